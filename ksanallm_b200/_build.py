@@ -77,12 +77,44 @@ def cuda_sources():
     return sorted((CSRC / "cuda").glob("*.cu"))
 
 
-def build_cuda(verbose: bool = False, ptxas_verbose: bool = False) -> Path:
+# Kernel sources of model families that can be served from a library of their own: enough to load one such model in a
+# fresh checkout without compiling every kernel of the package.
+FAMILY_SOURCES = {
+    "molopel": ("host_common", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2cta", "gemm_bf16_cluster_splitk",
+                "mixer_elementwise", "window_attention", "linear_attention"),
+}
+
+# Files compiled with IEEE division, square root and the accurate math functions: what they compute is specified in
+# 32-bit floats.
+EXACT_MATH = {"mixer_elementwise", "window_attention", "linear_attention"}
+
+
+def cuda_library(family: str = "") -> Path:
+    return LIB / (f"libksana_kernels_{family}.so" if family else "libksana_kernels.so")
+
+
+def _cuda_stale(srcs, out: Path) -> bool:
+    headers = sorted((CSRC / "cuda").glob("*.cuh")) + sorted((CSRC / "cuda").glob("*.h"))
+    return _newer([*srcs, *headers], out)
+
+
+def usable_library(family: str = "") -> Path:
+    """The library to load for a model of ``family``: the complete one when it is up to date, else (for a family that
+    has a list of its own) the family's, compiled first if needed."""
+    full = cuda_library()
+    if family not in FAMILY_SOURCES or (full.exists() and not _cuda_stale(cuda_sources(), full)):
+        return full if full.exists() else build_cuda()
+    return build_cuda(family=family)
+
+
+def build_cuda(verbose: bool = False, ptxas_verbose: bool = False, family: str = "") -> Path:
     LIB.mkdir(parents=True, exist_ok=True)
     OBJ.mkdir(parents=True, exist_ok=True)
-    out = LIB / "libksana_kernels.so"
+    out = cuda_library(family)
     headers = sorted((CSRC / "cuda").glob("*.cuh")) + sorted((CSRC / "cuda").glob("*.h"))
     srcs = cuda_sources()
+    if family:
+        srcs = [s for s in srcs if s.stem in FAMILY_SOURCES[family]]
     if not srcs:
         return out
     jobs = []
@@ -91,14 +123,15 @@ def build_cuda(verbose: bool = False, ptxas_verbose: bool = False) -> Path:
         o = OBJ / (s.stem + ".o")
         objs.append(o)
         if _newer([s, *headers], o):
-            cmd = [NVCC, *NVCC_FLAGS, "-I", CSRC / "cuda", "-c", s, "-o", o]
+            flags = [f for f in NVCC_FLAGS if f != "--use_fast_math" or s.stem not in EXACT_MATH]
+            cmd = [NVCC, *flags, "-I", CSRC / "cuda", "-c", s, "-o", o]
             if ptxas_verbose:
                 cmd += ["-Xptxas", "-v"]
             jobs.append(cmd)
     if jobs:
         with ThreadPoolExecutor(max_workers=min(8, len(jobs))) as ex:
             list(ex.map(lambda c: _run(c, verbose or ptxas_verbose), jobs))
-    if jobs or not out.exists():
+    if jobs or not out.exists() or _newer(objs, out):
         _run([NVCC, "-shared", "-o", out, *objs, "-lcudart"], verbose)
     return out
 

@@ -41,6 +41,49 @@ class QuantConfig:
 
 
 @dataclass
+class AttentionSpec:
+    """A softmax-attention mixer of one layer with sizes of its own."""
+    heads: int
+    kv_heads: int
+    dim: int
+    vdim: int
+    scale: float
+    window: int = 0          # keys a position sees, itself included (0: all earlier ones)
+    bias_max: float = 0.0    # learned distance bias: distance at which its log-spaced buckets end (0: no bias)
+    qkv_bias: bool = False
+    qk_norm: bool = False    # per-head RMS norm of q and k
+    out_scale: float = 1.0   # factor on the mixer's output
+
+
+@dataclass
+class LinearAttentionSpec:
+    """A linear-attention mixer with a fixed decay per head: S <- decay S + k v^T, o = S^T q."""
+    heads: int
+    dim: int
+    vdim: int
+    decay: List[float]
+    act: str = "none"        # activation on q, k and v after their projections: none | silu
+    rot_dims: int = 0        # leading dimensions of q and k that are rotated (half-split pairs)
+    rot_base: float = 10000.0
+    key_scale: float = 1.0   # factor on k after rotation
+    norm: str = "head"       # head: weightless RMS norm of each head | concat: one over all heads, with a weight
+    gate: str = "silu"       # output gate: silu | sigmoid of its own projection
+    out_scale: float = 1.0
+
+
+@dataclass
+class LayerSpec:
+    """One layer of a model whose layers differ: its mixers (side by side when there are both) and its feed-forward."""
+    attn: Optional[AttentionSpec] = None
+    linear: Optional[LinearAttentionSpec] = None
+    ff: int = 0              # feed-forward width (0: the layer has none)
+
+    @property
+    def state_shape(self):
+        return (self.linear.heads, self.linear.dim, self.linear.vdim) if self.linear else None
+
+
+@dataclass
 class ModelConfig:
     model_type: str = "llama"
     architectures: List[str] = field(default_factory=list)
@@ -118,6 +161,10 @@ class ModelConfig:
     reranker_start_layer: int = 0  # layer-wise reranker: depth of the first scoring head lm_head.0.linear_head
     num_register_token: int = 0  # parallel token prediction: register tokens appended per step (0 = off)
     reg_token_id: int = 0
+    # models described layer by layer (empty: every layer follows the fields above)
+    layers: List[LayerSpec] = field(default_factory=list)
+    logit_softcap: float = 0.0    # logits <- cap * tanh(logits / cap); 0 = off
+    residual_fp32: bool = False   # the residual stream is kept in 32-bit floats
     # quantisation
     quant: QuantConfig = field(default_factory=QuantConfig)
     raw: Dict[str, Any] = field(default_factory=dict)
@@ -132,6 +179,11 @@ class ModelConfig:
         if self.moe_layers:
             return layer_idx in self.moe_layers
         return layer_idx >= self.first_k_dense_replace and (layer_idx % max(self.moe_layer_freq, 1) == 0)
+
+    @property
+    def has_state(self) -> bool:
+        """Some layer carries a recurrent state from token to token."""
+        return any(l.linear is not None for l in self.layers)
 
     @property
     def q_head_dim(self) -> int:
@@ -185,7 +237,61 @@ def _quant(d: Optional[Dict[str, Any]]) -> QuantConfig:
     return q
 
 
+def _molopel_mixers(kind: str, c: Dict[str, Any]) -> LayerSpec:
+    if kind == "lightning":
+        return LayerSpec(linear=LinearAttentionSpec(
+            int(c["heads"]), int(c["dim"]), int(c["vdim"]), [float(x) for x in c["decay"]], act="silu",
+            norm="concat", gate="sigmoid"))
+    if kind == "parallel":
+        a, r = c["left"], c["right"]
+        return LayerSpec(
+            attn=AttentionSpec(int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), int(a["vdim"]), float(a["scale"]),
+                               window=int(a["mask"]["size"]), bias_max=float(a["bias_max"]), qkv_bias=True,
+                               qk_norm=True, out_scale=float(c["left_scale"])),
+            linear=LinearAttentionSpec(int(r["heads"]), int(r["dim"]), int(r["vdim"]), [float(x) for x in r["decay"]],
+                                       rot_dims=int(r["rot"]["dims"]), rot_base=float(r["rot"]["base"]),
+                                       key_scale=float(r["dim"]) ** -0.5, norm="head", gate="silu",
+                                       out_scale=float(c["right_scale"])))
+    raise ValueError(f"unknown Molopel layer type {kind!r}")
+
+
+def _molopel_config(c: Dict[str, Any]) -> ModelConfig:
+    """Molopel: layers of linear attention alone ("lightning") or of windowed attention beside retention
+    ("parallel"), each with sizes of its own; LayerNorm without bias, tied embeddings, soft-capped logits."""
+    m = ModelConfig(model_type="molopel", architectures=[str(c.get("architecture", "Molopel"))], raw=c)
+    m.vocab_size, m.hidden_size = int(c["vocab"]), int(c["width"])
+    for entry in c["layers"]:
+        spec = _molopel_mixers(str(entry["type"]), entry["mixer"])
+        mlp = entry.get("mlp")
+        if mlp is not None:
+            if str(mlp.get("kind", "dense")) != "dense":
+                raise ValueError(f"unknown Molopel feed-forward {mlp.get('kind')!r}")
+            spec.ff = int(mlp["ff"])
+        if spec.linear is not None and len(spec.linear.decay) != spec.linear.heads:
+            raise ValueError("one decay per head is needed")
+        m.layers.append(spec)
+    m.num_layers = len(m.layers)
+    attn = next((l.attn for l in m.layers if l.attn is not None), None)
+    if attn is not None:
+        m.num_heads, m.num_kv_heads, m.head_dim = attn.heads, attn.kv_heads, attn.dim
+    m.intermediate_size = max((l.ff for l in m.layers), default=0)
+    m.rms_norm_eps = float(c["norm"]["eps"])
+    m.norm_type, m.position_encoding, m.hidden_act = "layernorm", "none", "gelu_tanh"
+    m.tie_word_embeddings = True
+    m.emb_scale = float((c.get("embedding") or {}).get("scale", 1.0))
+    m.logit_softcap = float(c.get("logit_softcap") or 0.0)
+    m.residual_fp32 = True
+    m.max_position_embeddings = int(c.get("max_position_embeddings", 1 << 20))
+    m.torch_dtype = str(c.get("torch_dtype", "bfloat16"))
+    eos = c.get("eos_token_id")
+    m.eos_token_ids = [int(e) for e in eos] if isinstance(eos, (list, tuple)) else ([int(eos)] if eos is not None else [])
+    m.bos_token_id, m.pad_token_id = c.get("bos_token_id"), c.get("pad_token_id")
+    return m
+
+
 def model_config_from_dict(c: Dict[str, Any]) -> ModelConfig:
+    if str(c.get("architecture", "")).lower() == "molopel":
+        return _molopel_config(c)
     if isinstance(c.get("text_config"), dict) and str(c.get("model_type", "")).lower() in ("llama4",):
         # multimodal wrapper configs keep the language model under "text_config"
         inner = dict(c["text_config"])

@@ -1,0 +1,95 @@
+// Small helpers of the kernels behind layers with mixers of their own sizes: typed loads and stores that compute in
+// 32-bit floats whatever the storage type, and the accurate activations (these files are compiled without fast math).
+#pragma once
+#include "sm100.cuh"
+
+namespace ksana {
+
+template <typename T>
+__device__ __forceinline__ float to_f(T v);
+template <>
+__device__ __forceinline__ float to_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ float to_f<__nv_bfloat16>(__nv_bfloat16 v) { return __bfloat162float(v); }
+
+template <typename T>
+__device__ __forceinline__ T from_f(float v);
+template <>
+__device__ __forceinline__ float from_f<float>(float v) { return v; }
+template <>
+__device__ __forceinline__ __nv_bfloat16 from_f<__nv_bfloat16>(float v) { return __float2bfloat16_rn(v); }
+
+// N consecutive elements, N = 1, 4 or 8; for N > 1 the address is aligned to N elements.
+template <int N>
+__device__ __forceinline__ void load_n(const float* p, float* f) {
+  if constexpr (N == 1) {
+    f[0] = p[0];
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) {
+      float4 v = *reinterpret_cast<const float4*>(p + i);
+      f[i] = v.x; f[i + 1] = v.y; f[i + 2] = v.z; f[i + 3] = v.w;
+    }
+  }
+}
+template <int N>
+__device__ __forceinline__ void load_n(const __nv_bfloat16* p, float* f) {
+  if constexpr (N == 1) {
+    f[0] = __bfloat162float(p[0]);
+  } else if constexpr (N == 4) {
+    uint2 v = *reinterpret_cast<const uint2*>(p);
+    float2 a = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&v.x));
+    float2 b = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&v.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  } else {
+    uint4 v = *reinterpret_cast<const uint4*>(p);
+    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      uint32_t u = w[i];
+      float2 a = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&u));
+      f[2 * i] = a.x; f[2 * i + 1] = a.y;
+    }
+  }
+}
+template <int N>
+__device__ __forceinline__ void store_n(float* p, const float* f) {
+  if constexpr (N == 1) {
+    p[0] = f[0];
+  } else {
+#pragma unroll
+    for (int i = 0; i < N; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(f[i], f[i + 1], f[i + 2], f[i + 3]);
+  }
+}
+template <int N>
+__device__ __forceinline__ void store_n(__nv_bfloat16* p, const float* f) {
+  if constexpr (N == 1) {
+    p[0] = __float2bfloat16_rn(f[0]);
+  } else if constexpr (N == 4) {
+    *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]));
+  } else {
+    *reinterpret_cast<uint4*>(p) =
+        make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+  }
+}
+
+__device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
+__device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// 0.5 z (1 + tanh u) with u = sqrt(2 / pi) (z + 0.044715 z^3)
+__device__ __forceinline__ float gelu_tanh_f(float z) {
+  const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+  return z / (1.f + expf(-2.f * u));
+}
+
+// Sum over the block (a multiple of 32 threads, at most 1024); every thread gets it. `red` holds 32 floats.
+__device__ __forceinline__ float block_sum(float v, float* red) {
+  v = warp_sum(v);
+  __syncthreads();  // earlier readers of red are done
+  if ((threadIdx.x & 31) == 0) red[threadIdx.x >> 5] = v;
+  __syncthreads();
+  float t = 0.f;
+  for (unsigned i = 0; i < (blockDim.x >> 5); ++i) t += red[i];
+  return t;
+}
+
+}  // namespace ksana

@@ -61,6 +61,12 @@ PYBIND11_MODULE(_ksana_host, m) {
              if (!c.FlexibleReserve(seq, tokens, shared, min_len, &run)) return py::none();
              return py::make_tuple(run.dst_begin, run.src_slots, run.dst_slots, run.src_pos);
            })
+      .def("configure_states", &KVCacheManager::ConfigureStates, py::arg("num_device_slots"),
+           py::arg("num_host_slots") = 0)
+      .def_property_readonly("stateful", &KVCacheManager::stateful)
+      .def_property_readonly("num_state_slots", &KVCacheManager::num_state_slots)
+      .def_property_readonly("num_free_state_slots", &KVCacheManager::num_free_state_slots)
+      .def("state_slot", &KVCacheManager::StateSlot)
       .def("num_blocks", &KVCacheManager::NumBlocks)
       .def("free_seq", &KVCacheManager::FreeSeq)
       .def("truncate", &KVCacheManager::Truncate)
@@ -127,6 +133,9 @@ PYBIND11_MODULE(_ksana_host, m) {
       .def_property_readonly("swap_out", [](const StepPlan& p) { return PairsToArray(p.swap_out); })
       .def_property_readonly("swap_in", [](const StepPlan& p) { return PairsToArray(p.swap_in); })
       .def_property_readonly("block_copies", [](const StepPlan& p) { return PairsToArray(p.block_copies); })
+      .def_property_readonly("state_swap_out", [](const StepPlan& p) { return PairsToArray(p.state_swap_out); })
+      .def_property_readonly("state_swap_in", [](const StepPlan& p) { return PairsToArray(p.state_swap_in); })
+      .def_property_readonly("state_copies", [](const StepPlan& p) { return PairsToArray(p.state_copies); })
       .def_property_readonly("flexible",
                              [](const StepPlan& p) {
                                py::array_t<int32_t> a({static_cast<py::ssize_t>(p.flexible.size() / 4), py::ssize_t(4)});
@@ -212,6 +221,8 @@ PYBIND11_MODULE(_ksana_host, m) {
              return d;
            })
       .def("schedule", &Scheduler::Schedule, py::arg("now_ms") = 0)
+      .def("feed_given", &Scheduler::FeedGiven, py::arg("seq_id"), py::arg("tokens"))
+      .def("plan_given", &Scheduler::PlanGiven, py::arg("seq_ids"))
       .def("micro_batch_of", &Scheduler::MicroBatchOf)
       .def("set_hold_waiting", &Scheduler::SetHoldWaiting)
       .def("set_paused", &Scheduler::SetPaused)
@@ -239,6 +250,7 @@ PYBIND11_MODULE(_ksana_host, m) {
             d["q_starts"] = l.off_q_starts;
             d["logits_idx"] = l.off_logits_idx;
             d["block_tables"] = l.off_block_tables;
+            d["state_slots"] = l.off_state_slots;
             d["total_words"] = l.total_words;
             return d;
           },

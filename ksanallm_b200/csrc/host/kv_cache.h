@@ -81,6 +81,9 @@ struct SeqBlocks {
   std::vector<BlockId> own;         // private blocks after the shared ones
   std::vector<BlockId> host;        // host copies while swapped out (own blocks only)
   bool swapped = false;
+  // Recurrent-state slots (models with layers that carry a fixed-size state per sequence); -1: none.
+  int state = -1;
+  int host_state = -1;  // while swapped out
   bool no_commit = false;  // blocks never enter the prefix tree (token ids do not determine the KV: spliced embeddings)
   int NumBlocks() const { return static_cast<int>(shared.size() + own.size()); }
 };
@@ -110,6 +113,22 @@ class KVCacheManager {
     root_.key = 0x9E3779B97F4A7C15ull;
   }
   ~KVCacheManager() { FreeSubtree(&root_); }
+
+  // Models whose layers carry a recurrent state: every sequence then also holds one slot of a fixed pool. The state
+  // after a cached prefix is not kept, so prefix sharing is switched off. Called once, before any sequence exists.
+  void ConfigureStates(int num_device_slots, int num_host_slots) {
+    if (!seqs_.empty()) throw std::runtime_error("KVCacheManager: state slots configured after use");
+    states_ = BlockAllocator(num_device_slots);
+    host_states_ = BlockAllocator(num_host_slots);
+    stateful_ = num_device_slots > 0;
+    if (stateful_) prefix_ = false;
+  }
+  bool stateful() const { return stateful_; }
+  int num_state_slots() const { return states_.num_total(); }
+  int num_free_state_slots() const { return states_.num_free(); }
+  // Whether a new sequence would get what it needs besides blocks.
+  bool CanCreate() const { return !stateful_ || states_.num_free() > 0; }
+  int StateSlot(int64_t seq) const { return seqs_.at(seq).state; }
 
   int block_size() const { return block_size_; }
   bool prefix_enabled() const { return prefix_; }
@@ -143,7 +162,10 @@ class KVCacheManager {
   // Registers a sequence and pins its cached prefix. Returns number of prefix tokens reused.
   int CreateSeq(int64_t seq, const std::vector<int32_t>& tokens, bool use_prefix = true) {
     if (seqs_.count(seq)) throw std::runtime_error("KVCacheManager: duplicate seq");
+    int slot = -1;
+    if (stateful_ && !states_.Alloc(&slot)) throw std::runtime_error("KVCacheManager: no free state slot");
     SeqBlocks& sb = seqs_[seq];
+    sb.state = slot;
     sb.no_commit = !use_prefix;
     stats_.prefix_query_tokens += static_cast<int64_t>(tokens.size());
     if (!prefix_ || !use_prefix) return 0;
@@ -311,6 +333,8 @@ class KVCacheManager {
     for (auto* n : sb.shared) Unpin(n);
     for (auto b : sb.own) dev_.Release(b);
     for (auto b : sb.host) host_.Release(b);
+    if (sb.state >= 0) states_.Release(sb.state);
+    if (sb.host_state >= 0) host_states_.Release(sb.host_state);
     seqs_.erase(it);
   }
 
@@ -332,12 +356,18 @@ class KVCacheManager {
 
   // Copy-on-write fork: the child shares the parent's tree blocks and gets private copies of the
   // parent's private blocks. Returns false (nothing changed) when there are not enough blocks.
-  bool Fork(int64_t parent, int64_t child, std::vector<CopyPair>* copies) {
+  bool Fork(int64_t parent, int64_t child, std::vector<CopyPair>* copies,
+            std::vector<CopyPair>* state_copies = nullptr) {
     if (seqs_.count(child)) throw std::runtime_error("KVCacheManager: duplicate seq in fork");
     const SeqBlocks& p = seqs_.at(parent);
     if (p.swapped) return false;
     if (static_cast<int>(p.own.size()) > num_available_blocks()) return false;
+    if (stateful_ && (state_copies == nullptr || states_.num_free() == 0)) return false;
     SeqBlocks c;
+    if (stateful_) {
+      states_.Alloc(&c.state);
+      state_copies->push_back({p.state, c.state});
+    }
     c.no_commit = p.no_commit;
     for (auto* n : p.shared) {
       Pin(n);
@@ -358,10 +388,16 @@ class KVCacheManager {
 
   // Swap-out: private blocks go to host blocks; tree blocks stay pinned on the device (other
   // requests may share them). Returns false when the host tier is full.
-  bool SwapOut(int64_t seq, std::vector<CopyPair>* copies) {
+  bool SwapOut(int64_t seq, std::vector<CopyPair>* copies, std::vector<CopyPair>* state_copies = nullptr) {
     SeqBlocks& sb = seqs_.at(seq);
     if (sb.swapped) return true;
     if (static_cast<int>(sb.own.size()) > host_.num_free()) return false;
+    if (stateful_) {
+      if (state_copies == nullptr || !host_states_.Alloc(&sb.host_state)) return false;
+      state_copies->push_back({sb.state, sb.host_state});
+      states_.Release(sb.state);
+      sb.state = -1;
+    }
     for (auto b : sb.own) {
       BlockId h;
       host_.Alloc(&h);
@@ -377,10 +413,16 @@ class KVCacheManager {
 
   // Swap-in: needs the tree part to still be resident (pinned nodes never leave), then host
   // blocks come back into fresh device blocks. Returns false when memory is short.
-  bool SwapIn(int64_t seq, std::vector<CopyPair>* copies) {
+  bool SwapIn(int64_t seq, std::vector<CopyPair>* copies, std::vector<CopyPair>* state_copies = nullptr) {
     SeqBlocks& sb = seqs_.at(seq);
     if (!sb.swapped) return true;
     if (static_cast<int>(sb.host.size()) > num_available_blocks()) return false;
+    if (stateful_) {
+      if (state_copies == nullptr || !states_.Alloc(&sb.state)) return false;
+      state_copies->push_back({sb.host_state, sb.state});
+      host_states_.Release(sb.host_state);
+      sb.host_state = -1;
+    }
     for (auto h : sb.host) {
       BlockId b;
       if (!dev_.Alloc(&b)) {
@@ -486,6 +528,9 @@ class KVCacheManager {
 
   BlockAllocator dev_;
   BlockAllocator host_;
+  BlockAllocator states_{0};       // recurrent-state slots on the device
+  BlockAllocator host_states_{0};  // ... and of swapped-out sequences
+  bool stateful_ = false;
   int block_size_;
   bool prefix_;
   PrefixNode root_;

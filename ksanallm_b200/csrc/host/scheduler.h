@@ -130,6 +130,8 @@ struct StepPlan {
   std::vector<CopyPair> swap_out;       // device -> host
   std::vector<CopyPair> swap_in;        // host -> device
   std::vector<CopyPair> block_copies;   // device -> device (fork copy-on-write)
+  // the same three moves for recurrent-state slots
+  std::vector<CopyPair> state_swap_out, state_swap_in, state_copies;
   // flexible cache reuse, one row per token: (source slot, destination slot, source position, destination position);
   // executed before every other block operation of the step
   std::vector<int32_t> flexible;
@@ -166,7 +168,7 @@ struct SchedStats {
 struct PackedLayout {
   int32_t num_seqs, num_prefill, num_decode, total_tokens, total_logits, max_q_len, max_kv_len, max_blocks;
   int32_t off_input_ids, off_positions, off_slot_mapping, off_cu_q, off_kv_lens, off_q_starts;
-  int32_t off_logits_idx, off_block_tables, off_seq_of_token, total_words;
+  int32_t off_logits_idx, off_block_tables, off_seq_of_token, off_state_slots, total_words;
 };
 
 class Scheduler {
@@ -226,7 +228,7 @@ class Scheduler {
     if (it == seqs_.end() || seqs_.count(child)) return false;
     Sequence& p = *it->second;
     if (p.state != SEQ_RUNNING) return false;
-    if (!cache_->Fork(parent, child, &pending_copies_)) return false;
+    if (!cache_->Fork(parent, child, &pending_copies_, &pending_state_copies_)) return false;
     auto c = std::make_unique<Sequence>(p);
     c->id = child;
     c->drafts.clear();
@@ -366,6 +368,7 @@ class Scheduler {
     StepPlan plan;
     ++stats_.steps;
     plan.block_copies.swap(pending_copies_);
+    plan.state_copies.swap(pending_state_copies_);
     DropAbortedAndTimedOut(now_ms, &plan);
     BalanceMicroBatches();
 
@@ -463,7 +466,7 @@ class Scheduler {
       if (cache_->NumHostBlocks(id) + std::max(extra, 0) + headroom > cache_->num_available_blocks() &&
           !running_.empty())
         break;
-      if (!cache_->SwapIn(id, &plan.swap_in)) break;
+      if (!cache_->SwapIn(id, &plan.swap_in, &plan.state_swap_in)) break;
       if (!cache_->EnsureCapacity(id, s.num_computed + need_now + cfg_.lookahead_slots)) {
         // Could not grow after coming back: stay resident, run next step.
         swapped_.pop_front();
@@ -512,6 +515,7 @@ class Scheduler {
       int64_t id = waiting_.front();
       Sequence& s = *seqs_.at(id);
       size_t flex_mark = plan.flexible.size();
+      if (!cache_->Has(id) && !cache_->CanCreate()) break;  // no recurrent-state slot: wait for one to be released
       if (!cache_->Has(id)) {
         int hit = s.no_cache ? 0 : cache_->MatchPrefix(s.tokens);
         int remaining = static_cast<int>(s.tokens.size()) - hit;
@@ -576,6 +580,53 @@ class Scheduler {
       --batch_budget;
     }
 
+    FillPlan(&plan, std::move(prefill), std::move(decode));
+    return plan;
+  }
+
+  // ---- given tokens ---------------------------------------------------------------------------------------
+  // Replay of recorded token ids: the caller says which sequences run and how many of which tokens, instead of the
+  // queues and the sampler. Such a sequence holds blocks (and a state slot) like any other, is planned with
+  // PlanGiven, advances through Update() (its entries ask for no logits) and is ended with Finish().
+  bool FeedGiven(int64_t id, const std::vector<int32_t>& tokens) {
+    auto it = seqs_.find(id);
+    if (it == seqs_.end()) {
+      if (tokens.empty() || !cache_->CanCreate()) return false;
+      auto s = std::make_unique<Sequence>();
+      s->id = id;
+      s->tokens = tokens;
+      s->prompt_len = static_cast<int>(tokens.size());
+      s->no_cache = true;  // every token is computed in the step that brings it
+      s->state = SEQ_RUNNING;
+      cache_->CreateSeq(id, s->tokens, false);
+      seqs_[id] = std::move(s);
+      return true;
+    }
+    it->second->tokens.insert(it->second->tokens.end(), tokens.begin(), tokens.end());
+    return true;
+  }
+
+  // One step over the not yet computed tokens of `ids`. Throws when the cache cannot hold them.
+  StepPlan PlanGiven(const std::vector<int64_t>& ids) {
+    StepPlan plan;
+    ++stats_.steps;
+    std::vector<StepEntry> prefill, decode;
+    for (int64_t id : ids) {
+      Sequence& s = *seqs_.at(id);
+      int q_len = static_cast<int>(s.tokens.size()) - s.num_computed;
+      if (q_len <= 0) continue;
+      if (!cache_->EnsureCapacity(id, s.num_computed + q_len))
+        throw std::runtime_error("Scheduler: the cache pool is too small for the given tokens");
+      bool as_decode = s.num_computed > 0 && q_len <= cfg_.decode_token_threshold;
+      (as_decode ? decode : prefill).push_back({id, s.num_computed, q_len, 0, 0, as_decode});
+    }
+    FillPlan(&plan, std::move(prefill), std::move(decode));
+    return plan;
+  }
+
+ private:
+  void FillPlan(StepPlan* out, std::vector<StepEntry> prefill, std::vector<StepEntry> decode) {
+    StepPlan& plan = *out;
     // Order: prefill by new-token count (desc), then decode by q_len (desc) — equal-q_len decode
     // entries are contiguous so one kernel launch covers each group.
     std::stable_sort(prefill.begin(), prefill.end(),
@@ -597,8 +648,9 @@ class Scheduler {
       plan.max_kv_len = std::max(plan.max_kv_len, e.q_start + e.q_len);
       stats_.draft_proposed += e.n_drafts;
     }
-    return plan;
   }
+
+ public:
 
   // Words needed by Pack() for this plan.
   int64_t PackedWords(const StepPlan& plan, int max_blocks) const {
@@ -626,6 +678,7 @@ class Scheduler {
     int32_t* lg = buf + l.off_logits_idx;
     int32_t* bt = buf + l.off_block_tables;
     int32_t* sot = buf + l.off_seq_of_token;
+    int32_t* sst = buf + l.off_state_slots;
     int t = 0, li = 0, b = 0;
     cu[0] = 0;
     const int bs = cfg_.block_size;
@@ -647,6 +700,7 @@ class Scheduler {
       cu[b + 1] = t;
       kvl[b] = e.q_start + e.q_len;
       qs[b] = e.q_start;
+      sst[b] = cache_->StateSlot(e.seq_id);
       ++b;
     }
     return l;
@@ -779,6 +833,8 @@ class Scheduler {
     off = align(off + B);
     l->off_logits_idx = static_cast<int32_t>(off);
     off = align(off + plan.total_logits);
+    l->off_state_slots = static_cast<int32_t>(off);
+    off = align(off + B);
     l->off_block_tables = static_cast<int32_t>(off);
     off = align(off + static_cast<int64_t>(B) * max_blocks);
     l->total_words = static_cast<int32_t>(off);
@@ -828,7 +884,7 @@ class Scheduler {
     ++s.preempt_count;
     s.drafts.clear();
     bool mid_prefill = static_cast<int>(s.tokens.size()) - s.num_computed > 1;
-    if (cfg_.preempt_mode == 0 && !mid_prefill && cache_->SwapOut(id, &plan->swap_out)) {
+    if (cfg_.preempt_mode == 0 && !mid_prefill && cache_->SwapOut(id, &plan->swap_out, &plan->state_swap_out)) {
       s.state = SEQ_SWAPPED;
       swapped_.push_back(id);
       ++stats_.preempt_swap;
@@ -873,7 +929,7 @@ class Scheduler {
   std::unordered_map<int64_t, std::unique_ptr<Sequence>> seqs_;
   std::deque<int64_t> waiting_, running_, swapped_;
   std::unordered_set<int64_t> aborted_;
-  std::vector<CopyPair> pending_copies_;
+  std::vector<CopyPair> pending_copies_, pending_state_copies_;
   int mb_filter_ = -1, mb_count_ = 1;
   bool hold_waiting_ = false;
   bool preempted_this_step_ = false;

@@ -102,7 +102,7 @@ class LLMEngine:
     def __init__(self, model: TransformerModel, serving: ServingConfig, tp: Optional[TPGroup] = None,
                  num_blocks: Optional[int] = None, num_host_blocks: Optional[int] = None,
                  detokenize: Optional[Callable[[List[int]], str]] = None, seed: int = 0,
-                 kv_dtype: Optional[torch.dtype] = None, block_sync_group=None):
+                 kv_dtype: Optional[torch.dtype] = None, block_sync_group=None, num_state_slots: Optional[int] = None):
         self.model = model
         self._block_sync_group = block_sync_group  # pipeline stages: world group for the block-count agreement
         self.cfg: ModelConfig = model.cfg
@@ -111,6 +111,10 @@ class LLMEngine:
         self.detokenize = detokenize
         bs_cfg, bm_cfg = serving.setting.batch_scheduler, serving.setting.block_manager
         self.block_size = 64 if self.cfg.use_mla and bm_cfg.block_token_num == 16 else bm_cfg.block_token_num
+        # every running sequence of a model with recurrent layers holds a state slot
+        self.num_state_slots = (num_state_slots or bs_cfg.max_batch_size) if self.cfg.has_state else 0
+        if self.cfg.has_state:
+            self._check_recurrent(model)
         if num_blocks is None:
             num_blocks = self._derive_num_blocks(kv_dtype)
         if num_host_blocks is None:
@@ -118,15 +122,19 @@ class LLMEngine:
             num_host_blocks = min(num_host_blocks, self._host_block_cap(kv_dtype))
         self.num_blocks = num_blocks
         max_blocks_per_seq = (bs_cfg.max_token_len + self.block_size - 1) // self.block_size + 1
+        num_host_states = self.num_state_slots if num_host_blocks > 0 else 0
         self.runner = ModelRunner(model, num_blocks, self.block_size, num_host_blocks, bs_cfg.max_step_tokens,
-                                  bs_cfg.max_batch_size, max_blocks_per_seq, kv_dtype, seed)
+                                  bs_cfg.max_batch_size, max_blocks_per_seq, kv_dtype, seed, self.num_state_slots,
+                                  num_host_states)
         self.runner.sampler.eos_token_ids = list(model.cfg.eos_token_ids)
         self.is_driver = self.tp.rank == 0  # with pipeline stages: re-set by attach_pipeline (global rank 0 drives)
         # drafts per step from the first next-n module (applied repeatedly for more than one; tensor-parallel peers
         # receive each further pass's rows from the driver)
         self.mtp_steps = bs_cfg.mtp_step_num if (bs_cfg.enable_speculative_decoding or bs_cfg.mtp_step_num) \
             and model.mtp_layers else 0
-        self.trie_drafts = 3 if (bs_cfg.enable_speculative_decoding and not model.mtp_layers) else 0
+        # (a recurrent state cannot step back over rejected drafts)
+        self.trie_drafts = 3 if (bs_cfg.enable_speculative_decoding and not model.mtp_layers
+                                 and not self.cfg.has_state) else 0
         sc = _host.SchedulerConfig()
         sc.block_size = self.block_size
         sc.max_batch_size = bs_cfg.max_batch_size
@@ -152,6 +160,8 @@ class LLMEngine:
         sc.decode_token_threshold = 1 + sc.max_draft_tokens
         self.cache = _host.KVCacheManager(num_blocks, num_host_blocks, self.block_size,
                                           bool(bs_cfg.enable_auto_prefix_cache))
+        if self.num_state_slots:
+            self.cache.configure_states(self.num_state_slots, num_host_states)
         self.sched = _host.Scheduler(sc, self.cache)
         self.sched_cfg = sc
         self._ids = itertools.count(1)
@@ -204,6 +214,18 @@ class LLMEngine:
         self._dp_arrivals = 0
         self.dp_any_work = True
 
+    def _check_recurrent(self, model) -> None:
+        """What a model with recurrent layers cannot be combined with: all of it splits or re-uses a sequence at
+        places where its state is not kept."""
+        g, cn = self.serving.setting.global_, self.serving.setting.connector
+        if self.tp.size > 1 or self._block_sync_group is not None or g.pipeline_para_size > 1 or \
+                g.attn_data_para_size > 1:
+            raise NotImplementedError("models with recurrent layers run on one GPU")
+        if cn.group_role in ("prefill", "decode", "both"):
+            raise NotImplementedError("models with recurrent layers do not hand requests over between instances")
+        if getattr(model.cfg, "num_register_token", 0):
+            raise NotImplementedError("models with recurrent layers do not take register tokens")
+
     @staticmethod
     def _flexible_cache_min(bs_cfg, model, kv_dtype) -> int:
         """setting.batch_scheduler.min_flexible_cache_num when the model's cached keys can be moved to another
@@ -211,7 +233,7 @@ class LLMEngine:
         0 (off) otherwise."""
         want = int(getattr(bs_cfg, "min_flexible_cache_num", 0) or 0)
         cfg = model.cfg
-        if want <= 0 or not bs_cfg.enable_auto_prefix_cache:
+        if want <= 0 or not bs_cfg.enable_auto_prefix_cache or cfg.layers:
             return 0
         movable = (cfg.position_encoding in ("rope", "alibi") and not cfg.qk_norm_after_rope and not cfg.qk_l2_norm
                    and not cfg.rope_layers and not cfg.rope_scaling.mrope_section and not cfg.index_topk
@@ -221,10 +243,11 @@ class LLMEngine:
     # ---- sizing ----------------------------------------------------------------------------------------
     def _derive_num_blocks(self, kv_dtype) -> int:
         bm = self.serving.setting.block_manager
-        per_block = self.model.kv_block_bytes(self.block_size, kv_dtype)
+        per_block = max(self.model.kv_block_bytes(self.block_size, kv_dtype), 1)
         if self.model.device.type == "cuda":
             free, total = torch.cuda.mem_get_info(self.model.device)
             budget = free - int(total * bm.reserved_device_memory_ratio) - (8 << 30)
+            budget -= self.num_state_slots * self.model.state_slot_bytes()
             if bm.block_device_memory_ratio > 0:
                 budget = min(budget, int(total * bm.block_device_memory_ratio))
             n = max(int(budget // per_block), 16)
@@ -440,6 +463,8 @@ class LLMEngine:
         with self._phase("PrepareForwarding", nb, nt):
             self.runner.apply_flexible(plan.flexible)
             self.runner.apply_block_ops(plan.swap_out, plan.swap_in, plan.block_copies)
+            if self.num_state_slots:
+                self.runner.apply_state_ops(plan.state_copies, plan.state_swap_out, plan.state_swap_in)
             meta = self.runner.upload(layout)
             if mrope is not None:
                 meta.mrope_positions = mrope.to(self.runner.device)
@@ -481,6 +506,35 @@ class LLMEngine:
                           "schedule_s": t1 - t0, "forward_s": t2 - t1, "prefill": meta.num_prefill,
                           "decode": meta.num_decode})
         return n_new
+
+    # ---- replay of given tokens ------------------------------------------------------------------------------------
+    def replay(self, entries: Sequence[Tuple[int, Sequence[int], Sequence[int]]], end: Sequence[int] = ()) -> torch.Tensor:
+        """One step over given token ids instead of scheduled requests: ``entries`` = (sequence id, its next tokens,
+        the places among them whose logits are wanted). The step is planned, packed, run and committed by the same
+        scheduler, cache manager and runner that generation uses; nothing is sampled. A sequence is admitted at its
+        first entry and released after the step that names it in ``end``. Returns the wanted logits (fp32, in the
+        order of the entries and of their places)."""
+        with self.lock:
+            for sid, tokens, _ in entries:
+                if not self.sched.feed_given(sid, [int(t) for t in tokens]):
+                    raise EngineError(_host.RET_EXCEED_CAPACITY, "no room for another sequence")
+            plan = self.sched.plan_given([sid for sid, _, _ in entries])
+            out = torch.empty(0, self.cfg.vocab_size, dtype=torch.float32)
+            if not plan.empty():
+                layout = self.sched.pack(plan, self.runner.staging.host_np, self.runner.max_blocks_per_seq)
+                meta = self.runner.upload(layout)
+                hidden = self.runner.forward(meta)
+                first = {e.seq_id: int(r) for e, r in zip(plan.entries, meta.cu_q_host)}
+                rows = [first[sid] + int(p) for sid, _, want in entries for p in want]
+                if rows:
+                    out = self.runner.logits(hidden, meta, rows).to("cpu")
+                self.sched.update(plan, [], int(time.time() * 1000))
+                self.runner.check_device_status()
+                self.step_count += 1
+            for sid in end:
+                self.sched.finish(sid, _host.FINISH_LENGTH)
+                self.sched.forget(sid)
+        return out
 
     # ---- asynchronous scheduling ---------------------------------------------------------------------------------
     @staticmethod
@@ -532,6 +586,8 @@ class LLMEngine:
         with self._phase("LaunchStep", nb, nt):
             self.runner.apply_flexible(plan.flexible)
             self.runner.apply_block_ops(plan.swap_out, plan.swap_in, plan.block_copies)
+            if self.num_state_slots:
+                self.runner.apply_state_ops(plan.state_copies, plan.state_swap_out, plan.state_swap_in)
             meta = self.runner.upload(layout)
             if fix:
                 self.runner.fixup_inputs(meta)
@@ -986,7 +1042,7 @@ class LLMEngine:
                         mrope=None, noplan: bool = False) -> None:
         keys = ["num_seqs", "num_prefill", "num_decode", "total_tokens", "total_logits", "max_q_len", "max_kv_len",
                 "max_blocks", "input_ids", "positions", "slot_mapping", "seq_of_token", "cu_q", "kv_lens", "q_starts",
-                "logits_idx", "block_tables", "total_words"]
+                "logits_idx", "block_tables", "total_words", "state_slots"]
         h = self._hdr
         h[:] = 0
         h[0] = 2 if stop else (3 if noplan else 1)
@@ -1023,7 +1079,7 @@ class LLMEngine:
         """Step loop of a non-driver rank: receive plan, run the shard, join the collectives."""
         keys = ["num_seqs", "num_prefill", "num_decode", "total_tokens", "total_logits", "max_q_len", "max_kv_len",
                 "max_blocks", "input_ids", "positions", "slot_mapping", "seq_of_token", "cu_q", "kv_lens", "q_starts",
-                "logits_idx", "block_tables", "total_words"]
+                "logits_idx", "block_tables", "total_words", "state_slots"]
         hdr = torch.zeros(64, dtype=torch.int32)
         while True:
             dist.broadcast(hdr, src=self._ctl_src, group=self._ctl)

@@ -21,7 +21,8 @@ from .step_input import StepInput, StepStaging
 class ModelRunner:
     def __init__(self, model: TransformerModel, num_blocks: int, block_size: int, num_host_blocks: int = 0,
                  max_step_tokens: int = 4096, max_batch_size: int = 128, max_blocks_per_seq: int = 128,
-                 kv_dtype: Optional[torch.dtype] = None, seed: int = 0):
+                 kv_dtype: Optional[torch.dtype] = None, seed: int = 0, num_state_slots: int = 0,
+                 num_host_state_slots: int = 0):
         self.model = model
         self.device = model.device
         self.block_size = block_size
@@ -32,6 +33,13 @@ class ModelRunner:
             pin = self.device.type == "cuda"
             self.host_caches = [torch.empty((num_host_blocks,) + tuple(c.shape[1:]), dtype=c.dtype, pin_memory=pin)
                                 for c in self.kv_caches]
+        # recurrent-state pools, one slot per live sequence (None: the model has no such layers)
+        self.states = model.allocate_state(num_state_slots) if num_state_slots else None
+        self.host_states = None
+        if self.states is not None and num_host_state_slots > 0:
+            self.host_states = [torch.empty((num_host_state_slots,) + tuple(s.shape[1:]), dtype=s.dtype,
+                                            pin_memory=self.device.type == "cuda") for s in self.states]
+        model.reserve_positions(max_blocks_per_seq * block_size)
         self.max_blocks_per_seq = max_blocks_per_seq
         words = 8 * (max_step_tokens + 64) + 8 * (max_batch_size + 64) + max_batch_size * (max_blocks_per_seq + 32) + 4096
         self.staging = StepStaging(words, self.device)
@@ -73,13 +81,36 @@ class ModelRunner:
             for dev in self.kv_caches:
                 dev[dst] = dev[src]
 
+    def apply_state_ops(self, copies: np.ndarray, swap_out: np.ndarray, swap_in: np.ndarray) -> None:
+        """The moves of recurrent-state slots, on the compute stream ahead of the forward. Forks come first: they were
+        asked for before this step was planned, and a slot they read may be released and refilled by it."""
+        if self.states is None:
+            return
+        if len(copies):
+            # a later fork of the same batch may read what an earlier one wrote: follow every source to its origin,
+            # then gather before scattering
+            origin: Dict[int, int] = {}
+            for s, d in copies[:, :2].tolist():
+                origin[d] = origin.get(s, s)
+            dst = torch.tensor(list(origin.keys()), device=self.device)
+            src = torch.tensor(list(origin.values()), device=self.device)
+            for pool in self.states:
+                if pool.numel():
+                    pool[dst] = pool.index_select(0, src)
+        for pairs, back in ((swap_out, False), (swap_in, True)):
+            for s, d in (pairs[:, :2].tolist() if len(pairs) else ()):
+                for dev, host in zip(self.states, self.host_states):
+                    if dev.numel():
+                        (dev[d] if back else host[d]).copy_(host[s] if back else dev[s], non_blocking=True)
+
     def _mover_ok(self) -> bool:
         """Prepares (once) the per-layer base-address tables of the device cache and the pinned host pool."""
         ok = getattr(self, "_mover", None)
         if ok is None:
             c0 = self.kv_caches[0]
             self._block_bytes = c0[0].numel() * c0.element_size()
-            ok = self._block_bytes % 16 == 0 and all(c.is_contiguous() for c in self.kv_caches)
+            ok = self._block_bytes % 16 == 0 and self._block_bytes > 0 and \
+                all(c.is_contiguous() and c[0].numel() == c0[0].numel() for c in self.kv_caches)
             if ok:
                 self._dev_ptrs = torch.tensor([c.data_ptr() for c in self.kv_caches], dtype=torch.int64,
                                               device=self.device)
@@ -149,7 +180,10 @@ class ModelRunner:
 
     @torch.inference_mode()
     def forward(self, meta: StepInput, refit=None) -> torch.Tensor:
-        hidden = self.model.forward(meta, self.kv_caches, refit)
+        if self.states is not None:
+            hidden = self.model.forward(meta, self.kv_caches, refit, states=self.states)
+        else:
+            hidden = self.model.forward(meta, self.kv_caches, refit)
         self.last_hidden = hidden
         return hidden
 
@@ -243,5 +277,7 @@ class ModelRunner:
         return host.tolist()
 
     @torch.inference_mode()
-    def logits(self, hidden: torch.Tensor, meta: StepInput) -> torch.Tensor:
-        return self.model.compute_logits(hidden, meta.logits_idx)
+    def logits(self, hidden: torch.Tensor, meta: StepInput, rows: Optional[Sequence[int]] = None) -> torch.Tensor:
+        """fp32 logits of the step's own logits rows, or of the given rows of the hidden states."""
+        idx = meta.logits_idx if rows is None else torch.tensor(rows, dtype=torch.int32, device=self.device)
+        return self.model.compute_logits(hidden, idx)

@@ -35,6 +35,7 @@ class StepInput:
     max_kv_len: int
     max_blocks: int
     h2d_bytes: int = 0
+    state_slots: Optional[torch.Tensor] = None  # [B] int32, recurrent-state slot of each sequence (-1: none)
     # host copies of the small per-sequence arrays (kernel launch decisions never sync the device)
     cu_q_host: Optional[np.ndarray] = None
     kv_lens_host: Optional[np.ndarray] = None
@@ -96,13 +97,14 @@ class StepStaging:
             num_seqs=B, num_prefill=layout["num_prefill"], num_decode=layout["num_decode"], total_tokens=T,
             total_logits=L, max_q_len=layout["max_q_len"], max_kv_len=layout["max_kv_len"], max_blocks=mb,
             h2d_bytes=n * 4,
+            state_slots=sl("state_slots", B) if "state_slots" in layout else None,
             cu_q_host=hn[layout["cu_q"]:layout["cu_q"] + B + 1].copy(),
             kv_lens_host=hn[layout["kv_lens"]:layout["kv_lens"] + B].copy(),
         )
 
 
 def make_step_input(input_ids, positions, slot_mapping, cu_q, kv_lens, block_tables, logits_idx=None,
-                    num_prefill=None, device="cpu") -> StepInput:
+                    num_prefill=None, device="cpu", state_slots=None) -> StepInput:
     """Builds a StepInput from plain lists/tensors (tests, offline forward, warm-up)."""
     dev = torch.device(device)
 
@@ -125,5 +127,6 @@ def make_step_input(input_ids, positions, slot_mapping, cu_q, kv_lens, block_tab
         cu_q=cu.to(dev), kv_lens=kl.to(dev), q_starts=(kl - qlens).to(dev), logits_idx=t(logits_idx),
         block_tables=bt.to(dev).contiguous(), num_seqs=B, num_prefill=num_prefill, num_decode=B - num_prefill,
         total_tokens=T, total_logits=int(torch.as_tensor(logits_idx).numel()), max_q_len=int(qlens.max()) if B else 0,
+        state_slots=None if state_slots is None else t(state_slots),
         max_kv_len=int(kl.max()) if B else 0, max_blocks=bt.shape[1] if bt.dim() == 2 else 0,
         cu_q_host=cu.numpy().copy(), kv_lens_host=kl.numpy().copy())

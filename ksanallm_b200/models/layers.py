@@ -315,7 +315,7 @@ class DenseFFN:
         if self.gated:
             if self.act in ("silu", "swish"):
                 return ops.silu_and_mul(u)
-            return ref.gelu_and_mul(u)
+            return ops.gelu_and_mul(u)
         return ops.activation(u, self.act)
 
 

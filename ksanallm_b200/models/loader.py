@@ -22,7 +22,7 @@ from typing import Dict, Iterable, Iterator, List, Optional, Tuple
 
 import torch
 
-from ..config.model_config import ModelConfig
+from ..config.model_config import LayerSpec, ModelConfig
 from ..ops import reference as ref
 
 # Block-scaled e4m3 linear weights are kept with power-of-two scales (KSANA_FP8_POW2_SCALES=0: the checkpoint's own
@@ -47,6 +47,11 @@ _RENAMES: Dict[str, List[Tuple[str, str]]] = {
                   (r"\.feed_forward\.w1\.", ".mlp.gate_proj."), (r"\.feed_forward\.w3\.", ".mlp.up_proj."),
                   (r"\.feed_forward\.w2\.", ".mlp.down_proj."), (r"\.attention_norm\.", ".input_layernorm."),
                   (r"\.ffn_norm\.", ".post_attention_layernorm.")],
+    "molopel": [(r"^embed$", "model.embed_tokens.weight"), (r"^final\.norm$", "model.norm.weight"),
+                (r"^l(\d+)\.norm1$", r"model.layers.\1.input_layernorm.weight"),
+                (r"^l(\d+)\.norm2$", r"model.layers.\1.post_attention_layernorm.weight"),
+                (r"^l(\d+)\.mix\.", r"model.layers.\1.mixer."),
+                (r"^l(\d+)\.mlp\.(gate|up|down)$", r"model.layers.\1.mlp.\2_proj.weight")],
     "baichuan": [(r"\.W_pack\.", ".wpack.")],
     "chatglm": [(r"^transformer\.embedding\.word_embeddings\.", "model.embed_tokens."),
                 (r"^transformer\.encoder\.layers\.", "model.layers."),
@@ -140,6 +145,9 @@ def synthetic_checkpoint(cfg: ModelConfig, seed: int = 0, std: float = 0.02, dev
     n_total = cfg.num_layers + cfg.num_nextn_predict_layers
     for i in range(n_total):
         p = f"model.layers.{i}"
+        if cfg.layers:
+            yield from _synthetic_mixer_layer(cfg.layers[i], p, H, rnd, ones)
+            continue
         yield p + ".input_layernorm.weight", ones(H)
         yield p + ".post_attention_layernorm.weight", ones(H)
         a = p + ".self_attn"
@@ -371,6 +379,62 @@ def _kv_rows(t: torch.Tensor, rank: int, size: int, num_kv_heads: int, d: int) -
     return t[hidx * d:(hidx + 1) * d]
 
 
+def mixer_prefixes(spec: LayerSpec) -> Tuple[Optional[str], Optional[str]]:
+    """Checkpoint prefixes of a layer's attention and linear-attention tensors (None: the layer has no such mixer)."""
+    both = spec.attn is not None and spec.linear is not None
+    return (("left." if both else "") if spec.attn is not None else None,
+            ("right." if both else "") if spec.linear is not None else None)
+
+
+def mixer_parts(spec: LayerSpec) -> set:
+    """Names of all tensors of a layer's mixers, below the layer's mixer prefix."""
+    pa, pl = mixer_prefixes(spec)
+    need = set()
+    if spec.attn is not None:
+        need |= {pa + x for x in "qkvo"}
+        if spec.attn.qkv_bias:
+            need |= {f"{pa}{x}.b" for x in "qkv"}
+        if spec.attn.qk_norm:
+            need |= {pa + "q.norm", pa + "k.norm"}
+        if spec.attn.bias_max:
+            need.add(pa + "rel")
+    if spec.linear is not None:
+        need |= {pl + x for x in "qkvgo"}
+        if spec.linear.norm == "concat":
+            need.add(pl + "norm")
+    return need
+
+
+def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterator[Tuple[str, torch.Tensor]]:
+    yield p + ".input_layernorm.weight", ones(H)
+    pa, pl = mixer_prefixes(spec)
+    m = p + ".mixer."
+    if spec.attn is not None:
+        a = spec.attn
+        for x, n in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)):
+            yield m + pa + x, rnd(n, H)
+            if a.qkv_bias:
+                yield f"{m}{pa}{x}.b", rnd(n)
+        if a.qk_norm:
+            yield m + pa + "q.norm", ones(a.dim)
+            yield m + pa + "k.norm", ones(a.dim)
+        if a.bias_max:
+            yield m + pa + "rel", rnd(32, a.heads)
+        yield m + pa + "o", rnd(H, a.heads * a.vdim)
+    if spec.linear is not None:
+        r = spec.linear
+        for x, n in (("q", r.dim), ("k", r.dim), ("v", r.vdim), ("g", r.vdim)):
+            yield m + pl + x, rnd(r.heads * n, H)
+        if r.norm == "concat":
+            yield m + pl + "norm", ones(r.heads * r.vdim)
+        yield m + pl + "o", rnd(H, r.heads * r.vdim)
+    if spec.ff:
+        yield p + ".post_attention_layernorm.weight", ones(H)
+        yield p + ".mlp.gate_proj.weight", rnd(spec.ff, H)
+        yield p + ".mlp.up_proj.weight", rnd(spec.ff, H)
+        yield p + ".mlp.down_proj.weight", rnd(H, spec.ff)
+
+
 class WeightLoader:
     def __init__(self, cfg: ModelConfig, tp_rank: int = 0, tp_size: int = 1, device="cpu",
                  dtype: Optional[torch.dtype] = None, quantize: Optional[str] = None,
@@ -575,7 +639,7 @@ class WeightLoader:
             else:
                 self._put(name, t)
             return
-        m = re.match(r"(model\.layers\.\d+)\.(self_attn|mlp)\.(.*)$", name)
+        m = re.match(r"(model\.layers\.\d+)\.(self_attn|mlp|mixer)\.(.*)$", name)
         if not m:
             mm = re.match(r"(model\.layers\.\d+)\.(eh_proj)\.(weight|weight_scale_inv)$", name)
             if mm:
@@ -725,6 +789,10 @@ class WeightLoader:
     def _maybe_flush(self, key: str) -> None:
         cfg = self.cfg
         p = self._pending[key]
+        if key.endswith(".mixer"):
+            if mixer_parts(cfg.layers[self._layer_of(key)]) <= set(p):
+                self._finish_mixer(key, self._pending.pop(key))
+            return
         if key.endswith(".self_attn"):
             if cfg.use_mla:
                 # (the *_layernorm weights never enter the pending set: norm tensors are placed directly)
@@ -782,6 +850,9 @@ class WeightLoader:
         for key, parts in list(self._pending.items()):
             if key.endswith(".eh_proj"):
                 self._put_linear(key, parts["weight"], parts.get("weight_scale_inv"))
+            elif key.endswith(".mixer"):
+                missing = mixer_parts(cfg.layers[self._layer_of(key)]) - set(parts)
+                raise KeyError(f"{key}: the checkpoint has no {', '.join(sorted(missing))}")
             elif key.endswith(".self_attn"):
                 if cfg.use_mla:
                     self._finish_mla(key, parts)
@@ -799,6 +870,32 @@ class WeightLoader:
         self._expert_pqs.clear()
         self._pending.clear()
         self._experts.clear()
+
+    def _finish_mixer(self, key: str, p: Dict[str, torch.Tensor]) -> None:
+        """All tensors of a layer's mixers: their input projections become one weight (attention q, k, v, then linear
+        attention q, k, v, gate) and their output projections one, side by side along the input. Both are padded with
+        zeros to the multiples of eight that the GEMM takes."""
+        spec = self.cfg.layers[self._layer_of(key)]
+        pa, pl = mixer_prefixes(spec)
+        rows, biases, outs = [], [], []
+        for pre, names, has_bias in ((pa, "qkv", spec.attn is not None and spec.attn.qkv_bias), (pl, "qkvg", False)):
+            if pre is None:
+                continue
+            for x in names:
+                w = p[pre + x]
+                rows.append(w)
+                biases.append(p[pre + x + ".b"] if has_bias else torch.zeros(w.shape[0], dtype=w.dtype, device=w.device))
+            outs.append(p[pre + "o"])
+        pad = torch.nn.functional.pad
+        w_in, w_out = torch.cat(rows, 0), torch.cat(outs, 1)
+        extra = -w_in.shape[0] % 8
+        self._put_linear(key + ".in_proj", pad(w_in, (0, 0, 0, extra)))
+        if spec.attn is not None and spec.attn.qkv_bias:
+            self._put(key + ".in_proj.bias", pad(torch.cat(biases, 0), (0, extra)))
+        self._put_linear(key + ".o_proj", pad(w_out, (0, -w_out.shape[1] % 8)))
+        for pre, name, out in ((pa, "q.norm", "q_norm"), (pa, "k.norm", "k_norm"), (pa, "rel", "rel"), (pl, "norm", "norm")):
+            if pre is not None and pre + name in p:
+                self.out[f"{key}.{out}"] = self._own(p[pre + name].float())
 
     def _finish_attn(self, key: str, p: Dict[str, torch.Tensor]) -> None:
         cfg, r, n = self.cfg, self.rank, self.size

@@ -33,6 +33,8 @@ FAMILIES: Dict[str, str] = {
     "deepseek_v3": "MLA + sigmoid routing with correction bias, 8 groups / top-4, MTP layer, fp8 block weights; "
                    "V3.2 / GLM DSA: sparse attention over the keys picked by the indexer",
     "kimi_k2": "deepseek_v3 architecture with 384 experts",
+    "molopel": "layers of linear attention with fixed decays, alone or beside windowed attention with a learned distance "
+               "bias; recurrent state slots, LayerNorm, 32-bit residual, soft-capped logits",
     "minicpm": "embedding / residual / logit scaling; reranker head",
 }
 

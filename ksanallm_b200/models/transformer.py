@@ -18,6 +18,7 @@ from ..config.model_config import ModelConfig
 from ..ops import reference as ref
 from ..parallel.comm import TPGroup
 from .layers import Attention, DenseFFN, LinearW, MLAttention, MoEFFN
+from .mixers import LayerCache, MixerLayer, RotaryTables
 
 
 class DecoderLayer:
@@ -95,8 +96,12 @@ class TransformerModel:
             self.rope_cache = ref.build_rope_cache(rd, maxp, cfg.rope_theta, cfg.rope_scaling, self.device)
         self.progress = None  # optional per-layer completion tracker (prefill/decode disaggregation)
         self.layer_ids = list(layer_range) if layer_range is not None else list(range(cfg.num_layers))
-        self.layers: List[DecoderLayer] = [DecoderLayer(cfg, weights, i, self.tp, self.rope_cache)
-                                           for i in self.layer_ids]
+        self.rotary_tables = RotaryTables(self.device)  # of the layers that bring their own rotation
+        if cfg.layers:
+            self.layers = [MixerLayer(cfg, weights, i, self.tp, self.rotary_tables) for i in self.layer_ids]
+            self.reserve_positions(min(max_positions or 1, maxp))
+        else:
+            self.layers = [DecoderLayer(cfg, weights, i, self.tp, self.rope_cache) for i in self.layer_ids]
         self.norm_w = weights.get("model.norm.weight")
         self.norm_b = weights.get("model.norm.bias")
         self.lm_head = weights.get("lm_head.weight")
@@ -109,7 +114,28 @@ class TransformerModel:
             if p + ".eh_proj.weight" in weights:
                 self.mtp_layers.append(MTPLayer(cfg, weights, cfg.num_layers + j, self.tp, self.rope_cache))
 
-    # ---- KV cache -------------------------------------------------------------------------------
+    def reserve_positions(self, length: int) -> None:
+        """Makes the position tables of layers that bring their own cover ``length`` positions."""
+        if self.cfg.layers:
+            self.rotary_tables.reserve(length)
+            for layer in self.layers:
+                layer.reserve(length)
+
+    # ---- KV cache and recurrent state ------------------------------------------------------------
+    def state_slot_bytes(self) -> int:
+        """Bytes of one sequence's recurrent state across all local layers."""
+        if not self.cfg.has_state:
+            return 0
+        return sum(4 * h * d * dv for h, d, dv in (layer.state_shape() for layer in self.layers))
+
+    def allocate_state(self, num_slots: int) -> Optional[List[torch.Tensor]]:
+        """One fp32 pool [num_slots, heads, dim, vdim] per layer (empty for a layer without state), or None for a
+        model without any. A slot needs no clearing: a sequence's first step does not read it."""
+        if not self.cfg.has_state:
+            return None
+        return [torch.zeros(num_slots, *layer.state_shape(), dtype=torch.float32, device=self.device)
+                for layer in self.layers]
+
     @property
     def num_cache_layers(self) -> int:
         return len(self.layers) + len(self.mtp_layers)
@@ -118,6 +144,8 @@ class TransformerModel:
         """Bytes of one block across all local layers (used to size the block pool)."""
         cfg = self.cfg
         esz = torch.empty(0, dtype=kv_dtype or self.dtype).element_size()
+        if cfg.layers:
+            return sum(layer.kv_width() for layer in self.layers) * block_size * esz
         if cfg.use_mla:
             per_layer = block_size * (cfg.kv_lora_rank + cfg.qk_rope_head_dim + cfg.index_head_dim * bool(cfg.index_topk)) * esz
         else:
@@ -128,6 +156,11 @@ class TransformerModel:
     def allocate_kv_cache(self, num_blocks: int, block_size: int, kv_dtype: Optional[torch.dtype] = None):
         cfg = self.cfg
         dt = kv_dtype or self.dtype
+        if cfg.layers:
+            if kv_dtype is not None and kv_dtype != self.dtype:
+                raise NotImplementedError("layers with mixers of their own keep their keys and values in the model dtype")
+            return [torch.zeros(num_blocks, block_size * layer.kv_width(), dtype=dt, device=self.device)
+                    for layer in self.layers]
         caches = []
         for _ in range(self.num_cache_layers):
             if cfg.use_mla:
@@ -142,7 +175,8 @@ class TransformerModel:
 
     # ---- forward --------------------------------------------------------------------------------
     def embed_tokens(self, meta, refit=None) -> torch.Tensor:
-        x = ops.embedding(meta.input_ids, self.embed, self.cfg.emb_scale)
+        x = ops.embedding(meta.input_ids, self.embed, self.cfg.emb_scale,
+                          torch.float32 if self.cfg.residual_fp32 else None)
         if self.pos_embed is not None:
             x = x + self.pos_embed[meta.positions.long()]
         if refit is not None:
@@ -152,13 +186,15 @@ class TransformerModel:
         return x
 
     def forward(self, meta, kv_caches, refit=None, cutoff_layer: Optional[int] = None,
-                hidden_in: Optional[torch.Tensor] = None) -> torch.Tensor:
+                hidden_in: Optional[torch.Tensor] = None, states: Optional[List[torch.Tensor]] = None) -> torch.Tensor:
         """Returns the final normalised hidden states [T, H]. ``self.last_residual`` then holds the
         un-normalised residual stream (the "transformer" probe target).
 
         Pipeline stages: ``hidden_in`` is the residual stream received from the previous stage (no embedding
         lookup); a stage built without ``model.norm.weight`` (not the last one) returns the un-normalised residual
-        stream for the next stage."""
+        stream for the next stage. ``states``: the recurrent-state pools of a model that has them."""
+        if self.cfg.layers:
+            kv_caches = [LayerCache(kv, st) for kv, st in zip(kv_caches, states)]
         x = self.embed_tokens(meta, refit) if hidden_in is None else hidden_in
         layers = self.layers if cutoff_layer is None else self.layers[:cutoff_layer]
         residual = x
@@ -200,12 +236,15 @@ class TransformerModel:
         if self.norm_w is None:
             return x
         if self.cfg.norm_type == "layernorm":
-            return ops.layer_norm(x, self.norm_w, self.norm_b, self.cfg.rms_norm_eps)
+            return ops.layer_norm(x, self.norm_w, self.norm_b, self.cfg.rms_norm_eps, None, self.dtype)
         return ops.rms_norm(x, self.norm_w, self.cfg.rms_norm_eps)
 
     def compute_logits(self, hidden: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """fp32 logits for the selected rows; vocab shards are gathered across the TP group."""
         h = hidden if rows is None else hidden.index_select(0, rows.long())
+        if self.cfg.logit_softcap:
+            return ops.softcap(ops.linear(h, self.lm_head, None, torch.float32)[:, :self.cfg.vocab_size],
+                               self.cfg.logit_softcap)
         logits = ops.linear(h, self.lm_head)
         if self.tp.size > 1 and self.lm_head.shape[0] < self.cfg.vocab_size:
             logits = self.tp.all_gather(logits, dim=-1)
@@ -218,6 +257,8 @@ class TransformerModel:
         """argmax over the full vocabulary without materialising gathered logits on every rank:
         local (max, index) pairs are exchanged instead (reference: greedy.cu:240-424 +
         common_model.cpp:591-617)."""
+        if self.cfg.logit_softcap:
+            return ops.argmax(self.compute_logits(hidden, rows))
         h = hidden.index_select(0, rows.long())
         logits = ops.linear(h, self.lm_head).float()
         if self.tp.size == 1 or self.lm_head.shape[0] >= self.cfg.vocab_size:

@@ -18,14 +18,21 @@ def _cuda():
     return _c
 
 
+def _mixer():
+    from . import cuda_mixer as _c
+    return _c
+
+
 def rms_norm(x, weight, eps, residual=None):
     if x.is_cuda:
         return _cuda().rms_norm(x, weight, eps, residual)
     return ref.rms_norm(x, weight, eps, residual)
 
 
-def layer_norm(x, weight, bias, eps, residual=None):
-    return ref.layer_norm(x, weight, bias, eps, residual)
+def layer_norm(x, weight, bias, eps, residual=None, out_dtype=None):
+    if x.is_cuda:
+        return _mixer().layer_norm(x, weight, bias, eps, residual, out_dtype)
+    return ref.layer_norm(x, weight, bias, eps, residual, out_dtype)
 
 
 def _library_baseline() -> bool:
@@ -35,12 +42,14 @@ def _library_baseline() -> bool:
     return os.environ.get("KSANA_LIBRARY_BASELINE", "0") == "1"
 
 
-def linear(x, weight, bias=None):
+def linear(x, weight, bias=None, out_dtype=None):
+    """``out_dtype`` float32: the accumulator leaves unrounded."""
     if x.is_cuda:
         if _library_baseline():
-            return torch.nn.functional.linear(x, weight, bias)
-        return _cuda().linear(x, weight, bias)
-    return ref.linear(x, weight, bias)
+            y = torch.nn.functional.linear(x, weight, bias)
+            return y if out_dtype is None else y.to(out_dtype)
+        return _cuda().linear(x, weight, bias, out_dtype)
+    return ref.linear(x, weight, bias, out_dtype)
 
 
 def linear_fp8_block(x, wq, w_scale_inv, bias=None, sfb=None, pow2=False):
@@ -63,14 +72,22 @@ def silu_and_mul(x):
     return ref.silu_and_mul(x)
 
 
+def gelu_and_mul(x):
+    if x.is_cuda:
+        return _mixer().gelu_and_mul(x)
+    return ref.gelu_and_mul(x)
+
+
 def activation(x, kind):
     return ref.activation(x, kind)
 
 
-def embedding(ids, table, scale=1.0):
+def embedding(ids, table, scale=1.0, out_dtype=None):
     if ids.is_cuda:
+        if out_dtype is not None:
+            return _mixer().embedding(ids, table, scale, out_dtype)
         return _cuda().embedding(ids, table, scale)
-    return ref.embedding(ids, table, scale)
+    return ref.embedding(ids, table, scale, out_dtype)
 
 
 def rope_qknorm_cache(q, k, v, positions, cos_sin, slot_mapping, kv_cache, q_norm_w=None, k_norm_w=None,
@@ -92,6 +109,40 @@ def paged_attention(q, kv_cache, meta, scale, alibi_slopes=None, k_scale=1.0, v_
         return _cuda().paged_attention(q, kv_cache, meta, scale, alibi_slopes, k_scale, v_scale, window)
     return ref.paged_attention(q, kv_cache, meta.block_tables, meta.cu_q, meta.kv_lens, scale, alibi_slopes,
                                k_scale, v_scale, window)
+
+
+def qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps):
+    f = _mixer() if q.is_cuda else ref
+    return f.qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps)
+
+
+def window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out):
+    """Writes heads * vdim columns of ``out`` [T, ...] (a column slice is fine)."""
+    if q.is_cuda:
+        _mixer().window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out)
+        return
+    out.copy_(ref.window_attention(q, cache, meta.block_tables, meta.cu_q, meta.kv_lens, block_size, kv_heads, vdim,
+                                   scale, window, bias, out_scale).flatten(1))
+
+
+def linear_attention(q, k, v, state, meta, decay, act, rotary, key_scale):
+    if q.is_cuda:
+        return _mixer().linear_attention(q, k, v, state, meta, decay, act, rotary, key_scale)
+    return ref.linear_attention(q, k, v, state, meta.state_slots, meta.cu_q, meta.kv_lens, meta.positions, decay, act,
+                                rotary, key_scale)
+
+
+def gated_norm(o, g, weight, eps, gate, out_scale, out):
+    if o.is_cuda:
+        _mixer().gated_norm(o, g, weight, eps, gate, out_scale, out)
+        return
+    out.copy_(ref.gated_norm(o, g, weight, eps, gate, out_scale))
+
+
+def softcap(logits, cap):
+    if logits.is_cuda:
+        return _mixer().softcap(logits, cap)
+    return ref.softcap(logits, cap)
 
 
 def mla_cache_append(latent, k_rope, slot_mapping, cache):

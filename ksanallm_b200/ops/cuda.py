@@ -20,18 +20,18 @@ _lib = None
 launch_count = 0  # number of kernel-library launches issued (each is at least one CUDA kernel)
 
 
-def lib():
+def lib(family: str = ""):
+    """The loaded kernel library. ``family``: on the first call, a model family whose kernels suffice (see
+    _build.FAMILY_SOURCES); launchers outside that family are then absent."""
     global _lib
     if _lib is None:
-        path = _build.LIB / "libksana_kernels.so"
+        path = _build.usable_library(family)
         if not path.exists():
-            _build.build_cuda()
-        if not path.exists():
-            raise RuntimeError("libksana_kernels.so is missing: run `python -m ksanallm_b200._build`")
+            raise RuntimeError(f"{path.name} is missing: run `python -m ksanallm_b200._build`")
         _lib = ctypes.CDLL(str(path))
         for name in dir(_Sig):
-            if name.startswith("ksana_"):
-                fn = getattr(_lib, name)
+            fn = getattr(_lib, name, None) if name.startswith("ksana_") else None
+            if fn is not None:
                 fn.argtypes, fn.restype = getattr(_Sig, name)
     return _lib
 
@@ -75,6 +75,14 @@ class _Sig:
     ksana_gemm_bf16_batched = ([P, LL, LL, P, P, LL, LL, I, I, I, I, P], I)
     ksana_mla_rope_append = ([P, LL, I, I, P, P, I, P, I, P, P, P, P, I, I, I, I, I, I, P], I)
     ksana_block_copy = ([P, P, I, P, I, LL, P], I)
+    ksana_layer_norm = ([P, I, P, I, P, P, P, I, I, I, F, I, P], I)
+    ksana_embedding_f32 = ([P, P, P, I, I, I, F, I, P], I)
+    ksana_gelu_mul = ([P, I, P, I, I, I, I, P], I)
+    ksana_qk_norm_cache = ([P, I, P, I, P, I, P, P, P, P, F, I, I, I, I, I, I, I, P], I)
+    ksana_gated_norm = ([P, P, I, P, P, I, I, I, I, F, I, F, I, P], I)
+    ksana_softcap = ([P, I, P, I, I, F, P], I)
+    ksana_window_attention_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
+    ksana_linear_recurrent = ([P, I, P, I, P, I, P, P, P, P, P, P, P, I, I, F, I, I, I, P, I, I, I, I, P], I)
     ksana_logits_process = ([P, I, I, I, P, P, P, P, P, P, P, P, P, P, P, I, P], I)
 
 
@@ -143,7 +151,8 @@ def gemm_bf16(x: torch.Tensor, w: torch.Tensor, bias: Optional[torch.Tensor] = N
     return out
 
 
-def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
+           out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     if x.dtype == torch.float32 or weight.dtype == torch.float32:
         # fp32 router / probe paths: tiny GEMMs outside the bf16 hot path
         y = x.float() @ weight.float().t()
@@ -152,9 +161,9 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
     x2 = x.reshape(-1, x.shape[-1])
     N, K = weight.shape
     if N % 8 or K % 8:
-        y = ref.linear(x2, weight, bias)
+        y = ref.linear(x2, weight, bias, out_dtype)
     else:
-        y = gemm_bf16(x2, weight, bias)
+        y = gemm_bf16(x2, weight, bias, out_dtype)
     return y.view(*lead, N)
 
 

@@ -1,0 +1,113 @@
+"""ctypes wrappers of the kernels behind layers with mixers of their own sizes (csrc/cuda/mixer_elementwise.cu,
+window_attention.cu, linear_attention.cu). bf16 and fp32 storage; everything is computed in 32-bit floats."""
+from __future__ import annotations
+
+from typing import Optional
+
+import torch
+
+from .cuda import _check, _ptr, _stream, lib
+
+_KIND = {torch.float32: 0, torch.bfloat16: 1}
+
+
+def _rows(x: torch.Tensor) -> torch.Tensor:
+    """[rows, H] view with a contiguous last dimension."""
+    x = x.reshape(-1, x.shape[-1])
+    return x if x.stride(1) == 1 else x.contiguous()
+
+
+def layer_norm(x, weight, bias, eps: float, residual: Optional[torch.Tensor] = None, out_dtype=None) -> torch.Tensor:
+    x2 = _rows(x)
+    out = torch.empty(x2.shape, dtype=out_dtype or x.dtype, device=x.device)
+    r2 = residual.view(-1, x2.shape[1]) if residual is not None else None
+    rk = _KIND[r2.dtype] if r2 is not None else (0 if x.dtype == torch.float32 else _KIND[out.dtype])
+    kinds = _KIND[x.dtype] | rk << 1 | _KIND[weight.dtype] << 2 | _KIND[out.dtype] << 3
+    if bias is not None:
+        bias = bias.to(weight.dtype)
+    _check(lib().ksana_layer_norm(_ptr(x2), x2.stride(0), _ptr(r2), r2.stride(0) if r2 is not None else 0, _ptr(weight),
+                                  _ptr(bias), _ptr(out), out.stride(0), x2.shape[0], x2.shape[1], float(eps), kinds,
+                                  _stream()), "layer_norm")
+    return out.view(x.shape)
+
+
+def embedding(ids, table, scale: float, out_dtype) -> torch.Tensor:
+    assert out_dtype == torch.float32 and table.is_contiguous()
+    T, H = ids.numel(), table.shape[1]
+    out = torch.empty(T, H, dtype=torch.float32, device=table.device)
+    _check(lib().ksana_embedding_f32(_ptr(ids), _ptr(table), _ptr(out), T, H, table.shape[0], float(scale),
+                                     _KIND[table.dtype], _stream()), "embedding_f32")
+    return out
+
+
+def gelu_and_mul(x: torch.Tensor) -> torch.Tensor:
+    T, two_i = x.shape
+    out = torch.empty(T, two_i // 2, dtype=x.dtype, device=x.device)
+    _check(lib().ksana_gelu_mul(_ptr(x), x.stride(0), _ptr(out), out.stride(0), T, two_i // 2, _KIND[x.dtype],
+                                _stream()), "gelu_mul")
+    return out
+
+
+def _packed_heads(x: torch.Tensor) -> torch.Tensor:
+    assert x.stride(2) == 1 and (x.shape[1] == 1 or x.stride(1) == x.shape[2])
+    return x
+
+
+def qk_norm_cache(q, k, v, slot_mapping, cache, block_size: int, q_norm, k_norm, eps: float) -> None:
+    T, h, d = q.shape
+    hk, dv = v.shape[1], v.shape[2]
+    for x in (q, k, v):
+        _packed_heads(x)
+    assert cache.dtype == q.dtype and cache.is_contiguous()
+    _check(lib().ksana_qk_norm_cache(_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0),
+                                     _ptr(slot_mapping), _ptr(cache), _ptr(q_norm), _ptr(k_norm), float(eps), T, h, hk,
+                                     d, dv, block_size, _KIND[q.dtype], _stream()), "qk_norm_cache")
+
+
+def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, scale: float, window: int, bias,
+                     out_scale: float, out: torch.Tensor) -> None:
+    T, h, d = q.shape
+    _packed_heads(q)
+    assert out.stride(1) == 1
+    _check(lib().ksana_window_attention_any(
+        _ptr(q), q.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks, _ptr(meta.cu_q),
+        _ptr(meta.kv_lens), _ptr(meta.seq_of_token), h, kv_heads, d, vdim, block_size, window, float(scale), _ptr(bias),
+        bias.shape[1] if bias is not None else 0, float(out_scale), _ptr(out), out.stride(0), 0, T, _KIND[q.dtype],
+        _stream()), "window_attention_any")
+
+
+def linear_attention(q, k, v, state, meta, decay, act: str, rotary, key_scale: float) -> torch.Tensor:
+    T, h, d = q.shape
+    dv = v.shape[2]
+    for x in (q, k, v):
+        _packed_heads(x)
+    out = torch.empty(T, h, dv, dtype=q.dtype, device=q.device)
+    rd = rotary.shape[1] if rotary is not None else 0
+    n_pre, n_dec = meta.num_prefill, meta.num_decode
+    one = n_dec > 0 and meta.num_decode_tokens == n_dec
+    for base, count, single in ((0, n_pre, 0), (n_pre, n_dec, 1 if one else 0)):
+        if count:
+            _check(lib().ksana_linear_recurrent(
+                _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(state), _ptr(meta.state_slots),
+                _ptr(meta.cu_q), _ptr(meta.kv_lens), _ptr(meta.positions), _ptr(decay), _ptr(rotary), rd,
+                1 if act == "silu" else 0, float(key_scale), h, d, dv, _ptr(out), base, count, single, _KIND[q.dtype],
+                _stream()), "linear_recurrent")
+    return out
+
+
+def gated_norm(o, g, weight, eps: float, gate: str, out_scale: float, out: torch.Tensor) -> None:
+    T, h, dv = o.shape
+    assert o.is_contiguous() and g.stride(1) == 1 and out.stride(1) == 1
+    _check(lib().ksana_gated_norm(_ptr(o), _ptr(g), g.stride(0), _ptr(weight), _ptr(out), out.stride(0), T, h, dv,
+                                  float(eps), 1 if gate == "sigmoid" else 0, float(out_scale), _KIND[o.dtype],
+                                  _stream()), "gated_norm")
+
+
+def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    rows, n = logits.shape
+    x = logits.float()
+    if x.stride(1) != 1:
+        x = x.contiguous()
+    out = torch.empty(rows, n, dtype=torch.float32, device=x.device)
+    _check(lib().ksana_softcap(_ptr(x), x.stride(0), _ptr(out), rows, n, float(cap), _stream()), "softcap")
+    return out

@@ -30,24 +30,25 @@ def rms_norm(x: torch.Tensor, weight: torch.Tensor, eps: float,
 
 
 def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float,
-               residual: Optional[torch.Tensor] = None) -> torch.Tensor:
+               residual: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     xf = x.float()
     if residual is not None:
         xf = xf + residual.float()
         residual.copy_(xf.to(residual.dtype))
         xf = residual.float()
     y = F.layer_norm(xf, (xf.shape[-1],), weight.float(), None if bias is None else bias.float(), eps)
-    return y.to(x.dtype)
+    return y.to(out_dtype or x.dtype)
 
 
 # ---- dense linear algebra -------------------------------------------------------------------------
 
-def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
+           out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """y[T, N] = x[T, K] @ weight[N, K]^T (+ bias), fp32 accumulation."""
     y = x.float() @ weight.float().t()
     if bias is not None:
         y = y + bias.float()
-    return y.to(x.dtype)
+    return y.to(out_dtype or x.dtype)
 
 
 def silu_and_mul(x: torch.Tensor) -> torch.Tensor:
@@ -80,8 +81,11 @@ def activation(x: torch.Tensor, kind: str) -> torch.Tensor:
     return y.to(x.dtype)
 
 
-def embedding(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0) -> torch.Tensor:
+def embedding(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0,
+              out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     y = table[ids.long()]
+    if out_dtype is not None and out_dtype != table.dtype:
+        return y.to(out_dtype) * scale
     return y if scale == 1.0 else (y.float() * scale).to(table.dtype)
 
 
@@ -324,6 +328,130 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_tables: torch
         p = torch.softmax(s, dim=-1)
         out[qs:qe] = torch.einsum("hqk,hkd->hqd", p, V).permute(1, 0, 2).to(q.dtype)
     return out
+
+
+# ---- layers with mixers of their own sizes: windowed attention with a distance bias, linear attention ---------------
+
+def split_kv_cache(cache: torch.Tensor, hk: int, bs: int, d: int, dv: int) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Views [nb, hk, bs, d] and [nb, hk, bs, dv] of a layer cache [nb, hk * bs * (d + dv)] (keys, then values)."""
+    nb, cut = cache.shape[0], hk * bs * d
+    return cache[:, :cut].view(nb, hk, bs, d), cache[:, cut:].view(nb, hk, bs, dv)
+
+
+def qk_norm_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, slot_mapping: torch.Tensor, cache: torch.Tensor,
+                  block_size: int, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float) -> None:
+    """Per-head RMS norm of q (in place) and k, then k and v go to their cache slots. q [T, h, d], k [T, hk, d],
+    v [T, hk, dv] may be row-strided views; the cache has the layout of :func:`split_kv_cache`."""
+    hk, d, dv = k.shape[1], k.shape[2], v.shape[2]
+
+    def unit(x, w):
+        xf = x.float()
+        return (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(x.dtype)
+
+    if q_norm is not None:
+        q.copy_(unit(q, q_norm))
+    kn = unit(k, k_norm) if k_norm is not None else k
+    K, V = split_kv_cache(cache, hk, block_size, d, dv)
+    slots = slot_mapping.long()
+    blk, off = slots // block_size, slots % block_size
+    K[blk, :, off] = kn.to(cache.dtype)
+    V[blk, :, off] = v.to(cache.dtype)
+
+
+def distance_bias(rel: torch.Tensor, bias_max: float, count: int) -> torch.Tensor:
+    """[heads, count] fp32: the learned bias of every distance 0 .. count - 1. ``rel`` [rows, heads]: the first half of
+    the rows belongs to one distance each, the rest to log-spaced ranges that end at ``bias_max``."""
+    rows = rel.shape[0]
+    half = rows // 2
+    n = torch.arange(count, dtype=torch.float64)
+    x = torch.log(n.clamp(min=max(half, 1)) / max(half, 1)) / math.log(bias_max / max(half, 1)) * (rows - half)
+    near = torch.round(x)  # a distance that lies exactly on a boundary must not fall below it by rounding
+    x = torch.where((x - near).abs() < 1e-9, near, torch.floor(x))
+    bucket = torch.where(n < half, n, (half + x).clamp(max=rows - 1)).long()
+    return rel.float()[bucket.to(rel.device)].t().contiguous()
+
+
+def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, cu_q: torch.Tensor,
+                     kv_lens: torch.Tensor, block_size: int, hk: int, dv: int, scale: float, window: int,
+                     bias: Optional[torch.Tensor], out_scale: float = 1.0) -> torch.Tensor:
+    """Softmax attention of each sequence's new tokens over its newest ``window`` keys (0: all), with a bias per head
+    and distance (``bias`` [h, >= reach], None: none). q [T, h, d]; returns [T, h, dv]."""
+    T, h, d = q.shape
+    K, V = split_kv_cache(cache, hk, block_size, d, dv)
+    out = torch.empty(T, h, dv, dtype=q.dtype, device=q.device)
+    cu, kl, group = cu_q.tolist(), kv_lens.tolist(), h // hk
+    for b in range(len(kl)):
+        ql, L = cu[b + 1] - cu[b], kl[b]
+        if ql == 0:
+            continue
+        lo = max(0, L - ql - window + 1) // block_size * block_size if window else 0
+        blocks = block_tables[b, lo // block_size:(L + block_size - 1) // block_size].long()
+        kb = K[blocks].permute(1, 0, 2, 3).reshape(hk, -1, d)[:, :L - lo].float().repeat_interleave(group, 0)
+        vb = V[blocks].permute(1, 0, 2, 3).reshape(hk, -1, dv)[:, :L - lo].float().repeat_interleave(group, 0)
+        s = torch.einsum("qhd,hkd->hqk", q[cu[b]:cu[b + 1]].float(), kb) * scale
+        dist = torch.arange(L - ql, L, device=q.device).unsqueeze(1) - torch.arange(lo, L, device=q.device)
+        if bias is not None:
+            s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
+        hidden = dist < 0
+        if window:
+            hidden = hidden | (dist >= window)
+        p = torch.softmax(s.masked_fill(hidden.unsqueeze(0), float("-inf")), dim=-1)
+        out[cu[b]:cu[b + 1]] = (torch.einsum("hqk,hkd->qhd", p, vb) * out_scale).to(q.dtype)
+    return out
+
+
+def rotary_table(dims: int, base: float, count: int, device="cpu") -> torch.Tensor:
+    """[count, dims] fp32 = [cos | sin] of position * base^(-2 i / dims)."""
+    inv = base ** (-torch.arange(0, dims // 2, dtype=torch.float64) * 2 / dims)
+    a = torch.arange(count, dtype=torch.float64).unsqueeze(1) * inv
+    return torch.cat((a.cos(), a.sin()), 1).float().to(device)
+
+
+def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
+                     cu_q: torch.Tensor, kv_lens: torch.Tensor, positions: torch.Tensor, decay: torch.Tensor,
+                     act: str = "none", rotary: Optional[torch.Tensor] = None, key_scale: float = 1.0) -> torch.Tensor:
+    """S <- decay S + k v^T, o = S^T q, the state of sequence b living in ``state[slots[b]]`` ([h, d, dv] fp32). A
+    sequence whose first token is among the new ones starts from zero whatever its slot holds. ``act`` is applied to
+    q, k and v first, then q and k are rotated by ``rotary`` and k is scaled."""
+    T, h, d = q.shape
+    qf, kf, vf = q.float(), k.float(), v.float()
+    if act == "silu":
+        qf, kf, vf = F.silu(qf), F.silu(kf), F.silu(vf).to(v.dtype).float()
+    if rotary is not None:
+        cs = rotary[positions.long()]
+        rd = cs.shape[1]
+        qf = apply_rope(qf, cs[:, :rd // 2], cs[:, rd // 2:], False, rd)
+        kf = apply_rope(kf, cs[:, :rd // 2], cs[:, rd // 2:], False, rd)
+    kf = kf * key_scale
+    out = torch.empty(T, h, v.shape[2], dtype=q.dtype, device=q.device)
+    cu, kl, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
+    dec = decay.float().view(h, 1, 1)
+    for b in range(len(kl)):
+        S = torch.zeros_like(state[0]) if kl[b] == cu[b + 1] - cu[b] else state[sl[b]].clone()
+        for t in range(cu[b], cu[b + 1]):
+            S = dec * S + kf[t].unsqueeze(2) * vf[t].unsqueeze(1)
+            out[t] = torch.einsum("hde,hd->he", S, qf[t]).to(q.dtype)
+        if cu[b + 1] > cu[b]:
+            state[sl[b]] = S
+    return out
+
+
+def gated_norm(o: torch.Tensor, g: torch.Tensor, weight: Optional[torch.Tensor], eps: float, gate: str,
+               out_scale: float = 1.0) -> torch.Tensor:
+    """RMS norm of o [T, h, dv] - per head without a weight, over all heads together with one - times gate(g),
+    g [T, h * dv]; returns [T, h * dv]."""
+    T = o.shape[0]
+    of = o.float() if weight is None else o.float().reshape(T, 1, -1)
+    of = (of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, -1)
+    if weight is not None:
+        of = of * weight.float()
+    gf = g.float()
+    gf = torch.sigmoid(gf) if gate == "sigmoid" else F.silu(gf)
+    return (of * gf * out_scale).to(o.dtype)
+
+
+def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:
+    return cap * torch.tanh(logits.float() / cap)
 
 
 def mla_cache_append(latent: torch.Tensor, k_rope: torch.Tensor, slot_mapping: torch.Tensor,

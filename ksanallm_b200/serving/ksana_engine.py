@@ -108,7 +108,8 @@ class EngineArgs:
         cfg_path = os.path.join(a.model_dir or "", "config.json")
         if os.path.isfile(cfg_path):
             with open(cfg_path, "r", encoding="utf-8") as f:
-                a.model_type = str(json.load(f).get("model_type", ""))
+                raw = json.load(f)
+            a.model_type = str(raw.get("model_type") or raw.get("architecture", "")).lower()
         return a
 
     @classmethod
