@@ -24,23 +24,7 @@ constexpr int PF_BQ = 128;   // query rows per CTA
 constexpr int PF_BKV = 128;  // kv tokens per tile
 constexpr int PF_PAGE = 16;
 
-__host__ __device__ constexpr uint32_t idesc_pv(int n) {
-  // bf16 x bf16 -> f32, A K-major, B MN-major (bit 16)
-  return (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | (static_cast<uint32_t>(n >> 3) << 17) |
-         (static_cast<uint32_t>(128 >> 4) << 24);
-}
-
-// MN-major 128-byte-swizzled operand: 64 elements contiguous along MN (one 128-byte row), 8 K-rows per 1024 bytes,
-// next 8 K-rows at +1024 (SBO), next 64 MN elements at +lbo_bytes (LBO).
-__device__ __forceinline__ uint64_t umma_desc_mn128(uint32_t smem_addr, uint32_t lbo_bytes) {
-  uint64_t d = 0;
-  d |= static_cast<uint64_t>((smem_addr >> 4) & 0x3FFF);
-  d |= static_cast<uint64_t>((lbo_bytes >> 4) & 0x3FFF) << 16;
-  d |= static_cast<uint64_t>(1024 >> 4) << 32;
-  d |= static_cast<uint64_t>(1) << 46;
-  d |= static_cast<uint64_t>(2) << 61;
-  return d;
-}
+__host__ __device__ constexpr uint32_t idesc_pv(int n) { return umma_idesc_major(128, n, false, true); }
 
 template <int D>
 struct PrefillSmem {

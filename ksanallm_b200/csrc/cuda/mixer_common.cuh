@@ -81,6 +81,14 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return z / (1.f + expf(-2.f * u));
 }
 
+// v = hi + lo with both parts bf16: the pair keeps 16 bits of the mantissa through 16-bit tensor-core operands. Packs
+// two values; *lo is exact up to its own rounding.
+__device__ __forceinline__ uint32_t split_bf16(float a, float b, uint32_t* lo) {
+  const uint32_t hi = pack_bf16(a, b);
+  *lo = pack_bf16(a - __uint_as_float(hi << 16), b - __uint_as_float(hi & 0xffff0000u));
+  return hi;
+}
+
 // Sum over the block (a multiple of 32 threads, at most 1024); every thread gets it. `red` holds 32 floats.
 __device__ __forceinline__ float block_sum(float v, float* red) {
   v = warp_sum(v);

@@ -207,6 +207,22 @@ __host__ __device__ constexpr uint32_t umma_idesc(int m, int n, int a_fmt, int b
          (static_cast<uint32_t>(n >> 3) << 17) | (static_cast<uint32_t>(m >> 4) << 24);
 }
 
+// bf16 x bf16 -> fp32 with either operand K-major or MN-major (bits 15 and 16).
+__host__ __device__ constexpr uint32_t umma_idesc_major(int m, int n, bool a_mn, bool b_mn) {
+  return umma_idesc(m, n, 1, 1) | (a_mn ? 1u << 15 : 0u) | (b_mn ? 1u << 16 : 0u);
+}
+// MN-major 128-byte-swizzled operand: 64 elements contiguous along MN (one 128-byte row), 8 K-rows per 1024 bytes,
+// next 8 K-rows at +1024 (SBO), next 64 MN elements at +lbo_bytes (LBO).
+__device__ __forceinline__ uint64_t umma_desc_mn128(uint32_t smem_addr, uint32_t lbo_bytes) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((smem_addr >> 4) & 0x3FFF);
+  d |= static_cast<uint64_t>((lbo_bytes >> 4) & 0x3FFF) << 16;
+  d |= static_cast<uint64_t>(1024 >> 4) << 32;
+  d |= static_cast<uint64_t>(1) << 46;
+  d |= static_cast<uint64_t>(2) << 61;
+  return d;
+}
+
 // D[tmem] (+)= A[smem] * B[smem]^T, bf16/fp16 inputs. One thread issues.
 __device__ __forceinline__ void umma_f16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc,
                                          uint32_t accumulate) {
@@ -323,6 +339,11 @@ __device__ __forceinline__ float4 ld_cluster_f4(uint32_t cluster_addr) {
                : "=f"(v.x), "=f"(v.y), "=f"(v.z), "=f"(v.w)
                : "r"(cluster_addr)
                : "memory");
+  return v;
+}
+__device__ __forceinline__ float ld_cluster_f1(uint32_t cluster_addr) {
+  float v;
+  asm volatile("ld.shared::cluster.f32 %0, [%1];" : "=f"(v) : "r"(cluster_addr) : "memory");
   return v;
 }
 __device__ __forceinline__ void cluster_sync_all() {

@@ -66,14 +66,48 @@ def qk_norm_cache(q, k, v, slot_mapping, cache, block_size: int, q_norm, k_norm,
 
 def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, scale: float, window: int, bias,
                      out_scale: float, out: torch.Tensor) -> None:
+    """bf16 prompts take the tensor-core kernel, bf16 single tokens the cache-streaming one; sizes those do not have,
+    and fp32, take the general kernel."""
     T, h, d = q.shape
     _packed_heads(q)
     assert out.stride(1) == 1
-    _check(lib().ksana_window_attention_any(
-        _ptr(q), q.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks, _ptr(meta.cu_q),
-        _ptr(meta.kv_lens), _ptr(meta.seq_of_token), h, kv_heads, d, vdim, block_size, window, float(scale), _ptr(bias),
-        bias.shape[1] if bias is not None else 0, float(out_scale), _ptr(out), out.stride(0), 0, T, _KIND[q.dtype],
-        _stream()), "window_attention_any")
+    n_pre, n_dec, pre_tokens = meta.num_prefill, meta.num_decode, meta.num_prefill_tokens
+    blen = bias.shape[1] if bias is not None else 0
+    sizes = (h, kv_heads, d, vdim, block_size, window, float(scale), _ptr(bias), blen, float(out_scale))
+
+    def general(first: int, count: int) -> None:
+        if count:
+            _check(lib().ksana_window_attention_any(
+                _ptr(q), q.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks, _ptr(meta.cu_q),
+                _ptr(meta.kv_lens), _ptr(meta.seq_of_token), *sizes, _ptr(out), out.stride(0), first, count,
+                _KIND[q.dtype], _stream()), "window_attention_any")
+
+    if q.dtype != torch.bfloat16:
+        return general(0, T)
+    cu = meta.cu_q_host
+    if n_pre:
+        max_q = int((cu[1:n_pre + 1] - cu[:n_pre]).max())
+        code = lib().ksana_window_prefill(_ptr(q), q.stride(0), T, _ptr(cache), cache.shape[0], _ptr(meta.block_tables),
+                                          meta.max_blocks, _ptr(meta.cu_q), _ptr(meta.kv_lens), *sizes, _ptr(out),
+                                          out.stride(0), 0, n_pre, max_q, _stream())
+        if code == -1:
+            general(0, pre_tokens)
+        else:
+            _check(code, "window_prefill")
+    if n_dec:
+        code = -1
+        if meta.num_decode_tokens == n_dec:
+            code = lib().ksana_window_decode(_ptr(q), q.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks,
+                                             _ptr(meta.cu_q), _ptr(meta.kv_lens), *sizes, _ptr(out), out.stride(0),
+                                             n_pre, n_dec, int(meta.kv_lens_host[n_pre:].max()), _stream())
+        if code == -1:
+            general(pre_tokens, T - pre_tokens)
+        else:
+            _check(code, "window_decode")
+
+
+# Prompt portions of more tokens than this go through the chunked form of linear attention.
+LINEAR_CHUNK_MIN_TOKENS = 16
 
 
 def linear_attention(q, k, v, state, meta, decay, act: str, rotary, key_scale: float) -> torch.Tensor:
@@ -84,14 +118,28 @@ def linear_attention(q, k, v, state, meta, decay, act: str, rotary, key_scale: f
     out = torch.empty(T, h, dv, dtype=q.dtype, device=q.device)
     rd = rotary.shape[1] if rotary is not None else 0
     n_pre, n_dec = meta.num_prefill, meta.num_decode
+    head = (_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(state), _ptr(meta.state_slots),
+            _ptr(meta.cu_q), _ptr(meta.kv_lens), _ptr(meta.positions), _ptr(decay), _ptr(rotary), rd,
+            1 if act == "silu" else 0, float(key_scale), h, d, dv, _ptr(out))
+    n_long = 0
+    if n_pre and q.dtype == torch.bfloat16:
+        lens = meta.cu_q_host[1:n_pre + 1] - meta.cu_q_host[:n_pre]
+        long = (lens > LINEAR_CHUNK_MIN_TOKENS).nonzero()[0]
+        n_long = int(long[-1]) + 1 if len(long) else 0  # a step lists its prompt portions longest first
+        if n_long:
+            tokens = int(meta.cu_q_host[n_long])
+            scratch = torch.empty(lib().ksana_linear_chunk_scratch(tokens, n_long, h, d, dv), dtype=torch.float32,
+                                  device=q.device)
+            code = lib().ksana_linear_chunked(*head, 0, n_long, int(lens[:n_long].max()), _ptr(scratch), _stream())
+            if code == -1:
+                n_long = 0
+            else:
+                _check(code, "linear_chunked")
     one = n_dec > 0 and meta.num_decode_tokens == n_dec
-    for base, count, single in ((0, n_pre, 0), (n_pre, n_dec, 1 if one else 0)):
+    for base, count, single in ((n_long, n_pre - n_long, 0), (n_pre, n_dec, 1 if one else 0)):
         if count:
-            _check(lib().ksana_linear_recurrent(
-                _ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(state), _ptr(meta.state_slots),
-                _ptr(meta.cu_q), _ptr(meta.kv_lens), _ptr(meta.positions), _ptr(decay), _ptr(rotary), rd,
-                1 if act == "silu" else 0, float(key_scale), h, d, dv, _ptr(out), base, count, single, _KIND[q.dtype],
-                _stream()), "linear_recurrent")
+            _check(lib().ksana_linear_recurrent(*head, base, count, single, _KIND[q.dtype], _stream()),
+                   "linear_recurrent")
     return out
 
 
