@@ -11,6 +11,11 @@ each case is small (at most a few GB on the device) and launches its kernel a ha
     python benchmarks/kernel_cases.py mla [B ctx h q_len]     # tcgen05 absorbed-MLA decode over the latent cache
     python benchmarks/kernel_cases.py rmsnorm [T H]
     python benchmarks/kernel_cases.py moe [T E k H I]
+    python benchmarks/kernel_cases.py window_prefill [T h hk d dv window]   # layers with mixers of their own sizes
+    python benchmarks/kernel_cases.py window_decode [B ctx h hk d dv window]
+    python benchmarks/kernel_cases.py linear_prefill [T h d dv rotary]
+    python benchmarks/kernel_cases.py linear_decode [B h d dv rotary]
+    python benchmarks/kernel_cases.py mixer_rows [T H h hk d]
     python benchmarks/kernel_cases.py all
 """
 import json
@@ -21,7 +26,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 from ksanallm_b200.engine.step_input import make_step_input  # noqa: E402
-from ksanallm_b200.ops import cuda, cuda_moe  # noqa: E402
+from ksanallm_b200.ops import cuda, cuda_mixer, cuda_moe  # noqa: E402
 from ksanallm_b200.ops import reference as ref  # noqa: E402
 
 DEV = "cuda"
@@ -190,8 +195,119 @@ def case_moe():
                 tflops=round(fl / us / 1e6, 1), frac_of_measured_bf16=round(fl / us / 1e6 / p["bf16_tflops"], 3))
 
 
+def _window_setup(q_lens, kv_lens, h, hk, d, dv, window, prefill):
+    q, _, bt, cu = _attn_setup(q_lens, kv_lens, h, 1)
+    q = (torch.randn(cu[-1], h, d, device=DEV) * 0.3).to(torch.bfloat16)
+    cache = (torch.randn(int(bt.max()) + 2, hk * 16 * (d + dv), device=DEV) * 0.3).to(torch.bfloat16)
+    T = cu[-1]
+    meta = make_step_input([0] * T, [0] * T, [0] * T, cu, kv_lens, bt, num_prefill=prefill, device=DEV)
+    bias = torch.randn(h, window or max(kv_lens), device=DEV)
+    out = torch.empty(T, h * dv, dtype=torch.bfloat16, device=DEV)
+    return lambda i: cuda_mixer.window_attention(q, cache, meta, 16, hk, dv, d ** -0.5, window, bias, 1.0, out)
+
+
+def case_window_prefill():
+    T, h, hk, d, dv, window = args_or([8192, 32, 8, 128, 128, 1024])
+    us = timeit(_window_setup([T], [T], h, hk, d, dv, window, 1), iters=5)
+    w = min(window or T, T)
+    pairs = w * (w + 1) / 2 + (T - w) * w
+    fl = 2.0 * h * (d + dv) * pairs
+    p = peaks()
+    return dict(kernel="window_prefill", T=T, h=h, hk=hk, d=d, dv=dv, window=window, us=round(us, 1),
+                tflops=round(fl / us / 1e6, 1), frac_of_measured_bf16=round(fl / us / 1e6 / p["bf16_tflops"], 3))
+
+
+def case_window_decode():
+    B, ctx, h, hk, d, dv, window = args_or([128, 4096, 32, 8, 128, 128, 1024])
+    us = timeit(_window_setup([1] * B, [ctx] * B, h, hk, d, dv, window, 0))
+    by = B * min(window or ctx, ctx) * hk * (d + dv) * 2
+    p = peaks()
+    return dict(kernel="window_decode", B=B, ctx=ctx, h=h, hk=hk, d=d, dv=dv, window=window, us=round(us, 1),
+                kv_gb=round(by / 1e9, 3), gbs=round(by / us / 1e3, 1),
+                frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+
+
+def _linear_setup(lens, q_lens, h, d, dv, rotary, prefill, copies=1):
+    B, T = len(lens), sum(q_lens)
+    cu = [0]
+    for q in q_lens:
+        cu.append(cu[-1] + q)
+    pos = [n - q + i for n, q in zip(lens, q_lens) for i in range(q)]
+    meta = make_step_input([0] * T, pos, [0] * T, cu, lens, torch.zeros(B, 1), num_prefill=prefill, device=DEV,
+                           state_slots=list(range(B)))
+    width = h * (2 * d + dv)
+    xs = [(torch.randn(T, width, device=DEV) * 0.3).to(torch.bfloat16) for _ in range(copies)]
+    states = [torch.zeros(B, h, d, dv, device=DEV) for _ in range(copies)]
+    decay = torch.full((h,), 0.99, device=DEV)
+    table = ref.rotary_table(d, 1e4, max(lens), DEV) if rotary else None
+
+    def run(i):
+        x = xs[i % copies]
+        q, k, v = x[:, :h * d], x[:, h * d:2 * h * d], x[:, 2 * h * d:]
+        cuda_mixer.linear_attention(q.unflatten(1, (h, d)), k.unflatten(1, (h, d)), v.unflatten(1, (h, dv)),
+                                    states[i % copies], meta, decay, "none" if rotary else "silu", table, 0.1)
+    return run
+
+
+def case_linear_prefill():
+    T, h, d, dv, rotary = args_or([8192, 32, 128, 128, 1])
+    us = timeit(_linear_setup([T], [T], h, d, dv, rotary, 1, 2), iters=5)
+    by = T * h * (2 * d + 2 * dv) * 2
+    fl = T * h * (2.0 * d * dv * 2 + 128 * (d + dv))  # state update and read-out + the causal half of a chunk of 128
+    p = peaks()
+    floor = max(by / p["hbm_gbs"] / 1e3, fl / p["bf16_tflops"] / 1e6)
+    return dict(kernel="linear_chunked", T=T, h=h, d=d, dv=dv, rotary=rotary, us=round(us, 1),
+                roofline_us=round(floor, 1), frac_of_roofline=round(floor / us, 3))
+
+
+def case_linear_decode():
+    B, h, d, dv, rotary = args_or([128, 32, 128, 128, 1])
+    us = timeit(_linear_setup([100] * B, [1] * B, h, d, dv, rotary, 0, 2))
+    by = 2 * B * h * d * dv * 4
+    p = peaks()
+    return dict(kernel="linear_recurrent", B=B, h=h, d=d, dv=dv, rotary=rotary, us=round(us, 1),
+                state_gb=round(by / 2e9, 3), gbs=round(by / us / 1e3, 1),
+                frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+
+
+def case_mixer_rows():
+    """The row-wise kernels, each beside its counterpart of the dense models."""
+    T, H, h, hk, d = args_or([8192, 4096, 32, 8, 128])
+    bf = lambda *s: torch.randn(*s, device=DEV).to(torch.bfloat16)  # noqa: E731
+    p, out = peaks(), {}
+
+    def add(name, us, by):
+        out[name] = dict(us=round(us, 1), gbs=round(by / us / 1e3, 1), frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+
+    xs, w = [bf(T, H) for _ in range(3)], torch.ones(H, device=DEV, dtype=torch.bfloat16)
+    r32, r16 = [torch.randn(T, H, device=DEV) for _ in range(3)], [bf(T, H) for _ in range(3)]
+    add("layer_norm", timeit(lambda i: cuda_mixer.layer_norm(xs[i % 3], w, None, 1e-6, r32[i % 3], torch.bfloat16)), T * H * 12)
+    add("rms_norm", timeit(lambda i: cuda.rms_norm(xs[i % 3], w, 1e-6, r16[i % 3])), T * H * 8)
+    us = [bf(T, 6 * H) for _ in range(2)]
+    add("gelu_mul", timeit(lambda i: cuda_mixer.gelu_and_mul(us[i % 2])), T * H * 18)
+    add("silu_mul", timeit(lambda i: cuda.silu_and_mul(us[i % 2])), T * H * 18)
+    o, g, y = bf(T, h, d), bf(T, 2 * h * d), torch.empty(T, h * d, device=DEV, dtype=torch.bfloat16)
+    gs = [g, g.clone()]
+    add("gated_head_norm", timeit(lambda i: cuda_mixer.gated_norm(o, gs[i % 2][:, :h * d], None, 1e-6, "silu", 1.1, y)), T * h * d * 6)
+    wn = torch.ones(h * d, device=DEV)
+    add("gated_row_norm", timeit(lambda i: cuda_mixer.gated_norm(o, gs[i % 2][:, :h * d], wn, 1e-6, "sigmoid", 1.0, y)), T * h * d * 6)
+    slots = torch.arange(T, dtype=torch.int32, device=DEV)
+    cache = torch.zeros((T + 15) // 16, 2, hk, 16, d, dtype=torch.bfloat16, device=DEV)
+    qkv = [bf(T, (h + 2 * hk) * d) for _ in range(3)]
+    wf, wb = torch.ones(d, device=DEV), torch.ones(d, device=DEV, dtype=torch.bfloat16)
+
+    def parts(x):
+        return x[:, :h * d].unflatten(1, (h, d)), x[:, h * d:(h + hk) * d].unflatten(1, (hk, d)), x[:, (h + hk) * d:].unflatten(1, (hk, d))
+    by = T * d * 2 * (2 * h + 4 * hk)
+    add("qk_norm_cache", timeit(lambda i: cuda_mixer.qk_norm_cache(*parts(qkv[i % 3]), slots, cache.view(cache.shape[0], -1), 16, wf, wf, 1e-6)), by)
+    table = torch.randn(T, d, device=DEV)
+    add("rope_cache", timeit(lambda i: cuda.rope_qknorm_cache(*parts(qkv[i % 3]), slots, table, slots, cache, wb, wb, 1e-6)), by)
+    return dict(kernel="mixer_rows", T=T, H=H, h=h, hk=hk, d=d, **out)
+
+
 CASES = dict(gemm=case_gemm, gemm_fp8=case_gemm_fp8, gemm_int4=case_gemm_int4, decode=case_decode, prefill=case_prefill, mla=case_mla, rmsnorm=case_rmsnorm,
-             moe=case_moe)
+             moe=case_moe, window_prefill=case_window_prefill, window_decode=case_window_decode,
+             linear_prefill=case_linear_prefill, linear_decode=case_linear_decode, mixer_rows=case_mixer_rows)
 
 if __name__ == "__main__":
     which = sys.argv[1] if len(sys.argv) > 1 else "all"

@@ -26,7 +26,8 @@ struct LinearAttnArgs {
 
 template <typename T>
 __device__ __forceinline__ float la_act(float x, int act) {
-  return act ? silu_f(x) : x;
+  if (!act) return x;
+  return sizeof(T) == 2 ? silu_fast(x) : silu_f(x);
 }
 
 // Element c of a head of q or k after activation and rotation.
@@ -75,6 +76,18 @@ linear_recurrent_kernel(LinearAttnArgs a, int seq_base) {
       store_n<VEC>(sS + r * 32 + tx * VEC, s);
     }
   }
+  // the single token's share of the state is requested before anything else (up to RMAX rows per thread)
+  constexpr int RMAX = ONE ? 8 : 1;
+  float pre[RMAX][VEC];
+  if (ONE && live) {
+#pragma unroll
+    for (int i = 0; i < RMAX; ++i) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) pre[i][j] = 0.f;
+      const int r = ty + i * TY;
+      if (r < a.d && !fresh) load_n<VEC>(S + static_cast<size_t>(r) * a.dv, pre[i]);
+    }
+  }
   for (int t = t0; t < t1; ++t) {
     const T* q = static_cast<const T*>(a.q) + static_cast<size_t>(t) * a.ldq + head * a.d;
     const T* k = static_cast<const T*>(a.k) + static_cast<size_t>(t) * a.ldk + head * a.d;
@@ -93,8 +106,23 @@ linear_recurrent_kernel(LinearAttnArgs a, int seq_base) {
       float vv[VEC];
 #pragma unroll
       for (int j = 0; j < VEC; ++j) vv[j] = sv[tx * VEC + j];
-#pragma unroll 8
-      for (int r = ty; r < a.d; r += TY) {
+      if (ONE) {
+#pragma unroll
+        for (int i = 0; i < RMAX; ++i) {
+          const int r = ty + i * TY;
+          if (r < a.d) {
+            const float kr = sk[r], qr = sq[r];
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) {
+              pre[i][j] = dec * pre[i][j] + kr * vv[j];
+              acc[j] += qr * pre[i][j];
+            }
+            store_n<VEC>(S + static_cast<size_t>(r) * a.dv, pre[i]);
+          }
+        }
+      }
+#pragma unroll 4
+      for (int r = ty + (ONE ? RMAX * TY : 0); r < a.d; r += TY) {
         float s[VEC];
         if (ONE) {
 #pragma unroll
@@ -154,29 +182,6 @@ __device__ __forceinline__ float decay_pow(float decay, int e) {
   return decay > 0.f ? exp2f(static_cast<float>(e) * log2f(decay)) : 0.f;
 }
 
-// Eight consecutive features of a head of q or k after activation and rotation (c0 % 8 == 0; rd % 16 == 0).
-__device__ __forceinline__ void la_feature8(const __nv_bfloat16* head, int c0, const float* cs, int rd, int act, float* f) {
-  load_n<8>(head + c0, f);
-  if (act) {
-#pragma unroll
-    for (int i = 0; i < 8; ++i) f[i] = silu_f(f[i]);
-  }
-  if (c0 < rd) {
-    const int half = rd >> 1;
-    const bool low = c0 < half;
-    const int i0 = low ? c0 : c0 - half;
-    float y[8], co[8], si[8];
-    load_n<8>(head + (low ? c0 + half : i0), y);
-    load_n<8>(cs + i0, co);
-    load_n<8>(cs + half + i0, si);
-#pragma unroll
-    for (int i = 0; i < 8; ++i) {
-      const float z = act ? silu_f(y[i]) : y[i];
-      f[i] = low ? f[i] * co[i] - z * si[i] : f[i] * co[i] + z * si[i];
-    }
-  }
-}
-
 // Row r, 8 features from c0 of a 128-row operand in the 128-byte swizzle (64-column panels of 16 KB).
 __device__ __forceinline__ uint4* operand_at(uint8_t* base, int r, int c0) {
   return reinterpret_cast<uint4*>(base + (c0 >> 6) * (128 * 128) + r * 128 + ((((c0 >> 3) & 7) ^ (r & 7)) << 4));
@@ -189,49 +194,68 @@ __device__ __forceinline__ void store_split8(uint8_t* hi, uint8_t* lo, int r, in
   *operand_at(lo, r, c0) = make_uint4(l[0], l[1], l[2], l[3]);
 }
 
-// n valid rows of q or k (scaled per row by rs[r], if given), zero elsewhere, as hi + lo operands of DK columns.
-template <int DK>
-__device__ __forceinline__ void stage_features(const LinearAttnArgs& a, const void* src, int ld, int head, int t0, int n,
-                                               float scale, const float* rs, uint8_t* hi, uint8_t* lo) {
-  for (int u = threadIdx.x; u < 128 * (DK / 8); u += 256) {
-    const int r = u / (DK / 8), c0 = (u % (DK / 8)) * 8;
-    float f[8];
-#pragma unroll
-    for (int i = 0; i < 8; ++i) f[i] = 0.f;
-    if (r < n && c0 < a.d) {
-      const int t = t0 + r;
-      const __nv_bfloat16* p = static_cast<const __nv_bfloat16*>(src) + static_cast<size_t>(t) * ld + head * a.d;
-      const float* cs = a.rotary ? a.rotary + static_cast<size_t>(a.positions[t]) * a.rd : nullptr;
-      la_feature8(p, c0, cs, a.rd, a.act, f);
-      const float m = rs ? scale * rs[r] : scale;
-#pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] *= m;
-    }
-    store_split8(hi, lo, r, c0, f);
-  }
+// Features of a head are handled in slots of 16: slot u < rd / 16 holds the 8 dimensions from 8 u and their rotation
+// partners half a rotation further, the others 16 consecutive ones. First dimension of each half of the slot:
+__device__ __forceinline__ void slot_dims(int u, int rd, int* lo, int* hi) {
+  const bool rot = u * 16 < rd;
+  *lo = rot ? u * 8 : u * 16;
+  *hi = rot ? *lo + (rd >> 1) : *lo + 8;
 }
 
-// n valid rows of v, columns [col0, col0 + DVT), zero elsewhere: one bf16 operand.
-template <int DVT>
-__device__ __forceinline__ void stage_values(const LinearAttnArgs& a, int head, int col0, int t0, int n, uint8_t* dst) {
-  for (int u = threadIdx.x; u < 128 * (DVT / 8); u += 256) {
-    const int r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
-    uint4 w = make_uint4(0, 0, 0, 0);
-    if (r < n && col0 + c0 < a.dv) {
-      const __nv_bfloat16* p =
-          static_cast<const __nv_bfloat16*>(a.v) + static_cast<size_t>(t0 + r) * a.ldv + head * a.dv + col0 + c0;
-      if (a.act) {
-        float f[8];
-        load_n<8>(p, f);
+// cos and sin of a slot's 8 pairs.
+struct SlotAngles {
+  float4 c[2], s[2];
+};
+__device__ __forceinline__ void load_angles(const LinearAttnArgs& a, int pos, int lo, SlotAngles* x) {
+  const float4* p = reinterpret_cast<const float4*>(a.rotary + static_cast<size_t>(pos) * a.rd + lo);
+  const float4* q = p + (a.rd >> 3);
+  x->c[0] = p[0]; x->c[1] = p[1];
+  x->s[0] = q[0]; x->s[1] = q[1];
+}
+
+// Activation, rotation and scale of one slot, then its hi and lo parts go to row r of the operands.
+__device__ __forceinline__ void finish_slot(uint4 w_lo, uint4 w_hi, bool rot, const SlotAngles& an, int act, float scale,
+                                            uint8_t* hi, uint8_t* lo, int r, int c_lo, int c_hi) {
+  float x[8], y[8];
+  unpack8(w_lo, x);
+  unpack8(w_hi, y);
+  if (act) {
 #pragma unroll
-        for (int i = 0; i < 8; ++i) f[i] = silu_f(f[i]);
-        w = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
-      } else {
-        w = *reinterpret_cast<const uint4*>(p);
-      }
+    for (int i = 0; i < 8; ++i) {
+      x[i] = silu_fast(x[i]);
+      y[i] = silu_fast(y[i]);
     }
-    *operand_at(dst, r, c0) = w;
   }
+  if (rot) {
+    const float* c = reinterpret_cast<const float*>(an.c);
+    const float* s = reinterpret_cast<const float*>(an.s);
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+      const float u = x[i] * c[i] - y[i] * s[i];
+      y[i] = y[i] * c[i] + x[i] * s[i];
+      x[i] = u;
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 8; ++i) {
+    x[i] *= scale;
+    y[i] *= scale;
+  }
+  store_split8(hi, lo, r, c_lo, x);
+  store_split8(hi, lo, r, c_hi, y);
+}
+
+__device__ __forceinline__ uint4 value_word(uint4 w, int act) {
+  if (!act) return w;
+  float f[8];
+  unpack8(w, f);
+#pragma unroll
+  for (int i = 0; i < 8; ++i) f[i] = silu_fast(f[i]);
+  return make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+}
+
+__device__ __forceinline__ const __nv_bfloat16* head_row(const void* base, int t, int ld, int off) {
+  return static_cast<const __nv_bfloat16*>(base) + static_cast<size_t>(t) * ld + off;
 }
 
 // Launch 1: L = sum_j decay^(n - 1 - j) k_j v_j^T of one (chunk, head, DVT value columns) -> scratch [entry][h][d][dv].
@@ -268,8 +292,43 @@ linear_chunk_kv_kernel(LinearAttnArgs a, int seq_base, int tiles, float* __restr
   __syncthreads();
   tc_fence_after();
   const uint32_t tmem = *holder;
-  stage_features<128>(a, a.k, a.ldk, head, t0, n, a.key_scale, rs, k_hi, k_lo);
-  stage_values<DVT>(a, head, col0, t0, n, sv);
+  const int pos0 = a.kv_lens[b] - (a.cu_q[b + 1] - t0);
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+  constexpr int UV = 128 * (DVT / 8) / 256;
+  uint4 vw[UV];
+#pragma unroll
+  for (int i = 0; i < UV; ++i) {
+    const int u = i * 256 + tid, r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
+    vw[i] = r < n && col0 + c0 < a.dv
+                ? *reinterpret_cast<const uint4*>(head_row(a.v, t0 + r, a.ldv, head * a.dv + col0 + c0)) : zero;
+  }
+#pragma unroll
+  for (int g = 0; g < 2; ++g) {
+    uint4 wl[2], wh[2];
+    SlotAngles an[2];
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int u = (g * 2 + i) * 256 + tid, r = u / 8, sl = u % 8;
+      int cl, ch;
+      slot_dims(sl, a.rd, &cl, &ch);
+      const __nv_bfloat16* p = head_row(a.k, t0 + r, a.ldk, head * a.d);
+      wl[i] = r < n && cl < a.d ? *reinterpret_cast<const uint4*>(p + cl) : zero;
+      wh[i] = r < n && ch < a.d ? *reinterpret_cast<const uint4*>(p + ch) : zero;
+      if (r < n && sl * 16 < a.rd) load_angles(a, pos0 + r, cl, &an[i]);
+    }
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const int u = (g * 2 + i) * 256 + tid, r = u / 8, sl = u % 8;
+      int cl, ch;
+      slot_dims(sl, a.rd, &cl, &ch);
+      finish_slot(wl[i], wh[i], r < n && sl * 16 < a.rd, an[i], a.act, a.key_scale * rs[r], k_hi, k_lo, r, cl, ch);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < UV; ++i) {
+    const int u = i * 256 + tid, r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
+    *operand_at(sv, r, c0) = value_word(vw[i], a.act);
+  }
   fence_async_smem();
   __syncthreads();
   if (tid == 0) {
@@ -348,8 +407,8 @@ struct ChunkOutSmem {
   static_assert(USED + 960 <= 232448, "does not fit");
 };
 
-template <int DK, int DVT>
-__global__ void __launch_bounds__(256)
+template <int DK, int DVT, int NT>
+__global__ void __launch_bounds__(NT)
 linear_chunk_out_kernel(LinearAttnArgs a, int seq_base, int tiles, const float* __restrict__ scratch, unsigned int* err) {
   using M_ = ChunkOutSmem<DK, DVT>;
   extern __shared__ uint8_t smem_raw[];
@@ -374,6 +433,33 @@ linear_chunk_out_kernel(LinearAttnArgs a, int seq_base, int tiles, const float* 
   volatile int* abort_flag = reinterpret_cast<volatile int*>(holder + 1);
   constexpr uint32_t COLS = 128 + 2 * DVT <= 256 ? 256 : 512;
   const int tid = threadIdx.x, warp = tid >> 5;
+  const uint4 zero = make_uint4(0, 0, 0, 0);
+
+  // ---- q, k and v: everything is requested before anything is used ----
+  constexpr int UQ = 128 * (DK / 16) / NT, UV = 128 * (DVT / 8) / NT, US = DK * (DVT / 8) / NT;
+  const int pos0 = a.kv_lens[b] - q_len + c * LC;
+  uint4 ql[UQ], qh[UQ], kl[UQ], kh[UQ], vw[UV];
+  SlotAngles an[UQ];
+#pragma unroll
+  for (int i = 0; i < UQ; ++i) {
+    const int u = i * NT + tid, r = u / (DK / 16), sl = u % (DK / 16);
+    int cl, ch;
+    slot_dims(sl, a.rd, &cl, &ch);
+    const __nv_bfloat16* q = head_row(a.q, t0 + r, a.ldq, head * a.d);
+    const __nv_bfloat16* k = head_row(a.k, t0 + r, a.ldk, head * a.d);
+    const bool in_lo = r < n && cl < a.d, in_hi = r < n && ch < a.d;
+    ql[i] = in_lo ? *reinterpret_cast<const uint4*>(q + cl) : zero;
+    qh[i] = in_hi ? *reinterpret_cast<const uint4*>(q + ch) : zero;
+    kl[i] = in_lo ? *reinterpret_cast<const uint4*>(k + cl) : zero;
+    kh[i] = in_hi ? *reinterpret_cast<const uint4*>(k + ch) : zero;
+    if (r < n && sl * 16 < a.rd) load_angles(a, pos0 + r, cl, &an[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < UV; ++i) {
+    const int u = i * NT + tid, r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
+    vw[i] = r < n && col0 + c0 < a.dv
+                ? *reinterpret_cast<const uint4*>(head_row(a.v, t0 + r, a.ldv, head * a.dv + col0 + c0)) : zero;
+  }
   if (tid == 0) {
     for (int i = 0; i < 3; ++i) mbar_init(&bar[i], 1);
     *abort_flag = 0;
@@ -383,9 +469,31 @@ linear_chunk_out_kernel(LinearAttnArgs a, int seq_base, int tiles, const float* 
     tmem_alloc(holder, COLS);
     tmem_relinquish();
   }
-  tab[tid] = tid >= 127 ? decay_pow(a.decay[head], tid - 127) : 0.f;
-  stage_features<DK>(a, a.q, a.ldq, head, t0, n, 1.f, nullptr, q_hi, q_lo);
-  stage_features<DK>(a, a.k, a.ldk, head, t0, n, a.key_scale, nullptr, k_hi, k_lo);
+  if (tid < 256) tab[tid] = tid >= 127 ? decay_pow(a.decay[head], tid - 127) : 0.f;
+#pragma unroll
+  for (int i = 0; i < UQ; ++i) {
+    const int u = i * NT + tid, r = u / (DK / 16), sl = u % (DK / 16);
+    int cl, ch;
+    slot_dims(sl, a.rd, &cl, &ch);
+    const bool rot = r < n && sl * 16 < a.rd;
+    finish_slot(ql[i], qh[i], rot, an[i], a.act, 1.f, q_hi, q_lo, r, cl, ch);
+    finish_slot(kl[i], kh[i], rot, an[i], a.act, a.key_scale, k_hi, k_lo, r, cl, ch);
+  }
+  // the state entering the chunk (fp32) is on its way while the scores are multiplied
+  float4 sw[US][2];
+  if (has_state) {
+    const float* src = scratch + (chunk_entry(a, seq_base, b, c) * a.h + head) * a.d * a.dv + col0;
+#pragma unroll
+    for (int i = 0; i < US; ++i) {
+      const int u = i * NT + tid, r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
+      sw[i][0] = sw[i][1] = make_float4(0.f, 0.f, 0.f, 0.f);
+      if (r < a.d && col0 + c0 < a.dv) {
+        const float4* p = reinterpret_cast<const float4*>(src + static_cast<size_t>(r) * a.dv + c0);
+        sw[i][0] = p[0];
+        sw[i][1] = p[1];
+      }
+    }
+  }
   fence_async_smem();
   tc_fence_before();
   __syncthreads();
@@ -404,19 +512,20 @@ linear_chunk_out_kernel(LinearAttnArgs a, int seq_base, int tiles, const float* 
       }
     umma_commit(&bar[0]);
   }
-  stage_values<DVT>(a, head, col0, t0, n, sv);
+#pragma unroll
+  for (int i = 0; i < UV; ++i) {
+    const int u = i * NT + tid, r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
+    *operand_at(sv, r, c0) = value_word(vw[i], a.act);
+  }
   if (has_state) {
     // state rows: panels of 64 columns, DK rows each
-    const float* src = scratch + (chunk_entry(a, seq_base, b, c) * a.h + head) * a.d * a.dv + col0;
-    for (int u = tid; u < DK * (DVT / 8); u += 256) {
-      const int r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
-      float f[8];
 #pragma unroll
-      for (int i = 0; i < 8; ++i) f[i] = 0.f;
-      if (r < a.d && col0 + c0 < a.dv) load_n<8>(src + static_cast<size_t>(r) * a.dv + c0, f);
+    for (int i = 0; i < US; ++i) {
+      const int u = i * NT + tid, r = u / (DVT / 8), c0 = (u % (DVT / 8)) * 8;
+      const float* f = reinterpret_cast<const float*>(sw[i]);
       uint32_t h[4], l[4];
 #pragma unroll
-      for (int i = 0; i < 4; ++i) h[i] = split_bf16(f[2 * i], f[2 * i + 1], &l[i]);
+      for (int j = 0; j < 4; ++j) h[j] = split_bf16(f[2 * j], f[2 * j + 1], &l[j]);
       const int off = (c0 >> 6) * (DK * 128) + r * 128 + ((((c0 >> 3) & 7) ^ (r & 7)) << 4);
       *reinterpret_cast<uint4*>(s_hi + off) = make_uint4(h[0], h[1], h[2], h[3]);
       *reinterpret_cast<uint4*>(s_lo + off) = make_uint4(l[0], l[1], l[2], l[3]);
@@ -434,30 +543,36 @@ linear_chunk_out_kernel(LinearAttnArgs a, int seq_base, int tiles, const float* 
                  umma_desc_mn128(smem_u32(p == 2 ? s_lo : s_hi) + k * (16 * 128), DK * 128), idesc, (p || k) ? 1u : 0u);
     umma_commit(&bar[1]);
   }
-  // scores -> decayed, causal weights, written over them as two bf16 matrices. A warp and the one four further on share
-  // 32 rows; each takes half of the columns.
+  // scores -> decayed, causal weights, written over them as two bf16 matrices. The warps whose numbers agree modulo 4
+  // share 32 rows; each takes its part of the columns.
+  constexpr int PARTS = NT / 128, PC = 128 / PARTS;
   const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
-  const int row = (warp & 3) * 32 + (tid & 31), half = warp >> 2;
+  const int row = (warp & 3) * 32 + (tid & 31), part = warp >> 2;
   int bad = !mbar_wait_bounded(&bar[0], 0, abort_flag, err);
   bad = __any_sync(0xffffffffu, bad);
-  uint32_t s[64];
+  uint32_t s[PC];
   if (!bad) {
     tc_fence_after();
-    tmem_ld32(tmem + lane_off + half * 64, s);
-    tmem_ld32(tmem + lane_off + half * 64 + 32, s + 32);
+#pragma unroll
+    for (int q = 0; q < PC / 32; ++q) tmem_ld32(tmem + lane_off + part * PC + q * 32, s + q * 32);
     tmem_wait_ld();
   }
-  if (__syncthreads_or(bad)) bad = 1;  // both halves of a row have been read
+  if (__syncthreads_or(bad)) bad = 1;  // every part of a row has been read
   if (!bad) {
-    uint32_t hi[32], lo[32];
+    uint32_t hi[PC / 2], lo[PC / 2];
 #pragma unroll
-    for (int j = 0; j < 32; ++j) {
-      const int c0 = half * 64 + 2 * j;
+    for (int j = 0; j < PC / 2; ++j) {
+      const int c0 = part * PC + 2 * j;
       hi[j] = split_bf16(__uint_as_float(s[2 * j]) * tab[row - c0 + 127],
                          __uint_as_float(s[2 * j + 1]) * tab[row - c0 + 126], &lo[j]);
     }
-    tmem_st32(tmem + lane_off + half * 32, hi);
-    tmem_st32(tmem + lane_off + 64 + half * 32, lo);
+    if constexpr (PC == 64) {
+      tmem_st32(tmem + lane_off + part * 32, hi);
+      tmem_st32(tmem + lane_off + 64 + part * 32, lo);
+    } else {
+      tmem_st16(tmem + lane_off + part * 16, hi);
+      tmem_st16(tmem + lane_off + 64 + part * 16, lo);
+    }
     tmem_wait_st();
   }
   tc_fence_before();
@@ -479,15 +594,16 @@ linear_chunk_out_kernel(LinearAttnArgs a, int seq_base, int tiles, const float* 
   if (!bad) {
     tc_fence_after();
     const float f = tab[128 + row];  // decay^(row + 1)
+    constexpr int OC = DVT / PARTS;  // 16, 32 or 64 output columns per thread
     __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + (static_cast<size_t>(t0 + row) * a.h + head) * a.dv + col0;
 #pragma unroll 1
-    for (int cc = half * (DVT / 2); cc < (half + 1) * (DVT / 2); cc += 32) {
-      uint32_t x[32], y[32];
-      tmem_ld32(tm_own + lane_off + cc, x);
-      if (has_state) tmem_ld32(tm_state + lane_off + cc, y);
+    for (int cc = part * OC; cc < (part + 1) * OC; cc += 16) {
+      uint32_t x[16], y[16];
+      tmem_ld16(tm_own + lane_off + cc, x);
+      if (has_state) tmem_ld16(tm_state + lane_off + cc, y);
       tmem_wait_ld();
 #pragma unroll
-      for (int j = 0; j < 32; j += 8) {
+      for (int j = 0; j < 16; j += 8) {
         float v[8];
 #pragma unroll
         for (int u = 0; u < 8; ++u) {
@@ -519,9 +635,10 @@ template <int DK, int DVT>
 static int launch_chunk_out(const LinearAttnArgs& a, int seq_base, int num_seqs, int max_q, const float* scratch,
                             cudaStream_t st) {
   const int tiles = (a.dv + DVT - 1) / DVT;
-  auto kern = linear_chunk_out_kernel<DK, DVT>;
+  constexpr int NT = DK == 64 && DVT == 64 ? 256 : 512;  // two CTAs per SM fit the smallest size only
+  auto kern = linear_chunk_out_kernel<DK, DVT, NT>;
   if (KSANA_SMEM_ONCE(kern, (ChunkOutSmem<DK, DVT>::TOTAL)) != 0) return -4;
-  kern<<<dim3((max_q + LC - 1) / LC, a.h * tiles, num_seqs), 256, ChunkOutSmem<DK, DVT>::TOTAL, st>>>(
+  kern<<<dim3((max_q + LC - 1) / LC, a.h * tiles, num_seqs), NT, ChunkOutSmem<DK, DVT>::TOTAL, st>>>(
       a, seq_base, tiles, scratch, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }

@@ -32,6 +32,15 @@ __device__ __forceinline__ void load_n(const float* p, float* f) {
     }
   }
 }
+// eight bf16 of one 16-byte word
+__device__ __forceinline__ void unpack8(uint4 v, float* f) {
+  const uint32_t w[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+  for (int i = 0; i < 4; ++i) {
+    f[2 * i] = __uint_as_float(w[i] << 16);
+    f[2 * i + 1] = __uint_as_float(w[i] & 0xffff0000u);
+  }
+}
 template <int N>
 __device__ __forceinline__ void load_n(const __nv_bfloat16* p, float* f) {
   if constexpr (N == 1) {
@@ -42,14 +51,7 @@ __device__ __forceinline__ void load_n(const __nv_bfloat16* p, float* f) {
     float2 b = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&v.y));
     f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
   } else {
-    uint4 v = *reinterpret_cast<const uint4*>(p);
-    const uint32_t w[4] = {v.x, v.y, v.z, v.w};
-#pragma unroll
-    for (int i = 0; i < 4; ++i) {
-      uint32_t u = w[i];
-      float2 a = __bfloat1622float2(*reinterpret_cast<__nv_bfloat162*>(&u));
-      f[2 * i] = a.x; f[2 * i + 1] = a.y;
-    }
+    unpack8(*reinterpret_cast<const uint4*>(p), f);
   }
 }
 template <int N>
@@ -75,6 +77,8 @@ __device__ __forceinline__ void store_n(__nv_bfloat16* p, const float* f) {
 
 __device__ __forceinline__ float sigmoid_f(float x) { return 1.f / (1.f + expf(-x)); }
 __device__ __forceinline__ float silu_f(float x) { return x / (1.f + expf(-x)); }
+// The same through the fast exponential and division (relative error about 1e-6): inputs and results here are 16-bit.
+__device__ __forceinline__ float silu_fast(float x) { return __fdividef(x, 1.f + __expf(-x)); }
 // 0.5 z (1 + tanh u) with u = sqrt(2 / pi) (z + 0.044715 z^3)
 __device__ __forceinline__ float gelu_tanh_f(float z) {
   const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);

@@ -204,32 +204,66 @@ qk_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ld
 }
 
 // ---- gated RMS norm behind linear attention -------------------------------------------------------------------------
-__device__ __forceinline__ float gate_f(float g, int kind) { return kind == 0 ? silu_f(g) : sigmoid_f(g); }
+template <typename T>
+__device__ __forceinline__ float gate_f(float g, int kind) {
+  if (sizeof(T) == 2) {
+    const float s = __fdividef(1.f, 1.f + __expf(-g));
+    return kind == 0 ? g * s : s;
+  }
+  return kind == 0 ? silu_f(g) : sigmoid_f(g);
+}
 
-// per head, no weight: one warp per (token, head)
-template <typename T, int N>
+// per head, no weight: a warp takes HEADS heads of a token at a time, up to 32 N columns each in registers
+template <typename T, int N, int HEADS>
 __global__ void __launch_bounds__(256)
 gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ g, int ldg, T* __restrict__ out, int ldo,
                        int tokens, int h, int dv, float eps, int gate, float out_scale) {
+  const int groups = (h + HEADS - 1) / HEADS;
   const long long unit = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
-  if (unit >= static_cast<long long>(tokens) * h) return;
-  const size_t t = unit / h;
-  const int hd = static_cast<int>(unit % h);
-  const T* src = o + unit * dv;
-  float f[N], gg[N], ss = 0.f;
-  for (int c = lane * N; c < dv; c += 32 * N) {
-    load_n<N>(src + c, f);
+  if (unit >= static_cast<long long>(tokens) * groups) return;
+  const size_t t = unit / groups;
+  const int h0 = static_cast<int>(unit % groups) * HEADS;
+  if (dv <= 32 * N) {
+    float f[HEADS][N], gg[HEADS][N];
+    const int c = lane * N;
 #pragma unroll
-    for (int j = 0; j < N; ++j) ss += f[j] * f[j];
+    for (int i = 0; i < HEADS; ++i) {
+#pragma unroll
+      for (int j = 0; j < N; ++j) f[i][j] = gg[i][j] = 0.f;
+      if (h0 + i < h && c < dv) {
+        load_n<N>(o + (t * h + h0 + i) * dv + c, f[i]);
+        load_n<N>(g + t * ldg + (h0 + i) * dv + c, gg[i]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < HEADS; ++i) {
+      float ss = 0.f;
+#pragma unroll
+      for (int j = 0; j < N; ++j) ss += f[i][j] * f[i][j];
+      const float inv = out_scale / sqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
+#pragma unroll
+      for (int j = 0; j < N; ++j) f[i][j] *= inv * gate_f<T>(gg[i][j], gate);
+      if (h0 + i < h && c < dv) store_n<N>(out + t * ldo + (h0 + i) * dv + c, f[i]);
+    }
+    return;
   }
-  const float inv = out_scale / sqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
-  for (int c = lane * N; c < dv; c += 32 * N) {
-    load_n<N>(src + c, f);
-    load_n<N>(g + t * ldg + hd * dv + c, gg);
+  for (int hd = h0; hd < min(h0 + HEADS, h); ++hd) {
+    const T* src = o + (t * h + hd) * dv;
+    float f[N], gg[N], ss = 0.f;
+    for (int c = lane * N; c < dv; c += 32 * N) {
+      load_n<N>(src + c, f);
 #pragma unroll
-    for (int j = 0; j < N; ++j) f[j] = f[j] * inv * gate_f(gg[j], gate);
-    store_n<N>(out + t * ldo + hd * dv + c, f);
+      for (int j = 0; j < N; ++j) ss += f[j] * f[j];
+    }
+    const float inv = out_scale / sqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
+    for (int c = lane * N; c < dv; c += 32 * N) {
+      load_n<N>(src + c, f);
+      load_n<N>(g + t * ldg + hd * dv + c, gg);
+#pragma unroll
+      for (int j = 0; j < N; ++j) f[j] *= inv * gate_f<T>(gg[j], gate);
+      store_n<N>(out + t * ldo + hd * dv + c, f);
+    }
   }
 }
 
@@ -251,7 +285,7 @@ gated_row_norm_kernel(const T* __restrict__ o, const T* __restrict__ g, int ldg,
     load_n<N>(o + t * width + c, f);
     load_n<N>(g + t * ldg + c, gg);
 #pragma unroll
-    for (int j = 0; j < N; ++j) f[j] = f[j] * inv * w[c + j] * gate_f(gg[j], gate);
+    for (int j = 0; j < N; ++j) f[j] = f[j] * inv * w[c + j] * gate_f<T>(gg[j], gate);
     store_n<N>(out + t * ldo + c, f);
   }
 }
@@ -342,19 +376,20 @@ KSANA_API int ksana_gated_norm(const void* o, const void* g, int ldg, const floa
   const int esz = kind ? 2 : 4;
   const int width = h * dv;
   const bool vec = !((dv | ldg | ldo) & 3) && aligned(o, 4 * esz) && aligned(g, 4 * esz) && aligned(out, 4 * esz);
-  const unsigned grid = static_cast<unsigned>((static_cast<long long>(tokens) * h + 7) / 8);
+  const bool wide = kind && !w && dv > 128 && !((dv | ldg | ldo) & 7) && aligned(o, 16) && aligned(g, 16) && aligned(out, 16);
+  const unsigned grid = static_cast<unsigned>((static_cast<long long>(tokens) * ((h + 3) / 4) + 7) / 8);
 #define KSANA_GN(T, N)                                                                                               \
   do {                                                                                                               \
     if (w)                                                                                                           \
       gated_row_norm_kernel<T, N><<<tokens, 256, 0, st>>>(static_cast<const T*>(o), static_cast<const T*>(g), ldg, w, \
                                                           static_cast<T*>(out), ldo, width, eps, gate, out_scale);   \
     else                                                                                                             \
-      gated_head_norm_kernel<T, N><<<grid, 256, 0, st>>>(static_cast<const T*>(o), static_cast<const T*>(g), ldg,    \
+      gated_head_norm_kernel<T, N, 4><<<grid, 256, 0, st>>>(static_cast<const T*>(o), static_cast<const T*>(g), ldg,    \
                                                          static_cast<T*>(out), ldo, tokens, h, dv, eps, gate,        \
                                                          out_scale);                                                 \
   } while (0)
   if (kind) {
-    if (vec) KSANA_GN(bf16, 4); else KSANA_GN(bf16, 1);
+    if (wide) KSANA_GN(bf16, 8); else if (vec) KSANA_GN(bf16, 4); else KSANA_GN(bf16, 1);
   } else {
     if (vec) KSANA_GN(float, 4); else KSANA_GN(float, 1);
   }
