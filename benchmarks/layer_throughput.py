@@ -1,0 +1,135 @@
+"""Prefill and decode throughput of Molopel at layer sizes of real models, each beside the dense model (Qwen3 blocks: QK
+norm, grouped-query attention, SwiGLU) of the same width, heads and depth whose feed-forward is as wide as makes the
+parameter counts equal. Random weights, bf16, one GPU; every number comes from ``LLMEngine.step()``.
+
+    python bench.py --throughput molopel
+
+prefill: prompts of 4096 tokens, 8192 tokens a step. decode: 128 sequences behind prompts of 1024 tokens, one token each
+per step. Weights and caches are larger than L2, so each step starts cold. CUDA events around the timed steps; the host
+clock around the same steps is given beside it.
+"""
+from __future__ import annotations
+
+import json
+import time
+
+import torch
+
+from ksanallm_b200.config.model_config import model_config_from_dict, molopel_config
+from ksanallm_b200.config.schema import parse_serving_config
+from ksanallm_b200.engine.llm_engine import LLMEngine
+from ksanallm_b200.engine.sampling_params import SamplingParams
+from ksanallm_b200.models.loader import load_model_weights
+from ksanallm_b200.models.transformer import TransformerModel
+from ksanallm_b200.ops import cuda
+
+# width, depth, feed-forward, heads, key / value heads, window
+SIZES = [(2048, 8, 6144, 16, 4, 1024), (4096, 8, 12288, 32, 8, 1024), (8192, 4, 24576, 64, 8, 2048)]
+PROMPT, STEP_TOKENS = 4096, 8192
+BATCH, CONTEXT, DECODE_STEPS = 128, 1024, 40
+
+
+def parameters(weights) -> int:
+    return sum(w.numel() for k, w in weights.items() if k.startswith("model.layers."))
+
+
+def dense_config(width, depth, ff, heads, kv_heads):
+    return model_config_from_dict(dict(
+        model_type="qwen3", hidden_size=width, num_hidden_layers=depth, num_attention_heads=heads,
+        num_key_value_heads=kv_heads, head_dim=128, intermediate_size=ff, rms_norm_eps=1e-6, vocab_size=32000,
+        max_position_embeddings=8192, torch_dtype="bfloat16", eos_token_id=2, tie_word_embeddings=True))
+
+
+def build(cfg):
+    weights = load_model_weights(cfg, synthetic_seed=0, device="cuda:0", dtype=torch.bfloat16)
+    n = parameters(weights)
+    return TransformerModel(cfg, weights, max_positions=8192), n
+
+
+def engine_of(model):
+    serving = parse_serving_config({"setting": {"batch_scheduler": {
+        "max_batch_size": BATCH, "max_step_tokens": STEP_TOKENS, "max_token_len": 8192, "enable_auto_prefix_cache": False}}})
+    blocks = BATCH * (CONTEXT + DECODE_STEPS + 64) // 16 + 2048
+    return LLMEngine(model, serving, num_blocks=blocks, num_host_blocks=0)
+
+
+def timed(fn) -> tuple:
+    e0, e1 = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    torch.cuda.synchronize()
+    t0 = time.perf_counter()
+    e0.record()
+    fn()
+    e1.record()
+    torch.cuda.synchronize()
+    return e0.elapsed_time(e1) / 1e3, time.perf_counter() - t0
+
+
+def drain(eng) -> int:
+    steps = 0
+    while eng.has_unfinished():
+        eng.step()
+        steps += 1
+    return steps
+
+
+def measure(model) -> dict:
+    gen = torch.Generator().manual_seed(1)
+    vocab = model.cfg.vocab_size
+
+    def prompt(n):
+        return torch.randint(3, vocab, (n,), generator=gen).tolist()
+
+    eng = engine_of(model)
+    one = SamplingParams(topk=1, max_new_tokens=1, ignore_eos=True)
+    out = {}
+    for wave in range(2):  # the first warms up
+        for _ in range(8):
+            eng.add_request(prompt(PROMPT), one)
+        dev, host = timed(lambda: drain(eng))
+    out["prefill_tok_s"] = round(8 * PROMPT / dev)
+    out["prefill_tok_s_host_clock"] = round(8 * PROMPT / host)
+    many = SamplingParams(topk=1, max_new_tokens=DECODE_STEPS + 8, ignore_eos=True)
+    for _ in range(BATCH):
+        eng.add_request(prompt(CONTEXT), many)
+    while eng.sched.num_waiting or any(not s.output_tokens for r in eng.requests.values() for s in r.seqs):
+        eng.step()
+    for _ in range(3):
+        eng.step()
+    before = cuda.launch_count
+    done = [0]
+
+    def run():
+        for _ in range(DECODE_STEPS - 20):
+            done[0] += eng.step()
+    dev, host = timed(run)
+    out["decode_tok_s"] = round(done[0] / dev)
+    out["decode_tok_s_host_clock"] = round(done[0] / host)
+    out["decode_ms_per_step"] = round(dev / (DECODE_STEPS - 20) * 1e3, 3)
+    out["decode_batch"] = round(done[0] / (DECODE_STEPS - 20))
+    out["launches_per_step"] = round((cuda.launch_count - before) / (DECODE_STEPS - 20))
+    drain(eng)
+    if cuda.read_error():
+        out["kernel_error_word"] = True
+    return out
+
+
+def run(design: str) -> None:
+    assert design == "molopel"
+    for width, depth, ff, heads, kv, window in SIZES:
+        rows = {}
+        model, n = build(molopel_config(width, depth, ff, heads, kv, 128, window))
+        rows["molopel"] = dict(parameters_m=round(n / 1e6), **measure(model))
+        del model
+        torch.cuda.empty_cache()
+        attn = depth * width * 128 * 2 * (heads + kv)
+        dense_ff = max((n - attn) // (3 * depth * width) // 128 * 128, 128)
+        model, n = build(dense_config(width, depth, dense_ff, heads, kv))
+        rows["dense"] = dict(parameters_m=round(n / 1e6), **measure(model))
+        del model
+        torch.cuda.empty_cache()
+        print(json.dumps(dict(metric="throughput", design=design, width=width, layers=depth, ff=ff, dense_ff=dense_ff,
+                              heads=heads, kv_heads=kv, window=window, dtype="bf16", data="synthetic", **rows)), flush=True)
+
+
+if __name__ == "__main__":
+    run("molopel")

@@ -81,7 +81,7 @@ def cuda_sources():
 # fresh checkout without compiling every kernel of the package.
 FAMILY_SOURCES = {
     "molopel": ("host_common", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2cta", "gemm_bf16_cluster_splitk",
-                "mixer_elementwise", "window_attention", "linear_attention"),
+                "mixer_elementwise", "window_attention", "linear_attention", "mixer_executor"),
 }
 
 # Files compiled with IEEE division, square root and the accurate math functions: what they compute is specified in

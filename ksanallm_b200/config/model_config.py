@@ -575,7 +575,33 @@ def tiny_moe_128_config() -> ModelConfig:
         rms_norm_eps=1e-6, max_position_embeddings=2048, torch_dtype="bfloat16", eos_token_id=2, bos_token_id=1))
 
 
+def molopel_config(width: int = 4096, layers: int = 32, ff: int = 12288, heads: int = 32, kv_heads: int = 8,
+                   dim: int = 128, window: int = 1024, vocab: int = 32000) -> ModelConfig:
+    """Molopel at the sizes of an ordinary decoder of that width: three windowed-attention + retention layers, then one
+    of linear attention alone. The retention half has half as many heads with values twice as wide."""
+    def decays(n):
+        return [1.0 - 2.0 ** (-5.0 - 4.0 * i / max(n - 1, 1)) for i in range(n)]
+    half = max(heads // 2, 1)
+    parallel = dict(type="parallel", mlp=dict(kind="dense", ff=ff), mixer=dict(
+        left=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, bias_max=max(window // 2, 17),
+                  mask=dict(size=window)),
+        right=dict(heads=half, dim=dim, vdim=2 * dim, decay=decays(half), rot=dict(dims=dim, base=10000.0)),
+        left_scale=0.5, right_scale=0.5))
+    lightning = dict(type="lightning", mlp=None, mixer=dict(heads=heads, dim=dim, vdim=dim, decay=decays(heads)))
+    return model_config_from_dict(dict(
+        architecture="Molopel", embedding=dict(scale=1.0), norm=dict(eps=1e-6), vocab=vocab, width=width,
+        logit_softcap=30.0, layers=[lightning if i % 4 == 3 else parallel for i in range(layers)], eos_token_id=2))
+
+
+def tiny_molopel_config() -> ModelConfig:
+    cfg = molopel_config(width=128, layers=4, ff=192, heads=4, kv_heads=2, dim=32, window=24)
+    cfg.torch_dtype = "float32"
+    return cfg
+
+
 NAMED_CONFIGS = {
+    "tiny-molopel": tiny_molopel_config,
+    "molopel": molopel_config,
     "tiny-llama": tiny_llama_config,
     "tiny-moe": tiny_moe_config,
     "tiny-moe-128": tiny_moe_128_config,

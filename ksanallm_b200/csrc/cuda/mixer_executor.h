@@ -1,0 +1,75 @@
+// Native forward pass of layers with mixers of their own sizes (windowed attention and / or linear attention, LayerNorm
+// over a 32-bit residual stream, gated FFN), driven from ONE call per step. Mirrored with ctypes on the Python side.
+#pragma once
+#include <cuda_runtime.h>
+
+extern "C" {
+
+struct KsanaMixerLayer {
+  // weights, bf16
+  const void* w_in;      // [n_in, H]: attention q, k, v, then linear attention q, k, v, gate
+  const void* b_in;      // optional bias [n_in]
+  const void* w_out;     // [H, k_out]: attention columns, then linear-attention columns, then zero padding
+  const void* ln2;       // norm before the FFN (null: the layer has none)
+  const void* w_gu;      // [2 I, H] gate rows, then up rows
+  const void* w_down;    // [H, I]
+  const void* next_ln;   // next layer's first norm, or the final norm
+  int n_in, k_out, inter;
+  // softmax attention (h == 0: none)
+  int h, hk, d, dv, window, bias_len;
+  float scale, attn_out_scale;
+  const float* q_norm;
+  const float* k_norm;
+  const float* bias;     // [h, bias_len]
+  void* kv;              // this layer's cache
+  // linear attention (lh == 0: none)
+  int lh, ld, ldv, rd, act, gate;
+  float key_scale, lin_out_scale;
+  const float* decay;
+  const float* rotary;
+  const float* norm_w;   // null: per-head norm without weight
+  float* state;          // this layer's state pool
+};
+
+struct KsanaMixerModel {
+  int hidden, block_size, num_blocks;
+  float eps;
+  // scratch for max_tokens rows
+  void* in_buf;    // [T, max n_in]
+  void* mix_buf;   // [T, max k_out]
+  void* o_buf;     // [T, max lh * ldv]
+  void* gu_buf;    // [T, 2 max I]
+  void* act_buf;   // [T, max I]
+  void* proj_buf;  // [T, H]
+  void* h_buf[2];  // [T, H]
+  float* chunk_buf;
+  long long chunk_floats;
+  float* gemm_ws;
+  long long gemm_ws_floats;
+  unsigned int* gemm_counters;
+  int n_counters;
+  const KsanaMixerLayer* layers;
+};
+
+struct KsanaMixerStep {
+  const int* positions;
+  const int* slot_mapping;
+  const int* seq_of_token;
+  const int* block_tables;
+  const int* cu_q;
+  const int* kv_lens;
+  const int* state_slots;
+  int total_tokens, max_blocks;
+  int num_prefill, num_decode, prefill_tokens;
+  int max_q_prefill, max_kv_decode;
+  int one_token;         // every decode sequence has exactly one new token
+  int num_long;          // leading prompt portions long enough for the chunked form of linear attention
+  int long_tokens;       // their tokens
+};
+
+// h: normalised input of layer `first` ([T, H] bf16), residual: [T, H] fp32 stream, updated in place. *out_h receives
+// the pointer of the normalised output. Returns 0, or (layer + 1) * 100 + step on failure with the failing call's code
+// in *fail_code.
+int ksana_mixer_forward(const KsanaMixerModel* m, const KsanaMixerStep* s, const void* h, float* residual, int first,
+                        int last, void** out_h, int* fail_code, int* launches, cudaStream_t stream);
+}

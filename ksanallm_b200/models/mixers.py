@@ -78,8 +78,9 @@ class DecayedLinearAttention:
         self.width = self.nv
         self.decay = torch.tensor(spec.decay, dtype=torch.float64).float().to(device)
         self.norm = w[prefix + ".norm"] if spec.norm == "concat" else None
-        if spec.rot_dims:
-            tables.get(spec.rot_dims, spec.rot_base)
+
+    def rotary(self) -> Optional[torch.Tensor]:
+        return self.tables.get(self.spec.rot_dims, self.spec.rot_base) if self.spec.rot_dims else None
 
     def run(self, x: torch.Tensor, meta, state: torch.Tensor, out: torch.Tensor) -> None:
         """x [T, rows] = the projected (q | k | v | gate); writes heads * vdim columns of ``out``."""
@@ -88,8 +89,7 @@ class DecayedLinearAttention:
         k = x[:, self.nq:2 * self.nq].unflatten(1, (s.heads, s.dim))
         v = x[:, 2 * self.nq:2 * self.nq + self.nv].unflatten(1, (s.heads, s.vdim))
         g = x[:, 2 * self.nq + self.nv:]
-        rotary = self.tables.get(s.rot_dims, s.rot_base) if s.rot_dims else None
-        o = ops.linear_attention(q, k, v, state, meta, self.decay, s.act, rotary, s.key_scale)
+        o = ops.linear_attention(q, k, v, state, meta, self.decay, s.act, self.rotary(), s.key_scale)
         ops.gated_norm(o, g, self.norm, self.eps, s.gate, s.out_scale, out)
 
 

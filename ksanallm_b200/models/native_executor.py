@@ -292,3 +292,148 @@ class DenseExecutor:
             return fc.hbuf[:T]
         out = self._out.value
         return (self._h[0] if out == self._h[0].data_ptr() else self._h[1])[:T]
+
+
+# ---- layers with mixers of their own sizes (csrc/cuda/mixer_executor.cu) ---------------------------------------------
+
+class _MixerLayer(ctypes.Structure):
+    _fields_ = [(n, P) for n in ("w_in", "b_in", "w_out", "ln2", "w_gu", "w_down", "next_ln")] + \
+        [(n, I) for n in ("n_in", "k_out", "inter", "h", "hk", "d", "dv", "window", "bias_len")] + \
+        [("scale", F), ("attn_out_scale", F), ("q_norm", P), ("k_norm", P), ("bias", P), ("kv", P)] + \
+        [(n, I) for n in ("lh", "ld", "ldv", "rd", "act", "gate")] + \
+        [("key_scale", F), ("lin_out_scale", F), ("decay", P), ("rotary", P), ("norm_w", P), ("state", P)]
+
+
+class _MixerModel(ctypes.Structure):
+    _fields_ = [("hidden", I), ("block_size", I), ("num_blocks", I), ("eps", F), ("in_buf", P), ("mix_buf", P),
+                ("o_buf", P), ("gu_buf", P), ("act_buf", P), ("proj_buf", P), ("h_buf", P * 2), ("chunk_buf", P),
+                ("chunk_floats", LL), ("gemm_ws", P), ("gemm_ws_floats", LL), ("gemm_counters", P), ("n_counters", I),
+                ("layers", P)]
+
+
+class _MixerStep(ctypes.Structure):
+    _fields_ = [(n, P) for n in ("positions", "slot_mapping", "seq_of_token", "block_tables", "cu_q", "kv_lens",
+                                 "state_slots")] + \
+        [(n, I) for n in ("total_tokens", "max_blocks", "num_prefill", "num_decode", "prefill_tokens", "max_q_prefill",
+                          "max_kv_decode", "one_token", "num_long", "long_tokens")]
+
+
+class MixerExecutor:
+    """The one-call-per-step path of bf16 models whose layers are :class:`~ksanallm_b200.models.mixers.MixerLayer`."""
+
+    @staticmethod
+    def eligible(model) -> bool:
+        if os.environ.get("KSANA_DISABLE_NATIVE_EXECUTOR", "0") == "1" or os.environ.get("KSANA_LIBRARY_BASELINE") == "1":
+            return False
+        if model.device.type != "cuda" or model.dtype != torch.bfloat16 or not model.layers or model.norm_w is None:
+            return False
+        for layer in model.layers:
+            lins = [layer.in_proj, layer.o_proj] + ([layer.ffn.up, layer.ffn.down] if layer.ffn is not None else [])
+            if any(lin.kind != "dense" or lin.pre is not None or lin.weight.dtype != torch.bfloat16 or
+                   not lin.weight.is_contiguous() or lin.weight.shape[0] % 8 or lin.weight.shape[1] % 8 for lin in lins):
+                return False
+            if layer.o_proj.bias is not None or layer.ffn is not None and (
+                    layer.ffn.up.bias is not None or layer.ffn.down.bias is not None or not layer.ffn.gated or
+                    layer.ffn.act != "gelu_tanh"):
+                return False
+        return True
+
+    def __init__(self, model):
+        self.model = model
+        n = len(model.layers)
+        self._layers = (_MixerLayer * n)()
+        for i, layer in enumerate(model.layers):
+            L = self._layers[i]
+            nxt = model.layers[i + 1].ln1 if i + 1 < n else model.norm_w
+            L.w_in, L.b_in, L.w_out = _p(layer.in_proj.weight), _p(layer.in_proj.bias), _p(layer.o_proj.weight)
+            L.n_in, L.k_out = layer.in_proj.weight.shape[0], layer.o_proj.weight.shape[1]
+            L.next_ln = _p(nxt)
+            if layer.ffn is not None:
+                L.ln2, L.w_gu, L.w_down = _p(layer.ln2), _p(layer.ffn.up.weight), _p(layer.ffn.down.weight)
+                L.inter = layer.ffn.down.weight.shape[1]
+            if layer.attn is not None:
+                a, s = layer.attn, layer.attn.spec
+                L.h, L.hk, L.d, L.dv, L.window = s.heads, s.kv_heads, s.dim, s.vdim, s.window
+                L.scale, L.attn_out_scale = s.scale, s.out_scale
+                L.q_norm, L.k_norm = _p(a.q_norm), _p(a.k_norm)
+            if layer.linear is not None:
+                a, s = layer.linear, layer.linear.spec
+                L.lh, L.ld, L.ldv, L.rd = s.heads, s.dim, s.vdim, s.rot_dims
+                L.act, L.gate = int(s.act == "silu"), int(s.gate == "sigmoid")
+                L.key_scale, L.lin_out_scale = s.key_scale, s.out_scale
+                L.decay, L.norm_w = _p(a.decay), _p(a.norm)
+        m = self._m = _MixerModel()
+        m.hidden, m.eps = model.cfg.hidden_size, float(model.cfg.rms_norm_eps)
+        ws = self._ws = kcuda.workspace(model.device)
+        m.gemm_ws, m.gemm_ws_floats = _p(ws.gemm_ws), ws.gemm_ws.numel()
+        m.gemm_counters, m.n_counters = _p(ws.gemm_counters), ws.gemm_counters.numel()
+        m.layers = ctypes.cast(self._layers, P)
+        self.cap, self._bufs, self._chunk = 0, [], None
+        self._key = self._tables = None
+        self._step = _MixerStep()
+        self._fn = kcuda.lib().ksana_mixer_forward
+        self._fn.argtypes, self._fn.restype = [P, P, P, P, I, I, P, P, P, P], I
+        self._out, self._fail, self._launches = P(), I(), I()
+
+    def _ensure(self, T: int) -> None:
+        if T <= self.cap:
+            return
+        cap = (max(T, 1024) + 1023) // 1024 * 1024
+        L, H = self._layers, self._m.hidden
+        cols = [max(max(f(x) for x in L), 8) for f in (
+            lambda x: x.n_in, lambda x: x.k_out, lambda x: x.lh * x.ldv, lambda x: 2 * x.inter, lambda x: x.inter)] + [H] * 3
+        self._bufs = [torch.empty(cap, c, dtype=torch.bfloat16, device=self.model.device) for c in cols]
+        m = self._m
+        m.in_buf, m.mix_buf, m.o_buf, m.gu_buf, m.act_buf, m.proj_buf, m.h_buf[0], m.h_buf[1] = (_p(b) for b in self._bufs)
+        self.cap = cap
+
+    def _bind(self, caches) -> None:
+        # the position tables grow with the longest sequence an engine asks for: they are part of the key
+        tables = [(layer.attn.bias if layer.attn else None, layer.linear.rotary() if layer.linear else None)
+                  for layer in self.model.layers]
+        key = tuple((c.kv.data_ptr(), c.kv.shape, c.state.data_ptr(), _p(b), _p(r)) for c, (b, r) in zip(caches, tables))
+        if key == self._key:
+            return
+        m = self._m
+        m.block_size = 1
+        for L, c, layer, (bias, rotary) in zip(self._layers, caches, self.model.layers, tables):
+            L.kv, L.state, L.bias, L.rotary = _p(c.kv), _p(c.state), _p(bias), _p(rotary)
+            L.bias_len = bias.shape[1] if bias is not None else 0
+            m.num_blocks = c.kv.shape[0]
+            if layer.attn is not None:
+                m.block_size = c.kv.shape[1] // layer.kv_width()
+        self._key, self._tables = key, tables
+
+    def can_run(self, meta, caches, n_layers: int) -> bool:
+        return meta.total_tokens > 0 and (meta.state_slots is not None or not self.model.cfg.has_state)
+
+    def forward(self, meta, caches, h: torch.Tensor, residual: torch.Tensor, n_layers: int) -> torch.Tensor:
+        """As DenseExecutor.forward; ``residual`` is the 32-bit stream."""
+        from ..ops.cuda_mixer import long_portions
+        T = meta.total_tokens
+        self._ensure(T)
+        self._bind(caches)
+        s, m = self._step, self._m
+        s.positions, s.slot_mapping, s.seq_of_token = _p(meta.positions), _p(meta.slot_mapping), _p(meta.seq_of_token)
+        s.block_tables, s.cu_q, s.kv_lens = _p(meta.block_tables), _p(meta.cu_q), _p(meta.kv_lens)
+        s.state_slots, s.total_tokens, s.max_blocks = _p(meta.state_slots), T, meta.max_blocks
+        n_pre, n_dec, cu = meta.num_prefill, meta.num_decode, meta.cu_q_host
+        s.num_prefill, s.num_decode, s.prefill_tokens = n_pre, n_dec, meta.num_prefill_tokens
+        s.max_q_prefill = int((cu[1:n_pre + 1] - cu[:n_pre]).max()) if n_pre else 0
+        s.max_kv_decode = int(meta.kv_lens_host[n_pre:].max()) if n_dec else 0
+        s.one_token = int(T - s.prefill_tokens == n_dec)
+        s.num_long = long_portions(meta)
+        s.long_tokens = int(cu[s.num_long])
+        if s.num_long:
+            need = max((s.long_tokens // 128 + s.num_long) * x.lh * x.ld * x.ldv for x in self._layers)
+            if need > m.chunk_floats:
+                self._chunk = torch.empty(need, dtype=torch.float32, device=self.model.device)
+                m.chunk_buf, m.chunk_floats = _p(self._chunk), need
+        rc = self._fn(ctypes.byref(m), ctypes.byref(s), h.data_ptr(), residual.data_ptr(), 0, n_layers,
+                      ctypes.byref(self._out), ctypes.byref(self._fail), ctypes.byref(self._launches),
+                      torch.cuda.current_stream().cuda_stream)
+        kcuda.launch_count += self._launches.value
+        if rc != 0:
+            raise RuntimeError(f"native mixer forward failed at layer {rc // 100 - 1}, step {rc % 100}, "
+                               f"code {self._fail.value}")
+        return self._bufs[6 if self._out.value == self._bufs[6].data_ptr() else 7][:T]

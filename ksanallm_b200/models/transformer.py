@@ -194,6 +194,7 @@ class TransformerModel:
         lookup); a stage built without ``model.norm.weight`` (not the last one) returns the un-normalised residual
         stream for the next stage. ``states``: the recurrent-state pools of a model that has them."""
         if self.cfg.layers:
+            states = states if states is not None else [kv.new_empty(0, dtype=torch.float32) for kv in kv_caches]
             kv_caches = [LayerCache(kv, st) for kv, st in zip(kv_caches, states)]
         x = self.embed_tokens(meta, refit) if hidden_in is None else hidden_in
         layers = self.layers if cutoff_layer is None else self.layers[:cutoff_layer]
@@ -228,8 +229,9 @@ class TransformerModel:
         first use; None when the model or the environment rules it out."""
         ex = getattr(self, "_native", False)
         if ex is False:
-            from .native_executor import DenseExecutor
-            ex = self._native = DenseExecutor(self) if DenseExecutor.eligible(self) else None
+            from .native_executor import DenseExecutor, MixerExecutor
+            kind = MixerExecutor if self.cfg.layers else DenseExecutor
+            ex = self._native = kind(self) if kind.eligible(self) else None
         return ex
 
     def _final_norm_only(self, x):

@@ -110,6 +110,15 @@ def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, 
 LINEAR_CHUNK_MIN_TOKENS = 16
 
 
+def long_portions(meta) -> int:
+    """How many leading prompt portions of the step go through the chunked form (a step lists them longest first; a
+    shorter one ahead of a longer one goes along)."""
+    n_pre = meta.num_prefill
+    lens = meta.cu_q_host[1:n_pre + 1] - meta.cu_q_host[:n_pre]
+    above = (lens > LINEAR_CHUNK_MIN_TOKENS).nonzero()[0]
+    return int(above[-1]) + 1 if len(above) else 0
+
+
 def linear_attention(q, k, v, state, meta, decay, act: str, rotary, key_scale: float) -> torch.Tensor:
     T, h, d = q.shape
     dv = v.shape[2]
@@ -121,20 +130,17 @@ def linear_attention(q, k, v, state, meta, decay, act: str, rotary, key_scale: f
     head = (_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0), _ptr(state), _ptr(meta.state_slots),
             _ptr(meta.cu_q), _ptr(meta.kv_lens), _ptr(meta.positions), _ptr(decay), _ptr(rotary), rd,
             1 if act == "silu" else 0, float(key_scale), h, d, dv, _ptr(out))
-    n_long = 0
-    if n_pre and q.dtype == torch.bfloat16:
-        lens = meta.cu_q_host[1:n_pre + 1] - meta.cu_q_host[:n_pre]
-        long = (lens > LINEAR_CHUNK_MIN_TOKENS).nonzero()[0]
-        n_long = int(long[-1]) + 1 if len(long) else 0  # a step lists its prompt portions longest first
-        if n_long:
-            tokens = int(meta.cu_q_host[n_long])
-            scratch = torch.empty(lib().ksana_linear_chunk_scratch(tokens, n_long, h, d, dv), dtype=torch.float32,
-                                  device=q.device)
-            code = lib().ksana_linear_chunked(*head, 0, n_long, int(lens[:n_long].max()), _ptr(scratch), _stream())
-            if code == -1:
-                n_long = 0
-            else:
-                _check(code, "linear_chunked")
+    n_long = long_portions(meta) if q.dtype == torch.bfloat16 else 0
+    if n_long:
+        cu = meta.cu_q_host
+        scratch = torch.empty(lib().ksana_linear_chunk_scratch(int(cu[n_long]), n_long, h, d, dv), dtype=torch.float32,
+                              device=q.device)
+        code = lib().ksana_linear_chunked(*head, 0, n_long, int((cu[1:n_long + 1] - cu[:n_long]).max()), _ptr(scratch),
+                                          _stream())
+        if code == -1:
+            n_long = 0
+        else:
+            _check(code, "linear_chunked")
     one = n_dec > 0 and meta.num_decode_tokens == n_dec
     for base, count, single in ((n_long, n_pre - n_long, 0), (n_pre, n_dec, 1 if one else 0)):
         if count:
