@@ -159,7 +159,7 @@ def greedy(cfg: dict, w: Dict[str, torch.Tensor], tokens: List[int], new: int) -
 
 
 # ---- random small models --------------------------------------------------------------------------------------
-def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
+def tensor_shapes(cfg: dict, bias_rows: int = 16) -> Dict[str, tuple]:
     W = cfg["width"]
     shapes = {"embed": (cfg["vocab"], W), "final.norm": (W,)}
     for i, layer in enumerate(cfg["layers"]):
@@ -183,7 +183,7 @@ def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
             for t, n in (("q", a["heads"] * a["dim"]), ("k", a["kv_heads"] * a["dim"]), ("v", a["kv_heads"] * a["vdim"])):
                 shapes[f"{p}.mix.left.{t}.b"] = (n,)
             shapes[p + ".mix.left.q.norm"] = shapes[p + ".mix.left.k.norm"] = (a["dim"],)
-            shapes[p + ".mix.left.rel"] = (a["bias_rows"], a["heads"])
+            shapes[p + ".mix.left.rel"] = (bias_rows, a["heads"])
             proj(p + ".mix.right", r["heads"], r["heads"], r["dim"], r["vdim"], "g")
         if layer["mlp"] is not None:
             shapes[p + ".norm2"] = (W,)
@@ -192,11 +192,11 @@ def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
     return shapes
 
 
-def random_weights(cfg: dict, seed: int) -> Dict[str, torch.Tensor]:
+def random_weights(cfg: dict, seed: int, bias_rows: int = 16) -> Dict[str, torch.Tensor]:
     """bfloat16 tensors whose sublayers all move the residual stream by about its own size."""
     g = torch.Generator().manual_seed(seed)
     out = {}
-    for name, shape in tensor_shapes(cfg).items():
+    for name, shape in tensor_shapes(cfg, bias_rows).items():
         r = torch.randn(*shape, generator=g, dtype=torch.float32)
         if "norm" in name.split(".")[-1]:
             t = 1 + 0.3 * r
