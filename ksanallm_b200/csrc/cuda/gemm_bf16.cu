@@ -341,6 +341,14 @@ KSANA_API int ksana_gemm_bf16_swiglu(const void* A, const void* W_interleaved, v
   return ksana::gemm_bf16_pair(A, W_interleaved, C, nullptr, M, N, K, lda, ldw, ldc, 0, 256, 1, stream);
 }
 
+// The same with the tanh form of GELU as the gate's activation.
+KSANA_API int ksana_gemm_bf16_geglu(const void* A, const void* W_interleaved, void* C, int M, int N, int K, int lda,
+                                    int ldw, int ldc, cudaStream_t stream) {
+  if (M <= 0 || N <= 0 || K <= 0) return 0;
+  if ((N & 31) || (K & 7) || (lda & 7) || (ldw & 7) || (ldc & 7)) return -1;
+  return ksana::gemm_bf16_pair(A, W_interleaved, C, nullptr, M, N, K, lda, ldw, ldc, 0, 256, 2, stream);
+}
+
 static unsigned long long* g_gemm_trace = nullptr;
 // Debug aid: device buffer of 8 uint64 that receives the timeline of CTA 0 of subsequent GEMM launches (nullptr: off).
 KSANA_API void ksana_gemm_set_trace(void* buf) { g_gemm_trace = reinterpret_cast<unsigned long long*>(buf); }

@@ -107,7 +107,8 @@ struct PairSched {
 
 // EPI 0: C = acc (+ bias).  EPI 1: gated activation. The W rows are interleaved in groups of 16 (16 gate rows, then
 // the 16 up rows of the same features), so every 32 accumulator columns hold 16 (gate, up) pairs:
-// C[row, col / 2 + j] = silu(acc[col + j]) * acc[col + 16 + j]; C is [M, N / 2].
+// C[row, col / 2 + j] = silu(acc[col + j]) * acc[col + 16 + j]; C is [M, N / 2].  EPI 2: the same with the tanh form of
+// GELU: gelu(z) = z / (1 + exp(-2 u)), u = sqrt(2 / pi) (z + 0.044715 z^3).
 template <int BN, int EPI, typename OutT>
 __global__ void __launch_bounds__(192, 1)
 gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
@@ -323,10 +324,13 @@ gemm_bf16_pair_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_cons
           for (int j = 0; j < 32; ++j)
             if (col0 + j < N) v[j] += __bfloat162float(bias[col0 + j]);
         }
-        if constexpr (EPI == 1) {
+        if constexpr (EPI != 0) {
           float o[16];
 #pragma unroll
-          for (int j = 0; j < 16; ++j) o[j] = v[j] / (1.f + __expf(-v[j])) * v[16 + j];
+          for (int j = 0; j < 16; ++j) {
+            const float e = EPI == 1 ? v[j] : 1.5957691216057308f * (v[j] + 0.044715f * v[j] * v[j] * v[j]);
+            o[j] = v[j] / (1.f + __expf(-e)) * v[16 + j];
+          }
           if (row_ok && col0 < N) {
             OutT* dst = crow + (col0 >> 1);
             if constexpr (sizeof(OutT) == 2) {
@@ -453,19 +457,21 @@ static int launch_pair(const void* A, const void* W, void* C, const void* bias, 
 
 void gemm_pair_set_lane(int lane) { g_pair_lane = lane & 1; }
 
-// epi 0: plain (+ bias); epi 1: gated SiLU over 16-row interleaved W (C is [M, N / 2], N % 32 == 0).
+// epi 0: plain (+ bias); epi 1 / 2: gated SiLU / GELU over 16-row interleaved W (C is [M, N / 2], N % 32 == 0).
 // bn: 128 or 256. Same argument rules as ksana_gemm_bf16.
 int gemm_bf16_pair(const void* A, const void* W, void* C, const void* bias, int M, int N, int K, int lda, int ldw,
                    int ldc, int out_fp32, int bn, int epi, cudaStream_t stream) {
-  if (epi == 1 && (N & 31)) return -1;
+  if (epi != 0 && (N & 31)) return -1;
 #define KSANA_PAIR_CASE(BN_, EPI_)                                                                       \
   return out_fp32 ? launch_pair<BN_, EPI_, float>(A, W, C, bias, M, N, K, lda, ldw, ldc, stream)         \
                   : launch_pair<BN_, EPI_, __nv_bfloat16>(A, W, C, bias, M, N, K, lda, ldw, ldc, stream)
   if (bn == 128) {
     if (epi == 1) { KSANA_PAIR_CASE(128, 1); }
+    if (epi == 2) return -1;
     KSANA_PAIR_CASE(128, 0);
   }
   if (epi == 1) { KSANA_PAIR_CASE(256, 1); }
+  if (epi == 2) { KSANA_PAIR_CASE(256, 2); }
   KSANA_PAIR_CASE(256, 0);
 #undef KSANA_PAIR_CASE
 }

@@ -9,6 +9,8 @@ extern "C" {
 int ksana_gemm_bf16(const void* A, const void* W, void* C, const void* bias, int M, int N, int K, int lda, int ldw,
                     int ldc, int out_fp32, int bn, int force_splits, float* ws, long long ws_floats,
                     unsigned int* counters, int num_counters, cudaStream_t stream);
+int ksana_gemm_bf16_geglu(const void* A, const void* W_interleaved, void* C, int M, int N, int K, int lda, int ldw,
+                          int ldc, cudaStream_t stream);
 int ksana_layer_norm(const void* x, int ldx, void* residual, int ldr, const void* w, const void* b, void* out, int ldo,
                      int rows, int H, float eps, int kinds, cudaStream_t st);
 int ksana_gelu_mul(const void* x, int ldx, void* out, int ldo, int rows, int I, int kind, cudaStream_t st);
@@ -147,8 +149,13 @@ struct Exec {
     if (!step(9, gemm(mix, w.k_out, w.w_out, nullptr, m->proj_buf, H, H))) return false;
     if (w.ln2 != nullptr) {
       if (!norm(10, m->proj_buf, w.ln2)) return false;
-      if (!step(11, gemm(h, H, w.w_gu, nullptr, m->gu_buf, 2 * w.inter, 2 * w.inter))) return false;
-      if (!step(12, ksana_gelu_mul(m->gu_buf, 2 * w.inter, m->act_buf, w.inter, T, w.inter, 1, st))) return false;
+      const int I = w.inter;
+      if (w.w_gu_il != nullptr && T >= 384) {
+        if (!step(11, ksana_gemm_bf16_geglu(h, w.w_gu_il, m->act_buf, T, 2 * I, H, H, H, I, st))) return false;
+      } else {
+        if (!step(11, gemm(h, H, w.w_gu, nullptr, m->gu_buf, 2 * I, 2 * I))) return false;
+        if (!step(12, ksana_gelu_mul(m->gu_buf, 2 * I, m->act_buf, I, T, I, 1, st))) return false;
+      }
       if (!step(13, gemm(m->act_buf, w.inter, w.w_down, nullptr, m->proj_buf, H, H))) return false;
     }
     return norm(14, m->proj_buf, w.next_ln);

@@ -12,6 +12,8 @@ struct KsanaMixerLayer {
   const void* w_out;     // [H, k_out]: attention columns, then linear-attention columns, then zero padding
   const void* ln2;       // norm before the FFN (null: the layer has none)
   const void* w_gu;      // [2 I, H] gate rows, then up rows
+  const void* w_gu_il;   // optional copy of w_gu, gate / up rows interleaved in groups of 16: prompt-sized steps then run
+                         // the activation as the GEMM's epilogue
   const void* w_down;    // [H, I]
   const void* next_ln;   // next layer's first norm, or the final norm
   int n_in, k_out, inter;

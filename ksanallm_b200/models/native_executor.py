@@ -297,7 +297,7 @@ class DenseExecutor:
 # ---- layers with mixers of their own sizes (csrc/cuda/mixer_executor.cu) ---------------------------------------------
 
 class _MixerLayer(ctypes.Structure):
-    _fields_ = [(n, P) for n in ("w_in", "b_in", "w_out", "ln2", "w_gu", "w_down", "next_ln")] + \
+    _fields_ = [(n, P) for n in ("w_in", "b_in", "w_out", "ln2", "w_gu", "w_gu_il", "w_down", "next_ln")] + \
         [(n, I) for n in ("n_in", "k_out", "inter", "h", "hk", "d", "dv", "window", "bias_len")] + \
         [("scale", F), ("attn_out_scale", F), ("q_norm", P), ("k_norm", P), ("bias", P), ("kv", P)] + \
         [(n, I) for n in ("lh", "ld", "ldv", "rd", "act", "gate")] + \
@@ -342,6 +342,7 @@ class MixerExecutor:
         self.model = model
         n = len(model.layers)
         self._layers = (_MixerLayer * n)()
+        self._wgu_il = []
         for i, layer in enumerate(model.layers):
             L = self._layers[i]
             nxt = model.layers[i + 1].ln1 if i + 1 < n else model.norm_w
@@ -351,6 +352,9 @@ class MixerExecutor:
             if layer.ffn is not None:
                 L.ln2, L.w_gu, L.w_down = _p(layer.ln2), _p(layer.ffn.up.weight), _p(layer.ffn.down.weight)
                 L.inter = layer.ffn.down.weight.shape[1]
+                if os.environ.get("KSANA_FUSED_SWIGLU", "0") == "1" and L.inter % 16 == 0:  # see DenseExecutor
+                    self._wgu_il.append(kcuda.interleave_gate_up(layer.ffn.up.weight))
+                    L.w_gu_il = _p(self._wgu_il[-1])
             if layer.attn is not None:
                 a, s = layer.attn, layer.attn.spec
                 L.h, L.hk, L.d, L.dv, L.window = s.heads, s.kv_heads, s.dim, s.vdim, s.window

@@ -44,6 +44,7 @@ class _Sig:
     ksana_sm_count = ([], I)
     ksana_gemm_bf16 = ([P, P, P, P, I, I, I, I, I, I, I, I, I, P, LL, P, I, P], I)
     ksana_gemm_bf16_swiglu = ([P, P, P, I, I, I, I, I, I, P], I)
+    ksana_gemm_bf16_geglu = ([P, P, P, I, I, I, I, I, I, P], I)
     ksana_gemm_fp8_block = ([P, P, P, P, P, P, I, I, I, I, I, I, I, I, P, LL, P, I, P], I)
     ksana_moe_route = ([P, I, P, I, I, I, I, I, I, I, F, P, P, P], I)
     ksana_moe_permute = ([P, I, P, I, I, I, I, I, P, P, P, P, P], I)
@@ -196,13 +197,15 @@ def interleave_gate_up(w: torch.Tensor) -> torch.Tensor:
     return torch.stack((w[:I_].view(I_ // 16, 16, -1), w[I_:].view(I_ // 16, 16, -1)), 1).reshape(w.shape).contiguous()
 
 
-def gemm_bf16_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor) -> torch.Tensor:
-    """SiLU(x Wg^T) * (x Wu^T) in one kernel: x [M, K] bf16, w_interleaved [2 I, K] from interleave_gate_up -> [M, I]."""
+def gemm_bf16_swiglu(x: torch.Tensor, w_interleaved: torch.Tensor, act: str = "silu") -> torch.Tensor:
+    """act(x Wg^T) * (x Wu^T) in one kernel: x [M, K] bf16, w_interleaved [2 I, K] from interleave_gate_up -> [M, I];
+    act silu | gelu_tanh."""
     M, K = x.shape
     N = w_interleaved.shape[0]
     out = torch.empty(M, N // 2, dtype=torch.bfloat16, device=x.device)
-    _check(lib().ksana_gemm_bf16_swiglu(_ptr(x), _ptr(w_interleaved), _ptr(out), M, N, K, x.stride(0),
-                                        w_interleaved.stride(0), out.stride(0), _stream()), "gemm_bf16_swiglu")
+    fn = lib().ksana_gemm_bf16_geglu if act == "gelu_tanh" else lib().ksana_gemm_bf16_swiglu
+    _check(fn(_ptr(x), _ptr(w_interleaved), _ptr(out), M, N, K, x.stride(0), w_interleaved.stride(0), out.stride(0),
+              _stream()), f"gemm_bf16_{act}")
     return out
 
 

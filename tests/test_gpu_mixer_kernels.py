@@ -1,7 +1,4 @@
 """CUDA kernels of layers with mixers of their own sizes against plain 32-bit statements of the same operations."""
-import math
-
-import numpy as np
 import pytest
 import torch
 
@@ -280,3 +277,13 @@ def test_gelu_softcap_embedding(dtype, width):
     ids = torch.tensor([3, 0, 10], dtype=torch.int32)
     e = cuda_mixer.embedding(ids.to(DEV), table.to(DEV), 7.5, torch.float32).cpu()
     assert torch.equal(e, table[ids.long()].float() * 7.5)
+
+
+@pytest.mark.parametrize("rows,K,ff", [(700, 256, 512), (130, 136, 48)])
+def test_gelu_gate_as_gemm_epilogue(rows, K, ff):
+    from ksanallm_b200.ops import cuda
+    g = torch.Generator().manual_seed(8)
+    x, w = torch.randn(rows, K, generator=g).to(torch.bfloat16), (torch.randn(2 * ff, K, generator=g) * 0.2).to(torch.bfloat16)
+    got = cuda.gemm_bf16_swiglu(x.to(DEV), cuda.interleave_gate_up(w.to(DEV)), "gelu_tanh").double().cpu()
+    want = M.gelu_tanh(x.double() @ w[:ff].double().T) * (x.double() @ w[ff:].double().T)
+    assert (got - want).abs().max() < 1e-2 * want.abs().max()

@@ -1,7 +1,5 @@
 """Molopel on the GPU: whole models through the engine's own step function against the plain oracle, in both number
 formats, and generation through the scheduler."""
-import os
-
 import pytest
 import torch
 
@@ -59,6 +57,18 @@ def test_layer_path_and_native_executor_agree(cases, monkeypatch):
     layers, m2 = run()
     assert m2._native is None
     assert torch.equal(native, layers)
+
+
+def test_activation_as_gemm_epilogue(cases, monkeypatch):
+    """KSANA_FUSED_SWIGLU=1: prompt-sized steps run GELU(gate) * up inside the GEMM."""
+    monkeypatch.setenv("KSANA_FUSED_SWIGLU", "1")
+    case = cases["even"]
+    eng = case.engine(torch.bfloat16, 512, "cuda")
+    toks = [case.tokens(130, i) for i in range(3)]
+    got = eng.replay([(i, t, list(range(130))) for i, t in enumerate(toks)])
+    assert eng.model._native._wgu_il
+    want = torch.cat([case.logits(t) for t in toks])
+    assert (((got.double() - want) ** 2).mean(1).sqrt() / want.std()).max() < 6e-2
 
 
 @pytest.mark.parametrize("bs", [dict(), dict(split_fuse_token_num=9), dict(enable_async=True)])
