@@ -377,18 +377,28 @@ linear_chunk_scan_kernel(LinearAttnArgs a, int seq_base, float* __restrict__ scr
   float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
   if (a.kv_lens[b] != q_len) s = *S;
   const int chunks = (q_len + LC - 1) / LC;
-  const float whole = decay_pow(a.decay[head], LC);
+  const float whole = decay_pow(a.decay[head], LC), last = decay_pow(a.decay[head], q_len - (chunks - 1) * LC);
   const size_t step = static_cast<size_t>(a.h) * per;
-  float4* p = reinterpret_cast<float4*>(scratch + (chunk_entry(a, seq_base, b, 0) * a.h + head) * per + e);
-  float4 next = *p;
-  for (int c = 0; c < chunks; ++c) {
-    const float4 v = next;
-    float4* here = p;
-    p = reinterpret_cast<float4*>(reinterpret_cast<float*>(p) + step);
-    if (c + 1 < chunks) next = *p;
-    *here = s;
-    const float f = c + 1 < chunks ? whole : decay_pow(a.decay[head], q_len - c * LC);
-    s.x = f * s.x + v.x; s.y = f * s.y + v.y; s.z = f * s.z + v.z; s.w = f * s.w + v.w;
+  float* p = scratch + (chunk_entry(a, seq_base, b, 0) * a.h + head) * per + e;
+  auto at = [&](int c) { return reinterpret_cast<float4*>(p + c * step); };
+  // the chain over the chunks is short arithmetic: what it costs is the loads, so AHEAD of them are kept in flight
+  constexpr int AHEAD = 8;
+  float4 ring[AHEAD];
+#pragma unroll
+  for (int i = 0; i < AHEAD; ++i)
+    if (i < chunks) ring[i] = *at(i);
+  for (int c0 = 0; c0 < chunks; c0 += AHEAD) {
+#pragma unroll
+    for (int i = 0; i < AHEAD; ++i) {
+      const int c = c0 + i;
+      if (c < chunks) {
+        const float4 v = ring[i];
+        if (c + AHEAD < chunks) ring[i] = *at(c + AHEAD);
+        *at(c) = s;
+        const float f = c + 1 < chunks ? whole : last;
+        s.x = f * s.x + v.x; s.y = f * s.y + v.y; s.z = f * s.z + v.z; s.w = f * s.w + v.w;
+      }
+    }
   }
   *S = s;
 }
