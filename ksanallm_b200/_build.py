@@ -80,13 +80,14 @@ def cuda_sources():
 # Kernel sources of model families that can be served from a library of their own: enough to load one such model in a
 # fresh checkout without compiling every kernel of the package.
 FAMILY_SOURCES = {
-    "molopel": ("host_common", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2cta", "gemm_bf16_cluster_splitk",
-                "mixer_elementwise", "window_attention", "linear_attention", "mixer_executor"),
+    family: ("host_common", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2cta", "gemm_bf16_cluster_splitk", "moe",
+             "moe_topk", "mixer_elementwise", "window_attention", "linear_attention", "mixer_executor")
+    for family in ("molopel", "givirax")
 }
 
 # Files compiled with IEEE division, square root and the accurate math functions: what they compute is specified in
 # 32-bit floats.
-EXACT_MATH = {"mixer_elementwise", "window_attention", "linear_attention"}
+EXACT_MATH = {"moe_topk", "mixer_elementwise", "window_attention", "linear_attention"}
 
 
 def cuda_library(family: str = "") -> Path:

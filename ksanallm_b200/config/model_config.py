@@ -11,7 +11,7 @@ from __future__ import annotations
 import json
 import os
 from dataclasses import dataclass, field
-from typing import Any, Dict, List, Optional
+from typing import Any, Dict, List, Optional, Tuple
 
 
 @dataclass
@@ -49,6 +49,8 @@ class AttentionSpec:
     vdim: int
     scale: float
     window: int = 0          # keys a position sees, itself included (0: all earlier ones)
+    keep_first: int = 0      # the first tokens of the sequence stay visible however far behind the window they are
+    shared_kv: bool = False  # the values are the keys: no value projection, one vector per token in the cache
     bias_max: float = 0.0    # learned distance bias: distance at which its log-spaced buckets end (0: no bias)
     qkv_bias: bool = False
     qk_norm: bool = False    # per-head RMS norm of q and k
@@ -72,15 +74,48 @@ class LinearAttentionSpec:
 
 
 @dataclass
+class ExpertsSpec:
+    """A mixture of gated-SiLU experts: the ``top`` largest router logits choose, and the softmax over the chosen logits
+    weights them."""
+    experts: int
+    top: int
+    ff: int
+    router_bias: bool = False  # a bias on the router logits, before the choice
+
+
+@dataclass
 class LayerSpec:
-    """One layer of a model whose layers differ: its mixers (side by side when there are both) and its feed-forward."""
+    """One layer of a model whose layers differ: its mixers (side by side when there are both) and its feed-forward,
+    which is dense (``ff``), routed (``moe``) or absent."""
     attn: Optional[AttentionSpec] = None
     linear: Optional[LinearAttentionSpec] = None
-    ff: int = 0              # feed-forward width (0: the layer has none)
+    ff: int = 0              # dense feed-forward width (0: none)
+    moe: Optional[ExpertsSpec] = None
+    gated: bool = True       # dense feed-forward: act(gate) * up, else act(up)
+    parallel: bool = False   # mixers and feed-forward read the same norm: x + (mixers(h) + ff(h))
 
     @property
     def state_shape(self):
         return (self.linear.heads, self.linear.dim, self.linear.vdim) if self.linear else None
+
+    @property
+    def has_ff(self) -> bool:
+        return self.ff > 0 or self.moe is not None
+
+    @property
+    def kv_width(self) -> int:
+        """Cache elements per token."""
+        a = self.attn
+        return a.kv_heads * (a.dim + (0 if a.shared_kv else a.vdim)) if a else 0
+
+
+@dataclass
+class LoopSpec:
+    """Layers start .. stop - 1 run ``times`` times in a row with the same weights. A learned vector per pass is added to
+    the stream ahead of the pass, and ahead of every pass but the first also the embedding output."""
+    start: int
+    stop: int
+    times: int
 
 
 @dataclass
@@ -165,6 +200,7 @@ class ModelConfig:
     layers: List[LayerSpec] = field(default_factory=list)
     logit_softcap: float = 0.0    # logits <- cap * tanh(logits / cap); 0 = off
     residual_fp32: bool = False   # the residual stream is kept in 32-bit floats
+    loop: Optional[LoopSpec] = None
     # quantisation
     quant: QuantConfig = field(default_factory=QuantConfig)
     raw: Dict[str, Any] = field(default_factory=dict)
@@ -174,6 +210,8 @@ class ModelConfig:
         return self.num_experts > 0
 
     def is_moe_layer(self, layer_idx: int) -> bool:
+        if self.layers:
+            return self.layers[layer_idx].moe is not None
         if not self.is_moe:
             return False
         if self.moe_layers:
@@ -184,6 +222,16 @@ class ModelConfig:
     def has_state(self) -> bool:
         """Some layer carries a recurrent state from token to token."""
         return any(l.linear is not None for l in self.layers)
+
+    def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
+        """The layers in the order they run, each with the number of the pass that starts with it (None: no pass does).
+        Every run has a cache of its own."""
+        order = list(range(self.num_layers))
+        if self.loop is None:
+            return [(i, None) for i in order]
+        lo, hi = self.loop.start, self.loop.stop
+        passes = [(i, t if i == lo else None) for t in range(self.loop.times) for i in order[lo:hi]]
+        return [(i, None) for i in order[:lo]] + passes + [(i, None) for i in order[hi:]]
 
     @property
     def q_head_dim(self) -> int:
@@ -255,11 +303,79 @@ def _molopel_mixers(kind: str, c: Dict[str, Any]) -> LayerSpec:
     raise ValueError(f"unknown Molopel layer type {kind!r}")
 
 
+def _layered_config(c: Dict[str, Any], model_type: str) -> ModelConfig:
+    """What the designs whose ``config.json`` lists their layers one by one have in common; reads ``m.layers``' sizes into
+    the fields other parts of the engine look at."""
+    m = ModelConfig(model_type=model_type, architectures=[str(c["architecture"])], raw=c)
+    m.vocab_size, m.hidden_size = int(c["vocab"]), int(c["width"])
+    m.rms_norm_eps = float(c["norm"]["eps"])
+    m.emb_scale = float((c.get("embedding") or {}).get("scale", 1.0))
+    m.residual_fp32 = True
+    m.hidden_act = "gelu_tanh"
+    m.torch_dtype = str(c.get("torch_dtype", "bfloat16"))
+    eos = c.get("eos_token_id")
+    m.eos_token_ids = [int(e) for e in eos] if isinstance(eos, (list, tuple)) else ([int(eos)] if eos is not None else [])
+    m.bos_token_id, m.pad_token_id = c.get("bos_token_id"), c.get("pad_token_id")
+    return m
+
+
+def _set_layers(m: ModelConfig, layers: List[LayerSpec]) -> None:
+    m.layers, m.num_layers = layers, len(layers)
+    attn = next((l.attn for l in layers if l.attn is not None), None)
+    if attn is not None:
+        m.num_heads, m.num_kv_heads, m.head_dim = attn.heads, attn.kv_heads, attn.dim
+    m.intermediate_size = max((l.ff for l in layers), default=0)
+    m.num_experts = max((l.moe.experts for l in layers if l.moe), default=0)
+    m.num_experts_per_tok = max((l.moe.top for l in layers if l.moe), default=0)
+    m.moe_intermediate_size = max((l.moe.ff for l in layers if l.moe), default=0)
+
+
+def _givirax_layer(entry: Dict[str, Any]) -> LayerSpec:
+    if str(entry["type"]) != "attention":
+        raise ValueError(f"unknown Givirax layer type {entry['type']!r}")
+    a, mlp = entry["mixer"], entry.get("mlp")
+    spec = LayerSpec(parallel=True, gated=False, attn=AttentionSpec(
+        int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), int(a["vdim"]), float(a["scale"]),
+        window=int(a["mask"]["size"]), keep_first=int(a["mask"]["keep_first"]), shared_kv=True))
+    if spec.attn.vdim != spec.attn.dim or spec.attn.heads % spec.attn.kv_heads:
+        raise ValueError("values that are the keys have the keys' size, and heads are a multiple of kv_heads")
+    if spec.attn.window < 1:
+        raise ValueError("a position sees at least itself: mask.size >= 1")
+    if mlp is not None:
+        kind = str(mlp.get("kind", "dense"))
+        if kind == "dense":
+            spec.ff = int(mlp["ff"])
+        elif kind == "moe":
+            r = mlp["router"]
+            spec.moe = ExpertsSpec(int(r["experts"]), int(r["top"]), int(mlp["expert"]["ff"]), router_bias=True)
+            if not 1 <= spec.moe.top <= spec.moe.experts:
+                raise ValueError("router.top must lie between 1 and router.experts")
+        else:
+            raise ValueError(f"unknown Givirax feed-forward {kind!r}")
+    return spec
+
+
+def _givirax_config(c: Dict[str, Any]) -> ModelConfig:
+    """Givirax: layers whose attention (a sliding window plus the first tokens, no rotation, values = keys) and
+    feed-forward (plain GELU or routed SiLU experts) read one norm side by side; learned positions, a range of layers that
+    runs several times, untied head."""
+    m = _layered_config(c, "givirax")
+    _set_layers(m, [_givirax_layer(e) for e in c["layers"]])
+    m.position_encoding, m.gated_mlp = "learned", False
+    m.max_position_embeddings = int(c["max_positions"])
+    loop = c.get("loop")
+    if loop:
+        m.loop = LoopSpec(int(loop["start"]), int(loop["stop"]), int(loop["times"]))
+        if not (0 <= m.loop.start < m.loop.stop <= m.num_layers and m.loop.times >= 1):
+            raise ValueError(f"loop {loop} does not fit {m.num_layers} layers")
+    return m
+
+
 def _molopel_config(c: Dict[str, Any]) -> ModelConfig:
     """Molopel: layers of linear attention alone ("lightning") or of windowed attention beside retention
     ("parallel"), each with sizes of its own; LayerNorm without bias, tied embeddings, soft-capped logits."""
-    m = ModelConfig(model_type="molopel", architectures=[str(c.get("architecture", "Molopel"))], raw=c)
-    m.vocab_size, m.hidden_size = int(c["vocab"]), int(c["width"])
+    m = _layered_config(c, "molopel")
+    layers = []
     for entry in c["layers"]:
         spec = _molopel_mixers(str(entry["type"]), entry["mixer"])
         mlp = entry.get("mlp")
@@ -269,29 +385,19 @@ def _molopel_config(c: Dict[str, Any]) -> ModelConfig:
             spec.ff = int(mlp["ff"])
         if spec.linear is not None and len(spec.linear.decay) != spec.linear.heads:
             raise ValueError("one decay per head is needed")
-        m.layers.append(spec)
-    m.num_layers = len(m.layers)
-    attn = next((l.attn for l in m.layers if l.attn is not None), None)
-    if attn is not None:
-        m.num_heads, m.num_kv_heads, m.head_dim = attn.heads, attn.kv_heads, attn.dim
-    m.intermediate_size = max((l.ff for l in m.layers), default=0)
-    m.rms_norm_eps = float(c["norm"]["eps"])
-    m.norm_type, m.position_encoding, m.hidden_act = "layernorm", "none", "gelu_tanh"
+        layers.append(spec)
+    _set_layers(m, layers)
+    m.norm_type, m.position_encoding = "layernorm", "none"
     m.tie_word_embeddings = True
-    m.emb_scale = float((c.get("embedding") or {}).get("scale", 1.0))
     m.logit_softcap = float(c.get("logit_softcap") or 0.0)
-    m.residual_fp32 = True
     m.max_position_embeddings = int(c.get("max_position_embeddings", 1 << 20))
-    m.torch_dtype = str(c.get("torch_dtype", "bfloat16"))
-    eos = c.get("eos_token_id")
-    m.eos_token_ids = [int(e) for e in eos] if isinstance(eos, (list, tuple)) else ([int(eos)] if eos is not None else [])
-    m.bos_token_id, m.pad_token_id = c.get("bos_token_id"), c.get("pad_token_id")
     return m
 
 
 def model_config_from_dict(c: Dict[str, Any]) -> ModelConfig:
-    if str(c.get("architecture", "")).lower() == "molopel":
-        return _molopel_config(c)
+    design = {"molopel": _molopel_config, "givirax": _givirax_config}.get(str(c.get("architecture", "")).lower())
+    if design is not None:
+        return design(c)
     if isinstance(c.get("text_config"), dict) and str(c.get("model_type", "")).lower() in ("llama4",):
         # multimodal wrapper configs keep the language model under "text_config"
         inner = dict(c["text_config"])
@@ -599,7 +705,31 @@ def tiny_molopel_config() -> ModelConfig:
     return cfg
 
 
+def givirax_config(width: int = 4096, layers: int = 16, ff: int = 12288, experts: int = 16, top: int = 2,
+                   expert_ff: int = 3072, heads: int = 32, kv_heads: int = 8, dim: int = 128, window: int = 1024,
+                   keep_first: int = 4, loop: Optional[Dict[str, int]] = None, vocab: int = 32000,
+                   max_positions: int = 8192) -> ModelConfig:
+    """Givirax at the sizes of an ordinary decoder of that width: dense and routed feed-forwards in turn."""
+    mixer = dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5,
+                 mask=dict(size=window, keep_first=keep_first))
+    dense = dict(kind="dense", ff=ff)
+    moe = dict(kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top))
+    return model_config_from_dict(dict(
+        architecture="Givirax", embedding=dict(scale=1.0), norm=dict(eps=1e-6), vocab=vocab, width=width,
+        max_positions=max_positions, loop=loop, eos_token_id=2,
+        layers=[dict(type="attention", mixer=mixer, mlp=moe if i % 2 else dense) for i in range(layers)]))
+
+
+def tiny_givirax_config() -> ModelConfig:
+    cfg = givirax_config(width=128, layers=3, ff=192, experts=6, expert_ff=48, heads=4, kv_heads=2, dim=32, window=24,
+                         keep_first=2, loop=dict(start=0, stop=2, times=3), max_positions=512)
+    cfg.torch_dtype = "float32"
+    return cfg
+
+
 NAMED_CONFIGS = {
+    "tiny-givirax": tiny_givirax_config,
+    "givirax": givirax_config,
     "tiny-molopel": tiny_molopel_config,
     "molopel": molopel_config,
     "tiny-llama": tiny_llama_config,

@@ -94,8 +94,8 @@ rms_norm_kernel(const __nv_bfloat16* __restrict__ x, int ldx, __nv_bfloat16* __r
 // ---- SiLU(gate) * up ------------------------------------------------------------------------------------------
 __global__ void silu_mul_kernel(const __nv_bfloat16* __restrict__ x, int ldx, __nv_bfloat16* __restrict__ out, int ldo,
                                 int I) {
-  const int row = blockIdx.y;
-  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  const int row = blockIdx.x;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
   if (c >= I) return;
   const __nv_bfloat16* xr = x + static_cast<size_t>(row) * ldx;
   float g[8], u[8], o[8];
@@ -336,7 +336,7 @@ KSANA_API int ksana_rms_norm(const void* x, int ldx, void* residual, int ldr, co
 KSANA_API int ksana_silu_mul(const void* x, int ldx, void* out, int ldo, int T, int I, cudaStream_t stream) {
   if (T <= 0) return 0;
   if ((I & 7) || (ldx & 7) || (ldo & 7)) return -1;
-  dim3 grid((I / 8 + 255) / 256, T);
+  dim3 grid(T, (I / 8 + 255) / 256);
   silu_mul_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const __nv_bfloat16*>(x), ldx,
                                             reinterpret_cast<__nv_bfloat16*>(out), ldo, I);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;

@@ -1,43 +1,104 @@
-// Bandwidth-bound steps of layers with mixers of their own sizes: LayerNorm over a 32-bit residual stream, embedding
-// into that stream, GELU(gate) * up, per-head QK norm with the paged cache append, the gated RMS norm behind linear
-// attention, and the logit soft cap. Everything is computed in 32-bit floats; T is the storage type of activations.
+// Bandwidth-bound steps of layers with mixers of their own sizes: norms over a 32-bit residual stream, embedding into
+// that stream, GELU (gated or not), the paged cache append (with per-head QK norm, or beside the activation), the gated
+// RMS norm behind linear attention, and the logit soft cap. Everything is computed in 32-bit floats; T is the storage type of activations.
 #include "host_common.h"
 #include "mixer_common.cuh"
 
 namespace ksana {
 
-// ---- LayerNorm (+ residual add) -----------------------------------------------------------------------------
-// residual (fp32 or T, may be null) += x; out = (r - mean) / sqrt(var + eps) * w (+ b). The row stays in registers:
-// VPT groups of 4 per thread.
+// ---- the stream and its norms -----------------------------------------------------------------------------------
+// A row of the stream (R) takes what a sublayer hands over and is normalised for the next one:
+//   v = res_in + (x + sum_j weights[t, j] y[pos[t, j]]) + add_rows + add_vec;  res_out = v
+//   out = v / sqrt(mean(v^2) + eps) * w                        (center 0)
+//   out = (v - mean(v)) / sqrt(var(v) + eps) * w (+ b)         (center 1)
+// Every term may be absent (null). y holds the rows of routed experts in sorted order (pos -1: another rank's expert).
+template <typename X, typename R, typename W, typename O>
+struct StreamNormArgs {
+  const X* x;
+  int ldx;
+  const R* res_in;
+  R* res_out;
+  int ldr;
+  const W* w;
+  const W* b;
+  O* out;
+  int ldo, H;
+  float eps;
+  int center;
+  const float* add_rows;  // [rows, H]
+  const float* add_vec;   // [H]
+  const X* y;             // [n, H]
+  const int* pos;
+  const float* weights;
+  int k;
+
+  // N columns of the new stream value of `row`
+  template <int N>
+  __device__ void value(size_t row, int c, float* v) const {
+#pragma unroll
+    for (int j = 0; j < N; ++j) v[j] = 0.f;
+    if (x) load_n<N>(x + row * ldx + c, v);
+    float f[N];
+    for (int e = 0; e < k; ++e) {
+      const int p = pos[row * k + e];
+      if (p < 0) continue;
+      const float g = weights[row * k + e];
+      load_n<N>(y + static_cast<size_t>(p) * H + c, f);
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] = fmaf(g, f[j], v[j]);
+    }
+    if (res_in) {
+      load_n<N>(res_in + row * ldr + c, f);
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] += f[j];
+    }
+    if (add_rows) {
+      load_n<N>(add_rows + row * H + c, f);
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] += f[j];
+    }
+    if (add_vec) {
+      load_n<N>(add_vec + c, f);
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[j] += f[j];
+    }
+  }
+  template <int N>
+  __device__ void keep(size_t row, int c, float* v) const {
+    if (res_out) {
+      store_n<N>(res_out + row * ldr + c, v);
+      if constexpr (sizeof(R) == 2) {  // the norm sees what the stream keeps
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[j] = to_f(from_f<R>(v[j]));
+      }
+    }
+  }
+};
+
+// The row stays in registers: VPT groups of 4 per thread.
 template <typename X, typename R, typename W, typename O, int VPT>
 __global__ void __launch_bounds__(256)
-layer_norm_kernel(const X* __restrict__ x, int ldx, R* __restrict__ residual, int ldr, const W* __restrict__ w,
-                  const W* __restrict__ b, O* __restrict__ out, int ldo, int H, float eps) {
+stream_norm_kernel(const StreamNormArgs<X, R, W, O> a) {
   __shared__ float red[32];
   const size_t row = blockIdx.x;
+  const int H = a.H;
   float v[VPT][4];
   float s = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (i * 256 + threadIdx.x) * 4;
+    if (c < H) a.template value<4>(row, c, v[i]);
+  }
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (i * 256 + threadIdx.x) * 4;
     if (c < H) {
-      load_n<4>(x + row * ldx + c, v[i]);
-      if (residual) {
-        float r[4];
-        load_n<4>(residual + row * ldr + c, r);
-#pragma unroll
-        for (int j = 0; j < 4; ++j) v[i][j] += r[j];
-        store_n<4>(residual + row * ldr + c, v[i]);
-        if constexpr (sizeof(R) == 2) {  // the norm sees what the stream keeps
-#pragma unroll
-          for (int j = 0; j < 4; ++j) v[i][j] = to_f(from_f<R>(v[i][j]));
-        }
-      }
+      a.template keep<4>(row, c, v[i]);
 #pragma unroll
       for (int j = 0; j < 4; ++j) s += v[i][j];
     }
   }
-  const float mean = block_sum(s, red) / static_cast<float>(H);
+  const float mean = a.center ? block_sum(s, red) / static_cast<float>(H) : 0.f;
   float ss = 0.f;
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
@@ -49,85 +110,97 @@ layer_norm_kernel(const X* __restrict__ x, int ldx, R* __restrict__ residual, in
       }
     }
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(H) + eps);
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(H) + a.eps);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (i * 256 + threadIdx.x) * 4;
     if (c < H) {
       float g[4], o[4];
-      load_n<4>(w + c, g);
+      load_n<4>(a.w + c, g);
 #pragma unroll
       for (int j = 0; j < 4; ++j) o[j] = v[i][j] * inv * g[j];
-      if (b) {
-        load_n<4>(b + c, g);
+      if (a.b) {
+        load_n<4>(a.b + c, g);
 #pragma unroll
         for (int j = 0; j < 4; ++j) o[j] += g[j];
       }
-      store_n<4>(out + row * ldo + c, o);
+      store_n<4>(a.out + row * a.ldo + c, o);
     }
   }
 }
 
-// Any width and alignment: the row is read again for each of the three passes.
+// Any width and alignment: the row's new value stays in shared memory.
 template <typename X, typename R, typename W, typename O>
 __global__ void __launch_bounds__(256)
-layer_norm_any_kernel(const X* __restrict__ x, int ldx, R* residual, int ldr, const W* __restrict__ w,
-                      const W* __restrict__ b, O* __restrict__ out, int ldo, int H, float eps) {
+stream_norm_any_kernel(const StreamNormArgs<X, R, W, O> a) {
+  extern __shared__ float row_v[];
   __shared__ float red[32];
   const size_t row = blockIdx.x;
-  auto value = [&](int c) { return residual ? to_f(residual[row * ldr + c]) : to_f(x[row * ldx + c]); };
+  const int H = a.H;
   float s = 0.f;
   for (int c = threadIdx.x; c < H; c += 256) {
-    if (residual) residual[row * ldr + c] = from_f<R>(to_f(residual[row * ldr + c]) + to_f(x[row * ldx + c]));
-    s += value(c);
+    float v;
+    a.template value<1>(row, c, &v);
+    a.template keep<1>(row, c, &v);
+    row_v[c] = v;  // only this thread reads it back
+    s += v;
   }
-  const float mean = block_sum(s, red) / static_cast<float>(H);
+  const float mean = a.center ? block_sum(s, red) / static_cast<float>(H) : 0.f;
   float ss = 0.f;
   for (int c = threadIdx.x; c < H; c += 256) {
-    const float d = value(c) - mean;
+    const float d = row_v[c] - mean;
     ss += d * d;
   }
-  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(H) + eps);
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(H) + a.eps);
   for (int c = threadIdx.x; c < H; c += 256) {
-    float o = (value(c) - mean) * inv * to_f(w[c]);
-    if (b) o += to_f(b[c]);
-    out[row * ldo + c] = from_f<O>(o);
+    float o = (row_v[c] - mean) * inv * to_f(a.w[c]);
+    if (a.b) o += to_f(a.b[c]);
+    a.out[row * a.ldo + c] = from_f<O>(o);
   }
 }
 
 template <typename X, typename R, typename W, typename O>
-static int launch_layer_norm(const void* x, int ldx, void* residual, int ldr, const void* w, const void* b, void* out,
-                             int ldo, int rows, int H, float eps, cudaStream_t st) {
-  auto px = static_cast<const X*>(x);
-  auto pr = static_cast<R*>(residual);
-  auto pw = static_cast<const W*>(w), pb = static_cast<const W*>(b);
-  auto po = static_cast<O*>(out);
+static int launch_stream_norm(const void* x, int ldx, const void* res_in, void* res_out, int ldr, const void* w,
+                              const void* b, void* out, int ldo, int rows, int H, float eps, int center,
+                              const float* add_rows, const float* add_vec, const void* y, const int* pos,
+                              const float* weights, int k, cudaStream_t st) {
+  const StreamNormArgs<X, R, W, O> a{static_cast<const X*>(x), ldx, static_cast<const R*>(res_in),
+                                     static_cast<R*>(res_out), ldr, static_cast<const W*>(w), static_cast<const W*>(b),
+                                     static_cast<O*>(out), ldo, H, eps, center, add_rows, add_vec,
+                                     static_cast<const X*>(y), pos, weights, y ? k : 0};
   const bool vec = !((H | ldx | ldr | ldo) & 3) && H <= 8192;
-#define KSANA_LN(V) layer_norm_kernel<X, R, W, O, V><<<rows, 256, 0, st>>>(px, ldx, pr, ldr, pw, pb, po, ldo, H, eps)
-  if (!vec)
-    layer_norm_any_kernel<X, R, W, O><<<rows, 256, 0, st>>>(px, ldx, pr, ldr, pw, pb, po, ldo, H, eps);
-  else if (H <= 1024)
-    KSANA_LN(1);
-  else if (H <= 2048)
-    KSANA_LN(2);
-  else if (H <= 4096)
-    KSANA_LN(4);
-  else
-    KSANA_LN(8);
-#undef KSANA_LN
+#define KSANA_SN(V) stream_norm_kernel<X, R, W, O, V><<<rows, 256, 0, st>>>(a)
+  if (!vec) {
+    if (H > 50 * 1024) return -1;
+    auto kern = stream_norm_any_kernel<X, R, W, O>;
+    if (H * 4 > 47 * 1024 && KSANA_SMEM_ONCE(kern, 200 * 1024) != 0) return -4;
+    kern<<<rows, 256, H * 4, st>>>(a);
+  } else if (H <= 1024) {
+    KSANA_SN(1);
+  } else if (H <= 2048) {
+    KSANA_SN(2);
+  } else if (H <= 4096) {
+    KSANA_SN(4);
+  } else {
+    KSANA_SN(8);
+  }
+#undef KSANA_SN
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
 // ---- embedding into a 32-bit stream ---------------------------------------------------------------------------
+// out = table[id] * scale (+ pos_table[position], unscaled)
 template <typename T>
 __global__ void embedding_f32_kernel(const int* __restrict__ ids, const T* __restrict__ table, float* __restrict__ out,
-                                     int H, int vocab, float scale) {
+                                     int H, int vocab, float scale, const int* __restrict__ positions,
+                                     const T* __restrict__ pos_table, int pos_rows) {
   const size_t row = blockIdx.y;
   const int c = blockIdx.x * blockDim.x + threadIdx.x;
   if (c >= H) return;
-  int id = ids[row];
-  id = id < 0 ? 0 : (id >= vocab ? vocab - 1 : id);
-  out[row * H + c] = to_f(table[static_cast<size_t>(id) * H + c]) * scale;
+  const int id = min(max(ids[row], 0), vocab - 1);
+  float v = to_f(table[static_cast<size_t>(id) * H + c]) * scale;
+  if (pos_table) v += to_f(pos_table[static_cast<size_t>(min(max(positions[row], 0), pos_rows - 1)) * H + c]);
+  out[row * H + c] = v;
 }
 
 // ---- GELU(gate) * up --------------------------------------------------------------------------------------------
@@ -145,8 +218,8 @@ __global__ void gelu_mul_kernel(const T* __restrict__ x, int ldx, T* __restrict_
 }
 
 // ---- per-head QK norm + cache append ------------------------------------------------------------------------------
-// One warp per (token, head): heads [0, h) are queries (normalised in place), the next hk keys (normalised into the
-// cache), the last hk values (copied into the cache). Cache: [block][keys hk x bs x d | values hk x bs x dv].
+// One warp per (token, head): heads [0, h) are queries (normalised in place; h is 0 when they are not), the next hk keys
+// (normalised into the cache), the last hk values (copied into the cache). Cache: [block][keys hk x bs x d | values hk x bs x dv].
 template <typename T, int N>
 __global__ void __launch_bounds__(256)
 qk_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ldk, const T* __restrict__ v, int ldv,
@@ -165,7 +238,6 @@ qk_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ld
     dst = q + static_cast<size_t>(t) * ldq + hd * d;
     src = dst;
     w = qw;
-    if (w == nullptr) return;
   } else {
     const int slot = slots[t];
     if (slot < 0) return;
@@ -201,6 +273,34 @@ qk_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ld
     }
     store_n<N>(dst + c, f);
   }
+}
+
+// ---- cache append beside an activation -----------------------------------------------------------------------------
+// A row of x holds new keys (nk columns, to the cache of keys alone: [block][hk x bs x d]) and, behind them, the input of
+// a feed-forward's activation: out = gelu(up), or gelu(gate) * up over 2 I columns. N columns per thread.
+template <typename T, int N>
+__global__ void __launch_bounds__(256)
+append_act_kernel(const T* __restrict__ k, const T* __restrict__ u, int ldx, const int* __restrict__ slots,
+                  T* __restrict__ cache, int nk, int d, int bs, T* __restrict__ out, int ldo, int I, int gated) {
+  const size_t row = blockIdx.x;
+  int c = (blockIdx.y * 256 + threadIdx.x) * N;
+  float f[N];
+  if (c < nk) {
+    const int slot = slots[row];
+    if (slot < 0) return;
+    load_n<N>(k + row * ldx + c, f);
+    store_n<N>(cache + static_cast<size_t>(slot / bs) * bs * nk + (static_cast<size_t>(c / d) * bs + slot % bs) * d + c % d,
+               f);
+    return;
+  }
+  c -= nk;
+  if (c >= I) return;
+  load_n<N>(u + row * ldx + c, f);
+  float g[N];
+  if (gated) load_n<N>(u + row * ldx + I + c, g);
+#pragma unroll
+  for (int j = 0; j < N; ++j) f[j] = gelu_tanh_f(f[j]) * (gated ? g[j] : 1.f);
+  store_n<N>(out + row * ldo + c, f);
 }
 
 // ---- gated RMS norm behind linear attention -------------------------------------------------------------------------
@@ -305,30 +405,45 @@ static int done() { return cudaGetLastError() == cudaSuccess ? 0 : -5; }
 using namespace ksana;
 using bf16 = __nv_bfloat16;
 
-// Storage types: 0 = fp32, 1 = bf16. `kinds` = x | residual << 1 | weight << 2 | out << 3. Row pitches in elements.
-KSANA_API int ksana_layer_norm(const void* x, int ldx, void* residual, int ldr, const void* w, const void* b, void* out,
-                               int ldo, int rows, int H, float eps, int kinds, cudaStream_t st) {
+// Storage types: 0 = fp32, 1 = bf16. `kinds` = x (and y) | stream << 1 | weight << 2 | out << 3. Row pitches in elements.
+KSANA_API int ksana_stream_norm(const void* x, int ldx, const void* res_in, void* res_out, int ldr, const void* w,
+                                const void* b, void* out, int ldo, int rows, int H, float eps, int kinds, int center,
+                                const float* add_rows, const float* add_vec, const void* y, const int* pos,
+                                const float* weights, int k, cudaStream_t st) {
   if (rows <= 0 || H <= 0) return 0;
-#define KSANA_LN_CASE(K, X, R, W, O) \
-  case K: return launch_layer_norm<X, R, W, O>(x, ldx, residual, ldr, w, b, out, ldo, rows, H, eps, st)
+#define KSANA_SN_CASE(K, X, R, W, O)                                                                             \
+  case K:                                                                                                        \
+    return launch_stream_norm<X, R, W, O>(x, ldx, res_in, res_out, ldr, w, b, out, ldo, rows, H, eps, center,    \
+                                          add_rows, add_vec, y, pos, weights, k, st)
   switch (kinds) {
-    KSANA_LN_CASE(0, float, float, float, float);
-    KSANA_LN_CASE(12, float, float, bf16, bf16);  // first norm of a bf16 model over its 32-bit stream
-    KSANA_LN_CASE(13, bf16, float, bf16, bf16);   // sublayer output into the 32-bit stream
-    KSANA_LN_CASE(15, bf16, bf16, bf16, bf16);
+    KSANA_SN_CASE(0, float, float, float, float);
+    KSANA_SN_CASE(12, float, float, bf16, bf16);  // first norm of a bf16 model over its 32-bit stream
+    KSANA_SN_CASE(13, bf16, float, bf16, bf16);   // sublayer output into the 32-bit stream
+    KSANA_SN_CASE(15, bf16, bf16, bf16, bf16);
     default: return -1;
   }
-#undef KSANA_LN_CASE
+#undef KSANA_SN_CASE
 }
 
+// residual (may be null) += x, and its LayerNorm
+KSANA_API int ksana_layer_norm(const void* x, int ldx, void* residual, int ldr, const void* w, const void* b, void* out,
+                               int ldo, int rows, int H, float eps, int kinds, cudaStream_t st) {
+  return ksana_stream_norm(x, ldx, residual, residual, ldr, w, b, out, ldo, rows, H, eps, kinds, 1, nullptr, nullptr,
+                           nullptr, nullptr, nullptr, 0, st);
+}
+
+// pos_table may be null (no learned positions); both tables have storage type `kind`.
 KSANA_API int ksana_embedding_f32(const int* ids, const void* table, float* out, int rows, int H, int vocab, float scale,
-                                  int kind, cudaStream_t st) {
+                                  const int* positions, const void* pos_table, int pos_rows, int kind,
+                                  cudaStream_t st) {
   if (rows <= 0) return 0;
   dim3 grid((H + 255) / 256, rows);
   if (kind)
-    embedding_f32_kernel<<<grid, 256, 0, st>>>(ids, static_cast<const bf16*>(table), out, H, vocab, scale);
+    embedding_f32_kernel<<<grid, 256, 0, st>>>(ids, static_cast<const bf16*>(table), out, H, vocab, scale, positions,
+                                               static_cast<const bf16*>(pos_table), pos_rows);
   else
-    embedding_f32_kernel<<<grid, 256, 0, st>>>(ids, static_cast<const float*>(table), out, H, vocab, scale);
+    embedding_f32_kernel<<<grid, 256, 0, st>>>(ids, static_cast<const float*>(table), out, H, vocab, scale, positions,
+                                               static_cast<const float*>(pos_table), pos_rows);
   return done();
 }
 
@@ -354,6 +469,7 @@ KSANA_API int ksana_qk_norm_cache(void* q, int ldq, const void* k, int ldk, cons
   const int esz = kind ? 2 : 4;
   const bool vec = !((ldq | ldk | ldv | d | dv) & 3) && aligned(q, 4 * esz) && aligned(k, 4 * esz) &&
                    aligned(v, 4 * esz) && aligned(cache, 4 * esz);
+  if (!qw) h = 0;
   const long long units = static_cast<long long>(tokens) * (h + 2 * hk);
   const unsigned grid = static_cast<unsigned>((units + 7) / 8);
 #define KSANA_QK(T, N)                                                                                              \
@@ -366,6 +482,28 @@ KSANA_API int ksana_qk_norm_cache(void* q, int ldq, const void* k, int ldk, cons
     if (vec) KSANA_QK(float, 4); else KSANA_QK(float, 1);
   }
 #undef KSANA_QK
+  return done();
+}
+
+// k: [tokens, hk * d] or null (hk 0: nothing to append); u: [tokens, I or 2 I] or null (I 0: no activation), both inside
+// rows of pitch ldx. The cache holds keys alone.
+KSANA_API int ksana_append_act(const void* k, const void* u, int ldx, const int* slots, void* cache, int tokens, int hk,
+                               int d, int bs, void* out, int ldo, int I, int gated, int kind, cudaStream_t st) {
+  const int nk = hk * d;
+  if (tokens <= 0 || nk + I <= 0) return 0;
+  const bool vec = !((ldx | d | I | ldo) & 7) && aligned(k, 16) && aligned(u, 16) &&
+                   aligned(cache, 16) && aligned(out, 16);
+  const int n = vec ? 8 : 1;
+  const dim3 grid(tokens, (nk + I + n * 256 - 1) / (n * 256));
+#define KSANA_AA(T, N)                                                                                             \
+  append_act_kernel<T, N><<<grid, 256, 0, st>>>(static_cast<const T*>(k), static_cast<const T*>(u), ldx, slots,    \
+                                                static_cast<T*>(cache), nk, d, bs, static_cast<T*>(out), ldo, I, gated)
+  if (kind) {
+    if (vec) KSANA_AA(bf16, 8); else KSANA_AA(bf16, 1);
+  } else {
+    if (vec) KSANA_AA(float, 8); else KSANA_AA(float, 1);
+  }
+#undef KSANA_AA
   return done();
 }
 

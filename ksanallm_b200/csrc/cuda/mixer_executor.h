@@ -1,5 +1,6 @@
-// Native forward pass of layers with mixers of their own sizes (windowed attention and / or linear attention, LayerNorm
-// over a 32-bit residual stream, gated FFN), driven from ONE call per step. Mirrored with ctypes on the Python side.
+// Native forward pass of layers with mixers of their own sizes (windowed attention and / or linear attention, a norm over
+// a 32-bit residual stream, a dense or routed FFN behind or beside the mixers), driven from ONE call per step. A layer
+// that runs several times is listed once per run. Mirrored with ctypes on the Python side.
 #pragma once
 #include <cuda_runtime.h>
 
@@ -7,18 +8,28 @@ extern "C" {
 
 struct KsanaMixerLayer {
   // weights, bf16
-  const void* w_in;      // [n_in, H]: attention q, k, v, then linear attention q, k, v, gate
+  const void* w_in;      // [n_in, H]: attention q, k, v, linear attention q, k, v, gate, then a parallel dense FFN's input
   const void* b_in;      // optional bias [n_in]
-  const void* w_out;     // [H, k_out]: attention columns, then linear-attention columns, then zero padding
-  const void* ln2;       // norm before the FFN (null: the layer has none)
+  const void* w_out;     // [H, k_out]: attention columns, linear-attention columns, a parallel dense FFN's, zero padding
+  const void* ln2;       // norm before the FFN (null: the layer has none, or it reads the mixers' norm)
   const void* w_gu;      // [2 I, H] gate rows, then up rows
   const void* w_gu_il;   // optional copy of w_gu, gate / up rows interleaved in groups of 16: prompt-sized steps then run
                          // the activation as the GEMM's epilogue
   const void* w_down;    // [H, I]
   const void* next_ln;   // next layer's first norm, or the final norm
   int n_in, k_out, inter;
+  // FFN beside the mixers: dense of width `inter` inside w_in / w_out, or routed experts (experts > 0)
+  int parallel, gated;
+  int experts, top, expert_inter, router_rows;
+  const void* w_router;         // [router_rows, H], rows from `experts` on are padding
+  const float* b_router;        // optional [experts]
+  const void* w_expert_gu;      // [experts, 2 expert_inter, H]
+  const void* w_expert_down;    // [experts, H, expert_inter]
+  // what the stream takes between this layer and the next norm
+  const float* next_vec;        // optional [H]
+  int next_start;               // add the embedding output
   // softmax attention (h == 0: none)
-  int h, hk, d, dv, window, bias_len;
+  int h, hk, d, dv, window, keep_first, shared_kv, bias_len;
   float scale, attn_out_scale;
   const float* q_norm;
   const float* k_norm;
@@ -34,7 +45,7 @@ struct KsanaMixerLayer {
 };
 
 struct KsanaMixerModel {
-  int hidden, block_size, num_blocks;
+  int hidden, block_size, num_blocks, center;  // center: LayerNorm, else RMS norm
   float eps;
   // scratch for max_tokens rows
   void* in_buf;    // [T, max n_in]
@@ -44,6 +55,18 @@ struct KsanaMixerModel {
   void* act_buf;   // [T, max I]
   void* proj_buf;  // [T, H]
   void* h_buf[2];  // [T, H]
+  // routed experts: [T, max router_rows], [T, max top] (ids, weights), [T max top] (sorted row of a pair, pair of a sorted
+  // row), the sort's counters, and rows in sorted order [T max top, H | 2 I | I | H]
+  float* router_buf;
+  int* expert_ids;
+  float* expert_weights;
+  int* pair_pos;
+  int* pair_src;
+  int* sort_meta;
+  void* rows_buf;
+  void* rows_gu_buf;
+  void* rows_act_buf;
+  void* rows_out_buf;
   float* chunk_buf;
   long long chunk_floats;
   float* gemm_ws;
@@ -61,6 +84,7 @@ struct KsanaMixerStep {
   const int* cu_q;
   const int* kv_lens;
   const int* state_slots;
+  const float* start;    // the embedding output [T, H] (layers with next_start)
   int total_tokens, max_blocks;
   int num_prefill, num_decode, prefill_tokens;
   int max_q_prefill, max_kv_decode;

@@ -135,7 +135,7 @@ moe_route_kernel(const float* __restrict__ logits, int ld, const float* __restri
 }
 
 // ---- counting sort by expert -----------------------------------------------------------------------------------------
-// counts[E_local] must be zero on entry (the scan kernel re-zeroes it for the next call through `cursor`).
+// counts[E_local] must be zero on entry.
 __global__ void moe_count_kernel(const int* __restrict__ ids, int n, int expert_offset, int E_local,
                                  int* __restrict__ counts) {
   const int i = blockIdx.x * blockDim.x + threadIdx.x;
@@ -143,7 +143,7 @@ __global__ void moe_count_kernel(const int* __restrict__ ids, int n, int expert_
   const int e = ids[i] - expert_offset;
   if (e >= 0 && e < E_local) atomicAdd(&counts[e], 1);
 }
-// offsets[e] = exclusive prefix sum of counts, offsets[E_local] = total; cursor[e] = 0; counts[e] = 0.
+// offsets[e] = exclusive prefix sum of counts, offsets[E_local] = total; cursor[e] = 0.
 __global__ void moe_scan_kernel(int* __restrict__ counts, int E_local, int* __restrict__ offsets,
                                 int* __restrict__ cursor) {
   if (threadIdx.x == 0) {
@@ -151,7 +151,6 @@ __global__ void moe_scan_kernel(int* __restrict__ counts, int E_local, int* __re
     for (int e = 0; e < E_local; ++e) {
       offsets[e] = acc;
       acc += counts[e];
-      counts[e] = 0;
       cursor[e] = 0;
     }
     offsets[E_local] = acc;
@@ -175,9 +174,9 @@ __global__ void moe_scatter_kernel(const int* __restrict__ ids, int n, int exper
 // xs[p] = x[row_src[p] / k] for the first offsets[E_local] rows.
 __global__ void moe_gather_kernel(const __nv_bfloat16* __restrict__ x, int ldx, const int* __restrict__ row_src, int k,
                                   const int* __restrict__ offsets, int E_local, __nv_bfloat16* __restrict__ xs, int H) {
-  const int p = blockIdx.y;
+  const int p = blockIdx.x;
   if (p >= offsets[E_local]) return;
-  const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * 8;
   if (c >= H) return;
   const int t = row_src[p] / k;
   *reinterpret_cast<uint4*>(xs + static_cast<size_t>(p) * H + c) =
@@ -396,6 +395,10 @@ moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_co
 
 using namespace ksana;
 
+extern "C" int ksana_moe_sort(const int* ids, int n, int expert_offset, int E, int* offsets, int* pos, int* row_src,
+                              cudaStream_t st);
+static constexpr int SORT_ONE_CTA_MAX = 32768;  // pairs that one CTA sorts faster than three launches
+
 KSANA_API int ksana_moe_route(const float* logits, int ld, const float* bias, int T, int E, int k, int scoring,
                               int norm_topk, int n_group, int topk_group, float routed_scale, int* ids, float* weights,
                               cudaStream_t stream) {
@@ -408,8 +411,9 @@ KSANA_API int ksana_moe_route(const float* logits, int ld, const float* bias, in
 }
 
 // Sorts the T*k (token, slot) pairs by local expert. meta: int workspace of at least 3 * E_local + 2 ints laid out as
-// counts[E_local] (zero on first use, kept zero by the kernel) | offsets[E_local + 1] | cursor[E_local].
-// pos: [T*k] sorted row or -1; row_src: [T*k]; xs: [T*k, H] gathered rows (only the first offsets[E_local] are valid).
+// counts[E_local] | offsets[E_local + 1] | cursor[E_local].
+// pos: [T*k] sorted row or -1; row_src: [T*k]; xs: [T*k, H] gathered rows (only the first offsets[E_local] are valid),
+// or null: sort only.
 KSANA_API int ksana_moe_permute(const void* x, int ldx, const int* ids, int T, int k, int H, int expert_offset,
                                 int E_local, int* meta, int* pos, int* row_src, void* xs, cudaStream_t stream) {
   const int n = T * k;
@@ -418,10 +422,18 @@ KSANA_API int ksana_moe_permute(const void* x, int ldx, const int* ids, int T, i
   int* counts = meta;
   int* offsets = meta + E_local;
   int* cursor = offsets + E_local + 1;
-  moe_count_kernel<<<(n + 255) / 256, 256, 0, stream>>>(ids, n, expert_offset, E_local, counts);
-  moe_scan_kernel<<<1, 32, 0, stream>>>(counts, E_local, offsets, cursor);
-  moe_scatter_kernel<<<(n + 255) / 256, 256, 0, stream>>>(ids, n, expert_offset, E_local, offsets, cursor, pos, row_src);
-  dim3 grid((H / 8 + 255) / 256, n);
+  int rc = -1;
+  if (n <= SORT_ONE_CTA_MAX) rc = ksana_moe_sort(ids, n, expert_offset, E_local, offsets, pos, row_src, stream);
+  if (rc == -1) {
+    if (cudaMemsetAsync(counts, 0, static_cast<size_t>(E_local) * sizeof(int), stream) != cudaSuccess) return -5;
+    moe_count_kernel<<<(n + 255) / 256, 256, 0, stream>>>(ids, n, expert_offset, E_local, counts);
+    moe_scan_kernel<<<1, 32, 0, stream>>>(counts, E_local, offsets, cursor);
+    moe_scatter_kernel<<<(n + 255) / 256, 256, 0, stream>>>(ids, n, expert_offset, E_local, offsets, cursor, pos, row_src);
+  } else if (rc != 0) {
+    return rc;
+  }
+  if (xs == nullptr) return cudaGetLastError() == cudaSuccess ? 0 : -5;
+  dim3 grid(n, (H / 8 + 255) / 256);
   moe_gather_kernel<<<grid, 256, 0, stream>>>(reinterpret_cast<const __nv_bfloat16*>(x), ldx, row_src, k, offsets,
                                               E_local, reinterpret_cast<__nv_bfloat16*>(xs), H);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
@@ -431,7 +443,7 @@ KSANA_API int ksana_moe_permute(const void* x, int ldx, const int* ids, int T, i
 KSANA_API int ksana_moe_grouped_gemm(const void* A, const void* W, void* C, const int* offsets, int E, int max_rows,
                                      int N, int K, cudaStream_t stream) {
   if (max_rows <= 0) return 0;
-  if ((N % G_BN) || (K & 7)) return -1;
+  if ((N & 7) || (K & 7)) return -1;  // (a last tile's columns past N are the next expert's: computed and dropped)
   CUtensorMap tmA, tmB;
   if (make_tmap_2d(&tmA, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, max_rows, K, K, G_BM, G_BK, CU_TENSOR_MAP_SWIZZLE_128B))
     return -2;

@@ -1,8 +1,11 @@
-// Attention over the paged cache of layers with sizes of their own: a sliding window, a learned bias per distance, and
-// key / value heads of different sizes. Scores, softmax and the accumulation are 32-bit.
+// Attention over the paged cache of layers with sizes of their own: a sliding window, first tokens that stay visible
+// behind it, a learned bias per distance, key / value heads of different sizes, or values that are the keys. Scores,
+// softmax and the accumulation are 32-bit.
 //
-// Cache of a layer: [block][keys hk x bs x d | values hk x bs x dv]. bias: [h][bias_len] fp32 (null: none), indexed by
-// the distance between query and key.
+// Cache of a layer: [block][keys hk x bs x d | values hk x bs x dv], the second part only where values are not the keys.
+// bias: [h][bias_len] fp32 (null: none), indexed by the distance between query and key.
+//
+// Query i sees key j when j <= i and (i - j < window or j < keep); window 0: every j <= i.
 #include "host_common.h"
 #include "mixer_common.cuh"
 
@@ -17,13 +20,17 @@ struct WindowAttnArgs {
   const int* cu_q;
   const int* kv_lens;
   const int* seq_of_token;
-  int h, hk, d, dv, bs, window;
+  int h, hk, d, dv, bs, window, keep, shared;  // shared: values are the keys (dv == d)
   float scale;
   const float* bias;
   int bias_len;
   float out_scale;
   void* out;
   int ldo;
+  __host__ __device__ size_t v_off() const { return shared ? 0 : static_cast<size_t>(hk) * bs * d; }
+  __host__ __device__ size_t block_elems() const { return static_cast<size_t>(hk) * bs * (d + (shared ? 0 : dv)); }
+  // oldest key inside the window of the query at `pos`
+  __device__ int window_start(int pos) const { return window > 0 && pos - window + 1 > 0 ? pos - window + 1 : 0; }
 };
 
 // ---- any size, any storage type ---------------------------------------------------------------------------------
@@ -46,17 +53,17 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
   __syncwarp();
   const int* bt = a.block_tables + static_cast<size_t>(b) * a.max_blocks;
   const T* cache = static_cast<const T*>(a.cache);
-  const size_t block_elems = static_cast<size_t>(a.hk) * a.bs * (a.d + a.dv);
-  const size_t v_off = static_cast<size_t>(a.hk) * a.bs * a.d;
+  const size_t block_elems = a.block_elems(), v_off = a.v_off();
   const float* bias = a.bias ? a.bias + static_cast<size_t>(head) * a.bias_len : nullptr;
-  const int lo = a.window > 0 && pos - a.window + 1 > 0 ? pos - a.window + 1 : 0;
+  const int lo = a.window_start(pos);
+  const int kept = min(a.keep, lo), n = kept + pos - lo + 1;  // the visible keys: [0, kept) and [lo, pos]
   float m = -INFINITY, l = 0.f, acc[NV];
 #pragma unroll
   for (int i = 0; i < NV; ++i) acc[i] = 0.f;
-  for (int j0 = lo; j0 <= pos; j0 += 32) {
-    const int j = j0 + lane;
+  for (int i0 = 0; i0 < n; i0 += 32) {
+    const int i = i0 + lane, j = i < kept ? i : lo + i - kept;
     float s = -INFINITY;
-    if (j <= pos) {
+    if (i < n) {
       const T* kp = cache + bt[j / a.bs] * block_elems + (static_cast<size_t>(kh) * a.bs + j % a.bs) * a.d;
       float dot = 0.f;
       for (int c = 0; c < a.d; ++c) dot += sq[c] * to_f(kp[c]);
@@ -65,15 +72,15 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
     }
     const float m_new = fmaxf(m, warp_max(s));
     const float f = expf(m - m_new);
-    const float p = j <= pos ? expf(s - m_new) : 0.f;
+    const float p = i < n ? expf(s - m_new) : 0.f;
     l = l * f + warp_sum(p);
     m = m_new;
 #pragma unroll
     for (int i = 0; i < NV; ++i) acc[i] *= f;
-    const int n = min(32, pos - j0 + 1);
-    for (int u = 0; u < n; ++u) {
+    const int count = min(32, n - i0);
+    for (int u = 0; u < count; ++u) {
       const float pu = __shfl_sync(0xffffffffu, p, u);
-      const int ju = j0 + u;
+      const int ju = i0 + u < kept ? i0 + u : lo + i0 + u - kept;
       const T* vp = cache + bt[ju / a.bs] * block_elems + v_off + (static_cast<size_t>(kh) * a.bs + ju % a.bs) * a.dv;
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
@@ -118,29 +125,35 @@ static int launch_any(const WindowAttnArgs& a, int tok_base, int tokens, cudaStr
 //   softmax         scores + bias in registers; the mask is part of the tile's bias table (one entry per distance,
 //                   -inf outside the window); running max with a lazy rescale of O
 //   O += P V        A = P from TMEM, written over S as two bf16 matrices hi + lo (the weights keep 16 mantissa bits)
-// Tiles start at the block of 128 keys that holds the first row's oldest visible key. Head sizes below DP / DVP are
-// filled up with zeros by TMA.
+// Tiles start at the block of 128 keys that holds the first row's oldest key in the window; the blocks of the kept first
+// tokens ahead of it come first. Where a block holds kept tokens its table has no window cut, and the scores are masked
+// one by one. Head sizes below DP / DVP are filled up with zeros by TMA.
+//
+// SHARED: the values are the keys. Both products read the same tile in shared memory - rows of keys are K-major for
+// Q K^T and MN-major for P V - and the values' room holds a third tile in flight.
 constexpr int WP_PAGE = 16;
 
-template <int DP, int DVP>
+template <int DP, int DVP, bool SHARED>
 struct WindowPrefillSmem {
+  static constexpr int STAGES = SHARED ? 3 : 2;
   static constexpr int Q_BYTES = 128 * DP * 2;
   static constexpr int K_BYTES = 128 * DP * 2;
   static constexpr int V_BYTES = 128 * DVP * 2;
   static constexpr int OFF_K = Q_BYTES;
-  static constexpr int OFF_V = OFF_K + 2 * K_BYTES;
-  static constexpr int OFF_TAB = OFF_V + 2 * V_BYTES;
+  static constexpr int OFF_V = OFF_K + STAGES * K_BYTES;
+  static constexpr int OFF_TAB = OFF_V + (SHARED ? 0 : 2) * V_BYTES;
   static constexpr int OFF_BAR = OFF_TAB + 2 * 256 * 4;
   static constexpr int USED = OFF_BAR + 256 + 1024;
   // at least half of the SM's shared memory: two CTAs would compete for the 512 TMEM columns each of them takes
   static constexpr int TOTAL = USED > 120 * 1024 ? USED : 120 * 1024;
 };
 
-template <int DP, int DVP>
+template <int DP, int DVP, bool SHARED>
 __global__ void __launch_bounds__(160, 1)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, WindowAttnArgs a, int seq_base, unsigned int* err) {
-  using L_ = WindowPrefillSmem<DP, DVP>;
+  using L_ = WindowPrefillSmem<DP, DVP, SHARED>;
+  constexpr int STAGES = L_::STAGES;
   const int b = blockIdx.y + seq_base, head = blockIdx.z, qt = blockIdx.x;
   const int q0 = a.cu_q[b];
   const int q_len = a.cu_q[b + 1] - q0;
@@ -157,8 +170,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   uint8_t* sV = smem + L_::OFF_V;
   float* tab = reinterpret_cast<float*>(smem + L_::OFF_TAB);  // [2][256]
   uint64_t* q_bar = reinterpret_cast<uint64_t*>(smem + L_::OFF_BAR);
-  uint64_t* k_full = q_bar + 1;   // [2]
-  uint64_t* v_full = k_full + 2;  // [2]
+  uint64_t* k_full = q_bar + 1;        // [STAGES]
+  uint64_t* v_full = k_full + STAGES;  // [2]
   uint64_t* s_done = v_full + 2;  // [2]
   uint64_t* p_ready = s_done + 2;
   uint64_t* o_done = p_ready + 1;
@@ -167,8 +180,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 
   if (tid == 0) {
     mbar_init(q_bar, 1);
+    for (int s = 0; s < STAGES; ++s) mbar_init(&k_full[s], 1);
     for (int s = 0; s < 2; ++s) {
-      mbar_init(&k_full[s], 1);
       mbar_init(&v_full[s], 1);
       mbar_init(&s_done[s], 1);
     }
@@ -187,10 +200,11 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   const uint32_t tmem_S = *tmem_holder;       // two buffers of 128 columns
   const uint32_t tmem_O = tmem_S + 256;
 
-  const int first_key = a.window > 0 ? max(0, row_pos - a.window + 1) : 0;
-  const int kt0 = first_key / 128;
+  const int kt0 = a.window_start(row_pos) / 128;
   const int kv_end = min(L, row_pos + 128);
-  const int n = (kv_end + 127) / 128 - kt0;   // >= 1
+  const int n_kept = min(a.keep / 128 + (a.keep % 128 != 0), kt0);  // tiles of kept tokens ahead of the window's
+  const int n = n_kept + (kv_end + 127) / 128 - kt0;  // >= 1
+  auto tile = [&](int i) { return i < n_kept ? i : kt0 + i - n_kept; };
   const int n_pages = (L + WP_PAGE - 1) / WP_PAGE;
   const int* bt = a.block_tables + static_cast<size_t>(b) * a.max_blocks;
 
@@ -198,22 +212,21 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     if ((tid & 31) == 0) {
       int k_loads = 0, v_loads = 0;
       // the pages of tile i of one operand; pages past the sequence repeat its last one (masked keys)
-      auto load = [&](const CUtensorMap& tm, uint8_t* base, int bytes, int halves, uint64_t* bar, int i) {
-        const int st = i & 1;
+      auto load = [&](const CUtensorMap& tm, uint8_t* base, int bytes, int halves, uint64_t* bar, int i, int st) {
         mbar_expect_tx(&bar[st], bytes);
         for (int p = 0; p < 128 / WP_PAGE; ++p) {
-          const int blk = bt[min((kt0 + i) * (128 / WP_PAGE) + p, n_pages - 1)];
+          const int blk = bt[min(tile(i) * (128 / WP_PAGE) + p, n_pages - 1)];
           for (int hf = 0; hf < halves; ++hf)
             tma_load_3d(base + st * bytes + hf * (128 * 128) + p * (WP_PAGE * 128), &tm, &bar[st], hf * 64,
                         kh * WP_PAGE, blk);
         }
       };
-      auto load_k = [&](int i) { load(tmK, sK, L_::K_BYTES, DP / 64, k_full, i); k_loads = i + 1; };
-      auto load_v = [&](int i) { load(tmV, sV, L_::V_BYTES, DVP / 64, v_full, i); v_loads = i + 1; };
+      auto load_k = [&](int i) { load(tmK, sK, L_::K_BYTES, DP / 64, k_full, i, i % STAGES); k_loads = i + 1; };
+      auto load_v = [&](int i) { load(tmV, sV, L_::V_BYTES, DVP / 64, v_full, i, i & 1); v_loads = i + 1; };
       auto issue_qk = [&](int i) {
         tc_fence_after();
         constexpr uint32_t idesc = umma_idesc(128, 128, 1, 1);
-        const uint32_t kb = smem_u32(sK + (i & 1) * L_::K_BYTES), qb = smem_u32(sQ);
+        const uint32_t kb = smem_u32(sK + (i % STAGES) * L_::K_BYTES), qb = smem_u32(sQ);
 #pragma unroll
         for (int k = 0; k < DP / 16; ++k) {
           const uint32_t off = (k >> 2) * (128 * 128) + (k & 3) * 32;
@@ -224,27 +237,30 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       mbar_expect_tx(q_bar, L_::Q_BYTES);
       for (int hf = 0; hf < DP / 64; ++hf) tma_load_3d(sQ + hf * (128 * 128), &tmQ, q_bar, hf * 64, head, q0 + qt * 128);
       load_k(0);
-      load_v(0);
-      if (n > 1) load_k(1);
+      if constexpr (!SHARED) load_v(0);
+      for (int i = 1; i < STAGES && i < n; ++i) load_k(i);
       bool ok = mbar_wait_bounded(q_bar, 0, abort_flag, err) && mbar_wait_bounded(&k_full[0], 0, abort_flag, err);
       if (ok) issue_qk(0);
       for (int i = 0; ok && i < n; ++i) {
         if (i > 0) ok = mbar_wait_bounded(o_done, (i - 1) & 1, abort_flag, err);
         if (!ok) break;
+        if (SHARED && i > 0 && i + 2 < n) load_k(i + 2);  // tile i - 1 has been multiplied twice
         if (i + 1 < n) {
-          load_v(i + 1);
-          ok = mbar_wait_bounded(&k_full[(i + 1) & 1], ((i + 1) >> 1) & 1, abort_flag, err);
+          if constexpr (!SHARED) load_v(i + 1);
+          ok = mbar_wait_bounded(&k_full[(i + 1) % STAGES], ((i + 1) / STAGES) & 1, abort_flag, err);
           if (!ok) break;
           issue_qk(i + 1);
         }
         ok = mbar_wait_bounded(p_ready, i & 1, abort_flag, err);
         if (!ok) break;
-        if (i + 2 < n) load_k(i + 2);  // the keys of tile i have been multiplied
-        ok = mbar_wait_bounded(&v_full[i & 1], (i >> 1) & 1, abort_flag, err);
-        if (!ok) break;
+        if constexpr (!SHARED) {
+          if (i + 2 < n) load_k(i + 2);  // the keys of tile i have been multiplied
+          ok = mbar_wait_bounded(&v_full[i & 1], (i >> 1) & 1, abort_flag, err);
+          if (!ok) break;
+        }
         tc_fence_after();
         constexpr uint32_t idesc = umma_idesc_major(128, DVP, false, true);
-        const uint32_t vb = smem_u32(sV + (i & 1) * L_::V_BYTES), pb = tmem_S + (i & 1) * 128;
+        const uint32_t vb = smem_u32(SHARED ? sK + (i % STAGES) * L_::K_BYTES : sV + (i & 1) * L_::V_BYTES), pb = tmem_S + (i & 1) * 128;
 #pragma unroll
         for (int k = 0; k < 16; ++k)  // hi, then lo
           umma_f16_ts(tmem_O, pb + k * 8, umma_desc_mn128(vb + (k & 7) * (16 * 128), 128 * 128), idesc,
@@ -253,14 +269,12 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       }
       if (!ok) {
         // copies in flight still write to this CTA's memory: give them their (bounded) time before leaving
-        for (int s = 0; s < 2; ++s) {
-          for (int which = 0; which < 2; ++which) {
-            const int cnt = which ? v_loads : k_loads;
-            const int last = cnt - 1 - ((cnt - 1 - s) & 1);
-            if (last < 0) continue;
-            for (int it = 0; it < (1 << 20) && !mbar_try_wait(which ? &v_full[s] : &k_full[s], (last >> 1) & 1); ++it) {}
-          }
-        }
+        auto drain = [](uint64_t* bar, int stages, int loads) {
+          for (int i = max(loads - stages, 0); i < loads; ++i)
+            for (int it = 0; it < (1 << 20) && !mbar_try_wait(&bar[i % stages], (i / stages) & 1); ++it) {}
+        };
+        drain(k_full, STAGES, k_loads);
+        drain(v_full, 2, v_loads);
       }
     }
     __syncwarp();
@@ -268,17 +282,20 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     const uint32_t lane_off = static_cast<uint32_t>(warp * 32) << 16;
     const float scale2 = a.scale * 1.4426950408889634f;
     const float* bias = a.bias ? a.bias + static_cast<size_t>(head) * a.bias_len : nullptr;
-    const int reach = a.window > 0 ? a.window : 0x7fffffff;
+    const int reach = a.window > 0 ? min(a.window, 1 << 30) : 1 << 30;
     float m_ref = -INFINITY, l = 0.f;
     bool ok = true;
     for (int i = 0; i < n; ++i) {
       float* tb = tab + (i & 1) * 256;
-      const int d0 = row_pos - (kt0 + i) * 128 - 127;  // distance of entry 0
+      const int key0 = tile(i) * 128;
+      const int d0 = row_pos - key0 - 127;   // distance of entry 0
+      const int kept = a.keep - key0;        // columns below this one are kept tokens
+      const int cut = kept > 0 ? 1 << 30 : reach;
 #pragma unroll
       for (int e = tid; e < 256; e += 128) {
         const int dist = d0 + e;
         float v = -INFINITY;
-        if (dist >= 0 && dist < reach) v = bias ? bias[min(dist, a.bias_len - 1)] * 1.4426950408889634f : 0.f;
+        if (dist >= 0 && dist < cut) v = bias ? bias[min(dist, a.bias_len - 1)] * 1.4426950408889634f : 0.f;
         tb[e] = v;
       }
       asm volatile("bar.sync 1, 128;" ::: "memory");
@@ -294,6 +311,12 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       for (int c = 0; c < 4; ++c) tmem_ld32(S + c * 32, reinterpret_cast<uint32_t*>(s) + c * 32);
       tmem_wait_ld();
       float m_tile = -INFINITY;
+      if (kept > 0) {
+        const int behind = row_pos + tid - key0 - reach;  // columns up to this one are behind the window
+#pragma unroll
+        for (int j = 0; j < 128; ++j)
+          if (j >= kept && j <= behind) s[j] = -INFINITY;
+      }
 #pragma unroll
       for (int j = 0; j < 128; ++j) {
         s[j] = fmaf(s[j], scale2, tb[tid - j + 127]);
@@ -371,12 +394,12 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   }
 }
 
-template <int DP, int DVP>
+template <int DP, int DVP, bool SHARED = false>
 static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blocks, int seq_base, int num_seqs,
                           int max_q, cudaStream_t st) {
-  using L_ = WindowPrefillSmem<DP, DVP>;
+  using L_ = WindowPrefillSmem<DP, DVP, SHARED>;
   CUtensorMap tq, tk, tv;
-  const uint64_t blk = static_cast<uint64_t>(a.hk) * a.bs * (a.d + a.dv) * 2;
+  const uint64_t blk = a.block_elems() * 2;
   const uint64_t d = a.d, dv = a.dv;
   {
     const uint64_t dims[3] = {d, static_cast<uint64_t>(a.h), static_cast<uint64_t>(total_tokens)};
@@ -391,13 +414,15 @@ static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blo
     const uint64_t str[2] = {d * 2, blk};
     if (make_tmap_nd(&tk, a.cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -3;
   }
-  {
+  if (SHARED) {
+    tv = tk;
+  } else {
     const uint64_t dims[3] = {dv, rows, static_cast<uint64_t>(num_blocks)};
     const uint64_t str[2] = {dv * 2, blk};
-    const void* base = static_cast<const char*>(a.cache) + rows * d * 2;
+    const void* base = static_cast<const char*>(a.cache) + a.v_off() * 2;
     if (make_tmap_nd(&tv, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -3;
   }
-  auto kern = window_prefill_kernel<DP, DVP>;
+  auto kern = window_prefill_kernel<DP, DVP, SHARED>;
   if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
   kern<<<dim3((max_q + 127) / 128, num_seqs, a.h), 160, L_::TOTAL, st>>>(tq, tk, tv, a, seq_base, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
@@ -437,15 +462,17 @@ window_decode_kernel(WindowAttnArgs a, int seq_base, int groups) {
 
   const int t = a.cu_q[b];
   const int pos = a.kv_lens[b] - 1;
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  const int p0 = lo >> 4, pages = (pos >> 4) - p0 + 1;
+  const int lo = a.window_start(pos);
+  const int p0 = lo >> 4;
+  const int n_kept = min((a.keep >> 4) + ((a.keep & 15) != 0), p0);  // pages of kept tokens ahead of the window's
+  const int pages = n_kept + (pos >> 4) - p0 + 1;
   const int per = (pages + splits - 1) / splits;
-  const int first = p0 + split * per, last = min(first + per, p0 + pages);
+  const int first = split * per, last = min(first + per, pages);
   const int* bt = a.block_tables + static_cast<size_t>(b) * a.max_blocks;
   const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(a.cache);
-  const size_t block_elems = static_cast<size_t>(a.hk) * 16 * (a.d + a.dv);
+  const size_t block_elems = a.block_elems();
   const size_t k_off = static_cast<size_t>(kh) * 16 * a.d;
-  const size_t v_off = static_cast<size_t>(a.hk) * 16 * a.d + static_cast<size_t>(kh) * 16 * a.dv;
+  const size_t v_off = a.v_off() + static_cast<size_t>(kh) * 16 * a.dv;
 
   uint32_t qf[2 * KD][4];
   {
@@ -469,7 +496,8 @@ window_decode_kernel(WindowAttnArgs a, int seq_base, int groups) {
     for (int u = 0; u < 4; ++u) o[i][u] = 0.f;
   float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
 
-  for (int pg = first + warp; pg < last; pg += 4) {
+  for (int i = first + warp; i < last; i += 4) {
+    const int pg = i < n_kept ? i : p0 + i - n_kept;
     const __nv_bfloat16* blk = cache + bt[pg] * block_elems;
     uint4 kf[2][KD], vf[4][ND];
 #pragma unroll
@@ -501,7 +529,7 @@ window_decode_kernel(WindowAttnArgs a, int seq_base, int groups) {
         const int key = pg * 16 + nt * 8 + j * 2 + (u & 1);
         const float* bias = (u >> 1) ? bias1 : bias0;
         float s = -INFINITY;
-        if (key >= lo && key <= pos) {
+        if ((key >= lo || key < a.keep) && key <= pos) {
           s = c[nt][u] * scale2;
           if (bias) s = fmaf(bias[min(pos - key, a.bias_len - 1)], 1.4426950408889634f, s);
         }
@@ -628,7 +656,7 @@ static int launch_decode(const WindowAttnArgs& a, int seq_base, int num_seqs, in
   const int smem = static_cast<int>(sizeof(float)) * (4 * g * ND * 64 + 64 + 64 + 32);
   auto kern = window_decode_kernel<KD, ND>;
   if (KSANA_SMEM_ONCE(kern, 4 * 16 * ND * 64 * 4 + 1024) != 0) return -4;
-  const int keys = a.window > 0 && a.window < max_kv ? a.window : max_kv;
+  const int keys = a.window > 0 && a.window < max_kv - a.keep ? a.window + a.keep : max_kv;
   const int pages = keys / 16 + 1;
   const long long base = static_cast<long long>(num_seqs) * a.hk * groups;
   int splits = 1;
@@ -657,15 +685,19 @@ using namespace ksana;
 // take (heads of at most 128 dimensions in multiples of 8, pages of 16 tokens, 16-byte aligned rows).
 KSANA_API int ksana_window_prefill(const void* q, int ldq, int total_tokens, const void* cache, int num_blocks,
                                    const int* block_tables, int max_blocks, const int* cu_q, const int* kv_lens, int h,
-                                   int hk, int d, int dv, int bs, int window, float scale, const float* bias,
-                                   int bias_len, float out_scale, void* out, int ldo, int seq_base, int num_seqs,
-                                   int max_q, cudaStream_t st) {
+                                   int hk, int d, int dv, int bs, int window, int keep, int shared, float scale,
+                                   const float* bias, int bias_len, float out_scale, void* out, int ldo, int seq_base,
+                                   int num_seqs, int max_q, cudaStream_t st) {
   if (num_seqs <= 0 || max_q <= 0) return 0;
+  if (keep < 0 || (shared && d != dv)) return -2;
   if (h % hk || bs != WP_PAGE || d > 128 || dv > 128 || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
       !rows16(out, ldo))
     return -1;
-  WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, scale,
-                   bias, bias_len, out_scale, out, ldo};
+  WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
+                   shared, scale, bias, bias_len, out_scale, out, ldo};
+  if (shared)
+    return d <= 64 ? launch_prefill<64, 64, true>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
+                   : launch_prefill<128, 128, true>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st);
   if (d <= 64)
     return dv <= 64 ? launch_prefill<64, 64>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
                     : launch_prefill<64, 128>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st);
@@ -677,14 +709,15 @@ KSANA_API int ksana_window_prefill(const void* q, int ldq, int total_tokens, con
 // take (d = 32, 64, 96 or 128, dv = 64 or 128, pages of 16 tokens, 16-byte aligned rows).
 KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, const int* block_tables, int max_blocks,
                                   const int* cu_q, const int* kv_lens, int h, int hk, int d, int dv, int bs, int window,
-                                  float scale, const float* bias, int bias_len, float out_scale, void* out, int ldo,
-                                  int seq_base, int num_seqs, int max_kv, cudaStream_t st) {
+                                  int keep, int shared, float scale, const float* bias, int bias_len, float out_scale,
+                                  void* out, int ldo, int seq_base, int num_seqs, int max_kv, cudaStream_t st) {
   if (num_seqs <= 0) return 0;
+  if (keep < 0 || (shared && d != dv)) return -2;
   if (h % hk || bs != 16 || (d & 31) || d > 128 || (dv & 63) || dv > 128 || !rows16(q, ldq) || !rows16(cache, 0) ||
       !rows16(out, ldo))
     return -1;
-  WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, scale,
-                   bias, bias_len, out_scale, out, ldo};
+  WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
+                   shared, scale, bias, bias_len, out_scale, out, ldo};
 #define KSANA_WD(KD) \
   case KD: return dv == 64 ? launch_decode<KD, 1>(a, seq_base, num_seqs, max_kv, st) \
                            : launch_decode<KD, 2>(a, seq_base, num_seqs, max_kv, st)
@@ -701,12 +734,12 @@ KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, con
 // Tokens [tok_base, tok_base + tokens) of the step, whatever sequences they belong to. kind: 0 fp32, 1 bf16.
 KSANA_API int ksana_window_attention_any(const void* q, int ldq, const void* cache, const int* block_tables,
                                          int max_blocks, const int* cu_q, const int* kv_lens, const int* seq_of_token,
-                                         int h, int hk, int d, int dv, int bs, int window, float scale,
-                                         const float* bias, int bias_len, float out_scale, void* out, int ldo,
-                                         int tok_base, int tokens, int kind, cudaStream_t st) {
+                                         int h, int hk, int d, int dv, int bs, int window, int keep, int shared,
+                                         float scale, const float* bias, int bias_len, float out_scale, void* out,
+                                         int ldo, int tok_base, int tokens, int kind, cudaStream_t st) {
   if (tokens <= 0) return 0;
-  if (h % hk) return -1;
-  WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, seq_of_token, h, hk, d, dv, bs, window, scale,
-                   bias, bias_len, out_scale, out, ldo};
+  if (h % hk || keep < 0 || (shared && d != dv)) return -2;
+  WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, seq_of_token, h, hk, d, dv, bs, window, keep,
+                   shared, scale, bias, bias_len, out_scale, out, ldo};
   return kind ? launch_any<__nv_bfloat16>(a, tok_base, tokens, st) : launch_any<float>(a, tok_base, tokens, st);
 }

@@ -617,6 +617,8 @@ class Scheduler {
       if (q_len <= 0) continue;
       if (!cache_->EnsureCapacity(id, s.num_computed + q_len))
         throw std::runtime_error("Scheduler: the cache pool is too small for the given tokens");
+      if (static_cast<int>(s.tokens.size()) >= cfg_.max_token_len)
+        throw std::runtime_error("Scheduler: the given tokens are longer than a sequence may be");
       bool as_decode = s.num_computed > 0 && q_len <= cfg_.decode_token_threshold;
       (as_decode ? decode : prefill).push_back({id, s.num_computed, q_len, 0, 0, as_decode});
     }

@@ -113,8 +113,8 @@ class LLMEngine:
         self.block_size = 64 if self.cfg.use_mla and bm_cfg.block_token_num == 16 else bm_cfg.block_token_num
         # every running sequence of a model with recurrent layers holds a state slot
         self.num_state_slots = (num_state_slots or bs_cfg.max_batch_size) if self.cfg.has_state else 0
-        if self.cfg.has_state:
-            self._check_recurrent(model)
+        if self.cfg.layers:
+            self._check_layered(model)
         if num_blocks is None:
             num_blocks = self._derive_num_blocks(kv_dtype)
         if num_host_blocks is None:
@@ -140,6 +140,8 @@ class LLMEngine:
         sc.max_batch_size = bs_cfg.max_batch_size
         sc.max_step_tokens = bs_cfg.max_step_tokens
         sc.max_token_len = bs_cfg.max_token_len
+        if model.pos_embed is not None:  # every token that is fed needs a row of the table of learned positions
+            sc.max_token_len = min(sc.max_token_len, model.pos_embed.shape[0] + 1)
         sc.max_waiting_queue_len = bs_cfg.max_waiting_queue_len
         sc.waiting_timeout_ms = bs_cfg.waiting_timeout_in_ms
         sc.split_fuse_token_num = bs_cfg.split_fuse_token_num
@@ -214,13 +216,15 @@ class LLMEngine:
         self._dp_arrivals = 0
         self.dp_any_work = True
 
-    def _check_recurrent(self, model) -> None:
-        """What a model with recurrent layers cannot be combined with: all of it splits or re-uses a sequence at
-        places where its state is not kept."""
+    def _check_layered(self, model) -> None:
+        """What a model described layer by layer cannot be combined with: several GPUs, and for one with recurrent layers
+        all that splits or re-uses a sequence at places where its state is not kept."""
         g, cn = self.serving.setting.global_, self.serving.setting.connector
         if self.tp.size > 1 or self._block_sync_group is not None or g.pipeline_para_size > 1 or \
                 g.attn_data_para_size > 1:
-            raise NotImplementedError("models with recurrent layers run on one GPU")
+            raise NotImplementedError("models described layer by layer run on one GPU")
+        if not model.cfg.has_state:
+            return
         if cn.group_role in ("prefill", "decode", "both"):
             raise NotImplementedError("models with recurrent layers do not hand requests over between instances")
         if getattr(model.cfg, "num_register_token", 0):

@@ -39,6 +39,7 @@ class StepInput:
     # host copies of the small per-sequence arrays (kernel launch decisions never sync the device)
     cu_q_host: Optional[np.ndarray] = None
     kv_lens_host: Optional[np.ndarray] = None
+    start: Optional[torch.Tensor] = None  # embedding output [T, H] of a model whose loop adds it again
     # multimodal RoPE: [3, T] (temporal, height, width) positions; None for plain text steps
     mrope_positions: Optional[torch.Tensor] = None
     _mrope_table: Optional[torch.Tensor] = None

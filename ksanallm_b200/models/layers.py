@@ -329,6 +329,7 @@ class MoEFFN:
         self.tp = tp
         self.gate_w = w[prefix + ".gate.weight"]
         self.bias = w.get(prefix + ".gate.e_score_correction_bias")
+        self.logit_bias = w.get(prefix + ".gate.bias")  # on the router logits, ahead of the choice (topk_softmax)
         self.w_gate_up = w.get(prefix + ".experts.up_gate_proj.weight")  # [E_local, 2I, H]
         self.w_down = w.get(prefix + ".experts.down_proj.weight")        # [E_local, H, I]
         # 4-bit group-quantised experts (GPTQ / AWQ checkpoints): packed words [E_local, N, K / 8] + scales / zeros
@@ -387,13 +388,10 @@ class MoEFFN:
         if (ep is not None and h.is_cuda and h.dtype == torch.bfloat16 and self.e_local < c.num_experts and
                 h.shape[0] <= ep.t_cap * ep.size):
             return self._partial_dispatch(h, ep)
-        logits = ops.linear(h.float() if self.gate_w.dtype == torch.float32 else h, self.gate_w)
         if c.moe_router == "llama4":
-            y = self._llama4_experts(h, logits)
+            y = self._llama4_experts(h, ops.linear(h.float() if self.gate_w.dtype == torch.float32 else h, self.gate_w))
         else:
-            ids, wts = ops.moe_route(logits, c.num_experts_per_tok, c.scoring_func, c.norm_topk_prob, c.n_group,
-                                     c.topk_group, c.routed_scaling_factor, self.bias)
-            ids = self._place(ids)
+            ids, wts = self.route(h)
             if self.s_gate_up is not None and self._grouped_fp8(h):
                 # block-scaled fp8 experts: device-side sort + grouped fp8 tcgen05 GEMMs, no host round trip
                 from ..ops import cuda_moe
@@ -410,6 +408,26 @@ class MoEFFN:
                 s = s * g
             y = y + s
         return y
+
+    def route(self, h: torch.Tensor):
+        """Expert ids [T, k] (as the expert kernels count them) and fp32 weights [T, k] of the rows of ``h``."""
+        c = self.cfg
+        if c.scoring_func == "topk_softmax":
+            # softmax over the chosen logits only, which stay in 32-bit
+            ids, wts = ops.moe_topk(ops.linear(h, self.gate_w, None, torch.float32), c.num_experts,
+                                    c.num_experts_per_tok, self.logit_bias)
+        else:
+            logits = ops.linear(h.float() if self.gate_w.dtype == torch.float32 else h, self.gate_w)
+            ids, wts = ops.moe_route(logits, c.num_experts_per_tok, c.scoring_func, c.norm_topk_prob, c.n_group,
+                                     c.topk_group, c.routed_scaling_factor, self.bias)
+        return self._place(ids), wts
+
+    def rows(self, h: torch.Tensor):
+        """The routed sum in the form a norm over the stream takes: (unweighted rows of the experts, the row of every
+        (token, slot) pair, weights [T, k]). Unquantised local experts without a shared one."""
+        ids, wts = self.route(h)
+        y, pos = ops.moe_expert_rows(h, ids, self.w_gate_up, self.w_down)
+        return y, pos, wts
 
     def _grouped_fp8(self, h: torch.Tensor) -> bool:
         ok = getattr(self, "_grouped_fp8_ok", None)
@@ -480,11 +498,7 @@ class MoEFFN:
     def _dp_exchange(self, h: torch.Tensor, ep) -> torch.Tensor:
         """Attention data parallelism: ``h`` holds only this rank's tokens (possibly none); the routed experts are
         reached through the exchange, whose slot stride for this step was agreed by the DP coordinator."""
-        c = self.cfg
-        logits = ops.linear(h.float() if self.gate_w.dtype == torch.float32 else h, self.gate_w)
-        ids, wts = ops.moe_route(logits, c.num_experts_per_tok, c.scoring_func, c.norm_topk_prob, c.n_group,
-                                 c.topk_group, c.routed_scaling_factor, self.bias)
-        ids = self._place(ids)
+        ids, wts = self.route(h)
         kw = dict(getattr(self, "_ep_kw", {}))
         if not kw and (self.s_gate_up is not None or self.q4 is not None):
             kw["experts_fn"] = self._fp8_experts  # quantised local experts over the gathered rows
@@ -506,15 +520,11 @@ class MoEFFN:
         """Expert-parallel path: this rank routes only its own slice of the tokens, sends each row to the ranks
         hosting its experts and gets the weighted outputs back. The result keeps the "partial sum" contract of
         ``partial`` (rows owned by other ranks are zero here), so the reduce that follows is unchanged."""
-        c = self.cfg
         T = h.shape[0]
         per = (T + ep.size - 1) // ep.size
         lo, hi = min(T, ep.rank * per), min(T, (ep.rank + 1) * per)
         mine = h[lo:hi]
-        logits = ops.linear(mine.float() if self.gate_w.dtype == torch.float32 else mine, self.gate_w)
-        ids, wts = ops.moe_route(logits, c.num_experts_per_tok, c.scoring_func, c.norm_topk_prob, c.n_group,
-                                 c.topk_group, c.routed_scaling_factor, self.bias)
-        ids = self._place(ids)
+        ids, wts = self.route(mine)
         y = torch.zeros_like(h)
         if self.shared is not None:
             s = self.shared.down(self.shared.core(h), add_bias=self.tp.rank == 0)

@@ -52,6 +52,15 @@ _RENAMES: Dict[str, List[Tuple[str, str]]] = {
                 (r"^l(\d+)\.norm2$", r"model.layers.\1.post_attention_layernorm.weight"),
                 (r"^l(\d+)\.mix\.", r"model.layers.\1.mixer."),
                 (r"^l(\d+)\.mlp\.(gate|up|down)$", r"model.layers.\1.mlp.\2_proj.weight")],
+    "givirax": [(r"^embed$", "model.embed_tokens.weight"), (r"^pos$", "model.embed_positions.weight"),
+                (r"^loop\.step$", "model.loop.step"), (r"^final\.norm$", "model.norm.weight"),
+                (r"^head$", "lm_head.weight"),
+                (r"^l(\d+)\.norm1$", r"model.layers.\1.input_layernorm.weight"),
+                (r"^l(\d+)\.mix\.", r"model.layers.\1.mixer."),
+                (r"^l(\d+)\.mlp\.(up|down)$", r"model.layers.\1.mixer.ff.\2"),
+                (r"^l(\d+)\.mlp\.e(\d+)\.(gate|up|down)$", r"model.layers.\1.mlp.experts.\2.\3_proj.weight"),
+                (r"^l(\d+)\.mlp\.router$", r"model.layers.\1.mlp.gate.weight"),
+                (r"^l(\d+)\.mlp\.router\.b$", r"model.layers.\1.mlp.gate.bias")],
     "baichuan": [(r"\.W_pack\.", ".wpack.")],
     "chatglm": [(r"^transformer\.embedding\.word_embeddings\.", "model.embed_tokens."),
                 (r"^transformer\.encoder\.layers\.", "model.layers."),
@@ -142,6 +151,10 @@ def synthetic_checkpoint(cfg: ModelConfig, seed: int = 0, std: float = 0.02, dev
 
     H, d = cfg.hidden_size, cfg.head_dim
     yield "model.embed_tokens.weight", rnd(cfg.vocab_size, H)
+    if cfg.layers and cfg.position_encoding == "learned":
+        yield "model.embed_positions.weight", rnd(cfg.max_position_embeddings, H)
+    if cfg.loop is not None:
+        yield "model.loop.step", rnd(cfg.loop.times, H)
     n_total = cfg.num_layers + cfg.num_nextn_predict_layers
     for i in range(n_total):
         p = f"model.layers.{i}"
@@ -391,7 +404,7 @@ def mixer_parts(spec: LayerSpec) -> set:
     pa, pl = mixer_prefixes(spec)
     need = set()
     if spec.attn is not None:
-        need |= {pa + x for x in "qkvo"}
+        need |= {pa + x for x in ("qko" if spec.attn.shared_kv else "qkvo")}
         if spec.attn.qkv_bias:
             need |= {f"{pa}{x}.b" for x in "qkv"}
         if spec.attn.qk_norm:
@@ -402,6 +415,8 @@ def mixer_parts(spec: LayerSpec) -> set:
         need |= {pl + x for x in "qkvgo"}
         if spec.linear.norm == "concat":
             need.add(pl + "norm")
+    if spec.parallel and spec.ff:  # a dense feed-forward beside the mixers shares their projections
+        need |= {"ff." + x for x in (("gate", "up", "down") if spec.gated else ("up", "down"))}
     return need
 
 
@@ -412,6 +427,8 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
     if spec.attn is not None:
         a = spec.attn
         for x, n in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)):
+            if x == "v" and a.shared_kv:
+                continue
             yield m + pa + x, rnd(n, H)
             if a.qkv_bias:
                 yield f"{m}{pa}{x}.b", rnd(n)
@@ -428,8 +445,23 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
         if r.norm == "concat":
             yield m + pl + "norm", ones(r.heads * r.vdim)
         yield m + pl + "o", rnd(H, r.heads * r.vdim)
-    if spec.ff:
+    if spec.ff and spec.parallel:
+        for x in ("gate", "up") if spec.gated else ("up",):
+            yield f"{m}ff.{x}", rnd(spec.ff, H)
+        yield m + "ff.down", rnd(H, spec.ff)
+        return
+    if spec.has_ff and not spec.parallel:
         yield p + ".post_attention_layernorm.weight", ones(H)
+    if spec.moe is not None:
+        e = spec.moe
+        yield p + ".mlp.gate.weight", rnd(e.experts, H)
+        if e.router_bias:
+            yield p + ".mlp.gate.bias", rnd(e.experts)
+        for i in range(e.experts):
+            yield f"{p}.mlp.experts.{i}.gate_proj.weight", rnd(e.ff, H)
+            yield f"{p}.mlp.experts.{i}.up_proj.weight", rnd(e.ff, H)
+            yield f"{p}.mlp.experts.{i}.down_proj.weight", rnd(H, e.ff)
+    if spec.ff:
         yield p + ".mlp.gate_proj.weight", rnd(spec.ff, H)
         yield p + ".mlp.up_proj.weight", rnd(spec.ff, H)
         yield p + ".mlp.down_proj.weight", rnd(H, spec.ff)
@@ -538,6 +570,13 @@ class WeightLoader:
             self.out[f"{layer_name}.mlp.expert_perm"] = torch.tensor(perm, dtype=torch.int32, device=self.device)
         return perm
 
+    def _num_experts(self, name: str) -> int:
+        """Routed experts of the layer ``name`` belongs to."""
+        if self.cfg.layers:
+            spec = self.cfg.layers[self._layer_of(name + ".")]
+            return spec.moe.experts if spec.moe is not None else 0
+        return self.cfg.num_experts
+
     def _layer_of(self, name: str) -> Optional[int]:
         m = re.match(r"model\.layers\.(\d+)\.", name)
         return int(m.group(1)) if m else None
@@ -612,8 +651,13 @@ class WeightLoader:
         if name == "model.embed_positions.weight":
             self._put(name, t)
             return
+        if name == "model.loop.step":
+            self._put(name, t.float(), keep_dtype=True)
+            return
         if name == "lm_head.weight":
             V = t.shape[0]
+            if cfg.layers:
+                t = torch.nn.functional.pad(t, (0, 0, 0, -V % 8))  # the rows the GEMM takes; logits are cut to the vocabulary
             if n > 1:
                 pad = (-V) % n
                 if pad:
@@ -654,7 +698,7 @@ class WeightLoader:
         if rest in ("experts.gate_up_proj", "experts.down_proj") and t.dim() == 3:
             if self.family == "llama4":
                 t = t.transpose(1, 2)  # Llama 4 keeps [E, in, out] for its batched matmul
-            per = max(cfg.num_experts // self.ep_size, 1)
+            per = max(self._num_experts(layer) // self.ep_size, 1)
             perm = self._perm_of(layer)
             for le in range(t.shape[0]):
                 e = perm[le] if perm else le  # physical slot of logical expert le
@@ -680,7 +724,7 @@ class WeightLoader:
             perm = self._perm_of(layer)
             if perm:
                 e = perm[e]
-            per = max(cfg.num_experts // self.ep_size, 1)
+            per = max(self._num_experts(layer) // self.ep_size, 1)
             if self.ep_size > 1 and not (self.ep_rank * per <= e < (self.ep_rank + 1) * per):
                 return
             self._experts[key][(e, em.group(2) + "." + em.group(3))] = t
@@ -824,6 +868,8 @@ class WeightLoader:
                                             (self._have(p, pre + "up_proj_t", b) and self._have(p, pre + "down_proj_t", b))))
             if moe:
                 ok = "gate.weight" in p
+                if cfg.layers and cfg.layers[li].moe.router_bias:
+                    ok = ok and "gate.bias" in p
                 if cfg.topk_method == "noaux_tc":
                     ok = ok and "gate.e_score_correction_bias" in p
                 if cfg.num_shared_experts:
@@ -837,7 +883,8 @@ class WeightLoader:
 
     def _maybe_flush_experts(self, key: str) -> None:
         ex = self._experts[key]
-        per = max(self.cfg.num_experts // max(self.ep_size, 1), 1) if self.ep_size > 1 else self.cfg.num_experts
+        experts = self._num_experts(key)
+        per = max(experts // max(self.ep_size, 1), 1) if self.ep_size > 1 else experts
         first = next(iter(ex.values()))
         want = per * 3 * (2 if any(self._fp8(t) for t in ex.values()) else 1)
         if len(ex) >= want:
@@ -870,15 +917,23 @@ class WeightLoader:
         self._expert_pqs.clear()
         self._pending.clear()
         self._experts.clear()
+        if cfg.layers:
+            need = {"model.embed_tokens.weight": True, "model.norm.weight": True,
+                    "lm_head.weight": not cfg.tie_word_embeddings, "model.loop.step": cfg.loop is not None,
+                    "model.embed_positions.weight": cfg.position_encoding == "learned"}
+            missing = [name for name, wanted in need.items() if wanted and name not in self.out]
+            if missing:
+                raise KeyError(f"the checkpoint has no {', '.join(missing)}")
 
     def _finish_mixer(self, key: str, p: Dict[str, torch.Tensor]) -> None:
         """All tensors of a layer's mixers: their input projections become one weight (attention q, k, v, then linear
-        attention q, k, v, gate) and their output projections one, side by side along the input. Both are padded with
-        zeros to the multiples of eight that the GEMM takes."""
+        attention q, k, v, gate, then the input of a dense feed-forward beside them) and their output projections one,
+        side by side along the input. Both are padded with zeros to the multiples of eight that the GEMM takes."""
         spec = self.cfg.layers[self._layer_of(key)]
         pa, pl = mixer_prefixes(spec)
         rows, biases, outs = [], [], []
-        for pre, names, has_bias in ((pa, "qkv", spec.attn is not None and spec.attn.qkv_bias), (pl, "qkvg", False)):
+        shared = spec.attn is not None and spec.attn.shared_kv
+        for pre, names, has_bias in ((pa, "qk" if shared else "qkv", spec.attn is not None and spec.attn.qkv_bias), (pl, "qkvg", False)):
             if pre is None:
                 continue
             for x in names:
@@ -886,6 +941,11 @@ class WeightLoader:
                 rows.append(w)
                 biases.append(p[pre + x + ".b"] if has_bias else torch.zeros(w.shape[0], dtype=w.dtype, device=w.device))
             outs.append(p[pre + "o"])
+        if spec.parallel and spec.ff:
+            for x in ("gate", "up") if spec.gated else ("up",):
+                rows.append(p["ff." + x])
+                biases.append(torch.zeros(spec.ff, dtype=rows[-1].dtype, device=rows[-1].device))
+            outs.append(p["ff.down"])
         pad = torch.nn.functional.pad
         w_in, w_out = torch.cat(rows, 0), torch.cat(outs, 1)
         extra = -w_in.shape[0] % 8
@@ -1016,7 +1076,12 @@ class WeightLoader:
                 if pre + b + ".bias" in p:
                     self._put(f"{key}.{pre}down_proj.bias", p[pre + b + ".bias"])
         if "gate.weight" in p:
-            self._put(f"{key}.gate.weight", p["gate.weight"], keep_dtype=p["gate.weight"].dtype == torch.float32)
+            gate = p["gate.weight"]
+            if cfg.layers:  # (the padding rows are no experts: the router looks at the first ones only)
+                gate = torch.nn.functional.pad(gate, (0, 0, 0, -gate.shape[0] % 8))
+            self._put(f"{key}.gate.weight", gate, keep_dtype=gate.dtype == torch.float32)
+        if "gate.bias" in p:
+            self._put(f"{key}.gate.bias", p["gate.bias"].float(), keep_dtype=True)
         if "gate.e_score_correction_bias" in p:
             self._put(f"{key}.gate.e_score_correction_bias", p["gate.e_score_correction_bias"].float(), keep_dtype=True)
         if "shared_expert_gate.weight" in p:
@@ -1035,6 +1100,14 @@ class WeightLoader:
                 self.out[f"{key}.experts.{name}.zeros"] = self._own(torch.stack([q.zeros for q in qs]).to(self.dtype))
             return
         has_scale = (ids[0], "gate_proj.weight_scale_inv") in ex
+        if self.cfg.layers:
+            want = {(e, x + "_proj.weight") for e in range(self._num_experts(key)) for x in ("gate", "up", "down")}
+            if want - set(ex):
+                raise KeyError(f"{key}: the checkpoint has no experts.{min(want - set(ex))[0]}.{min(want - set(ex))[1]}")
+            extra = -ex[(0, "down_proj.weight")].shape[1] % 8  # zero columns up to the multiple of eight the GEMM takes
+            if extra and not has_scale:
+                pad = torch.nn.functional.pad
+                ex = {(e, x): pad(t, (0, extra) if x[0] == "d" else (0, 0, 0, extra)) for (e, x), t in ex.items()}
         gu = torch.stack([torch.cat((ex[(e, "gate_proj.weight")], ex[(e, "up_proj.weight")]), 0) for e in ids])
         dn = torch.stack([ex[(e, "down_proj.weight")] for e in ids])
         if has_scale:

@@ -1,24 +1,28 @@
 """Layers whose sequence mixers have sizes of their own, described by :class:`LayerSpec`: softmax attention over a
-window with a learned distance bias, and linear attention with a fixed decay per head, alone or side by side.
+window (with a learned distance bias, first tokens that stay visible, or values that are the keys), and linear attention
+with a fixed decay per head, alone or side by side.
 
 Both mixers of a layer read the same normalised input, so their input projections are one GEMM and their outputs go
-into one buffer that a single output projection reads. A layer's cache is the pair (paged keys / values, state pool);
-either is an empty tensor where the layer does not have that mixer.
+into one buffer that a single output projection reads. A dense feed-forward that reads that input too (``parallel``) is
+part of the same two GEMMs. A layer's cache is the pair (paged keys / values, state pool); either is an empty tensor
+where the layer does not have that mixer. A layer that runs several times has one :class:`MixerLayer` per run, over the
+same weights.
 """
 from __future__ import annotations
 
-from typing import Dict, NamedTuple, Optional
+from dataclasses import replace
+from typing import Dict, NamedTuple, Optional, Tuple
 
 import torch
 
 from .. import ops
 from ..config.model_config import AttentionSpec, LayerSpec, LinearAttentionSpec, ModelConfig
 from ..ops import reference as ref
-from .layers import DenseFFN, LinearW
+from .layers import DenseFFN, LinearW, MoEFFN
 
 
 class LayerCache(NamedTuple):
-    kv: torch.Tensor     # [num_blocks, kv_heads * block_size * (dim + vdim)]
+    kv: torch.Tensor     # [num_blocks, kv_heads * block_size * (dim + vdim)], without the values where they are the keys
     state: torch.Tensor  # [num_slots, heads, dim, vdim] fp32
 
 
@@ -46,7 +50,10 @@ class RotaryTables:
 class WindowedAttention:
     def __init__(self, cfg: ModelConfig, spec: AttentionSpec, w: Dict[str, torch.Tensor], prefix: str):
         self.spec, self.eps = spec, cfg.rms_norm_eps
-        self.nq, self.nk, self.nv = spec.heads * spec.dim, spec.kv_heads * spec.dim, spec.kv_heads * spec.vdim
+        self.nq, self.nk = spec.heads * spec.dim, spec.kv_heads * spec.dim
+        self.nv = 0 if spec.shared_kv else spec.kv_heads * spec.vdim
+        if spec.shared_kv and (spec.qk_norm or spec.qkv_bias):
+            raise NotImplementedError("keys that are the values are cached as projected")
         self.rows = self.nq + self.nk + self.nv
         self.width = spec.heads * spec.vdim
         self.q_norm, self.k_norm = w.get(prefix + ".q_norm"), w.get(prefix + ".k_norm")
@@ -54,19 +61,26 @@ class WindowedAttention:
         self.bias: Optional[torch.Tensor] = None  # [heads, reach]: the bias of every distance a query can see
 
     def reserve(self, length: int) -> None:
-        reach = min(self.spec.window or length, length)
+        reach = length if self.spec.keep_first else min(self.spec.window or length, length)
         if self.rel is not None and (self.bias is None or self.bias.shape[1] < reach):
             self.bias = ref.distance_bias(self.rel, self.spec.bias_max, reach)
 
-    def run(self, x: torch.Tensor, meta, kv: torch.Tensor, out: torch.Tensor) -> None:
-        """x [T, rows] = the projected (q | k | v); writes heads * vdim columns of ``out``."""
-        s, T = self.spec, x.shape[0]
+    def run(self, x: torch.Tensor, meta, kv: torch.Tensor, out: torch.Tensor,
+            ff: Optional[Tuple[torch.Tensor, torch.Tensor, bool]] = None) -> None:
+        """x [T, rows] = the projected (q | k | v); writes heads * vdim columns of ``out``. ``ff`` = (input, output,
+        gated) of a feed-forward's activation that runs in the launch of the cache append (keys = values only)."""
+        s = self.spec
         q = x[:, :self.nq].unflatten(1, (s.heads, s.dim))
         k = x[:, self.nq:self.nq + self.nk].unflatten(1, (s.kv_heads, s.dim))
-        v = x[:, self.nq + self.nk:].unflatten(1, (s.kv_heads, s.vdim))
-        bs = kv.shape[1] // (s.kv_heads * (s.dim + s.vdim))
-        ops.qk_norm_cache(q, k, v, meta.slot_mapping, kv, bs, self.q_norm, self.k_norm, self.eps)
-        ops.window_attention(q, kv, meta, bs, s.kv_heads, s.vdim, s.scale, s.window, self.bias, s.out_scale, out)
+        bs = kv.shape[1] // (self.nk + self.nv)
+        if s.shared_kv:
+            u, act, gated = ff if ff is not None else (None, None, False)
+            ops.append_act(k, u, meta.slot_mapping, kv, bs, act, gated)
+        else:
+            v = x[:, self.nq + self.nk:].unflatten(1, (s.kv_heads, s.vdim))
+            ops.qk_norm_cache(q, k, v, meta.slot_mapping, kv, bs, self.q_norm, self.k_norm, self.eps)
+        ops.window_attention(q, kv, meta, bs, s.kv_heads, s.vdim, s.scale, s.window, self.bias, s.out_scale, out,
+                             s.keep_first)
 
 
 class DecayedLinearAttention:
@@ -93,29 +107,53 @@ class DecayedLinearAttention:
         ops.gated_norm(o, g, self.norm, self.eps, s.gate, s.out_scale, out)
 
 
-class MixerLayer:
-    """x <- x + mixers(norm1(x)); x <- x + ff(norm2(x)) unless the layer has no feed-forward."""
+class PassStart(NamedTuple):
+    """What the stream takes ahead of one pass of a loop."""
+    step: torch.Tensor      # [H] fp32, the pass's learned vector
+    add_start: bool         # also the embedding output: every pass but the first
 
-    def __init__(self, cfg: ModelConfig, w: Dict[str, torch.Tensor], idx: int, tp, tables: RotaryTables):
+
+class MixerLayer:
+    """One run of a layer: x <- x + mixers(norm1(x)); x <- x + ff(norm2(x)) unless the layer has no feed-forward; or, in
+    parallel, h = norm1(x); x <- x + (mixers(h) + ff(h))."""
+
+    def __init__(self, cfg: ModelConfig, w: Dict[str, torch.Tensor], idx: int, tp, tables: RotaryTables,
+                 number: Optional[int] = None):
+        """``number``: this run starts that pass of the loop."""
         if tp.size > 1:
-            raise NotImplementedError("models with recurrent layers run on one GPU (tensor_para_size 1)")
+            raise NotImplementedError("models described layer by layer run on one GPU (tensor_para_size 1)")
         p = f"model.layers.{idx}"
         spec: LayerSpec = cfg.layers[idx]
         self.cfg, self.tp, self.idx, self.spec = cfg, tp, idx, spec
-        self.is_moe = False
+        self.is_moe = spec.moe is not None
+        self.pass_start = PassStart(w["model.loop.step"][number].contiguous(), number > 0) if number is not None else None
         self.ln1, self.ln1_b = w[p + ".input_layernorm.weight"], None
         self.ln2, self.ln2_b = w.get(p + ".post_attention_layernorm.weight"), None
         self.in_proj, self.o_proj = LinearW(w, p + ".mixer.in_proj"), LinearW(w, p + ".mixer.o_proj")
         device = self.ln1.device
         self.attn = WindowedAttention(cfg, spec.attn, w, p + ".mixer") if spec.attn else None
         self.linear = DecayedLinearAttention(cfg, spec.linear, w, p + ".mixer", device, tables) if spec.linear else None
-        self.ffn = DenseFFN(cfg, w, p + ".mlp", tp) if spec.ff else None
+        self.ffn = DenseFFN(cfg, w, p + ".mlp", tp) if spec.ff and not spec.parallel else None
+        self.experts = None
+        if spec.moe is not None:
+            m = spec.moe
+            self.experts = MoEFFN(replace(cfg, layers=[], num_experts=m.experts, num_experts_per_tok=m.top,
+                                          moe_intermediate_size=m.ff, scoring_func="topk_softmax",
+                                          num_shared_experts=0), w, p + ".mlp", tp)
+            if m.router_bias and self.experts.logit_bias is None:
+                raise KeyError(f"missing {p}.mlp.gate.bias")
+            if self.experts.q4 is not None or self.experts.s_gate_up is not None:
+                raise NotImplementedError("routed experts of models described layer by layer are not quantised")
+        self.parallel_ff = spec.ff if spec.parallel else 0
+        if self.parallel_ff and (self.linear is not None or self.attn is None or not spec.attn.shared_kv):
+            raise NotImplementedError("a dense feed-forward runs beside attention whose values are its keys")
+        if self.experts is not None and not spec.parallel:
+            raise NotImplementedError("routed experts run beside the mixers")
 
     # ---- per-sequence memory ---------------------------------------------------------------------------------
     def kv_width(self) -> int:
         """Cache elements per token."""
-        a = self.spec.attn
-        return a.kv_heads * (a.dim + a.vdim) if a else 0
+        return self.spec.kv_width
 
     def state_shape(self):
         return self.spec.state_shape or (0, 0, 0)
@@ -125,16 +163,30 @@ class MixerLayer:
             self.attn.reserve(length)
 
     # ---- forward ---------------------------------------------------------------------------------------------
-    def _norm(self, x, wgt, bias, residual):
-        return ops.layer_norm(x, wgt, bias, self.cfg.rms_norm_eps, residual, self.ln1.dtype)
+    def _norm(self, y, wgt, residual, **more):
+        """The stream takes ``y`` (and ``more``); returns the normalised sum."""
+        return ops.stream_norm(y, wgt, self.cfg.rms_norm_eps, self.cfg.norm_type == "layernorm", residual, residual,
+                               self.ln1.dtype, **more)
+
+    def start(self, x: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+        """First layer of the model: (its normalised input, the stream) from the embedding output, which stays as it is."""
+        residual = torch.empty_like(x)
+        h = ops.stream_norm(None, self.ln1, self.cfg.rms_norm_eps, self.cfg.norm_type == "layernorm", x, residual,
+                            self.ln1.dtype, add_vec=self.pass_start.step if self.pass_start else None)
+        return h, residual
 
     def mix(self, h: torch.Tensor, meta, cache: LayerCache) -> torch.Tensor:
         x = self.in_proj(h)
-        widths = [m.width for m in (self.attn, self.linear) if m is not None]
-        K = self.o_proj.in_features
+        widths = [m.width for m in (self.attn, self.linear) if m is not None] + [self.parallel_ff]
+        K, used = self.o_proj.in_features, sum(widths)
         buf = torch.empty(h.shape[0], K, dtype=h.dtype, device=h.device)
-        if K > sum(widths):
-            buf[:, sum(widths):].zero_()  # padding of the output projection's input
+        if K > used:
+            buf[:, used:].zero_()  # padding of the output projection's input
+        if self.parallel_ff:
+            n = self.parallel_ff * (2 if self.spec.gated else 1)
+            ff = (x[:, self.attn.rows:self.attn.rows + n], buf[:, widths[0]:used], self.spec.gated)
+            self.attn.run(x[:, :self.attn.rows], meta, cache.kv, buf[:, :widths[0]], ff)
+            return buf
         row = col = 0
         for m, mem in ((self.attn, cache.kv), (self.linear, cache.state)):
             if m is not None:
@@ -142,13 +194,21 @@ class MixerLayer:
                 row, col = row + m.rows, col + m.width
         return buf
 
-    def forward(self, h: torch.Tensor, residual: torch.Tensor, meta, cache: LayerCache, next_norm, next_norm_b=None):
-        """Same contract as DecoderLayer.forward: consumes the normalised input, returns the next layer's."""
+    def forward(self, h: torch.Tensor, residual: torch.Tensor, meta, cache: LayerCache, next_norm, next_norm_b=None,
+                pass_start: Optional[PassStart] = None):
+        """Same contract as DecoderLayer.forward: consumes the normalised input, returns the next layer's.
+        ``pass_start``: the next run's, if it starts a pass; the embedding output is ``meta.start``."""
         y = self.o_proj(self.mix(h, meta, cache))
         if self.ffn is not None:
-            h = self._norm(y, self.ln2, None, residual)
+            h = self._norm(y, self.ln2, residual)
             y = self.ffn.down(self.ffn.core(h))
         if next_norm is None:
+            assert self.experts is None  # (only a pipeline stage ends without a norm)
             residual.add_(y)
             return residual
-        return self._norm(y, next_norm, next_norm_b, residual)
+        more = {}
+        if self.experts is not None:
+            more["routed"] = self.experts.rows(h)
+        if pass_start is not None:
+            more.update(add_vec=pass_start.step, add_rows=meta.start if pass_start.add_start else None)
+        return self._norm(y, next_norm, residual, **more)

@@ -298,22 +298,28 @@ class DenseExecutor:
 
 class _MixerLayer(ctypes.Structure):
     _fields_ = [(n, P) for n in ("w_in", "b_in", "w_out", "ln2", "w_gu", "w_gu_il", "w_down", "next_ln")] + \
-        [(n, I) for n in ("n_in", "k_out", "inter", "h", "hk", "d", "dv", "window", "bias_len")] + \
+        [(n, I) for n in ("n_in", "k_out", "inter", "parallel", "gated", "experts", "top", "expert_inter",
+                          "router_rows")] + \
+        [(n, P) for n in ("w_router", "b_router", "w_expert_gu", "w_expert_down", "next_vec")] + \
+        [(n, I) for n in ("next_start", "h", "hk", "d", "dv", "window", "keep_first", "shared_kv", "bias_len")] + \
         [("scale", F), ("attn_out_scale", F), ("q_norm", P), ("k_norm", P), ("bias", P), ("kv", P)] + \
         [(n, I) for n in ("lh", "ld", "ldv", "rd", "act", "gate")] + \
         [("key_scale", F), ("lin_out_scale", F), ("decay", P), ("rotary", P), ("norm_w", P), ("state", P)]
 
 
 class _MixerModel(ctypes.Structure):
-    _fields_ = [("hidden", I), ("block_size", I), ("num_blocks", I), ("eps", F), ("in_buf", P), ("mix_buf", P),
-                ("o_buf", P), ("gu_buf", P), ("act_buf", P), ("proj_buf", P), ("h_buf", P * 2), ("chunk_buf", P),
+    _fields_ = [("hidden", I), ("block_size", I), ("num_blocks", I), ("center", I), ("eps", F), ("in_buf", P),
+                ("mix_buf", P), ("o_buf", P), ("gu_buf", P), ("act_buf", P), ("proj_buf", P), ("h_buf", P * 2)] + \
+               [(n, P) for n in ("router_buf", "expert_ids", "expert_weights", "pair_pos", "pair_src", "sort_meta",
+                                 "rows_buf", "rows_gu_buf", "rows_act_buf", "rows_out_buf")] + \
+               [("chunk_buf", P),
                 ("chunk_floats", LL), ("gemm_ws", P), ("gemm_ws_floats", LL), ("gemm_counters", P), ("n_counters", I),
                 ("layers", P)]
 
 
 class _MixerStep(ctypes.Structure):
     _fields_ = [(n, P) for n in ("positions", "slot_mapping", "seq_of_token", "block_tables", "cu_q", "kv_lens",
-                                 "state_slots")] + \
+                                 "state_slots", "start")] + \
         [(n, I) for n in ("total_tokens", "max_blocks", "num_prefill", "num_decode", "prefill_tokens", "max_q_prefill",
                           "max_kv_decode", "one_token", "num_long", "long_tokens")]
 
@@ -336,29 +342,50 @@ class MixerExecutor:
                     layer.ffn.up.bias is not None or layer.ffn.down.bias is not None or not layer.ffn.gated or
                     layer.ffn.act != "gelu_tanh"):
                 return False
+            e = layer.experts
+            if e is not None:
+                H, two_i = model.cfg.hidden_size, e.w_gate_up.shape[1]
+                if e.perm is not None or e._eplb_counts is not None or e.gate_w.dtype != torch.bfloat16 or H % 8 or \
+                        two_i % 16 or any(t.dtype != torch.bfloat16 or not t.is_contiguous()
+                                          for t in (e.gate_w, e.w_gate_up, e.w_down)) or layer.spec.moe.experts > 2048:
+                    return False
         return True
 
     def __init__(self, model):
         self.model = model
         n = len(model.layers)
         self._layers = (_MixerLayer * n)()
-        self._wgu_il = []
+        self._wgu_il = {}
         for i, layer in enumerate(model.layers):
             L = self._layers[i]
             nxt = model.layers[i + 1].ln1 if i + 1 < n else model.norm_w
             L.w_in, L.b_in, L.w_out = _p(layer.in_proj.weight), _p(layer.in_proj.bias), _p(layer.o_proj.weight)
             L.n_in, L.k_out = layer.in_proj.weight.shape[0], layer.o_proj.weight.shape[1]
             L.next_ln = _p(nxt)
+            L.parallel, L.gated = int(layer.spec.parallel), int(layer.spec.gated)
+            if layer.parallel_ff:
+                L.inter = layer.parallel_ff
+            if layer.experts is not None:
+                e, s = layer.experts, layer.spec.moe
+                L.experts, L.top, L.expert_inter = s.experts, s.top, e.w_down.shape[2]
+                L.router_rows, L.w_router, L.b_router = e.gate_w.shape[0], _p(e.gate_w), _p(e.logit_bias)
+                L.w_expert_gu, L.w_expert_down = _p(e.w_gate_up), _p(e.w_down)
+            start = model.layers[i + 1].pass_start if i + 1 < n else None
+            if start is not None:
+                L.next_vec, L.next_start = _p(start.step), int(start.add_start)
             if layer.ffn is not None:
                 L.ln2, L.w_gu, L.w_down = _p(layer.ln2), _p(layer.ffn.up.weight), _p(layer.ffn.down.weight)
                 L.inter = layer.ffn.down.weight.shape[1]
                 if os.environ.get("KSANA_FUSED_SWIGLU", "0") == "1" and L.inter % 16 == 0:  # see DenseExecutor
-                    self._wgu_il.append(kcuda.interleave_gate_up(layer.ffn.up.weight))
-                    L.w_gu_il = _p(self._wgu_il[-1])
+                    key = layer.ffn.up.weight.data_ptr()  # (the runs of a looped layer share one copy)
+                    if key not in self._wgu_il:
+                        self._wgu_il[key] = kcuda.interleave_gate_up(layer.ffn.up.weight)
+                    L.w_gu_il = _p(self._wgu_il[key])
             if layer.attn is not None:
                 a, s = layer.attn, layer.attn.spec
                 L.h, L.hk, L.d, L.dv, L.window = s.heads, s.kv_heads, s.dim, s.vdim, s.window
                 L.scale, L.attn_out_scale = s.scale, s.out_scale
+                L.keep_first, L.shared_kv = s.keep_first, int(s.shared_kv)
                 L.q_norm, L.k_norm = _p(a.q_norm), _p(a.k_norm)
             if layer.linear is not None:
                 a, s = layer.linear, layer.linear.spec
@@ -368,6 +395,7 @@ class MixerExecutor:
                 L.decay, L.norm_w = _p(a.decay), _p(a.norm)
         m = self._m = _MixerModel()
         m.hidden, m.eps = model.cfg.hidden_size, float(model.cfg.rms_norm_eps)
+        m.center = int(model.cfg.norm_type == "layernorm")
         ws = self._ws = kcuda.workspace(model.device)
         m.gemm_ws, m.gemm_ws_floats = _p(ws.gemm_ws), ws.gemm_ws.numel()
         m.gemm_counters, m.n_counters = _p(ws.gemm_counters), ws.gemm_counters.numel()
@@ -385,10 +413,24 @@ class MixerExecutor:
         cap = (max(T, 1024) + 1023) // 1024 * 1024
         L, H = self._layers, self._m.hidden
         cols = [max(max(f(x) for x in L), 8) for f in (
-            lambda x: x.n_in, lambda x: x.k_out, lambda x: x.lh * x.ldv, lambda x: 2 * x.inter, lambda x: x.inter)] + [H] * 3
-        self._bufs = [torch.empty(cap, c, dtype=torch.bfloat16, device=self.model.device) for c in cols]
+            lambda x: x.n_in, lambda x: x.k_out, lambda x: x.lh * x.ldv, lambda x: 0 if x.parallel else 2 * x.inter,
+            lambda x: 0 if x.parallel else x.inter)] + [H] * 3
+        dev = self.model.device
+        self._bufs = [torch.empty(cap, c, dtype=torch.bfloat16, device=dev) for c in cols]
         m = self._m
         m.in_buf, m.mix_buf, m.o_buf, m.gu_buf, m.act_buf, m.proj_buf, m.h_buf[0], m.h_buf[1] = (_p(b) for b in self._bufs)
+        routed = [x for x in L if x.experts]
+        if routed:
+            top = max(x.top for x in routed)
+            self._routed = [torch.empty(cap, max(x.router_rows for x in routed), dtype=torch.float32, device=dev)]
+            self._routed += [torch.empty(cap, top, dtype=t, device=dev)
+                             for t in (torch.int32, torch.float32, torch.int32, torch.int32)]
+            self._routed.append(torch.zeros(3 * max(x.experts for x in routed) + 2, dtype=torch.int32, device=dev))
+            self._routed += [torch.empty(cap * top, c, dtype=torch.bfloat16, device=dev)
+                             for c in (H, max(2 * x.expert_inter for x in routed), max(x.expert_inter for x in routed), H)]
+            for name, b in zip(("router_buf", "expert_ids", "expert_weights", "pair_pos", "pair_src", "sort_meta",
+                                "rows_buf", "rows_gu_buf", "rows_act_buf", "rows_out_buf"), self._routed):
+                setattr(m, name, _p(b))
         self.cap = cap
 
     def _bind(self, caches) -> None:
@@ -421,12 +463,13 @@ class MixerExecutor:
         s.positions, s.slot_mapping, s.seq_of_token = _p(meta.positions), _p(meta.slot_mapping), _p(meta.seq_of_token)
         s.block_tables, s.cu_q, s.kv_lens = _p(meta.block_tables), _p(meta.cu_q), _p(meta.kv_lens)
         s.state_slots, s.total_tokens, s.max_blocks = _p(meta.state_slots), T, meta.max_blocks
+        s.start = _p(meta.start)
         n_pre, n_dec, cu = meta.num_prefill, meta.num_decode, meta.cu_q_host
         s.num_prefill, s.num_decode, s.prefill_tokens = n_pre, n_dec, meta.num_prefill_tokens
         s.max_q_prefill = int((cu[1:n_pre + 1] - cu[:n_pre]).max()) if n_pre else 0
         s.max_kv_decode = int(meta.kv_lens_host[n_pre:].max()) if n_dec else 0
         s.one_token = int(T - s.prefill_tokens == n_dec)
-        s.num_long = long_portions(meta)
+        s.num_long = long_portions(meta) if self.model.cfg.has_state else 0
         s.long_tokens = int(cu[s.num_long])
         if s.num_long:
             need = max((s.long_tokens // 128 + s.num_long) * x.lh * x.ld * x.ldv for x in self._layers)

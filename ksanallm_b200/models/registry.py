@@ -35,6 +35,8 @@ FAMILIES: Dict[str, str] = {
     "kimi_k2": "deepseek_v3 architecture with 384 experts",
     "molopel": "layers of linear attention with fixed decays, alone or beside windowed attention with a learned distance "
                "bias; recurrent state slots, LayerNorm, 32-bit residual, soft-capped logits",
+    "givirax": "attention over a window and the first tokens whose values are its keys, beside a GELU or routed "
+               "feed-forward under one norm; learned positions, looped layers, 32-bit residual",
     "minicpm": "embedding / residual / logit scaling; reranker head",
 }
 

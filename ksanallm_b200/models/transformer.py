@@ -98,7 +98,10 @@ class TransformerModel:
         self.layer_ids = list(layer_range) if layer_range is not None else list(range(cfg.num_layers))
         self.rotary_tables = RotaryTables(self.device)  # of the layers that bring their own rotation
         if cfg.layers:
-            self.layers = [MixerLayer(cfg, weights, i, self.tp, self.rotary_tables) for i in self.layer_ids]
+            if layer_range is not None and len(self.layer_ids) != cfg.num_layers:
+                raise NotImplementedError("models described layer by layer run on one GPU (pipeline_para_size 1)")
+            # one entry per run: a layer inside a loop appears once per pass, with a cache of its own
+            self.layers = [MixerLayer(cfg, weights, i, self.tp, self.rotary_tables, t) for i, t in cfg.layer_runs()]
             self.reserve_positions(min(max_positions or 1, maxp))
         else:
             self.layers = [DecoderLayer(cfg, weights, i, self.tp, self.rope_cache) for i in self.layer_ids]
@@ -176,9 +179,7 @@ class TransformerModel:
     # ---- forward --------------------------------------------------------------------------------
     def embed_tokens(self, meta, refit=None) -> torch.Tensor:
         x = ops.embedding(meta.input_ids, self.embed, self.cfg.emb_scale,
-                          torch.float32 if self.cfg.residual_fp32 else None)
-        if self.pos_embed is not None:
-            x = x + self.pos_embed[meta.positions.long()]
+                          torch.float32 if self.cfg.residual_fp32 else None, meta.positions, self.pos_embed)
         if refit is not None:
             # multimodal: rows of precomputed embeddings replace token embeddings at given positions
             for pos, emb in refit:
@@ -203,9 +204,13 @@ class TransformerModel:
             self.last_residual = residual
             return self._final_norm_only(residual)
         first = layers[0]
-        h = first._norm(x, first.ln1, first.ln1_b, None)
-        if h.data_ptr() == residual.data_ptr():
-            residual = x.clone()
+        if self.cfg.layers:
+            meta.start = x
+            h, residual = first.start(x)
+        else:
+            h = first._norm(x, first.ln1, first.ln1_b, None)
+            if h.data_ptr() == residual.data_ptr():
+                residual = x.clone()
         native = self._native_executor()
         if native is not None and cutoff_layer is None and native.can_run(meta, kv_caches, len(layers)):
             if not residual.is_contiguous():
@@ -218,7 +223,8 @@ class TransformerModel:
         for li, layer in enumerate(layers):
             nxt = layers[li + 1] if li + 1 < len(layers) else None
             nw, nb = (nxt.ln1, nxt.ln1_b) if nxt is not None else (self.norm_w, self.norm_b)
-            h = layer.forward(h, residual, meta, kv_caches[li], nw, nb)
+            more = (nxt.pass_start,) if self.cfg.loop is not None and nxt is not None else ()
+            h = layer.forward(h, residual, meta, kv_caches[li], nw, nb, *more)
             if self.progress is not None:
                 self.progress.record(li)  # parallel.transfer.LayerProgressTracker: KV of layer li may leave now
         self.last_residual = residual
@@ -237,6 +243,9 @@ class TransformerModel:
     def _final_norm_only(self, x):
         if self.norm_w is None:
             return x
+        if self.cfg.layers:
+            return ops.stream_norm(None, self.norm_w, self.cfg.rms_norm_eps, self.cfg.norm_type == "layernorm", x, None,
+                                   self.dtype)
         if self.cfg.norm_type == "layernorm":
             return ops.layer_norm(x, self.norm_w, self.norm_b, self.cfg.rms_norm_eps, None, self.dtype)
         return ops.rms_norm(x, self.norm_w, self.cfg.rms_norm_eps)
@@ -244,9 +253,9 @@ class TransformerModel:
     def compute_logits(self, hidden: torch.Tensor, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
         """fp32 logits for the selected rows; vocab shards are gathered across the TP group."""
         h = hidden if rows is None else hidden.index_select(0, rows.long())
-        if self.cfg.logit_softcap:
-            return ops.softcap(ops.linear(h, self.lm_head, None, torch.float32)[:, :self.cfg.vocab_size],
-                               self.cfg.logit_softcap)
+        if self.cfg.residual_fp32:  # the accumulator of the head leaves unrounded
+            logits = ops.linear(h, self.lm_head, None, torch.float32)[:, :self.cfg.vocab_size]
+            return ops.softcap(logits, self.cfg.logit_softcap) if self.cfg.logit_softcap else logits
         logits = ops.linear(h, self.lm_head)
         if self.tp.size > 1 and self.lm_head.shape[0] < self.cfg.vocab_size:
             logits = self.tp.all_gather(logits, dim=-1)
@@ -259,7 +268,7 @@ class TransformerModel:
         """argmax over the full vocabulary without materialising gathered logits on every rank:
         local (max, index) pairs are exchanged instead (reference: greedy.cu:240-424 +
         common_model.cpp:591-617)."""
-        if self.cfg.logit_softcap:
+        if self.cfg.residual_fp32:
             return ops.argmax(self.compute_logits(hidden, rows))
         h = hidden.index_select(0, rows.long())
         logits = ops.linear(h, self.lm_head).float()

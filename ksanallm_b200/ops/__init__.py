@@ -35,6 +35,13 @@ def layer_norm(x, weight, bias, eps, residual=None, out_dtype=None):
     return ref.layer_norm(x, weight, bias, eps, residual, out_dtype)
 
 
+def stream_norm(x, weight, eps, center, stream_in, stream_out=None, out_dtype=None, add_rows=None, add_vec=None,
+                routed=None):
+    """The 32-bit residual stream takes ``x`` (and more) and is normalised; see ``reference.stream_norm``."""
+    f = _mixer() if stream_in.is_cuda else ref
+    return f.stream_norm(x, weight, eps, center, stream_in, stream_out, out_dtype, add_rows, add_vec, routed)
+
+
 def _library_baseline() -> bool:
     """KSANA_LIBRARY_BASELINE=1 routes dense GEMMs to cuBLAS (torch.matmul): the measured stand-in for the
     reference's cuBLAS + NCCL build, never the default."""
@@ -79,15 +86,18 @@ def gelu_and_mul(x):
 
 
 def activation(x, kind):
+    if x.is_cuda and kind == "gelu_tanh":
+        return _mixer().gelu(x)
     return ref.activation(x, kind)
 
 
-def embedding(ids, table, scale=1.0, out_dtype=None):
-    if ids.is_cuda:
-        if out_dtype is not None:
-            return _mixer().embedding(ids, table, scale, out_dtype)
+def embedding(ids, table, scale=1.0, out_dtype=None, positions=None, pos_table=None):
+    """``pos_table``: learned position vectors, added unscaled."""
+    if ids.is_cuda and out_dtype is not None:
+        return _mixer().embedding(ids, table, scale, out_dtype, positions, pos_table)
+    if ids.is_cuda and pos_table is None:
         return _cuda().embedding(ids, table, scale)
-    return ref.embedding(ids, table, scale, out_dtype)
+    return ref.embedding(ids, table, scale, out_dtype, positions, pos_table)
 
 
 def rope_qknorm_cache(q, k, v, positions, cos_sin, slot_mapping, kv_cache, q_norm_w=None, k_norm_w=None,
@@ -116,13 +126,21 @@ def qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps)
     return f.qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps)
 
 
-def window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out):
-    """Writes heads * vdim columns of ``out`` [T, ...] (a column slice is fine)."""
+def append_act(k, u, slot_mapping, cache, block_size, out, gated=False):
+    """Keys to a cache of keys alone and / or a GELU feed-forward's activation; see ``reference.append_act``."""
+    f = _mixer() if (k if k is not None else u).is_cuda else ref
+    f.append_act(k, u, slot_mapping, cache, block_size, out, gated)
+
+
+def window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out, keep_first=0):
+    """Writes heads * vdim columns of ``out`` [T, ...] (a column slice is fine). Whether the cache holds values of their
+    own or the keys are the values shows in its width."""
     if q.is_cuda:
-        _mixer().window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out)
+        _mixer().window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out,
+                                  keep_first)
         return
     out.copy_(ref.window_attention(q, cache, meta.block_tables, meta.cu_q, meta.kv_lens, block_size, kv_heads, vdim,
-                                   scale, window, bias, out_scale).flatten(1))
+                                   scale, window, bias, out_scale, keep_first).flatten(1))
 
 
 def linear_attention(q, k, v, state, meta, decay, act, rotary, key_scale):
@@ -162,6 +180,20 @@ def moe_route(logits, top_k, scoring="softmax", norm_topk=False, n_group=1, topk
     if logits.is_cuda:
         return _cuda().moe_route(logits, top_k, scoring, norm_topk, n_group, topk_group, routed_scale, correction_bias)
     return ref.moe_route(logits, top_k, scoring, norm_topk, n_group, topk_group, routed_scale, correction_bias)
+
+
+def moe_topk(logits, experts, top_k, bias=None):
+    if logits.is_cuda:
+        from . import cuda_moe
+        return cuda_moe.moe_topk(logits, experts, top_k, bias)
+    return ref.moe_topk(logits, experts, top_k, bias)
+
+
+def moe_expert_rows(x, ids, w_gate_up, w_down):
+    if x.is_cuda:
+        from . import cuda_moe
+        return cuda_moe.expert_pipeline(x, ids, w_gate_up, w_down)
+    return ref.moe_expert_rows(x, ids, w_gate_up, w_down)
 
 
 def moe_experts(x, ids, weights, w_gate_up, w_down, expert_offset=0):

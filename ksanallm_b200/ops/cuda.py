@@ -76,15 +76,21 @@ class _Sig:
     ksana_gemm_bf16_batched = ([P, LL, LL, P, P, LL, LL, I, I, I, I, P], I)
     ksana_mla_rope_append = ([P, LL, I, I, P, P, I, P, I, P, P, P, P, I, I, I, I, I, I, P], I)
     ksana_block_copy = ([P, P, I, P, I, LL, P], I)
+    ksana_stream_norm = ([P, I, P, P, I, P, P, P, I, I, I, F, I, I, P, P, P, P, P, I, P], I)
     ksana_layer_norm = ([P, I, P, I, P, P, P, I, I, I, F, I, P], I)
-    ksana_embedding_f32 = ([P, P, P, I, I, I, F, I, P], I)
+    ksana_embedding_f32 = ([P, P, P, I, I, I, F, P, P, I, I, P], I)
+    ksana_append_act = ([P, P, I, P, P, I, I, I, I, P, I, I, I, I, P], I)
+    ksana_moe_topk = ([P, I, P, I, I, I, P, P, P], I)
+    ksana_moe_sort = ([P, I, I, I, P, P, P, P], I)
+    ksana_moe_gemm_any = ([P, I, P, I, P, P, P, I, I, I, I, I, P], I)
+    ksana_silu_mul_any = ([P, P, I, I, I, P], I)
     ksana_gelu_mul = ([P, I, P, I, I, I, I, P], I)
     ksana_qk_norm_cache = ([P, I, P, I, P, I, P, P, P, P, F, I, I, I, I, I, I, I, P], I)
     ksana_gated_norm = ([P, P, I, P, P, I, I, I, I, F, I, F, I, P], I)
     ksana_softcap = ([P, I, P, I, I, F, P], I)
-    ksana_window_attention_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
-    ksana_window_prefill = ([P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
-    ksana_window_decode = ([P, I, P, P, I, P, P, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
+    ksana_window_attention_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
+    ksana_window_prefill = ([P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
+    ksana_window_decode = ([P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
     ksana_linear_chunk_scratch = ([I, I, I, I, I], LL)
     ksana_linear_chunked = ([P, I, P, I, P, I, P, P, P, P, P, P, P, I, I, F, I, I, I, P, I, I, I, P, P], I)
     ksana_linear_recurrent = ([P, I, P, I, P, I, P, P, P, P, P, P, P, I, I, F, I, I, I, P, I, I, I, I, P], I)

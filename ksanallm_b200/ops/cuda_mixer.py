@@ -31,12 +31,33 @@ def layer_norm(x, weight, bias, eps: float, residual: Optional[torch.Tensor] = N
     return out.view(x.shape)
 
 
-def embedding(ids, table, scale: float, out_dtype) -> torch.Tensor:
+def stream_norm(x, weight, eps: float, center: bool, stream_in, stream_out=None, out_dtype=None, add_rows=None,
+                add_vec=None, routed=None) -> torch.Tensor:
+    T, H = stream_in.shape
+    out = torch.empty(T, H, dtype=out_dtype or stream_in.dtype, device=stream_in.device)
+    y, pos, wts = routed if routed is not None else (None, None, None)
+    assert stream_in.is_contiguous() and (stream_out is None or stream_out.is_contiguous())
+    assert all(t is None or t.is_contiguous() for t in (add_rows, add_vec, y, pos, wts))
+    xk = x if x is not None else y
+    kinds = (_KIND[xk.dtype] if xk is not None else 0) | _KIND[stream_in.dtype] << 1 | _KIND[weight.dtype] << 2 | \
+        _KIND[out.dtype] << 3
+    assert x is None or x.stride(1) == 1
+    _check(lib().ksana_stream_norm(_ptr(x), x.stride(0) if x is not None else 0, _ptr(stream_in), _ptr(stream_out), H,
+                                   _ptr(weight), None, _ptr(out), H, T, H, float(eps), kinds, int(center),
+                                   _ptr(add_rows), _ptr(add_vec), _ptr(y), _ptr(pos), _ptr(wts),
+                                   wts.shape[1] if wts is not None else 0, _stream()), "stream_norm")
+    return out
+
+
+def embedding(ids, table, scale: float, out_dtype, positions=None, pos_table=None) -> torch.Tensor:
     assert out_dtype == torch.float32 and table.is_contiguous()
+    assert pos_table is None or pos_table.is_contiguous() and pos_table.dtype == table.dtype
     T, H = ids.numel(), table.shape[1]
     out = torch.empty(T, H, dtype=torch.float32, device=table.device)
     _check(lib().ksana_embedding_f32(_ptr(ids), _ptr(table), _ptr(out), T, H, table.shape[0], float(scale),
-                                     _KIND[table.dtype], _stream()), "embedding_f32")
+                                     _ptr(positions) if pos_table is not None else None, _ptr(pos_table),
+                                     pos_table.shape[0] if pos_table is not None else 0, _KIND[table.dtype],
+                                     _stream()), "embedding_f32")
     return out
 
 
@@ -46,6 +67,30 @@ def gelu_and_mul(x: torch.Tensor) -> torch.Tensor:
     _check(lib().ksana_gelu_mul(_ptr(x), x.stride(0), _ptr(out), out.stride(0), T, two_i // 2, _KIND[x.dtype],
                                 _stream()), "gelu_mul")
     return out
+
+
+def append_act(k, u, slot_mapping, cache, block_size: int, out, gated: bool = False) -> None:
+    """k and u are column slices of one matrix (or one of them is None)."""
+    T = (k if k is not None else u).shape[0]
+    hk, d = (k.shape[1], k.shape[2]) if k is not None else (0, 8)
+    ld = k.stride(0) if k is not None else u.stride(0)
+    dt = k.dtype if k is not None else u.dtype
+    if k is not None:
+        _packed_heads(k)
+        assert cache.is_contiguous() and cache.dtype == dt
+    if u is not None:
+        assert u.stride(1) == 1 and u.stride(0) == ld and out.stride(1) == 1 and out.dtype == dt
+    cols = 0 if u is None else u.shape[1] // 2 if gated else u.shape[1]
+    _check(lib().ksana_append_act(_ptr(k), _ptr(u), ld, _ptr(slot_mapping), _ptr(cache), T, hk, d, block_size, _ptr(out),
+                                  out.stride(0) if u is not None else 0, cols, int(gated), _KIND[dt], _stream()),
+           "append_act")
+
+
+def gelu(x: torch.Tensor) -> torch.Tensor:
+    x2 = _rows(x)
+    out = torch.empty(x2.shape, dtype=x.dtype, device=x.device)
+    append_act(None, x2, None, None, 1, out)
+    return out.view(x.shape)
 
 
 def _packed_heads(x: torch.Tensor) -> torch.Tensor:
@@ -65,7 +110,7 @@ def qk_norm_cache(q, k, v, slot_mapping, cache, block_size: int, q_norm, k_norm,
 
 
 def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, scale: float, window: int, bias,
-                     out_scale: float, out: torch.Tensor) -> None:
+                     out_scale: float, out: torch.Tensor, keep_first: int = 0) -> None:
     """bf16 prompts take the tensor-core kernel, bf16 single tokens the cache-streaming one; sizes those do not have,
     and fp32, take the general kernel."""
     T, h, d = q.shape
@@ -73,7 +118,9 @@ def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, 
     assert out.stride(1) == 1
     n_pre, n_dec, pre_tokens = meta.num_prefill, meta.num_decode, meta.num_prefill_tokens
     blen = bias.shape[1] if bias is not None else 0
-    sizes = (h, kv_heads, d, vdim, block_size, window, float(scale), _ptr(bias), blen, float(out_scale))
+    shared = int(cache.shape[1] == kv_heads * block_size * d)
+    sizes = (h, kv_heads, d, vdim, block_size, window, keep_first, shared, float(scale), _ptr(bias), blen,
+             float(out_scale))
 
     def general(first: int, count: int) -> None:
         if count:

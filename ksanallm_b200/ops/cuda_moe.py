@@ -30,10 +30,50 @@ def moe_route(logits, top_k, scoring="softmax", norm_topk=False, n_group=1, topk
     return ids, w
 
 
+def moe_topk(logits, experts, top_k, bias=None):
+    """The ``top_k`` largest of the first ``experts`` logits (+ bias) of each token, softmax over just those."""
+    from . import cuda
+    T = logits.shape[0]
+    x = logits if logits.dtype == torch.float32 and logits.stride(1) == 1 else logits.float().contiguous()
+    ids = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
+    w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
+    code = cuda.lib().ksana_moe_topk(cuda._ptr(x), x.stride(0), cuda._ptr(bias), T, experts, top_k, cuda._ptr(ids),
+                                     cuda._ptr(w), cuda._stream())
+    if code == -1:
+        return ref.moe_topk(logits, experts, top_k, bias)
+    cuda._check(code, "moe_topk")
+    return ids, w
+
+
+def _pipeline_any(x, ids, w_gate_up, w_down, expert_offset):
+    """expert_pipeline for fp32, and for sizes the tensor-core GEMM does not take: the same sort, plain GEMMs."""
+    from . import cuda
+    T, H = x.shape
+    k, (E, two_i, _) = ids.shape[1], w_gate_up.shape
+    n, dev, kind = T * k, x.device, 0 if x.dtype == torch.float32 else 1
+    assert w_gate_up.dtype == w_down.dtype == x.dtype and x.stride(1) == 1
+    offsets = torch.empty(E + 1, dtype=torch.int32, device=dev)
+    pos, row_src = (torch.empty(n, dtype=torch.int32, device=dev) for _ in range(2))
+    lib, st, p = cuda.lib(), cuda._stream(), cuda._ptr
+    cuda._check(lib.ksana_moe_sort(p(ids.contiguous()), n, expert_offset, E, p(offsets), p(pos), p(row_src), st),
+                "moe_sort")
+    h1 = torch.empty(n, two_i, dtype=x.dtype, device=dev)
+    cuda._check(lib.ksana_moe_gemm_any(p(x), x.stride(0), p(row_src), k, p(w_gate_up.contiguous()), p(h1), p(offsets), E,
+                                       n, two_i, H, kind, st), "moe_gemm_any(gate_up)")
+    a = torch.empty(n, two_i // 2, dtype=x.dtype, device=dev)
+    cuda._check(lib.ksana_silu_mul_any(p(h1), p(a), n, two_i // 2, kind, st), "silu_mul_any")
+    y = torch.empty(n, H, dtype=x.dtype, device=dev)
+    cuda._check(lib.ksana_moe_gemm_any(p(a), two_i // 2, None, 1, p(w_down.contiguous()), p(y), p(offsets), E, n, H,
+                                       two_i // 2, kind, st), "moe_gemm_any(down)")
+    return y, pos
+
+
 def expert_pipeline(x, ids, w_gate_up, w_down, expert_offset=0):
     """Sort the (token, slot) pairs by local expert and run gate_up -> SiLU*mul -> down on the sorted rows.
     Returns (y [T*k, H] sorted expert outputs, pos [T*k] sorted row of each pair or -1 for non-local experts)."""
     from . import cuda
+    if not supports(x, w_gate_up, w_down):
+        return _pipeline_any(x, ids, w_gate_up, w_down, expert_offset)
     T, H = x.shape
     k = ids.shape[1]
     E_local, two_i, _ = w_gate_up.shape
@@ -66,8 +106,8 @@ def expert_pipeline(x, ids, w_gate_up, w_down, expert_offset=0):
 
 def supports(x, w_gate_up, w_down) -> bool:
     two_i, H = w_gate_up.shape[1], x.shape[1]
-    return (x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and two_i % 128 == 0 and H % 128 == 0 and
-            (two_i // 2) % 8 == 0 and w_gate_up.is_contiguous() and w_down.is_contiguous())
+    return (x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and two_i % 16 == 0 and H % 8 == 0 and
+            w_gate_up.is_contiguous() and w_down.is_contiguous())
 
 
 def moe_experts(x, ids, weights, w_gate_up, w_down, expert_offset=0):

@@ -40,6 +40,33 @@ def layer_norm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tenso
     return y.to(out_dtype or x.dtype)
 
 
+def stream_norm(x: Optional[torch.Tensor], weight: torch.Tensor, eps: float, center: bool, stream_in: torch.Tensor,
+                stream_out: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
+                add_rows: Optional[torch.Tensor] = None, add_vec: Optional[torch.Tensor] = None,
+                routed: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None) -> torch.Tensor:
+    """The residual stream takes a sublayer's output and is normalised for the next one (``center``: LayerNorm without
+    bias, else RMS norm). ``routed`` = (rows, position of every (token, slot) pair among them or -1, weights [T, k]):
+    the weighted rows of routed experts belong to the sublayer's output. ``add_rows`` [T, H] and ``add_vec`` [H] follow.
+    The sum goes to ``stream_out`` (``stream_in`` itself is fine)."""
+    xf = x.float() if x is not None else torch.zeros_like(stream_in, dtype=torch.float32)
+    if routed is not None:
+        y, pos, w = routed
+        p = pos.view(w.shape).long()
+        w = w.masked_fill(p < 0, 0.0)
+        xf = xf + torch.einsum("tk,tkh->th", w, y[p.clamp(min=0)].float())
+    v = stream_in.float() + xf
+    if add_rows is not None:
+        v = v + add_rows
+    if add_vec is not None:
+        v = v + add_vec
+    if stream_out is not None:
+        stream_out.copy_(v)
+        v = stream_out.float()
+    if center:
+        v = v - v.mean(-1, keepdim=True)
+    return (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(out_dtype or stream_in.dtype)
+
+
 # ---- dense linear algebra -------------------------------------------------------------------------
 
 def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
@@ -68,7 +95,7 @@ def activation(x: torch.Tensor, kind: str) -> torch.Tensor:
     xf = x.float()
     if kind in ("gelu", "gelu_python"):
         y = F.gelu(xf)
-    elif kind in ("gelu_new", "gelu_fast", "gelu_pytorch_tanh"):
+    elif kind in ("gelu_new", "gelu_fast", "gelu_pytorch_tanh", "gelu_tanh"):
         y = F.gelu(xf, approximate="tanh")
     elif kind == "relu":
         y = F.relu(xf)
@@ -82,7 +109,12 @@ def activation(x: torch.Tensor, kind: str) -> torch.Tensor:
 
 
 def embedding(ids: torch.Tensor, table: torch.Tensor, scale: float = 1.0,
-              out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
+              out_dtype: Optional[torch.dtype] = None, positions: Optional[torch.Tensor] = None,
+              pos_table: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Scaled token rows (+ the unscaled rows of a table of learned positions)."""
+    if pos_table is not None:
+        y = table[ids.long()].to(out_dtype or table.dtype)
+        return (y if scale == 1.0 else y * scale) + pos_table[positions.long()].to(y.dtype)
     y = table[ids.long()]
     if out_dtype is not None and out_dtype != table.dtype:
         return y.to(out_dtype) * scale
@@ -333,8 +365,12 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_tables: torch
 # ---- layers with mixers of their own sizes: windowed attention with a distance bias, linear attention ---------------
 
 def split_kv_cache(cache: torch.Tensor, hk: int, bs: int, d: int, dv: int) -> Tuple[torch.Tensor, torch.Tensor]:
-    """Views [nb, hk, bs, d] and [nb, hk, bs, dv] of a layer cache [nb, hk * bs * (d + dv)] (keys, then values)."""
+    """Views [nb, hk, bs, d] and [nb, hk, bs, dv] of a layer cache [nb, hk * bs * (d + dv)] (keys, then values), or of a
+    cache of keys alone that are the values too."""
     nb, cut = cache.shape[0], hk * bs * d
+    if cache.shape[1] == cut:
+        K = cache.view(nb, hk, bs, d)
+        return K, K
     return cache[:, :cut].view(nb, hk, bs, d), cache[:, cut:].view(nb, hk, bs, dv)
 
 
@@ -358,6 +394,18 @@ def qk_norm_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, slot_mappin
     V[blk, :, off] = v.to(cache.dtype)
 
 
+def append_act(k: Optional[torch.Tensor], u: Optional[torch.Tensor], slot_mapping: torch.Tensor,
+               cache: Optional[torch.Tensor], block_size: int, out: Optional[torch.Tensor], gated: bool = False) -> None:
+    """New keys k [T, hk, d] go to their slots of a cache of keys alone; out = gelu(u), or gelu(gate) * up of u's two
+    halves (tanh form). Either half of the work may be absent (None)."""
+    if k is not None:
+        slots = slot_mapping.long()
+        K, _ = split_kv_cache(cache, k.shape[1], block_size, k.shape[2], k.shape[2])
+        K[slots // block_size, :, slots % block_size] = k.to(cache.dtype)
+    if u is not None:
+        out.copy_(gelu_and_mul(u) if gated else activation(u, "gelu_tanh"))
+
+
 def distance_bias(rel: torch.Tensor, bias_max: float, count: int) -> torch.Tensor:
     """[heads, count] fp32: the learned bias of every distance 0 .. count - 1. ``rel`` [rows, heads]: the first half of
     the rows belongs to one distance each, the rest to log-spaced ranges that end at ``bias_max``."""
@@ -373,9 +421,10 @@ def distance_bias(rel: torch.Tensor, bias_max: float, count: int) -> torch.Tenso
 
 def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, cu_q: torch.Tensor,
                      kv_lens: torch.Tensor, block_size: int, hk: int, dv: int, scale: float, window: int,
-                     bias: Optional[torch.Tensor], out_scale: float = 1.0) -> torch.Tensor:
-    """Softmax attention of each sequence's new tokens over its newest ``window`` keys (0: all), with a bias per head
-    and distance (``bias`` [h, >= reach], None: none). q [T, h, d]; returns [T, h, dv]."""
+                     bias: Optional[torch.Tensor], out_scale: float = 1.0, keep_first: int = 0) -> torch.Tensor:
+    """Softmax attention of each sequence's new tokens over its newest ``window`` keys (0: all) and its first
+    ``keep_first`` ones, with a bias per head and distance (``bias`` [h, >= reach], None: none). q [T, h, d]; returns
+    [T, h, dv]."""
     T, h, d = q.shape
     K, V = split_kv_cache(cache, hk, block_size, d, dv)
     out = torch.empty(T, h, dv, dtype=q.dtype, device=q.device)
@@ -384,7 +433,7 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
         ql, L = cu[b + 1] - cu[b], kl[b]
         if ql == 0:
             continue
-        lo = max(0, L - ql - window + 1) // block_size * block_size if window else 0
+        lo = max(0, L - ql - window + 1) // block_size * block_size if window and not keep_first else 0
         blocks = block_tables[b, lo // block_size:(L + block_size - 1) // block_size].long()
         kb = K[blocks].permute(1, 0, 2, 3).reshape(hk, -1, d)[:, :L - lo].float().repeat_interleave(group, 0)
         vb = V[blocks].permute(1, 0, 2, 3).reshape(hk, -1, dv)[:, :L - lo].float().repeat_interleave(group, 0)
@@ -394,7 +443,7 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
             s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
         hidden = dist < 0
         if window:
-            hidden = hidden | (dist >= window)
+            hidden = hidden | (dist >= window) & (torch.arange(lo, L, device=q.device) >= keep_first)
         p = torch.softmax(s.masked_fill(hidden.unsqueeze(0), float("-inf")), dim=-1)
         out[cu[b]:cu[b + 1]] = (torch.einsum("hqk,hkd->qhd", p, vb) * out_scale).to(q.dtype)
     return out
@@ -556,6 +605,29 @@ def moe_route(logits: torch.Tensor, top_k: int, scoring: str = "softmax", norm_t
         w = w / w.sum(-1, keepdim=True).clamp_min(1e-20)
     w = w * routed_scale
     return ids.to(torch.int32), w
+
+
+def moe_topk(logits: torch.Tensor, experts: int, top_k: int,
+             bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+    """Router over the first ``experts`` columns of ``logits``: the ``top_k`` largest (after ``bias``) and the softmax
+    over just those. Returns (ids [T, k] int32, weights [T, k] fp32)."""
+    z = logits[:, :experts].float()
+    if bias is not None:
+        z = z + bias.float()
+    top, ids = z.topk(top_k, dim=-1)
+    return ids.to(torch.int32), torch.softmax(top, dim=-1)
+
+
+def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, w_gate_up: torch.Tensor,
+                    w_down: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
+    """The unweighted output of every (token, slot) pair's expert: (rows [T * k, H], the row of each pair)."""
+    k = ids.shape[1]
+    flat = ids.reshape(-1).long()
+    y = torch.empty(flat.numel(), x.shape[1], dtype=x.dtype, device=x.device)
+    for e in flat.unique().tolist():
+        at = (flat == e).nonzero()[:, 0]
+        y[at] = linear(silu_and_mul(linear(x[at // k], w_gate_up[e])), w_down[e])
+    return y, torch.arange(flat.numel(), dtype=torch.int32, device=x.device)
 
 
 def moe_experts(x: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, w_gate_up: torch.Tensor,
