@@ -73,13 +73,14 @@ def append_act(k, u, slot_mapping, cache, block_size: int, out, gated: bool = Fa
     """k and u are column slices of one matrix (or one of them is None)."""
     T = (k if k is not None else u).shape[0]
     hk, d = (k.shape[1], k.shape[2]) if k is not None else (0, 8)
-    ld = k.stride(0) if k is not None else u.stride(0)
+    ld = u.stride(0) if u is not None else k.stride(0)
     dt = k.dtype if k is not None else u.dtype
     if k is not None:
         _packed_heads(k)
         assert cache.is_contiguous() and cache.dtype == dt
     if u is not None:
-        assert u.stride(1) == 1 and u.stride(0) == ld and out.stride(1) == 1 and out.dtype == dt
+        assert u.stride(1) == 1 and (T == 1 or k is None or k.stride(0) == ld)
+        assert out.stride(1) == 1 and out.dtype == dt
     cols = 0 if u is None else u.shape[1] // 2 if gated else u.shape[1]
     _check(lib().ksana_append_act(_ptr(k), _ptr(u), ld, _ptr(slot_mapping), _ptr(cache), T, hk, d, block_size, _ptr(out),
                                   out.stride(0) if u is not None else 0, cols, int(gated), _KIND[dt], _stream()),
