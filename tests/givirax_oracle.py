@@ -93,8 +93,11 @@ def route(logits, top):
     return order, x / x.sum()
 
 
-def moe_ff(h, top, w, p):
+def moe_ff(h, top, w, p, margins=None):
     z = h @ w[p + ".router"].T + w[p + ".router.b"]
+    if margins is not None and top < z.shape[1]:  # how far each token's choice is from another one
+        s = z.sort(-1, descending=True).values
+        margins.append(s[:, top - 1] - s[:, top])
     rows = []
     for t in range(h.shape[0]):
         ids, weights = route(z[t], top)
@@ -102,13 +105,15 @@ def moe_ff(h, top, w, p):
     return torch.stack(rows)
 
 
-def feed_forward(h, mlp, w, p):
-    return dense_ff(h, w, p) if mlp["kind"] == "dense" else moe_ff(h, mlp["router"]["top"], w, p)
+def feed_forward(h, mlp, w, p, margins=None):
+    return dense_ff(h, w, p) if mlp["kind"] == "dense" else moe_ff(h, mlp["router"]["top"], w, p, margins)
 
 
 # ---- whole model ----------------------------------------------------------------------------------------------
-def forward(cfg: dict, w: Dict[str, torch.Tensor], tokens: List[int], residuals: Optional[list] = None):
-    """Logits [n, vocab] of one whole sequence; ``residuals`` collects the stream after every layer run."""
+def forward(cfg: dict, w: Dict[str, torch.Tensor], tokens: List[int], residuals: Optional[list] = None,
+            margins: Optional[list] = None):
+    """Logits [n, vocab] of one whole sequence; ``residuals`` collects the stream after every layer run, ``margins`` how
+    clear each routing decision was."""
     eps = cfg["norm"]["eps"]
     start = embed(tokens, w["embed"], cfg["embedding"]["scale"], w["pos"])
     x = start
@@ -121,7 +126,7 @@ def forward(cfg: dict, w: Dict[str, torch.Tensor], tokens: List[int], residuals:
         h = rms_norm(x, w[f"l{i}.norm1"], eps)
         y = attention_mixer(h, layer["mixer"], w, f"l{i}.mix")
         if layer["mlp"] is not None:
-            y = y + feed_forward(h, layer["mlp"], w, f"l{i}.mlp")
+            y = y + feed_forward(h, layer["mlp"], w, f"l{i}.mlp", margins)
         x = x + y
         if residuals is not None:
             residuals.append(x)
