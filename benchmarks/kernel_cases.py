@@ -11,8 +11,8 @@ each case is small (at most a few GB on the device) and launches its kernel a ha
     python benchmarks/kernel_cases.py mla [B ctx h q_len]     # tcgen05 absorbed-MLA decode over the latent cache
     python benchmarks/kernel_cases.py rmsnorm [T H]
     python benchmarks/kernel_cases.py moe [T E k H I]
-    python benchmarks/kernel_cases.py window_prefill [T h hk d dv window]   # layers with mixers of their own sizes
-    python benchmarks/kernel_cases.py window_decode [B ctx h hk d dv window]
+    python benchmarks/kernel_cases.py window_prefill [T h hk d dv window keep shared]   # layers with mixers of their own sizes
+    python benchmarks/kernel_cases.py window_decode [B ctx h hk d dv window keep shared]
     python benchmarks/kernel_cases.py linear_prefill [T h d dv rotary]
     python benchmarks/kernel_cases.py linear_decode [B h d dv rotary]
     python benchmarks/kernel_cases.py mixer_rows [T H h hk d]
@@ -195,34 +195,34 @@ def case_moe():
                 tflops=round(fl / us / 1e6, 1), frac_of_measured_bf16=round(fl / us / 1e6 / p["bf16_tflops"], 3))
 
 
-def _window_setup(q_lens, kv_lens, h, hk, d, dv, window, prefill):
+def _window_setup(q_lens, kv_lens, h, hk, d, dv, window, prefill, keep=0, shared=0):
     q, _, bt, cu = _attn_setup(q_lens, kv_lens, h, 1)
     q = (torch.randn(cu[-1], h, d, device=DEV) * 0.3).to(torch.bfloat16)
-    cache = (torch.randn(int(bt.max()) + 2, hk * 16 * (d + dv), device=DEV) * 0.3).to(torch.bfloat16)
+    cache = (torch.randn(int(bt.max()) + 2, hk * 16 * (d + (0 if shared else dv)), device=DEV) * 0.3).to(torch.bfloat16)
     T = cu[-1]
     meta = make_step_input([0] * T, [0] * T, [0] * T, cu, kv_lens, bt, num_prefill=prefill, device=DEV)
-    bias = torch.randn(h, window or max(kv_lens), device=DEV)
+    bias = None if shared else torch.randn(h, max(kv_lens) if keep else window or max(kv_lens), device=DEV)
     out = torch.empty(T, h * dv, dtype=torch.bfloat16, device=DEV)
-    return lambda i: cuda_mixer.window_attention(q, cache, meta, 16, hk, dv, d ** -0.5, window, bias, 1.0, out)
+    return lambda i: cuda_mixer.window_attention(q, cache, meta, 16, hk, dv, d ** -0.5, window, bias, 1.0, out, keep)
 
 
 def case_window_prefill():
-    T, h, hk, d, dv, window = args_or([8192, 32, 8, 128, 128, 1024])
-    us = timeit(_window_setup([T], [T], h, hk, d, dv, window, 1), iters=5)
+    T, h, hk, d, dv, window, keep, shared = args_or([8192, 32, 8, 128, 128, 1024, 0, 0])
+    us = timeit(_window_setup([T], [T], h, hk, d, dv, window, 1, keep, shared), iters=5)
     w = min(window or T, T)
     pairs = w * (w + 1) / 2 + (T - w) * w
     fl = 2.0 * h * (d + dv) * pairs
     p = peaks()
-    return dict(kernel="window_prefill", T=T, h=h, hk=hk, d=d, dv=dv, window=window, us=round(us, 1),
+    return dict(kernel="window_prefill", T=T, h=h, hk=hk, d=d, dv=dv, window=window, keep=keep, shared=shared, us=round(us, 1),
                 tflops=round(fl / us / 1e6, 1), frac_of_measured_bf16=round(fl / us / 1e6 / p["bf16_tflops"], 3))
 
 
 def case_window_decode():
-    B, ctx, h, hk, d, dv, window = args_or([128, 4096, 32, 8, 128, 128, 1024])
-    us = timeit(_window_setup([1] * B, [ctx] * B, h, hk, d, dv, window, 0))
-    by = B * min(window or ctx, ctx) * hk * (d + dv) * 2
+    B, ctx, h, hk, d, dv, window, keep, shared = args_or([128, 4096, 32, 8, 128, 128, 1024, 0, 0])
+    us = timeit(_window_setup([1] * B, [ctx] * B, h, hk, d, dv, window, 0, keep, shared))
+    by = B * min(window + keep if window else ctx, ctx) * hk * (d + (0 if shared else dv)) * 2
     p = peaks()
-    return dict(kernel="window_decode", B=B, ctx=ctx, h=h, hk=hk, d=d, dv=dv, window=window, us=round(us, 1),
+    return dict(kernel="window_decode", B=B, ctx=ctx, h=h, hk=hk, d=d, dv=dv, window=window, keep=keep, shared=shared, us=round(us, 1),
                 kv_gb=round(by / 1e9, 3), gbs=round(by / us / 1e3, 1),
                 frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
 
@@ -300,6 +300,30 @@ def case_mixer_rows():
         return x[:, :h * d].unflatten(1, (h, d)), x[:, h * d:(h + hk) * d].unflatten(1, (hk, d)), x[:, (h + hk) * d:].unflatten(1, (hk, d))
     by = T * d * 2 * (2 * h + 4 * hk)
     add("qk_norm_cache", timeit(lambda i: cuda_mixer.qk_norm_cache(*parts(qkv[i % 3]), slots, cache.view(cache.shape[0], -1), 16, wf, wf, 1e-6)), by)
+    # cache append beside a plain GELU feed-forward, routed norm, router and sort
+    keys = torch.zeros((T + 15) // 16, hk * 16 * d, dtype=torch.bfloat16, device=DEV)
+    wide = [bf(T, (h + hk) * d + 4 * H) for _ in range(2)]
+    mixed = torch.empty(T, h * d + 4 * H, dtype=torch.bfloat16, device=DEV)
+    add("append_act", timeit(lambda i: cuda_mixer.append_act(
+        wide[i % 2][:, h * d:(h + hk) * d].unflatten(1, (hk, d)), wide[i % 2][:, (h + hk) * d:], slots, keys, 16,
+        mixed[:, h * d:])), T * (hk * d + 4 * H) * 4)
+    add("stream_norm", timeit(lambda i: cuda_mixer.stream_norm(xs[i % 3], w, 1e-6, False, r32[i % 3], r32[i % 3], torch.bfloat16)), T * H * 12)
+    k, E = 2, 16
+    y2, pos = bf(T * k, H), torch.randperm(T * k, dtype=torch.int32, device=DEV)
+    z = torch.randn(T, E, device=DEV)
+    ids, wts = cuda_moe.moe_topk(z, E, k)
+    add("stream_norm_routed", timeit(lambda i: cuda_mixer.stream_norm(xs[i % 3], w, 1e-6, False, r32[i % 3], r32[i % 3], torch.bfloat16,
+                                                                      routed=(y2, pos, wts))), T * H * (12 + 2 * k))
+    add("stream_norm_pass", timeit(lambda i: cuda_mixer.stream_norm(xs[i % 3], w, 1e-6, False, r32[i % 3], r32[i % 3], torch.bfloat16,
+                                                                    add_rows=r32[(i + 1) % 3], add_vec=r32[0][0])), T * H * 16)
+    comb = bf(T, H)
+    add("moe_combine", timeit(lambda i: cuda.lib().ksana_moe_combine(y2.data_ptr(), pos.data_ptr(), wts.data_ptr(), T, k, H, comb.data_ptr(),
+                                                                      torch.cuda.current_stream().cuda_stream)), T * H * (2 + 2 * k))
+    add("moe_topk", timeit(lambda i: cuda_moe.moe_topk(z, E, k)), T * (E + 2 * k) * 4)
+    add("moe_route", timeit(lambda i: cuda_moe.moe_route(z, k, "softmax", True)), T * (E + 2 * k) * 4)
+    offs, src = torch.empty(E + 1, dtype=torch.int32, device=DEV), torch.empty(T * k, dtype=torch.int32, device=DEV)
+    add("moe_sort", timeit(lambda i: cuda.lib().ksana_moe_sort(ids.data_ptr(), T * k, 0, E, offs.data_ptr(), pos.data_ptr(), src.data_ptr(),
+                                                               torch.cuda.current_stream().cuda_stream)), T * k * 12)
     table = torch.randn(T, d, device=DEV)
     add("rope_cache", timeit(lambda i: cuda.rope_qknorm_cache(*parts(qkv[i % 3]), slots, table, slots, cache, wb, wb, 1e-6)), by)
     return dict(kernel="mixer_rows", T=T, H=H, h=h, hk=hk, d=d, **out)

@@ -1,8 +1,13 @@
-"""Prefill and decode throughput of Molopel at layer sizes of real models, each beside the dense model (Qwen3 blocks: QK
-norm, grouped-query attention, SwiGLU) of the same width, heads and depth whose feed-forward is as wide as makes the
-parameter counts equal. Random weights, bf16, one GPU; every number comes from ``LLMEngine.step()``.
+"""Prefill and decode throughput of the designs described layer by layer, at layer sizes of real models, each beside the
+closest other model of the same width, heads and depth. Random weights, bf16, one GPU; every number comes from
+``LLMEngine.step()``.
 
     python bench.py --throughput molopel
+    python bench.py --throughput givirax
+
+Molopel: beside the dense model (Qwen3 blocks: QK norm, grouped-query attention, SwiGLU) whose feed-forward is as wide as
+makes the parameter counts equal. Givirax (half of its layers run twice): beside Qwen3-MoE blocks, dense and routed in
+turn, as many layers as Givirax has runs, with the same experts and a gated feed-forward of the same number of weights.
 
 prefill: prompts of 4096 tokens, 8192 tokens a step. decode: 128 sequences behind prompts of 1024 tokens, one token each
 per step. Weights and caches are larger than L2, so each step starts cold. CUDA events around the timed steps; the host
@@ -15,7 +20,7 @@ import time
 
 import torch
 
-from ksanallm_b200.config.model_config import model_config_from_dict, molopel_config
+from ksanallm_b200.config.model_config import givirax_config, model_config_from_dict, molopel_config
 from ksanallm_b200.config.schema import parse_serving_config
 from ksanallm_b200.engine.llm_engine import LLMEngine
 from ksanallm_b200.engine.sampling_params import SamplingParams
@@ -25,6 +30,9 @@ from ksanallm_b200.ops import cuda
 
 # width, depth, feed-forward, heads, key / value heads, window
 SIZES = [(2048, 8, 6144, 16, 4, 1024), (4096, 8, 12288, 32, 8, 1024), (8192, 4, 24576, 64, 8, 2048)]
+# width, depth, feed-forward, experts, experts per token, expert width, heads, key / value heads, window
+GIVIRAX_SIZES = [(2048, 8, 8192, 16, 2, 2048, 16, 4, 1024), (4096, 8, 16384, 16, 2, 4096, 32, 8, 1024),
+                 (8192, 4, 32768, 8, 2, 8192, 64, 8, 2048)]
 PROMPT, STEP_TOKENS = 4096, 8192
 BATCH, CONTEXT, DECODE_STEPS = 128, 1024, 40
 
@@ -38,6 +46,15 @@ def dense_config(width, depth, ff, heads, kv_heads):
         model_type="qwen3", hidden_size=width, num_hidden_layers=depth, num_attention_heads=heads,
         num_key_value_heads=kv_heads, head_dim=128, intermediate_size=ff, rms_norm_eps=1e-6, vocab_size=32000,
         max_position_embeddings=8192, torch_dtype="bfloat16", eos_token_id=2, tie_word_embeddings=True))
+
+
+def moe_config(width, depth, ff, experts, top, expert_ff, heads, kv_heads):
+    return model_config_from_dict(dict(
+        model_type="qwen3_moe", hidden_size=width, num_hidden_layers=depth, num_attention_heads=heads,
+        num_key_value_heads=kv_heads, head_dim=128, intermediate_size=ff, moe_intermediate_size=expert_ff,
+        num_experts=experts, num_experts_per_tok=top, norm_topk_prob=True, rms_norm_eps=1e-6, vocab_size=32000,
+        mlp_layer_types=["sparse" if i % 2 else "dense" for i in range(depth)],
+        max_position_embeddings=8192, torch_dtype="bfloat16", eos_token_id=2))
 
 
 def build(cfg):
@@ -113,7 +130,26 @@ def measure(model) -> dict:
     return out
 
 
+def run_givirax() -> None:
+    for width, depth, ff, experts, top, expert_ff, heads, kv, window in GIVIRAX_SIZES:
+        loop = dict(start=depth // 4, stop=depth // 4 + depth // 2, times=2)
+        runs = depth + depth // 2
+        rows = {}
+        # the other model's layers are its own: the kinds of feed-forward follow the order of Givirax' runs
+        for name, cfg in (("givirax", givirax_config(width, depth, ff, experts, top, expert_ff, heads, kv, 128, window, 4, loop)),
+                          ("moe", moe_config(width, runs, ff * 2 // 3 // 128 * 128, experts, top, expert_ff, heads, kv))):
+            model, n = build(cfg)
+            rows[name] = dict(parameters_m=round(n / 1e6), **measure(model))
+            del model
+            torch.cuda.empty_cache()
+        print(json.dumps(dict(metric="throughput", design="givirax", width=width, layers=depth, layer_runs=runs, ff=ff,
+                              experts=experts, top=top, expert_ff=expert_ff, heads=heads, kv_heads=kv, window=window,
+                              keep_first=4, dtype="bf16", data="synthetic", **rows)), flush=True)
+
+
 def run(design: str) -> None:
+    if design == "givirax":
+        return run_givirax()
     assert design == "molopel"
     for width, depth, ff, heads, kv, window in SIZES:
         rows = {}

@@ -32,36 +32,33 @@ struct StreamNormArgs {
   const float* weights;
   int k;
 
-  // N columns of the new stream value of `row`
-  template <int N>
-  __device__ void value(size_t row, int c, float* v) const {
+  // V groups of N columns of the new stream value of `row`, `step` columns apart. Each term is loaded for all groups at
+  // once, so that its loads are in flight together.
+  template <int N, int V>
+  __device__ void value(size_t row, int c0, int step, float (*v)[N]) const {
 #pragma unroll
-    for (int j = 0; j < N; ++j) v[j] = 0.f;
-    if (x) load_n<N>(x + row * ldx + c, v);
-    float f[N];
+    for (int i = 0; i < V; ++i)
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[i][j] = 0.f;
+    auto add = [&](const auto* p, float w) {
+      float f[V][N];
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+        if (c0 + i * step < H) load_n<N>(p + c0 + i * step, f[i]);
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+        if (c0 + i * step < H)
+#pragma unroll
+          for (int j = 0; j < N; ++j) v[i][j] = fmaf(w, f[i][j], v[i][j]);
+    };
+    if (x) add(x + row * ldx, 1.f);
     for (int e = 0; e < k; ++e) {
       const int p = pos[row * k + e];
-      if (p < 0) continue;
-      const float g = weights[row * k + e];
-      load_n<N>(y + static_cast<size_t>(p) * H + c, f);
-#pragma unroll
-      for (int j = 0; j < N; ++j) v[j] = fmaf(g, f[j], v[j]);
+      if (p >= 0) add(y + static_cast<size_t>(p) * H, weights[row * k + e]);
     }
-    if (res_in) {
-      load_n<N>(res_in + row * ldr + c, f);
-#pragma unroll
-      for (int j = 0; j < N; ++j) v[j] += f[j];
-    }
-    if (add_rows) {
-      load_n<N>(add_rows + row * H + c, f);
-#pragma unroll
-      for (int j = 0; j < N; ++j) v[j] += f[j];
-    }
-    if (add_vec) {
-      load_n<N>(add_vec + c, f);
-#pragma unroll
-      for (int j = 0; j < N; ++j) v[j] += f[j];
-    }
+    if (res_in) add(res_in + row * ldr, 1.f);
+    if (add_rows) add(add_rows + row * H, 1.f);
+    if (add_vec) add(add_vec, 1.f);
   }
   template <int N>
   __device__ void keep(size_t row, int c, float* v) const {
@@ -84,11 +81,7 @@ stream_norm_kernel(const StreamNormArgs<X, R, W, O> a) {
   const int H = a.H;
   float v[VPT][4];
   float s = 0.f;
-#pragma unroll
-  for (int i = 0; i < VPT; ++i) {
-    const int c = (i * 256 + threadIdx.x) * 4;
-    if (c < H) a.template value<4>(row, c, v[i]);
-  }
+  a.template value<4, VPT>(row, threadIdx.x * 4, 1024, v);
 #pragma unroll
   for (int i = 0; i < VPT; ++i) {
     const int c = (i * 256 + threadIdx.x) * 4;
@@ -139,11 +132,11 @@ stream_norm_any_kernel(const StreamNormArgs<X, R, W, O> a) {
   const int H = a.H;
   float s = 0.f;
   for (int c = threadIdx.x; c < H; c += 256) {
-    float v;
-    a.template value<1>(row, c, &v);
-    a.template keep<1>(row, c, &v);
-    row_v[c] = v;  // only this thread reads it back
-    s += v;
+    float v[1][1];
+    a.template value<1, 1>(row, c, 0, v);
+    a.template keep<1>(row, c, v[0]);
+    row_v[c] = v[0][0];  // only this thread reads it back
+    s += v[0][0];
   }
   const float mean = a.center ? block_sum(s, red) / static_cast<float>(H) : 0.f;
   float ss = 0.f;

@@ -36,7 +36,7 @@ int ksana_window_prefill(const void* q, int ldq, int total_tokens, const void* c
                          int d, int dv, int bs, int window, int keep, int shared, float scale, const float* bias,
                          int bias_len, float out_scale, void* out, int ldo, int seq_base, int num_seqs, int max_q,
                          cudaStream_t st);
-int ksana_window_decode(const void* q, int ldq, const void* cache, const int* block_tables, int max_blocks,
+int ksana_window_decode(const void* q, int ldq, const void* cache, int num_blocks, const int* block_tables, int max_blocks,
                         const int* cu_q, const int* kv_lens, int h, int hk, int d, int dv, int bs, int window,
                         int keep, int shared, float scale, const float* bias, int bias_len, float out_scale, void* out,
                         int ldo, int seq_base, int num_seqs, int max_kv, cudaStream_t st);
@@ -123,7 +123,7 @@ struct Exec {
     if (s->num_decode > 0) {
       int rc = -1;
       if (s->one_token)
-        rc = ksana_window_decode(x, ld, w.kv, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, w.h, w.hk, w.d, w.dv,
+        rc = ksana_window_decode(x, ld, w.kv, m->num_blocks, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, w.h, w.hk, w.d, w.dv,
                                  m->block_size, w.window, w.keep_first, w.shared_kv, w.scale, w.bias, w.bias_len,
                                  w.attn_out_scale, out, w.k_out, s->num_prefill, s->num_decode, s->max_kv_decode, st);
       if (rc == -1) rc = general(s->prefill_tokens, T - s->prefill_tokens);

@@ -394,71 +394,103 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   }
 }
 
+// The tensor maps of a layer's cache: pages of 16 keys (values) of one head, 64 columns at a time.
+static int cache_maps(const WindowAttnArgs& a, int num_blocks, CUtensorMap* tk, CUtensorMap* tv) {
+  const uint32_t box[3] = {64, WP_PAGE, 1};
+  const uint64_t rows = static_cast<uint64_t>(a.hk) * a.bs, blk = a.block_elems() * 2;
+  for (int which = 0; which < (a.shared ? 1 : 2); ++which) {
+    const uint64_t cols = which ? a.dv : a.d;
+    const uint64_t dims[3] = {cols, rows, static_cast<uint64_t>(num_blocks)};
+    const uint64_t str[2] = {cols * 2, blk};
+    const void* base = static_cast<const char*>(a.cache) + (which ? a.v_off() * 2 : 0);
+    if (make_tmap_nd(which ? tv : tk, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B))
+      return -3;
+  }
+  if (a.shared) *tv = *tk;
+  return 0;
+}
+
 template <int DP, int DVP, bool SHARED = false>
 static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blocks, int seq_base, int num_seqs,
                           int max_q, cudaStream_t st) {
   using L_ = WindowPrefillSmem<DP, DVP, SHARED>;
   CUtensorMap tq, tk, tv;
-  const uint64_t blk = a.block_elems() * 2;
-  const uint64_t d = a.d, dv = a.dv;
   {
-    const uint64_t dims[3] = {d, static_cast<uint64_t>(a.h), static_cast<uint64_t>(total_tokens)};
-    const uint64_t str[2] = {d * 2, static_cast<uint64_t>(a.ldq) * 2};
+    const uint64_t dims[3] = {static_cast<uint64_t>(a.d), static_cast<uint64_t>(a.h), static_cast<uint64_t>(total_tokens)};
+    const uint64_t str[2] = {static_cast<uint64_t>(a.d) * 2, static_cast<uint64_t>(a.ldq) * 2};
     const uint32_t box[3] = {64, 1, 128};
     if (make_tmap_nd(&tq, a.q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -2;
   }
-  const uint32_t box[3] = {64, WP_PAGE, 1};
-  const uint64_t rows = static_cast<uint64_t>(a.hk) * a.bs;
-  {
-    const uint64_t dims[3] = {d, rows, static_cast<uint64_t>(num_blocks)};
-    const uint64_t str[2] = {d * 2, blk};
-    if (make_tmap_nd(&tk, a.cache, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -3;
-  }
-  if (SHARED) {
-    tv = tk;
-  } else {
-    const uint64_t dims[3] = {dv, rows, static_cast<uint64_t>(num_blocks)};
-    const uint64_t str[2] = {dv * 2, blk};
-    const void* base = static_cast<const char*>(a.cache) + a.v_off() * 2;
-    if (make_tmap_nd(&tv, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -3;
-  }
+  if (int rc = cache_maps(a, num_blocks, &tk, &tv)) return rc;
   auto kern = window_prefill_kernel<DP, DVP, SHARED>;
   if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
   kern<<<dim3((max_q + 127) / 128, num_seqs, a.h), 160, L_::TOTAL, st>>>(tq, tk, tv, a, seq_base, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
-// ---- one new token: mma.sync over register-resident pages --------------------------------------------------------------
+// ---- one new token: mma.sync over pages streamed through shared memory --------------------------------------------------
 // One CTA of 4 warps = (sequence, key / value head, split of the visible pages); the splits of a head form a cluster
-// and merge through distributed shared memory. A warp takes one 16-key page at a time: its K and V rows go straight
-// from the cache into MMA fragments with 16-byte loads (dimensions and value columns are permuted the same way on both
-// sides of each product, so no transposition is needed). The rows of the fragments are the query heads that share the
-// key head. The kernel is a stream over the cache; the tensor instructions only keep the arithmetic out of its way.
+// and merge through distributed shared memory. Every warp streams its own 16-key pages: one lane keeps a ring of them
+// in flight with TMA, the warp multiplies. Keys are the rows of the products and the (up to 8 NT) query heads that share
+// the key head their columns:
+//   S^T = K Q^T     16 keys x 8 NT heads, K by ldmatrix
+//   O^T += V^T P^T  V^T by ldmatrix.trans, P^T = P transposed in registers, as two bf16 matrices hi + lo
+// so nothing is computed for more than 8 NT - heads columns of padding. SHARED: values are keys, both products read the
+// same page. Head sizes below DP / DVP are filled up with zeros by TMA. The kernel is a stream over the cache; the tensor
+// instructions only keep the arithmetic out of its way.
 __device__ __forceinline__ void mma_16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
   asm volatile(
       "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
       : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
       : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
 }
+template <bool TRANS>
+__device__ __forceinline__ void ldmatrix_x4(uint32_t* r, uint32_t addr) {
+  if constexpr (TRANS)
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+  else
+    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
+                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
+}
+// an 8 x 8 matrix of 16-bit values held across the warp, transposed
+__device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
+  uint32_t r;
+  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
+  return r;
+}
 
-template <int KD, int ND>  // d = 32 KD, dv = 64 ND
+template <int DP, int DVP, bool SHARED>
+struct WindowDecodeSmem {
+  static constexpr int K_BYTES = 16 * DP * 2;
+  static constexpr int PAGE = K_BYTES + (SHARED ? 0 : 16 * DVP * 2);
+  static constexpr int STAGES = PAGE <= 2048 ? 4 : PAGE <= 4096 ? 3 : 2;
+  static constexpr int RING = 4 * STAGES * PAGE;
+  static constexpr int LDO = DVP + 4;
+  static constexpr int MERGE = 4 * 16 * LDO * 4;  // over the ring, once every page has been multiplied
+  static constexpr int TOTAL = (RING > MERGE ? RING : MERGE) + 1024;
+};
+
+template <int DP, int DVP, int NT, bool SHARED>
 __global__ void __launch_bounds__(128)
-window_decode_kernel(WindowAttnArgs a, int seq_base, int groups) {
-  extern __shared__ float sm[];
+window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_constant__ CUtensorMap tmV, WindowAttnArgs a,
+                     int seq_base, int groups, unsigned int* err) {
+  using L_ = WindowDecodeSmem<DP, DVP, SHARED>;
+  constexpr int STAGES = L_::STAGES, LDO = L_::LDO;
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ uint64_t full[4][STAGES];
+  __shared__ float sM[4][16], sL[4][16], cM[16], cL[16];
+  __shared__ int abort_word;
+  volatile int* abort_flag = &abort_word;
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int splits = gridDim.x, split = blockIdx.x;
   const int kh = blockIdx.y / groups, part = blockIdx.y % groups;
   const int b = blockIdx.z + seq_base;
   const int gq = a.h / a.hk;
   const int head0 = kh * gq + part * 16;
-  const int g = min(16, gq - part * 16);        // query heads of this CTA
+  const int g = min(16, gq - part * 16);        // query heads of this CTA, at most 8 NT
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
-  const int r = lane >> 2, j = lane & 3;
-  constexpr int DV = ND * 64;
-  float* sO = sm;                               // [4][g][DV]
-  float* sM = sO + 4 * g * DV;                  // [4][16]
-  float* sL = sM + 64;                          // [4][16]
-  float* cM = sL + 64;                          // [16] of this CTA
-  float* cL = cM + 16;
+  const int r = lane >> 2, j2 = (lane & 3) * 2;
 
   const int t = a.cu_q[b];
   const int pos = a.kv_lens[b] - 1;
@@ -467,157 +499,216 @@ window_decode_kernel(WindowAttnArgs a, int seq_base, int groups) {
   const int n_kept = min((a.keep >> 4) + ((a.keep & 15) != 0), p0);  // pages of kept tokens ahead of the window's
   const int pages = n_kept + (pos >> 4) - p0 + 1;
   const int per = (pages + splits - 1) / splits;
-  const int first = split * per, last = min(first + per, pages);
+  const int first = split * per + warp, last = min(split * per + per, pages);
+  const int count = first < last ? (last - first + 3) / 4 : 0;  // of this warp
   const int* bt = a.block_tables + static_cast<size_t>(b) * a.max_blocks;
-  const __nv_bfloat16* cache = static_cast<const __nv_bfloat16*>(a.cache);
-  const size_t block_elems = a.block_elems();
-  const size_t k_off = static_cast<size_t>(kh) * 16 * a.d;
-  const size_t v_off = a.v_off() + static_cast<size_t>(kh) * 16 * a.dv;
+  auto page = [&](int n) {
+    const int i = first + 4 * n;
+    return i < n_kept ? i : p0 + i - n_kept;
+  };
 
-  uint32_t qf[2 * KD][4];
-  {
-    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + static_cast<size_t>(t) * a.ldq + head0 * a.d;
+  if (tid == 0) {
+    for (int w = 0; w < 4; ++w)
+      for (int s = 0; s < STAGES; ++s) mbar_init(&full[w][s], 1);
+    abort_word = 0;
+    fence_mbar_init();
+  }
+  __syncthreads();
+
+  uint8_t* ring = smem + warp * STAGES * L_::PAGE;
+  int my_block = 0, issued = 0;  // lane l holds the block of this warp's page 32 c + l
+  auto issue = [&](int n) {
+    if ((n & 31) == 0) my_block = n + lane < count ? bt[page(n + lane)] : 0;
+    const int blk = __shfl_sync(0xffffffffu, my_block, n & 31);
+    if (lane == 0) {
+      uint8_t* dst = ring + (n % STAGES) * L_::PAGE;
+      uint64_t* bar = &full[warp][n % STAGES];
+      mbar_expect_tx(bar, L_::PAGE);
 #pragma unroll
-    for (int kb = 0; kb < KD; ++kb) {
-      uint4 x = make_uint4(0, 0, 0, 0), y = x;
-      if (r < g) x = *reinterpret_cast<const uint4*>(q + r * a.d + kb * 32 + j * 8);
-      if (r + 8 < g) y = *reinterpret_cast<const uint4*>(q + (r + 8) * a.d + kb * 32 + j * 8);
-      qf[2 * kb][0] = x.x; qf[2 * kb][1] = y.x; qf[2 * kb][2] = x.y; qf[2 * kb][3] = y.y;
-      qf[2 * kb + 1][0] = x.z; qf[2 * kb + 1][1] = y.z; qf[2 * kb + 1][2] = x.w; qf[2 * kb + 1][3] = y.w;
+      for (int hf = 0; hf < DP / 64; ++hf) tma_load_3d(dst + hf * 2048, &tmK, bar, hf * 64, kh * 16, blk);
+      if constexpr (!SHARED) {
+#pragma unroll
+        for (int hf = 0; hf < DVP / 64; ++hf)
+          tma_load_3d(dst + L_::K_BYTES + hf * 2048, &tmV, bar, hf * 64, kh * 16, blk);
+      }
     }
+    issued = n + 1;
+  };
+  for (int n = 0; n < STAGES && n < count; ++n) issue(n);
+
+  uint32_t qf[DP / 16][NT][2];
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt) {
+    const int hd = nt * 8 + r;
+    const __nv_bfloat16* q = static_cast<const __nv_bfloat16*>(a.q) + static_cast<size_t>(t) * a.ldq + (head0 + hd) * a.d;
+#pragma unroll
+    for (int kb = 0; kb < DP / 16; ++kb)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const int c = kb * 16 + u * 8 + j2;
+        qf[kb][nt][u] = hd < g && c < a.d ? *reinterpret_cast<const uint32_t*>(q + c) : 0u;
+      }
   }
   const float scale2 = a.scale * 1.4426950408889634f;
-  const float* bias0 = a.bias ? a.bias + static_cast<size_t>(head0 + min(r, g - 1)) * a.bias_len : nullptr;
-  const float* bias1 = a.bias ? a.bias + static_cast<size_t>(head0 + min(r + 8, g - 1)) * a.bias_len : nullptr;
-  float o[ND * 8][4];
+  float acc[DVP / 16][NT][4];
 #pragma unroll
-  for (int i = 0; i < ND * 8; ++i)
+  for (int i = 0; i < DVP / 16; ++i)
 #pragma unroll
-    for (int u = 0; u < 4; ++u) o[i][u] = 0.f;
-  float m[2] = {-INFINITY, -INFINITY}, l[2] = {0.f, 0.f};
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int u = 0; u < 4; ++u) acc[i][nt][u] = 0.f;
+  float m[NT][2], l[NT][2];  // of heads nt * 8 + j2 + {0, 1}; l: this thread's keys only
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt) m[nt][0] = m[nt][1] = -INFINITY, l[nt][0] = l[nt][1] = 0.f;
 
-  for (int i = first + warp; i < last; i += 4) {
-    const int pg = i < n_kept ? i : p0 + i - n_kept;
-    const __nv_bfloat16* blk = cache + bt[pg] * block_elems;
-    uint4 kf[2][KD], vf[4][ND];
+  // this lane's row and 16-byte column of the four 8 x 8 matrices of an ldmatrix
+  const int k_row = (lane & 7) + (lane & 8), k_col = lane >> 4;
+  const int v_row = (lane & 7) + ((lane >> 4) << 3), v_col = (lane >> 3) & 1;
+  bool ok = true;
+  for (int n = 0; n < count; ++n) {
+    ok = mbar_wait_bounded(&full[warp][n % STAGES], (n / STAGES) & 1, abort_flag, err);
+    if (!__all_sync(0xffffffffu, ok)) {
+      ok = false;
+      // copies in flight still write to this CTA's memory: give them their (bounded) time before leaving
+      for (int i = n; i < issued; ++i)
+        for (int it = 0; it < (1 << 20) && !mbar_try_wait(&full[warp][i % STAGES], (i / STAGES) & 1); ++it) {}
+      break;
+    }
+    const uint32_t kb0 = smem_u32(ring + (n % STAGES) * L_::PAGE), vb0 = kb0 + (SHARED ? 0 : L_::K_BYTES);
+    float c[NT][4];
 #pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-      for (int kb = 0; kb < KD; ++kb)
-        kf[nt][kb] = *reinterpret_cast<const uint4*>(blk + k_off + (nt * 8 + r) * a.d + kb * 32 + j * 8);
-#pragma unroll
-    for (int u = 0; u < 4; ++u)
-#pragma unroll
-      for (int nb = 0; nb < ND; ++nb)
-        vf[u][nb] = *reinterpret_cast<const uint4*>(blk + v_off + (j * 2 + (u & 1) + (u >> 1) * 8) * a.dv + nb * 64 + r * 8);
-    float c[2][4];
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt) {
+    for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
       for (int u = 0; u < 4; ++u) c[nt][u] = 0.f;
 #pragma unroll
-      for (int kb = 0; kb < KD; ++kb) {
-        mma_16816(c[nt], qf[2 * kb], kf[nt][kb].x, kf[nt][kb].y);
-        mma_16816(c[nt], qf[2 * kb + 1], kf[nt][kb].z, kf[nt][kb].w);
-      }
+    for (int kb = 0; kb < DP / 16; ++kb) {
+      uint32_t f[4];
+      const int ch = kb * 2 + k_col;
+      ldmatrix_x4<false>(f, kb0 + (ch >> 3) * 2048 + k_row * 128 + (((ch & 7) ^ (k_row & 7)) << 4));
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) mma_16816(c[nt], f, qf[kb][nt][0], qf[kb][nt][1]);
     }
-    float mx[2] = {-INFINITY, -INFINITY};
+    const int key0 = page(n) * 16 + r;
 #pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
+    for (int u = 0; u < 2; ++u) {
+      const int key = key0 + u * 8;
+      const bool seen = (key >= lo || key < a.keep) && key <= pos;
 #pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        const int key = pg * 16 + nt * 8 + j * 2 + (u & 1);
-        const float* bias = (u >> 1) ? bias1 : bias0;
-        float s = -INFINITY;
-        if ((key >= lo || key < a.keep) && key <= pos) {
-          s = c[nt][u] * scale2;
-          if (bias) s = fmaf(bias[min(pos - key, a.bias_len - 1)], 1.4426950408889634f, s);
-        }
-        c[nt][u] = s;
-        mx[u >> 1] = fmaxf(mx[u >> 1], s);
-      }
-    float f[2];
+      for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-    for (int q = 0; q < 2; ++q) {
-      mx[q] = fmaxf(mx[q], __shfl_xor_sync(0xffffffffu, mx[q], 1));
-      mx[q] = fmaxf(mx[q], __shfl_xor_sync(0xffffffffu, mx[q], 2));
-      mx[q] = fmaxf(mx[q], m[q]);  // finite: every page of the range holds a visible key
-      f[q] = exp2f(m[q] - mx[q]);
-      m[q] = mx[q];
-      l[q] *= f[q];
-    }
-    uint32_t ph[4], pl[4];
-#pragma unroll
-    for (int nt = 0; nt < 2; ++nt)
-#pragma unroll
-      for (int q = 0; q < 2; ++q) {
-        const float x = exp2f(c[nt][2 * q] - m[q]), y = exp2f(c[nt][2 * q + 1] - m[q]);
-        l[q] += x + y;
-        ph[nt * 2 + q] = split_bf16(x, y, &pl[nt * 2 + q]);
-      }
-#pragma unroll
-    for (int nb = 0; nb < ND; ++nb) {
-      const uint32_t* w0 = reinterpret_cast<const uint32_t*>(&vf[0][nb]);
-      const uint32_t* w1 = reinterpret_cast<const uint32_t*>(&vf[1][nb]);
-      const uint32_t* w2 = reinterpret_cast<const uint32_t*>(&vf[2][nb]);
-      const uint32_t* w3 = reinterpret_cast<const uint32_t*>(&vf[3][nb]);
-#pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        const uint32_t sel = (e & 1) ? 0x7632 : 0x5410;
-        const uint32_t b0 = __byte_perm(w0[e >> 1], w1[e >> 1], sel), b1 = __byte_perm(w2[e >> 1], w3[e >> 1], sel);
-        float* acc = o[nb * 8 + e];
-        acc[0] *= f[0]; acc[1] *= f[0]; acc[2] *= f[1]; acc[3] *= f[1];
-        mma_16816(acc, ph, b0, b1);
-        mma_16816(acc, pl, b0, b1);
-      }
-    }
-  }
-#pragma unroll
-  for (int q = 0; q < 2; ++q) {
-    l[q] += __shfl_xor_sync(0xffffffffu, l[q], 1);
-    l[q] += __shfl_xor_sync(0xffffffffu, l[q], 2);
-    const int row = r + q * 8;
-    if (row < g) {
-      if (j == 0) {
-        sM[warp * 16 + row] = m[q];
-        sL[warp * 16 + row] = l[q];
-      }
-      float* dst = sO + (static_cast<size_t>(warp) * g + row) * DV;
-#pragma unroll
-      for (int nb = 0; nb < ND; ++nb)
-#pragma unroll
-        for (int u = 0; u < 2; ++u) {
-          float* p = dst + nb * 64 + (j * 2 + u) * 8;
-          *reinterpret_cast<float4*>(p) = make_float4(o[nb * 8][q * 2 + u], o[nb * 8 + 1][q * 2 + u],
-                                                      o[nb * 8 + 2][q * 2 + u], o[nb * 8 + 3][q * 2 + u]);
-          *reinterpret_cast<float4*>(p + 4) = make_float4(o[nb * 8 + 4][q * 2 + u], o[nb * 8 + 5][q * 2 + u],
-                                                          o[nb * 8 + 6][q * 2 + u], o[nb * 8 + 7][q * 2 + u]);
+        for (int e = 0; e < 2; ++e) {
+          float s = c[nt][u * 2 + e] * scale2;
+          if (a.bias) {
+            const int hd = min(nt * 8 + j2 + e, g - 1);
+            const float* bias = a.bias + static_cast<size_t>(head0 + hd) * a.bias_len;
+            if (seen) s = fmaf(bias[min(pos - key, a.bias_len - 1)], 1.4426950408889634f, s);
+          }
+          c[nt][u * 2 + e] = seen ? s : -INFINITY;
         }
     }
+    float mx[NT][2];
+    bool grown = false;
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        float v = fmaxf(c[nt][e], c[nt][2 + e]);
+        v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 4));
+        v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 8));
+        v = fmaxf(v, __shfl_xor_sync(0xffffffffu, v, 16));
+        mx[nt][e] = fmaxf(v, m[nt][e]);  // finite: every page of the range holds a visible key
+        grown = grown || mx[nt][e] > m[nt][e] + 8.f;
+      }
+    if (__any_sync(0xffffffffu, grown)) {
+      // exponents stay relative to m until some head's maximum has grown by more than 8 (x 256)
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          const float f = exp2f(m[nt][e] - mx[nt][e]);
+          m[nt][e] = mx[nt][e];
+          l[nt][e] *= f;
+#pragma unroll
+          for (int i = 0; i < DVP / 16; ++i) {
+            acc[i][nt][e] *= f;
+            acc[i][nt][2 + e] *= f;
+          }
+        }
+    }
+    uint32_t ph[NT][2], pl[NT][2];
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int u = 0; u < 2; ++u) {
+        const float x = exp2f(c[nt][u * 2] - m[nt][0]), y = exp2f(c[nt][u * 2 + 1] - m[nt][1]);
+        l[nt][0] += x;
+        l[nt][1] += y;
+        uint32_t low;
+        ph[nt][u] = transpose_8x8(split_bf16(x, y, &low));
+        pl[nt][u] = transpose_8x8(low);
+      }
+#pragma unroll
+    for (int i = 0; i < DVP / 16; ++i) {
+      uint32_t f[4];
+      const int ch = i * 2 + v_col;
+      ldmatrix_x4<true>(f, vb0 + (ch >> 3) * 2048 + v_row * 128 + (((ch & 7) ^ (v_row & 7)) << 4));
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) {
+        mma_16816(acc[i][nt], f, ph[nt][0], ph[nt][1]);
+        mma_16816(acc[i][nt], f, pl[nt][0], pl[nt][1]);
+      }
+    }
+    __syncwarp();  // every lane has read this page
+    if (n + STAGES < count) issue(n + STAGES);
   }
+  __syncthreads();  // the ring is free: the warps' parts go over it
+  float* sO = reinterpret_cast<float*>(smem);  // [4][g][LDO]
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+    for (int e = 0; e < 2; ++e) {
+      float s = l[nt][e];
+      s += __shfl_xor_sync(0xffffffffu, s, 4);
+      s += __shfl_xor_sync(0xffffffffu, s, 8);
+      s += __shfl_xor_sync(0xffffffffu, s, 16);
+      const int hd = nt * 8 + j2 + e;
+      if (hd < g) {
+        if (r == 0) {
+          sM[warp][hd] = m[nt][e];
+          sL[warp][hd] = s;
+        }
+        float* dst = sO + (warp * g + hd) * LDO + r;
+#pragma unroll
+        for (int i = 0; i < DVP / 16; ++i) {
+          dst[i * 16] = acc[i][nt][e];
+          dst[i * 16 + 8] = acc[i][nt][2 + e];
+        }
+      }
+    }
   __syncthreads();
   // the four warps' parts -> one per CTA, in place of warp 0's
   if (tid < g) {
     float M = -INFINITY, S = 0.f;
-    for (int w = 0; w < 4; ++w) M = fmaxf(M, sM[w * 16 + tid]);
+    for (int w = 0; w < 4; ++w) M = fmaxf(M, sM[w][tid]);
     for (int w = 0; w < 4; ++w) {
-      const float f = M == -INFINITY ? 0.f : exp2f(sM[w * 16 + tid] - M);
-      S += sL[w * 16 + tid] * f;
-      sL[w * 16 + tid] = f;  // from here on the warp's weight
+      const float f = M == -INFINITY ? 0.f : exp2f(sM[w][tid] - M);
+      S += sL[w][tid] * f;
+      sL[w][tid] = f;  // from here on the warp's weight
     }
     cM[tid] = M;
     cL[tid] = S;
   }
   __syncthreads();
-  for (int e = tid * 4; e < g * DV; e += 512) {
-    const int row = e / DV;
+  const int quads = a.dv / 4;
+  for (int e = tid; e < g * quads; e += 128) {
+    const int hd = e / quads, col = e % quads * 4;
     float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
     for (int w = 0; w < 4; ++w) {
-      const float f = sL[w * 16 + row];
-      const float4 v = *reinterpret_cast<const float4*>(sO + static_cast<size_t>(w) * g * DV + e);
+      const float f = sL[w][hd];
+      const float4 v = *reinterpret_cast<const float4*>(sO + (w * g + hd) * LDO + col);
       s.x += f * v.x; s.y += f * v.y; s.z += f * v.z; s.w += f * v.w;
     }
-    *reinterpret_cast<float4*>(sO + e) = s;  // only this thread reads or writes these elements of warp 0's part
+    *reinterpret_cast<float4*>(sO + hd * LDO + col) = s;  // only this thread reads or writes these elements of warp 0's part
   }
   __syncwarp();
   if (splits > 1)
@@ -625,46 +716,50 @@ window_decode_kernel(WindowAttnArgs a, int seq_base, int groups) {
   else
     __syncthreads();
   __nv_bfloat16* out = static_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(t) * a.ldo + head0 * a.dv;
-  for (int e = (split * 128 + tid) * 4; e < g * DV; e += splits * 512) {
-    const int row = e / DV;
-    float M = -INFINITY, S = 0.f, acc[4] = {0.f, 0.f, 0.f, 0.f};
+  for (int e = split * 128 + tid; e < g * quads; e += splits * 128) {
+    const int hd = e / quads, col = e % quads * 4;
+    float M = -INFINITY, S = 0.f, o[4] = {0.f, 0.f, 0.f, 0.f};
     if (splits == 1) {
-      S = cL[row];
-      const float4 v = *reinterpret_cast<const float4*>(sO + e);
-      acc[0] = v.x; acc[1] = v.y; acc[2] = v.z; acc[3] = v.w;
+      S = cL[hd];
+      const float4 v = *reinterpret_cast<const float4*>(sO + hd * LDO + col);
+      o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
     } else {
-      for (int s = 0; s < splits; ++s) M = fmaxf(M, ld_cluster_f1(mapa_u32(smem_u32(cM + row), s)));
+      for (int s = 0; s < splits; ++s) M = fmaxf(M, ld_cluster_f1(mapa_u32(smem_u32(cM + hd), s)));
       for (int s = 0; s < splits; ++s) {
-        const float f = exp2f(ld_cluster_f1(mapa_u32(smem_u32(cM + row), s)) - M);
-        S += f * ld_cluster_f1(mapa_u32(smem_u32(cL + row), s));
-        const float4 v = ld_cluster_f4(mapa_u32(smem_u32(sO + e), s));
-        acc[0] += f * v.x; acc[1] += f * v.y; acc[2] += f * v.z; acc[3] += f * v.w;
+        const float f = exp2f(ld_cluster_f1(mapa_u32(smem_u32(cM + hd), s)) - M);
+        S += f * ld_cluster_f1(mapa_u32(smem_u32(cL + hd), s));
+        const float4 v = ld_cluster_f4(mapa_u32(smem_u32(sO + hd * LDO + col), s));
+        o[0] += f * v.x; o[1] += f * v.y; o[2] += f * v.z; o[3] += f * v.w;
       }
     }
     const float inv = a.out_scale / S;
 #pragma unroll
-    for (int u = 0; u < 4; ++u) acc[u] *= inv;
-    store_n<4>(out + row * a.dv + e % DV, acc);
+    for (int u = 0; u < 4; ++u) o[u] *= inv;
+    store_n<4>(out + hd * a.dv + col, o);
   }
   __syncwarp();
   if (splits > 1) cluster_sync_all();  // nobody leaves while its memory is still read
 }
 
-template <int KD, int ND>
-static int launch_decode(const WindowAttnArgs& a, int seq_base, int num_seqs, int max_kv, cudaStream_t st) {
-  const int gq = a.h / a.hk, groups = (gq + 15) / 16, g = gq < 16 ? gq : 16;
-  const int smem = static_cast<int>(sizeof(float)) * (4 * g * ND * 64 + 64 + 64 + 32);
-  auto kern = window_decode_kernel<KD, ND>;
-  if (KSANA_SMEM_ONCE(kern, 4 * 16 * ND * 64 * 4 + 1024) != 0) return -4;
+template <int DP, int DVP, int NT, bool SHARED>
+static int launch_decode(const WindowAttnArgs& a, int num_blocks, int seq_base, int num_seqs, int max_kv,
+                         cudaStream_t st) {
+  using L_ = WindowDecodeSmem<DP, DVP, SHARED>;
+  const int gq = a.h / a.hk, groups = (gq + 15) / 16;
+  CUtensorMap tk, tv;
+  if (int rc = cache_maps(a, num_blocks, &tk, &tv)) return rc;
+  auto kern = window_decode_kernel<DP, DVP, NT, SHARED>;
+  if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
   const int keys = a.window > 0 && a.window < max_kv - a.keep ? a.window + a.keep : max_kv;
   const int pages = keys / 16 + 1;
   const long long base = static_cast<long long>(num_seqs) * a.hk * groups;
+  // enough CTAs for a few waves of what the SMs hold (whose last one is then short), as long as a warp gets some pages
   int splits = 1;
-  while (splits < 8 && base * splits < 3 * sm_count() && pages / (splits * 2) >= 8) splits *= 2;
+  while (splits < 8 && base * splits < 8 * sm_count() && pages / (splits * 2) >= 8) splits *= 2;
   cudaLaunchConfig_t cfg = {};
   cfg.gridDim = dim3(splits, a.hk * groups, num_seqs);
   cfg.blockDim = dim3(128);
-  cfg.dynamicSmemBytes = smem;
+  cfg.dynamicSmemBytes = L_::TOTAL;
   cfg.stream = st;
   cudaLaunchAttribute at[1];
   at[0].id = cudaLaunchAttributeClusterDimension;
@@ -672,7 +767,7 @@ static int launch_decode(const WindowAttnArgs& a, int seq_base, int num_seqs, in
   at[0].val.clusterDim.y = at[0].val.clusterDim.z = 1;
   cfg.attrs = at;
   cfg.numAttrs = 1;
-  return cudaLaunchKernelEx(&cfg, kern, a, seq_base, groups) == cudaSuccess ? 0 : -5;
+  return cudaLaunchKernelEx(&cfg, kern, tk, tv, a, seq_base, groups, error_word()) == cudaSuccess ? 0 : -5;
 }
 
 static bool rows16(const void* p, int ld) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && (ld & 7) == 0; }
@@ -706,29 +801,31 @@ KSANA_API int ksana_window_prefill(const void* q, int ldq, int total_tokens, con
 }
 
 // bf16. Sequences [seq_base, seq_base + num_seqs) with exactly one new token each. Returns -1 for sizes it does not
-// take (d = 32, 64, 96 or 128, dv = 64 or 128, pages of 16 tokens, 16-byte aligned rows).
-KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, const int* block_tables, int max_blocks,
-                                  const int* cu_q, const int* kv_lens, int h, int hk, int d, int dv, int bs, int window,
-                                  int keep, int shared, float scale, const float* bias, int bias_len, float out_scale,
-                                  void* out, int ldo, int seq_base, int num_seqs, int max_kv, cudaStream_t st) {
+// take (heads of at most 128 dimensions in multiples of 8, pages of 16 tokens, 16-byte aligned rows).
+KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, int num_blocks, const int* block_tables,
+                                  int max_blocks, const int* cu_q, const int* kv_lens, int h, int hk, int d, int dv,
+                                  int bs, int window, int keep, int shared, float scale, const float* bias, int bias_len,
+                                  float out_scale, void* out, int ldo, int seq_base, int num_seqs, int max_kv,
+                                  cudaStream_t st) {
   if (num_seqs <= 0) return 0;
   if (keep < 0 || (shared && d != dv)) return -2;
-  if (h % hk || bs != 16 || (d & 31) || d > 128 || (dv & 63) || dv > 128 || !rows16(q, ldq) || !rows16(cache, 0) ||
+  if (h % hk || bs != WP_PAGE || d > 128 || dv > 128 || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
       !rows16(out, ldo))
     return -1;
   WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
                    shared, scale, bias, bias_len, out_scale, out, ldo};
-#define KSANA_WD(KD) \
-  case KD: return dv == 64 ? launch_decode<KD, 1>(a, seq_base, num_seqs, max_kv, st) \
-                           : launch_decode<KD, 2>(a, seq_base, num_seqs, max_kv, st)
-  switch (d / 32) {
-    KSANA_WD(1);
-    KSANA_WD(2);
-    KSANA_WD(3);
-    KSANA_WD(4);
+#define KSANA_WD(DP, DVP, SHARED)                                                                             \
+  return h / hk <= 8 ? launch_decode<DP, DVP, 1, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)       \
+                     : launch_decode<DP, DVP, 2, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)
+  if (shared) {
+    if (d <= 64) KSANA_WD(64, 64, true);
+    KSANA_WD(128, 128, true);
   }
+  if (d <= 64 && dv <= 64) KSANA_WD(64, 64, false);
+  if (d <= 64) KSANA_WD(64, 128, false);
+  if (dv <= 64) KSANA_WD(128, 64, false);
+  KSANA_WD(128, 128, false);
 #undef KSANA_WD
-  return -1;
 }
 
 // Tokens [tok_base, tok_base + tokens) of the step, whatever sequences they belong to. kind: 0 fp32, 1 bf16.

@@ -90,7 +90,7 @@ class _Sig:
     ksana_softcap = ([P, I, P, I, I, F, P], I)
     ksana_window_attention_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
     ksana_window_prefill = ([P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
-    ksana_window_decode = ([P, I, P, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
+    ksana_window_decode = ([P, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
     ksana_linear_chunk_scratch = ([I, I, I, I, I], LL)
     ksana_linear_chunked = ([P, I, P, I, P, I, P, P, P, P, P, P, P, I, I, F, I, I, I, P, I, I, I, P, P], I)
     ksana_linear_recurrent = ([P, I, P, I, P, I, P, P, P, P, P, P, P, I, I, F, I, I, I, P, I, I, I, I, P], I)

@@ -145,8 +145,8 @@ def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, 
     if n_dec:
         code = -1
         if meta.num_decode_tokens == n_dec:
-            code = lib().ksana_window_decode(_ptr(q), q.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks,
-                                             _ptr(meta.cu_q), _ptr(meta.kv_lens), *sizes, _ptr(out), out.stride(0),
+            code = lib().ksana_window_decode(_ptr(q), q.stride(0), _ptr(cache), cache.shape[0], _ptr(meta.block_tables),
+                                             meta.max_blocks, _ptr(meta.cu_q), _ptr(meta.kv_lens), *sizes, _ptr(out), out.stride(0),
                                              n_pre, n_dec, int(meta.kv_lens_host[n_pre:].max()), _stream())
         if code == -1:
             general(pre_tokens, T - pre_tokens)
