@@ -85,6 +85,17 @@ __device__ __forceinline__ float gelu_tanh_f(float z) {
   return z / (1.f + expf(-2.f * u));
 }
 
+// For storage type T: 16-bit results take the fast exponential and division.
+template <typename T>
+__device__ __forceinline__ float gelu_tanh_as(float z) {
+  if constexpr (sizeof(T) == 2) {
+    const float u = 0.7978845608028654f * (z + 0.044715f * z * z * z);
+    return __fdividef(z, 1.f + __expf(-2.f * u));
+  } else {
+    return gelu_tanh_f(z);
+  }
+}
+
 // v = hi + lo with both parts bf16: the pair keeps 16 bits of the mantissa through 16-bit tensor-core operands. Packs
 // two values; *lo is exact up to its own rounding.
 __device__ __forceinline__ uint32_t split_bf16(float a, float b, uint32_t* lo) {

@@ -206,7 +206,7 @@ __global__ void gelu_mul_kernel(const T* __restrict__ x, int ldx, T* __restrict_
   load_n<N>(x + row * ldx + c, g);
   load_n<N>(x + row * ldx + I + c, u);
 #pragma unroll
-  for (int j = 0; j < N; ++j) g[j] = gelu_tanh_f(g[j]) * u[j];
+  for (int j = 0; j < N; ++j) g[j] = gelu_tanh_as<T>(g[j]) * u[j];
   store_n<N>(out + row * ldo + c, g);
 }
 
@@ -292,7 +292,7 @@ append_act_kernel(const T* __restrict__ k, const T* __restrict__ u, int ldx, con
   float g[N];
   if (gated) load_n<N>(u + row * ldx + I + c, g);
 #pragma unroll
-  for (int j = 0; j < N; ++j) f[j] = gelu_tanh_f(f[j]) * (gated ? g[j] : 1.f);
+  for (int j = 0; j < N; ++j) f[j] = gelu_tanh_as<T>(f[j]) * (gated ? g[j] : 1.f);
   store_n<N>(out + row * ldo + c, f);
 }
 

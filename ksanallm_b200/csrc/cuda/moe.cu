@@ -215,10 +215,15 @@ __global__ void moe_combine_kernel(const __nv_bfloat16* __restrict__ y, const in
 // Same pipeline as gemm_bf16_kernel (TMA producer warp / MMA warp / 4 epilogue warps, double-buffered TMEM
 // accumulator); the persistent tile loop walks (expert, m-tile, n-tile) using the device-side offsets, so ragged and
 // empty experts cost nothing. A tile's trailing rows may belong to the next expert: they are computed and dropped.
-constexpr int G_BM = 128, G_BN = 128, G_BK = 64, G_STAGES = 6;
-constexpr int G_A_BYTES = G_BM * G_BK * 2, G_B_BYTES = G_BN * G_BK * 2, G_STAGE = G_A_BYTES + G_B_BYTES;
-constexpr int G_BAR = G_STAGES * G_STAGE;
-constexpr int G_SMEM = G_BAR + 256 + 1024;
+// BN: 256 where experts get whole row tiles (half the reads of A), 128 where the weights are the traffic.
+constexpr int G_BM = 128, G_BK = 64, G_A_BYTES = G_BM * G_BK * 2;
+template <int BN>
+struct GroupedSmem {
+  static constexpr int STAGES = BN == 256 ? 4 : 6;
+  static constexpr int STAGE = G_A_BYTES + BN * G_BK * 2;
+  static constexpr int BAR = STAGES * STAGE;
+  static constexpr int TOTAL = BAR + 256 + 1024;
+};
 
 struct GroupedTileIter {
   const int* offsets;
@@ -226,16 +231,19 @@ struct GroupedTileIter {
   int e, base;                   // current expert and the global index of its first tile
   __device__ GroupedTileIter(const int* off, int E_, int tiles_n_, int first, int stride_)
       : offsets(off), E(E_), tiles_n(tiles_n_), stride(stride_), next(first), e(0), base(0) {}
-  // Returns false when no tile is left; otherwise fills (expert, m-tile, n-tile).
+  // Returns false when no tile is left; otherwise fills (expert, m-tile, n-tile). Within an expert, groups of 8 row tiles
+  // go through all column tiles, rows first: CTAs that run together share weight tiles, and a group's rows stay in L2.
   __device__ bool get(int* expert, int* mt, int* nt) {
     while (e < E) {
       const int rows = offsets[e + 1] - offsets[e];
-      const int tiles = ((rows + G_BM - 1) / G_BM) * tiles_n;
+      const int tiles_m = (rows + G_BM - 1) / G_BM, tiles = tiles_m * tiles_n;
       if (next < base + tiles) {
         const int local = next - base;
         *expert = e;
-        *mt = local / tiles_n;
-        *nt = local - (*mt) * tiles_n;
+        const int m0 = local / (8 * tiles_n) * 8, in_group = local - m0 * tiles_n;
+        const int height = min(8, tiles_m - m0);
+        *nt = in_group / height;
+        *mt = m0 + in_group - *nt * height;
         next += stride;
         return true;
       }
@@ -246,13 +254,15 @@ struct GroupedTileIter {
   }
 };
 
+template <int G_BN>
 __global__ void __launch_bounds__(192, 1)
 moe_grouped_gemm_kernel(const __grid_constant__ CUtensorMap tmA, const __grid_constant__ CUtensorMap tmB,
                         __nv_bfloat16* __restrict__ C, const int* __restrict__ offsets, int E, int N, int K, int ldc,
                         unsigned int* err) {
+  constexpr int G_STAGES = GroupedSmem<G_BN>::STAGES, G_STAGE = GroupedSmem<G_BN>::STAGE;
   extern __shared__ uint8_t smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
-  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + G_BAR);
+  uint64_t* full_bar = reinterpret_cast<uint64_t*>(smem + GroupedSmem<G_BN>::BAR);
   uint64_t* empty_bar = full_bar + G_STAGES;
   uint64_t* acc_full = empty_bar + G_STAGES;
   uint64_t* acc_empty = acc_full + 2;
@@ -439,21 +449,31 @@ KSANA_API int ksana_moe_permute(const void* x, int ldx, const int* ids, int T, i
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
+template <int BN>
+static int launch_grouped(const CUtensorMap& tmA, const void* W, void* C, const int* offsets, int E, int N, int K,
+                          cudaStream_t stream) {
+  CUtensorMap tmB;
+  if (make_tmap_2d(&tmB, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, static_cast<uint64_t>(E) * N, K, K, BN, G_BK,
+                   CU_TENSOR_MAP_SWIZZLE_128B))
+    return -3;
+  auto kern = moe_grouped_gemm_kernel<BN>;
+  if (KSANA_SMEM_ONCE(kern, GroupedSmem<BN>::TOTAL) != 0) return -4;
+  kern<<<sm_count(), 192, GroupedSmem<BN>::TOTAL, stream>>>(tmA, tmB, reinterpret_cast<__nv_bfloat16*>(C), offsets, E, N,
+                                                            K, N, error_word());
+  return cudaGetLastError() == cudaSuccess ? 0 : -5;
+}
+
 // C[sorted rows, N] = A[sorted rows, K] * W[e]^T per expert. W: [E, N, K] bf16 contiguous; max_rows = rows of A.
 KSANA_API int ksana_moe_grouped_gemm(const void* A, const void* W, void* C, const int* offsets, int E, int max_rows,
                                      int N, int K, cudaStream_t stream) {
   if (max_rows <= 0) return 0;
   if ((N & 7) || (K & 7)) return -1;  // (a last tile's columns past N are the next expert's: computed and dropped)
-  CUtensorMap tmA, tmB;
+  CUtensorMap tmA;
   if (make_tmap_2d(&tmA, A, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, max_rows, K, K, G_BM, G_BK, CU_TENSOR_MAP_SWIZZLE_128B))
     return -2;
-  if (make_tmap_2d(&tmB, W, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, static_cast<uint64_t>(E) * N, K, K, G_BN, G_BK,
-                   CU_TENSOR_MAP_SWIZZLE_128B))
-    return -3;
-  if (KSANA_SMEM_ONCE(moe_grouped_gemm_kernel, G_SMEM) != 0) return -4;
-  moe_grouped_gemm_kernel<<<sm_count(), 192, G_SMEM, stream>>>(tmA, tmB, reinterpret_cast<__nv_bfloat16*>(C), offsets, E,
-                                                              N, K, N, error_word());
-  return cudaGetLastError() == cudaSuccess ? 0 : -5;
+  if (N % 256 == 0 && max_rows >= 2 * G_BM * E)
+    return launch_grouped<256>(tmA, W, C, offsets, E, N, K, stream);
+  return launch_grouped<128>(tmA, W, C, offsets, E, N, K, stream);
 }
 
 KSANA_API int ksana_moe_combine(const void* y, const int* pos, const float* weights, int T, int k, int H, void* out,
