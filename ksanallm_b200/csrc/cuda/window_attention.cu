@@ -148,7 +148,7 @@ struct WindowPrefillSmem {
   static constexpr int TOTAL = USED > 120 * 1024 ? USED : 120 * 1024;
 };
 
-template <int DP, int DVP, bool SHARED>
+template <int DP, int DVP, bool SHARED, bool KEEP>
 __global__ void __launch_bounds__(160, 1)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, WindowAttnArgs a, int seq_base, unsigned int* err) {
@@ -202,7 +202,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
 
   const int kt0 = a.window_start(row_pos) / 128;
   const int kv_end = min(L, row_pos + 128);
-  const int n_kept = min(a.keep / 128 + (a.keep % 128 != 0), kt0);  // tiles of kept tokens ahead of the window's
+  // tiles of kept tokens ahead of the window's
+  const int n_kept = KEEP ? min(a.keep / 128 + (a.keep % 128 != 0), kt0) : 0;
   const int n = n_kept + (kv_end + 127) / 128 - kt0;  // >= 1
   auto tile = [&](int i) { return i < n_kept ? i : kt0 + i - n_kept; };
   const int n_pages = (L + WP_PAGE - 1) / WP_PAGE;
@@ -288,8 +289,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     for (int i = 0; i < n; ++i) {
       float* tb = tab + (i & 1) * 256;
       const int key0 = tile(i) * 128;
-      const int d0 = row_pos - key0 - 127;   // distance of entry 0
-      const int kept = a.keep - key0;        // columns below this one are kept tokens
+      const int d0 = row_pos - key0 - 127;        // distance of entry 0
+      const int kept = KEEP ? a.keep - key0 : 0;  // columns below this one are kept tokens
       const int cut = kept > 0 ? 1 << 30 : reach;
 #pragma unroll
       for (int e = tid; e < 256; e += 128) {
@@ -311,7 +312,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       for (int c = 0; c < 4; ++c) tmem_ld32(S + c * 32, reinterpret_cast<uint32_t*>(s) + c * 32);
       tmem_wait_ld();
       float m_tile = -INFINITY;
-      if (kept > 0) {
+      if (KEEP && kept > 0) {
         const int behind = row_pos + tid - key0 - reach;  // columns up to this one are behind the window
 #pragma unroll
         for (int j = 0; j < 128; ++j)
@@ -410,7 +411,7 @@ static int cache_maps(const WindowAttnArgs& a, int num_blocks, CUtensorMap* tk, 
   return 0;
 }
 
-template <int DP, int DVP, bool SHARED = false>
+template <int DP, int DVP, bool SHARED, bool KEEP>
 static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blocks, int seq_base, int num_seqs,
                           int max_q, cudaStream_t st) {
   using L_ = WindowPrefillSmem<DP, DVP, SHARED>;
@@ -422,7 +423,7 @@ static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blo
     if (make_tmap_nd(&tq, a.q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -2;
   }
   if (int rc = cache_maps(a, num_blocks, &tk, &tv)) return rc;
-  auto kern = window_prefill_kernel<DP, DVP, SHARED>;
+  auto kern = window_prefill_kernel<DP, DVP, SHARED, KEEP>;
   if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
   kern<<<dim3((max_q + 127) / 128, num_seqs, a.h), 160, L_::TOTAL, st>>>(tq, tk, tv, a, seq_base, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
@@ -790,14 +791,18 @@ KSANA_API int ksana_window_prefill(const void* q, int ldq, int total_tokens, con
     return -1;
   WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
                    shared, scale, bias, bias_len, out_scale, out, ldo};
-  if (shared)
-    return d <= 64 ? launch_prefill<64, 64, true>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
-                   : launch_prefill<128, 128, true>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st);
-  if (d <= 64)
-    return dv <= 64 ? launch_prefill<64, 64>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
-                    : launch_prefill<64, 128>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st);
-  return dv <= 64 ? launch_prefill<128, 64>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
-                  : launch_prefill<128, 128>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st);
+#define KSANA_WP(DP, DVP, SHARED)                                                                                      \
+  return keep ? launch_prefill<DP, DVP, SHARED, true>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)      \
+              : launch_prefill<DP, DVP, SHARED, false>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
+  if (shared) {
+    if (d <= 64) KSANA_WP(64, 64, true);
+    KSANA_WP(128, 128, true);
+  }
+  if (d <= 64 && dv <= 64) KSANA_WP(64, 64, false);
+  if (d <= 64) KSANA_WP(64, 128, false);
+  if (dv <= 64) KSANA_WP(128, 64, false);
+  KSANA_WP(128, 128, false);
+#undef KSANA_WP
 }
 
 // bf16. Sequences [seq_base, seq_base + num_seqs) with exactly one new token each. Returns -1 for sizes it does not
