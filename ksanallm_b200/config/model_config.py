@@ -9,6 +9,7 @@ model-type dispatch of src/ksana_llm/runtime/model_instance.cpp:50-145.
 from __future__ import annotations
 
 import json
+import math
 import os
 from dataclasses import dataclass, field
 from typing import Any, Dict, List, Optional, Tuple
@@ -27,6 +28,7 @@ class RopeScaling:
     mscale_all_dim: float = 0.0
     mrope_section: List[int] = field(default_factory=list)
     alpha: float = 0.0  # dynamic-NTK "alpha" flavour
+    attention_factor: float = 0.0  # YaRN: magnitude of cos and sin as given (0: from factor and mscale)
 
 
 @dataclass
@@ -38,6 +40,14 @@ class QuantConfig:
     weight_block_size: List[int] = field(default_factory=list)  # [128, 128] for block-scaled fp8
     zero_point: bool = False
     modules_to_not_convert: List[str] = field(default_factory=list)
+
+
+@dataclass
+class RotarySpec:
+    """Rotation of the leading ``dims`` dimensions of q and k, neighbouring entries (2i, 2i + 1) being a pair."""
+    dims: int
+    base: float
+    scaling: RopeScaling = field(default_factory=RopeScaling)
 
 
 @dataclass
@@ -55,6 +65,42 @@ class AttentionSpec:
     qkv_bias: bool = False
     qk_norm: bool = False    # per-head RMS norm of q and k
     out_scale: float = 1.0   # factor on the mixer's output
+    rot: Optional[RotarySpec] = None
+    softcap: float = 0.0     # score <- cap * tanh(score / cap), 0: off
+    sink: bool = False       # the softmax's denominator has one more term exp(0)
+    head_gate: bool = False  # each head's output times the sigmoid of a number of its own, projected from the mixer's input
+    o_bias: bool = False
+    kv_from: Optional[int] = None  # reads the keys and values of that earlier layer: no projections, no cache of its own
+
+
+@dataclass
+class LatentAttentionSpec:
+    """Attention over a cached latent of ``rank`` numbers per token (RMS-normed) and one rotated key part shared by all
+    heads; keys of ``dim`` unrotated dimensions and values are linear maps of the latent, per head."""
+    heads: int
+    dim: int
+    rot_dim: int
+    vdim: int
+    rank: int
+    scale: float
+    rot: RotarySpec = None
+    head_gate: bool = False
+
+    @property
+    def width(self) -> int:
+        """Cache elements per token."""
+        return self.rank + self.rot_dim
+
+
+@dataclass
+class RecurrenceSpec:
+    """A gated linear recurrence per channel behind a short causal convolution, times a GELU branch:
+    log a = -decay_scale * r * softplus(lam), S <- a S + sqrt(1 - a^2) i u, the gates r and i being block-diagonal maps
+    of u."""
+    width: int
+    blocks: int
+    taps: int
+    decay_scale: float = 8.0
 
 
 @dataclass
@@ -75,12 +121,20 @@ class LinearAttentionSpec:
 
 @dataclass
 class ExpertsSpec:
-    """A mixture of gated-SiLU experts: the ``top`` largest router logits choose, and the softmax over the chosen logits
-    weights them."""
+    """A mixture of gated experts: the ``top`` largest router logits choose, and the softmax over the chosen logits weights
+    them (which is the softmax over all experts, divided by the chosen ones' sum). With ``groups`` > 1, equal groups of
+    neighbouring experts are ranked by their largest logit first, and only experts of the best ``keep`` groups count.
+
+    An expert is silu(gate) * up; with ``limit`` > 0, g * sigmoid(``alpha`` g) * (u + 1) with g = min(gate, limit) and
+    u = up clamped to +-limit."""
     experts: int
     top: int
     ff: int
     router_bias: bool = False  # a bias on the router logits, before the choice
+    groups: int = 1
+    keep: int = 1
+    limit: float = 0.0
+    alpha: float = 1.0
 
 
 @dataclass
@@ -89,13 +143,20 @@ class LayerSpec:
     which is dense (``ff``), routed (``moe``) or absent."""
     attn: Optional[AttentionSpec] = None
     linear: Optional[LinearAttentionSpec] = None
+    latent: Optional[LatentAttentionSpec] = None
+    recurrence: Optional[RecurrenceSpec] = None
     ff: int = 0              # dense feed-forward width (0: none)
     moe: Optional[ExpertsSpec] = None
     gated: bool = True       # dense feed-forward: act(gate) * up, else act(up)
     parallel: bool = False   # mixers and feed-forward read the same norm: x + (mixers(h) + ff(h))
+    ff_bias: bool = False    # biases of the dense feed-forward's projections
+    ff_act: str = ""         # its activation ("": the model's)
+    layer_scale: bool = False  # each sublayer's result times a learned vector
 
     @property
     def state_shape(self):
+        if self.recurrence is not None:  # the recurrent state, then the convolution's last inputs, oldest first
+            return (1, self.recurrence.taps, self.recurrence.width)
         return (self.linear.heads, self.linear.dim, self.linear.vdim) if self.linear else None
 
     @property
@@ -106,7 +167,11 @@ class LayerSpec:
     def kv_width(self) -> int:
         """Cache elements per token."""
         a = self.attn
-        return a.kv_heads * (a.dim + (0 if a.shared_kv else a.vdim)) if a else 0
+        if self.latent is not None:
+            return self.latent.width
+        if a is None or a.kv_from is not None:
+            return 0
+        return a.kv_heads * (a.dim + (0 if a.shared_kv else a.vdim))
 
 
 @dataclass
@@ -201,6 +266,9 @@ class ModelConfig:
     logit_softcap: float = 0.0    # logits <- cap * tanh(logits / cap); 0 = off
     residual_fp32: bool = False   # the residual stream is kept in 32-bit floats
     loop: Optional[LoopSpec] = None
+    # hyper-connections: the residual is this many streams; each sublayer reads a weighted sum of them, and every stream
+    # becomes a weighted sum of all old ones and the sublayer's result (0: one plain residual)
+    streams: int = 0
     # quantisation
     quant: QuantConfig = field(default_factory=QuantConfig)
     raw: Dict[str, Any] = field(default_factory=dict)
@@ -221,7 +289,7 @@ class ModelConfig:
     @property
     def has_state(self) -> bool:
         """Some layer carries a recurrent state from token to token."""
-        return any(l.linear is not None for l in self.layers)
+        return any(l.state_shape is not None for l in self.layers)
 
     def layer_runs(self) -> List[Tuple[int, Optional[int]]]:
         """The layers in the order they run, each with the number of the pass that starts with it (None: no pass does).
@@ -322,8 +390,11 @@ def _layered_config(c: Dict[str, Any], model_type: str) -> ModelConfig:
 def _set_layers(m: ModelConfig, layers: List[LayerSpec]) -> None:
     m.layers, m.num_layers = layers, len(layers)
     attn = next((l.attn for l in layers if l.attn is not None), None)
+    latent = next((l.latent for l in layers if l.latent is not None), None)
     if attn is not None:
         m.num_heads, m.num_kv_heads, m.head_dim = attn.heads, attn.kv_heads, attn.dim
+    elif latent is not None:
+        m.num_heads, m.num_kv_heads, m.head_dim = latent.heads, 1, latent.dim + latent.rot_dim
     m.intermediate_size = max((l.ff for l in layers), default=0)
     m.num_experts = max((l.moe.experts for l in layers if l.moe), default=0)
     m.num_experts_per_tok = max((l.moe.top for l in layers if l.moe), default=0)
@@ -394,8 +465,89 @@ def _molopel_config(c: Dict[str, Any]) -> ModelConfig:
     return m
 
 
+def _ladusun_rotary(r: Dict[str, Any], kind: str) -> RotarySpec:
+    s = r.get("scaling")
+    if not s:
+        return RotarySpec(int(r["dims"]), float(r["base"]))
+    rs = RopeScaling(type=kind, factor=float(s["factor"]), original_max_position_embeddings=int(s["original"]))
+    if kind == "yarn":
+        rs.beta_fast, rs.beta_slow = float(s["fast"]), float(s["slow"])
+        rs.attention_factor = 0.1 * math.log(rs.factor) + 1.0
+    else:
+        rs.low_freq_factor, rs.high_freq_factor = float(s["low"]), float(s["high"])
+    spec = RotarySpec(int(r["dims"]), float(r["base"]), rs)
+    if spec.dims % 2:
+        raise ValueError("rot.dims counts pairs of dimensions")
+    return spec
+
+
+def _ladusun_layer(entry: Dict[str, Any]) -> LayerSpec:
+    kind, c, mlp = str(entry["type"]), entry["mixer"], entry.get("mlp")
+    spec = LayerSpec(gated=False, layer_scale=True)
+    if kind == "rglru":
+        spec.recurrence = RecurrenceSpec(int(c["width"]), int(c["blocks"]), int(c["conv"]))
+        if spec.recurrence.width % spec.recurrence.blocks or spec.recurrence.taps < 1:
+            raise ValueError("the recurrence's width is a multiple of its blocks, and the convolution has at least one tap")
+    elif kind == "attention":
+        kv_from = c.get("kv_from")
+        spec.attn = AttentionSpec(
+            int(c["heads"]), int(c["kv_heads"]), int(c["dim"]), int(c["vdim"]), float(c["scale"]), qkv_bias=True,
+            rot=_ladusun_rotary(c["rot"], "llama3"), softcap=float(c.get("softcap") or 0.0), sink=True, head_gate=True, o_bias=True,
+            kv_from=None if kv_from is None else int(kv_from))
+        if spec.attn.heads % spec.attn.kv_heads or spec.attn.rot.dims > spec.attn.dim:
+            raise ValueError("heads are a multiple of kv_heads, and at most a whole head is rotated")
+    elif kind == "latent_attention":
+        spec.latent = LatentAttentionSpec(
+            int(c["heads"]), int(c["dim"]), int(c["rot_dim"]), int(c["vdim"]), int(c["kv_rank"]), float(c["scale"]),
+            rot=_ladusun_rotary(c["rot"], "yarn"), head_gate=True)
+        if spec.latent.rot.dims != spec.latent.rot_dim:
+            raise ValueError("the rotated part is rotated as a whole: rot.dims = rot_dim")
+    else:
+        raise ValueError(f"unknown Ladusun layer type {kind!r}")
+    if mlp is None:
+        return spec
+    ff = str(mlp.get("kind", "dense"))
+    if ff == "dense":
+        spec.ff, spec.ff_bias, spec.ff_act = int(mlp["ff"]), True, "relu2"
+    elif ff == "moe":
+        r, e = mlp["router"], mlp["expert"]
+        g = r.get("groups") or dict(count=1, keep=1)
+        spec.moe = ExpertsSpec(int(r["experts"]), int(r["top"]), int(e["ff"]), groups=int(g["count"]), keep=int(g["keep"]),
+                               limit=float(e["limit"]), alpha=1.702)
+        m = spec.moe
+        if m.groups < 1 or m.experts % m.groups or not 1 <= m.keep <= m.groups or \
+                not 1 <= m.top <= m.experts // m.groups * m.keep or m.limit <= 0:
+            raise ValueError(f"router {r} does not fit, or the experts' limit is not positive")
+    else:
+        raise ValueError(f"unknown Ladusun feed-forward {ff!r}")
+    return spec
+
+
+def _ladusun_config(c: Dict[str, Any]) -> ModelConfig:
+    """Ladusun: layers of latent attention, capped attention with a sink (some read another layer's keys and values), or
+    a gated linear recurrence; squared-ReLU or routed clamped experts; several residual streams joined by
+    hyper-connections; tied embeddings."""
+    m = _layered_config(c, "ladusun")
+    layers = [_ladusun_layer(e) for e in c["layers"]]
+    for i, l in enumerate(layers):
+        if l.attn is None or l.attn.kv_from is None:
+            continue
+        j = l.attn.kv_from
+        src = layers[j].attn if 0 <= j < i else None
+        if src is None or src.kv_from is not None or (src.kv_heads, src.dim, src.vdim, src.rot) != \
+                (l.attn.kv_heads, l.attn.dim, l.attn.vdim, l.attn.rot):
+            raise ValueError(f"layer {i} cannot read the keys and values of layer {j}")
+    _set_layers(m, layers)
+    m.streams = int(c["streams"])
+    if m.streams < 1:
+        raise ValueError("streams counts residual streams, at least one")
+    m.position_encoding, m.gated_mlp, m.tie_word_embeddings = "none", False, True
+    m.max_position_embeddings = int(c.get("max_position_embeddings", 1 << 20))
+    return m
+
+
 def model_config_from_dict(c: Dict[str, Any]) -> ModelConfig:
-    design = {"molopel": _molopel_config, "givirax": _givirax_config}.get(str(c.get("architecture", "")).lower())
+    design = {"molopel": _molopel_config, "givirax": _givirax_config, "ladusun": _ladusun_config}.get(str(c.get("architecture", "")).lower())
     if design is not None:
         return design(c)
     if isinstance(c.get("text_config"), dict) and str(c.get("model_type", "")).lower() in ("llama4",):
@@ -727,7 +879,45 @@ def tiny_givirax_config() -> ModelConfig:
     return cfg
 
 
+def ladusun_config(width: int = 4096, layers: int = 8, ff: int = 12288, experts: int = 16, top: int = 2,
+                   expert_ff: int = 3072, heads: int = 32, kv_heads: int = 8, dim: int = 128, rank: int = 512,
+                   rot_dim: int = 64, streams: int = 4, vocab: int = 32000, groups: int = 4, keep: int = 2) -> ModelConfig:
+    """Ladusun at the sizes of an ordinary decoder of that width: latent attention, the recurrence, attention, and every
+    second attention layer reading the one before it; dense and routed feed-forwards in turn."""
+    latent = dict(type="latent_attention", mixer=dict(
+        heads=heads, dim=dim, rot_dim=rot_dim, vdim=dim, kv_rank=rank, scale=(dim + rot_dim) ** -0.5,
+        rot=dict(dims=rot_dim, base=1e5, scaling=dict(factor=4.0, original=4096, fast=32.0, slow=1.0))))
+    rec = dict(type="rglru", mixer=dict(width=width, blocks=max(width // 128, 1), conv=4))
+    attn = dict(type="attention", mixer=dict(
+        heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, softcap=50.0,
+        rot=dict(dims=dim, base=5e5, scaling=dict(factor=8.0, low=1.0, high=4.0, original=8192))))
+    out, owner = [], None
+    for i in range(layers):
+        entry = json.loads(json.dumps((latent, rec, attn, rec)[i % 4]))
+        if entry["type"] == "attention":
+            if owner is None:
+                owner = i
+            else:
+                entry["mixer"]["kv_from"], owner = owner, None
+        entry["mlp"] = dict(kind="dense", ff=ff) if i % 2 == 0 else dict(
+            kind="moe", expert=dict(ff=expert_ff, limit=7.0),
+            router=dict(experts=experts, top=top, groups=dict(count=groups, keep=keep)))
+        out.append(entry)
+    return model_config_from_dict(dict(
+        architecture="Ladusun", embedding=dict(scale=1.0), norm=dict(eps=1e-6), vocab=vocab, width=width, streams=streams,
+        layers=out, eos_token_id=2))
+
+
+def tiny_ladusun_config() -> ModelConfig:
+    cfg = ladusun_config(width=128, layers=7, ff=192, experts=6, expert_ff=48, heads=4, kv_heads=2, dim=32, rank=48,
+                         rot_dim=16, streams=3, groups=3)
+    cfg.torch_dtype = "float32"
+    return cfg
+
+
 NAMED_CONFIGS = {
+    "tiny-ladusun": tiny_ladusun_config,
+    "ladusun": ladusun_config,
     "tiny-givirax": tiny_givirax_config,
     "givirax": givirax_config,
     "tiny-molopel": tiny_molopel_config,

@@ -1,6 +1,6 @@
 // Bandwidth-bound steps of layers with mixers of their own sizes: norms over a 32-bit residual stream, embedding into
-// that stream, GELU (gated or not), the paged cache append (with per-head QK norm, or beside the activation), the gated
-// RMS norm behind linear attention, and the logit soft cap. Everything is computed in 32-bit floats; T is the storage type of activations.
+// that stream, GELU (gated or not), squared ReLU and clamped gates, the paged cache append (with per-head QK norm and
+// rotation, or beside the activation), the gated RMS norm behind linear attention, and the logit soft cap. Everything is computed in 32-bit floats; T is the storage type of activations.
 #include "host_common.h"
 #include "mixer_common.cuh"
 
@@ -210,14 +210,47 @@ __global__ void gelu_mul_kernel(const T* __restrict__ x, int ldx, T* __restrict_
   store_n<N>(out + row * ldo + c, g);
 }
 
-// ---- per-head QK norm + cache append ------------------------------------------------------------------------------
-// One warp per (token, head): heads [0, h) are queries (normalised in place; h is 0 when they are not), the next hk keys
-// (normalised into the cache), the last hk values (copied into the cache). Cache: [block][keys hk x bs x d | values hk x bs x dv].
+// ---- squared ReLU; gate and up clamped -------------------------------------------------------------------------------
+template <typename T, int N>
+__global__ void relu2_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n) {
+  const size_t i = (static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x) * N;
+  if (i >= n) return;
+  float f[N];
+  load_n<N>(x + i, f);
+#pragma unroll
+  for (int j = 0; j < N; ++j) f[j] = fmaxf(f[j], 0.f) * fmaxf(f[j], 0.f);
+  store_n<N>(out + i, f);
+}
+
+// out = g sigmoid(alpha g) (u + 1) with g = min(gate, limit), u = up clamped to +-limit, over rows [gate | up]
+template <typename T, int N>
+__global__ void clamped_gate_mul_kernel(const T* __restrict__ x, T* __restrict__ out, int I, float limit, float alpha) {
+  const size_t row = blockIdx.x;
+  const int c = (blockIdx.y * blockDim.x + threadIdx.x) * N;
+  if (c >= I) return;
+  float g[N], u[N];
+  load_n<N>(x + row * 2 * I + c, g);
+  load_n<N>(x + row * 2 * I + I + c, u);
+#pragma unroll
+  for (int j = 0; j < N; ++j) {
+    g[j] = fminf(g[j], limit);
+    const float s = sizeof(T) == 2 ? __fdividef(1.f, 1.f + __expf(-alpha * g[j])) : sigmoid_f(alpha * g[j]);
+    g[j] *= s * (fminf(fmaxf(u[j], -limit), limit) + 1.f);
+  }
+  store_n<N>(out + row * I + c, g);
+}
+
+// ---- per-head QK norm, rotation, cache append -----------------------------------------------------------------------
+// One warp per (token, head): heads [0, h) are queries (in place; h is 0 when nothing happens to them), the next hk keys
+// (into the cache), the last hk values (copied into the cache). Queries and keys are normalised where there is a weight,
+// then the pairs (2i, 2i + 1) of their first rd dimensions are rotated where there is a table. Cache: [block][keys hk x bs
+// x d | values hk x bs x dv].
 template <typename T, int N>
 __global__ void __launch_bounds__(256)
 qk_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ldk, const T* __restrict__ v, int ldv,
                      const int* __restrict__ slots, T* __restrict__ cache, const float* __restrict__ qw,
-                     const float* __restrict__ kw, float eps, int tokens, int h, int hk, int d, int dv, int bs) {
+                     const float* __restrict__ kw, float eps, const int* __restrict__ positions,
+                     const float* __restrict__ rotary, int rd, int tokens, int h, int hk, int d, int dv, int bs) {
   const int heads = h + 2 * hk;
   const long long unit = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -258,13 +291,34 @@ qk_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ld
     }
     inv = 1.f / sqrtf(warp_sum(ss) / static_cast<float>(n) + eps);
   }
-  for (int c = lane * N; c < n; c += 32 * N) {
-    load_n<N>(src + c, f);
-    if (w) {
+  const bool turn = rotary != nullptr && hd < h + hk;
+  const float* cs = turn ? rotary + static_cast<size_t>(positions[t]) * rd : nullptr;
+  for (int c0 = 0; c0 < n; c0 += 32 * N) {
+    const int c = c0 + lane * N;
+    if (c < n) load_n<N>(src + c, f);
+    if (w && c < n) {
 #pragma unroll
       for (int j = 0; j < N; ++j) f[j] = f[j] * inv * w[c + j];
     }
-    store_n<N>(dst + c, f);
+    if (turn) {
+      if constexpr (N == 1) {
+        const float other = __shfl_xor_sync(0xffffffffu, f[0], 1);
+        if (c < rd) {
+          const float co = cs[c >> 1], si = cs[rd / 2 + (c >> 1)];
+          f[0] = c & 1 ? f[0] * co + other * si : f[0] * co - other * si;
+        }
+      } else {
+#pragma unroll
+        for (int j = 0; j < N; j += 2)
+          if (c + j < rd) {
+            const int i = (c + j) >> 1;
+            const float co = cs[i], si = cs[rd / 2 + i], a = f[j], b = f[j + 1];
+            f[j] = a * co - b * si;
+            f[j + 1] = b * co + a * si;
+          }
+      }
+    }
+    if (c < n) store_n<N>(dst + c, f);
   }
 }
 
@@ -455,20 +509,56 @@ KSANA_API int ksana_gelu_mul(const void* x, int ldx, void* out, int ldo, int row
   return done();
 }
 
+KSANA_API int ksana_relu2(const void* x, void* out, long long n, int kind, cudaStream_t st) {
+  if (n <= 0) return 0;
+  const bool vec = !(n & 7) && aligned(x, 16) && aligned(out, 16);
+#define KSANA_R2(T, N)                                                                                        \
+  relu2_kernel<T, N><<<static_cast<unsigned>((n / N + (n % N ? 1 : 0) + 255) / 256), 256, 0, st>>>(           \
+      static_cast<const T*>(x), static_cast<T*>(out), static_cast<size_t>(n))
+  if (kind) {
+    if (vec) KSANA_R2(bf16, 8); else KSANA_R2(bf16, 1);
+  } else {
+    if (vec) KSANA_R2(float, 8); else KSANA_R2(float, 1);
+  }
+#undef KSANA_R2
+  return done();
+}
+
+// x: [rows, 2 I] contiguous, out: [rows, I].
+KSANA_API int ksana_clamped_gate_mul(const void* x, void* out, int rows, int I, float limit, float alpha, int kind,
+                                     cudaStream_t st) {
+  if (rows <= 0 || I <= 0) return 0;
+  const bool vec = !(I & 7) && aligned(x, 16) && aligned(out, 16);
+  const int n = vec ? 8 : 1;
+  const dim3 grid(rows, (I + n * 256 - 1) / (n * 256));
+#define KSANA_CG(T, N) \
+  clamped_gate_mul_kernel<T, N><<<grid, 256, 0, st>>>(static_cast<const T*>(x), static_cast<T*>(out), I, limit, alpha)
+  if (kind) {
+    if (vec) KSANA_CG(bf16, 8); else KSANA_CG(bf16, 1);
+  } else {
+    if (vec) KSANA_CG(float, 8); else KSANA_CG(float, 1);
+  }
+#undef KSANA_CG
+  return done();
+}
+
 KSANA_API int ksana_qk_norm_cache(void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const int* slots,
-                                  void* cache, const float* qw, const float* kw, float eps, int tokens, int h, int hk,
-                                  int d, int dv, int bs, int kind, cudaStream_t st) {
+                                  void* cache, const float* qw, const float* kw, float eps, const int* positions,
+                                  const float* rotary, int rd, int tokens, int h, int hk, int d, int dv, int bs, int kind,
+                                  cudaStream_t st) {
   if (tokens <= 0) return 0;
+  if (rotary && (rd < 0 || rd > d || (rd & 1))) return -2;
   const int esz = kind ? 2 : 4;
   const bool vec = !((ldq | ldk | ldv | d | dv) & 3) && aligned(q, 4 * esz) && aligned(k, 4 * esz) &&
                    aligned(v, 4 * esz) && aligned(cache, 4 * esz);
-  if (!qw) h = 0;
+  if (!qw && !rotary) h = 0;
+  if (h + hk <= 0) return 0;
   const long long units = static_cast<long long>(tokens) * (h + 2 * hk);
   const unsigned grid = static_cast<unsigned>((units + 7) / 8);
 #define KSANA_QK(T, N)                                                                                              \
   qk_norm_cache_kernel<T, N><<<grid, 256, 0, st>>>(static_cast<T*>(q), ldq, static_cast<const T*>(k), ldk,          \
                                                    static_cast<const T*>(v), ldv, slots, static_cast<T*>(cache), qw, \
-                                                   kw, eps, tokens, h, hk, d, dv, bs)
+                                                   kw, eps, positions, rotary, rd, tokens, h, hk, d, dv, bs)
   if (kind) {
     if (vec) KSANA_QK(bf16, 4); else KSANA_QK(bf16, 1);
   } else {

@@ -7,17 +7,55 @@
 namespace ksana {
 
 // ---- router: top-k of logits (+ bias), softmax over the chosen ones ------------------------------------------------
-// One warp per token; the token's logits sit in shared memory. Ties go to the lower index.
+// One warp per token; the token's logits sit in shared memory. Ties go to the lower index. Of `groups` equal groups of
+// neighbours only the `keep` with the largest logits take part.
+__device__ __forceinline__ void warp_argmax(float& v, int& i) {
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) {
+    const float ov = __shfl_xor_sync(0xffffffffu, v, o);
+    const int oi = __shfl_xor_sync(0xffffffffu, i, o);
+    if (ov > v || (ov == v && oi < i)) {
+      v = ov;
+      i = oi;
+    }
+  }
+}
 __global__ void __launch_bounds__(128)
 moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int T, int E, int k,
-                int* __restrict__ ids, float* __restrict__ weights) {
+                int groups, int keep, int* __restrict__ ids, float* __restrict__ weights) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
   if (t >= T) return;
-  float* z = sm + warp * E;
+  const int G = keep < groups ? groups : 0, size = E / groups;
+  float* z = sm + warp * (E + 2 * G);
   for (int e = lane; e < E; e += 32) z[e] = logits[static_cast<size_t>(t) * ld + e] + (bias ? bias[e] : 0.f);
   __syncwarp();
+  if (G > 0) {
+    float *best = z + E, *open = best + G;
+    for (int g = lane; g < G; g += 32) {
+      float v = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) v = fmaxf(v, z[e]);
+      best[g] = v;
+      open[g] = 0.f;
+    }
+    __syncwarp();
+    for (int r = 0; r < keep; ++r) {
+      float v = -INFINITY;
+      int vi = G;
+      for (int g = lane; g < G; g += 32)
+        if (open[g] == 0.f && (best[g] > v || vi == G)) {
+          v = best[g];
+          vi = g;
+        }
+      warp_argmax(v, vi);
+      if (lane == 0 && vi < G) open[vi] = 1.f;
+      __syncwarp();
+    }
+    for (int e = lane; e < E; e += 32)
+      if (open[e / size] == 0.f) z[e] = -INFINITY;
+    __syncwarp();
+  }
   int* my_ids = ids + static_cast<size_t>(t) * k;
   float* my_w = weights + static_cast<size_t>(t) * k;
   float top = 0.f, sum = 0.f;
@@ -29,15 +67,7 @@ moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restric
         v = z[e];
         vi = e;
       }
-#pragma unroll
-    for (int o = 16; o > 0; o >>= 1) {
-      const float ov = __shfl_xor_sync(0xffffffffu, v, o);
-      const int oi = __shfl_xor_sync(0xffffffffu, vi, o);
-      if (ov > v || (ov == v && oi < vi)) {
-        v = ov;
-        vi = oi;
-      }
-    }
+    warp_argmax(v, vi);
     if (vi >= E) vi = 0;  // (no finite logit is left)
     if (r == 0) top = v;
     const float p = v == -INFINITY ? 0.f : expf(v - top);
@@ -171,12 +201,13 @@ static int launched() { return cudaGetLastError() == cudaSuccess ? 0 : -5; }
 
 using namespace ksana;
 
-KSANA_API int ksana_moe_topk(const float* logits, int ld, const float* bias, int T, int E, int k, int* ids,
-                             float* weights, cudaStream_t st) {
+KSANA_API int ksana_moe_topk(const float* logits, int ld, const float* bias, int T, int E, int k, int groups, int keep,
+                             int* ids, float* weights, cudaStream_t st) {
   if (T <= 0) return 0;
-  if (k < 1 || k > E || E > 2048) return -1;
-  moe_topk_kernel<<<(T + 3) / 4, 128, 4 * E * static_cast<int>(sizeof(float)), st>>>(logits, ld, bias, T, E, k, ids,
-                                                                                      weights);
+  if (groups < 1 || E % groups || keep < 1 || keep > groups || k > E / groups * keep) return -2;
+  const int smem = 4 * (E + (keep < groups ? 2 * groups : 0)) * static_cast<int>(sizeof(float));
+  if (k < 1 || E > 2048 || smem > 48 * 1024) return -1;
+  moe_topk_kernel<<<(T + 3) / 4, 128, smem, st>>>(logits, ld, bias, T, E, k, groups, keep, ids, weights);
   return launched();
 }
 

@@ -415,18 +415,18 @@ class MoEFFN:
         if c.scoring_func == "topk_softmax":
             # softmax over the chosen logits only, which stay in 32-bit
             ids, wts = ops.moe_topk(ops.linear(h, self.gate_w, None, torch.float32), c.num_experts,
-                                    c.num_experts_per_tok, self.logit_bias)
+                                    c.num_experts_per_tok, self.logit_bias, c.n_group, c.topk_group)
         else:
             logits = ops.linear(h.float() if self.gate_w.dtype == torch.float32 else h, self.gate_w)
             ids, wts = ops.moe_route(logits, c.num_experts_per_tok, c.scoring_func, c.norm_topk_prob, c.n_group,
                                      c.topk_group, c.routed_scaling_factor, self.bias)
         return self._place(ids), wts
 
-    def rows(self, h: torch.Tensor):
+    def rows(self, h: torch.Tensor, limit: float = 0.0, alpha: float = 1.0):
         """The routed sum in the form a norm over the stream takes: (unweighted rows of the experts, the row of every
-        (token, slot) pair, weights [T, k]). Unquantised local experts without a shared one."""
+        (token, slot) pair, weights [T, k]). Unquantised local experts without a shared one; ``limit`` > 0: clamped ones."""
         ids, wts = self.route(h)
-        y, pos = ops.moe_expert_rows(h, ids, self.w_gate_up, self.w_down)
+        y, pos = ops.moe_expert_rows(h, ids, self.w_gate_up, self.w_down, limit, alpha)
         return y, pos, wts
 
     def _grouped_fp8(self, h: torch.Tensor) -> bool:

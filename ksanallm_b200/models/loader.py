@@ -61,6 +61,15 @@ _RENAMES: Dict[str, List[Tuple[str, str]]] = {
                 (r"^l(\d+)\.mlp\.e(\d+)\.(gate|up|down)$", r"model.layers.\1.mlp.experts.\2.\3_proj.weight"),
                 (r"^l(\d+)\.mlp\.router$", r"model.layers.\1.mlp.gate.weight"),
                 (r"^l(\d+)\.mlp\.router\.b$", r"model.layers.\1.mlp.gate.bias")],
+    "ladusun": [(r"^embed$", "model.embed_tokens.weight"), (r"^final\.norm$", "model.norm.weight"),
+                (r"^l(\d+)\.norm1$", r"model.layers.\1.input_layernorm.weight"),
+                (r"^l(\d+)\.norm2$", r"model.layers.\1.post_attention_layernorm.weight"),
+                (r"^l(\d+)\.(ls\d|hc\d\.\w+)$", r"model.layers.\1.\2"),
+                (r"^l(\d+)\.mix\.", r"model.layers.\1.mixer."),
+                (r"^l(\d+)\.mlp\.(up|down)$", r"model.layers.\1.mlp.\2_proj.weight"),
+                (r"^l(\d+)\.mlp\.(up|down)\.b$", r"model.layers.\1.mlp.\2_proj.bias"),
+                (r"^l(\d+)\.mlp\.e(\d+)\.(gate|up|down)$", r"model.layers.\1.mlp.experts.\2.\3_proj.weight"),
+                (r"^l(\d+)\.mlp\.router$", r"model.layers.\1.mlp.gate.weight")],
     "baichuan": [(r"\.W_pack\.", ".wpack.")],
     "chatglm": [(r"^transformer\.embedding\.word_embeddings\.", "model.embed_tokens."),
                 (r"^transformer\.encoder\.layers\.", "model.layers."),
@@ -155,6 +164,12 @@ def synthetic_checkpoint(cfg: ModelConfig, seed: int = 0, std: float = 0.02, dev
         yield "model.embed_positions.weight", rnd(cfg.max_position_embeddings, H)
     if cfg.loop is not None:
         yield "model.loop.step", rnd(cfg.loop.times, H)
+    for i, spec in enumerate(cfg.layers if cfg.streams else ()):
+        S = cfg.streams
+        for n in (1, 2) if spec.has_ff else (1,):  # streams that are read in equal parts and stay apart
+            yield f"model.layers.{i}.hc{n}.in", ones(S) / S
+            yield f"model.layers.{i}.hc{n}.out", ones(S)
+            yield f"model.layers.{i}.hc{n}.mix", torch.eye(S, device=device, dtype=dtype)
     n_total = cfg.num_layers + cfg.num_nextn_predict_layers
     for i in range(n_total):
         p = f"model.layers.{i}"
@@ -404,19 +419,43 @@ def mixer_parts(spec: LayerSpec) -> set:
     pa, pl = mixer_prefixes(spec)
     need = set()
     if spec.attn is not None:
-        need |= {pa + x for x in ("qko" if spec.attn.shared_kv else "qkvo")}
-        if spec.attn.qkv_bias:
-            need |= {f"{pa}{x}.b" for x in "qkv"}
-        if spec.attn.qk_norm:
+        a = spec.attn
+        proj = "q" if a.kv_from is not None else "qk" if a.shared_kv else "qkv"
+        need |= {pa + x for x in proj + "o"}
+        if a.qkv_bias:
+            need |= {f"{pa}{x}.b" for x in proj}
+        if a.o_bias:
+            need.add(pa + "o.b")
+        if a.head_gate:
+            need.add(pa + "g")
+        if a.qk_norm:
             need |= {pa + "q.norm", pa + "k.norm"}
-        if spec.attn.bias_max:
+        if a.bias_max:
             need.add(pa + "rel")
+    if spec.latent is not None:
+        need |= {"q", "dkv", "dkv.norm", "uk", "uv", "o"} | ({"g"} if spec.latent.head_gate else set())
+    if spec.recurrence is not None:
+        need |= {"y", "y.b", "x", "x.b", "conv", "conv.b", "ra", "ra.b", "ri", "ri.b", "lam", "o"}
     if spec.linear is not None:
         need |= {pl + x for x in "qkvgo"}
         if spec.linear.norm == "concat":
             need.add(pl + "norm")
     if spec.parallel and spec.ff:  # a dense feed-forward beside the mixers shares their projections
         need |= {"ff." + x for x in (("gate", "up", "down") if spec.gated else ("up", "down"))}
+    return need
+
+
+def layer_parts(cfg: ModelConfig, i: int) -> set:
+    """Names of the tensors that surround a layer's mixers and feed-forward."""
+    spec, p = cfg.layers[i], f"model.layers.{i}"
+    need = {p + ".input_layernorm.weight"}
+    if spec.has_ff and not spec.parallel:
+        need.add(p + ".post_attention_layernorm.weight")
+    for n in (1, 2) if spec.has_ff else (1,):
+        if spec.layer_scale:
+            need.add(f"{p}.ls{n}")
+        if cfg.streams:
+            need |= {f"{p}.hc{n}.{x}" for x in ("in", "out", "mix")}
     return need
 
 
@@ -427,7 +466,7 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
     if spec.attn is not None:
         a = spec.attn
         for x, n in (("q", a.heads * a.dim), ("k", a.kv_heads * a.dim), ("v", a.kv_heads * a.vdim)):
-            if x == "v" and a.shared_kv:
+            if x == "v" and a.shared_kv or x != "q" and a.kv_from is not None:
                 continue
             yield m + pa + x, rnd(n, H)
             if a.qkv_bias:
@@ -437,7 +476,34 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
             yield m + pa + "k.norm", ones(a.dim)
         if a.bias_max:
             yield m + pa + "rel", rnd(32, a.heads)
+        if a.head_gate:
+            yield m + pa + "g", rnd(a.heads, H)
         yield m + pa + "o", rnd(H, a.heads * a.vdim)
+        if a.o_bias:
+            yield m + pa + "o.b", rnd(H)
+    if spec.latent is not None:
+        a = spec.latent
+        yield m + "q", rnd(a.heads * (a.dim + a.rot_dim), H)
+        yield m + "dkv", rnd(a.rank + a.rot_dim, H)
+        yield m + "dkv.norm", ones(a.rank)
+        yield m + "uk", rnd(a.heads * a.dim, a.rank)
+        yield m + "uv", rnd(a.heads * a.vdim, a.rank)
+        if a.head_gate:
+            yield m + "g", rnd(a.heads, H)
+        yield m + "o", rnd(H, a.heads * a.vdim)
+    if spec.recurrence is not None:
+        r = spec.recurrence
+        C, B = r.width, r.blocks
+        for x in ("y", "x"):
+            yield m + x, rnd(C, H)
+            yield f"{m}{x}.b", rnd(C)
+        yield m + "conv", rnd(C, r.taps)
+        yield m + "conv.b", rnd(C)
+        for x in ("ra", "ri"):
+            yield m + x, rnd(B, C // B, C // B)
+            yield f"{m}{x}.b", rnd(B, C // B)
+        yield m + "lam", rnd(C)
+        yield m + "o", rnd(H, C)
     if spec.linear is not None:
         r = spec.linear
         for x, n in (("q", r.dim), ("k", r.dim), ("v", r.vdim), ("g", r.vdim)):
@@ -452,6 +518,9 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
         return
     if spec.has_ff and not spec.parallel:
         yield p + ".post_attention_layernorm.weight", ones(H)
+    if spec.layer_scale:
+        for n in (1, 2) if spec.has_ff else (1,):
+            yield f"{p}.ls{n}", ones(H)
     if spec.moe is not None:
         e = spec.moe
         yield p + ".mlp.gate.weight", rnd(e.experts, H)
@@ -462,9 +531,13 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
             yield f"{p}.mlp.experts.{i}.up_proj.weight", rnd(e.ff, H)
             yield f"{p}.mlp.experts.{i}.down_proj.weight", rnd(H, e.ff)
     if spec.ff:
-        yield p + ".mlp.gate_proj.weight", rnd(spec.ff, H)
+        if spec.gated:
+            yield p + ".mlp.gate_proj.weight", rnd(spec.ff, H)
         yield p + ".mlp.up_proj.weight", rnd(spec.ff, H)
         yield p + ".mlp.down_proj.weight", rnd(H, spec.ff)
+        if spec.ff_bias:
+            yield p + ".mlp.up_proj.bias", rnd(spec.ff)
+            yield p + ".mlp.down_proj.bias", rnd(H)
 
 
 class WeightLoader:
@@ -651,7 +724,7 @@ class WeightLoader:
         if name == "model.embed_positions.weight":
             self._put(name, t)
             return
-        if name == "model.loop.step":
+        if name == "model.loop.step" or re.match(r"model\.layers\.\d+\.(ls\d|hc\d\.\w+)$", name):
             self._put(name, t.float(), keep_dtype=True)
             return
         if name == "lm_head.weight":
@@ -858,13 +931,14 @@ class WeightLoader:
         if key.endswith(".mlp"):
             li = self._layer_of(key + ".")
             moe = cfg.is_moe_layer(li) or (cfg.is_moe and li >= cfg.num_layers)
-            b = cfg.mlp_bias
+            spec = cfg.layers[li] if cfg.layers else None
+            b, gated = (spec.ff_bias, spec.gated) if spec is not None else (cfg.mlp_bias, cfg.gated_mlp)
 
             def ffn_ok(pre):
                 return (self._have(p, pre + "gate_proj") and self._have(p, pre + "up_proj") and
                         self._have(p, pre + "down_proj")) or \
                     (self._have(p, pre + "gate_up_proj") and self._have(p, pre + "down_proj")) or \
-                    (not cfg.gated_mlp and ((self._have(p, pre + "up_proj", b) and self._have(p, pre + "down_proj", b)) or
+                    (not gated and ((self._have(p, pre + "up_proj", b) and self._have(p, pre + "down_proj", b)) or
                                             (self._have(p, pre + "up_proj_t", b) and self._have(p, pre + "down_proj_t", b))))
             if moe:
                 ok = "gate.weight" in p
@@ -921,39 +995,67 @@ class WeightLoader:
             need = {"model.embed_tokens.weight": True, "model.norm.weight": True,
                     "lm_head.weight": not cfg.tie_word_embeddings, "model.loop.step": cfg.loop is not None,
                     "model.embed_positions.weight": cfg.position_encoding == "learned"}
+            need.update((name, True) for i in range(len(cfg.layers)) for name in layer_parts(cfg, i))
+            for i, spec in enumerate(cfg.layers):
+                m = f"model.layers.{i}.m"
+                need[m + "ixer.in_proj.weight"] = True
+                need[m + ("lp.gate.weight" if spec.moe else "lp.down_proj.weight")] = spec.has_ff and not (
+                    spec.parallel and spec.ff)
+                need[m + "lp.experts.down_proj.weight"] = spec.moe is not None
             missing = [name for name, wanted in need.items() if wanted and name not in self.out]
             if missing:
                 raise KeyError(f"the checkpoint has no {', '.join(missing)}")
+            if cfg.tie_word_embeddings and self.out["model.embed_tokens.weight"].shape[0] % 8:
+                e = self.out["model.embed_tokens.weight"]  # the head is a padded copy: the rows the GEMM takes
+                self.out["lm_head.weight"] = torch.nn.functional.pad(e, (0, 0, 0, -e.shape[0] % 8))
 
     def _finish_mixer(self, key: str, p: Dict[str, torch.Tensor]) -> None:
-        """All tensors of a layer's mixers: their input projections become one weight (attention q, k, v, then linear
-        attention q, k, v, gate, then the input of a dense feed-forward beside them) and their output projections one,
-        side by side along the input. Both are padded with zeros to the multiples of eight that the GEMM takes."""
+        """All tensors of a layer's mixers: their input projections become one weight (attention q, k, v and gate, or
+        q, latent and gate, or the recurrence's two branches, then linear attention q, k, v, gate, then the input of a
+        dense feed-forward beside them) and their output projections one, side by side along the input. Both are padded
+        with zeros to the multiples of eight that the GEMM takes."""
         spec = self.cfg.layers[self._layer_of(key)]
         pa, pl = mixer_prefixes(spec)
-        rows, biases, outs = [], [], []
-        shared = spec.attn is not None and spec.attn.shared_kv
-        for pre, names, has_bias in ((pa, "qk" if shared else "qkv", spec.attn is not None and spec.attn.qkv_bias), (pl, "qkvg", False)):
-            if pre is None:
-                continue
-            for x in names:
-                w = p[pre + x]
-                rows.append(w)
-                biases.append(p[pre + x + ".b"] if has_bias else torch.zeros(w.shape[0], dtype=w.dtype, device=w.device))
-            outs.append(p[pre + "o"])
+        names, outs = [], []
+        if spec.attn is not None:
+            a = spec.attn
+            names += [pa + x for x in ("q" if a.kv_from is not None else "qk" if a.shared_kv else "qkv")]
+            names += [pa + "g"] if a.head_gate else []
+            outs.append(pa + "o")
+        if spec.latent is not None:
+            names += ["q", "dkv"] + (["g"] if spec.latent.head_gate else [])
+            outs.append("o")
+        if spec.recurrence is not None:
+            names += ["y", "x"]
+            outs.append("o")
+        if spec.linear is not None:
+            names += [pl + x for x in "qkvg"]
+            outs.append(pl + "o")
         if spec.parallel and spec.ff:
-            for x in ("gate", "up") if spec.gated else ("up",):
-                rows.append(p["ff." + x])
-                biases.append(torch.zeros(spec.ff, dtype=rows[-1].dtype, device=rows[-1].device))
-            outs.append(p["ff.down"])
+            names += ["ff.gate", "ff.up"] if spec.gated else ["ff.up"]
+            outs.append("ff.down")
         pad = torch.nn.functional.pad
-        w_in, w_out = torch.cat(rows, 0), torch.cat(outs, 1)
+        w_in, w_out = torch.cat([p[n] for n in names], 0), torch.cat([p[n] for n in outs], 1)
         extra = -w_in.shape[0] % 8
         self._put_linear(key + ".in_proj", pad(w_in, (0, 0, 0, extra)))
-        if spec.attn is not None and spec.attn.qkv_bias:
+        if any(n + ".b" in p for n in names):
+            biases = [p[n + ".b"] if n + ".b" in p else p[n].new_zeros(p[n].shape[0]) for n in names]
             self._put(key + ".in_proj.bias", pad(torch.cat(biases, 0), (0, extra)))
         self._put_linear(key + ".o_proj", pad(w_out, (0, -w_out.shape[1] % 8)))
-        for pre, name, out in ((pa, "q.norm", "q_norm"), (pa, "k.norm", "k_norm"), (pa, "rel", "rel"), (pl, "norm", "norm")):
+        if spec.attn is not None and spec.attn.o_bias:
+            self._put(key + ".o_proj.bias", p[pa + "o.b"])
+        if spec.latent is not None:
+            a = spec.latent
+            self._put(key + ".w_uk", p["uk"].view(a.heads, a.dim, a.rank))
+            self._put(key + ".w_uv", p["uv"].view(a.heads, a.vdim, a.rank))
+        f32 = [(pa, "q.norm", "q_norm"), (pa, "k.norm", "k_norm"), (pa, "rel", "rel"), (pl, "norm", "norm")]
+        if spec.latent is not None:
+            f32.append(("", "dkv.norm", "latent_norm"))
+        if spec.recurrence is not None:
+            f32 += [("", "conv", "conv"), ("", "conv.b", "conv_b"), ("", "lam", "lam")]
+            self._put(key + ".gates", torch.stack((p["ra"], p["ri"])))
+            self._put(key + ".gates_b", torch.stack((p["ra.b"].reshape(-1), p["ri.b"].reshape(-1))).float(), keep_dtype=True)
+        for pre, name, out in f32:
             if pre is not None and pre + name in p:
                 self.out[f"{key}.{out}"] = self._own(p[pre + name].float())
 
@@ -1061,6 +1163,13 @@ class WeightLoader:
                 gate, up = gu[:half], gu[half:]
             if up is None:
                 continue
+            extra = -up.shape[0] % 8 if cfg.layers else 0
+            if extra:  # zero columns up to the multiple of eight the GEMM takes (every activation here maps 0 to 0)
+                pad = torch.nn.functional.pad
+                gate = pad(gate, (0, 0, 0, extra)) if gate is not None else None
+                up, down = pad(up, (0, 0, 0, extra)), pad(down, (0, extra))
+                if pre + "up_proj.bias" in p:
+                    p[pre + "up_proj.bias"] = pad(p[pre + "up_proj.bias"], (0, extra))
             gs, us, ds = (p.get(pre + f"{x}_proj.weight_scale_inv") for x in ("gate", "up", "down"))
             if gate is not None:
                 fused = _cat0((_rows(gate, r, n), _rows(up, r, n)))

@@ -1,12 +1,15 @@
 """Layers whose sequence mixers have sizes of their own, described by :class:`LayerSpec`: softmax attention over a
-window (with a learned distance bias, first tokens that stay visible, or values that are the keys), and linear attention
-with a fixed decay per head, alone or side by side.
+window or everything (with rotation, a learned distance bias, first tokens that stay visible, values that are the keys,
+capped scores, a sink, a gate per head, or another layer's keys and values), latent attention, a gated linear recurrence,
+and linear attention with a fixed decay per head, alone or beside windowed attention.
 
-Both mixers of a layer read the same normalised input, so their input projections are one GEMM and their outputs go
+All mixers of a layer read the same normalised input, so their input projections are one GEMM and their outputs go
 into one buffer that a single output projection reads. A dense feed-forward that reads that input too (``parallel``) is
-part of the same two GEMMs. A layer's cache is the pair (paged keys / values, state pool); either is an empty tensor
-where the layer does not have that mixer. A layer that runs several times has one :class:`MixerLayer` per run, over the
-same weights.
+part of the same two GEMMs. A layer's cache is the pair (paged keys / values or latents, state pool); either is an empty
+tensor where the layer does not have that mixer. A layer that runs several times has one :class:`MixerLayer` per run, over
+the same weights.
+
+Where the model has ``streams``, the residual is [T, streams, H] and each sublayer has a :class:`HyperConnection`.
 """
 from __future__ import annotations
 
@@ -16,45 +19,58 @@ from typing import Dict, NamedTuple, Optional, Tuple
 import torch
 
 from .. import ops
-from ..config.model_config import AttentionSpec, LayerSpec, LinearAttentionSpec, ModelConfig
+from ..config.model_config import (AttentionSpec, LatentAttentionSpec, LayerSpec, LinearAttentionSpec, ModelConfig,
+                                   RecurrenceSpec, RotarySpec)
 from ..ops import reference as ref
 from .layers import DenseFFN, LinearW, MoEFFN
 
 
 class LayerCache(NamedTuple):
-    kv: torch.Tensor     # [num_blocks, kv_heads * block_size * (dim + vdim)], without the values where they are the keys
-    state: torch.Tensor  # [num_slots, heads, dim, vdim] fp32
+    # [num_blocks, kv_heads * block_size * (dim + vdim)], without the values where they are the keys, or
+    # [num_blocks, block_size * (rank + rot_dim)] of latents
+    kv: torch.Tensor
+    state: torch.Tensor  # [num_slots, *state_shape] fp32
 
 
 class RotaryTables:
-    """cos / sin rows of every (dims, base) pair the model's layers use, grown to the longest position needed."""
+    """cos / sin rows of every rotation the model's layers use, grown to the longest position needed."""
 
     def __init__(self, device):
         self.device = device
         self.length = 0
-        self._tables: Dict[tuple, torch.Tensor] = {}
+        self._specs: Dict[str, RotarySpec] = {}
+        self._tables: Dict[str, torch.Tensor] = {}
+
+    def _build(self, key: str) -> None:
+        r = self._specs[key]
+        self._tables[key] = ref.rotary_table(r.dims, r.base, max(self.length, 1), self.device, r.scaling)
 
     def reserve(self, length: int) -> None:
         if length > self.length:
             self.length = length
-            for dims, base in self._tables:
-                self._tables[(dims, base)] = ref.rotary_table(dims, base, length, self.device)
+            for key in self._tables:
+                self._build(key)
 
-    def get(self, dims: int, base: float) -> torch.Tensor:
-        t = self._tables.get((dims, base))
-        if t is None:
-            t = self._tables[(dims, base)] = ref.rotary_table(dims, base, max(self.length, 1), self.device)
-        return t
+    def get(self, spec: RotarySpec) -> torch.Tensor:
+        key = repr(spec)
+        if key not in self._tables:
+            self._specs[key] = spec
+            self._build(key)
+        return self._tables[key]
 
 
 class WindowedAttention:
-    def __init__(self, cfg: ModelConfig, spec: AttentionSpec, w: Dict[str, torch.Tensor], prefix: str):
-        self.spec, self.eps = spec, cfg.rms_norm_eps
+    def __init__(self, cfg: ModelConfig, spec: AttentionSpec, w: Dict[str, torch.Tensor], prefix: str,
+                 tables: RotaryTables):
+        self.spec, self.eps, self.tables = spec, cfg.rms_norm_eps, tables
         self.nq, self.nk = spec.heads * spec.dim, spec.kv_heads * spec.dim
         self.nv = 0 if spec.shared_kv else spec.kv_heads * spec.vdim
-        if spec.shared_kv and (spec.qk_norm or spec.qkv_bias):
+        if spec.shared_kv and (spec.qk_norm or spec.qkv_bias or spec.rot or spec.head_gate or spec.kv_from is not None):
             raise NotImplementedError("keys that are the values are cached as projected")
-        self.rows = self.nq + self.nk + self.nv
+        self.page = self.nk + self.nv  # cache elements per token
+        if spec.kv_from is not None:
+            self.nk = self.nv = 0
+        self.rows = self.nq + self.nk + self.nv + (spec.heads if spec.head_gate else 0)
         self.width = spec.heads * spec.vdim
         self.q_norm, self.k_norm = w.get(prefix + ".q_norm"), w.get(prefix + ".k_norm")
         self.rel = w.get(prefix + ".rel")
@@ -65,22 +81,83 @@ class WindowedAttention:
         if self.rel is not None and (self.bias is None or self.bias.shape[1] < reach):
             self.bias = ref.distance_bias(self.rel, self.spec.bias_max, reach)
 
+    def rotary(self) -> Optional[torch.Tensor]:
+        return self.tables.get(self.spec.rot) if self.spec.rot is not None else None
+
     def run(self, x: torch.Tensor, meta, kv: torch.Tensor, out: torch.Tensor,
             ff: Optional[Tuple[torch.Tensor, torch.Tensor, bool]] = None) -> None:
         """x [T, rows] = the projected (q | k | v); writes heads * vdim columns of ``out``. ``ff`` = (input, output,
         gated) of a feed-forward's activation that runs in the launch of the cache append (keys = values only)."""
         s = self.spec
         q = x[:, :self.nq].unflatten(1, (s.heads, s.dim))
-        k = x[:, self.nq:self.nq + self.nk].unflatten(1, (s.kv_heads, s.dim))
-        bs = kv.shape[1] // (self.nk + self.nv)
+        k = x[:, self.nq:self.nq + self.nk].unflatten(1, (s.kv_heads, s.dim)) if self.nk else None
+        end = self.nq + self.nk + self.nv
+        bs = kv.shape[1] // self.page
         if s.shared_kv:
             u, act, gated = ff if ff is not None else (None, None, False)
             ops.append_act(k, u, meta.slot_mapping, kv, bs, act, gated)
         else:
-            v = x[:, self.nq + self.nk:].unflatten(1, (s.kv_heads, s.vdim))
-            ops.qk_norm_cache(q, k, v, meta.slot_mapping, kv, bs, self.q_norm, self.k_norm, self.eps)
+            v = x[:, self.nq + self.nk:end].unflatten(1, (s.kv_heads, s.vdim)) if self.nk else None
+            if k is not None or s.rot is not None or self.q_norm is not None:
+                ops.qk_norm_cache(q, k, v, meta.slot_mapping, kv, bs, self.q_norm, self.k_norm, self.eps, meta.positions,
+                                  self.rotary())
         ops.window_attention(q, kv, meta, bs, s.kv_heads, s.vdim, s.scale, s.window, self.bias, s.out_scale, out,
-                             s.keep_first)
+                             s.keep_first, s.softcap, s.sink, x[:, end:end + s.heads] if s.head_gate else None)
+
+
+class LatentWeights:
+    """The maps from the latent to keys and values, in the layouts its kernels want."""
+
+    def __init__(self, uk: torch.Tensor, uv: torch.Tensor):
+        self.uk, self.uv = uk, uv                             # [h, dim, rank], [h, vdim, rank]
+        self.h, self.dim, self.rank = uk.shape
+        self.vdim = uv.shape[1]
+        self.uk_t = uk.transpose(1, 2).contiguous()           # [h, rank, dim]: absorbed into the query
+        # [h * (dim + vdim), rank]: all heads' keys, then all heads' values, written out by one GEMM
+        self.expand = torch.cat((uk.reshape(-1, self.rank), uv.reshape(-1, self.rank)), 0).contiguous()
+
+
+class LatentAttention:
+    def __init__(self, cfg: ModelConfig, spec: LatentAttentionSpec, w: Dict[str, torch.Tensor], prefix: str,
+                 tables: RotaryTables):
+        self.spec, self.eps, self.tables = spec, cfg.rms_norm_eps, tables
+        self.nq, self.na = spec.heads * (spec.dim + spec.rot_dim), spec.rank + spec.rot_dim
+        self.rows = self.nq + self.na + (spec.heads if spec.head_gate else 0)
+        self.width = spec.heads * spec.vdim
+        self.norm = w[prefix + ".latent_norm"]
+        self.w = LatentWeights(w[prefix + ".w_uk"], w[prefix + ".w_uv"])
+
+    def reserve(self, length: int) -> None:
+        pass
+
+    def rotary(self) -> torch.Tensor:
+        return self.tables.get(self.spec.rot)
+
+    def run(self, x: torch.Tensor, meta, kv: torch.Tensor, out: torch.Tensor) -> None:
+        """x [T, rows] = the projected (q | latent, rotated key part | gate); writes heads * vdim columns of ``out``."""
+        s = self.spec
+        q = x[:, :self.nq].unflatten(1, (s.heads, s.dim + s.rot_dim))
+        bs = kv.shape[1] // s.width
+        ops.latent_append(q, x[:, self.nq:self.nq + self.na], self.norm, self.eps, meta.positions, self.rotary(),
+                          meta.slot_mapping, kv, bs)
+        gate = x[:, self.nq + self.na:self.nq + self.na + s.heads] if s.head_gate else None
+        ops.latent_attention(q, kv, meta, bs, self.w, s.scale, gate, out)
+
+
+class GatedRecurrence:
+    def __init__(self, cfg: ModelConfig, spec: RecurrenceSpec, w: Dict[str, torch.Tensor], prefix: str):
+        self.spec = spec
+        self.rows, self.width = 2 * spec.width, spec.width
+        self.conv, self.conv_b = w[prefix + ".conv"], w[prefix + ".conv_b"]        # [C, K], [C] fp32
+        self.gates, self.gates_b = w[prefix + ".gates"], w[prefix + ".gates_b"]    # [2, B, C / B, C / B], [2, C] fp32
+        lam = w[prefix + ".lam"].double()
+        self.rate = (spec.decay_scale * torch.nn.functional.softplus(lam, threshold=100)).float()
+
+    def run(self, x: torch.Tensor, meta, state: torch.Tensor, out: torch.Tensor) -> None:
+        """x [T, rows] = the projected (y | x); writes ``width`` columns of ``out``."""
+        C = self.spec.width
+        ops.gated_recurrence(x[:, :C], x[:, C:2 * C], state, meta, self.conv, self.conv_b, self.gates, self.gates_b,
+                             self.rate, out)
 
 
 class DecayedLinearAttention:
@@ -94,7 +171,7 @@ class DecayedLinearAttention:
         self.norm = w[prefix + ".norm"] if spec.norm == "concat" else None
 
     def rotary(self) -> Optional[torch.Tensor]:
-        return self.tables.get(self.spec.rot_dims, self.spec.rot_base) if self.spec.rot_dims else None
+        return self.tables.get(RotarySpec(self.spec.rot_dims, self.spec.rot_base)) if self.spec.rot_dims else None
 
     def run(self, x: torch.Tensor, meta, state: torch.Tensor, out: torch.Tensor) -> None:
         """x [T, rows] = the projected (q | k | v | gate); writes heads * vdim columns of ``out``."""
@@ -111,6 +188,14 @@ class PassStart(NamedTuple):
     """What the stream takes ahead of one pass of a loop."""
     step: torch.Tensor      # [H] fp32, the pass's learned vector
     add_start: bool         # also the embedding output: every pass but the first
+
+
+class HyperConnection:
+    """How one sublayer reads the residual streams and what they become: u = sum_s inp[s] x_s;
+    x_t <- sum_s mix[s, t] x_s + out[t] y."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str):
+        self.inp, self.out, self.mix = (w[f"{prefix}.{n}"].contiguous() for n in ("in", "out", "mix"))
 
 
 class MixerLayer:
@@ -131,15 +216,24 @@ class MixerLayer:
         self.ln2, self.ln2_b = w.get(p + ".post_attention_layernorm.weight"), None
         self.in_proj, self.o_proj = LinearW(w, p + ".mixer.in_proj"), LinearW(w, p + ".mixer.o_proj")
         device = self.ln1.device
-        self.attn = WindowedAttention(cfg, spec.attn, w, p + ".mixer") if spec.attn else None
+        self.attn = WindowedAttention(cfg, spec.attn, w, p + ".mixer", tables) if spec.attn else None
+        self.latent = LatentAttention(cfg, spec.latent, w, p + ".mixer", tables) if spec.latent else None
+        self.recurrence = GatedRecurrence(cfg, spec.recurrence, w, p + ".mixer") if spec.recurrence else None
         self.linear = DecayedLinearAttention(cfg, spec.linear, w, p + ".mixer", device, tables) if spec.linear else None
-        self.ffn = DenseFFN(cfg, w, p + ".mlp", tp) if spec.ff and not spec.parallel else None
+        self.hyper = [HyperConnection(w, f"{p}.hc{n}") for n in ((1, 2) if spec.has_ff else (1,))] if cfg.streams else []
+        self.ls1, self.ls2 = (w.get(f"{p}.ls{n}") if spec.layer_scale else None for n in (1, 2))
+        if spec.layer_scale and not cfg.streams:
+            raise NotImplementedError("scales per layer come with residual streams")
+        self.ffn = None
+        if spec.ff and not spec.parallel:
+            self.ffn = DenseFFN(replace(cfg, layers=[], hidden_act=spec.ff_act or cfg.hidden_act, gated_mlp=spec.gated), w,
+                                p + ".mlp", tp)
         self.experts = None
         if spec.moe is not None:
             m = spec.moe
             self.experts = MoEFFN(replace(cfg, layers=[], num_experts=m.experts, num_experts_per_tok=m.top,
-                                          moe_intermediate_size=m.ff, scoring_func="topk_softmax",
-                                          num_shared_experts=0), w, p + ".mlp", tp)
+                                          moe_intermediate_size=m.ff, scoring_func="topk_softmax", n_group=m.groups,
+                                          topk_group=m.keep, num_shared_experts=0), w, p + ".mlp", tp)
             if m.router_bias and self.experts.logit_bias is None:
                 raise KeyError(f"missing {p}.mlp.gate.bias")
             if self.experts.q4 is not None or self.experts.s_gate_up is not None:
@@ -147,8 +241,8 @@ class MixerLayer:
         self.parallel_ff = spec.ff if spec.parallel else 0
         if self.parallel_ff and (self.linear is not None or self.attn is None or not spec.attn.shared_kv):
             raise NotImplementedError("a dense feed-forward runs beside attention whose values are its keys")
-        if self.experts is not None and not spec.parallel:
-            raise NotImplementedError("routed experts run beside the mixers")
+        if self.experts is not None and spec.parallel == bool(cfg.streams):
+            raise NotImplementedError("routed experts run beside the mixers, or behind them over several streams")
 
     # ---- per-sequence memory ---------------------------------------------------------------------------------
     def kv_width(self) -> int:
@@ -157,6 +251,10 @@ class MixerLayer:
 
     def state_shape(self):
         return self.spec.state_shape or (0, 0, 0)
+
+    def kv_from(self) -> Optional[int]:
+        """The layer whose cache this one reads (None: its own)."""
+        return self.spec.attn.kv_from if self.spec.attn is not None else None
 
     def reserve(self, length: int) -> None:
         if self.attn is not None:
@@ -169,7 +267,12 @@ class MixerLayer:
                                self.ln1.dtype, **more)
 
     def start(self, x: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
-        """First layer of the model: (its normalised input, the stream) from the embedding output, which stays as it is."""
+        """First layer of the model: (its normalised input, the stream) from the embedding output, which stays as it is.
+        With several streams all of them equal it until the first sublayer's result arrives: nothing is copied."""
+        if self.hyper:
+            h = ops.hyper_norm(None, None, None, x, None, None, None, self.hyper[0].inp, self.ln1, self.cfg.rms_norm_eps,
+                               self.ln1.dtype)
+            return h, torch.empty(x.shape[0], self.cfg.streams, x.shape[1], dtype=torch.float32, device=x.device)
         residual = torch.empty_like(x)
         h = ops.stream_norm(None, self.ln1, self.cfg.rms_norm_eps, self.cfg.norm_type == "layernorm", x, residual,
                             self.ln1.dtype, add_vec=self.pass_start.step if self.pass_start else None)
@@ -177,7 +280,8 @@ class MixerLayer:
 
     def mix(self, h: torch.Tensor, meta, cache: LayerCache) -> torch.Tensor:
         x = self.in_proj(h)
-        widths = [m.width for m in (self.attn, self.linear) if m is not None] + [self.parallel_ff]
+        widths = [m.width for m in (self.attn, self.latent, self.linear, self.recurrence) if m is not None]
+        widths.append(self.parallel_ff)
         K, used = self.o_proj.in_features, sum(widths)
         buf = torch.empty(h.shape[0], K, dtype=h.dtype, device=h.device)
         if K > used:
@@ -188,16 +292,36 @@ class MixerLayer:
             self.attn.run(x[:, :self.attn.rows], meta, cache.kv, buf[:, :widths[0]], ff)
             return buf
         row = col = 0
-        for m, mem in ((self.attn, cache.kv), (self.linear, cache.state)):
+        for m, mem in ((self.attn, cache.kv), (self.latent, cache.kv), (self.linear, cache.state),
+                       (self.recurrence, cache.state)):
             if m is not None:
                 m.run(x[:, row:row + m.rows], meta, mem, buf[:, col:col + m.width])
                 row, col = row + m.rows, col + m.width
         return buf
 
+    def _streams(self, h: torch.Tensor, residual: torch.Tensor, meta, cache: LayerCache, next_norm, next_in):
+        eps, dtype = self.cfg.rms_norm_eps, self.ln1.dtype
+        y = self.o_proj(self.mix(h, meta, cache))
+        old = meta.start if self.idx == 0 else residual  # ahead of the first result all streams are the embedding output
+        c = self.hyper[0]
+        if not self.spec.has_ff:
+            return ops.hyper_norm(y, self.ls1, None, old, c.mix, c.out, residual, next_in, next_norm, eps, dtype)
+        h = ops.hyper_norm(y, self.ls1, None, old, c.mix, c.out, residual, self.hyper[1].inp, self.ln2, eps, dtype)
+        y = routed = None
+        if self.experts is not None:
+            routed = self.experts.rows(h, self.spec.moe.limit, self.spec.moe.alpha)
+        else:
+            y = self.ffn.down(self.ffn.core(h))
+        c = self.hyper[1]
+        return ops.hyper_norm(y, self.ls2, routed, residual, c.mix, c.out, residual, next_in, next_norm, eps, dtype)
+
     def forward(self, h: torch.Tensor, residual: torch.Tensor, meta, cache: LayerCache, next_norm, next_norm_b=None,
-                pass_start: Optional[PassStart] = None):
+                pass_start: Optional[PassStart] = None, next_in: Optional[torch.Tensor] = None):
         """Same contract as DecoderLayer.forward: consumes the normalised input, returns the next layer's.
-        ``pass_start``: the next run's, if it starts a pass; the embedding output is ``meta.start``."""
+        ``pass_start``: the next run's, if it starts a pass; the embedding output is ``meta.start``. ``next_in``: how the
+        next sublayer reads the streams, where there are several."""
+        if self.hyper:
+            return self._streams(h, residual, meta, cache, next_norm, next_in)
         y = self.o_proj(self.mix(h, meta, cache))
         if self.ffn is not None:
             h = self._norm(y, self.ln2, residual)

@@ -37,6 +37,8 @@ FAMILIES: Dict[str, str] = {
                "bias; recurrent state slots, LayerNorm, 32-bit residual, soft-capped logits",
     "givirax": "attention over a window and the first tokens whose values are its keys, beside a GELU or routed "
                "feed-forward under one norm; learned positions, looped layers, 32-bit residual",
+    "ladusun": "latent attention, capped attention with a sink (keys and values shared between layers) or a gated linear "
+               "recurrence; clamped experts routed by groups, hyper-connected residual streams in 32-bit",
     "minicpm": "embedding / residual / logit scaling; reranker head",
 }
 

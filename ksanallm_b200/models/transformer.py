@@ -103,6 +103,9 @@ class TransformerModel:
             # one entry per run: a layer inside a loop appears once per pass, with a cache of its own
             self.layers = [MixerLayer(cfg, weights, i, self.tp, self.rotary_tables, t) for i, t in cfg.layer_runs()]
             self.reserve_positions(min(max_positions or 1, maxp))
+            self.stream_sum = torch.ones(cfg.streams, device=self.device) if cfg.streams else None
+            if cfg.loop is not None and (cfg.streams or any(l.kv_from() is not None for l in self.layers)):
+                raise NotImplementedError("loops over layers with several streams or shared keys")
         else:
             self.layers = [DecoderLayer(cfg, weights, i, self.tp, self.rope_cache) for i in self.layer_ids]
         self.norm_w = weights.get("model.norm.weight")
@@ -196,7 +199,8 @@ class TransformerModel:
         stream for the next stage. ``states``: the recurrent-state pools of a model that has them."""
         if self.cfg.layers:
             states = states if states is not None else [kv.new_empty(0, dtype=torch.float32) for kv in kv_caches]
-            kv_caches = [LayerCache(kv, st) for kv, st in zip(kv_caches, states)]
+            owner = [i if layer.kv_from() is None else layer.kv_from() for i, layer in enumerate(self.layers)]
+            kv_caches = [LayerCache(kv_caches[i], st) for i, st in zip(owner, states)]
         x = self.embed_tokens(meta, refit) if hidden_in is None else hidden_in
         layers = self.layers if cutoff_layer is None else self.layers[:cutoff_layer]
         residual = x
@@ -224,6 +228,8 @@ class TransformerModel:
             nxt = layers[li + 1] if li + 1 < len(layers) else None
             nw, nb = (nxt.ln1, nxt.ln1_b) if nxt is not None else (self.norm_w, self.norm_b)
             more = (nxt.pass_start,) if self.cfg.loop is not None and nxt is not None else ()
+            if self.cfg.streams:
+                more = (None, nxt.hyper[0].inp if nxt is not None else self.stream_sum)
             h = layer.forward(h, residual, meta, kv_caches[li], nw, nb, *more)
             if self.progress is not None:
                 self.progress.record(li)  # parallel.transfer.LayerProgressTracker: KV of layer li may leave now

@@ -42,6 +42,13 @@ def stream_norm(x, weight, eps, center, stream_in, stream_out=None, out_dtype=No
     return f.stream_norm(x, weight, eps, center, stream_in, stream_out, out_dtype, add_rows, add_vec, routed)
 
 
+def hyper_norm(x, scale, routed, streams, mix, out_w, streams_out, in_w, weight, eps, out_dtype):
+    """Residual streams take a sublayer's result and the next sublayer's input is normalised; see
+    ``reference.hyper_norm``."""
+    f = _mixer() if streams.is_cuda else ref
+    return f.hyper_norm(x, scale, routed, streams, mix, out_w, streams_out, in_w, weight, eps, out_dtype)
+
+
 def _library_baseline() -> bool:
     """KSANA_LIBRARY_BASELINE=1 routes dense GEMMs to cuBLAS (torch.matmul): the measured stand-in for the
     reference's cuBLAS + NCCL build, never the default."""
@@ -88,6 +95,8 @@ def gelu_and_mul(x):
 def activation(x, kind):
     if x.is_cuda and kind == "gelu_tanh":
         return _mixer().gelu(x)
+    if x.is_cuda and kind == "relu2":
+        return _mixer().relu2(x)
     return ref.activation(x, kind)
 
 
@@ -121,9 +130,34 @@ def paged_attention(q, kv_cache, meta, scale, alibi_slopes=None, k_scale=1.0, v_
                                k_scale, v_scale, window)
 
 
-def qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps):
+def qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps, positions=None, rotary=None):
     f = _mixer() if q.is_cuda else ref
-    return f.qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps)
+    return f.qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps, positions, rotary)
+
+
+def latent_append(q, a, norm_w, eps, positions, rotary, slot_mapping, cache, block_size):
+    f = _mixer() if q.is_cuda else ref
+    f.latent_append(q, a, norm_w, eps, positions, rotary, slot_mapping, cache, block_size)
+
+
+def latent_attention(q, cache, meta, block_size, w, scale, gate, out):
+    """``w``: :class:`~ksanallm_b200.models.mixers.LatentWeights`. Writes heads * vdim columns of ``out``."""
+    if q.is_cuda:
+        from . import cuda_latent
+        cuda_latent.latent_attention(q, cache, meta, block_size, w, scale, gate, out)
+        return
+    out.copy_(ref.latent_attention(q, cache, meta.block_tables, meta.cu_q, meta.kv_lens, block_size, w.uk, w.uv, scale,
+                                   gate).flatten(1))
+
+
+def gated_recurrence(y, x, state, meta, conv_w, conv_b, w_gates, b_gates, rate, out):
+    """Writes ``out`` [T, C] (a column slice is fine)."""
+    if x.is_cuda:
+        from . import cuda_recurrence
+        cuda_recurrence.gated_recurrence(y, x, state, meta, conv_w, conv_b, w_gates, b_gates, rate, out)
+        return
+    out.copy_(ref.gated_recurrence(y, x, state, meta.state_slots, meta.cu_q, meta.kv_lens, conv_w, conv_b, w_gates,
+                                   b_gates, rate))
 
 
 def append_act(k, u, slot_mapping, cache, block_size, out, gated=False):
@@ -132,15 +166,16 @@ def append_act(k, u, slot_mapping, cache, block_size, out, gated=False):
     f.append_act(k, u, slot_mapping, cache, block_size, out, gated)
 
 
-def window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out, keep_first=0):
+def window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out, keep_first=0,
+                     softcap=0.0, sink=False, gate=None):
     """Writes heads * vdim columns of ``out`` [T, ...] (a column slice is fine). Whether the cache holds values of their
     own or the keys are the values shows in its width."""
     if q.is_cuda:
         _mixer().window_attention(q, cache, meta, block_size, kv_heads, vdim, scale, window, bias, out_scale, out,
-                                  keep_first)
+                                  keep_first, softcap, sink, gate)
         return
     out.copy_(ref.window_attention(q, cache, meta.block_tables, meta.cu_q, meta.kv_lens, block_size, kv_heads, vdim,
-                                   scale, window, bias, out_scale, keep_first).flatten(1))
+                                   scale, window, bias, out_scale, keep_first, softcap, sink, gate).flatten(1))
 
 
 def linear_attention(q, k, v, state, meta, decay, act, rotary, key_scale):
@@ -182,18 +217,18 @@ def moe_route(logits, top_k, scoring="softmax", norm_topk=False, n_group=1, topk
     return ref.moe_route(logits, top_k, scoring, norm_topk, n_group, topk_group, routed_scale, correction_bias)
 
 
-def moe_topk(logits, experts, top_k, bias=None):
+def moe_topk(logits, experts, top_k, bias=None, groups=1, keep=1):
     if logits.is_cuda:
         from . import cuda_moe
-        return cuda_moe.moe_topk(logits, experts, top_k, bias)
-    return ref.moe_topk(logits, experts, top_k, bias)
+        return cuda_moe.moe_topk(logits, experts, top_k, bias, groups, keep)
+    return ref.moe_topk(logits, experts, top_k, bias, groups, keep)
 
 
-def moe_expert_rows(x, ids, w_gate_up, w_down):
+def moe_expert_rows(x, ids, w_gate_up, w_down, limit=0.0, alpha=1.0):
     if x.is_cuda:
         from . import cuda_moe
-        return cuda_moe.expert_pipeline(x, ids, w_gate_up, w_down)
-    return ref.moe_expert_rows(x, ids, w_gate_up, w_down)
+        return cuda_moe.expert_pipeline(x, ids, w_gate_up, w_down, 0, limit, alpha)
+    return ref.moe_expert_rows(x, ids, w_gate_up, w_down, limit, alpha)
 
 
 def moe_experts(x, ids, weights, w_gate_up, w_down, expert_offset=0):

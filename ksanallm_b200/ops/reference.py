@@ -67,6 +67,32 @@ def stream_norm(x: Optional[torch.Tensor], weight: torch.Tensor, eps: float, cen
     return (v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(out_dtype or stream_in.dtype)
 
 
+def hyper_norm(x: Optional[torch.Tensor], scale: Optional[torch.Tensor], routed, streams: torch.Tensor,
+               mix: Optional[torch.Tensor], out_w: Optional[torch.Tensor], streams_out: Optional[torch.Tensor],
+               in_w: torch.Tensor, weight: torch.Tensor, eps: float, out_dtype: torch.dtype) -> torch.Tensor:
+    """Hyper-connected residual streams between two sublayers. With y = (x + weighted rows of ``routed``, see
+    :func:`stream_norm`) * scale, every stream becomes sum_s mix[s, t] streams[s] + out_w[t] y (``mix`` None: the streams
+    stay as they are); returns the RMS norm of sum_t in_w[t] of the new ones. ``streams`` [T, S, H] fp32, or [T, H] where
+    all S are still equal; the new ones go to ``streams_out`` [T, S, H] (``streams`` itself is fine, None: nowhere)."""
+    S = in_w.shape[0]
+    v = streams.float()
+    if v.dim() == 2:
+        v = v.unsqueeze(1).expand(-1, S, -1)
+    if mix is not None:
+        y = x.float() if x is not None else torch.zeros_like(v[:, 0])
+        if routed is not None:
+            rows, pos, w = routed
+            p = pos.view(w.shape).long()
+            y = y + torch.einsum("tk,tkh->th", w.masked_fill(p < 0, 0.0), rows[p.clamp(min=0)].float())
+        if scale is not None:
+            y = y * scale
+        v = torch.einsum("st,nsh->nth", mix, v) + out_w.view(1, S, 1) * y.unsqueeze(1)
+        if streams_out is not None:
+            streams_out.copy_(v)
+    u = torch.einsum("s,nsh->nh", in_w, v)
+    return (u / torch.sqrt(u.pow(2).mean(-1, keepdim=True) + eps) * weight.float()).to(out_dtype)
+
+
 # ---- dense linear algebra -------------------------------------------------------------------------
 
 def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] = None,
@@ -99,6 +125,8 @@ def activation(x: torch.Tensor, kind: str) -> torch.Tensor:
         y = F.gelu(xf, approximate="tanh")
     elif kind == "relu":
         y = F.relu(xf)
+    elif kind == "relu2":
+        y = F.relu(xf).square()
     elif kind in ("silu", "swish"):
         y = F.silu(xf)
     elif kind == "sigmoid":
@@ -366,27 +394,40 @@ def paged_attention(q: torch.Tensor, kv_cache: torch.Tensor, block_tables: torch
 
 def split_kv_cache(cache: torch.Tensor, hk: int, bs: int, d: int, dv: int) -> Tuple[torch.Tensor, torch.Tensor]:
     """Views [nb, hk, bs, d] and [nb, hk, bs, dv] of a layer cache [nb, hk * bs * (d + dv)] (keys, then values), or of a
-    cache of keys alone that are the values too."""
+    cache of keys alone whose first dv numbers are the values too."""
     nb, cut = cache.shape[0], hk * bs * d
     if cache.shape[1] == cut:
         K = cache.view(nb, hk, bs, d)
-        return K, K
+        return K, K[..., :dv]
     return cache[:, :cut].view(nb, hk, bs, d), cache[:, cut:].view(nb, hk, bs, dv)
 
 
-def qk_norm_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, slot_mapping: torch.Tensor, cache: torch.Tensor,
-                  block_size: int, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor], eps: float) -> None:
-    """Per-head RMS norm of q (in place) and k, then k and v go to their cache slots. q [T, h, d], k [T, hk, d],
-    v [T, hk, dv] may be row-strided views; the cache has the layout of :func:`split_kv_cache`."""
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, rotary: torch.Tensor) -> torch.Tensor:
+    """The leading dimensions of x [T, heads, d] that ``rotary`` ([positions, dims] = [cos | sin]) covers, in neighbouring
+    pairs, turned by each token's row."""
+    cs = rotary[positions.long()]
+    half = cs.shape[1] // 2
+    return apply_rope(x, cs[:, :half], cs[:, half:], True, cs.shape[1])
+
+
+def qk_norm_cache(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], slot_mapping: torch.Tensor,
+                  cache: torch.Tensor, block_size: int, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor],
+                  eps: float, positions: Optional[torch.Tensor] = None, rotary: Optional[torch.Tensor] = None) -> None:
+    """Per-head RMS norm (if any), then rotation (if any), of q (in place) and k; then k and v go to their cache slots.
+    q [T, h, d], k [T, hk, d], v [T, hk, dv] may be row-strided views, k and v None (nothing is appended); the cache has
+    the layout of :func:`split_kv_cache`."""
+    def ready(x, w):
+        if w is not None:
+            xf = x.float()
+            x = (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(x.dtype)
+        return rotate_pairs(x, positions, rotary) if rotary is not None else x
+
+    if q_norm is not None or rotary is not None:
+        q.copy_(ready(q, q_norm))
+    if k is None:
+        return
     hk, d, dv = k.shape[1], k.shape[2], v.shape[2]
-
-    def unit(x, w):
-        xf = x.float()
-        return (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(x.dtype)
-
-    if q_norm is not None:
-        q.copy_(unit(q, q_norm))
-    kn = unit(k, k_norm) if k_norm is not None else k
+    kn = ready(k, k_norm)
     K, V = split_kv_cache(cache, hk, block_size, d, dv)
     slots = slot_mapping.long()
     blk, off = slots // block_size, slots % block_size
@@ -421,10 +462,12 @@ def distance_bias(rel: torch.Tensor, bias_max: float, count: int) -> torch.Tenso
 
 def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, cu_q: torch.Tensor,
                      kv_lens: torch.Tensor, block_size: int, hk: int, dv: int, scale: float, window: int,
-                     bias: Optional[torch.Tensor], out_scale: float = 1.0, keep_first: int = 0) -> torch.Tensor:
+                     bias: Optional[torch.Tensor], out_scale: float = 1.0, keep_first: int = 0, softcap: float = 0.0,
+                     sink: bool = False, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Softmax attention of each sequence's new tokens over its newest ``window`` keys (0: all) and its first
-    ``keep_first`` ones, with a bias per head and distance (``bias`` [h, >= reach], None: none). q [T, h, d]; returns
-    [T, h, dv]."""
+    ``keep_first`` ones, with a bias per head and distance (``bias`` [h, >= reach], None: none). ``softcap``: scores pass
+    through cap * tanh(score / cap) first. ``sink``: the denominator has one more term exp(0). ``gate`` [T, h]: each
+    head's result times its sigmoid. q [T, h, d]; returns [T, h, dv]."""
     T, h, d = q.shape
     K, V = split_kv_cache(cache, hk, block_size, d, dv)
     out = torch.empty(T, h, dv, dtype=q.dtype, device=q.device)
@@ -438,22 +481,88 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
         kb = K[blocks].permute(1, 0, 2, 3).reshape(hk, -1, d)[:, :L - lo].float().repeat_interleave(group, 0)
         vb = V[blocks].permute(1, 0, 2, 3).reshape(hk, -1, dv)[:, :L - lo].float().repeat_interleave(group, 0)
         s = torch.einsum("qhd,hkd->hqk", q[cu[b]:cu[b + 1]].float(), kb) * scale
+        if softcap:
+            s = softcap * torch.tanh(s / softcap)
         dist = torch.arange(L - ql, L, device=q.device).unsqueeze(1) - torch.arange(lo, L, device=q.device)
         if bias is not None:
             s = s + bias[:, dist.clamp(0, bias.shape[1] - 1)]
         hidden = dist < 0
         if window:
             hidden = hidden | (dist >= window) & (torch.arange(lo, L, device=q.device) >= keep_first)
-        p = torch.softmax(s.masked_fill(hidden.unsqueeze(0), float("-inf")), dim=-1)
-        out[cu[b]:cu[b + 1]] = (torch.einsum("hqk,hkd->qhd", p, vb) * out_scale).to(q.dtype)
+        s = s.masked_fill(hidden.unsqueeze(0), float("-inf"))
+        p = torch.softmax(torch.nn.functional.pad(s, (1, 0)), dim=-1)[..., 1:] if sink else torch.softmax(s, dim=-1)
+        o = torch.einsum("hqk,hkd->qhd", p, vb) * out_scale
+        if gate is not None:
+            o = o * torch.sigmoid(gate[cu[b]:cu[b + 1]].float()).unsqueeze(2)
+        out[cu[b]:cu[b + 1]] = o.to(q.dtype)
     return out
 
 
-def rotary_table(dims: int, base: float, count: int, device="cpu") -> torch.Tensor:
-    """[count, dims] fp32 = [cos | sin] of position * base^(-2 i / dims)."""
-    inv = base ** (-torch.arange(0, dims // 2, dtype=torch.float64) * 2 / dims)
-    a = torch.arange(count, dtype=torch.float64).unsqueeze(1) * inv
-    return torch.cat((a.cos(), a.sin()), 1).float().to(device)
+def latent_append(q: torch.Tensor, a: torch.Tensor, norm_w: torch.Tensor, eps: float, positions: torch.Tensor,
+                  rotary: torch.Tensor, slot_mapping: torch.Tensor, cache: torch.Tensor, block_size: int) -> None:
+    """What latent attention does between its projections and its scores: the rotated part of q (its last dimensions,
+    [T, h, dim + rot], in place) turns, and a [T, rank + rot] goes to the cache ([blocks, block_size * (rank + rot)]) as
+    [RMS-normed latent | rotated key part]."""
+    rd = rotary.shape[1]
+    rank = a.shape[1] - rd
+    q[..., -rd:] = rotate_pairs(q[..., -rd:], positions, rotary)
+    lat = a[:, :rank].float()
+    lat = lat / torch.sqrt(lat.pow(2).mean(-1, keepdim=True) + eps) * norm_w.float()
+    r = rotate_pairs(a[:, None, rank:], positions, rotary)[:, 0]
+    rows = cache.view(-1, block_size, rank + rd)
+    slots = slot_mapping.long()
+    rows[slots // block_size, slots % block_size] = torch.cat((lat, r.float()), 1).to(cache.dtype)
+
+
+def latent_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, cu_q: torch.Tensor,
+                     kv_lens: torch.Tensor, block_size: int, w_uk: torch.Tensor, w_uv: torch.Tensor, scale: float,
+                     gate: Optional[torch.Tensor]) -> torch.Tensor:
+    """q [T, h, dim + rot] (rotated) over the latent cache, with w_uk [h, dim, rank] absorbed into the query and
+    w_uv [h, vdim, rank] applied to the weighted latent. Returns [T, h, vdim]."""
+    dim, rank = w_uk.shape[1:]
+    q_lat = torch.einsum("thd,hdr->thr", q[..., :dim].float(), w_uk.float()).to(q.dtype)
+    o = window_attention(torch.cat((q_lat, q[..., dim:]), 2), cache, block_tables, cu_q, kv_lens, block_size, 1, rank,
+                         scale, 0, None, 1.0, 0, 0.0, False, gate)
+    return torch.einsum("thr,hvr->thv", o.float(), w_uv.float()).to(q.dtype)
+
+
+def gated_recurrence(y: torch.Tensor, x: torch.Tensor, state: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor,
+                     kv_lens: torch.Tensor, conv_w: torch.Tensor, conv_b: torch.Tensor, w_gates: torch.Tensor,
+                     b_gates: torch.Tensor, rate: torch.Tensor) -> torch.Tensor:
+    """The core of a gated linear recurrent block. x, y [T, C]: the two branches' projections (y before its GELU).
+    conv_w [C, K]: causal taps, the last one meets the current token. w_gates [2, B, C / B, C / B] ([out, in]) and
+    b_gates [2, C]: the block-diagonal maps of r and i. rate [C] = decay_scale * softplus(lam). A sequence's memory is
+    ``state[slot]`` [1, K, C] fp32: the recurrent state, then the last K - 1 inputs of the convolution, oldest first; a
+    sequence whose first token is among the new ones starts from zeros whatever its slot holds."""
+    T, C = x.shape
+    K, B = conv_w.shape[1], w_gates.shape[1]
+    out = torch.empty(T, C, dtype=x.dtype, device=x.device)
+    cu, kl, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
+    for b in range(len(kl)):
+        lo, hi = cu[b], cu[b + 1]
+        if hi == lo:
+            continue
+        mem = state[sl[b], 0]
+        if kl[b] == hi - lo:
+            mem = torch.zeros_like(mem)
+        xs = torch.cat((mem[1:], x[lo:hi].float()), 0)  # [K - 1 + n, C]
+        u = sum(xs[j:j + hi - lo] * conv_w[:, j] for j in range(K)) + conv_b
+        u = u.to(x.dtype).float()
+        z = torch.einsum("nbi,gboi->gnbo", u.view(-1, B, C // B), w_gates.float()).reshape(2, -1, C) + b_gates.unsqueeze(1)
+        la = -torch.sigmoid(z[0]) * rate
+        a, inp = torch.exp(la), torch.sqrt(-torch.expm1(2 * la)) * torch.sigmoid(z[1]) * u
+        S, rows = mem[0].clone(), []
+        for t in range(hi - lo):
+            S = a[t] * S + inp[t]
+            rows.append(S)
+        out[lo:hi] = (torch.stack(rows) * F.gelu(y[lo:hi].float(), approximate="tanh")).to(x.dtype)
+        state[sl[b], 0] = torch.cat((S.unsqueeze(0), xs[hi - lo:]), 0)
+    return out
+
+
+def rotary_table(dims: int, base: float, count: int, device="cpu", scaling=None) -> torch.Tensor:
+    """[count, dims] fp32 = [cos | sin] of position * base^(-2 i / dims), or of scaled frequencies (a ``RopeScaling``)."""
+    return build_rope_cache(dims, count, base, scaling, device)
 
 
 def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: torch.Tensor, slots: torch.Tensor,
@@ -607,26 +716,41 @@ def moe_route(logits: torch.Tensor, top_k: int, scoring: str = "softmax", norm_t
     return ids.to(torch.int32), w
 
 
-def moe_topk(logits: torch.Tensor, experts: int, top_k: int,
-             bias: Optional[torch.Tensor] = None) -> Tuple[torch.Tensor, torch.Tensor]:
+def moe_topk(logits: torch.Tensor, experts: int, top_k: int, bias: Optional[torch.Tensor] = None, groups: int = 1,
+             keep: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
     """Router over the first ``experts`` columns of ``logits``: the ``top_k`` largest (after ``bias``) and the softmax
-    over just those. Returns (ids [T, k] int32, weights [T, k] fp32)."""
+    over just those. Of ``groups`` > 1 equal groups of neighbours only the ``keep`` with the largest logits take part.
+    Returns (ids [T, k] int32, weights [T, k] fp32)."""
     z = logits[:, :experts].float()
     if bias is not None:
         z = z + bias.float()
+    if keep < groups:
+        g = z.view(z.shape[0], groups, -1)
+        best = g.amax(-1).topk(keep, dim=-1).indices
+        open_ = torch.zeros(g.shape[:2], dtype=torch.bool, device=z.device).scatter_(1, best, True)
+        z = g.masked_fill(~open_.unsqueeze(-1), float("-inf")).flatten(1)
     top, ids = z.topk(top_k, dim=-1)
     return ids.to(torch.int32), torch.softmax(top, dim=-1)
 
 
-def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, w_gate_up: torch.Tensor,
-                    w_down: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
-    """The unweighted output of every (token, slot) pair's expert: (rows [T * k, H], the row of each pair)."""
+def clamped_gate_mul(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    """x = [gate | up]: g * sigmoid(alpha g) * (u + 1), g = min(gate, limit), u = up clamped to +-limit."""
+    d = x.shape[-1] // 2
+    g, u = x[..., :d].float().clamp(max=limit), x[..., d:].float().clamp(-limit, limit)
+    return (g * torch.sigmoid(alpha * g) * (u + 1)).to(x.dtype)
+
+
+def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
+                    limit: float = 0.0, alpha: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+    """The unweighted output of every (token, slot) pair's expert: (rows [T * k, H], the row of each pair). ``limit`` > 0:
+    clamped experts, see :func:`clamped_gate_mul`."""
     k = ids.shape[1]
     flat = ids.reshape(-1).long()
     y = torch.empty(flat.numel(), x.shape[1], dtype=x.dtype, device=x.device)
     for e in flat.unique().tolist():
         at = (flat == e).nonzero()[:, 0]
-        y[at] = linear(silu_and_mul(linear(x[at // k], w_gate_up[e])), w_down[e])
+        h = linear(x[at // k], w_gate_up[e])
+        y[at] = linear(clamped_gate_mul(h, limit, alpha) if limit else silu_and_mul(h), w_down[e])
     return y, torch.arange(flat.numel(), dtype=torch.int32, device=x.device)
 
 
@@ -775,13 +899,12 @@ def build_rope_cache(rotary_dim: int, max_pos: int, theta: float, scaling=None, 
         orig = scaling.original_max_position_embeddings or max_pos
         low = max(math.floor(_yarn_find_dim(scaling.beta_fast, rotary_dim, base, orig)), 0)
         high = min(math.ceil(_yarn_find_dim(scaling.beta_slow, rotary_dim, base, orig)), rotary_dim - 1)
-        if low == high:
-            high += 0.001
-        ramp = ((torch.arange(half, dtype=torch.float64) - low) / (high - low)).clamp(0, 1)
+        ramp = ((torch.arange(half, dtype=torch.float64) - low) / max(high - low, 0.001)).clamp(0, 1)
         inv_mask = 1.0 - ramp
         inv = inv / factor * (1 - inv_mask) + inv * inv_mask
         mscale = yarn_mscale(factor, scaling.mscale) / yarn_mscale(factor, scaling.mscale_all_dim) \
             if scaling.mscale_all_dim else yarn_mscale(factor, 1.0)
+        mscale = getattr(scaling, "attention_factor", 0.0) or mscale
     freqs = torch.outer(pos, inv)
     out = torch.cat((freqs.cos() * mscale, freqs.sin() * mscale), dim=-1).float()
     return out.to(device)
