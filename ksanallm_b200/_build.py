@@ -81,13 +81,15 @@ def cuda_sources():
 # fresh checkout without compiling every kernel of the package.
 FAMILY_SOURCES = {
     family: ("host_common", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2cta", "gemm_bf16_cluster_splitk", "moe",
-             "moe_topk", "mixer_elementwise", "window_attention", "linear_attention", "mixer_executor")
-    for family in ("molopel", "givirax")
+             "moe_topk", "mixer_elementwise", "window_attention", "linear_attention", "hyper_connections", "head_gemm",
+             "gemm_batched", "latent_attention", "gated_recurrence", "mixer_executor")
+    for family in ("molopel", "givirax", "ladusun")
 }
 
 # Files compiled with IEEE division, square root and the accurate math functions: what they compute is specified in
 # 32-bit floats.
-EXACT_MATH = {"moe_topk", "mixer_elementwise", "window_attention", "linear_attention"}
+EXACT_MATH = {"moe_topk", "mixer_elementwise", "window_attention", "linear_attention", "hyper_connections", "head_gemm",
+              "latent_attention", "gated_recurrence"}
 
 
 def cuda_library(family: str = "") -> Path:

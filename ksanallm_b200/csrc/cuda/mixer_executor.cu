@@ -17,8 +17,8 @@ int ksana_stream_norm(const void* x, int ldx, const void* res_in, void* res_out,
                       cudaStream_t st);
 int ksana_append_act(const void* k, const void* u, int ldx, const int* slots, void* cache, int tokens, int hk, int d,
                      int bs, void* out, int ldo, int I, int gated, int kind, cudaStream_t st);
-int ksana_moe_topk(const float* logits, int ld, const float* bias, int T, int E, int k, int* ids, float* weights,
-                   cudaStream_t st);
+int ksana_moe_topk(const float* logits, int ld, const float* bias, int T, int E, int k, int groups, int keep, int* ids,
+                   float* weights, cudaStream_t st);
 int ksana_moe_permute(const void* x, int ldx, const int* ids, int T, int k, int H, int expert_offset, int E_local,
                       int* meta, int* pos, int* row_src, void* xs, cudaStream_t stream);
 int ksana_moe_grouped_gemm(const void* A, const void* W, void* C, const int* offsets, int E, int max_rows, int N, int K,
@@ -27,24 +27,25 @@ int ksana_silu_mul(const void* x, int ldx, void* out, int ldo, int rows, int I, 
 int ksana_silu_mul_any(const void* x, void* out, int rows, int I, int kind, cudaStream_t st);
 int ksana_gelu_mul(const void* x, int ldx, void* out, int ldo, int rows, int I, int kind, cudaStream_t st);
 int ksana_qk_norm_cache(void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const int* slots, void* cache,
-                        const float* qw, const float* kw, float eps, int tokens, int h, int hk, int d, int dv, int bs,
-                        int kind, cudaStream_t st);
+                        const float* qw, const float* kw, float eps, const int* positions, const float* rotary, int rd,
+                        int tokens, int h, int hk, int d, int dv, int bs, int kind, cudaStream_t st);
 int ksana_gated_norm(const void* o, const void* g, int ldg, const float* w, void* out, int ldo, int tokens, int h, int dv,
                      float eps, int gate, float out_scale, int kind, cudaStream_t st);
 int ksana_window_prefill(const void* q, int ldq, int total_tokens, const void* cache, int num_blocks,
                          const int* block_tables, int max_blocks, const int* cu_q, const int* kv_lens, int h, int hk,
                          int d, int dv, int bs, int window, int keep, int shared, float scale, const float* bias,
-                         int bias_len, float out_scale, void* out, int ldo, int seq_base, int num_seqs, int max_q,
-                         cudaStream_t st);
+                         int bias_len, float out_scale, float softcap, int sink, const void* gate, int ldg, void* out,
+                         int ldo, int seq_base, int num_seqs, int max_q, cudaStream_t st);
 int ksana_window_decode(const void* q, int ldq, const void* cache, int num_blocks, const int* block_tables, int max_blocks,
                         const int* cu_q, const int* kv_lens, int h, int hk, int d, int dv, int bs, int window,
-                        int keep, int shared, float scale, const float* bias, int bias_len, float out_scale, void* out,
-                        int ldo, int seq_base, int num_seqs, int max_kv, cudaStream_t st);
+                        int keep, int shared, float scale, const float* bias, int bias_len, float out_scale,
+                        float softcap, int sink, const void* gate, int ldg, void* out, int ldo, int seq_base, int num_seqs,
+                        int max_kv, cudaStream_t st);
 int ksana_window_attention_any(const void* q, int ldq, const void* cache, const int* block_tables, int max_blocks,
                                const int* cu_q, const int* kv_lens, const int* seq_of_token, int h, int hk, int d, int dv,
                                int bs, int window, int keep, int shared, float scale, const float* bias, int bias_len,
-                               float out_scale, void* out, int ldo, int tok_base, int tokens, int kind,
-                               cudaStream_t st);
+                               float out_scale, float softcap, int sink, const void* gate, int ldg, void* out, int ldo,
+                               int tok_base, int tokens, int kind, cudaStream_t st);
 long long ksana_linear_chunk_scratch(int tokens, int num_seqs, int h, int d, int dv);
 int ksana_linear_chunked(const void* q, int ldq, const void* k, int ldk, const void* v, int ldv, float* state,
                          const int* slots, const int* cu_q, const int* kv_lens, const int* positions, const float* decay,
@@ -104,19 +105,21 @@ struct Exec {
                                     static_cast<char*>(out) + static_cast<size_t>(w.h * w.dv) * 2, w.k_out, I, w.gated, 1,
                                     st)))
         return false;
-    } else if (!step(2, ksana_qk_norm_cache(x, ld, k, ld, v, ld, s->slot_mapping, w.kv, w.q_norm, w.k_norm, m->eps, T,
-                                            w.h, w.hk, w.d, w.dv, m->block_size, 1, st))) {
+    } else if (!step(2, ksana_qk_norm_cache(x, ld, k, ld, v, ld, s->slot_mapping, w.kv, w.q_norm, w.k_norm, m->eps,
+                                            nullptr, nullptr, 0, T, w.h, w.hk, w.d, w.dv, m->block_size, 1, st))) {
       return false;
     }
     auto general = [&](int first, int count) {
       return ksana_window_attention_any(x, ld, w.kv, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, s->seq_of_token,
                                         w.h, w.hk, w.d, w.dv, m->block_size, w.window, w.keep_first, w.shared_kv,
-                                        w.scale, w.bias, w.bias_len, w.attn_out_scale, out, w.k_out, first, count, 1, st);
+                                        w.scale, w.bias, w.bias_len, w.attn_out_scale, 0.f, 0, nullptr, 0, out, w.k_out, first,
+                                        count, 1, st);
     };
     if (s->num_prefill > 0) {
       int rc = ksana_window_prefill(x, ld, T, w.kv, m->num_blocks, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens,
                                     w.h, w.hk, w.d, w.dv, m->block_size, w.window, w.keep_first, w.shared_kv, w.scale,
-                                    w.bias, w.bias_len, w.attn_out_scale, out, w.k_out, 0, s->num_prefill, s->max_q_prefill, st);
+                                    w.bias, w.bias_len, w.attn_out_scale, 0.f, 0, nullptr, 0, out, w.k_out, 0, s->num_prefill,
+                                    s->max_q_prefill, st);
       if (rc == -1) rc = general(0, s->prefill_tokens);
       if (!step(3, rc)) return false;
     }
@@ -125,7 +128,8 @@ struct Exec {
       if (s->one_token)
         rc = ksana_window_decode(x, ld, w.kv, m->num_blocks, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, w.h, w.hk, w.d, w.dv,
                                  m->block_size, w.window, w.keep_first, w.shared_kv, w.scale, w.bias, w.bias_len,
-                                 w.attn_out_scale, out, w.k_out, s->num_prefill, s->num_decode, s->max_kv_decode, st);
+                                 w.attn_out_scale, 0.f, 0, nullptr, 0, out, w.k_out, s->num_prefill, s->num_decode,
+                                 s->max_kv_decode, st);
       if (rc == -1) rc = general(s->prefill_tokens, T - s->prefill_tokens);
       if (!step(4, rc)) return false;
     }
@@ -165,7 +169,7 @@ struct Exec {
     const int T = s->total_tokens, H = m->hidden, I = w.expert_inter, n = T * w.top;
     const int* offsets = m->sort_meta + w.experts;
     if (!step(15, gemm(h, H, w.w_router, nullptr, m->router_buf, w.router_rows, w.router_rows, 1))) return false;
-    if (!step(16, ksana_moe_topk(m->router_buf, w.router_rows, w.b_router, T, w.experts, w.top, m->expert_ids,
+    if (!step(16, ksana_moe_topk(m->router_buf, w.router_rows, w.b_router, T, w.experts, w.top, 1, 1, m->expert_ids,
                                  m->expert_weights, st)))
       return false;
     ++*launches;

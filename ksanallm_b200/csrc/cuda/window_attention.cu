@@ -6,6 +6,10 @@
 // bias: [h][bias_len] fp32 (null: none), indexed by the distance between query and key.
 //
 // Query i sees key j when j <= i and (i - j < window or j < keep); window 0: every j <= i.
+//
+// softcap > 0: a score becomes cap * tanh(score / cap) before anything else. sink: the softmax's denominator has one more
+// term exp(0). gate: each head's result is multiplied by the sigmoid of gate[token][head] (the storage type of q). Where
+// the cache holds keys alone, a key's first dv numbers are its value.
 #include "host_common.h"
 #include "mixer_common.cuh"
 
@@ -20,13 +24,17 @@ struct WindowAttnArgs {
   const int* cu_q;
   const int* kv_lens;
   const int* seq_of_token;
-  int h, hk, d, dv, bs, window, keep, shared;  // shared: values are the keys (dv == d)
+  int h, hk, d, dv, bs, window, keep, shared;  // shared: values are the keys (their first dv numbers)
   float scale;
   const float* bias;
   int bias_len;
   float out_scale;
   void* out;
   int ldo;
+  float softcap;
+  int sink;
+  const void* gate;
+  int ldg;
   __host__ __device__ size_t v_off() const { return shared ? 0 : static_cast<size_t>(hk) * bs * d; }
   __host__ __device__ size_t block_elems() const { return static_cast<size_t>(hk) * bs * (d + (shared ? 0 : dv)); }
   // oldest key inside the window of the query at `pos`
@@ -68,6 +76,7 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
       float dot = 0.f;
       for (int c = 0; c < a.d; ++c) dot += sq[c] * to_f(kp[c]);
       s = dot * a.scale;
+      if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
       if (bias) s += bias[min(pos - j, a.bias_len - 1)];
     }
     const float m_new = fmaxf(m, warp_max(s));
@@ -81,7 +90,8 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
     for (int u = 0; u < count; ++u) {
       const float pu = __shfl_sync(0xffffffffu, p, u);
       const int ju = i0 + u < kept ? i0 + u : lo + i0 + u - kept;
-      const T* vp = cache + bt[ju / a.bs] * block_elems + v_off + (static_cast<size_t>(kh) * a.bs + ju % a.bs) * a.dv;
+      const T* vp = cache + bt[ju / a.bs] * block_elems + v_off +
+                    (static_cast<size_t>(kh) * a.bs + ju % a.bs) * (a.shared ? a.d : a.dv);
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = i * 32 + lane;
@@ -90,7 +100,14 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
     }
   }
   T* o = static_cast<T*>(a.out) + static_cast<size_t>(t) * a.ldo + head * a.dv;
-  const float inv = a.out_scale / l;
+  if (a.sink) {  // relative to the larger of the running maximum and the sink's own score
+    const float top = fmaxf(m, 0.f), f = expf(m - top);
+    l = l * f + expf(-top);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) acc[i] *= f;
+  }
+  float inv = a.out_scale / l;
+  if (a.gate) inv *= sigmoid_f(to_f(static_cast<const T*>(a.gate)[static_cast<size_t>(t) * a.ldg + head]));
 #pragma unroll
   for (int i = 0; i < NV; ++i) {
     const int c = i * 32 + lane;
@@ -148,7 +165,24 @@ struct WindowPrefillSmem {
   static constexpr int TOTAL = USED > 120 * 1024 ? USED : 120 * 1024;
 };
 
-template <int DP, int DVP, bool SHARED, bool KEEP>
+// The cap of a score, in units where exp2 is the exponential: s -> c tanh(s / c) with c in those units. Tiles whose scores
+// are small against the cap take a polynomial, odd to degree 11 (error below 1e-7 of the cap up to |s / c| = 0.4); others
+// the exponential form.
+constexpr float CAP_POLY = 0.4f;
+__device__ __forceinline__ float cap_small(float s, float inv_c) {
+  const float x = s * inv_c, z = x * x;
+  float p = fmaf(z, -1382.f / 155925.f, 62.f / 2835.f);
+  p = fmaf(p, z, -17.f / 315.f);
+  p = fmaf(p, z, 2.f / 15.f);
+  p = fmaf(p, z, -1.f / 3.f);
+  return fmaf(p * z, s, s);
+}
+__device__ __forceinline__ float cap_any(float s, float c, float inv_c) {
+  const float x = fminf(fmaxf(s * inv_c, -20.f), 20.f);
+  return c - __fdividef(2.f * c, 1.f + __expf(2.f * x));
+}
+
+template <int DP, int DVP, bool SHARED, bool KEEP, bool CAP>
 __global__ void __launch_bounds__(160, 1)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
                       const __grid_constant__ CUtensorMap tmV, WindowAttnArgs a, int seq_base, unsigned int* err) {
@@ -282,6 +316,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
   } else {
     const uint32_t lane_off = static_cast<uint32_t>(warp * 32) << 16;
     const float scale2 = a.scale * 1.4426950408889634f;
+    const float cap2 = CAP ? a.softcap * 1.4426950408889634f : 0.f, inv_cap2 = CAP ? 1.f / cap2 : 0.f;
     const float* bias = a.bias ? a.bias + static_cast<size_t>(head) * a.bias_len : nullptr;
     const int reach = a.window > 0 ? min(a.window, 1 << 30) : 1 << 30;
     float m_ref = -INFINITY, l = 0.f;
@@ -312,6 +347,21 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       for (int c = 0; c < 4; ++c) tmem_ld32(S + c * 32, reinterpret_cast<uint32_t*>(s) + c * 32);
       tmem_wait_ld();
       float m_tile = -INFINITY;
+      if constexpr (CAP) {
+        float big = 0.f;
+#pragma unroll
+        for (int j = 0; j < 128; ++j) {
+          s[j] *= scale2;
+          big = fmaxf(big, fabsf(s[j]));
+        }
+        if (__any_sync(0xffffffffu, big > CAP_POLY * cap2)) {
+#pragma unroll
+          for (int j = 0; j < 128; ++j) s[j] = cap_any(s[j], cap2, inv_cap2);
+        } else {
+#pragma unroll
+          for (int j = 0; j < 128; ++j) s[j] = cap_small(s[j], inv_cap2);
+        }
+      }
       if (KEEP && kept > 0) {
         const int behind = row_pos + tid - key0 - reach;  // columns up to this one are behind the window
 #pragma unroll
@@ -320,7 +370,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       }
 #pragma unroll
       for (int j = 0; j < 128; ++j) {
-        s[j] = fmaf(s[j], scale2, tb[tid - j + 127]);
+        s[j] = CAP ? s[j] + tb[tid - j + 127] : fmaf(s[j], scale2, tb[tid - j + 127]);
         m_tile = fmaxf(m_tile, s[j]);
       }
       const float m_new = fmaxf(m_ref, m_tile);
@@ -369,7 +419,10 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
     if (__all_sync(0xffffffffu, ok)) {
       tc_fence_after();
       const bool valid = qt * 128 + tid < q_len;
-      const float inv = l > 0.f ? a.out_scale / l : 0.f;
+      if (a.sink && m_ref != -INFINITY) l += exp2f(-m_ref);
+      float inv = l > 0.f ? a.out_scale / l : 0.f;
+      if (a.gate && valid)
+        inv *= sigmoid_f(__bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[static_cast<size_t>(q0 + qt * 128 + tid) * a.ldg + head]));
       __nv_bfloat16* orow = static_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(q0 + qt * 128 + tid) * a.ldo +
                             head * a.dv;
 #pragma unroll 1
@@ -411,7 +464,7 @@ static int cache_maps(const WindowAttnArgs& a, int num_blocks, CUtensorMap* tk, 
   return 0;
 }
 
-template <int DP, int DVP, bool SHARED, bool KEEP>
+template <int DP, int DVP, bool SHARED, bool KEEP, bool CAP>
 static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blocks, int seq_base, int num_seqs,
                           int max_q, cudaStream_t st) {
   using L_ = WindowPrefillSmem<DP, DVP, SHARED>;
@@ -423,7 +476,7 @@ static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blo
     if (make_tmap_nd(&tq, a.q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -2;
   }
   if (int rc = cache_maps(a, num_blocks, &tk, &tv)) return rc;
-  auto kern = window_prefill_kernel<DP, DVP, SHARED, KEEP>;
+  auto kern = window_prefill_kernel<DP, DVP, SHARED, KEEP, CAP>;
   if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
   kern<<<dim3((max_q + 127) / 128, num_seqs, a.h), 160, L_::TOTAL, st>>>(tq, tk, tv, a, seq_base, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
@@ -551,6 +604,7 @@ window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
       }
   }
   const float scale2 = a.scale * 1.4426950408889634f;
+  const float cap2 = a.softcap * 1.4426950408889634f, inv_cap2 = a.softcap > 0.f ? 1.f / cap2 : 0.f;
   float acc[DVP / 16][NT][4];
 #pragma unroll
   for (int i = 0; i < DVP / 16; ++i)
@@ -599,6 +653,7 @@ window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
 #pragma unroll
         for (int e = 0; e < 2; ++e) {
           float s = c[nt][u * 2 + e] * scale2;
+          if (a.softcap > 0.f) s = cap_any(s, cap2, inv_cap2);
           if (a.bias) {
             const int hd = min(nt * 8 + j2 + e, g - 1);
             const float* bias = a.bias + static_cast<size_t>(head0 + hd) * a.bias_len;
@@ -721,6 +776,7 @@ window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
     const int hd = e / quads, col = e % quads * 4;
     float M = -INFINITY, S = 0.f, o[4] = {0.f, 0.f, 0.f, 0.f};
     if (splits == 1) {
+      M = cM[hd];
       S = cL[hd];
       const float4 v = *reinterpret_cast<const float4*>(sO + hd * LDO + col);
       o[0] = v.x; o[1] = v.y; o[2] = v.z; o[3] = v.w;
@@ -733,7 +789,9 @@ window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
         o[0] += f * v.x; o[1] += f * v.y; o[2] += f * v.z; o[3] += f * v.w;
       }
     }
-    const float inv = a.out_scale / S;
+    if (a.sink) S += exp2f(-M);
+    float inv = a.out_scale / S;
+    if (a.gate) inv *= sigmoid_f(__bfloat162float(static_cast<const __nv_bfloat16*>(a.gate)[static_cast<size_t>(t) * a.ldg + head0 + hd]));
 #pragma unroll
     for (int u = 0; u < 4; ++u) o[u] *= inv;
     store_n<4>(out + hd * a.dv + col, o);
@@ -782,18 +840,22 @@ using namespace ksana;
 KSANA_API int ksana_window_prefill(const void* q, int ldq, int total_tokens, const void* cache, int num_blocks,
                                    const int* block_tables, int max_blocks, const int* cu_q, const int* kv_lens, int h,
                                    int hk, int d, int dv, int bs, int window, int keep, int shared, float scale,
-                                   const float* bias, int bias_len, float out_scale, void* out, int ldo, int seq_base,
-                                   int num_seqs, int max_q, cudaStream_t st) {
+                                   const float* bias, int bias_len, float out_scale, float softcap, int sink,
+                                   const void* gate, int ldg, void* out, int ldo, int seq_base, int num_seqs, int max_q,
+                                   cudaStream_t st) {
   if (num_seqs <= 0 || max_q <= 0) return 0;
   if (keep < 0 || (shared && d != dv)) return -2;
   if (h % hk || bs != WP_PAGE || d > 128 || dv > 128 || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
       !rows16(out, ldo))
     return -1;
   WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
-                   shared, scale, bias, bias_len, out_scale, out, ldo};
+                   shared, scale, bias, bias_len, out_scale, out, ldo, softcap, sink, gate, ldg};
+  if (softcap > 0.f && (keep || shared)) return -1;
 #define KSANA_WP(DP, DVP, SHARED)                                                                                      \
-  return keep ? launch_prefill<DP, DVP, SHARED, true>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)      \
-              : launch_prefill<DP, DVP, SHARED, false>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
+  return keep ? launch_prefill<DP, DVP, SHARED, true, false>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st) \
+         : softcap > 0.f                                                                                               \
+             ? launch_prefill<DP, DVP, SHARED, false, !SHARED>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st) \
+             : launch_prefill<DP, DVP, SHARED, false, false>(a, total_tokens, num_blocks, seq_base, num_seqs, max_q, st)
   if (shared) {
     if (d <= 64) KSANA_WP(64, 64, true);
     KSANA_WP(128, 128, true);
@@ -810,15 +872,15 @@ KSANA_API int ksana_window_prefill(const void* q, int ldq, int total_tokens, con
 KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, int num_blocks, const int* block_tables,
                                   int max_blocks, const int* cu_q, const int* kv_lens, int h, int hk, int d, int dv,
                                   int bs, int window, int keep, int shared, float scale, const float* bias, int bias_len,
-                                  float out_scale, void* out, int ldo, int seq_base, int num_seqs, int max_kv,
-                                  cudaStream_t st) {
+                                  float out_scale, float softcap, int sink, const void* gate, int ldg, void* out,
+                                  int ldo, int seq_base, int num_seqs, int max_kv, cudaStream_t st) {
   if (num_seqs <= 0) return 0;
   if (keep < 0 || (shared && d != dv)) return -2;
   if (h % hk || bs != WP_PAGE || d > 128 || dv > 128 || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
       !rows16(out, ldo))
     return -1;
   WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
-                   shared, scale, bias, bias_len, out_scale, out, ldo};
+                   shared, scale, bias, bias_len, out_scale, out, ldo, softcap, sink, gate, ldg};
 #define KSANA_WD(DP, DVP, SHARED)                                                                             \
   return h / hk <= 8 ? launch_decode<DP, DVP, 1, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)       \
                      : launch_decode<DP, DVP, 2, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)
@@ -837,11 +899,12 @@ KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, int
 KSANA_API int ksana_window_attention_any(const void* q, int ldq, const void* cache, const int* block_tables,
                                          int max_blocks, const int* cu_q, const int* kv_lens, const int* seq_of_token,
                                          int h, int hk, int d, int dv, int bs, int window, int keep, int shared,
-                                         float scale, const float* bias, int bias_len, float out_scale, void* out,
-                                         int ldo, int tok_base, int tokens, int kind, cudaStream_t st) {
+                                         float scale, const float* bias, int bias_len, float out_scale, float softcap,
+                                         int sink, const void* gate, int ldg, void* out, int ldo, int tok_base,
+                                         int tokens, int kind, cudaStream_t st) {
   if (tokens <= 0) return 0;
-  if (h % hk || keep < 0 || (shared && d != dv)) return -2;
+  if (h % hk || keep < 0 || (shared && d < dv)) return -2;
   WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, seq_of_token, h, hk, d, dv, bs, window, keep,
-                   shared, scale, bias, bias_len, out_scale, out, ldo};
+                   shared, scale, bias, bias_len, out_scale, out, ldo, softcap, sink, gate, ldg};
   return kind ? launch_any<__nv_bfloat16>(a, tok_base, tokens, st) : launch_any<float>(a, tok_base, tokens, st);
 }

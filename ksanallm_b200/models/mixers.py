@@ -138,26 +138,32 @@ class LatentAttention:
         s = self.spec
         q = x[:, :self.nq].unflatten(1, (s.heads, s.dim + s.rot_dim))
         bs = kv.shape[1] // s.width
-        ops.latent_append(q, x[:, self.nq:self.nq + self.na], self.norm, self.eps, meta.positions, self.rotary(),
-                          meta.slot_mapping, kv, bs)
         gate = x[:, self.nq + self.na:self.nq + self.na + s.heads] if s.head_gate else None
-        ops.latent_attention(q, kv, meta, bs, self.w, s.scale, gate, out)
+        ops.latent_attention(q, x[:, self.nq:self.nq + self.na], self.norm, self.eps, self.rotary(), kv, meta, bs, self.w,
+                             s.scale, gate, out)
+
+
+class RecurrenceWeights:
+    """What a gated recurrence needs behind its input projections."""
+
+    def __init__(self, w: Dict[str, torch.Tensor], prefix: str, decay_scale: float):
+        self.conv, self.conv_b = w[prefix + ".conv"], w[prefix + ".conv_b"]        # [C, K], [C] fp32
+        self.gates, self.gates_b = w[prefix + ".gates"], w[prefix + ".gates_b"]    # [2, B, C / B, C / B], [2, C] fp32
+        lam = w[prefix + ".lam"].double()
+        self.rate = (decay_scale * torch.nn.functional.softplus(lam, threshold=100)).float()  # [C]
+        self.gates_by_block = torch.cat((self.gates[0], self.gates[1]), 1).contiguous()  # [B, 2 C / B, C / B]
 
 
 class GatedRecurrence:
     def __init__(self, cfg: ModelConfig, spec: RecurrenceSpec, w: Dict[str, torch.Tensor], prefix: str):
         self.spec = spec
         self.rows, self.width = 2 * spec.width, spec.width
-        self.conv, self.conv_b = w[prefix + ".conv"], w[prefix + ".conv_b"]        # [C, K], [C] fp32
-        self.gates, self.gates_b = w[prefix + ".gates"], w[prefix + ".gates_b"]    # [2, B, C / B, C / B], [2, C] fp32
-        lam = w[prefix + ".lam"].double()
-        self.rate = (spec.decay_scale * torch.nn.functional.softplus(lam, threshold=100)).float()
+        self.w = RecurrenceWeights(w, prefix, spec.decay_scale)
 
     def run(self, x: torch.Tensor, meta, state: torch.Tensor, out: torch.Tensor) -> None:
         """x [T, rows] = the projected (y | x); writes ``width`` columns of ``out``."""
         C = self.spec.width
-        ops.gated_recurrence(x[:, :C], x[:, C:2 * C], state, meta, self.conv, self.conv_b, self.gates, self.gates_b,
-                             self.rate, out)
+        ops.gated_recurrence(x[:, :C], x[:, C:2 * C], state, meta, self.w, out)
 
 
 class DecayedLinearAttention:

@@ -135,29 +135,26 @@ def qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps,
     return f.qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps, positions, rotary)
 
 
-def latent_append(q, a, norm_w, eps, positions, rotary, slot_mapping, cache, block_size):
-    f = _mixer() if q.is_cuda else ref
-    f.latent_append(q, a, norm_w, eps, positions, rotary, slot_mapping, cache, block_size)
-
-
-def latent_attention(q, cache, meta, block_size, w, scale, gate, out):
-    """``w``: :class:`~ksanallm_b200.models.mixers.LatentWeights`. Writes heads * vdim columns of ``out``."""
+def latent_attention(q, a, norm_w, eps, rotary, cache, meta, block_size, w, scale, gate, out):
+    """Rotation, cache append and attention; ``w``: :class:`~ksanallm_b200.models.mixers.LatentWeights`. Writes
+    heads * vdim columns of ``out``."""
     if q.is_cuda:
         from . import cuda_latent
-        cuda_latent.latent_attention(q, cache, meta, block_size, w, scale, gate, out)
+        cuda_latent.latent_attention(q, a, norm_w, eps, rotary, cache, meta, block_size, w, scale, gate, out)
         return
+    ref.latent_append(q, a, norm_w, eps, meta.positions, rotary, meta.slot_mapping, cache, block_size)
     out.copy_(ref.latent_attention(q, cache, meta.block_tables, meta.cu_q, meta.kv_lens, block_size, w.uk, w.uv, scale,
                                    gate).flatten(1))
 
 
-def gated_recurrence(y, x, state, meta, conv_w, conv_b, w_gates, b_gates, rate, out):
-    """Writes ``out`` [T, C] (a column slice is fine)."""
+def gated_recurrence(y, x, state, meta, w, out):
+    """``w``: :class:`~ksanallm_b200.models.mixers.RecurrenceWeights`. Writes ``out`` [T, C] (a column slice is fine)."""
     if x.is_cuda:
         from . import cuda_recurrence
-        cuda_recurrence.gated_recurrence(y, x, state, meta, conv_w, conv_b, w_gates, b_gates, rate, out)
+        cuda_recurrence.gated_recurrence(y, x, state, meta, w, out)
         return
-    out.copy_(ref.gated_recurrence(y, x, state, meta.state_slots, meta.cu_q, meta.kv_lens, conv_w, conv_b, w_gates,
-                                   b_gates, rate))
+    out.copy_(ref.gated_recurrence(y, x, state, meta.state_slots, meta.cu_q, meta.kv_lens, w.conv, w.conv_b, w.gates,
+                                   w.gates_b, w.rate))
 
 
 def append_act(k, u, slot_mapping, cache, block_size, out, gated=False):

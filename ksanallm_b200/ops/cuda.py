@@ -80,17 +80,24 @@ class _Sig:
     ksana_layer_norm = ([P, I, P, I, P, P, P, I, I, I, F, I, P], I)
     ksana_embedding_f32 = ([P, P, P, I, I, I, F, P, P, I, I, P], I)
     ksana_append_act = ([P, P, I, P, P, I, I, I, I, P, I, I, I, I, P], I)
-    ksana_moe_topk = ([P, I, P, I, I, I, P, P, P], I)
+    ksana_moe_topk = ([P, I, P, I, I, I, I, I, P, P, P], I)
     ksana_moe_sort = ([P, I, I, I, P, P, P, P], I)
     ksana_moe_gemm_any = ([P, I, P, I, P, P, P, I, I, I, I, I, P], I)
     ksana_silu_mul_any = ([P, P, I, I, I, P], I)
     ksana_gelu_mul = ([P, I, P, I, I, I, I, P], I)
-    ksana_qk_norm_cache = ([P, I, P, I, P, I, P, P, P, P, F, I, I, I, I, I, I, I, P], I)
+    ksana_qk_norm_cache = ([P, I, P, I, P, I, P, P, P, P, F, P, P, I, I, I, I, I, I, I, I, P], I)
+    ksana_relu2 = ([P, P, LL, I, P], I)
+    ksana_clamped_gate_mul = ([P, P, I, I, F, F, I, P], I)
+    ksana_hyper_norm = ([P, I, P, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, F, I, P], I)
+    ksana_head_gemm_any = ([P, LL, LL, P, P, LL, LL, I, I, I, I, I, P], I)
+    ksana_latent_append = ([P, I, I, P, I, P, I, P, F, P, P, P, P, I, I, I, I, I, P], I)
+    ksana_recurrence_conv = ([P, I, P, P, P, P, P, P, P, I, I, P, I, I, I, P], I)
+    ksana_recurrence_scan = ([P, I, P, I, P, P, P, P, P, P, P, P, I, I, I, P, I, I, I, I, I, P], I)
     ksana_gated_norm = ([P, P, I, P, P, I, I, I, I, F, I, F, I, P], I)
     ksana_softcap = ([P, I, P, I, I, F, P], I)
-    ksana_window_attention_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
-    ksana_window_prefill = ([P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
-    ksana_window_decode = ([P, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, P, I, I, I, I, P], I)
+    ksana_window_attention_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, F, F, I, P, I, P, I, I, I, I, P], I)
+    ksana_window_prefill = ([P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, F, I, P, I, P, I, I, I, I, P], I)
+    ksana_window_decode = ([P, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, F, I, P, I, P, I, I, I, I, P], I)
     ksana_linear_chunk_scratch = ([I, I, I, I, I], LL)
     ksana_linear_chunked = ([P, I, P, I, P, I, P, P, P, P, P, P, P, I, I, F, I, I, I, P, I, I, I, P, P], I)
     ksana_linear_recurrent = ([P, I, P, I, P, I, P, P, P, P, P, P, P, I, I, F, I, I, I, P, I, I, I, I, P], I)

@@ -49,6 +49,38 @@ def stream_norm(x, weight, eps: float, center: bool, stream_in, stream_out=None,
     return out
 
 
+def hyper_norm(x, scale, routed, streams, mix, out_w, streams_out, in_w, weight, eps: float, out_dtype) -> torch.Tensor:
+    S, H = in_w.shape[0], weight.shape[0]
+    T = streams.shape[0]
+    rows, pos, wts = routed if routed is not None else (None, None, None)
+    assert streams.is_contiguous() and streams.dtype == torch.float32 and weight.dtype == out_dtype
+    assert x is None or x.stride(1) == 1 and x.dtype == out_dtype
+    assert all(t is None or t.is_contiguous() for t in (scale, rows, pos, wts, mix, out_w, streams_out, in_w))
+    out = torch.empty(T, H, dtype=out_dtype, device=streams.device)
+    _check(lib().ksana_hyper_norm(_ptr(x), x.stride(0) if x is not None else 0, _ptr(scale), _ptr(rows), _ptr(pos),
+                                  _ptr(wts), wts.shape[1] if wts is not None else 0, _ptr(streams),
+                                  int(streams.dim() == 2), _ptr(mix), _ptr(out_w), _ptr(streams_out), _ptr(in_w),
+                                  _ptr(weight), _ptr(out), T, H, S, float(eps), _KIND[out_dtype], _stream()),
+           "hyper_norm")
+    return out
+
+
+def relu2(x: torch.Tensor) -> torch.Tensor:
+    x = x.contiguous()
+    out = torch.empty_like(x)
+    _check(lib().ksana_relu2(_ptr(x), _ptr(out), x.numel(), _KIND[x.dtype], _stream()), "relu2")
+    return out
+
+
+def clamped_gate_mul(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
+    T, two_i = x.shape
+    assert x.is_contiguous()
+    out = torch.empty(T, two_i // 2, dtype=x.dtype, device=x.device)
+    _check(lib().ksana_clamped_gate_mul(_ptr(x), _ptr(out), T, two_i // 2, float(limit), float(alpha), _KIND[x.dtype],
+                                        _stream()), "clamped_gate_mul")
+    return out
+
+
 def embedding(ids, table, scale: float, out_dtype, positions=None, pos_table=None) -> torch.Tensor:
     assert out_dtype == torch.float32 and table.is_contiguous()
     assert pos_table is None or pos_table.is_contiguous() and pos_table.dtype == table.dtype
@@ -99,19 +131,24 @@ def _packed_heads(x: torch.Tensor) -> torch.Tensor:
     return x
 
 
-def qk_norm_cache(q, k, v, slot_mapping, cache, block_size: int, q_norm, k_norm, eps: float) -> None:
+def qk_norm_cache(q, k, v, slot_mapping, cache, block_size: int, q_norm, k_norm, eps: float, positions=None,
+                  rotary=None) -> None:
     T, h, d = q.shape
-    hk, dv = v.shape[1], v.shape[2]
+    hk, dv = (v.shape[1], v.shape[2]) if v is not None else (0, 0)
     for x in (q, k, v):
-        _packed_heads(x)
+        if x is not None:
+            _packed_heads(x)
     assert cache.dtype == q.dtype and cache.is_contiguous()
-    _check(lib().ksana_qk_norm_cache(_ptr(q), q.stride(0), _ptr(k), k.stride(0), _ptr(v), v.stride(0),
-                                     _ptr(slot_mapping), _ptr(cache), _ptr(q_norm), _ptr(k_norm), float(eps), T, h, hk,
-                                     d, dv, block_size, _KIND[q.dtype], _stream()), "qk_norm_cache")
+    _check(lib().ksana_qk_norm_cache(_ptr(q), q.stride(0), _ptr(k), k.stride(0) if k is not None else 0, _ptr(v),
+                                     v.stride(0) if v is not None else 0, _ptr(slot_mapping), _ptr(cache), _ptr(q_norm),
+                                     _ptr(k_norm), float(eps), _ptr(positions) if rotary is not None else None,
+                                     _ptr(rotary), rotary.shape[1] if rotary is not None else 0, T, h, hk, d, dv,
+                                     block_size, _KIND[q.dtype], _stream()), "qk_norm_cache")
 
 
 def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, scale: float, window: int, bias,
-                     out_scale: float, out: torch.Tensor, keep_first: int = 0) -> None:
+                     out_scale: float, out: torch.Tensor, keep_first: int = 0, softcap: float = 0.0, sink: bool = False,
+                     gate=None) -> None:
     """bf16 prompts take the tensor-core kernel, bf16 single tokens the cache-streaming one; sizes those do not have,
     and fp32, take the general kernel."""
     T, h, d = q.shape
@@ -121,7 +158,8 @@ def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, 
     blen = bias.shape[1] if bias is not None else 0
     shared = int(cache.shape[1] == kv_heads * block_size * d)
     sizes = (h, kv_heads, d, vdim, block_size, window, keep_first, shared, float(scale), _ptr(bias), blen,
-             float(out_scale))
+             float(out_scale), float(softcap), int(sink), _ptr(gate), gate.stride(0) if gate is not None else 0)
+    assert gate is None or gate.dtype == q.dtype and gate.stride(1) == 1
 
     def general(first: int, count: int) -> None:
         if count:
