@@ -54,9 +54,40 @@ latent_append_kernel(T* __restrict__ q, int ldq, int dim, T* __restrict__ q_cat,
   }
 }
 
+// The contexts of sequences [seq_base, seq_base + gridDim.y), row by row behind one another: [rows][rank + rot]. One warp
+// per row, 16 bytes per lane.
+__global__ void __launch_bounds__(256)
+latent_gather_kernel(const uint4* __restrict__ cache, const int* __restrict__ block_tables, int max_blocks,
+                     const int* __restrict__ kv_lens, int seq_base, int bs, int words, uint4* __restrict__ out) {
+  const int b = seq_base + blockIdx.y, L = kv_lens[b];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int j0 = blockIdx.x * 32;
+  if (j0 >= L) return;
+  int row0 = 0;
+  for (int i = seq_base + lane; i < b; i += 32) row0 += kv_lens[i];
+#pragma unroll
+  for (int o = 16; o > 0; o >>= 1) row0 += __shfl_xor_sync(0xffffffffu, row0, o);
+  for (int j = j0 + warp; j < min(j0 + 32, L); j += 8) {
+    const uint4* src = cache + (static_cast<size_t>(block_tables[static_cast<size_t>(b) * max_blocks + j / bs]) * bs + j % bs) * words;
+    uint4* dst = out + static_cast<size_t>(row0 + j) * words;
+    for (int i = lane; i < words; i += 32) dst[i] = src[i];
+  }
+}
+
 }  // namespace ksana
 
 using namespace ksana;
+
+// bf16. -1: rows are not multiples of 16 bytes.
+KSANA_API int ksana_latent_gather(const void* cache, const int* block_tables, int max_blocks, const int* kv_lens,
+                                  int seq_base, int num_seqs, int max_kv, int bs, int width, void* out, cudaStream_t st) {
+  if (num_seqs <= 0 || max_kv <= 0) return 0;
+  if (width & 7) return -1;
+  latent_gather_kernel<<<dim3((max_kv + 31) / 32, num_seqs), 256, 0, st>>>(
+      static_cast<const uint4*>(cache), block_tables, max_blocks, kv_lens, seq_base, bs, width / 8,
+      static_cast<uint4*>(out));
+  return cudaGetLastError() == cudaSuccess ? 0 : -5;
+}
 
 // q: [tokens, h * (dim + rot)] (pitch ldq); q_cat: [tokens - cat_from, h, rank + rot] or null; x: [tokens, rank + rot]
 // (pitch ldx). A slot is a row of the cache. kind: 0 fp32, 1 bf16.

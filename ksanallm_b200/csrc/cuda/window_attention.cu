@@ -73,9 +73,13 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
     float s = -INFINITY;
     if (i < n) {
       const T* kp = cache + bt[j / a.bs] * block_elems + (static_cast<size_t>(kh) * a.bs + j % a.bs) * a.d;
-      float dot = 0.f;
-      for (int c = 0; c < a.d; ++c) dot += sq[c] * to_f(kp[c]);
-      s = dot * a.scale;
+      float dot[4] = {0.f, 0.f, 0.f, 0.f};
+      int c = 0;
+      for (; c + 4 <= a.d; c += 4)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) dot[u] = fmaf(sq[c + u], to_f(kp[c + u]), dot[u]);
+      for (; c < a.d; ++c) dot[0] = fmaf(sq[c], to_f(kp[c]), dot[0]);
+      s = ((dot[0] + dot[1]) + (dot[2] + dot[3])) * a.scale;
       if (a.softcap > 0.f) s = a.softcap * tanhf(s / a.softcap);
       if (bias) s += bias[min(pos - j, a.bias_len - 1)];
     }
@@ -84,8 +88,9 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
     const float p = i < n ? expf(s - m_new) : 0.f;
     l = l * f + warp_sum(p);
     m = m_new;
+    float part[NV];  // of these 32 keys: long sums in two steps keep their rounding small
 #pragma unroll
-    for (int i = 0; i < NV; ++i) acc[i] *= f;
+    for (int i = 0; i < NV; ++i) part[i] = 0.f;
     const int count = min(32, n - i0);
     for (int u = 0; u < count; ++u) {
       const float pu = __shfl_sync(0xffffffffu, p, u);
@@ -95,9 +100,11 @@ window_attention_any_kernel(WindowAttnArgs a, int tok_base, int tokens) {
 #pragma unroll
       for (int i = 0; i < NV; ++i) {
         const int c = i * 32 + lane;
-        if (c < a.dv) acc[i] += pu * to_f(vp[c]);
+        if (c < a.dv) part[i] = fmaf(pu, to_f(vp[c]), part[i]);
       }
     }
+#pragma unroll
+    for (int i = 0; i < NV; ++i) acc[i] = fmaf(acc[i], f, part[i]);
   }
   T* o = static_cast<T*>(a.out) + static_cast<size_t>(t) * a.ldo + head * a.dv;
   if (a.sink) {  // relative to the larger of the running maximum and the sink's own score
@@ -146,6 +153,9 @@ static int launch_any(const WindowAttnArgs& a, int tok_base, int tokens, cudaStr
 // tokens ahead of it come first. Where a block holds kept tokens its table has no window cut, and the scores are masked
 // one by one. Head sizes below DP / DVP are filled up with zeros by TMA.
 //
+// LATENT: keys and values of every head have been written out of the latents, [row][h x d keys | h x dv values] with the
+// contexts of the sequences behind one another; the last 64 columns of a key are the rotated part all heads share.
+//
 // SHARED: the values are the keys. Both products read the same tile in shared memory - rows of keys are K-major for
 // Q K^T and MN-major for P V - and the values' room holds a third tile in flight.
 constexpr int WP_PAGE = 16;
@@ -182,10 +192,12 @@ __device__ __forceinline__ float cap_any(float s, float c, float inv_c) {
   return c - __fdividef(2.f * c, 1.f + __expf(2.f * x));
 }
 
-template <int DP, int DVP, bool SHARED, bool KEEP, bool CAP>
+template <int DP, int DVP, bool SHARED, bool KEEP, bool CAP, bool LATENT = false>
 __global__ void __launch_bounds__(160, 1)
 window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK,
-                      const __grid_constant__ CUtensorMap tmV, WindowAttnArgs a, int seq_base, unsigned int* err) {
+                      const __grid_constant__ CUtensorMap tmV, const __grid_constant__ CUtensorMap tmR,
+                      WindowAttnArgs a, int seq_base, unsigned int* err) {
+  constexpr int DN = LATENT ? DP - 64 : DP;  // columns of a key's own
   using L_ = WindowPrefillSmem<DP, DVP, SHARED>;
   constexpr int STAGES = L_::STAGES;
   const int b = blockIdx.y + seq_base, head = blockIdx.z, qt = blockIdx.x;
@@ -256,8 +268,31 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
                         kh * WP_PAGE, blk);
         }
       };
-      auto load_k = [&](int i) { load(tmK, sK, L_::K_BYTES, DP / 64, k_full, i, i % STAGES); k_loads = i + 1; };
-      auto load_v = [&](int i) { load(tmV, sV, L_::V_BYTES, DVP / 64, v_full, i, i & 1); v_loads = i + 1; };
+      int ctx0 = 0;  // LATENT: the sequence's first row
+      if constexpr (LATENT)
+        for (int i = seq_base; i < b; ++i) ctx0 += a.kv_lens[i];
+      auto load_k = [&](int i) {
+        if constexpr (LATENT) {
+          uint8_t* dst = sK + (i % STAGES) * L_::K_BYTES;
+          uint64_t* bar = &k_full[i % STAGES];
+          mbar_expect_tx(bar, L_::K_BYTES);
+          for (int hf = 0; hf < DN / 64; ++hf) tma_load_3d(dst + hf * (128 * 128), &tmK, bar, hf * 64, head, ctx0 + i * 128);
+          tma_load_2d(dst + (DN / 64) * (128 * 128), &tmR, bar, 0, ctx0 + i * 128);
+        } else {
+          load(tmK, sK, L_::K_BYTES, DP / 64, k_full, i, i % STAGES);
+        }
+        k_loads = i + 1;
+      };
+      auto load_v = [&](int i) {
+        if constexpr (LATENT) {
+          mbar_expect_tx(&v_full[i & 1], L_::V_BYTES);
+          for (int hf = 0; hf < DVP / 64; ++hf)
+            tma_load_3d(sV + (i & 1) * L_::V_BYTES + hf * (128 * 128), &tmV, &v_full[i & 1], hf * 64, head, ctx0 + i * 128);
+        } else {
+          load(tmV, sV, L_::V_BYTES, DVP / 64, v_full, i, i & 1);
+        }
+        v_loads = i + 1;
+      };
       auto issue_qk = [&](int i) {
         tc_fence_after();
         constexpr uint32_t idesc = umma_idesc(128, 128, 1, 1);
@@ -270,7 +305,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
         umma_commit(&s_done[i & 1]);
       };
       mbar_expect_tx(q_bar, L_::Q_BYTES);
-      for (int hf = 0; hf < DP / 64; ++hf) tma_load_3d(sQ + hf * (128 * 128), &tmQ, q_bar, hf * 64, head, q0 + qt * 128);
+      for (int hf = 0; hf < DP / 64; ++hf)
+        tma_load_3d(sQ + hf * (128 * 128), &tmQ, q_bar, LATENT && hf == DN / 64 ? a.d : hf * 64, head, q0 + qt * 128);
       load_k(0);
       if constexpr (!SHARED) load_v(0);
       for (int i = 1; i < STAGES && i < n; ++i) load_k(i);
@@ -478,7 +514,30 @@ static int launch_prefill(const WindowAttnArgs& a, int total_tokens, int num_blo
   if (int rc = cache_maps(a, num_blocks, &tk, &tv)) return rc;
   auto kern = window_prefill_kernel<DP, DVP, SHARED, KEEP, CAP>;
   if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
-  kern<<<dim3((max_q + 127) / 128, num_seqs, a.h), 160, L_::TOTAL, st>>>(tq, tk, tv, a, seq_base, error_word());
+  kern<<<dim3((max_q + 127) / 128, num_seqs, a.h), 160, L_::TOTAL, st>>>(tq, tk, tv, tk, a, seq_base, error_word());
+  return cudaGetLastError() == cudaSuccess ? 0 : -5;
+}
+
+// d, dv: a head's unrotated key and value sizes; kv: [rows][h * d | h * dv] (pitch ldkv); rot: [rows][rd] (pitch ldr)
+template <int DP, int DVP>
+static int launch_latent(const WindowAttnArgs& a, int total_tokens, const void* kv, int ldkv, const void* rot, int ldr,
+                         int rd, int rows, int seq_base, int num_seqs, int max_q, cudaStream_t st) {
+  using L_ = WindowPrefillSmem<DP, DVP, false>;
+  CUtensorMap tq, tk, tv, tr;
+  auto heads_map = [&](CUtensorMap* m, const void* base, int cols, int pitch, int count) {
+    const uint64_t dims[3] = {static_cast<uint64_t>(cols), static_cast<uint64_t>(a.h), static_cast<uint64_t>(count)};
+    const uint64_t str[2] = {static_cast<uint64_t>(cols) * 2, static_cast<uint64_t>(pitch) * 2};
+    const uint32_t box[3] = {64, 1, 128};
+    return make_tmap_nd(m, base, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B);
+  };
+  if (heads_map(&tq, a.q, a.d + rd, a.ldq, total_tokens) || heads_map(&tk, kv, a.d, ldkv, rows) ||
+      heads_map(&tv, static_cast<const char*>(kv) + static_cast<size_t>(a.h) * a.d * 2, a.dv, ldkv, rows))
+    return -2;
+  if (make_tmap_2d(&tr, rot, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, rd, ldr, 128, 64, CU_TENSOR_MAP_SWIZZLE_128B))
+    return -3;
+  auto kern = window_prefill_kernel<DP, DVP, false, false, false, true>;
+  if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
+  kern<<<dim3((max_q + 127) / 128, num_seqs, a.h), 160, L_::TOTAL, st>>>(tq, tk, tv, tr, a, seq_base, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
@@ -521,7 +580,7 @@ struct WindowDecodeSmem {
   static constexpr int STAGES = PAGE <= 2048 ? 4 : PAGE <= 4096 ? 3 : 2;
   static constexpr int RING = 4 * STAGES * PAGE;
   static constexpr int LDO = DVP + 4;
-  static constexpr int MERGE = 4 * 16 * LDO * 4;  // over the ring, once every page has been multiplied
+  static constexpr int MERGE = 4 * (DVP > 256 ? 8 : 16) * LDO * 4;  // over the ring, once every page has been multiplied
   static constexpr int TOTAL = (RING > MERGE ? RING : MERGE) + 1024;
 };
 
@@ -538,11 +597,11 @@ window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
   volatile int* abort_flag = &abort_word;
   uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
   const int splits = gridDim.x, split = blockIdx.x;
-  const int kh = blockIdx.y / groups, part = blockIdx.y % groups;
+  const int kh = blockIdx.y / groups, hpart = blockIdx.y % groups;
   const int b = blockIdx.z + seq_base;
   const int gq = a.h / a.hk;
-  const int head0 = kh * gq + part * 16;
-  const int g = min(16, gq - part * 16);        // query heads of this CTA, at most 8 NT
+  const int head0 = kh * gq + hpart * 8 * NT;
+  const int g = min(8 * NT, gq - hpart * 8 * NT);  // query heads of this CTA
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
   const int r = lane >> 2, j2 = (lane & 3) * 2;
 
@@ -630,19 +689,30 @@ window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
       break;
     }
     const uint32_t kb0 = smem_u32(ring + (n % STAGES) * L_::PAGE), vb0 = kb0 + (SHARED ? 0 : L_::K_BYTES);
-    float c[NT][4];
+    constexpr int CHAINS = DP > 128 ? 4 : 1;  // independent sums over long keys
+    float c[NT][4], part[CHAINS][NT][4];
 #pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
+    for (int x = 0; x < CHAINS; ++x)
 #pragma unroll
-      for (int u = 0; u < 4; ++u) c[nt][u] = 0.f;
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int u = 0; u < 4; ++u) part[x][nt][u] = 0.f;
 #pragma unroll
     for (int kb = 0; kb < DP / 16; ++kb) {
       uint32_t f[4];
       const int ch = kb * 2 + k_col;
       ldmatrix_x4<false>(f, kb0 + (ch >> 3) * 2048 + k_row * 128 + (((ch & 7) ^ (k_row & 7)) << 4));
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) mma_16816(c[nt], f, qf[kb][nt][0], qf[kb][nt][1]);
+      for (int nt = 0; nt < NT; ++nt) mma_16816(part[kb % CHAINS][nt], f, qf[kb][nt][0], qf[kb][nt][1]);
     }
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+      for (int u = 0; u < 4; ++u) {
+        c[nt][u] = part[0][nt][u];
+#pragma unroll
+        for (int x = 1; x < CHAINS; ++x) c[nt][u] += part[x][nt][u];
+      }
     const int key0 = page(n) * 16 + r;
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
@@ -804,7 +874,7 @@ template <int DP, int DVP, int NT, bool SHARED>
 static int launch_decode(const WindowAttnArgs& a, int num_blocks, int seq_base, int num_seqs, int max_kv,
                          cudaStream_t st) {
   using L_ = WindowDecodeSmem<DP, DVP, SHARED>;
-  const int gq = a.h / a.hk, groups = (gq + 15) / 16;
+  const int gq = a.h / a.hk, groups = (gq + 8 * NT - 1) / (8 * NT);
   CUtensorMap tk, tv;
   if (int rc = cache_maps(a, num_blocks, &tk, &tv)) return rc;
   auto kern = window_decode_kernel<DP, DVP, NT, SHARED>;
@@ -875,12 +945,24 @@ KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, int
                                   float out_scale, float softcap, int sink, const void* gate, int ldg, void* out,
                                   int ldo, int seq_base, int num_seqs, int max_kv, cudaStream_t st) {
   if (num_seqs <= 0) return 0;
-  if (keep < 0 || (shared && d != dv)) return -2;
-  if (h % hk || bs != WP_PAGE || d > 128 || dv > 128 || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
+  if (keep < 0 || (shared && d < dv)) return -2;
+  const int top = shared ? 576 : 128;
+  if (h % hk || bs != WP_PAGE || d > top || dv > top || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
       !rows16(out, ldo))
     return -1;
   WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
                    shared, scale, bias, bias_len, out_scale, out, ldo, softcap, sink, gate, ldg};
+  if (shared && (d > 128 || d != dv)) {  // latents: long keys, values the first part of them
+#define KSANA_WL(DP, DVP) \
+  if (d <= DP && dv <= DVP) return launch_decode<DP, DVP, 1, true>(a, num_blocks, seq_base, num_seqs, max_kv, st)
+    KSANA_WL(64, 64);
+    KSANA_WL(128, 128);
+    KSANA_WL(192, 128);
+    KSANA_WL(320, 256);
+    KSANA_WL(576, 512);
+#undef KSANA_WL
+    return -1;
+  }
 #define KSANA_WD(DP, DVP, SHARED)                                                                             \
   return h / hk <= 8 ? launch_decode<DP, DVP, 1, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)       \
                      : launch_decode<DP, DVP, 2, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)
@@ -893,6 +975,26 @@ KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, int
   if (dv <= 64) KSANA_WD(128, 64, false);
   KSANA_WD(128, 128, false);
 #undef KSANA_WD
+}
+
+// Prompts over keys and values that were written out of latents (see launch_latent). bf16; -1 for sizes it does not take.
+KSANA_API int ksana_latent_prefill(const void* q, int ldq, int total_tokens, const void* kv, int ldkv, const void* rot,
+                                   int ldr, int rows, const int* cu_q, const int* kv_lens, int h, int d, int rd, int dv,
+                                   float scale, const void* gate, int ldg, void* out, int ldo, int seq_base, int num_seqs,
+                                   int max_q, cudaStream_t st) {
+  if (num_seqs <= 0 || max_q <= 0) return 0;
+  if (d > 128 || dv > 128 || rd > 64 || (d & 7) || (dv & 7) || (rd & 7) || !rows16(q, ldq) || !rows16(kv, ldkv) ||
+      !rows16(rot, ldr) || !rows16(out, ldo))
+    return -1;
+  WindowAttnArgs a{q, ldq, nullptr, nullptr, 0, cu_q, kv_lens, nullptr, h, h, d, dv, WP_PAGE, 0, 0, 0, scale, nullptr, 0,
+                   1.f, out, ldo, 0.f, 0, gate, ldg};
+#define KSANA_LP(DP, DVP) \
+  return launch_latent<DP, DVP>(a, total_tokens, kv, ldkv, rot, ldr, rd, rows, seq_base, num_seqs, max_q, st)
+  if (d <= 64 && dv <= 64) KSANA_LP(128, 64);
+  if (d <= 64) KSANA_LP(128, 128);
+  if (dv <= 64) KSANA_LP(192, 64);
+  KSANA_LP(192, 128);
+#undef KSANA_LP
 }
 
 // Tokens [tok_base, tok_base + tokens) of the step, whatever sequences they belong to. kind: 0 fp32, 1 bf16.

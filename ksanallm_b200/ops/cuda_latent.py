@@ -3,8 +3,8 @@ from __future__ import annotations
 
 import torch
 
-from .cuda import _check, _ptr, _stream, lib
-from .cuda_mixer import _KIND, window_attention
+from .cuda import _check, _ptr, _stream, gemm_bf16, lib
+from .cuda_mixer import _KIND
 
 
 def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tensor:
@@ -23,22 +23,76 @@ def head_gemm(a: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> torch.Tens
     return out
 
 
+# Keys and values that prompts have written out at a time: more contexts than this go in several rounds.
+EXPAND_BYTES = 1 << 30
+
+
+def _prompts(q, cache, meta, block_size: int, w, scale: float, gate, out) -> bool:
+    """The step's prompt portions over keys and values written out per head. False: sizes the kernel does not take."""
+    T, h, qd = q.shape
+    rank, dim, vdim = w.rank, w.dim, w.vdim
+    rot, width = qd - dim, rank + qd - dim
+    if q.dtype != torch.bfloat16 or (rank | rot | dim | vdim) % 8 or dim > 128 or vdim > 128 or rot > 64:
+        return False
+    n_pre, cu, kl = meta.num_prefill, meta.cu_q_host, meta.kv_lens_host
+    per_row = 2 * h * (dim + vdim)
+    lo = 0
+    while lo < n_pre:
+        hi, rows = lo, 0
+        while hi < n_pre and (hi == lo or (rows + int(kl[hi])) * per_row <= EXPAND_BYTES):
+            rows += int(kl[hi])
+            hi += 1
+        lat = torch.empty(rows, width, dtype=q.dtype, device=q.device)
+        _check(lib().ksana_latent_gather(_ptr(cache), _ptr(meta.block_tables), meta.max_blocks, _ptr(meta.kv_lens), lo,
+                                         hi - lo, int(kl[lo:hi].max()), block_size, width, _ptr(lat), _stream()),
+               "latent_gather")
+        kv = gemm_bf16(lat[:, :rank], w.expand)
+        code = lib().ksana_latent_prefill(
+            _ptr(q), q.stride(0), T, _ptr(kv), kv.stride(0), lat.data_ptr() + 2 * rank, width, rows, _ptr(meta.cu_q),
+            _ptr(meta.kv_lens), h, dim, rot, vdim, float(scale), _ptr(gate), gate.stride(0) if gate is not None else 0,
+            _ptr(out), out.stride(0), lo, hi - lo, int((cu[lo + 1:hi + 1] - cu[lo:hi]).max()), _stream())
+        if code == -1:
+            return False
+        _check(code, "latent_prefill")
+        lo = hi
+    return True
+
+
 def latent_attention(q, a, norm_w, eps: float, rotary, cache, meta, block_size: int, w, scale: float, gate,
                      out: torch.Tensor) -> None:
-    """See ``reference.latent_append`` and ``reference.latent_attention``."""
+    """See ``reference.latent_append`` and ``reference.latent_attention``. bf16 prompts attend to keys and values that are
+    written out of the latents per head; single tokens, fp32 and other sizes to the latents themselves."""
     T, h, qd = q.shape
     rank, dim, vdim = w.rank, w.dim, w.vdim
     rot = qd - dim
     assert q.stride(2) == 1 and q.stride(1) == qd and a.stride(1) == 1 and out.stride(1) == 1 and cache.is_contiguous()
-    q_cat = torch.empty(T, h, rank + rot, dtype=q.dtype, device=q.device)
-    _check(lib().ksana_latent_append(_ptr(q), q.stride(0), dim, _ptr(q_cat), 0, _ptr(a), a.stride(0), _ptr(norm_w),
+    n_pre, n_dec = meta.num_prefill, meta.num_decode
+    first = meta.num_prefill_tokens if q.dtype == torch.bfloat16 and n_pre else 0  # tokens from here on: absorbed queries
+    q_cat = torch.empty(T - first, h, rank + rot, dtype=q.dtype, device=q.device)
+    _check(lib().ksana_latent_append(_ptr(q), q.stride(0), dim, _ptr(q_cat), first, _ptr(a), a.stride(0), _ptr(norm_w),
                                      float(eps), _ptr(meta.positions), _ptr(rotary), _ptr(meta.slot_mapping),
                                      _ptr(cache), T, h, rank, rot, _KIND[q.dtype], _stream()), "latent_append")
-    head_gemm(q[..., :dim], w.uk_t, q_cat[..., :rank])
-    o = torch.empty(T, h * rank, dtype=q.dtype, device=q.device)
-    _check(lib().ksana_window_attention_any(
-        _ptr(q_cat), q_cat.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks, _ptr(meta.cu_q),
-        _ptr(meta.kv_lens), _ptr(meta.seq_of_token), h, 1, rank + rot, rank, block_size, 0, 0, 1, float(scale), None, 0,
-        1.0, 0.0, 0, _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(o), o.stride(0), 0, T, _KIND[q.dtype],
-        _stream()), "latent_attention_any")
-    head_gemm(o.view(T, h, rank), w.uv, out.unflatten(1, (h, vdim)))
+    if first and not _prompts(q, cache, meta, block_size, w, scale, gate, out):
+        q_cat = torch.empty(T, h, rank + rot, dtype=q.dtype, device=q.device)
+        q_cat[..., rank:] = q[..., dim:]
+        first = 0
+    if first == T:
+        return
+    head_gemm(q[first:, :, :dim], w.uk_t, q_cat[..., :rank])
+    o = torch.empty(T - first, h * rank, dtype=q.dtype, device=q.device)
+    # the kernels index tokens of the whole step
+    at = [x.data_ptr() - first * x.stride(0) * x.element_size() for x in (q_cat, o)]
+    shape = (h, 1, rank + rot, rank, block_size, 0, 0, 1, float(scale), None, 0, 1.0, 0.0, 0, _ptr(gate),
+             gate.stride(0) if gate is not None else 0)
+    code = -1
+    if q.dtype == torch.bfloat16 and n_dec == T - first:
+        code = lib().ksana_window_decode(at[0], q_cat.stride(0), _ptr(cache), cache.shape[0], _ptr(meta.block_tables),
+                                         meta.max_blocks, _ptr(meta.cu_q), _ptr(meta.kv_lens), *shape, at[1], o.stride(0),
+                                         n_pre, n_dec, int(meta.kv_lens_host[n_pre:].max()), _stream())
+    if code == -1:
+        code = lib().ksana_window_attention_any(
+            at[0], q_cat.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks, _ptr(meta.cu_q),
+            _ptr(meta.kv_lens), _ptr(meta.seq_of_token), *shape, at[1], o.stride(0), first, T - first, _KIND[q.dtype],
+            _stream())
+    _check(code, "latent_attention")
+    head_gemm(o.view(T - first, h, rank), w.uv, out[first:].unflatten(1, (h, vdim)))
