@@ -980,6 +980,12 @@ class WeightLoader:
                 else:
                     self._finish_attn(key, parts)
             else:
+                spec = cfg.layers[self._layer_of(key)] if cfg.layers else None
+                if spec is not None and spec.ff:
+                    need = {f"{x}_proj.{y}" for x in (("gate", "up", "down") if spec.gated else ("up", "down"))
+                            for y in (("weight", "bias") if spec.ff_bias else ("weight",))}
+                    if need - set(parts):
+                        raise KeyError(f"{key}: the checkpoint has no {', '.join(sorted(need - set(parts)))}")
                 self._finish_mlp(key, parts)
         for key, ex in list(self._experts.items()):
             self._finish_experts(key, ex)
