@@ -4,10 +4,13 @@ closest other model of the same width, heads and depth. Random weights, bf16, on
 
     python bench.py --throughput molopel
     python bench.py --throughput givirax
+    python bench.py --throughput ladusun
 
 Molopel: beside the dense model (Qwen3 blocks: QK norm, grouped-query attention, SwiGLU) whose feed-forward is as wide as
 makes the parameter counts equal. Givirax (half of its layers run twice): beside Qwen3-MoE blocks, dense and routed in
 turn, as many layers as Givirax has runs, with the same experts and a gated feed-forward of the same number of weights.
+Ladusun (four residual streams): beside DeepSeek blocks (latent attention, routed experts) of the same width, depth, heads
+and latent size, dense and routed in turn, with the same experts and a gated feed-forward of the same number of weights.
 
 prefill: prompts of 4096 tokens, 8192 tokens a step. decode: 128 sequences behind prompts of 1024 tokens, one token each
 per step. Weights and caches are larger than L2, so each step starts cold. CUDA events around the timed steps; the host
@@ -20,7 +23,7 @@ import time
 
 import torch
 
-from ksanallm_b200.config.model_config import givirax_config, model_config_from_dict, molopel_config
+from ksanallm_b200.config.model_config import givirax_config, ladusun_config, model_config_from_dict, molopel_config
 from ksanallm_b200.config.schema import parse_serving_config
 from ksanallm_b200.engine.llm_engine import LLMEngine
 from ksanallm_b200.engine.sampling_params import SamplingParams
@@ -33,6 +36,9 @@ SIZES = [(2048, 8, 6144, 16, 4, 1024), (4096, 8, 12288, 32, 8, 1024), (8192, 4, 
 # width, depth, feed-forward, experts, experts per token, expert width, heads, key / value heads, window
 GIVIRAX_SIZES = [(2048, 8, 8192, 16, 2, 2048, 16, 4, 1024), (4096, 8, 16384, 16, 2, 4096, 32, 8, 1024),
                  (8192, 4, 32768, 8, 2, 8192, 64, 8, 2048)]
+# width, depth, feed-forward, experts, experts per token, expert width, heads, key / value heads, latent size
+LADUSUN_SIZES = [(2048, 8, 8192, 16, 2, 2048, 16, 4, 512), (4096, 8, 16384, 16, 2, 4096, 32, 8, 512),
+                 (8192, 4, 32768, 8, 2, 8192, 64, 8, 512)]
 PROMPT, STEP_TOKENS = 4096, 8192
 BATCH, CONTEXT, DECODE_STEPS = 128, 1024, 40
 
@@ -55,6 +61,16 @@ def moe_config(width, depth, ff, experts, top, expert_ff, heads, kv_heads):
         num_experts=experts, num_experts_per_tok=top, norm_topk_prob=True, rms_norm_eps=1e-6, vocab_size=32000,
         mlp_layer_types=["sparse" if i % 2 else "dense" for i in range(depth)],
         max_position_embeddings=8192, torch_dtype="bfloat16", eos_token_id=2))
+
+
+def mla_config(width, depth, ff, experts, top, expert_ff, heads, rank):
+    return model_config_from_dict(dict(
+        model_type="deepseek_v2", hidden_size=width, num_hidden_layers=depth, num_attention_heads=heads,
+        num_key_value_heads=heads, intermediate_size=ff, moe_intermediate_size=expert_ff, n_routed_experts=experts,
+        num_experts_per_tok=top, n_group=4, topk_group=2, topk_method="group_limited_greedy", scoring_func="softmax",
+        norm_topk_prob=True, kv_lora_rank=rank, qk_nope_head_dim=128, qk_rope_head_dim=64, v_head_dim=128,
+        mlp_layer_types=["sparse" if i % 2 else "dense" for i in range(depth)], rms_norm_eps=1e-6, vocab_size=32000,
+        max_position_embeddings=8192, torch_dtype="bfloat16", eos_token_id=2, tie_word_embeddings=True))
 
 
 def build(cfg):
@@ -147,9 +163,25 @@ def run_givirax() -> None:
                               keep_first=4, dtype="bf16", data="synthetic", **rows)), flush=True)
 
 
+def run_ladusun() -> None:
+    for width, depth, ff, experts, top, expert_ff, heads, kv, rank in LADUSUN_SIZES:
+        rows = {}
+        for name, cfg in (("ladusun", ladusun_config(width, depth, ff, experts, top, expert_ff, heads, kv, 128, rank)),
+                          ("latent_moe", mla_config(width, depth, ff * 2 // 3 // 128 * 128, experts, top, expert_ff, heads, rank))):
+            model, n = build(cfg)
+            rows[name] = dict(parameters_m=round(n / 1e6), **measure(model))
+            del model
+            torch.cuda.empty_cache()
+        print(json.dumps(dict(metric="throughput", design="ladusun", width=width, layers=depth, ff=ff, experts=experts, top=top,
+                              expert_ff=expert_ff, heads=heads, kv_heads=kv, rank=rank, streams=4, dtype="bf16",
+                              data="synthetic", **rows)), flush=True)
+
+
 def run(design: str) -> None:
     if design == "givirax":
         return run_givirax()
+    if design == "ladusun":
+        return run_ladusun()
     assert design == "molopel"
     for width, depth, ff, heads, kv, window in SIZES:
         rows = {}

@@ -1,6 +1,7 @@
-// Native forward pass of layers with mixers of their own sizes (windowed attention and / or linear attention, a norm over
-// a 32-bit residual stream, a dense or routed FFN behind or beside the mixers), driven from ONE call per step. A layer
-// that runs several times is listed once per run. Mirrored with ctypes on the Python side.
+// Native forward pass of layers with mixers of their own sizes (windowed attention and / or linear attention, latent
+// attention, a gated recurrence; a norm over a 32-bit residual stream, or over several hyper-connected ones; a dense or
+// routed FFN behind or beside the mixers), driven from ONE call per step. A layer that runs several times is listed once
+// per run. Mirrored with ctypes on the Python side.
 #pragma once
 #include <cuda_runtime.h>
 
@@ -8,19 +9,25 @@ extern "C" {
 
 struct KsanaMixerLayer {
   // weights, bf16
-  const void* w_in;      // [n_in, H]: attention q, k, v, linear attention q, k, v, gate, then a parallel dense FFN's input
+  const void* w_in;      // [n_in, H]: attention q, k, v, head gates (or latent q, latent, head gates, or the recurrence's
+                         // y, x), linear attention q, k, v, gate, then a parallel dense FFN's input
   const void* b_in;      // optional bias [n_in]
   const void* w_out;     // [H, k_out]: attention columns, linear-attention columns, a parallel dense FFN's, zero padding
+  const void* b_out;     // optional bias [H]
   const void* ln2;       // norm before the FFN (null: the layer has none, or it reads the mixers' norm)
-  const void* w_gu;      // [2 I, H] gate rows, then up rows
+  const void* w_gu;      // [2 I, H] gate rows, then up rows; plain: [I, H]
+  const void* b_up;      // plain: optional bias [I]
+  const void* b_down;    // plain: optional bias [H]
   const void* w_gu_il;   // optional copy of w_gu, gate / up rows interleaved in groups of 16: prompt-sized steps then run
                          // the activation as the GEMM's epilogue
   const void* w_down;    // [H, I]
   const void* next_ln;   // next layer's first norm, or the final norm
   int n_in, k_out, inter;
+  int plain;             // FFN behind the mixers: squared ReLU instead of gated GELU
   // FFN beside the mixers: dense of width `inter` inside w_in / w_out, or routed experts (experts > 0)
   int parallel, gated;
-  int experts, top, expert_inter, router_rows;
+  int experts, top, expert_inter, router_rows, groups, keep_groups;
+  float limit, alpha;           // limit > 0: clamped gates
   const void* w_router;         // [router_rows, H], rows from `experts` on are padding
   const float* b_router;        // optional [experts]
   const void* w_expert_gu;      // [experts, 2 expert_inter, H]
@@ -30,7 +37,10 @@ struct KsanaMixerLayer {
   int next_start;               // add the embedding output
   // softmax attention (h == 0: none)
   int h, hk, d, dv, window, keep_first, shared_kv, bias_len;
-  float scale, attn_out_scale;
+  float scale, attn_out_scale, softcap;
+  int sink, head_gate, reads;  // reads: another layer's keys and values, nothing is appended
+  int rot;                     // rotated dimensions (of latent attention: its shared part)
+  const float* rot_table;
   const float* q_norm;
   const float* k_norm;
   const float* bias;     // [h, bias_len]
@@ -42,10 +52,32 @@ struct KsanaMixerLayer {
   const float* rotary;
   const float* norm_w;   // null: per-head norm without weight
   float* state;          // this layer's state pool
+  // latent attention (ah == 0: none)
+  int ah, adim, avdim, arank;
+  float ascale;
+  const float* anorm;
+  const void* a_uk_t;    // [ah, arank, adim]
+  const void* a_uv;      // [ah, avdim, arank]
+  const void* a_expand;  // [ah (adim + avdim), arank]
+  // gated recurrence (rc == 0: none)
+  int rc, rk, rb;
+  const float* conv_w;
+  const float* conv_b;
+  const void* gates;           // [2, rb, rc / rb, rc / rb]
+  const void* gates_by_block;  // [rb, 2 rc / rb, rc / rb]
+  const float* gates_b;
+  const float* rate;
+  // hyper-connections of the two sublayers, and their layer scales
+  const float* ls[2];
+  const float* hc_in[2];
+  const float* hc_mix[2];
+  const float* hc_out[2];
+  const float* next_in;        // how the next layer (or the final norm) reads the streams
 };
 
 struct KsanaMixerModel {
   int hidden, block_size, num_blocks, center;  // center: LayerNorm, else RMS norm
+  int streams;                                 // 0: one residual stream
   float eps;
   // scratch for max_tokens rows
   void* in_buf;    // [T, max n_in]
@@ -69,6 +101,8 @@ struct KsanaMixerModel {
   void* rows_out_buf;
   float* chunk_buf;
   long long chunk_floats;
+  void* lat_buf;           // scratch of latent attention
+  long long lat_bytes, expand_bytes;  // expand_bytes: keys and values that prompts have written out at a time
   float* gemm_ws;
   long long gemm_ws_floats;
   unsigned int* gemm_counters;
@@ -91,11 +125,16 @@ struct KsanaMixerStep {
   int one_token;         // every decode sequence has exactly one new token
   int num_long;          // leading prompt portions long enough for the chunked form of linear attention
   int long_tokens;       // their tokens
+  const int* cu_q_host;
+  const int* kv_lens_host;
 };
 
 // h: normalised input of layer `first` ([T, H] bf16), residual: [T, H] fp32 stream, updated in place. *out_h receives
 // the pointer of the normalised output. Returns 0, or (layer + 1) * 100 + step on failure with the failing call's code
 // in *fail_code.
+// Bytes of lat_buf that a step needs (the largest layer's).
+long long ksana_mixer_latent_bytes(const KsanaMixerModel* m, const KsanaMixerStep* s, int layers);
+
 int ksana_mixer_forward(const KsanaMixerModel* m, const KsanaMixerStep* s, const void* h, float* residual, int first,
                         int last, void** out_h, int* fail_code, int* launches, cudaStream_t stream);
 }

@@ -15,6 +15,7 @@ import numpy as np
 import torch
 
 from ..ops import cuda as kcuda
+from ..ops import cuda_latent
 
 P, I, F, LL = ctypes.c_void_p, ctypes.c_int, ctypes.c_float, ctypes.c_longlong
 
@@ -297,23 +298,29 @@ class DenseExecutor:
 # ---- layers with mixers of their own sizes (csrc/cuda/mixer_executor.cu) ---------------------------------------------
 
 class _MixerLayer(ctypes.Structure):
-    _fields_ = [(n, P) for n in ("w_in", "b_in", "w_out", "ln2", "w_gu", "w_gu_il", "w_down", "next_ln")] + \
-        [(n, I) for n in ("n_in", "k_out", "inter", "parallel", "gated", "experts", "top", "expert_inter",
-                          "router_rows")] + \
+    _fields_ = [(n, P) for n in ("w_in", "b_in", "w_out", "b_out", "ln2", "w_gu", "b_up", "b_down", "w_gu_il", "w_down",
+                                 "next_ln")] + \
+        [(n, I) for n in ("n_in", "k_out", "inter", "plain", "parallel", "gated", "experts", "top", "expert_inter",
+                          "router_rows", "groups", "keep_groups")] + [("limit", F), ("alpha", F)] + \
         [(n, P) for n in ("w_router", "b_router", "w_expert_gu", "w_expert_down", "next_vec")] + \
         [(n, I) for n in ("next_start", "h", "hk", "d", "dv", "window", "keep_first", "shared_kv", "bias_len")] + \
-        [("scale", F), ("attn_out_scale", F), ("q_norm", P), ("k_norm", P), ("bias", P), ("kv", P)] + \
+        [("scale", F), ("attn_out_scale", F), ("softcap", F)] + [(n, I) for n in ("sink", "head_gate", "reads", "rot")] + \
+        [(n, P) for n in ("rot_table", "q_norm", "k_norm", "bias", "kv")] + \
         [(n, I) for n in ("lh", "ld", "ldv", "rd", "act", "gate")] + \
-        [("key_scale", F), ("lin_out_scale", F), ("decay", P), ("rotary", P), ("norm_w", P), ("state", P)]
+        [("key_scale", F), ("lin_out_scale", F), ("decay", P), ("rotary", P), ("norm_w", P), ("state", P)] + \
+        [(n, I) for n in ("ah", "adim", "avdim", "arank")] + [("ascale", F)] + \
+        [(n, P) for n in ("anorm", "a_uk_t", "a_uv", "a_expand")] + [(n, I) for n in ("rc", "rk", "rb")] + \
+        [(n, P) for n in ("conv_w", "conv_b", "gates", "gates_by_block", "gates_b", "rate")] + \
+        [(n, P * 2) for n in ("ls", "hc_in", "hc_mix", "hc_out")] + [("next_in", P)]
 
 
 class _MixerModel(ctypes.Structure):
-    _fields_ = [("hidden", I), ("block_size", I), ("num_blocks", I), ("center", I), ("eps", F), ("in_buf", P),
+    _fields_ = [("hidden", I), ("block_size", I), ("num_blocks", I), ("center", I), ("streams", I), ("eps", F), ("in_buf", P),
                 ("mix_buf", P), ("o_buf", P), ("gu_buf", P), ("act_buf", P), ("proj_buf", P), ("h_buf", P * 2)] + \
                [(n, P) for n in ("router_buf", "expert_ids", "expert_weights", "pair_pos", "pair_src", "sort_meta",
                                  "rows_buf", "rows_gu_buf", "rows_act_buf", "rows_out_buf")] + \
                [("chunk_buf", P),
-                ("chunk_floats", LL), ("gemm_ws", P), ("gemm_ws_floats", LL), ("gemm_counters", P), ("n_counters", I),
+                ("chunk_floats", LL), ("lat_buf", P), ("lat_bytes", LL), ("expand_bytes", LL), ("gemm_ws", P), ("gemm_ws_floats", LL), ("gemm_counters", P), ("n_counters", I),
                 ("layers", P)]
 
 
@@ -321,7 +328,8 @@ class _MixerStep(ctypes.Structure):
     _fields_ = [(n, P) for n in ("positions", "slot_mapping", "seq_of_token", "block_tables", "cu_q", "kv_lens",
                                  "state_slots", "start")] + \
         [(n, I) for n in ("total_tokens", "max_blocks", "num_prefill", "num_decode", "prefill_tokens", "max_q_prefill",
-                          "max_kv_decode", "one_token", "num_long", "long_tokens")]
+                          "max_kv_decode", "one_token", "num_long", "long_tokens")] + \
+        [("cu_q_host", P), ("kv_lens_host", P)]
 
 
 class MixerExecutor:
@@ -333,16 +341,14 @@ class MixerExecutor:
             return False
         if model.device.type != "cuda" or model.dtype != torch.bfloat16 or not model.layers or model.norm_w is None:
             return False
-        if model.cfg.streams:
-            return False
         for layer in model.layers:
             lins = [layer.in_proj, layer.o_proj] + ([layer.ffn.up, layer.ffn.down] if layer.ffn is not None else [])
             if any(lin.kind != "dense" or lin.pre is not None or lin.weight.dtype != torch.bfloat16 or
                    not lin.weight.is_contiguous() or lin.weight.shape[0] % 8 or lin.weight.shape[1] % 8 for lin in lins):
                 return False
-            if layer.o_proj.bias is not None or layer.ffn is not None and (
-                    layer.ffn.up.bias is not None or layer.ffn.down.bias is not None or not layer.ffn.gated or
-                    layer.ffn.act != "gelu_tanh"):
+            f = layer.ffn
+            if f is not None and (f.gated, f.act) != (False, "relu2") and (
+                    f.up.bias is not None or f.down.bias is not None or not f.gated or f.act != "gelu_tanh"):
                 return False
             e = layer.experts
             if e is not None:
@@ -363,13 +369,20 @@ class MixerExecutor:
             nxt = model.layers[i + 1].ln1 if i + 1 < n else model.norm_w
             L.w_in, L.b_in, L.w_out = _p(layer.in_proj.weight), _p(layer.in_proj.bias), _p(layer.o_proj.weight)
             L.n_in, L.k_out = layer.in_proj.weight.shape[0], layer.o_proj.weight.shape[1]
-            L.next_ln = _p(nxt)
+            L.b_out, L.next_ln = _p(layer.o_proj.bias), _p(nxt)
+            for j, c in enumerate(layer.hyper):
+                L.hc_in[j], L.hc_mix[j], L.hc_out[j] = _p(c.inp), _p(c.mix), _p(c.out)
+                L.ls[j] = _p((layer.ls1, layer.ls2)[j])
+            if layer.hyper:
+                L.next_in = _p(model.layers[i + 1].hyper[0].inp if i + 1 < n else model.stream_sum)
             L.parallel, L.gated = int(layer.spec.parallel), int(layer.spec.gated)
             if layer.parallel_ff:
                 L.inter = layer.parallel_ff
             if layer.experts is not None:
                 e, s = layer.experts, layer.spec.moe
                 L.experts, L.top, L.expert_inter = s.experts, s.top, e.w_down.shape[2]
+                L.groups, L.keep_groups, L.limit, L.alpha = s.groups, s.keep, s.limit, s.alpha
+                L.ln2 = _p(layer.ln2)
                 L.router_rows, L.w_router, L.b_router = e.gate_w.shape[0], _p(e.gate_w), _p(e.logit_bias)
                 L.w_expert_gu, L.w_expert_down = _p(e.w_gate_up), _p(e.w_down)
             start = model.layers[i + 1].pass_start if i + 1 < n else None
@@ -378,7 +391,8 @@ class MixerExecutor:
             if layer.ffn is not None:
                 L.ln2, L.w_gu, L.w_down = _p(layer.ln2), _p(layer.ffn.up.weight), _p(layer.ffn.down.weight)
                 L.inter = layer.ffn.down.weight.shape[1]
-                if os.environ.get("KSANA_FUSED_SWIGLU", "0") == "1" and L.inter % 16 == 0:  # see DenseExecutor
+                L.plain, L.b_up, L.b_down = int(not layer.ffn.gated), _p(layer.ffn.up.bias), _p(layer.ffn.down.bias)
+                if layer.ffn.gated and os.environ.get("KSANA_FUSED_SWIGLU", "0") == "1" and L.inter % 16 == 0:  # see DenseExecutor
                     key = layer.ffn.up.weight.data_ptr()  # (the runs of a looped layer share one copy)
                     if key not in self._wgu_il:
                         self._wgu_il[key] = kcuda.interleave_gate_up(layer.ffn.up.weight)
@@ -389,6 +403,18 @@ class MixerExecutor:
                 L.scale, L.attn_out_scale = s.scale, s.out_scale
                 L.keep_first, L.shared_kv = s.keep_first, int(s.shared_kv)
                 L.q_norm, L.k_norm = _p(a.q_norm), _p(a.k_norm)
+                L.softcap, L.sink, L.head_gate = s.softcap, int(s.sink), int(s.head_gate)
+                L.reads, L.rot = int(s.kv_from is not None), s.rot.dims if s.rot else 0
+            if layer.latent is not None:
+                a, s = layer.latent, layer.latent.spec
+                L.ah, L.adim, L.avdim, L.arank, L.rot, L.ascale = s.heads, s.dim, s.vdim, s.rank, s.rot_dim, s.scale
+                L.head_gate, L.anorm = int(s.head_gate), _p(a.norm)
+                L.a_uk_t, L.a_uv, L.a_expand = _p(a.w.uk_t), _p(a.w.uv), _p(a.w.expand)
+            if layer.recurrence is not None:
+                a, s = layer.recurrence.w, layer.recurrence.spec
+                L.rc, L.rk, L.rb = s.width, s.taps, s.blocks
+                L.conv_w, L.conv_b, L.gates, L.gates_by_block = _p(a.conv), _p(a.conv_b), _p(a.gates), _p(a.gates_by_block)
+                L.gates_b, L.rate = _p(a.gates_b), _p(a.rate)
             if layer.linear is not None:
                 a, s = layer.linear, layer.linear.spec
                 L.lh, L.ld, L.ldv, L.rd = s.heads, s.dim, s.vdim, s.rot_dims
@@ -397,16 +423,20 @@ class MixerExecutor:
                 L.decay, L.norm_w = _p(a.decay), _p(a.norm)
         m = self._m = _MixerModel()
         m.hidden, m.eps = model.cfg.hidden_size, float(model.cfg.rms_norm_eps)
-        m.center = int(model.cfg.norm_type == "layernorm")
+        m.center, m.streams = int(model.cfg.norm_type == "layernorm"), model.cfg.streams
+        m.expand_bytes = cuda_latent.EXPAND_BYTES
         ws = self._ws = kcuda.workspace(model.device)
         m.gemm_ws, m.gemm_ws_floats = _p(ws.gemm_ws), ws.gemm_ws.numel()
         m.gemm_counters, m.n_counters = _p(ws.gemm_counters), ws.gemm_counters.numel()
         m.layers = ctypes.cast(self._layers, P)
-        self.cap, self._bufs, self._chunk = 0, [], None
+        self.cap, self._bufs, self._chunk, self._latent = 0, [], None, None
+        self._rec_width = max(x.rc for x in self._layers)
         self._key = self._tables = None
         self._step = _MixerStep()
         self._fn = kcuda.lib().ksana_mixer_forward
         self._fn.argtypes, self._fn.restype = [P, P, P, P, I, I, P, P, P, P], I
+        self._lat_fn = kcuda.lib().ksana_mixer_latent_bytes
+        self._lat_fn.argtypes, self._lat_fn.restype = [P, P, I], LL
         self._out, self._fail, self._launches = P(), I(), I()
 
     def _ensure(self, T: int) -> None:
@@ -437,7 +467,8 @@ class MixerExecutor:
 
     def _bind(self, caches) -> None:
         # the position tables grow with the longest sequence an engine asks for: they are part of the key
-        tables = [(layer.attn.bias if layer.attn else None, layer.linear.rotary() if layer.linear else None)
+        tables = [(layer.attn.bias if layer.attn else None,
+                   next((x.rotary() for x in (layer.linear, layer.attn, layer.latent) if x and x.rotary() is not None), None))
                   for layer in self.model.layers]
         key = tuple((c.kv.data_ptr(), c.kv.shape, c.state.data_ptr(), _p(b), _p(r)) for c, (b, r) in zip(caches, tables))
         if key == self._key:
@@ -446,11 +477,17 @@ class MixerExecutor:
         m.block_size = 1
         for L, c, layer, (bias, rotary) in zip(self._layers, caches, self.model.layers, tables):
             L.kv, L.state, L.bias, L.rotary = _p(c.kv), _p(c.state), _p(bias), _p(rotary)
+            L.rot_table = L.rotary if L.rot else None
             L.bias_len = bias.shape[1] if bias is not None else 0
             m.num_blocks = c.kv.shape[0]
-            if layer.attn is not None:
+            if layer.kv_width():
                 m.block_size = c.kv.shape[1] // layer.kv_width()
         self._key, self._tables = key, tables
+
+    def _chunk_floats(self, need: int) -> None:
+        if need > self._m.chunk_floats:
+            self._chunk = torch.empty(need, dtype=torch.float32, device=self.model.device)
+            self._m.chunk_buf, self._m.chunk_floats = _p(self._chunk), need
 
     def can_run(self, meta, caches, n_layers: int) -> bool:
         return meta.total_tokens > 0 and (meta.state_slots is not None or not self.model.cfg.has_state)
@@ -471,13 +508,18 @@ class MixerExecutor:
         s.max_q_prefill = int((cu[1:n_pre + 1] - cu[:n_pre]).max()) if n_pre else 0
         s.max_kv_decode = int(meta.kv_lens_host[n_pre:].max()) if n_dec else 0
         s.one_token = int(T - s.prefill_tokens == n_dec)
-        s.num_long = long_portions(meta) if self.model.cfg.has_state else 0
+        s.num_long = long_portions(meta) if any(x.lh for x in self._layers) else 0
         s.long_tokens = int(cu[s.num_long])
         if s.num_long:
-            need = max((s.long_tokens // 128 + s.num_long) * x.lh * x.ld * x.ldv for x in self._layers)
-            if need > m.chunk_floats:
-                self._chunk = torch.empty(need, dtype=torch.float32, device=self.model.device)
-                m.chunk_buf, m.chunk_floats = _p(self._chunk), need
+            self._chunk_floats(max((s.long_tokens // 128 + s.num_long) * x.lh * x.ld * x.ldv for x in self._layers))
+        if self._rec_width:  # chunks of prompts, or the gates' products where the general kernels run
+            self._chunk_floats(max(T * self._rec_width * 5 // 2 + 4, kcuda.lib().ksana_recurrence_scratch(
+                s.prefill_tokens, n_pre, s.max_q_prefill, self._rec_width)))
+        s.cu_q_host, s.kv_lens_host = cu.ctypes.data, meta.kv_lens_host.ctypes.data
+        need = self._lat_fn(ctypes.byref(m), ctypes.byref(s), n_layers)
+        if need > m.lat_bytes:
+            self._latent = torch.empty(need, dtype=torch.uint8, device=self.model.device)
+            m.lat_buf, m.lat_bytes = _p(self._latent), need
         rc = self._fn(ctypes.byref(m), ctypes.byref(s), h.data_ptr(), residual.data_ptr(), 0, n_layers,
                       ctypes.byref(self._out), ctypes.byref(self._fail), ctypes.byref(self._launches),
                       torch.cuda.current_stream().cuda_stream)

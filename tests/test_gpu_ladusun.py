@@ -126,6 +126,25 @@ def test_long_decode(cases, dtype):
         R.run_long_decode(cases[dtype][name], cases[dtype][name].engine(dtype, 320, "cuda"), tolerance(dtype, name))
 
 
+@pytest.mark.parametrize("name", ["even", "wide"])
+def test_layer_path_and_native_executor_agree(cases, name, monkeypatch):
+    """One call per step and one call per kernel launch the same kernels."""
+    case = cases[BF16][name]
+    toks = [case.tokens(n, n) for n in (140, 20, 33, 1)]
+
+    def run():
+        eng = case.engine(BF16, 512, "cuda")
+        a = eng.replay([(i, t[:-1] or t, [0]) for i, t in enumerate(toks)], [2, 3])
+        b = eng.replay([(i, t[-1:], [0]) for i, t in enumerate(toks[:2])] + [(9, toks[2], [32])])
+        return torch.cat((a, b)), eng.model
+    native, m1 = run()
+    assert type(m1._native).__name__ == "MixerExecutor"
+    monkeypatch.setenv("KSANA_DISABLE_NATIVE_EXECUTOR", "1")
+    layers, m2 = run()
+    assert m2._native is None
+    assert torch.equal(native, layers)
+
+
 @pytest.mark.parametrize("bs", [dict(), dict(split_fuse_token_num=9), dict(enable_async=True)])
 def test_greedy_generation(cases, bs):
     greedy_check(cases[F32]["odd"], serve(cases[F32]["odd"], device="cuda", **bs), [1, 2, 30, 17, 41, 8], 6)
