@@ -11,11 +11,16 @@ each case is small (at most a few GB on the device) and launches its kernel a ha
     python benchmarks/kernel_cases.py mla [B ctx h q_len]     # tcgen05 absorbed-MLA decode over the latent cache
     python benchmarks/kernel_cases.py rmsnorm [T H]
     python benchmarks/kernel_cases.py moe [T E k H I]
-    python benchmarks/kernel_cases.py window_prefill [T h hk d dv window keep shared]   # layers with mixers of their own sizes
-    python benchmarks/kernel_cases.py window_decode [B ctx h hk d dv window keep shared]
+    python benchmarks/kernel_cases.py window_prefill [T h hk d dv window keep shared cap]   # layers with mixers of their own sizes
+    python benchmarks/kernel_cases.py window_decode [B ctx h hk d dv window keep shared cap]
     python benchmarks/kernel_cases.py linear_prefill [T h d dv rotary]
     python benchmarks/kernel_cases.py linear_decode [B h d dv rotary]
     python benchmarks/kernel_cases.py mixer_rows [T H h hk d]
+    python benchmarks/kernel_cases.py latent_prefill [T h dim rot vdim rank]
+    python benchmarks/kernel_cases.py latent_decode [B ctx h dim rot vdim rank]
+    python benchmarks/kernel_cases.py recurrence_prefill [T C blocks taps sequences]
+    python benchmarks/kernel_cases.py recurrence_decode [B C blocks taps]
+    python benchmarks/kernel_cases.py ladusun_rows [T H streams h hk d rank rot]
     python benchmarks/kernel_cases.py all
 """
 import json
@@ -26,7 +31,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 from ksanallm_b200.engine.step_input import make_step_input  # noqa: E402
-from ksanallm_b200.ops import cuda, cuda_mixer, cuda_moe  # noqa: E402
+from ksanallm_b200.ops import cuda, cuda_latent, cuda_mixer, cuda_moe, cuda_recurrence  # noqa: E402
 from ksanallm_b200.ops import reference as ref  # noqa: E402
 
 DEV = "cuda"
@@ -52,6 +57,18 @@ def timeit(fn, iters=10, warm=3):
     e1.record()
     torch.cuda.synchronize()
     return e0.elapsed_time(e1) / iters * 1e3  # us
+
+
+def timeit_graph(fn, count=48):
+    """For kernels shorter than their launch from Python: ``count`` launches in one CUDA graph."""
+    for i in range(count):
+        fn(i)
+    torch.cuda.synchronize()
+    graph = torch.cuda.CUDAGraph()
+    with torch.cuda.graph(graph):
+        for i in range(count):
+            fn(i)
+    return timeit(lambda i: graph.replay(), iters=5) / count
 
 
 def args_or(default):
@@ -195,34 +212,36 @@ def case_moe():
                 tflops=round(fl / us / 1e6, 1), frac_of_measured_bf16=round(fl / us / 1e6 / p["bf16_tflops"], 3))
 
 
-def _window_setup(q_lens, kv_lens, h, hk, d, dv, window, prefill, keep=0, shared=0):
+def _window_setup(q_lens, kv_lens, h, hk, d, dv, window, prefill, keep=0, shared=0, cap=0):
     q, _, bt, cu = _attn_setup(q_lens, kv_lens, h, 1)
     q = (torch.randn(cu[-1], h, d, device=DEV) * 0.3).to(torch.bfloat16)
     cache = (torch.randn(int(bt.max()) + 2, hk * 16 * (d + (0 if shared else dv)), device=DEV) * 0.3).to(torch.bfloat16)
     T = cu[-1]
     meta = make_step_input([0] * T, [0] * T, [0] * T, cu, kv_lens, bt, num_prefill=prefill, device=DEV)
-    bias = None if shared else torch.randn(h, max(kv_lens) if keep else window or max(kv_lens), device=DEV)
+    bias = None if shared or cap else torch.randn(h, max(kv_lens) if keep else window or max(kv_lens), device=DEV)
     out = torch.empty(T, h * dv, dtype=torch.bfloat16, device=DEV)
-    return lambda i: cuda_mixer.window_attention(q, cache, meta, 16, hk, dv, d ** -0.5, window, bias, 1.0, out, keep)
+    gate = torch.randn(T, (h + 7) // 8 * 8, device=DEV).to(torch.bfloat16)[:, :h] if cap else None
+    return lambda i: cuda_mixer.window_attention(q, cache, meta, 16, hk, dv, d ** -0.5, window, bias, 1.0, out, keep,
+                                                 float(cap), bool(cap), gate)
 
 
 def case_window_prefill():
-    T, h, hk, d, dv, window, keep, shared = args_or([8192, 32, 8, 128, 128, 1024, 0, 0])
-    us = timeit(_window_setup([T], [T], h, hk, d, dv, window, 1, keep, shared), iters=5)
+    T, h, hk, d, dv, window, keep, shared, cap = args_or([8192, 32, 8, 128, 128, 1024, 0, 0, 0])
+    us = timeit(_window_setup([T], [T], h, hk, d, dv, window, 1, keep, shared, cap), iters=5)
     w = min(window or T, T)
     pairs = w * (w + 1) / 2 + (T - w) * w
     fl = 2.0 * h * (d + dv) * pairs
     p = peaks()
-    return dict(kernel="window_prefill", T=T, h=h, hk=hk, d=d, dv=dv, window=window, keep=keep, shared=shared, us=round(us, 1),
+    return dict(kernel="window_prefill", T=T, h=h, hk=hk, d=d, dv=dv, window=window, keep=keep, shared=shared, cap=cap, us=round(us, 1),
                 tflops=round(fl / us / 1e6, 1), frac_of_measured_bf16=round(fl / us / 1e6 / p["bf16_tflops"], 3))
 
 
 def case_window_decode():
-    B, ctx, h, hk, d, dv, window, keep, shared = args_or([128, 4096, 32, 8, 128, 128, 1024, 0, 0])
-    us = timeit(_window_setup([1] * B, [ctx] * B, h, hk, d, dv, window, 0, keep, shared))
+    B, ctx, h, hk, d, dv, window, keep, shared, cap = args_or([128, 4096, 32, 8, 128, 128, 1024, 0, 0, 0])
+    us = timeit(_window_setup([1] * B, [ctx] * B, h, hk, d, dv, window, 0, keep, shared, cap))
     by = B * min(window + keep if window else ctx, ctx) * hk * (d + (0 if shared else dv)) * 2
     p = peaks()
-    return dict(kernel="window_decode", B=B, ctx=ctx, h=h, hk=hk, d=d, dv=dv, window=window, keep=keep, shared=shared, us=round(us, 1),
+    return dict(kernel="window_decode", B=B, ctx=ctx, h=h, hk=hk, d=d, dv=dv, window=window, keep=keep, shared=shared, cap=cap, us=round(us, 1),
                 kv_gb=round(by / 1e9, 3), gbs=round(by / us / 1e3, 1),
                 frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
 
@@ -268,6 +287,156 @@ def case_linear_decode():
     return dict(kernel="linear_recurrent", B=B, h=h, d=d, dv=dv, rotary=rotary, us=round(us, 1),
                 state_gb=round(by / 2e9, 3), gbs=round(by / us / 1e3, 1),
                 frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+
+
+def _latent_setup(q_lens, kv_lens, h, dim, rot, vdim, rank, prefill):
+    """The operator's inputs, and what its kernels get in between."""
+    from ksanallm_b200.models.mixers import LatentWeights
+    _, _, bt, cu = _attn_setup(q_lens, kv_lens, 1, 1)
+    T = cu[-1]
+    bf = lambda *s: (torch.randn(*s, device=DEV) * 0.3).to(torch.bfloat16)  # noqa: E731
+    cache = bf(int(bt.max()) + 2, 16 * (rank + rot))
+    pos = [n - q + i for n, q in zip(kv_lens, q_lens) for i in range(q)]
+    slots = [int(bt[b, p // 16]) * 16 + p % 16 for b, (n, q) in enumerate(zip(kv_lens, q_lens)) for p in range(n - q, n)]
+    meta = make_step_input([0] * T, pos, slots, cu, kv_lens, bt, num_prefill=prefill, device=DEV)
+    x = bf(T, (h * (dim + rot) + rank + rot + h + 7) // 8 * 8)
+    nq, na = h * (dim + rot), rank + rot
+    w = LatentWeights(bf(h, dim, rank), bf(h, vdim, rank))
+    out, norm, table = bf(T, h * vdim), torch.ones(rank, device=DEV), ref.rotary_table(rot, 1e4, max(kv_lens), DEV)
+    return x[:, :nq].unflatten(1, (h, dim + rot)), x[:, nq:nq + na], x[:, nq + na:nq + na + h], w, cache, meta, out, norm, table
+
+
+def case_latent_prefill():
+    """The attention kernel alone, and the whole operator: append, gather, keys and values per head, attention."""
+    T, h, dim, rot, vdim, rank = args_or([8192, 32, 128, 64, 128, 512])
+    q, a, gate, w, cache, meta, out, norm, table = _latent_setup([T], [T], h, dim, rot, vdim, rank, 1)
+    lat = (torch.randn(T, rank + rot, device=DEV) * 0.3).to(torch.bfloat16)
+    kv = cuda.gemm_bf16(lat[:, :rank], w.expand)
+    st = torch.cuda.current_stream().cuda_stream
+
+    def kernel(i):
+        assert cuda.lib().ksana_latent_prefill(
+            q.data_ptr(), q.stride(0), T, kv.data_ptr(), kv.stride(0), lat.data_ptr() + 2 * rank, rank + rot, T,
+            meta.cu_q.data_ptr(), meta.kv_lens.data_ptr(), h, dim, rot, vdim, 0.07, gate.data_ptr(), gate.stride(0),
+            out.data_ptr(), out.stride(0), 0, 1, T, st) == 0
+    us = timeit(kernel, iters=5)
+    op = timeit(lambda i: cuda_latent.latent_attention(q, a, norm, 1e-6, table, cache, meta, 16, w, 0.07, gate, out), iters=5)
+    gather = timeit(lambda i: cuda.lib().ksana_latent_gather(cache.data_ptr(), meta.block_tables.data_ptr(), meta.max_blocks,
+                                                             meta.kv_lens.data_ptr(), 0, 1, T, 16, rank + rot, lat.data_ptr(), st))
+    fl, p = 2.0 * h * (dim + rot + vdim) * T * (T + 1) / 2, peaks()
+    return dict(kernel="latent_prefill", T=T, h=h, dim=dim, rot=rot, vdim=vdim, rank=rank, us=round(us, 1),
+                tflops=round(fl / us / 1e6, 1), frac_of_measured_bf16=round(fl / us / 1e6 / p["bf16_tflops"], 3),
+                operator_us=round(op, 1), gather_us=round(gather, 1),
+                gather_frac_of_measured_hbm=round(T * (rank + rot) * 4 / gather / 1e3 / p["hbm_gbs"], 3))
+
+
+def case_latent_decode():
+    B, ctx, h, dim, rot, vdim, rank = args_or([64, 4096, 32, 128, 64, 128, 512])
+    q, a, gate, w, cache, meta, out, norm, table = _latent_setup([1] * B, [ctx] * B, h, dim, rot, vdim, rank, 0)
+    qc = (torch.randn(B, h * (rank + rot), device=DEV) * 0.3).to(torch.bfloat16)
+    o = torch.empty(B, h * rank, dtype=torch.bfloat16, device=DEV)
+    st = torch.cuda.current_stream().cuda_stream
+
+    def kernel(i):
+        assert cuda.lib().ksana_window_decode(
+            qc.data_ptr(), qc.stride(0), cache.data_ptr(), cache.shape[0], meta.block_tables.data_ptr(), meta.max_blocks,
+            meta.cu_q.data_ptr(), meta.kv_lens.data_ptr(), h, 1, rank + rot, rank, 16, 0, 0, 1, 0.07, None, 0, 1.0, 0.0, 0,
+            gate.data_ptr(), gate.stride(0), o.data_ptr(), o.stride(0), 0, B, ctx, st) == 0
+    us = timeit(kernel)
+    op = timeit(lambda i: cuda_latent.latent_attention(q, a, norm, 1e-6, table, cache, meta, 16, w, 0.07, gate, out))
+    by, p = B * ctx * (rank + rot) * 2, peaks()
+    return dict(kernel="latent_decode", B=B, ctx=ctx, h=h, rank=rank, rot=rot, us=round(us, 1), kv_gb=round(by / 1e9, 3),
+                gbs=round(by / us / 1e3, 1), frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3),
+                tflops=round(2.0 * B * h * ctx * (2 * rank + rot) / us / 1e6, 1), operator_us=round(op, 1))
+
+
+def _recurrence_setup(lens, q_lens, C, blocks, K, prefill, copies=2):
+    from ksanallm_b200.models.mixers import RecurrenceWeights
+    B, T = len(lens), sum(q_lens)
+    cu = [0]
+    for q in q_lens:
+        cu.append(cu[-1] + q)
+    meta = make_step_input([0] * T, [0] * T, [0] * T, cu, lens, torch.zeros(B, 1), num_prefill=prefill, device=DEV,
+                           state_slots=list(range(B)))
+    s, r = C // blocks, lambda *a: torch.randn(*a, device=DEV) * 0.3  # noqa: E731
+    w = RecurrenceWeights({"p.conv": r(C, K), "p.conv_b": r(C), "p.gates": r(2, blocks, s, s).to(torch.bfloat16),
+                           "p.gates_b": r(2, C), "p.lam": r(C) - 3}, "p", 8.0)
+    xs = [r(T, 2 * C).to(torch.bfloat16) for _ in range(copies)]
+    states = [torch.zeros(B, 1, K, C, device=DEV) for _ in range(copies)]
+    out = torch.empty(T, C, dtype=torch.bfloat16, device=DEV)
+    return lambda i: cuda_recurrence.gated_recurrence(xs[i % copies][:, :C], xs[i % copies][:, C:], states[i % copies], meta, w, out)
+
+
+def case_recurrence_prefill():
+    T, C, blocks, K, n = args_or([8192, 4096, 32, 4, 1])
+    us = timeit(_recurrence_setup([T // n] * n, [T // n] * n, C, blocks, K, n), iters=5)
+    by, fl, p = T * C * 6, 4.0 * T * C * (C // blocks), peaks()
+    floor = max(by / p["hbm_gbs"] / 1e3, fl / p["bf16_tflops"] / 1e6)
+    return dict(kernel="recurrence_prompts", T=T, C=C, blocks=blocks, K=K, sequences=n, us=round(us, 1),
+                roofline_us=round(floor, 1), frac_of_roofline=round(floor / us, 3))
+
+
+def case_recurrence_decode():
+    B, C, blocks, K = args_or([128, 4096, 32, 4])
+    # enough layers' states and inputs that L2 holds none of them
+    us = timeit_graph(_recurrence_setup([100] * B, [1] * B, C, blocks, K, 0, 24))
+    by, p = B * C * (8 * K + 6) + 4 * C * (C // blocks), peaks()
+    return dict(kernel="recurrence_step", B=B, C=C, blocks=blocks, K=K, us=round(us, 1), mb=round(by / 1e6, 1),
+                gbs=round(by / us / 1e3, 1), frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+
+
+def case_ladusun_rows():
+    """Row-wise kernels of hyper-connected streams, latent attention and clamped experts."""
+    T, H, S, h, hk, d, rank, rot = args_or([8192, 4096, 4, 32, 8, 128, 512, 64])
+    bf = lambda *s: torch.randn(*s, device=DEV).to(torch.bfloat16)  # noqa: E731
+    f32 = lambda *s: torch.randn(*s, device=DEV)  # noqa: E731
+    p, out, st = peaks(), {}, torch.cuda.current_stream().cuda_stream
+
+    def add(name, us, by):
+        out[name] = dict(us=round(us, 1), gbs=round(by / us / 1e3, 1), frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+    xs, streams, w = [bf(T, H) for _ in range(2)], [f32(T, S, H) for _ in range(2)], bf(H)
+    mix, ow, iw, ls = torch.eye(S, device=DEV), f32(S), f32(S) / S, torch.ones(H, device=DEV)
+    add("hyper_norm", timeit(lambda i: cuda_mixer.hyper_norm(xs[i % 2], ls, None, streams[i % 2], mix, ow, streams[i % 2], iw, w,
+                                                             1e-6, torch.bfloat16)), T * H * (8 * S + 4))
+    k = 2
+    y2, pos, wts = bf(T * k, H), torch.randperm(T * k, dtype=torch.int32, device=DEV), torch.rand(T, k, device=DEV)
+    add("hyper_norm_routed", timeit(lambda i: cuda_mixer.hyper_norm(None, ls, (y2, pos, wts), streams[i % 2], mix, ow, streams[i % 2],
+                                                                    iw, w, 1e-6, torch.bfloat16)), T * H * (8 * S + 2 + 2 * k))
+    add("rms_norm", timeit(lambda i: cuda.rms_norm(xs[i % 2], w, 1e-6, xs[1 - i % 2])), T * H * 8)
+    us = [bf(T, 6 * H) for _ in range(2)]
+    add("clamped_gate_mul", timeit(lambda i: cuda_mixer.clamped_gate_mul(us[i % 2], 7.0, 1.702)), T * H * 18)
+    add("silu_mul", timeit(lambda i: cuda.silu_and_mul(us[i % 2])), T * H * 18)
+    add("relu2", timeit(lambda i: cuda_mixer.relu2(us[i % 2])), T * H * 24)
+    slots, table = torch.arange(T, dtype=torch.int32, device=DEV), torch.randn(T, d, device=DEV)
+    cache = torch.zeros((T + 15) // 16, hk * 16 * 2 * d, dtype=torch.bfloat16, device=DEV)
+    qkv = [bf(T, (h + 2 * hk) * d) for _ in range(3)]
+
+    def parts(x):
+        return x[:, :h * d].unflatten(1, (h, d)), x[:, h * d:(h + hk) * d].unflatten(1, (hk, d)), x[:, (h + hk) * d:].unflatten(1, (hk, d))
+    by = T * d * 2 * (2 * h + 4 * hk)
+    add("rotate_cache", timeit(lambda i: cuda_mixer.qk_norm_cache(*parts(qkv[i % 3]), slots, cache, 16, None, None, 1e-6, slots, table)), by)
+    add("rope_cache", timeit(lambda i: cuda.rope_qknorm_cache(*parts(qkv[i % 3]), slots, table, slots, cache.view(-1, 2, hk, 16, d))), by)
+    lat, lt = torch.zeros((T + 15) // 16, 16 * (rank + rot), dtype=torch.bfloat16, device=DEV), torch.randn(T, rot, device=DEV)
+    ql = [bf(T, h * (d + rot) + rank + rot) for _ in range(2)]
+    nq, nw = h * (d + rot), torch.ones(rank, device=DEV)
+
+    def append(i):
+        x = ql[i % 2]
+        assert cuda.lib().ksana_latent_append(x.data_ptr(), x.stride(0), d, None, 0, x.data_ptr() + 2 * nq, x.stride(0), nw.data_ptr(),
+                                              1e-6, slots.data_ptr(), lt.data_ptr(), slots.data_ptr(), lat.data_ptr(), T, h, rank, rot, 1, st) == 0
+    add("latent_append", timeit(append), T * 4 * (h * rot + rank + rot))
+    q, qc = bf(T, h, d + rot), bf(T, h, rank + rot)
+    kr, lt2 = bf(T, rot), bf(T, rank)
+
+    def mla_append(i):
+        assert cuda.lib().ksana_mla_rope_append(q.data_ptr(), q.stride(0), q.stride(1), d, qc.data_ptr(), kr.data_ptr(), rot, lt2.data_ptr(),
+                                                rank, slots.data_ptr(), lt.data_ptr(), slots.data_ptr(), lat.data_ptr(), rank + rot, T, h, rank, rot,
+                                                1, st) == 0
+    add("mla_rope_append", timeit(mla_append), T * 4 * (h * rot + rank + rot))
+    z = torch.randn(T, 16, device=DEV)
+    add("moe_topk_groups", timeit(lambda i: cuda_moe.moe_topk(z, 16, 2, None, 4, 2)), T * (16 + 4) * 4)
+    add("moe_route", timeit(lambda i: cuda_moe.moe_route(z, 2, "softmax", True, 4, 2)), T * (16 + 4) * 4)
+    return dict(kernel="ladusun_rows", T=T, H=H, streams=S, **out)
 
 
 def case_mixer_rows():
@@ -331,7 +500,9 @@ def case_mixer_rows():
 
 CASES = dict(gemm=case_gemm, gemm_fp8=case_gemm_fp8, gemm_int4=case_gemm_int4, decode=case_decode, prefill=case_prefill, mla=case_mla, rmsnorm=case_rmsnorm,
              moe=case_moe, window_prefill=case_window_prefill, window_decode=case_window_decode,
-             linear_prefill=case_linear_prefill, linear_decode=case_linear_decode, mixer_rows=case_mixer_rows)
+             linear_prefill=case_linear_prefill, linear_decode=case_linear_decode, mixer_rows=case_mixer_rows,
+             latent_prefill=case_latent_prefill, latent_decode=case_latent_decode, recurrence_prefill=case_recurrence_prefill,
+             recurrence_decode=case_recurrence_decode, ladusun_rows=case_ladusun_rows)
 
 if __name__ == "__main__":
     which = sys.argv[1] if len(sys.argv) > 1 else "all"
