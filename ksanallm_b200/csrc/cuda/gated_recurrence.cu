@@ -27,7 +27,7 @@ struct RecurrenceArgs {
   const int* slots;
   const int* cu_q;
   const int* kv_lens;
-  const float* conv_w;     // [C, K]
+  const float* conv_w;     // [K, C]
   const float* conv_b;
   const float* gates_b;    // [2, C]
   const float* rate;       // [C]
@@ -55,7 +55,7 @@ recurrence_conv_kernel(RecurrenceArgs a, const int* __restrict__ seq_of_token, T
       v = to_f(x[static_cast<size_t>(q0 + back) * a.ldx + c]);
     else if (!fresh)
       v = mem[static_cast<size_t>(a.K + back) * a.C + c];
-    s = fmaf(a.conv_w[static_cast<size_t>(c) * a.K + j], v, s);
+    s = fmaf(a.conv_w[static_cast<size_t>(j) * a.C + c], v, s);
   }
   u[static_cast<size_t>(t - tok_base) * a.C + c] = from_f<T>(s);
 }
@@ -99,15 +99,15 @@ recurrence_scan_kernel(RecurrenceArgs a, const T* __restrict__ u, const float* _
 }
 
 // ---- bf16 on the tensor cores ---------------------------------------------------------------------------------------
-// One CTA = 128 output channels of one block x TC columns, 128 threads. A column is a token of one chunk of a prompt, or
-// (STEP) the single new token of one sequence.
+// One CTA = 128 output channels of one block x TC columns, 256 threads. A column is a token of a prompt, or (STEP) the
+// single new token of one sequence.
 //   convolution   u of the block's channels -> shared memory, bf16, K-major with 128-byte swizzle
 //   products      Z_r = W_r u^T and Z_i = W_i u^T: 128 x TC x s, the channels on the MMA rows -> TMEM
-//   gates         thread m owns channel m (TMEM lane m) and walks along its columns
-// so the recurrence over a chunk is a loop in registers. Prompts: every chunk of 128 tokens runs on its own from S = 0 and
-// leaves S and the running sum of log a per token; recurrence_carry_kernel takes the states from chunk to chunk and
-// recurrence_finish_kernel adds each chunk's entering state, S_t + exp(sum log a) S_in, and multiplies by the other
-// branch. STEP: the state is read, advanced and written here.
+//   gates         thread (g, m) owns channel m (TMEM lane m) and walks along half g of the columns
+// so the recurrence over a chunk (half a tile) is a loop in registers. Prompts: every chunk of 64 tokens runs on its own
+// from S = 0 and leaves S and the running sum of log2 a per token; recurrence_carry_kernel takes the states from chunk to
+// chunk and recurrence_finish_kernel adds each chunk's entering state, S_t + 2^(sum log2 a) S_in, and multiplies by the
+// other branch. STEP: the state is read, advanced and written here.
 constexpr int RG_MAX_PART = 256;  // channels of a block
 
 template <int TC>
@@ -117,24 +117,47 @@ struct RecurrenceSmem {
   __host__ __device__ static int total(int kc) { return kc * (U_BYTES + 2 * W_BYTES) + 256 + 1024; }
 };
 
-// log a <= 0 -> a and sqrt(1 - a^2), relative error about 1e-6 (the gates were computed from 16-bit numbers)
-__device__ __forceinline__ void decay_fast(float la, float* a, float* in) {
-  const float e = __expf(la), x = 2.f * la;
-  const float small = -x * fmaf(x, fmaf(x, fmaf(x, fmaf(x, fmaf(x, 1.f / 720.f, 1.f / 120.f), 1.f / 24.f), 1.f / 6.f), 0.5f), 1.f);
-  const float w = fmaxf(x > -0.3f ? small : fmaf(-e, e, 1.f), 1e-37f);
-  *a = e;
-  *in = x == 0.f ? 0.f : w * rsqrtf(w);
+// Hardware approximations (relative error about 1e-7) without the handling of denormal numbers around them.
+__device__ __forceinline__ float ex2_ftz(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
 }
-__device__ __forceinline__ float sigmoid_fast(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
+__device__ __forceinline__ float rcp_ftz(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+__device__ __forceinline__ float rsqrt_ftz(float x) {
+  float r;
+  asm("rsqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+constexpr float LOG2E = 1.4426950408889634f;
+// 1 / (1 + 2^x): the sigmoid of -x ln 2
+__device__ __forceinline__ float sigmoid_log2(float x) { return rcp_ftz(1.f + ex2_ftz(x)); }
+// l = log2 a <= 0 -> a and sqrt(1 - a^2). 1 - a^2 = -expm1(2 l ln 2) is a power series where the difference would cancel.
+__device__ __forceinline__ void decay_fast(float l, float* a, float* in) {
+  const float e = ex2_ftz(l);
+  constexpr float c = 1.3862943611198906f;  // 2 ln 2
+  const float small = -l * fmaf(l, fmaf(l, fmaf(l, c * c * c * c / 24.f, c * c * c / 6.f), c * c / 2.f), c);
+  const float w = fmaxf(l > -0.05f ? small : fmaf(-e, e, 1.f), 1e-30f);
+  *a = e;
+  *in = w * rsqrt_ftz(w);
+}
 
 template <int TC, int KT, bool STEP>
-__global__ void __launch_bounds__(128)
+__global__ void __launch_bounds__(256)
 recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a, int seq_base, int num_seqs,
                        float* __restrict__ local, float* __restrict__ decay, int tok_base, unsigned int* err) {
   using L_ = RecurrenceSmem<TC>;
   const int part = a.C / a.B, groups = (part + 127) / 128;
   const int blk = blockIdx.y / groups, m0 = blockIdx.y % groups * 128;
   const int tid = threadIdx.x, warp = tid >> 5;
+  constexpr int HALF = TC / 2;  // columns per thread
+  const int m = m0 + (tid & 127), half0 = (tid >> 7) * HALF;
+  const bool mine = m < part;
+  const int ch = blk * part + (mine ? m : 0);
   // columns: tokens [q0 + i0, + n) of one sequence, or sequences [first, + n)
   int b = 0, q0 = 0, i0 = 0, n;
   bool fresh = false;
@@ -175,10 +198,25 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
     tmem_relinquish();
   }
 
+  // STEP: what the gates will meet is under way while the products are made
+  [[maybe_unused]] float old[STEP ? HALF : 1], yy[STEP ? HALF : 1];
+  [[maybe_unused]] float* mem_at[STEP ? HALF : 1];
+  [[maybe_unused]] int row_at[STEP ? HALF : 1];
+  if constexpr (STEP) {
+#pragma unroll
+    for (int j = 0; j < HALF; ++j) {
+      const int sb = i0 + min(half0 + j, n - 1);
+      row_at[j] = a.cu_q[sb];
+      mem_at[j] = a.state + static_cast<size_t>(a.slots[sb]) * a.K * a.C + ch;
+      old[j] = a.kv_lens[sb] == 1 ? 0.f : *mem_at[j];
+      yy[j] = __bfloat162float(static_cast<const __nv_bfloat16*>(a.y)[static_cast<size_t>(row_at[j]) * a.ldy + ch]);
+    }
+  }
+
   // ---- u -> shared memory
   const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(a.x) + blk * part;
   const int vecs = part / 8, strips = STEP ? TC : TC / 16;
-  for (int w = tid; w < kc * 8 * strips; w += 128) {
+  for (int w = tid; w < kc * 8 * strips; w += 256) {
     const int v = w % (kc * 8), strip = w / (kc * 8), c = v * 8;
     uint8_t* dst = sU + (v >> 3) * L_::U_BYTES;
     auto put = [&](int r, const float* f) {
@@ -195,10 +233,14 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
     float taps[KT][8], bias[8], win[KT][8];  // taps[KT - 1] meets the newest input
     load_n<8>(a.conv_b + ch, bias);
 #pragma unroll
-    for (int j = 0; j < KT; ++j)
+    for (int j = 0; j < KT; ++j) {
+      if (j >= KT - a.K) {
+        load_n<8>(a.conv_w + static_cast<size_t>(j - (KT - a.K)) * a.C + ch, taps[j]);
+      } else {
 #pragma unroll
-      for (int e = 0; e < 8; ++e)
-        taps[j][e] = j >= KT - a.K ? a.conv_w[static_cast<size_t>(ch + e) * a.K + j - (KT - a.K)] : 0.f;
+        for (int e = 0; e < 8; ++e) taps[j][e] = 0.f;
+      }
+    }
     if constexpr (STEP) {
       const int sb = i0 + strip, t = a.cu_q[sb];
       const bool first = a.kv_lens[sb] == 1;
@@ -221,7 +263,7 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
         for (int j = 0; j < KT; ++j) f[e] = fmaf(taps[j][e], win[j][e], f[e]);
       }
       put(strip, f);
-      if (m0 == 0) {  // a block of one CTA column: nobody else reads these rows
+      if (groups == 1) {  // else other CTAs read these rows: recurrence_shift_kernel moves them afterwards
 #pragma unroll
         for (int j = 0; j < KT - 1; ++j) {
           const int row = a.K - (KT - 1) + j;
@@ -243,6 +285,7 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
       const int r0 = strip * 16;
 #pragma unroll
       for (int j = 0; j < KT - 1; ++j) input(i0 + r0 - (KT - 1) + j, win[j + 1]);
+#pragma unroll KT
       for (int r = 0; r < 16; ++r) {
         if (r0 + r >= n) {
           put(r0 + r, zero);
@@ -286,60 +329,63 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
   ok = mbar_wait_bounded(z_done, 0, abort_flag, err);
   if (__all_sync(0xffffffffu, ok)) {
     tc_fence_after();
-    const int m = m0 + tid;
-    const bool mine = m < part;
-    const int ch = blk * part + (mine ? m : 0);
-    const float rate = a.rate[ch], br = a.gates_b[ch], bi = a.gates_b[a.C + ch];
-    const uint32_t lane_off = static_cast<uint32_t>(warp * 32) << 16;
+    const float rate2 = -a.rate[ch] * LOG2E, br2 = -a.gates_b[ch] * LOG2E, bi2 = -a.gates_b[a.C + ch] * LOG2E;
+    const uint32_t tm = tmem + (static_cast<uint32_t>((warp & 3) * 32) << 16);
     const uint8_t* u_col = sU + (m >> 6) * L_::U_BYTES + (m & 7) * 2;
     const int u_vec = (m >> 3) & 7;
     float S = 0.f, sum = 0.f;
+    constexpr int N = HALF < 16 ? 8 : 16;
+    static_assert(HALF % N == 0, "a thread's columns come in whole loads");
+    const int end = min(half0 + HALF, n);
+    float* lp = nullptr;
+    float* dp = nullptr;
+    if constexpr (!STEP) {
+      const size_t at = static_cast<size_t>(q0 - tok_base + i0 + half0) * a.C + ch;
+      lp = local + at;
+      dp = decay + at;
+    }
 #pragma unroll 1
-    for (int c0 = 0; c0 < n; c0 += 16) {
-      uint32_t zr[16], zi[16];
-      tmem_ld16(tmem + lane_off + c0, zr);
-      tmem_ld16(tmem + lane_off + TC + c0, zi);
+    for (int c0 = half0; c0 < end; c0 += N) {  // uniform over the warp
+      uint32_t zr[N], zi[N];
+      __syncwarp();
+      if constexpr (N == 8) {
+        tmem_ld8(tm + c0, zr);
+        tmem_ld8(tm + TC + c0, zi);
+      } else {
+        tmem_ld16(tm + c0, zr);
+        tmem_ld16(tm + TC + c0, zi);
+      }
       tmem_wait_ld();
-      float dec[16], in[16], la[16];
+      float dec[N], in[N], l2[N];
 #pragma unroll
-      for (int j = 0; j < 16; ++j) {
+      for (int j = 0; j < N; ++j) {
         const int r = c0 + j;
         const float u = mine ? __bfloat162float(*reinterpret_cast<const __nv_bfloat16*>(u_col + r * 128 + ((u_vec ^ (r & 7)) << 4))) : 0.f;
-        la[j] = -sigmoid_fast(__uint_as_float(zr[j]) + br) * rate;
-        decay_fast(la[j], &dec[j], &in[j]);
-        in[j] *= sigmoid_fast(__uint_as_float(zi[j]) + bi) * u;
+        l2[j] = sigmoid_log2(fmaf(__uint_as_float(zr[j]), -LOG2E, br2)) * rate2;
+        decay_fast(l2[j], &dec[j], &in[j]);
+        in[j] *= sigmoid_log2(fmaf(__uint_as_float(zi[j]), -LOG2E, bi2)) * u;
       }
-      if (!mine) continue;
       if constexpr (STEP) {
-        float old[16], yy[16];
-        float* mem[16];
-        size_t row[16];
 #pragma unroll
-        for (int j = 0; j < 16; ++j) {
-          const int sb = i0 + min(c0 + j, n - 1);
-          row[j] = a.cu_q[sb];
-          mem[j] = a.state + static_cast<size_t>(a.slots[sb]) * a.K * a.C + ch;
-          old[j] = a.kv_lens[sb] == 1 ? 0.f : *mem[j];
-          yy[j] = __bfloat162float(static_cast<const __nv_bfloat16*>(a.y)[row[j] * a.ldy + ch]);
-        }
-#pragma unroll
-        for (int j = 0; j < 16; ++j)
-          if (c0 + j < n) {
+        for (int j = 0; j < N; ++j)
+          if (mine && c0 + j < n) {
             const float s = fmaf(dec[j], old[j], in[j]);
-            *mem[j] = s;
-            static_cast<__nv_bfloat16*>(a.out)[row[j] * a.ldo + ch] =
+            *mem_at[j] = s;
+            static_cast<__nv_bfloat16*>(a.out)[static_cast<size_t>(row_at[j]) * a.ldo + ch] =
                 __float2bfloat16_rn(s * gelu_tanh_as<__nv_bfloat16>(yy[j]));
           }
       } else {
-        const size_t at = static_cast<size_t>(q0 - tok_base + i0 + c0) * a.C + ch;
 #pragma unroll
-        for (int j = 0; j < 16; ++j)
-          if (c0 + j < n) {
-            S = fmaf(dec[j], S, in[j]);
-            sum += la[j];
-            local[at + static_cast<size_t>(j) * a.C] = S;
-            decay[at + static_cast<size_t>(j) * a.C] = sum;
+        for (int j = 0; j < N; ++j) {
+          S = fmaf(dec[j], S, in[j]);
+          sum += l2[j];
+          if (mine && c0 + j < n) {
+            *lp = S;
+            *dp = sum;
           }
+          lp += a.C;
+          dp += a.C;
+        }
       }
     }
   }
@@ -380,7 +426,7 @@ recurrence_carry_kernel(RecurrenceArgs a, int seq_base, const float* __restrict_
     for (int j = 0; j < U; ++j)
       if (j0 + j < chunks) {
         carry[(static_cast<size_t>(blockIdx.y) * max_chunks + j0 + j) * a.C + c] = S;
-        S = fmaf(expf(d[j]), S, s[j]);
+        S = fmaf(exp2f(d[j]), S, s[j]);
       }
   }
   mem[0] = S;
@@ -396,7 +442,7 @@ recurrence_carry_kernel(RecurrenceArgs a, int seq_base, const float* __restrict_
   }
 }
 
-// out = (S of the chunk alone + exp(sum of log a) * entering state) * gelu(y); 4 channels per thread
+// out = (S of the chunk alone + a's product so far * entering state) * gelu(y); 4 channels per thread
 template <int TC>
 __global__ void __launch_bounds__(256)
 recurrence_finish_kernel(RecurrenceArgs a, const int* __restrict__ seq_of_token, int seq_base,
@@ -412,15 +458,30 @@ recurrence_finish_kernel(RecurrenceArgs a, const int* __restrict__ seq_of_token,
   load_n<4>(carry + (static_cast<size_t>(b - seq_base) * max_chunks + chunk) * a.C + c, in);
   load_n<4>(static_cast<const __nv_bfloat16*>(a.y) + static_cast<size_t>(t) * a.ldy + c, y);
 #pragma unroll
-  for (int j = 0; j < 4; ++j) s[j] = fmaf(__expf(d[j]), in[j], s[j]) * gelu_tanh_as<__nv_bfloat16>(y[j]);
+  for (int j = 0; j < 4; ++j) s[j] = fmaf(ex2_ftz(d[j]), in[j], s[j]) * gelu_tanh_as<__nv_bfloat16>(y[j]);
   store_n<4>(static_cast<__nv_bfloat16*>(a.out) + static_cast<size_t>(t) * a.ldo + c, s);
+}
+
+// One step's inputs move into the last rows of the memory, where recurrence_tile_kernel could not do it.
+__global__ void __launch_bounds__(256)
+recurrence_shift_kernel(RecurrenceArgs a, int seq_base) {
+  const int c = blockIdx.x * 256 + threadIdx.x, b = seq_base + blockIdx.y;
+  if (c >= a.C) return;
+  float* mem = a.state + static_cast<size_t>(a.slots[b]) * a.K * a.C + c;
+  const bool first = a.kv_lens[b] == 1;
+  for (int j = 1; j < a.K; ++j)
+    mem[static_cast<size_t>(j) * a.C] =
+        j == a.K - 1 ? __bfloat162float(static_cast<const __nv_bfloat16*>(a.x)[static_cast<size_t>(a.cu_q[b]) * a.ldx + c])
+        : first      ? 0.f
+                     : mem[static_cast<size_t>(j + 1) * a.C];
 }
 
 static bool tile_sizes(const RecurrenceArgs& a, const void* gates) {
   auto rows16 = [](const void* p, int ld) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && (ld & 7) == 0; };
   const int part = a.C / a.B;
   return part % 8 == 0 && part <= RG_MAX_PART && a.K >= 1 && a.K <= 8 && rows16(a.x, a.ldx) && rows16(a.y, a.ldy) &&
-         rows16(a.out, a.ldo) && rows16(gates, 0) && rows16(a.state, 0) && rows16(a.conv_b, 0);
+         rows16(a.out, a.ldo) && rows16(gates, 0) && rows16(a.state, 0) &&
+         rows16(a.conv_w, 0) && rows16(a.conv_b, 0);
 }
 
 template <int TC, int KT, bool STEP>
@@ -434,11 +495,11 @@ static int launch_tile(const RecurrenceArgs& a, const void* gates, int seq_base,
   auto kern = recurrence_tile_kernel<TC, KT, STEP>;
   if (KSANA_SMEM_ONCE(kern, RecurrenceSmem<TC>::total(RG_MAX_PART / 64)) != 0) return -4;
   const dim3 grid((columns + TC - 1) / TC, a.B * ((part + 127) / 128), STEP ? 1 : num_seqs);
-  kern<<<grid, 128, smem, st>>>(tw, a, seq_base, num_seqs, local, decay, tok_base, error_word());
+  kern<<<grid, 256, smem, st>>>(tw, a, seq_base, num_seqs, local, decay, tok_base, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
-constexpr int RG_CHUNK = 128, RG_STEP = 16;
+constexpr int RG_TILE = 128, RG_CHUNK = RG_TILE / 2, RG_STEP = 16;
 
 }  // namespace ksana
 
@@ -450,7 +511,7 @@ KSANA_API long long ksana_recurrence_scratch(int tokens, int num_seqs, int max_q
 }
 
 // bf16. Sequences [seq_base, seq_base + num_seqs), whose tokens are [tok_base, tok_base + tokens), at most max_q each.
-// gates: [2, B, C / B, C / B]. -1: sizes it does not take.
+// conv_w: [K, C], gates: [2, B, C / B, C / B]. -1: sizes it does not take.
 KSANA_API int ksana_recurrence_prompts(const void* y, int ldy, const void* x, int ldx, float* state, const int* slots,
                                        const int* cu_q, const int* kv_lens, const int* seq_of_token, const float* conv_w,
                                        const float* conv_b, const void* gates, const float* gates_b, const float* rate,
@@ -462,8 +523,8 @@ KSANA_API int ksana_recurrence_prompts(const void* y, int ldy, const void* x, in
   if (!tile_sizes(a, gates)) return -1;
   const int max_chunks = (max_q + RG_CHUNK - 1) / RG_CHUNK;
   float *local = scratch, *decay = local + static_cast<size_t>(tokens) * C, *carry = decay + static_cast<size_t>(tokens) * C;
-  const int rc = K <= 4 ? launch_tile<RG_CHUNK, 4, false>(a, gates, seq_base, num_seqs, max_q, local, decay, tok_base, st)
-                        : launch_tile<RG_CHUNK, 8, false>(a, gates, seq_base, num_seqs, max_q, local, decay, tok_base, st);
+  const int rc = K <= 4 ? launch_tile<RG_TILE, 4, false>(a, gates, seq_base, num_seqs, max_q, local, decay, tok_base, st)
+                        : launch_tile<RG_TILE, 8, false>(a, gates, seq_base, num_seqs, max_q, local, decay, tok_base, st);
   if (rc) return rc;
   recurrence_carry_kernel<RG_CHUNK><<<dim3((C + 127) / 128, num_seqs), 128, 0, st>>>(a, seq_base, local, decay, carry,
                                                                                      max_chunks, tok_base);
@@ -480,9 +541,12 @@ KSANA_API int ksana_recurrence_step(const void* y, int ldy, const void* x, int l
   if (num_seqs <= 0) return 0;
   if (B < 1 || C % B || K < 1) return -2;
   RecurrenceArgs a{y, ldy, x, ldx, state, slots, cu_q, kv_lens, conv_w, conv_b, gates_b, rate, out, ldo, C, K, B};
-  if (!tile_sizes(a, gates) || C / B > 128) return -1;
-  return K <= 4 ? launch_tile<RG_STEP, 4, true>(a, gates, seq_base, num_seqs, num_seqs, nullptr, nullptr, 0, st)
-                : launch_tile<RG_STEP, 8, true>(a, gates, seq_base, num_seqs, num_seqs, nullptr, nullptr, 0, st);
+  if (!tile_sizes(a, gates)) return -1;
+  const int rc = K <= 4 ? launch_tile<RG_STEP, 4, true>(a, gates, seq_base, num_seqs, num_seqs, nullptr, nullptr, 0, st)
+                        : launch_tile<RG_STEP, 8, true>(a, gates, seq_base, num_seqs, num_seqs, nullptr, nullptr, 0, st);
+  if (rc || C / B <= 128 || K == 1) return rc;
+  recurrence_shift_kernel<<<dim3((C + 255) / 256, num_seqs), 256, 0, st>>>(a, seq_base);
+  return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
 KSANA_API int ksana_recurrence_conv(const void* x, int ldx, const float* state, const int* slots, const int* cu_q,

@@ -149,6 +149,7 @@ class RecurrenceWeights:
     def __init__(self, w: Dict[str, torch.Tensor], prefix: str, decay_scale: float):
         self.conv, self.conv_b = w[prefix + ".conv"], w[prefix + ".conv_b"]        # [C, K], [C] fp32
         self.gates, self.gates_b = w[prefix + ".gates"], w[prefix + ".gates_b"]    # [2, B, C / B, C / B], [2, C] fp32
+        self.conv_t = self.conv.t().contiguous()                                   # [K, C]: one load for neighbours
         lam = w[prefix + ".lam"].double()
         self.rate = (decay_scale * torch.nn.functional.softplus(lam, threshold=100)).float()  # [C]
         self.gates_by_block = torch.cat((self.gates[0], self.gates[1]), 1).contiguous()  # [B, 2 C / B, C / B]

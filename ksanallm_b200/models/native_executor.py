@@ -413,7 +413,7 @@ class MixerExecutor:
             if layer.recurrence is not None:
                 a, s = layer.recurrence.w, layer.recurrence.spec
                 L.rc, L.rk, L.rb = s.width, s.taps, s.blocks
-                L.conv_w, L.conv_b, L.gates, L.gates_by_block = _p(a.conv), _p(a.conv_b), _p(a.gates), _p(a.gates_by_block)
+                L.conv_w, L.conv_b, L.gates, L.gates_by_block = _p(a.conv_t), _p(a.conv_b), _p(a.gates), _p(a.gates_by_block)
                 L.gates_b, L.rate = _p(a.gates_b), _p(a.rate)
             if layer.linear is not None:
                 a, s = layer.linear, layer.linear.spec

@@ -18,7 +18,7 @@ def gated_recurrence(y, x, state, meta, w, out: torch.Tensor) -> None:
     n_pre, n_dec, pre_tokens = meta.num_prefill, meta.num_decode, meta.num_prefill_tokens
     rows = (_ptr(y), y.stride(0), _ptr(x), x.stride(0), _ptr(state), _ptr(meta.state_slots), _ptr(meta.cu_q),
             _ptr(meta.kv_lens))
-    maps = (_ptr(w.conv), _ptr(w.conv_b), _ptr(w.gates), _ptr(w.gates_b), _ptr(w.rate), C, K, B, _ptr(out), out.stride(0))
+    maps = (_ptr(w.conv_t), _ptr(w.conv_b), _ptr(w.gates), _ptr(w.gates_b), _ptr(w.rate), C, K, B, _ptr(out), out.stride(0))
 
     def general(seq_base: int, seqs: int, tok_base: int, tokens: int) -> None:
         if not seqs or not tokens:
@@ -26,7 +26,7 @@ def gated_recurrence(y, x, state, meta, w, out: torch.Tensor) -> None:
         kind = _KIND[x.dtype]
         u = torch.empty(tokens, C, dtype=x.dtype, device=x.device)
         _check(lib().ksana_recurrence_conv(_ptr(x), x.stride(0), _ptr(state), _ptr(meta.state_slots), _ptr(meta.cu_q),
-                                           _ptr(meta.kv_lens), _ptr(meta.seq_of_token), _ptr(w.conv), _ptr(w.conv_b), C,
+                                           _ptr(meta.kv_lens), _ptr(meta.seq_of_token), _ptr(w.conv_t), _ptr(w.conv_b), C,
                                            K, _ptr(u), tok_base, tokens, kind, _stream()), "recurrence_conv")
         z = torch.empty(tokens, B, 2 * (C // B), dtype=torch.float32, device=x.device)
         head_gemm(u.view(tokens, B, C // B), w.gates_by_block, z)
