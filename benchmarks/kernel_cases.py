@@ -338,10 +338,10 @@ def case_latent_decode():
     st = torch.cuda.current_stream().cuda_stream
 
     def kernel(i):
-        assert cuda.lib().ksana_window_decode(
-            qc.data_ptr(), qc.stride(0), cache.data_ptr(), cache.shape[0], meta.block_tables.data_ptr(), meta.max_blocks,
-            meta.cu_q.data_ptr(), meta.kv_lens.data_ptr(), h, 1, rank + rot, rank, 16, 0, 0, 1, 0.07, None, 0, 1.0, 0.0, 0,
-            gate.data_ptr(), gate.stride(0), o.data_ptr(), o.stride(0), 0, B, ctx, st) == 0
+        assert cuda.lib().ksana_latent_decode(
+            qc.data_ptr(), qc.stride(0), B, cache.data_ptr(), cache.shape[0], meta.block_tables.data_ptr(), meta.max_blocks,
+            meta.cu_q.data_ptr(), meta.kv_lens.data_ptr(), h, rank, rot, 16, 0.07, gate.data_ptr(), gate.stride(0),
+            o.data_ptr(), o.stride(0), 0, B, 1, ctx, st) == 0
     us = timeit(kernel)
     op = timeit(lambda i: cuda_latent.latent_attention(q, a, norm, 1e-6, table, cache, meta, 16, w, 0.07, gate, out))
     by, p = B * ctx * (rank + rot) * 2, peaks()

@@ -117,23 +117,6 @@ struct RecurrenceSmem {
   __host__ __device__ static int total(int kc) { return kc * (U_BYTES + 2 * W_BYTES) + 256 + 1024; }
 };
 
-// Hardware approximations (relative error about 1e-7) without the handling of denormal numbers around them.
-__device__ __forceinline__ float ex2_ftz(float x) {
-  float r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-__device__ __forceinline__ float rcp_ftz(float x) {
-  float r;
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-__device__ __forceinline__ float rsqrt_ftz(float x) {
-  float r;
-  asm("rsqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
-  return r;
-}
-constexpr float LOG2E = 1.4426950408889634f;
 // 1 / (1 + 2^x): the sigmoid of -x ln 2
 __device__ __forceinline__ float sigmoid_log2(float x) { return rcp_ftz(1.f + ex2_ftz(x)); }
 // l = log2 a <= 0 -> a and sqrt(1 - a^2). 1 - a^2 = -expm1(2 l ln 2) is a power series where the difference would cancel.
@@ -215,7 +198,7 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
 
   // ---- u -> shared memory
   const __nv_bfloat16* x = static_cast<const __nv_bfloat16*>(a.x) + blk * part;
-  const int vecs = part / 8, strips = STEP ? TC : TC / 16;
+  const int vecs = part / 8, strips = STEP ? TC : TC / 8;
   for (int w = tid; w < kc * 8 * strips; w += 256) {
     const int v = w % (kc * 8), strip = w / (kc * 8), c = v * 8;
     uint8_t* dst = sU + (v >> 3) * L_::U_BYTES;
@@ -224,13 +207,31 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
           make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
     };
     const float zero[8] = {0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f, 0.f};
-    constexpr int ROWS = STEP ? 1 : 16;
+    constexpr int ROWS = STEP ? 1 : 8;
     if (v >= vecs || strip * ROWS >= n) {
       for (int r = 0; r < ROWS; ++r) put(strip * ROWS + r, zero);
       continue;
     }
     const int ch = blk * part + c;
-    float taps[KT][8], bias[8], win[KT][8];  // taps[KT - 1] meets the newest input
+    // STEP: the inputs before this one and this one; else the strip's and those before it, all loads in flight together
+    [[maybe_unused]] uint4 raw[STEP ? 1 : ROWS + KT - 1];
+    if constexpr (!STEP) {
+      const float* mem = a.state + static_cast<size_t>(a.slots[b]) * a.K * a.C + ch;
+#pragma unroll
+      for (int j = 0; j < ROWS + KT - 1; ++j) {
+        const int i = i0 + strip * ROWS + j - (KT - 1);  // token of this portion, or what came before it
+        raw[j] = make_uint4(0u, 0u, 0u, 0u);
+        if (i >= 0) {
+          if (i < i0 + n) raw[j] = *reinterpret_cast<const uint4*>(x + static_cast<size_t>(q0 + i) * a.ldx + c);
+        } else if (!fresh && i > -a.K) {
+          float f[8];
+          load_n<8>(mem + static_cast<size_t>(a.K + i) * a.C, f);
+          raw[j] = make_uint4(pack_bf16(f[0], f[1]), pack_bf16(f[2], f[3]), pack_bf16(f[4], f[5]), pack_bf16(f[6], f[7]));
+        }
+      }
+    }
+    float taps[KT][8], bias[8];  // taps[KT - 1] meets the newest input
+    [[maybe_unused]] float win[STEP ? KT : 1][8];
     load_n<8>(a.conv_b + ch, bias);
 #pragma unroll
     for (int j = 0; j < KT; ++j) {
@@ -271,39 +272,21 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
         }
       }
     } else {
-      const float* mem = a.state + static_cast<size_t>(a.slots[b]) * a.K * a.C + ch;
-      auto input = [&](int i, float* f) {  // token i of this portion, or what came before it
-        if (i >= 0) {
-          load_n<8>(x + static_cast<size_t>(q0 + i) * a.ldx + c, f);
-        } else if (!fresh && i > -a.K) {
-          load_n<8>(mem + static_cast<size_t>(a.K + i) * a.C, f);
-        } else {
+      float in[KT][8];
 #pragma unroll
-          for (int e = 0; e < 8; ++e) f[e] = 0.f;
-        }
-      };
-      const int r0 = strip * 16;
+      for (int j = 0; j < KT - 1; ++j) unpack8(raw[j], in[j]);
 #pragma unroll
-      for (int j = 0; j < KT - 1; ++j) input(i0 + r0 - (KT - 1) + j, win[j + 1]);
-#pragma unroll KT
-      for (int r = 0; r < 16; ++r) {
-        if (r0 + r >= n) {
-          put(r0 + r, zero);
-          continue;
-        }
-#pragma unroll
-        for (int j = 0; j < KT - 1; ++j)
-#pragma unroll
-          for (int e = 0; e < 8; ++e) win[j][e] = win[j + 1][e];
-        input(i0 + r0 + r, win[KT - 1]);
+      for (int r = 0; r < ROWS; ++r) {
+        unpack8(raw[r + KT - 1], in[(r + KT - 1) % KT]);
         float f[8];
 #pragma unroll
         for (int e = 0; e < 8; ++e) {
           f[e] = bias[e];
 #pragma unroll
-          for (int j = 0; j < KT; ++j) f[e] = fmaf(taps[j][e], win[j][e], f[e]);
+          for (int j = 0; j < KT; ++j) f[e] = fmaf(taps[j][e], in[(r + j) % KT][e], f[e]);
+          if (strip * ROWS + r >= n) f[e] = 0.f;
         }
-        put(r0 + r, f);
+        put(strip * ROWS + r, f);
       }
     }
   }

@@ -96,6 +96,24 @@ __device__ __forceinline__ float gelu_tanh_as(float z) {
   }
 }
 
+// Hardware approximations (relative error about 1e-7) without the handling of denormal numbers around them.
+__device__ __forceinline__ float ex2_ftz(float x) {
+  float r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+__device__ __forceinline__ float rcp_ftz(float x) {
+  float r;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+__device__ __forceinline__ float rsqrt_ftz(float x) {
+  float r;
+  asm("rsqrt.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(x));
+  return r;
+}
+constexpr float LOG2E = 1.4426950408889634f;
+
 // v = hi + lo with both parts bf16: the pair keeps 16 bits of the mantissa through 16-bit tensor-core operands. Packs
 // two values; *lo is exact up to its own rounding.
 __device__ __forceinline__ uint32_t split_bf16(float a, float b, uint32_t* lo) {

@@ -72,6 +72,10 @@ int ksana_latent_append(void* q, int ldq, int dim, void* q_cat, int cat_from, co
                         int h, int rank, int rot, int kind, cudaStream_t st);
 int ksana_latent_gather(const void* cache, const int* block_tables, int max_blocks, const int* kv_lens, int seq_base,
                         int num_seqs, int max_kv, int bs, int width, void* out, cudaStream_t st);
+int ksana_latent_decode(const void* q, int ldq, int total_tokens, const void* cache, int num_blocks,
+                        const int* block_tables, int max_blocks, const int* cu_q, const int* kv_lens, int h, int rank,
+                        int rot, int bs, float scale, const void* gate, int ldg, void* out, int ldo, int seq_base,
+                        int num_seqs, int max_q, int max_kv, cudaStream_t st);
 int ksana_latent_prefill(const void* q, int ldq, int total_tokens, const void* kv, int ldkv, const void* rot, int ldr,
                          int rows, const int* cu_q, const int* kv_lens, int h, int d, int rd, int dv, float scale,
                          const void* gate, int ldg, void* out, int ldo, int seq_base, int num_seqs, int max_q,
@@ -233,10 +237,10 @@ struct Exec {
     const char* qc = q_cat - static_cast<size_t>(p.first) * ldc * 2;
     char* oc = o - static_cast<size_t>(p.first) * ldo * 2;
     int rc = -1;
-    if (s->num_decode == rows)
-      rc = ksana_window_decode(qc, ldc, w.kv, m->num_blocks, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, w.ah, 1,
-                               width, w.arank, m->block_size, 0, 0, 1, w.ascale, nullptr, 0, 1.f, 0.f, 0, gate, ld, oc, ldo,
-                               s->num_prefill, s->num_decode, s->max_kv_decode, st);
+    if (p.first == s->prefill_tokens)  // only the sequences behind the prompts
+      rc = ksana_latent_decode(qc, ldc, T, w.kv, m->num_blocks, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, w.ah,
+                               w.arank, w.rot, m->block_size, w.ascale, gate, ld, oc, ldo, s->num_prefill, s->num_decode,
+                               s->max_q_decode, s->max_kv_decode, st);
     if (rc == -1)
       rc = ksana_window_attention_any(qc, ldc, w.kv, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, s->seq_of_token,
                                       w.ah, 1, width, w.arank, m->block_size, 0, 0, 1, w.ascale, nullptr, 0, 1.f, 0.f, 0,

@@ -125,6 +125,7 @@ struct KsanaMixerStep {
   int one_token;         // every decode sequence has exactly one new token
   int num_long;          // leading prompt portions long enough for the chunked form of linear attention
   int long_tokens;       // their tokens
+  int max_q_decode;
   const int* cu_q_host;
   const int* kv_lens_host;
 };

@@ -179,13 +179,30 @@ struct WindowPrefillSmem {
 // are small against the cap take a polynomial, odd to degree 11 (error below 1e-7 of the cap up to |s / c| = 0.4); others
 // the exponential form.
 constexpr float CAP_POLY = 0.4f;
-__device__ __forceinline__ float cap_small(float s, float inv_c) {
-  const float x = s * inv_c, z = x * x;
-  float p = fmaf(z, -1382.f / 155925.f, 62.f / 2835.f);
-  p = fmaf(p, z, -17.f / 315.f);
-  p = fmaf(p, z, 2.f / 15.f);
-  p = fmaf(p, z, -1.f / 3.f);
-  return fmaf(p * z, s, s);
+// two 32-bit floats in one register pair; FMAs on them issue as one
+__device__ __forceinline__ uint64_t pair(float a, float b) {
+  uint64_t r;
+  asm("mov.b64 %0, {%1, %2};" : "=l"(r) : "f"(a), "f"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
+  uint64_t r;
+  asm("mul.rn.f32x2 %0, %1, %2;" : "=l"(r) : "l"(a), "l"(b));
+  return r;
+}
+__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
+  uint64_t r;
+  asm("fma.rn.f32x2 %0, %1, %2, %3;" : "=l"(r) : "l"(a), "l"(b), "l"(c));
+  return r;
+}
+__device__ __forceinline__ void cap_small2(float* s, float inv_c) {
+  const uint64_t v = pair(s[0], s[1]), x = mul2(v, pair(inv_c, inv_c)), z = mul2(x, x);
+  uint64_t p = fma2(z, pair(-1382.f / 155925.f, -1382.f / 155925.f), pair(62.f / 2835.f, 62.f / 2835.f));
+  p = fma2(p, z, pair(-17.f / 315.f, -17.f / 315.f));
+  p = fma2(p, z, pair(2.f / 15.f, 2.f / 15.f));
+  p = fma2(p, z, pair(-1.f / 3.f, -1.f / 3.f));
+  p = fma2(mul2(p, z), v, v);
+  asm("mov.b64 {%0, %1}, %2;" : "=f"(s[0]), "=f"(s[1]) : "l"(p));
 }
 __device__ __forceinline__ float cap_any(float s, float c, float inv_c) {
   const float x = fminf(fmaxf(s * inv_c, -20.f), 20.f);
@@ -386,16 +403,17 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_cons
       if constexpr (CAP) {
         float big = 0.f;
 #pragma unroll
-        for (int j = 0; j < 128; ++j) {
-          s[j] *= scale2;
-          big = fmaxf(big, fabsf(s[j]));
+        for (int j = 0; j < 128; j += 2) {
+          const uint64_t v = mul2(pair(s[j], s[j + 1]), pair(scale2, scale2));
+          asm("mov.b64 {%0, %1}, %2;" : "=f"(s[j]), "=f"(s[j + 1]) : "l"(v));
+          big = fmaxf(big, fmaxf(fabsf(s[j]), fabsf(s[j + 1])));
         }
         if (__any_sync(0xffffffffu, big > CAP_POLY * cap2)) {
 #pragma unroll
           for (int j = 0; j < 128; ++j) s[j] = cap_any(s[j], cap2, inv_cap2);
         } else {
 #pragma unroll
-          for (int j = 0; j < 128; ++j) s[j] = cap_small(s[j], inv_cap2);
+          for (int j = 0; j < 128; j += 2) cap_small2(s + j, inv_cap2);
         }
       }
       if (KEEP && kept > 0) {
@@ -580,7 +598,7 @@ struct WindowDecodeSmem {
   static constexpr int STAGES = PAGE <= 2048 ? 4 : PAGE <= 4096 ? 3 : 2;
   static constexpr int RING = 4 * STAGES * PAGE;
   static constexpr int LDO = DVP + 4;
-  static constexpr int MERGE = 4 * (DVP > 256 ? 8 : 16) * LDO * 4;  // over the ring, once every page has been multiplied
+  static constexpr int MERGE = 4 * 16 * LDO * 4;  // over the ring, once every page has been multiplied
   static constexpr int TOTAL = (RING > MERGE ? RING : MERGE) + 1024;
 };
 
@@ -689,30 +707,19 @@ window_decode_kernel(const __grid_constant__ CUtensorMap tmK, const __grid_const
       break;
     }
     const uint32_t kb0 = smem_u32(ring + (n % STAGES) * L_::PAGE), vb0 = kb0 + (SHARED ? 0 : L_::K_BYTES);
-    constexpr int CHAINS = DP > 128 ? 4 : 1;  // independent sums over long keys
-    float c[NT][4], part[CHAINS][NT][4];
+    float c[NT][4];
 #pragma unroll
-    for (int x = 0; x < CHAINS; ++x)
+    for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-        for (int u = 0; u < 4; ++u) part[x][nt][u] = 0.f;
+      for (int u = 0; u < 4; ++u) c[nt][u] = 0.f;
 #pragma unroll
     for (int kb = 0; kb < DP / 16; ++kb) {
       uint32_t f[4];
       const int ch = kb * 2 + k_col;
       ldmatrix_x4<false>(f, kb0 + (ch >> 3) * 2048 + k_row * 128 + (((ch & 7) ^ (k_row & 7)) << 4));
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) mma_16816(part[kb % CHAINS][nt], f, qf[kb][nt][0], qf[kb][nt][1]);
+      for (int nt = 0; nt < NT; ++nt) mma_16816(c[nt], f, qf[kb][nt][0], qf[kb][nt][1]);
     }
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-      for (int u = 0; u < 4; ++u) {
-        c[nt][u] = part[0][nt][u];
-#pragma unroll
-        for (int x = 1; x < CHAINS; ++x) c[nt][u] += part[x][nt][u];
-      }
     const int key0 = page(n) * 16 + r;
 #pragma unroll
     for (int u = 0; u < 2; ++u) {
@@ -946,23 +953,11 @@ KSANA_API int ksana_window_decode(const void* q, int ldq, const void* cache, int
                                   int ldo, int seq_base, int num_seqs, int max_kv, cudaStream_t st) {
   if (num_seqs <= 0) return 0;
   if (keep < 0 || (shared && d < dv)) return -2;
-  const int top = shared ? 576 : 128;
-  if (h % hk || bs != WP_PAGE || d > top || dv > top || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
+  if (h % hk || bs != WP_PAGE || d > 128 || dv > 128 || (shared && d != dv) || (d & 7) || (dv & 7) || !rows16(q, ldq) || !rows16(cache, 0) ||
       !rows16(out, ldo))
     return -1;
   WindowAttnArgs a{q, ldq, cache, block_tables, max_blocks, cu_q, kv_lens, nullptr, h, hk, d, dv, bs, window, keep,
                    shared, scale, bias, bias_len, out_scale, out, ldo, softcap, sink, gate, ldg};
-  if (shared && (d > 128 || d != dv)) {  // latents: long keys, values the first part of them
-#define KSANA_WL(DP, DVP) \
-  if (d <= DP && dv <= DVP) return launch_decode<DP, DVP, 1, true>(a, num_blocks, seq_base, num_seqs, max_kv, st)
-    KSANA_WL(64, 64);
-    KSANA_WL(128, 128);
-    KSANA_WL(192, 128);
-    KSANA_WL(320, 256);
-    KSANA_WL(576, 512);
-#undef KSANA_WL
-    return -1;
-  }
 #define KSANA_WD(DP, DVP, SHARED)                                                                             \
   return h / hk <= 8 ? launch_decode<DP, DVP, 1, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)       \
                      : launch_decode<DP, DVP, 2, SHARED>(a, num_blocks, seq_base, num_seqs, max_kv, st)

@@ -328,8 +328,8 @@ class _MixerStep(ctypes.Structure):
     _fields_ = [(n, P) for n in ("positions", "slot_mapping", "seq_of_token", "block_tables", "cu_q", "kv_lens",
                                  "state_slots", "start")] + \
         [(n, I) for n in ("total_tokens", "max_blocks", "num_prefill", "num_decode", "prefill_tokens", "max_q_prefill",
-                          "max_kv_decode", "one_token", "num_long", "long_tokens")] + \
-        [("cu_q_host", P), ("kv_lens_host", P)]
+                          "max_kv_decode", "one_token", "num_long", "long_tokens",
+                          "max_q_decode")] + [("cu_q_host", P), ("kv_lens_host", P)]
 
 
 class MixerExecutor:
@@ -508,6 +508,7 @@ class MixerExecutor:
         s.max_q_prefill = int((cu[1:n_pre + 1] - cu[:n_pre]).max()) if n_pre else 0
         s.max_kv_decode = int(meta.kv_lens_host[n_pre:].max()) if n_dec else 0
         s.one_token = int(T - s.prefill_tokens == n_dec)
+        s.max_q_decode = int((cu[n_pre + 1:] - cu[n_pre:-1]).max()) if n_dec else 0
         s.num_long = long_portions(meta) if any(x.lh for x in self._layers) else 0
         s.long_tokens = int(cu[s.num_long])
         if s.num_long:

@@ -91,6 +91,7 @@ class _Sig:
     ksana_hyper_norm = ([P, I, P, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, F, I, P], I)
     ksana_head_gemm_any = ([P, LL, LL, P, P, LL, LL, I, I, I, I, I, P], I)
     ksana_latent_append = ([P, I, I, P, I, P, I, P, F, P, P, P, P, I, I, I, I, I, P], I)
+    ksana_latent_decode = ([P, I, I, P, I, P, I, P, P, I, I, I, I, F, P, I, P, I, I, I, I, I, P], I)
     ksana_latent_gather = ([P, P, I, P, I, I, I, I, I, P, P], I)
     ksana_latent_prefill = ([P, I, I, P, I, P, I, I, P, P, I, I, I, I, F, P, I, P, I, I, I, I, P], I)
     ksana_recurrence_scratch = ([I, I, I, I], LL)

@@ -82,17 +82,18 @@ def latent_attention(q, a, norm_w, eps: float, rotary, cache, meta, block_size: 
     o = torch.empty(T - first, h * rank, dtype=q.dtype, device=q.device)
     # the kernels index tokens of the whole step
     at = [x.data_ptr() - first * x.stride(0) * x.element_size() for x in (q_cat, o)]
-    shape = (h, 1, rank + rot, rank, block_size, 0, 0, 1, float(scale), None, 0, 1.0, 0.0, 0, _ptr(gate),
-             gate.stride(0) if gate is not None else 0)
+    gates = (_ptr(gate), gate.stride(0) if gate is not None else 0)
     code = -1
-    if q.dtype == torch.bfloat16 and n_dec == T - first:
-        code = lib().ksana_window_decode(at[0], q_cat.stride(0), _ptr(cache), cache.shape[0], _ptr(meta.block_tables),
-                                         meta.max_blocks, _ptr(meta.cu_q), _ptr(meta.kv_lens), *shape, at[1], o.stride(0),
-                                         n_pre, n_dec, int(meta.kv_lens_host[n_pre:].max()), _stream())
+    if q.dtype == torch.bfloat16 and first == meta.num_prefill_tokens:  # only the sequences behind the prompts
+        cu = meta.cu_q_host[n_pre:]
+        code = lib().ksana_latent_decode(
+            at[0], q_cat.stride(0), T, _ptr(cache), cache.shape[0], _ptr(meta.block_tables), meta.max_blocks,
+            _ptr(meta.cu_q), _ptr(meta.kv_lens), h, rank, rot, block_size, float(scale), *gates, at[1], o.stride(0), n_pre,
+            n_dec, int((cu[1:] - cu[:-1]).max()), int(meta.kv_lens_host[n_pre:].max()), _stream())
     if code == -1:
         code = lib().ksana_window_attention_any(
             at[0], q_cat.stride(0), _ptr(cache), _ptr(meta.block_tables), meta.max_blocks, _ptr(meta.cu_q),
-            _ptr(meta.kv_lens), _ptr(meta.seq_of_token), *shape, at[1], o.stride(0), first, T - first, _KIND[q.dtype],
-            _stream())
+            _ptr(meta.kv_lens), _ptr(meta.seq_of_token), h, 1, rank + rot, rank, block_size, 0, 0, 1, float(scale), None, 0,
+            1.0, 0.0, 0, *gates, at[1], o.stride(0), first, T - first, _KIND[q.dtype], _stream())
     _check(code, "latent_attention")
     head_gemm(o.view(T - first, h, rank), w.uv, out[first:].unflatten(1, (h, vdim)))
