@@ -12,10 +12,11 @@
 
 namespace ksana {
 
-// sqrt(1 - a^2) and a itself from log a <= 0
-__device__ __forceinline__ void decay_of(float la, float* a, float* in) {
-  *a = expf(la);
-  *in = sqrtf(-expm1f(2.f * la));
+// a - 1 and sqrt(1 - a^2) from log a <= 0. The recurrence runs as S + (a - 1) S: over thousands of tokens the rounding of
+// an a close to 1 would add up.
+__device__ __forceinline__ void decay_of(float la, float* am1, float* in) {
+  *am1 = expm1f(la);
+  *in = sqrtf(-*am1 * (2.f + *am1));
 }
 
 struct RecurrenceArgs {
@@ -79,9 +80,9 @@ recurrence_scan_kernel(RecurrenceArgs a, const T* __restrict__ u, const float* _
   for (int t = q0; t < q0 + n; ++t) {
     const size_t row = t - tok_base;
     const float* zt = z + (row * a.B + blk) * 2 * part + off;
-    float dec, in;
-    decay_of(-sigmoid_f(zt[0] + br) * rate, &dec, &in);
-    S = fmaf(dec, S, in * sigmoid_f(zt[part] + bi) * to_f(u[row * a.C + c]));
+    float am1, in;
+    decay_of(-sigmoid_f(zt[0] + br) * rate, &am1, &in);
+    S = fmaf(am1, S, S) + in * sigmoid_f(zt[part] + bi) * to_f(u[row * a.C + c]);
     out[static_cast<size_t>(t) * a.ldo + c] = from_f<T>(S * gelu_tanh_f(to_f(y[static_cast<size_t>(t) * a.ldy + c])));
   }
   mem[0] = S;
@@ -119,13 +120,13 @@ struct RecurrenceSmem {
 
 // 1 / (1 + 2^x): the sigmoid of -x ln 2
 __device__ __forceinline__ float sigmoid_log2(float x) { return rcp_ftz(1.f + ex2_ftz(x)); }
-// l = log2 a <= 0 -> a and sqrt(1 - a^2). 1 - a^2 = -expm1(2 l ln 2) is a power series where the difference would cancel.
-__device__ __forceinline__ void decay_fast(float l, float* a, float* in) {
-  const float e = ex2_ftz(l);
-  constexpr float c = 1.3862943611198906f;  // 2 ln 2
-  const float small = -l * fmaf(l, fmaf(l, fmaf(l, c * c * c * c / 24.f, c * c * c / 6.f), c * c / 2.f), c);
-  const float w = fmaxf(l > -0.05f ? small : fmaf(-e, e, 1.f), 1e-30f);
-  *a = e;
+// l = log2 a <= 0 -> a - 1 and sqrt(1 - a^2). a - 1 = expm1(l ln 2) is a power series where the difference would cancel.
+__device__ __forceinline__ void decay_fast(float l, float* am1, float* in) {
+  constexpr float c = 0.6931471805599453f;  // ln 2
+  const float small = l * fmaf(l, fmaf(l, fmaf(l, c * c * c * c / 24.f, c * c * c / 6.f), c * c / 2.f), c);
+  const float d = l > -0.05f ? small : ex2_ftz(l) - 1.f;
+  const float w = fmaxf(-d * (2.f + d), 1e-30f);
+  *am1 = d;
   *in = w * rsqrt_ftz(w);
 }
 
@@ -352,7 +353,7 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
 #pragma unroll
         for (int j = 0; j < N; ++j)
           if (mine && c0 + j < n) {
-            const float s = fmaf(dec[j], old[j], in[j]);
+            const float s = fmaf(dec[j], old[j], old[j]) + in[j];
             *mem_at[j] = s;
             static_cast<__nv_bfloat16*>(a.out)[static_cast<size_t>(row_at[j]) * a.ldo + ch] =
                 __float2bfloat16_rn(s * gelu_tanh_as<__nv_bfloat16>(yy[j]));
@@ -360,7 +361,7 @@ recurrence_tile_kernel(const __grid_constant__ CUtensorMap tmW, RecurrenceArgs a
       } else {
 #pragma unroll
         for (int j = 0; j < N; ++j) {
-          S = fmaf(dec[j], S, in[j]);
+          S = fmaf(dec[j], S, S) + in[j];
           sum += l2[j];
           if (mine && c0 + j < n) {
             *lp = S;

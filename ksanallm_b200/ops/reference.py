@@ -550,10 +550,11 @@ def gated_recurrence(y: torch.Tensor, x: torch.Tensor, state: torch.Tensor, slot
         u = u.to(x.dtype).float()
         z = torch.einsum("nbi,gboi->gnbo", u.view(-1, B, C // B), w_gates.float()).reshape(2, -1, C) + b_gates.unsqueeze(1)
         la = -torch.sigmoid(z[0]) * rate
-        a, inp = torch.exp(la), torch.sqrt(-torch.expm1(2 * la)) * torch.sigmoid(z[1]) * u
+        am1 = torch.expm1(la)  # S + (a - 1) S: the rounding of an a close to 1 would add up over many tokens
+        inp = torch.sqrt(-am1 * (2 + am1)) * torch.sigmoid(z[1]) * u
         S, rows = mem[0].clone(), []
         for t in range(hi - lo):
-            S = a[t] * S + inp[t]
+            S = S + am1[t] * S + inp[t]
             rows.append(S)
         out[lo:hi] = (torch.stack(rows) * F.gelu(y[lo:hi].float(), approximate="tanh")).to(x.dtype)
         state[sl[b], 0] = torch.cat((S.unsqueeze(0), xs[hi - lo:]), 0)

@@ -62,6 +62,11 @@ def test_slow_and_fast_decays(dtype, lam):
     M.recurrence_case(dtype, "cuda", lam_mean=lam)
 
 
+def test_slow_decays_keep_their_precision():
+    """Decays within 1e-5 of 1: rounding them would add up over the tokens."""
+    M.recurrence_case(F32, "cuda", 64, 2, 2, n=1500, lam_mean=-14.0, tol=2e-6)
+
+
 @pytest.mark.parametrize("dtype", [F32, BF16])
 @pytest.mark.parametrize("C,B,K", [(128, 2, 4), (60, 3, 3), (192, 1, 5)])
 def test_recurrence_batch(dtype, C, B, K):

@@ -53,6 +53,10 @@ def test_gated_recurrence(C, B, K):
     M.recurrence_case(F32, "cpu", C, B, K, n=150)
 
 
+def test_slow_decays_keep_their_precision():
+    M.recurrence_case(F32, "cpu", 16, 2, 2, n=600, lam_mean=-14.0, tol=2e-6)
+
+
 def test_recurrence_batch():
     M.recurrence_batch(F32, "cpu", 24, 2, 3)
 
