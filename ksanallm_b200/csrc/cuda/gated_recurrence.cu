@@ -396,7 +396,7 @@ recurrence_carry_kernel(RecurrenceArgs a, int seq_base, const float* __restrict_
   float* mem = a.state + static_cast<size_t>(a.slots[b]) * a.K * a.C + c;
   float S = fresh ? 0.f : mem[0];
   const int chunks = (n + TC - 1) / TC;
-  constexpr int U = 8;
+  constexpr int U = 16;
   for (int j0 = 0; j0 < chunks; j0 += U) {
     float s[U], d[U];
 #pragma unroll
