@@ -526,8 +526,10 @@ KSANA_API int ksana_recurrence_step(const void* y, int ldy, const void* x, int l
   if (B < 1 || C % B || K < 1) return -2;
   RecurrenceArgs a{y, ldy, x, ldx, state, slots, cu_q, kv_lens, conv_w, conv_b, gates_b, rate, out, ldo, C, K, B};
   if (!tile_sizes(a, gates)) return -1;
-  const int rc = K <= 4 ? launch_tile<RG_STEP, 4, true>(a, gates, seq_base, num_seqs, num_seqs, nullptr, nullptr, 0, st)
-                        : launch_tile<RG_STEP, 8, true>(a, gates, seq_base, num_seqs, num_seqs, nullptr, nullptr, 0, st);
+#define KSANA_RS(TC, KT) launch_tile<TC, KT, true>(a, gates, seq_base, num_seqs, num_seqs, nullptr, nullptr, 0, st)
+  // wide blocks: fewer CTAs load their gates (one CTA fills an SM's shared memory with them)
+  const int rc = K > 4 ? KSANA_RS(RG_STEP, 8) : C / B > 128 ? KSANA_RS(2 * RG_STEP, 4) : KSANA_RS(RG_STEP, 4);
+#undef KSANA_RS
   if (rc || C / B <= 128 || K == 1) return rc;
   recurrence_shift_kernel<<<dim3((C + 255) / 256, num_seqs), 256, 0, st>>>(a, seq_base);
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
