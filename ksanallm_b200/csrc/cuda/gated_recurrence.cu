@@ -120,7 +120,8 @@ struct RecurrenceSmem {
 
 // 1 / (1 + 2^x): the sigmoid of -x ln 2
 __device__ __forceinline__ float sigmoid_log2(float x) { return rcp_ftz(1.f + ex2_ftz(x)); }
-// l = log2 a <= 0 -> a - 1 and sqrt(1 - a^2). a - 1 = expm1(l ln 2) is a power series where the difference would cancel.
+// l = log2 a <= 0 -> a - 1 and sqrt(1 - a^2). a - 1 = e^(l ln 2) - 1 is its Taylor series
+// where the difference would cancel.
 __device__ __forceinline__ void decay_fast(float l, float* am1, float* in) {
   constexpr float c = 0.6931471805599453f;  // ln 2
   const float small = l * fmaf(l, fmaf(l, fmaf(l, c * c * c * c / 24.f, c * c * c / 6.f), c * c / 2.f), c);

@@ -1,6 +1,7 @@
 // Bandwidth-bound steps of layers with mixers of their own sizes: norms over a 32-bit residual stream, embedding into
 // that stream, GELU (gated or not), squared ReLU and clamped gates, the paged cache append (with per-head QK norm and
-// rotation, or beside the activation), the gated RMS norm behind linear attention, and the logit soft cap. Everything is computed in 32-bit floats; T is the storage type of activations.
+// rotation, or beside the activation), the gated RMS norm behind linear attention, and the logit soft cap. Everything is
+// computed in 32-bit floats; T is the storage type of activations.
 #include "host_common.h"
 #include "mixer_common.cuh"
 

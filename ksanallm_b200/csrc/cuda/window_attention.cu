@@ -176,7 +176,7 @@ struct WindowPrefillSmem {
 };
 
 // The cap of a score, in units where exp2 is the exponential: s -> c tanh(s / c) with c in those units. Tiles whose scores
-// are small against the cap take a polynomial, odd to degree 11 (error below 1e-7 of the cap up to |s / c| = 0.4); others
+// are small against the cap take the Taylor series of tanh to degree 11 (error below 1e-7 of the cap up to |s / c| = 0.4); others
 // the exponential form.
 constexpr float CAP_POLY = 0.4f;
 // two 32-bit floats in one register pair; FMAs on them issue as one
