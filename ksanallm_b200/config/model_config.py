@@ -44,10 +44,12 @@ class QuantConfig:
 
 @dataclass
 class RotarySpec:
-    """Rotation of the leading ``dims`` dimensions of q and k, neighbouring entries (2i, 2i + 1) being a pair."""
+    """Rotation of the leading ``dims`` dimensions of q and k, neighbouring entries (2i, 2i + 1) being a pair, or the
+    entries i and i + dims / 2 (``halves``)."""
     dims: int
     base: float
     scaling: RopeScaling = field(default_factory=RopeScaling)
+    halves: bool = False
 
 
 @dataclass
@@ -71,6 +73,11 @@ class AttentionSpec:
     head_gate: bool = False  # each head's output times the sigmoid of a number of its own, projected from the mixer's input
     o_bias: bool = False
     kv_from: Optional[int] = None  # reads the keys and values of that earlier layer: no projections, no cache of its own
+    qk_norm_all: bool = False  # RMS norm of q (and of k) over all heads together, ahead of the rotation
+    # every head's softmax weights become a learned mix of all heads' weights (talking heads); the softmax's denominator
+    # has one more term exp(s) with a learned s per head
+    talk: bool = False
+    out_gate: bool = False  # the heads' output times sigmoid of a projection of the mixer's input, number by number
 
 
 @dataclass
@@ -120,6 +127,17 @@ class LinearAttentionSpec:
 
 
 @dataclass
+class TimeMixSpec:
+    """A linear recurrence whose decay is a function of the token, per head and key channel: o = (S + diag(u) k v^T)^T r,
+    then S <- diag(w) S + k v^T. Its five inputs read the token's own vector moved towards the previous token's, each by a
+    learned amount per coordinate; w = exp(-exp(.)) comes out of a low-rank map."""
+    heads: int
+    dim: int
+    width: int               # of the model: the state also holds the previous token's vector
+    out_scale: float = 1.0
+
+
+@dataclass
 class ExpertsSpec:
     """A mixture of gated experts: the ``top`` largest router logits choose, and the softmax over the chosen logits weights
     them (which is the softmax over all experts, divided by the chosen ones' sum). With ``groups`` > 1, equal groups of
@@ -135,6 +153,11 @@ class ExpertsSpec:
     keep: int = 1
     limit: float = 0.0
     alpha: float = 1.0
+    plain: bool = False      # an expert is down(relu(up)^2): no gate
+    # sigmoid: the weights are the chosen logits' sigmoids times ``scale``, not normalised
+    scoring: str = "softmax"
+    scale: float = 1.0
+    shared_ff: int = 0       # a shared expert beside the routed ones, times the sigmoid of one number per token (0: none)
 
 
 @dataclass
@@ -143,6 +166,7 @@ class LayerSpec:
     which is dense (``ff``), routed (``moe``) or absent."""
     attn: Optional[AttentionSpec] = None
     linear: Optional[LinearAttentionSpec] = None
+    timemix: Optional[TimeMixSpec] = None
     latent: Optional[LatentAttentionSpec] = None
     recurrence: Optional[RecurrenceSpec] = None
     ff: int = 0              # dense feed-forward width (0: none)
@@ -152,9 +176,15 @@ class LayerSpec:
     ff_bias: bool = False    # biases of the dense feed-forward's projections
     ff_act: str = ""         # its activation ("": the model's)
     layer_scale: bool = False  # each sublayer's result times a learned vector
+    # mixers and feed-forward run side by side over norms of their own of the same stream, and each one's result is
+    # multiplied, number by number, by the sigmoid of a map of what it read
+    gated_residual: bool = False
 
     @property
     def state_shape(self):
+        if self.timemix is not None:  # every head's state [key][value], then the previous token's vector
+            t = self.timemix
+            return (1, 1, t.heads * t.dim * t.dim + t.width)
         if self.recurrence is not None:  # the recurrent state, then the convolution's last inputs, oldest first
             return (1, self.recurrence.taps, self.recurrence.width)
         return (self.linear.heads, self.linear.dim, self.linear.vdim) if self.linear else None
@@ -546,8 +576,45 @@ def _ladusun_config(c: Dict[str, Any]) -> ModelConfig:
     return m
 
 
+def _vibunex_layer(entry: Dict[str, Any], width: int) -> LayerSpec:
+    if str(entry["type"]) != "parallel":
+        raise ValueError(f"unknown Vibunex layer type {entry['type']!r}")
+    c, mlp = entry["mixer"], entry.get("mlp")
+    a, r = c["left"], c["right"]
+    rot = _ladusun_rotary(a["rot"], "yarn")
+    rot.halves = True
+    spec = LayerSpec(
+        parallel=True, gated=False, gated_residual=True,
+        attn=AttentionSpec(int(a["heads"]), int(a["kv_heads"]), int(a["dim"]), int(a["vdim"]), float(a["scale"]), rot=rot,
+                           out_scale=float(c["left_scale"]), qk_norm_all=True, talk=True, out_gate=True),
+        timemix=TimeMixSpec(int(r["heads"]), int(r["dim"]), width, float(c["right_scale"])))
+    if spec.attn.heads % spec.attn.kv_heads or rot.dims > spec.attn.dim or rot.dims % 2:
+        raise ValueError("heads are a multiple of kv_heads, and pairs of at most a whole head are rotated")
+    if mlp is not None:
+        if str(mlp.get("kind", "moe")) != "moe":
+            raise ValueError(f"unknown Vibunex feed-forward {mlp.get('kind')!r}")
+        q = mlp["router"]
+        spec.moe = ExpertsSpec(int(q["experts"]), int(q["top"]), int(mlp["expert"]["ff"]), plain=True, scoring="sigmoid",
+                               scale=float(q["scale"]), shared_ff=int(mlp["shared"]["ff"]))
+        if not 1 <= spec.moe.top <= spec.moe.experts:
+            raise ValueError("router.top must lie between 1 and router.experts")
+    return spec
+
+
+def _vibunex_config(c: Dict[str, Any]) -> ModelConfig:
+    """Vibunex: attention whose heads' weights are mixed, beside time mixing with token-dependent decays, beside routed
+    squared-ReLU experts and a shared one; sublayers gated into one scaled residual; norms with one number; untied head."""
+    m = _layered_config(c, "vibunex")
+    _set_layers(m, [_vibunex_layer(e, m.hidden_size) for e in c["layers"]])
+    m.residual_scale = float(c["residual_mult"])
+    m.position_encoding, m.gated_mlp = "none", False
+    m.max_position_embeddings = int(c.get("max_position_embeddings", 1 << 20))
+    return m
+
+
 def model_config_from_dict(c: Dict[str, Any]) -> ModelConfig:
-    design = {"molopel": _molopel_config, "givirax": _givirax_config, "ladusun": _ladusun_config}.get(str(c.get("architecture", "")).lower())
+    design = {"molopel": _molopel_config, "givirax": _givirax_config, "ladusun": _ladusun_config,
+              "vibunex": _vibunex_config}.get(str(c.get("architecture", "")).lower())
     if design is not None:
         return design(c)
     if isinstance(c.get("text_config"), dict) and str(c.get("model_type", "")).lower() in ("llama4",):
@@ -915,7 +982,31 @@ def tiny_ladusun_config() -> ModelConfig:
     return cfg
 
 
+def vibunex_config(width: int = 4096, layers: int = 8, experts: int = 16, top: int = 2, expert_ff: int = 4096,
+                   shared_ff: int = 4096, heads: int = 32, kv_heads: int = 8, dim: int = 128, mix_heads: int = 64,
+                   mix_dim: int = 64, vocab: int = 32000) -> ModelConfig:
+    """Vibunex at the sizes of an ordinary decoder of that width."""
+    layer = dict(type="parallel", mixer=dict(
+        left=dict(heads=heads, kv_heads=kv_heads, dim=dim, vdim=dim, scale=dim ** -0.5, rot=dict(
+            dims=dim // 2, base=5e5, scaling=dict(factor=4.0, original=8192, fast=32.0, slow=1.0))),
+        right=dict(heads=mix_heads, dim=mix_dim), left_scale=0.7, right_scale=0.7),
+        mlp=dict(kind="moe", expert=dict(ff=expert_ff), router=dict(experts=experts, top=top, scale=1.5),
+                 shared=dict(ff=shared_ff)))
+    return model_config_from_dict(dict(
+        architecture="Vibunex", norm=dict(eps=1e-6), vocab=vocab, width=width, residual_mult=0.5,
+        layers=[json.loads(json.dumps(layer)) for _ in range(layers)], eos_token_id=2))
+
+
+def tiny_vibunex_config() -> ModelConfig:
+    cfg = vibunex_config(width=128, layers=3, experts=6, expert_ff=48, shared_ff=80, heads=4, kv_heads=2, dim=32,
+                         mix_heads=3, mix_dim=24)
+    cfg.torch_dtype = "float32"
+    return cfg
+
+
 NAMED_CONFIGS = {
+    "tiny-vibunex": tiny_vibunex_config,
+    "vibunex": vibunex_config,
     "tiny-ladusun": tiny_ladusun_config,
     "ladusun": ladusun_config,
     "tiny-givirax": tiny_givirax_config,

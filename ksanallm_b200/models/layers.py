@@ -409,24 +409,27 @@ class MoEFFN:
             y = y + s
         return y
 
-    def route(self, h: torch.Tensor):
+    def route(self, h: torch.Tensor, logits: Optional[torch.Tensor] = None):
         """Expert ids [T, k] (as the expert kernels count them) and fp32 weights [T, k] of the rows of ``h``."""
         c = self.cfg
-        if c.scoring_func == "topk_softmax":
-            # softmax over the chosen logits only, which stay in 32-bit
-            ids, wts = ops.moe_topk(ops.linear(h, self.gate_w, None, torch.float32), c.num_experts,
-                                    c.num_experts_per_tok, self.logit_bias, c.n_group, c.topk_group)
+        if c.scoring_func in ("topk_softmax", "topk_sigmoid"):
+            # softmax over the chosen logits only, or each one's sigmoid; the logits stay in 32-bit
+            z = ops.linear(h, self.gate_w, None, torch.float32) if logits is None else logits
+            ids, wts = ops.moe_topk(z, c.num_experts, c.num_experts_per_tok, self.logit_bias, c.n_group, c.topk_group,
+                                    c.scoring_func[5:], c.routed_scaling_factor)
         else:
             logits = ops.linear(h.float() if self.gate_w.dtype == torch.float32 else h, self.gate_w)
             ids, wts = ops.moe_route(logits, c.num_experts_per_tok, c.scoring_func, c.norm_topk_prob, c.n_group,
                                      c.topk_group, c.routed_scaling_factor, self.bias)
         return self._place(ids), wts
 
-    def rows(self, h: torch.Tensor, limit: float = 0.0, alpha: float = 1.0):
+    def rows(self, h: torch.Tensor, limit: float = 0.0, alpha: float = 1.0, plain: bool = False,
+             logits: Optional[torch.Tensor] = None):
         """The routed sum in the form a norm over the stream takes: (unweighted rows of the experts, the row of every
-        (token, slot) pair, weights [T, k]). Unquantised local experts without a shared one; ``limit`` > 0: clamped ones."""
-        ids, wts = self.route(h)
-        y, pos = ops.moe_expert_rows(h, ids, self.w_gate_up, self.w_down, limit, alpha)
+        (token, slot) pair, weights [T, k]). Unquantised local experts without a shared one; ``limit`` > 0: clamped ones;
+        ``plain``: ungated ones. ``logits``: the router's, where they are there already (topk_softmax, topk_sigmoid)."""
+        ids, wts = self.route(h, logits)
+        y, pos = ops.moe_expert_rows(h, ids, self.w_gate_up, self.w_down, limit, alpha, plain)
         return y, pos, wts
 
     def _grouped_fp8(self, h: torch.Tensor) -> bool:

@@ -70,6 +70,17 @@ _RENAMES: Dict[str, List[Tuple[str, str]]] = {
                 (r"^l(\d+)\.mlp\.(up|down)\.b$", r"model.layers.\1.mlp.\2_proj.bias"),
                 (r"^l(\d+)\.mlp\.e(\d+)\.(gate|up|down)$", r"model.layers.\1.mlp.experts.\2.\3_proj.weight"),
                 (r"^l(\d+)\.mlp\.router$", r"model.layers.\1.mlp.gate.weight")],
+    "vibunex": [(r"^embed$", "model.embed_tokens.weight"), (r"^final\.norm$", "model.norm.weight"),
+                (r"^head$", "lm_head.weight"),
+                (r"^l(\d+)\.norm1$", r"model.layers.\1.input_layernorm.weight"),
+                (r"^l(\d+)\.norm2$", r"model.layers.\1.post_attention_layernorm.weight"),
+                (r"^l(\d+)\.mix\.", r"model.layers.\1.mixer."),
+                (r"^l(\d+)\.rg1", r"model.layers.\1.mixer.rg"),
+                (r"^l(\d+)\.rg2$", r"model.layers.\1.mlp.rg.weight"), (r"^l(\d+)\.rg2\.b$", r"model.layers.\1.mlp.rg.bias"),
+                (r"^l(\d+)\.mlp\.e(\d+)\.(up|down)$", r"model.layers.\1.mlp.experts.\2.\3_proj.weight"),
+                (r"^l(\d+)\.mlp\.shared\.(up|down)$", r"model.layers.\1.mlp.shared_expert.\2_proj.weight"),
+                (r"^l(\d+)\.mlp\.shared\.sg$", r"model.layers.\1.mlp.shared_expert_gate.weight"),
+                (r"^l(\d+)\.mlp\.router$", r"model.layers.\1.mlp.gate.weight")],
     "baichuan": [(r"\.W_pack\.", ".wpack.")],
     "chatglm": [(r"^transformer\.embedding\.word_embeddings\.", "model.embed_tokens."),
                 (r"^transformer\.encoder\.layers\.", "model.layers."),
@@ -408,10 +419,11 @@ def _kv_rows(t: torch.Tensor, rank: int, size: int, num_kv_heads: int, d: int) -
 
 
 def mixer_prefixes(spec: LayerSpec) -> Tuple[Optional[str], Optional[str]]:
-    """Checkpoint prefixes of a layer's attention and linear-attention tensors (None: the layer has no such mixer)."""
-    both = spec.attn is not None and spec.linear is not None
-    return (("left." if both else "") if spec.attn is not None else None,
-            ("right." if both else "") if spec.linear is not None else None)
+    """Checkpoint prefixes of a layer's attention and linear-attention or time-mixing tensors (None: the layer has no such
+    mixer)."""
+    other = spec.linear is not None or spec.timemix is not None
+    both = spec.attn is not None and other
+    return (("left." if both else "") if spec.attn is not None else None, ("right." if both else "") if other else None)
 
 
 def mixer_parts(spec: LayerSpec) -> set:
@@ -426,9 +438,11 @@ def mixer_parts(spec: LayerSpec) -> set:
             need |= {f"{pa}{x}.b" for x in proj}
         if a.o_bias:
             need.add(pa + "o.b")
-        if a.head_gate:
+        if a.head_gate or a.out_gate:
             need.add(pa + "g")
-        if a.qk_norm:
+        if a.talk:
+            need |= {pa + "talk", pa + "sink"}
+        if a.qk_norm or a.qk_norm_all:
             need |= {pa + "q.norm", pa + "k.norm"}
         if a.bias_max:
             need.add(pa + "rel")
@@ -440,8 +454,24 @@ def mixer_parts(spec: LayerSpec) -> set:
         need |= {pl + x for x in "qkvgo"}
         if spec.linear.norm == "concat":
             need.add(pl + "norm")
+    if spec.timemix is not None:
+        need |= {pl + x for x in ("r", "k", "v", "g", "w1", "w2", "w0", "u", "norm", "o")} | {f"{pl}mu.{x}" for x in "rkvgw"}
+    if spec.gated_residual:
+        need |= {"rg", "rg.b"}
     if spec.parallel and spec.ff:  # a dense feed-forward beside the mixers shares their projections
         need |= {"ff." + x for x in (("gate", "up", "down") if spec.gated else ("up", "down"))}
+    return need
+
+
+def moe_parts(spec: LayerSpec) -> set:
+    """Names of the tensors around a layer's routed experts, below the layer's feed-forward prefix."""
+    need = {"gate.weight"}
+    if spec.moe.router_bias:
+        need.add("gate.bias")
+    if spec.moe.shared_ff:
+        need |= {"shared_expert.up_proj.weight", "shared_expert.down_proj.weight", "shared_expert_gate.weight"}
+    if spec.gated_residual:
+        need |= {"rg.weight", "rg.bias"}
     return need
 
 
@@ -449,7 +479,7 @@ def layer_parts(cfg: ModelConfig, i: int) -> set:
     """Names of the tensors that surround a layer's mixers and feed-forward."""
     spec, p = cfg.layers[i], f"model.layers.{i}"
     need = {p + ".input_layernorm.weight"}
-    if spec.has_ff and not spec.parallel:
+    if spec.has_ff and (not spec.parallel or spec.gated_residual):
         need.add(p + ".post_attention_layernorm.weight")
     for n in (1, 2) if spec.has_ff else (1,):
         if spec.layer_scale:
@@ -471,9 +501,14 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
             yield m + pa + x, rnd(n, H)
             if a.qkv_bias:
                 yield f"{m}{pa}{x}.b", rnd(n)
-        if a.qk_norm:
-            yield m + pa + "q.norm", ones(a.dim)
-            yield m + pa + "k.norm", ones(a.dim)
+        if a.qk_norm or a.qk_norm_all:
+            yield m + pa + "q.norm", ones(a.dim * (a.heads if a.qk_norm_all else 1))
+            yield m + pa + "k.norm", ones(a.dim * (a.kv_heads if a.qk_norm_all else 1))
+        if a.talk:
+            yield m + pa + "talk", rnd(a.heads, a.heads)
+            yield m + pa + "sink", rnd(a.heads)
+        if a.out_gate:
+            yield m + pa + "g", rnd(a.heads * a.vdim, H)
         if a.bias_max:
             yield m + pa + "rel", rnd(32, a.heads)
         if a.head_gate:
@@ -504,6 +539,22 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
             yield f"{m}{x}.b", rnd(B, C // B)
         yield m + "lam", rnd(C)
         yield m + "o", rnd(H, C)
+    if spec.timemix is not None:
+        r = spec.timemix
+        n, rank = r.heads * r.dim, max(r.dim, 32)
+        for x in "rkvg":
+            yield m + pl + x, rnd(n, H)
+        for x in "rkvgw":
+            yield f"{m}{pl}mu.{x}", rnd(H)
+        yield m + pl + "w1", rnd(rank, H)
+        yield m + pl + "w2", rnd(n, rank)
+        yield m + pl + "w0", rnd(n)
+        yield m + pl + "u", rnd(r.heads, r.dim)
+        yield m + pl + "norm", ones(n)
+        yield m + pl + "o", rnd(H, n)
+    if spec.gated_residual:
+        yield m + "rg", rnd(H, H)
+        yield m + "rg.b", rnd(H)
     if spec.linear is not None:
         r = spec.linear
         for x, n in (("q", r.dim), ("k", r.dim), ("v", r.vdim), ("g", r.vdim)):
@@ -516,7 +567,7 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
             yield f"{m}ff.{x}", rnd(spec.ff, H)
         yield m + "ff.down", rnd(H, spec.ff)
         return
-    if spec.has_ff and not spec.parallel:
+    if spec.has_ff and (not spec.parallel or spec.gated_residual):
         yield p + ".post_attention_layernorm.weight", ones(H)
     if spec.layer_scale:
         for n in (1, 2) if spec.has_ff else (1,):
@@ -526,8 +577,16 @@ def _synthetic_mixer_layer(spec: LayerSpec, p: str, H: int, rnd, ones) -> Iterat
         yield p + ".mlp.gate.weight", rnd(e.experts, H)
         if e.router_bias:
             yield p + ".mlp.gate.bias", rnd(e.experts)
+        if spec.gated_residual:
+            yield p + ".mlp.rg.weight", rnd(H, H)
+            yield p + ".mlp.rg.bias", rnd(H)
+        if e.shared_ff:
+            yield p + ".mlp.shared_expert.up_proj.weight", rnd(e.shared_ff, H)
+            yield p + ".mlp.shared_expert.down_proj.weight", rnd(H, e.shared_ff)
+            yield p + ".mlp.shared_expert_gate.weight", rnd(1, H)
         for i in range(e.experts):
-            yield f"{p}.mlp.experts.{i}.gate_proj.weight", rnd(e.ff, H)
+            if not e.plain:
+                yield f"{p}.mlp.experts.{i}.gate_proj.weight", rnd(e.ff, H)
             yield f"{p}.mlp.experts.{i}.up_proj.weight", rnd(e.ff, H)
             yield f"{p}.mlp.experts.{i}.down_proj.weight", rnd(H, e.ff)
     if spec.ff:
@@ -740,7 +799,7 @@ class WeightLoader:
             return
         if name.startswith("model.norm.") or "layernorm" in name or name.endswith("norm.weight") \
                 or name.endswith("norm.bias") or ".enorm." in name or ".hnorm." in name:
-            self._put(name, t)
+            self._put(name, t.reshape(1).expand(cfg.hidden_size) if cfg.layers and t.dim() == 0 else t)  # (one number for all)
             return
         if ".self_attn.indexer." in name:
             # sparse-attention indexer (DeepSeek-V3.2 / GLM DSA): small replicated projections; block-scaled fp8
@@ -942,8 +1001,8 @@ class WeightLoader:
                                             (self._have(p, pre + "up_proj_t", b) and self._have(p, pre + "down_proj_t", b))))
             if moe:
                 ok = "gate.weight" in p
-                if cfg.layers and cfg.layers[li].moe.router_bias:
-                    ok = ok and "gate.bias" in p
+                if cfg.layers:
+                    ok = not moe_parts(spec) - set(p)
                 if cfg.topk_method == "noaux_tc":
                     ok = ok and "gate.e_score_correction_bias" in p
                 if cfg.num_shared_experts:
@@ -960,7 +1019,8 @@ class WeightLoader:
         experts = self._num_experts(key)
         per = max(experts // max(self.ep_size, 1), 1) if self.ep_size > 1 else experts
         first = next(iter(ex.values()))
-        want = per * 3 * (2 if any(self._fp8(t) for t in ex.values()) else 1)
+        plain = self.cfg.layers and self.cfg.layers[self._layer_of(key + ".")].moe.plain
+        want = per * (2 if plain else 3) * (2 if any(self._fp8(t) for t in ex.values()) else 1)
         if len(ex) >= want:
             self._finish_experts(key, self._experts.pop(key))
 
@@ -984,8 +1044,12 @@ class WeightLoader:
                 if spec is not None and spec.ff:
                     need = {f"{x}_proj.{y}" for x in (("gate", "up", "down") if spec.gated else ("up", "down"))
                             for y in (("weight", "bias") if spec.ff_bias else ("weight",))}
-                    if need - set(parts):
-                        raise KeyError(f"{key}: the checkpoint has no {', '.join(sorted(need - set(parts)))}")
+                elif spec is not None and spec.moe is not None:
+                    need = moe_parts(spec)
+                else:
+                    need = set()
+                if need - set(parts):
+                    raise KeyError(f"{key}: the checkpoint has no {', '.join(sorted(need - set(parts)))}")
                 self._finish_mlp(key, parts)
         for key, ex in list(self._experts.items()):
             self._finish_experts(key, ex)
@@ -1026,7 +1090,7 @@ class WeightLoader:
         if spec.attn is not None:
             a = spec.attn
             names += [pa + x for x in ("q" if a.kv_from is not None else "qk" if a.shared_kv else "qkv")]
-            names += [pa + "g"] if a.head_gate else []
+            names += [pa + "g"] if a.head_gate or a.out_gate else []
             outs.append(pa + "o")
         if spec.latent is not None:
             names += ["q", "dkv"] + (["g"] if spec.latent.head_gate else [])
@@ -1037,6 +1101,11 @@ class WeightLoader:
         if spec.linear is not None:
             names += [pl + x for x in "qkvg"]
             outs.append(pl + "o")
+        if spec.timemix is not None:  # (its inputs are mixes of two tokens': projections of their own)
+            outs.append(pl + "o")
+            self._finish_timemix(key, pl, p)
+        if spec.gated_residual:
+            names.append("rg")
         if spec.parallel and spec.ff:
             names += ["ff.gate", "ff.up"] if spec.gated else ["ff.up"]
             outs.append("ff.down")
@@ -1054,7 +1123,8 @@ class WeightLoader:
             a = spec.latent
             self._put(key + ".w_uk", p["uk"].view(a.heads, a.dim, a.rank))
             self._put(key + ".w_uv", p["uv"].view(a.heads, a.vdim, a.rank))
-        f32 = [(pa, "q.norm", "q_norm"), (pa, "k.norm", "k_norm"), (pa, "rel", "rel"), (pl, "norm", "norm")]
+        f32 = [(pa, "q.norm", "q_norm"), (pa, "k.norm", "k_norm"), (pa, "rel", "rel"), (pl, "norm", "norm"),
+               (pa, "talk", "talk"), (pa, "sink", "sink"), (pl, "u", "u"), (pl, "w0", "w0")]
         if spec.latent is not None:
             f32.append(("", "dkv.norm", "latent_norm"))
         if spec.recurrence is not None:
@@ -1064,6 +1134,20 @@ class WeightLoader:
         for pre, name, out in f32:
             if pre is not None and pre + name in p:
                 self.out[f"{key}.{out}"] = self._own(p[pre + name].float())
+
+    def _finish_timemix(self, key: str, pre: str, p: Dict[str, torch.Tensor]) -> None:
+        """Time mixing's projections: r, k, v and gate as one stack, and the two maps of the decay. Their rows are
+        zero-padded to the multiples of eight that the GEMM takes."""
+        pad = torch.nn.functional.pad
+        stack = torch.stack([p[pre + x] for x in "rkvg"])
+        self._put(key + ".mix_proj", pad(stack, (0, 0, 0, -stack.shape[1] % 8)))
+        w1, w2 = p[pre + "w1"], p[pre + "w2"]
+        rank = -w1.shape[0] % 8
+        self._put(key + ".w1", pad(w1, (0, 0, 0, rank)))
+        # twice along the input: the tanh in front of it arrives as two 16-bit parts
+        w2 = pad(w2, (0, rank, 0, -w2.shape[0] % 8))
+        self._put(key + ".w2", torch.cat((w2, w2), 1) if self.dtype != torch.float32 else w2)
+        self.out[key + ".mu"] = self._own(torch.stack([p[f"{pre}mu.{x}"].float() for x in "rkvgw"]))
 
     def _finish_attn(self, key: str, p: Dict[str, torch.Tensor]) -> None:
         cfg, r, n = self.cfg, self.rank, self.size
@@ -1177,6 +1261,11 @@ class WeightLoader:
                 if pre + "up_proj.bias" in p:
                     p[pre + "up_proj.bias"] = pad(p[pre + "up_proj.bias"], (0, extra))
             gs, us, ds = (p.get(pre + f"{x}_proj.weight_scale_inv") for x in ("gate", "up", "down"))
+            if pre and cfg.layers and "rg.weight" in p:  # beside the residual gate, which reads the same input
+                self._put_linear(f"{key}.in_proj", torch.cat((p["rg.weight"], up), 0))
+                self._put(f"{key}.in_proj.bias", torch.cat((p["rg.bias"], up.new_zeros(up.shape[0])), 0))
+                self._put_linear(f"{key}.{pre}down_proj", down)
+                continue
             if gate is not None:
                 fused = _cat0((_rows(gate, r, n), _rows(up, r, n)))
                 fs = None if gs is None else torch.cat((_rows(gs, r, n), _rows(us, r, n)), 0)
@@ -1193,6 +1282,8 @@ class WeightLoader:
         if "gate.weight" in p:
             gate = p["gate.weight"]
             if cfg.layers:  # (the padding rows are no experts: the router looks at the first ones only)
+                if "shared_expert_gate.weight" in p:  # the row behind the experts': the shared expert's gate
+                    gate = torch.cat((gate, p.pop("shared_expert_gate.weight")), 0)
                 gate = torch.nn.functional.pad(gate, (0, 0, 0, -gate.shape[0] % 8))
             self._put(f"{key}.gate.weight", gate, keep_dtype=gate.dtype == torch.float32)
         if "gate.bias" in p:
@@ -1204,7 +1295,7 @@ class WeightLoader:
 
     def _finish_experts(self, key: str, ex: Dict[Tuple[int, str], torch.Tensor]) -> None:
         ids = sorted({e for e, _ in ex})
-        if isinstance(ex[(ids[0], "gate_proj.weight")], QuantW):
+        if isinstance(ex[(ids[0], "down_proj.weight")], QuantW):
             # GPTQ / AWQ experts: stacked packed words + group scales / zeros, [gate | up] rows fused per expert
             gus = [QuantW.cat0((ex[(e, "gate_proj.weight")], ex[(e, "up_proj.weight")])) for e in ids]
             dns = [ex[(e, "down_proj.weight")] for e in ids]
@@ -1216,14 +1307,17 @@ class WeightLoader:
             return
         has_scale = (ids[0], "gate_proj.weight_scale_inv") in ex
         if self.cfg.layers:
-            want = {(e, x + "_proj.weight") for e in range(self._num_experts(key)) for x in ("gate", "up", "down")}
+            plain = self.cfg.layers[self._layer_of(key + ".")].moe.plain
+            stems = ("up", "down") if plain else ("gate", "up", "down")
+            want = {(e, x + "_proj.weight") for e in range(self._num_experts(key)) for x in stems}
             if want - set(ex):
                 raise KeyError(f"{key}: the checkpoint has no experts.{min(want - set(ex))[0]}.{min(want - set(ex))[1]}")
             extra = -ex[(0, "down_proj.weight")].shape[1] % 8  # zero columns up to the multiple of eight the GEMM takes
             if extra and not has_scale:
                 pad = torch.nn.functional.pad
                 ex = {(e, x): pad(t, (0, extra) if x[0] == "d" else (0, 0, 0, extra)) for (e, x), t in ex.items()}
-        gu = torch.stack([torch.cat((ex[(e, "gate_proj.weight")], ex[(e, "up_proj.weight")]), 0) for e in ids])
+        gu = torch.stack([torch.cat([ex[(e, x)] for x in ("gate_proj.weight", "up_proj.weight") if (e, x) in ex], 0)
+                          for e in ids])
         dn = torch.stack([ex[(e, "down_proj.weight")] for e in ids])
         if has_scale:
             self.out[f"{key}.experts.up_gate_proj.weight"] = gu.to(self.device).contiguous()

@@ -1,7 +1,8 @@
 """Layers whose sequence mixers have sizes of their own, described by :class:`LayerSpec`: softmax attention over a
 window or everything (with rotation, a learned distance bias, first tokens that stay visible, values that are the keys,
-capped scores, a sink, a gate per head, or another layer's keys and values), latent attention, a gated linear recurrence,
-and linear attention with a fixed decay per head, alone or beside windowed attention.
+capped scores, a sink, a gate per head, another layer's keys and values, or weights that are mixed across heads), latent
+attention, a gated linear recurrence, linear attention with a fixed decay per head, and time mixing with token-dependent
+decays, the last two alone or beside attention.
 
 All mixers of a layer read the same normalised input, so their input projections are one GEMM and their outputs go
 into one buffer that a single output projection reads. A dense feed-forward that reads that input too (``parallel``) is
@@ -9,7 +10,9 @@ part of the same two GEMMs. A layer's cache is the pair (paged keys / values or 
 tensor where the layer does not have that mixer. A layer that runs several times has one :class:`MixerLayer` per run, over
 the same weights.
 
-Where the model has ``streams``, the residual is [T, streams, H] and each sublayer has a :class:`HyperConnection`.
+Where the model has ``streams``, the residual is [T, streams, H] and each sublayer has a :class:`HyperConnection`. Where
+a layer's sublayers are gated into the residual (``gated_residual``), its normalised input is [1 or 2, T, H]: one norm for the
+mixers, one for the feed-forward.
 """
 from __future__ import annotations
 
@@ -20,7 +23,7 @@ import torch
 
 from .. import ops
 from ..config.model_config import (AttentionSpec, LatentAttentionSpec, LayerSpec, LinearAttentionSpec, ModelConfig,
-                                   RecurrenceSpec, RotarySpec)
+                                   RecurrenceSpec, RotarySpec, TimeMixSpec)
 from ..ops import reference as ref
 from .layers import DenseFFN, LinearW, MoEFFN
 
@@ -70,8 +73,11 @@ class WindowedAttention:
         self.page = self.nk + self.nv  # cache elements per token
         if spec.kv_from is not None:
             self.nk = self.nv = 0
-        self.rows = self.nq + self.nk + self.nv + (spec.heads if spec.head_gate else 0)
         self.width = spec.heads * spec.vdim
+        self.rows = self.nq + self.nk + self.nv + (spec.heads if spec.head_gate else self.width if spec.out_gate else 0)
+        if spec.talk and (spec.window or spec.bias_max or spec.shared_kv or spec.softcap or spec.sink or spec.head_gate):
+            raise NotImplementedError("weights are mixed across heads in attention to all keys with plain scores")
+        self.talk, self.sink = w.get(prefix + ".talk"), w.get(prefix + ".sink")
         self.q_norm, self.k_norm = w.get(prefix + ".q_norm"), w.get(prefix + ".k_norm")
         self.rel = w.get(prefix + ".rel")
         self.bias: Optional[torch.Tensor] = None  # [heads, reach]: the bias of every distance a query can see
@@ -100,7 +106,11 @@ class WindowedAttention:
             v = x[:, self.nq + self.nk:end].unflatten(1, (s.kv_heads, s.vdim)) if self.nk else None
             if k is not None or s.rot is not None or self.q_norm is not None:
                 ops.qk_norm_cache(q, k, v, meta.slot_mapping, kv, bs, self.q_norm, self.k_norm, self.eps, meta.positions,
-                                  self.rotary())
+                                  self.rotary(), s.qk_norm_all, s.rot is not None and s.rot.halves)
+        if s.talk:
+            ops.talking_attention(q, kv, meta, bs, s.kv_heads, s.vdim, s.scale, self.sink, self.talk, s.out_scale, out,
+                                  x[:, end:end + self.width] if s.out_gate else None)
+            return
         ops.window_attention(q, kv, meta, bs, s.kv_heads, s.vdim, s.scale, s.window, self.bias, s.out_scale, out,
                              s.keep_first, s.softcap, s.sink, x[:, end:end + s.heads] if s.head_gate else None)
 
@@ -191,6 +201,25 @@ class DecayedLinearAttention:
         ops.gated_norm(o, g, self.norm, self.eps, s.gate, s.out_scale, out)
 
 
+class TimeMixing:
+    def __init__(self, cfg: ModelConfig, spec: TimeMixSpec, w: Dict[str, torch.Tensor], prefix: str):
+        self.spec, self.eps = spec, cfg.rms_norm_eps
+        self.rows, self.width = 0, spec.heads * spec.dim
+        self.mu, self.proj = w[prefix + ".mu"], w[prefix + ".mix_proj"]  # [5, W] fp32 (r, k, v, gate, decay), [4, n, W]
+        self.w1, self.w2, self.w0 = w[prefix + ".w1"], w[prefix + ".w2"], w[prefix + ".w0"]
+        self.u, self.norm = w[prefix + ".u"].contiguous(), w[prefix + ".norm"]
+
+    def run(self, h: torch.Tensor, meta, state: torch.Tensor, out: torch.Tensor) -> None:
+        """h [T, W] = the mixer's input; writes heads * dim columns of ``out``."""
+        n = self.width
+        m = ops.token_mix(h, self.mu, state, meta)
+        r, k, v, g = (ops.linear(m[i], self.proj[i])[:, :n] for i in range(4))
+        t = ops.tanh_parts(ops.linear(m[4], self.w1, None, torch.float32), h.dtype)
+        z = ops.linear(t, self.w2, None, torch.float32)[:, :n]
+        o = ops.time_mix(r, k, v, z, self.w0, self.u, state, meta)
+        ops.gated_norm(o, g, self.norm, self.eps, "silu", self.spec.out_scale, out, per_head=True)
+
+
 class PassStart(NamedTuple):
     """What the stream takes ahead of one pass of a loop."""
     step: torch.Tensor      # [H] fp32, the pass's learned vector
@@ -207,7 +236,8 @@ class HyperConnection:
 
 class MixerLayer:
     """One run of a layer: x <- x + mixers(norm1(x)); x <- x + ff(norm2(x)) unless the layer has no feed-forward; or, in
-    parallel, h = norm1(x); x <- x + (mixers(h) + ff(h))."""
+    parallel, h = norm1(x); x <- x + (mixers(h) + ff(h)); or, with a gated residual, x <- x + scale * (mixers(norm1(x)) *
+    gate1 + ff(norm2(x)) * gate2)."""
 
     def __init__(self, cfg: ModelConfig, w: Dict[str, torch.Tensor], idx: int, tp, tables: RotaryTables,
                  number: Optional[int] = None):
@@ -226,6 +256,7 @@ class MixerLayer:
         self.attn = WindowedAttention(cfg, spec.attn, w, p + ".mixer", tables) if spec.attn else None
         self.latent = LatentAttention(cfg, spec.latent, w, p + ".mixer", tables) if spec.latent else None
         self.recurrence = GatedRecurrence(cfg, spec.recurrence, w, p + ".mixer") if spec.recurrence else None
+        self.timemix = TimeMixing(cfg, spec.timemix, w, p + ".mixer") if spec.timemix else None
         self.linear = DecayedLinearAttention(cfg, spec.linear, w, p + ".mixer", device, tables) if spec.linear else None
         self.hyper = [HyperConnection(w, f"{p}.hc{n}") for n in ((1, 2) if spec.has_ff else (1,))] if cfg.streams else []
         self.ls1, self.ls2 = (w.get(f"{p}.ls{n}") if spec.layer_scale else None for n in (1, 2))
@@ -239,12 +270,25 @@ class MixerLayer:
         if spec.moe is not None:
             m = spec.moe
             self.experts = MoEFFN(replace(cfg, layers=[], num_experts=m.experts, num_experts_per_tok=m.top,
-                                          moe_intermediate_size=m.ff, scoring_func="topk_softmax", n_group=m.groups,
-                                          topk_group=m.keep, num_shared_experts=0), w, p + ".mlp", tp)
+                                          moe_intermediate_size=m.ff, scoring_func="topk_" + m.scoring, n_group=m.groups,
+                                          topk_group=m.keep, routed_scaling_factor=m.scale, num_shared_experts=0), w,
+                                  p + ".mlp", tp)
             if m.router_bias and self.experts.logit_bias is None:
                 raise KeyError(f"missing {p}.mlp.gate.bias")
             if self.experts.q4 is not None or self.experts.s_gate_up is not None:
                 raise NotImplementedError("routed experts of models described layer by layer are not quantised")
+        # a gated layer's feed-forward: residual gate and shared expert's input as one projection, the shared expert's output
+        self.ff_in = self.shared_down = None
+        if spec.gated_residual:
+            if spec.ff or not spec.parallel or cfg.loop is not None or cfg.streams or spec.attn is None:
+                raise NotImplementedError("gated residuals join attention and routed experts that run side by side")
+            if spec.moe is not None:
+                if not spec.moe.shared_ff:
+                    raise NotImplementedError("routed experts of a gated layer come with a shared one")
+                self.ff_in = LinearW(w, p + ".mlp.in_proj")
+                self.shared_down = LinearW(w, p + ".mlp.shared_expert.down_proj")
+        elif spec.timemix is not None or spec.moe is not None and spec.moe.shared_ff:
+            raise NotImplementedError("time mixing and shared experts are part of layers with a gated residual")
         self.parallel_ff = spec.ff if spec.parallel else 0
         if self.parallel_ff and (self.linear is not None or self.attn is None or not spec.attn.shared_kv):
             raise NotImplementedError("a dense feed-forward runs beside attention whose values are its keys")
@@ -276,6 +320,11 @@ class MixerLayer:
     def start(self, x: torch.Tensor) -> Tuple[torch.Tensor, torch.Tensor]:
         """First layer of the model: (its normalised input, the stream) from the embedding output, which stays as it is.
         With several streams all of them equal it until the first sublayer's result arrives: nothing is copied."""
+        if self.spec.gated_residual:
+            residual = torch.empty_like(x)
+            h = ops.gated_stream_norm(None, None, None, None, None, None, self.cfg.residual_scale, x, residual, self.norms(),
+                                      self.cfg.rms_norm_eps, self.ln1.dtype)
+            return h, residual
         if self.hyper:
             h = ops.hyper_norm(None, None, None, x, None, None, None, self.hyper[0].inp, self.ln1, self.cfg.rms_norm_eps,
                                self.ln1.dtype)
@@ -284,6 +333,32 @@ class MixerLayer:
         h = ops.stream_norm(None, self.ln1, self.cfg.rms_norm_eps, self.cfg.norm_type == "layernorm", x, residual,
                             self.ln1.dtype, add_vec=self.pass_start.step if self.pass_start else None)
         return h, residual
+
+    def norms(self):
+        """A gated layer's norm weights: the mixers', then the feed-forward's if there is one."""
+        return [self.ln1, self.ln2] if self.ln2 is not None else [self.ln1]
+
+    def _gated(self, h: torch.Tensor, residual: torch.Tensor, meta, cache: LayerCache, next_norms):
+        H, attn = residual.shape[1], self.attn
+        x = self.in_proj(h[0])
+        K, n = self.o_proj.in_features, attn.width + (self.timemix.width if self.timemix else 0)
+        buf = torch.empty(h.shape[1], K, dtype=h.dtype, device=h.device)
+        if K > n:
+            buf[:, n:].zero_()
+        attn.run(x[:, :attn.rows], meta, cache.kv, buf[:, :attn.width])
+        if self.timemix is not None:
+            self.timemix.run(h[0], meta, cache.state, buf[:, attn.width:n])
+        routed = y = y_scale = y_gate = None
+        if self.experts is not None:
+            m = self.spec.moe
+            z = ops.linear(h[1], self.experts.gate_w, None, torch.float32)
+            routed = self.experts.rows(h[1], m.limit, m.alpha, m.plain, z)
+            f = self.ff_in(h[1])
+            y_scale, y_gate = z[:, m.experts], f[:, :H]
+            y = self.shared_down(ops.activation(f[:, H:], "relu2"))
+        return ops.gated_stream_norm(self.o_proj(buf), x[:, attn.rows:attn.rows + H], routed, y, y_scale, y_gate,
+                                     self.cfg.residual_scale, residual, residual, next_norms, self.cfg.rms_norm_eps,
+                                     self.ln1.dtype)
 
     def mix(self, h: torch.Tensor, meta, cache: LayerCache) -> torch.Tensor:
         x = self.in_proj(h)
@@ -323,10 +398,14 @@ class MixerLayer:
         return ops.hyper_norm(y, self.ls2, routed, residual, c.mix, c.out, residual, next_in, next_norm, eps, dtype)
 
     def forward(self, h: torch.Tensor, residual: torch.Tensor, meta, cache: LayerCache, next_norm, next_norm_b=None,
-                pass_start: Optional[PassStart] = None, next_in: Optional[torch.Tensor] = None):
+                pass_start: Optional[PassStart] = None, next_in: Optional[torch.Tensor] = None,
+                next_norm2: Optional[torch.Tensor] = None):
         """Same contract as DecoderLayer.forward: consumes the normalised input, returns the next layer's.
         ``pass_start``: the next run's, if it starts a pass; the embedding output is ``meta.start``. ``next_in``: how the
-        next sublayer reads the streams, where there are several."""
+        next sublayer reads the streams, where there are several. ``next_norm2``: a gated next layer's second norm."""
+        if self.spec.gated_residual:
+            h = self._gated(h, residual, meta, cache, [next_norm] if next_norm2 is None else [next_norm, next_norm2])
+            return h
         if self.hyper:
             return self._streams(h, residual, meta, cache, next_norm, next_in)
         y = self.o_proj(self.mix(h, meta, cache))

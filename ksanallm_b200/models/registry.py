@@ -39,6 +39,8 @@ FAMILIES: Dict[str, str] = {
                "feed-forward under one norm; learned positions, looped layers, 32-bit residual",
     "ladusun": "latent attention, capped attention with a sink (keys and values shared between layers) or a gated linear "
                "recurrence; clamped experts routed by groups, hyper-connected residual streams in 32-bit",
+    "vibunex": "attention whose heads' softmax weights are mixed, beside time mixing with token-dependent decays, beside "
+               "routed and shared squared-ReLU experts; gated sublayers, 32-bit residual",
     "minicpm": "embedding / residual / logit scaling; reranker head",
 }
 

@@ -96,6 +96,7 @@ class TransformerModel:
             self.rope_cache = ref.build_rope_cache(rd, maxp, cfg.rope_theta, cfg.rope_scaling, self.device)
         self.progress = None  # optional per-layer completion tracker (prefill/decode disaggregation)
         self.layer_ids = list(layer_range) if layer_range is not None else list(range(cfg.num_layers))
+        self.gated_layers = False
         self.rotary_tables = RotaryTables(self.device)  # of the layers that bring their own rotation
         if cfg.layers:
             if layer_range is not None and len(self.layer_ids) != cfg.num_layers:
@@ -103,6 +104,9 @@ class TransformerModel:
             # one entry per run: a layer inside a loop appears once per pass, with a cache of its own
             self.layers = [MixerLayer(cfg, weights, i, self.tp, self.rotary_tables, t) for i, t in cfg.layer_runs()]
             self.reserve_positions(min(max_positions or 1, maxp))
+            self.gated_layers = any(l.spec.gated_residual for l in self.layers)
+            if self.gated_layers and not all(l.spec.gated_residual for l in self.layers):
+                raise NotImplementedError("layers with and without a gated residual in one model")
             self.stream_sum = torch.ones(cfg.streams, device=self.device) if cfg.streams else None
             if cfg.loop is not None and (cfg.streams or any(l.kv_from() is not None for l in self.layers)):
                 raise NotImplementedError("loops over layers with several streams or shared keys")
@@ -230,7 +234,11 @@ class TransformerModel:
             more = (nxt.pass_start,) if self.cfg.loop is not None and nxt is not None else ()
             if self.cfg.streams:
                 more = (None, nxt.hyper[0].inp if nxt is not None else self.stream_sum)
+            if self.gated_layers:
+                more = (None, None, nxt.ln2 if nxt is not None else None)
             h = layer.forward(h, residual, meta, kv_caches[li], nw, nb, *more)
+            if nxt is None and self.gated_layers:
+                h = h[0]
             if self.progress is not None:
                 self.progress.record(li)  # parallel.transfer.LayerProgressTracker: KV of layer li may leave now
         self.last_residual = residual

@@ -130,9 +130,53 @@ def paged_attention(q, kv_cache, meta, scale, alibi_slopes=None, k_scale=1.0, v_
                                k_scale, v_scale, window)
 
 
-def qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps, positions=None, rotary=None):
+def qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps, positions=None, rotary=None,
+                  norm_all=False, halves=False):
     f = _mixer() if q.is_cuda else ref
-    return f.qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps, positions, rotary)
+    return f.qk_norm_cache(q, k, v, slot_mapping, cache, block_size, q_norm, k_norm, eps, positions, rotary, norm_all,
+                           halves)
+
+
+def talking_attention(q, cache, meta, block_size, kv_heads, vdim, scale, sink, talk, out_scale, out, gate=None):
+    """Writes heads * vdim columns of ``out`` [T, ...] (a column slice is fine); see ``reference.talking_attention``."""
+    if q.is_cuda:
+        from . import cuda_talking
+        cuda_talking.talking_attention(q, cache, meta, block_size, kv_heads, vdim, scale, sink, talk, out_scale, out, gate)
+        return
+    out.copy_(ref.talking_attention(q, cache, meta.block_tables, meta.cu_q, meta.kv_lens, block_size, kv_heads, vdim, scale,
+                                    sink, talk, out_scale, gate).flatten(1))
+
+
+def token_mix(h, mu, state, meta):
+    """``state`` [slots, 1, 1, n]: the previous token's vector is the last W numbers of a slot."""
+    if h.is_cuda:
+        from . import cuda_timemix
+        return cuda_timemix.token_mix(h, mu, state, meta)
+    return ref.token_mix(h, mu, state.flatten(1)[:, -h.shape[1]:], meta.state_slots, meta.cu_q, meta.kv_lens)
+
+
+def tanh_parts(x, dtype):
+    if x.is_cuda:
+        from . import cuda_timemix
+        return cuda_timemix.tanh_parts(x, dtype)
+    return ref.tanh_parts(x, dtype)
+
+
+def time_mix(r, k, v, z, w0, u, state, meta):
+    """``state`` as in :func:`token_mix`: the heads' states are the first h * d * d numbers of a slot."""
+    if r.is_cuda:
+        from . import cuda_timemix
+        return cuda_timemix.time_mix(r, k, v, z, w0, u, state, meta)
+    h, d = u.shape
+    S = state.flatten(1)[:, :h * d * d].unflatten(1, (h, d, d))
+    return ref.time_mix(r, k, v, z, w0, u, S, meta.state_slots, meta.cu_q, meta.kv_lens)
+
+
+def gated_stream_norm(x, x_gate, routed, y, y_scale, y_gate, scale, stream_in, stream_out, weights, eps, out_dtype):
+    f = ref
+    if stream_in.is_cuda:
+        f = _mixer()
+    return f.gated_stream_norm(x, x_gate, routed, y, y_scale, y_gate, scale, stream_in, stream_out, weights, eps, out_dtype)
 
 
 def latent_attention(q, a, norm_w, eps, rotary, cache, meta, block_size, w, scale, gate, out):
@@ -182,11 +226,11 @@ def linear_attention(q, k, v, state, meta, decay, act, rotary, key_scale):
                                 rotary, key_scale)
 
 
-def gated_norm(o, g, weight, eps, gate, out_scale, out):
+def gated_norm(o, g, weight, eps, gate, out_scale, out, per_head=False):
     if o.is_cuda:
-        _mixer().gated_norm(o, g, weight, eps, gate, out_scale, out)
+        _mixer().gated_norm(o, g, weight, eps, gate, out_scale, out, per_head)
         return
-    out.copy_(ref.gated_norm(o, g, weight, eps, gate, out_scale))
+    out.copy_(ref.gated_norm(o, g, weight, eps, gate, out_scale, per_head))
 
 
 def softcap(logits, cap):
@@ -214,18 +258,18 @@ def moe_route(logits, top_k, scoring="softmax", norm_topk=False, n_group=1, topk
     return ref.moe_route(logits, top_k, scoring, norm_topk, n_group, topk_group, routed_scale, correction_bias)
 
 
-def moe_topk(logits, experts, top_k, bias=None, groups=1, keep=1):
+def moe_topk(logits, experts, top_k, bias=None, groups=1, keep=1, scoring="softmax", scale=1.0):
     if logits.is_cuda:
         from . import cuda_moe
-        return cuda_moe.moe_topk(logits, experts, top_k, bias, groups, keep)
-    return ref.moe_topk(logits, experts, top_k, bias, groups, keep)
+        return cuda_moe.moe_topk(logits, experts, top_k, bias, groups, keep, scoring, scale)
+    return ref.moe_topk(logits, experts, top_k, bias, groups, keep, scoring, scale)
 
 
-def moe_expert_rows(x, ids, w_gate_up, w_down, limit=0.0, alpha=1.0):
+def moe_expert_rows(x, ids, w_gate_up, w_down, limit=0.0, alpha=1.0, plain=False):
     if x.is_cuda:
         from . import cuda_moe
-        return cuda_moe.expert_pipeline(x, ids, w_gate_up, w_down, 0, limit, alpha)
-    return ref.moe_expert_rows(x, ids, w_gate_up, w_down, limit, alpha)
+        return cuda_moe.expert_pipeline(x, ids, w_gate_up, w_down, 0, limit, alpha, plain)
+    return ref.moe_expert_rows(x, ids, w_gate_up, w_down, limit, alpha, plain)
 
 
 def moe_experts(x, ids, weights, w_gate_up, w_down, expert_offset=0):

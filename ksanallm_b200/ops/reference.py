@@ -402,25 +402,30 @@ def split_kv_cache(cache: torch.Tensor, hk: int, bs: int, d: int, dv: int) -> Tu
     return cache[:, :cut].view(nb, hk, bs, d), cache[:, cut:].view(nb, hk, bs, dv)
 
 
-def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, rotary: torch.Tensor) -> torch.Tensor:
-    """The leading dimensions of x [T, heads, d] that ``rotary`` ([positions, dims] = [cos | sin]) covers, in neighbouring
-    pairs, turned by each token's row."""
+def rotate_pairs(x: torch.Tensor, positions: torch.Tensor, rotary: torch.Tensor, neighbours: bool = True) -> torch.Tensor:
+    """The leading dimensions of x [T, heads, d] that ``rotary`` ([positions, dims] = [cos | sin]) covers, in pairs of
+    ``neighbours`` or of entries half of ``dims`` apart, turned by each token's row."""
     cs = rotary[positions.long()]
     half = cs.shape[1] // 2
-    return apply_rope(x, cs[:, :half], cs[:, half:], True, cs.shape[1])
+    return apply_rope(x, cs[:, :half], cs[:, half:], neighbours, cs.shape[1])
 
 
 def qk_norm_cache(q: torch.Tensor, k: Optional[torch.Tensor], v: Optional[torch.Tensor], slot_mapping: torch.Tensor,
                   cache: torch.Tensor, block_size: int, q_norm: Optional[torch.Tensor], k_norm: Optional[torch.Tensor],
-                  eps: float, positions: Optional[torch.Tensor] = None, rotary: Optional[torch.Tensor] = None) -> None:
-    """Per-head RMS norm (if any), then rotation (if any), of q (in place) and k; then k and v go to their cache slots.
+                  eps: float, positions: Optional[torch.Tensor] = None, rotary: Optional[torch.Tensor] = None,
+                  norm_all: bool = False, halves: bool = False) -> None:
+    """RMS norm (if any) per head, or over all heads together (``norm_all``), then rotation (if any) of neighbouring pairs
+    or of ``halves``, of q (in place) and k; then k and v go to their cache slots.
     q [T, h, d], k [T, hk, d], v [T, hk, dv] may be row-strided views, k and v None (nothing is appended); the cache has
     the layout of :func:`split_kv_cache`."""
     def ready(x, w):
-        if w is not None:
+        if w is not None and norm_all:
+            xf = x.float().flatten(1)
+            x = (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()).view(x.shape).to(x.dtype)
+        elif w is not None:
             xf = x.float()
             x = (xf * torch.rsqrt(xf.pow(2).mean(-1, keepdim=True) + eps) * w.float()).to(x.dtype)
-        return rotate_pairs(x, positions, rotary) if rotary is not None else x
+        return rotate_pairs(x, positions, rotary, not halves) if rotary is not None else x
 
     if q_norm is not None or rotary is not None:
         q.copy_(ready(q, q_norm))
@@ -496,6 +501,104 @@ def window_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.T
             o = o * torch.sigmoid(gate[cu[b]:cu[b + 1]].float()).unsqueeze(2)
         out[cu[b]:cu[b + 1]] = o.to(q.dtype)
     return out
+
+
+def talking_attention(q: torch.Tensor, cache: torch.Tensor, block_tables: torch.Tensor, cu_q: torch.Tensor,
+                      kv_lens: torch.Tensor, block_size: int, hk: int, dv: int, scale: float, sink: torch.Tensor,
+                      talk: torch.Tensor, out_scale: float = 1.0, gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """Softmax attention of each sequence's new tokens over all their keys whose weights are mixed across heads: with
+    p_g(i, j) = exp(s) / (sum over keys of exp(s) + exp(sink_g)), head h sums up sum_g talk[h, g] p_g(i, j) times the values
+    of its own key / value head. ``gate`` [T, h * dv]: the result times its sigmoid. q [T, h, d]; returns [T, h, dv]."""
+    T, h, d = q.shape
+    K, V = split_kv_cache(cache, hk, block_size, d, dv)
+    out = torch.empty(T, h, dv, dtype=q.dtype, device=q.device)
+    cu, kl, group = cu_q.tolist(), kv_lens.tolist(), h // hk
+    for b in range(len(kl)):
+        ql, L = cu[b + 1] - cu[b], kl[b]
+        if ql == 0:
+            continue
+        blocks = block_tables[b, :(L + block_size - 1) // block_size].long()
+        kb = K[blocks].permute(1, 0, 2, 3).reshape(hk, -1, d)[:, :L].float().repeat_interleave(group, 0)
+        vb = V[blocks].permute(1, 0, 2, 3).reshape(hk, -1, dv)[:, :L].float().repeat_interleave(group, 0)
+        s = torch.einsum("qhd,hkd->hqk", q[cu[b]:cu[b + 1]].float(), kb) * scale
+        dist = torch.arange(L - ql, L, device=q.device).unsqueeze(1) - torch.arange(L, device=q.device)
+        s = s.masked_fill((dist < 0).unsqueeze(0), float("-inf"))
+        p = torch.softmax(torch.cat((sink.float().view(h, 1, 1).expand(h, ql, 1), s), 2), dim=-1)[..., 1:]
+        p = torch.einsum("hg,gqk->hqk", talk.float(), p)
+        o = torch.einsum("hqk,hkd->qhd", p, vb) * out_scale
+        if gate is not None:
+            o = o * torch.sigmoid(gate[cu[b]:cu[b + 1]].float()).view(o.shape)
+        out[cu[b]:cu[b + 1]] = o.to(q.dtype)
+    return out
+
+
+def token_mix(h: torch.Tensor, mu: torch.Tensor, last: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor,
+              kv_lens: torch.Tensor) -> torch.Tensor:
+    """[n, T, W]: h + (h' - h) mu[n] for each row of ``mu`` [n, W], h' being the previous token's h. A sequence's first new
+    token finds it in ``last[slot]`` (fp32; zeros at the start of a sequence), which then takes the last new token's."""
+    hf = h.float()
+    prev = torch.cat((torch.zeros_like(hf[:1]), hf[:-1]))
+    cu, kl, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
+    for b in range(len(kl)):
+        if cu[b + 1] > cu[b]:
+            prev[cu[b]] = 0 if kl[b] == cu[b + 1] - cu[b] else last[sl[b]]
+            last[sl[b]] = hf[cu[b + 1] - 1]
+    return (hf + (prev - hf) * mu.unsqueeze(1)).to(h.dtype)
+
+
+def tanh_parts(x: torch.Tensor, dtype: torch.dtype) -> torch.Tensor:
+    """tanh of x [T, n] fp32; for a 16-bit ``dtype`` as two parts [T, 2 n] = [hi | lo] whose sum keeps 16 bits."""
+    t = torch.tanh(x)
+    if dtype == torch.float32:
+        return t
+    hi = t.to(dtype)
+    return torch.cat((hi, (t - hi.float()).to(dtype)), 1)
+
+
+def time_mix(r: torch.Tensor, k: torch.Tensor, v: torch.Tensor, z: torch.Tensor, w0: torch.Tensor, u: torch.Tensor,
+             state: torch.Tensor, slots: torch.Tensor, cu_q: torch.Tensor, kv_lens: torch.Tensor) -> torch.Tensor:
+    """With w = exp(-exp(z + w0)) per token, head and key channel: o_t = (S + diag(u) k_t v_t^T)^T r_t, then
+    S <- diag(w_t) S + k_t v_t^T, the state of sequence b being ``state[slots[b]]`` [h, d, d] fp32 ([key][value]). r, k, v
+    [T, h * d]; z [T, h * d] fp32; u [h, d]. A sequence whose first token is among the new ones starts from zero."""
+    T, (h, d) = r.shape[0], u.shape
+    rf, kf, vf = (x.float().reshape(T, h, d) for x in (r, k, v))
+    # S + (w - 1) S: the rounding of a w close to 1 would add up over many tokens
+    wm1 = torch.expm1(-torch.exp(z.float() + w0)).view(T, h, d)
+    out = torch.empty(T, h, d, dtype=r.dtype, device=r.device)
+    cu, kl, sl = cu_q.tolist(), kv_lens.tolist(), slots.tolist()
+    for b in range(len(kl)):
+        if cu[b + 1] == cu[b]:
+            continue
+        S = torch.zeros_like(state[0]) if kl[b] == cu[b + 1] - cu[b] else state[sl[b]].clone()
+        for t in range(cu[b], cu[b + 1]):
+            own = (rf[t] * u * kf[t]).sum(-1, keepdim=True)
+            out[t] = (torch.einsum("hde,hd->he", S, rf[t]) + own * vf[t]).to(r.dtype)
+            S = S + (wm1[t].unsqueeze(2) * S + kf[t].unsqueeze(2) * vf[t].unsqueeze(1))
+        state[sl[b]] = S
+    return out
+
+
+def gated_stream_norm(x: Optional[torch.Tensor], x_gate: Optional[torch.Tensor], routed, y: Optional[torch.Tensor],
+                      y_scale: Optional[torch.Tensor], y_gate: Optional[torch.Tensor], scale: float,
+                      stream_in: torch.Tensor, stream_out: Optional[torch.Tensor], weights, eps: float,
+                      out_dtype: torch.dtype) -> torch.Tensor:
+    """The 32-bit stream takes two gated sublayers' results and is RMS-normalised, once per weight in ``weights``:
+    stream + scale (x sigmoid(x_gate) + (sum of ``routed`` rows, see :func:`stream_norm`, + y sigmoid(y_scale)) sigmoid(y_gate)).
+    x, y and the gates [T, H]; ``y_scale`` [T] fp32; either sublayer may be absent. Returns [len(weights), T, H]."""
+    v = stream_in.float()
+    if x is not None:
+        v = v + scale * (x.float() * torch.sigmoid(x_gate.float()))
+    if y is not None:
+        f = y.float() * torch.sigmoid(y_scale.float()).unsqueeze(1)
+        if routed is not None:
+            rows, pos, w = routed
+            p = pos.view(w.shape).long()
+            f = f + torch.einsum("tk,tkh->th", w.masked_fill(p < 0, 0.0), rows[p.clamp(min=0)].float())
+        v = v + scale * (f * torch.sigmoid(y_gate.float()))
+    if stream_out is not None:
+        stream_out.copy_(v)
+    n = v / torch.sqrt(v.pow(2).mean(-1, keepdim=True) + eps)
+    return torch.stack([(n * w.float()).to(out_dtype) for w in weights])
 
 
 def latent_append(q: torch.Tensor, a: torch.Tensor, norm_w: torch.Tensor, eps: float, positions: torch.Tensor,
@@ -596,11 +699,11 @@ def linear_attention(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, state: t
 
 
 def gated_norm(o: torch.Tensor, g: torch.Tensor, weight: Optional[torch.Tensor], eps: float, gate: str,
-               out_scale: float = 1.0) -> torch.Tensor:
-    """RMS norm of o [T, h, dv] - per head without a weight, over all heads together with one - times gate(g),
-    g [T, h * dv]; returns [T, h * dv]."""
+               out_scale: float = 1.0, per_head: bool = False) -> torch.Tensor:
+    """RMS norm of o [T, h, dv] - per head without a weight, over all heads together with one (``per_head``: per head
+    nevertheless) - times gate(g), g [T, h * dv]; returns [T, h * dv]."""
     T = o.shape[0]
-    of = o.float() if weight is None else o.float().reshape(T, 1, -1)
+    of = o.float() if weight is None or per_head else o.float().reshape(T, 1, -1)
     of = (of * torch.rsqrt(of.pow(2).mean(-1, keepdim=True) + eps)).reshape(T, -1)
     if weight is not None:
         of = of * weight.float()
@@ -718,9 +821,9 @@ def moe_route(logits: torch.Tensor, top_k: int, scoring: str = "softmax", norm_t
 
 
 def moe_topk(logits: torch.Tensor, experts: int, top_k: int, bias: Optional[torch.Tensor] = None, groups: int = 1,
-             keep: int = 1) -> Tuple[torch.Tensor, torch.Tensor]:
+             keep: int = 1, scoring: str = "softmax", scale: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
     """Router over the first ``experts`` columns of ``logits``: the ``top_k`` largest (after ``bias``) and the softmax
-    over just those. Of ``groups`` > 1 equal groups of neighbours only the ``keep`` with the largest logits take part.
+    over just those, or (``scoring`` sigmoid) each one's sigmoid, times ``scale``. Of ``groups`` > 1 equal groups of neighbours only the ``keep`` with the largest logits take part.
     Returns (ids [T, k] int32, weights [T, k] fp32)."""
     z = logits[:, :experts].float()
     if bias is not None:
@@ -731,7 +834,7 @@ def moe_topk(logits: torch.Tensor, experts: int, top_k: int, bias: Optional[torc
         open_ = torch.zeros(g.shape[:2], dtype=torch.bool, device=z.device).scatter_(1, best, True)
         z = g.masked_fill(~open_.unsqueeze(-1), float("-inf")).flatten(1)
     top, ids = z.topk(top_k, dim=-1)
-    return ids.to(torch.int32), torch.softmax(top, dim=-1)
+    return ids.to(torch.int32), scale * (torch.sigmoid(top) if scoring == "sigmoid" else torch.softmax(top, dim=-1))
 
 
 def clamped_gate_mul(x: torch.Tensor, limit: float, alpha: float) -> torch.Tensor:
@@ -742,16 +845,17 @@ def clamped_gate_mul(x: torch.Tensor, limit: float, alpha: float) -> torch.Tenso
 
 
 def moe_expert_rows(x: torch.Tensor, ids: torch.Tensor, w_gate_up: torch.Tensor, w_down: torch.Tensor,
-                    limit: float = 0.0, alpha: float = 1.0) -> Tuple[torch.Tensor, torch.Tensor]:
+                    limit: float = 0.0, alpha: float = 1.0, plain: bool = False) -> Tuple[torch.Tensor, torch.Tensor]:
     """The unweighted output of every (token, slot) pair's expert: (rows [T * k, H], the row of each pair). ``limit`` > 0:
-    clamped experts, see :func:`clamped_gate_mul`."""
+    clamped experts, see :func:`clamped_gate_mul`. ``plain``: w_gate_up is [E, I, H], the activation squared ReLU."""
     k = ids.shape[1]
     flat = ids.reshape(-1).long()
     y = torch.empty(flat.numel(), x.shape[1], dtype=x.dtype, device=x.device)
     for e in flat.unique().tolist():
         at = (flat == e).nonzero()[:, 0]
         h = linear(x[at // k], w_gate_up[e])
-        y[at] = linear(clamped_gate_mul(h, limit, alpha) if limit else silu_and_mul(h), w_down[e])
+        a = activation(h, "relu2") if plain else clamped_gate_mul(h, limit, alpha) if limit else silu_and_mul(h)
+        y[at] = linear(a, w_down[e])
     return y, torch.arange(flat.numel(), dtype=torch.int32, device=x.device)
 
 
