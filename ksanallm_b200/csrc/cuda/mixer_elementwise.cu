@@ -1,7 +1,7 @@
-// Bandwidth-bound steps of layers with mixers of their own sizes: norms over a 32-bit residual stream, embedding into
-// that stream, GELU (gated or not), squared ReLU and clamped gates, the paged cache append (with per-head QK norm and
-// rotation, or beside the activation), the gated RMS norm behind linear attention, and the logit soft cap. Everything is
-// computed in 32-bit floats; T is the storage type of activations.
+// Bandwidth-bound steps of layers with mixers of their own sizes: norms over a 32-bit residual stream (which may take gated
+// sublayers), embedding into that stream, GELU (gated or not), squared ReLU and clamped gates, the paged cache append (with
+// QK norm per head or per row and rotation, or beside the activation), the gated RMS norm behind linear attention, and the
+// logit soft cap. Everything is computed in 32-bit floats; T is the storage type of activations.
 #include "host_common.h"
 #include "mixer_common.cuh"
 
@@ -182,6 +182,158 @@ static int launch_stream_norm(const void* x, int ldx, const void* res_in, void* 
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 
+// ---- gated sublayers into the stream ------------------------------------------------------------------------------
+// v = in + scale (x sig(xg) + (sum_j weights[t, j] rows[pos[t, j]] + y sig(ys[t])) sig(yg));  stream = v
+// out[n] = v / sqrt(mean(v^2) + eps) * w[n] for up to two weights. Every term may be absent (null).
+template <typename T>
+__device__ __forceinline__ float sigmoid_as(float x) {
+  if constexpr (sizeof(T) == 2) return __fdividef(1.f, 1.f + __expf(-x));
+  return sigmoid_f(x);
+}
+
+template <typename T>
+struct GatedNormArgs {
+  const T *x, *xg, *rows, *y, *yg;
+  int ldx, ldxg, ldy, ldyg, ldys, k, H, norms;
+  const int* pos;
+  const float *weights, *ys;
+  float scale, eps;
+  const float* in;  // [rows, H]
+  float* stream;    // [rows, H] (in itself is fine; null: nowhere)
+  const T* w[2];
+  T* out;           // [norms][tokens][H]
+  size_t plane;     // tokens * H
+
+  template <int N, int V>
+  __device__ void value(size_t row, int c0, int step, float (*v)[N]) const {
+    auto load = [&](const auto* p, float (*f)[N]) {
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+        if (c0 + i * step < H) load_n<N>(p + c0 + i * step, f[i]);
+    };
+    float a[V][N], b[V][N];
+#pragma unroll
+    for (int i = 0; i < V; ++i)
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[i][j] = a[i][j] = b[i][j] = 0.f;
+    if (y) {
+      load(y + row * ldy, a);
+      load(yg + row * ldyg, b);
+      const float s = sigmoid_as<T>(ys[row * ldys]);
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[i][j] = a[i][j] * s;
+      for (int e = 0; e < k; ++e) {
+        const int p = pos[row * k + e];
+        if (p < 0) continue;
+        const float we = weights[row * k + e];
+        load(rows + static_cast<size_t>(p) * H, a);
+#pragma unroll
+        for (int i = 0; i < V; ++i)
+#pragma unroll
+          for (int j = 0; j < N; ++j) v[i][j] = fmaf(we, a[i][j], v[i][j]);
+      }
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[i][j] *= sigmoid_as<T>(b[i][j]);
+    }
+    if (x) {
+      load(x + row * ldx, a);
+      load(xg + row * ldxg, b);
+#pragma unroll
+      for (int i = 0; i < V; ++i)
+#pragma unroll
+        for (int j = 0; j < N; ++j) v[i][j] = fmaf(a[i][j], sigmoid_as<T>(b[i][j]), v[i][j]);
+    }
+    load(in + row * H, a);
+#pragma unroll
+    for (int i = 0; i < V; ++i)
+#pragma unroll
+      for (int j = 0; j < N; ++j) v[i][j] = fmaf(scale, v[i][j], a[i][j]);
+  }
+};
+
+template <typename T, int VPT>
+__global__ void __launch_bounds__(256)
+gated_stream_norm_kernel(const GatedNormArgs<T> a) {
+  __shared__ float red[32];
+  const size_t row = blockIdx.x;
+  const int H = a.H;
+  float v[VPT][4], ss = 0.f;
+  a.template value<4, VPT>(row, threadIdx.x * 4, 1024, v);
+#pragma unroll
+  for (int i = 0; i < VPT; ++i) {
+    const int c = (i * 256 + threadIdx.x) * 4;
+    if (c < H) {
+      if (a.stream) store_n<4>(a.stream + row * H + c, v[i]);
+#pragma unroll
+      for (int j = 0; j < 4; ++j) ss += v[i][j] * v[i][j];
+    }
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(H) + a.eps);
+  for (int n = 0; n < a.norms; ++n) {
+#pragma unroll
+    for (int i = 0; i < VPT; ++i) {
+      const int c = (i * 256 + threadIdx.x) * 4;
+      if (c < H) {
+        float g[4];
+        load_n<4>(a.w[n] + c, g);
+#pragma unroll
+        for (int j = 0; j < 4; ++j) g[j] *= v[i][j] * inv;
+        store_n<4>(a.out + n * a.plane + row * H + c, g);
+      }
+    }
+  }
+}
+
+template <typename T>
+__global__ void __launch_bounds__(256)
+gated_stream_norm_any_kernel(const GatedNormArgs<T> a) {
+  extern __shared__ float row_v[];
+  __shared__ float red[32];
+  const size_t row = blockIdx.x;
+  const int H = a.H;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < H; c += 256) {
+    float v[1][1];
+    a.template value<1, 1>(row, c, 0, v);
+    if (a.stream) a.stream[row * H + c] = v[0][0];
+    row_v[c] = v[0][0];  // only this thread reads it back
+    ss += v[0][0] * v[0][0];
+  }
+  const float inv = 1.f / sqrtf(block_sum(ss, red) / static_cast<float>(H) + a.eps);
+  for (int n = 0; n < a.norms; ++n)
+    for (int c = threadIdx.x; c < H; c += 256)
+      a.out[n * a.plane + row * H + c] = from_f<T>(row_v[c] * inv * to_f(a.w[n][c]));
+}
+
+template <typename T>
+static int launch_gated_norm(const GatedNormArgs<T>& a, int rows, cudaStream_t st) {
+  auto al = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & (4 * sizeof(T) - 1)) == 0; };
+  const int H = a.H;
+  const bool vec = !((H | a.ldx | a.ldxg | a.ldy | a.ldyg) & 3) && H <= 8192 && al(a.x) && al(a.xg) && al(a.y) && al(a.yg) &&
+                   al(a.rows) && al(a.out) && al(a.w[0]) && al(a.w[1]);
+#define KSANA_GSN(V) gated_stream_norm_kernel<T, V><<<rows, 256, 0, st>>>(a)
+  if (!vec) {
+    if (H > 50 * 1024) return -1;
+    auto kern = gated_stream_norm_any_kernel<T>;
+    if (H * 4 > 47 * 1024 && KSANA_SMEM_ONCE(kern, 200 * 1024) != 0) return -4;
+    kern<<<rows, 256, H * 4, st>>>(a);
+  } else if (H <= 1024) {
+    KSANA_GSN(1);
+  } else if (H <= 2048) {
+    KSANA_GSN(2);
+  } else if (H <= 4096) {
+    KSANA_GSN(4);
+  } else {
+    KSANA_GSN(8);
+  }
+#undef KSANA_GSN
+  return cudaGetLastError() == cudaSuccess ? 0 : -5;
+}
+
 // ---- embedding into a 32-bit stream ---------------------------------------------------------------------------
 // out = table[id] * scale (+ pos_table[position], unscaled)
 template <typename T>
@@ -213,11 +365,11 @@ __global__ void gelu_mul_kernel(const T* __restrict__ x, int ldx, T* __restrict_
 
 // ---- squared ReLU; gate and up clamped -------------------------------------------------------------------------------
 template <typename T, int N>
-__global__ void relu2_kernel(const T* __restrict__ x, T* __restrict__ out, size_t n) {
+__global__ void relu2_kernel(const T* __restrict__ x, int ldx, T* __restrict__ out, int cols, size_t n) {
   const size_t i = (static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x) * N;
   if (i >= n) return;
   float f[N];
-  load_n<N>(x + i, f);
+  load_n<N>(ldx == cols ? x + i : x + i / cols * ldx + i % cols, f);
 #pragma unroll
   for (int j = 0; j < N; ++j) f[j] = fmaxf(f[j], 0.f) * fmaxf(f[j], 0.f);
   store_n<N>(out + i, f);
@@ -323,6 +475,68 @@ qk_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ld
   }
 }
 
+// ---- QK norm over whole rows, rotation of halves, cache append -------------------------------------------------------
+// One CTA per token. All heads of q are normalised together, then all of k; then entries i and i + rd / 2 of every head
+// turn; q stays in place, k and v go to their cache slots. N consecutive columns per thread.
+template <typename T, int N>
+__global__ void __launch_bounds__(256)
+qk_row_norm_cache_kernel(T* __restrict__ q, int ldq, const T* __restrict__ k, int ldk, const T* __restrict__ v, int ldv,
+                         const int* __restrict__ slots, T* __restrict__ cache, const float* __restrict__ qw,
+                         const float* __restrict__ kw, float eps, const int* __restrict__ positions,
+                         const float* __restrict__ rotary, int rd, int h, int hk, int d, int dv, int bs) {
+  extern __shared__ float row_qk[];  // [h * d] queries, [hk * d] keys
+  __shared__ float red[32];
+  const int t = blockIdx.x, nq = h * d, nk = hk * d;
+  q += static_cast<size_t>(t) * ldq;
+  k += static_cast<size_t>(t) * ldk;
+  v += static_cast<size_t>(t) * ldv;
+  float f[N], sq = 0.f, sk = 0.f;
+  for (int c = threadIdx.x * N; c < nq + nk; c += 256 * N) {
+    const bool is_q = c < nq;
+    load_n<N>(is_q ? q + c : k + c - nq, f);
+    float s = 0.f;
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      row_qk[c + j] = f[j];
+      s += f[j] * f[j];
+    }
+    if (is_q) sq += s; else sk += s;
+  }
+  const float iq = 1.f / sqrtf(block_sum(sq, red) / static_cast<float>(nq) + eps);
+  const float ik = 1.f / sqrtf(block_sum(sk, red) / static_cast<float>(nk) + eps);  // (its barriers: the row is complete)
+  const float* cs = rotary ? rotary + static_cast<size_t>(positions[t]) * rd : nullptr;
+  const int slot = slots[t], half = rd >> 1;
+  T* block = cache + static_cast<size_t>(max(slot, 0) / bs) * (static_cast<size_t>(hk) * bs * (d + dv));
+  const int off = max(slot, 0) % bs;
+  for (int c = threadIdx.x * N; c < nq + nk; c += 256 * N) {
+    const bool is_q = c < nq;
+    const float inv = is_q ? iq : ik;
+    const float* w = is_q ? qw : kw - nq;
+    const int hd = (is_q ? c : c - nq) / d, i0 = (is_q ? c : c - nq) % d;
+#pragma unroll
+    for (int j = 0; j < N; ++j) {
+      const int i = i0 + j;
+      float x = row_qk[c + j] * inv * w[c + j];
+      if (i < rd && cs) {
+        const bool low = i < half;
+        const int p = low ? c + j + half : c + j - half, a = low ? i : i - half;
+        const float y = row_qk[p] * inv * w[p];
+        x = low ? x * cs[a] - y * cs[half + a] : x * cs[a] + y * cs[half + a];
+      }
+      f[j] = x;
+    }
+    if (is_q)
+      store_n<N>(q + c, f);
+    else if (slot >= 0)
+      store_n<N>(block + (static_cast<size_t>(hd) * bs + off) * d + i0, f);
+  }
+  if (slot < 0) return;
+  for (int c = threadIdx.x * N; c < hk * dv; c += 256 * N) {
+    load_n<N>(v + c, f);
+    store_n<N>(block + static_cast<size_t>(hk) * bs * d + (static_cast<size_t>(c / dv) * bs + off) * dv + c % dv, f);
+  }
+}
+
 // ---- cache append beside an activation -----------------------------------------------------------------------------
 // A row of x holds new keys (nk columns, to the cache of keys alone: [block][hk x bs x d]) and, behind them, the input of
 // a feed-forward's activation: out = gelu(up), or gelu(gate) * up over 2 I columns. N columns per thread.
@@ -361,11 +575,11 @@ __device__ __forceinline__ float gate_f(float g, int kind) {
   return kind == 0 ? silu_f(g) : sigmoid_f(g);
 }
 
-// per head, no weight: a warp takes HEADS heads of a token at a time, up to 32 N columns each in registers
+// per head (w: null, or a factor per column of all heads): a warp takes HEADS heads of a token at a time, up to 32 N columns each in registers
 template <typename T, int N, int HEADS>
 __global__ void __launch_bounds__(256)
-gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ g, int ldg, T* __restrict__ out, int ldo,
-                       int tokens, int h, int dv, float eps, int gate, float out_scale) {
+gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ g, int ldg, const float* __restrict__ w,
+                       T* __restrict__ out, int ldo, int tokens, int h, int dv, float eps, int gate, float out_scale) {
   const int groups = (h + HEADS - 1) / HEADS;
   const long long unit = static_cast<long long>(blockIdx.x) * 8 + (threadIdx.x >> 5);
   const int lane = threadIdx.x & 31;
@@ -392,6 +606,12 @@ gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ g, int ldg
       const float inv = out_scale / sqrtf(warp_sum(ss) / static_cast<float>(dv) + eps);
 #pragma unroll
       for (int j = 0; j < N; ++j) f[i][j] *= inv * gate_f<T>(gg[i][j], gate);
+      if (w && h0 + i < h && c < dv) {
+        float ww[N];
+        load_n<N>(w + (h0 + i) * dv + c, ww);
+#pragma unroll
+        for (int j = 0; j < N; ++j) f[i][j] *= ww[j];
+      }
       if (h0 + i < h && c < dv) store_n<N>(out + t * ldo + (h0 + i) * dv + c, f[i]);
     }
     return;
@@ -409,7 +629,7 @@ gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ g, int ldg
       load_n<N>(src + c, f);
       load_n<N>(g + t * ldg + hd * dv + c, gg);
 #pragma unroll
-      for (int j = 0; j < N; ++j) f[j] *= inv * gate_f<T>(gg[j], gate);
+      for (int j = 0; j < N; ++j) f[j] *= inv * gate_f<T>(gg[j], gate) * (w ? w[hd * dv + c + j] : 1.f);
       store_n<N>(out + t * ldo + hd * dv + c, f);
     }
   }
@@ -510,12 +730,14 @@ KSANA_API int ksana_gelu_mul(const void* x, int ldx, void* out, int ldo, int row
   return done();
 }
 
-KSANA_API int ksana_relu2(const void* x, void* out, long long n, int kind, cudaStream_t st) {
-  if (n <= 0) return 0;
-  const bool vec = !(n & 7) && aligned(x, 16) && aligned(out, 16);
+// x: [rows, cols] with pitch ldx, out: contiguous.
+KSANA_API int ksana_relu2(const void* x, int ldx, void* out, int rows, int cols, int kind, cudaStream_t st) {
+  if (rows <= 0 || cols <= 0) return 0;
+  const size_t n = static_cast<size_t>(rows) * cols;
+  const bool vec = !(n & 7) && (ldx == cols || !((ldx | cols) & 7)) && aligned(x, 16) && aligned(out, 16);
 #define KSANA_R2(T, N)                                                                                        \
   relu2_kernel<T, N><<<static_cast<unsigned>((n / N + (n % N ? 1 : 0) + 255) / 256), 256, 0, st>>>(           \
-      static_cast<const T*>(x), static_cast<T*>(out), static_cast<size_t>(n))
+      static_cast<const T*>(x), ldx, static_cast<T*>(out), cols, n)
   if (kind) {
     if (vec) KSANA_R2(bf16, 8); else KSANA_R2(bf16, 1);
   } else {
@@ -591,22 +813,69 @@ KSANA_API int ksana_append_act(const void* k, const void* u, int ldx, const int*
   return done();
 }
 
-// gate: 0 silu, 1 sigmoid. w == nullptr: per head, no weight. o is [tokens, h, dv] contiguous.
+// The stream takes two gated sublayers, see GatedNormArgs. All activations have storage type `kind` (0 fp32, 1 bf16);
+// norms 1 or 2.
+KSANA_API int ksana_gated_stream_norm(const void* x, int ldx, const void* xg, int ldxg, const void* rows, const int* pos,
+                                      const float* weights, int k, const void* y, int ldy, const float* ys, int ldys,
+                                      const void* yg, int ldyg, float scale, const float* in, float* stream,
+                                      const void* w0, const void* w1, void* out, int tokens, int H, float eps, int kind,
+                                      cudaStream_t st) {
+  if (tokens <= 0 || H <= 0) return 0;
+#define KSANA_GSN_ARGS(T)                                                                                                 \
+  GatedNormArgs<T>{static_cast<const T*>(x), static_cast<const T*>(xg), static_cast<const T*>(rows),                      \
+                   static_cast<const T*>(y), static_cast<const T*>(yg), ldx, ldxg, ldy, ldyg, ldys, rows ? k : 0, H,       \
+                   w1 ? 2 : 1, pos, weights, ys, scale, eps, in, stream,                                                   \
+                   {static_cast<const T*>(w0), static_cast<const T*>(w1)}, static_cast<T*>(out),                           \
+                   static_cast<size_t>(tokens) * H}
+  return kind ? launch_gated_norm<bf16>(KSANA_GSN_ARGS(bf16), tokens, st)
+              : launch_gated_norm<float>(KSANA_GSN_ARGS(float), tokens, st);
+#undef KSANA_GSN_ARGS
+}
+
+KSANA_API int ksana_qk_row_norm_cache(void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const int* slots,
+                                      void* cache, const float* qw, const float* kw, float eps, const int* positions,
+                                      const float* rotary, int rd, int tokens, int h, int hk, int d, int dv, int bs,
+                                      int kind, cudaStream_t st) {
+  if (tokens <= 0) return 0;
+  if (rotary && (rd < 0 || rd > d || (rd & 1))) return -2;
+  const int esz = kind ? 2 : 4, smem = (h + hk) * d * 4;
+  if (smem > 200 * 1024) return -1;
+  const bool vec = !((ldq | ldk | ldv | d | dv) & 3) && aligned(q, 4 * esz) && aligned(k, 4 * esz) &&
+                   aligned(v, 4 * esz) && aligned(cache, 4 * esz);
+#define KSANA_QR(T, N)                                                                                                  \
+  do {                                                                                                                  \
+    auto kern = qk_row_norm_cache_kernel<T, N>;                                                                         \
+    if (smem > 47 * 1024 && KSANA_SMEM_ONCE(kern, 200 * 1024) != 0) return -4;                                          \
+    kern<<<tokens, 256, smem, st>>>(static_cast<T*>(q), ldq, static_cast<const T*>(k), ldk, static_cast<const T*>(v),   \
+                                    ldv, slots, static_cast<T*>(cache), qw, kw, eps, positions, rotary, rd, h, hk, d,   \
+                                    dv, bs);                                                                            \
+  } while (0)
+  if (kind) {
+    if (vec) KSANA_QR(bf16, 4); else KSANA_QR(bf16, 1);
+  } else {
+    if (vec) KSANA_QR(float, 4); else KSANA_QR(float, 1);
+  }
+#undef KSANA_QR
+  return done();
+}
+
+// gate: 0 silu, 1 sigmoid. w == nullptr: per head, no weight; per_head: per head, then w over all columns. o is [tokens, h, dv] contiguous.
 KSANA_API int ksana_gated_norm(const void* o, const void* g, int ldg, const float* w, void* out, int ldo, int tokens,
-                               int h, int dv, float eps, int gate, float out_scale, int kind, cudaStream_t st) {
+                               int h, int dv, float eps, int gate, float out_scale, int per_head, int kind,
+                               cudaStream_t st) {
   if (tokens <= 0) return 0;
   const int esz = kind ? 2 : 4;
   const int width = h * dv;
   const bool vec = !((dv | ldg | ldo) & 3) && aligned(o, 4 * esz) && aligned(g, 4 * esz) && aligned(out, 4 * esz);
-  const bool wide = kind && !w && dv > 128 && !((dv | ldg | ldo) & 7) && aligned(o, 16) && aligned(g, 16) && aligned(out, 16);
+  const bool wide = kind && (!w || per_head) && dv > 128 && !((dv | ldg | ldo) & 7) && aligned(o, 16) && aligned(g, 16) && aligned(out, 16);
   const unsigned grid = static_cast<unsigned>((static_cast<long long>(tokens) * ((h + 3) / 4) + 7) / 8);
 #define KSANA_GN(T, N)                                                                                               \
   do {                                                                                                               \
-    if (w)                                                                                                           \
+    if (w && !per_head)                                                                                              \
       gated_row_norm_kernel<T, N><<<tokens, 256, 0, st>>>(static_cast<const T*>(o), static_cast<const T*>(g), ldg, w, \
                                                           static_cast<T*>(out), ldo, width, eps, gate, out_scale);   \
     else                                                                                                             \
-      gated_head_norm_kernel<T, N, 4><<<grid, 256, 0, st>>>(static_cast<const T*>(o), static_cast<const T*>(g), ldg,    \
+      gated_head_norm_kernel<T, N, 4><<<grid, 256, 0, st>>>(static_cast<const T*>(o), static_cast<const T*>(g), ldg, w, \
                                                          static_cast<T*>(out), ldo, tokens, h, dv, eps, gate,        \
                                                          out_scale);                                                 \
   } while (0)

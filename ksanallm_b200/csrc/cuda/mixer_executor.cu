@@ -17,8 +17,8 @@ int ksana_stream_norm(const void* x, int ldx, const void* res_in, void* res_out,
                       cudaStream_t st);
 int ksana_append_act(const void* k, const void* u, int ldx, const int* slots, void* cache, int tokens, int hk, int d,
                      int bs, void* out, int ldo, int I, int gated, int kind, cudaStream_t st);
-int ksana_moe_topk(const float* logits, int ld, const float* bias, int T, int E, int k, int groups, int keep, int* ids,
-                   float* weights, cudaStream_t st);
+int ksana_moe_topk(const float* logits, int ld, const float* bias, int T, int E, int k, int groups, int keep, int scoring,
+                   float scale, int* ids, float* weights, cudaStream_t st);
 int ksana_moe_permute(const void* x, int ldx, const int* ids, int T, int k, int H, int expert_offset, int E_local,
                       int* meta, int* pos, int* row_src, void* xs, cudaStream_t stream);
 int ksana_moe_grouped_gemm(const void* A, const void* W, void* C, const int* offsets, int E, int max_rows, int N, int K,
@@ -30,7 +30,7 @@ int ksana_qk_norm_cache(void* q, int ldq, const void* k, int ldk, const void* v,
                         const float* qw, const float* kw, float eps, const int* positions, const float* rotary, int rd,
                         int tokens, int h, int hk, int d, int dv, int bs, int kind, cudaStream_t st);
 int ksana_gated_norm(const void* o, const void* g, int ldg, const float* w, void* out, int ldo, int tokens, int h, int dv,
-                     float eps, int gate, float out_scale, int kind, cudaStream_t st);
+                     float eps, int gate, float out_scale, int per_head, int kind, cudaStream_t st);
 int ksana_window_prefill(const void* q, int ldq, int total_tokens, const void* cache, int num_blocks,
                          const int* block_tables, int max_blocks, const int* cu_q, const int* kv_lens, int h, int hk,
                          int d, int dv, int bs, int window, int keep, int shared, float scale, const float* bias,
@@ -59,7 +59,7 @@ int ksana_hyper_norm(const void* x, int ldx, const float* scale, const void* row
                      int k, const float* streams, int one, const float* mix, const float* out_w, float* res,
                      const float* in_w, const void* w, void* out, int tokens, int H, int S, float eps, int kind,
                      cudaStream_t st);
-int ksana_relu2(const void* x, void* out, long long n, int kind, cudaStream_t st);
+int ksana_relu2(const void* x, int ldx, void* out, int rows, int cols, int kind, cudaStream_t st);
 int ksana_clamped_gate_mul(const void* x, void* out, int rows, int I, float limit, float alpha, int kind,
                            cudaStream_t st);
 int ksana_gemm_bf16_batched(const void* A, long long a_row_stride, long long a_batch_stride, const void* W, void* C,
@@ -360,7 +360,7 @@ struct Exec {
                                           base[i], count[i], i == 1 && s->one_token, 1, st)))
         return false;
     return step(7, ksana_gated_norm(m->o_buf, g, ld, w.norm_w, out, w.k_out, s->total_tokens, w.lh, w.ldv, m->eps, w.gate,
-                                    w.lin_out_scale, 1, st));
+                                    w.lin_out_scale, 0, 1, st));
   }
 
   // experts of the tokens in `h`; their rows stay in sorted order for the norm that adds them up
@@ -369,7 +369,7 @@ struct Exec {
     const int* offsets = m->sort_meta + w.experts;
     if (!step(15, gemm(h, H, w.w_router, nullptr, m->router_buf, w.router_rows, w.router_rows, 1))) return false;
     if (!step(16, ksana_moe_topk(m->router_buf, w.router_rows, w.b_router, T, w.experts, w.top, w.groups, w.keep_groups,
-                                 m->expert_ids, m->expert_weights, st)))
+                                 0, 1.f, m->expert_ids, m->expert_weights, st)))
       return false;
     ++*launches;
     if (!step(17, ksana_moe_permute(h, H, m->expert_ids, T, w.top, H, 0, w.experts, m->sort_meta, m->pair_pos,
@@ -389,7 +389,7 @@ struct Exec {
     const int T = s->total_tokens, H = m->hidden, I = w.inter;
     if (w.plain) {
       if (!step(11, gemm(h, H, w.w_gu, w.b_up, m->gu_buf, I, I))) return false;
-      if (!step(12, ksana_relu2(m->gu_buf, m->act_buf, static_cast<long long>(T) * I, 1, st))) return false;
+      if (!step(12, ksana_relu2(m->gu_buf, I, m->act_buf, T, I, 1, st))) return false;
     } else if (w.w_gu_il != nullptr && T >= 384) {
       if (!step(11, ksana_gemm_bf16_geglu(h, w.w_gu_il, m->act_buf, T, 2 * I, H, H, H, I, st))) return false;
     } else {

@@ -6,7 +6,7 @@
 
 namespace ksana {
 
-// ---- router: top-k of logits (+ bias), softmax over the chosen ones ------------------------------------------------
+// ---- router: top-k of logits (+ bias), softmax over the chosen ones or (sigmoid) each one's sigmoid, times scale ------------------------------------------------
 // One warp per token; the token's logits sit in shared memory. Ties go to the lower index. Of `groups` equal groups of
 // neighbours only the `keep` with the largest logits take part.
 __device__ __forceinline__ void warp_argmax(float& v, int& i) {
@@ -22,7 +22,7 @@ __device__ __forceinline__ void warp_argmax(float& v, int& i) {
 }
 __global__ void __launch_bounds__(128)
 moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restrict__ bias, int T, int E, int k,
-                int groups, int keep, int* __restrict__ ids, float* __restrict__ weights) {
+                int groups, int keep, int sigmoid, float scale, int* __restrict__ ids, float* __restrict__ weights) {
   extern __shared__ float sm[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * 4 + warp;
@@ -70,7 +70,7 @@ moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restric
     warp_argmax(v, vi);
     if (vi >= E) vi = 0;  // (no finite logit is left)
     if (r == 0) top = v;
-    const float p = v == -INFINITY ? 0.f : expf(v - top);
+    const float p = v == -INFINITY ? 0.f : sigmoid ? sigmoid_f(v) : expf(v - top);
     sum += p;
     if (lane == 0) {
       my_ids[r] = vi;
@@ -79,7 +79,7 @@ moe_topk_kernel(const float* __restrict__ logits, int ld, const float* __restric
     }
     __syncwarp();
   }
-  for (int r = lane; r < k; r += 32) my_w[r] = sum > 0.f ? my_w[r] / sum : 0.f;
+  for (int r = lane; r < k; r += 32) my_w[r] = sigmoid ? my_w[r] * scale : sum > 0.f ? my_w[r] / sum * scale : 0.f;
 }
 
 // ---- counting sort by expert in one CTA ----------------------------------------------------------------------------
@@ -201,13 +201,15 @@ static int launched() { return cudaGetLastError() == cudaSuccess ? 0 : -5; }
 
 using namespace ksana;
 
+// scoring: 0 softmax over the chosen logits, 1 each one's sigmoid.
 KSANA_API int ksana_moe_topk(const float* logits, int ld, const float* bias, int T, int E, int k, int groups, int keep,
-                             int* ids, float* weights, cudaStream_t st) {
+                             int scoring, float scale, int* ids, float* weights, cudaStream_t st) {
   if (T <= 0) return 0;
   if (groups < 1 || E % groups || keep < 1 || keep > groups || k > E / groups * keep) return -2;
   const int smem = 4 * (E + (keep < groups ? 2 * groups : 0)) * static_cast<int>(sizeof(float));
   if (k < 1 || E > 2048 || smem > 48 * 1024) return -1;
-  moe_topk_kernel<<<(T + 3) / 4, 128, smem, st>>>(logits, ld, bias, T, E, k, groups, keep, ids, weights);
+  moe_topk_kernel<<<(T + 3) / 4, 128, smem, st>>>(logits, ld, bias, T, E, k, groups, keep, scoring, scale,
+                                                    ids, weights);
   return launched();
 }
 

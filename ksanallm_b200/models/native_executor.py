@@ -341,6 +341,8 @@ class MixerExecutor:
             return False
         if model.device.type != "cuda" or model.dtype != torch.bfloat16 or not model.layers or model.norm_w is None:
             return False
+        if model.gated_layers:
+            return False
         for layer in model.layers:
             lins = [layer.in_proj, layer.o_proj] + ([layer.ffn.up, layer.ffn.down] if layer.ffn is not None else [])
             if any(lin.kind != "dense" or lin.pre is not None or lin.weight.dtype != torch.bfloat16 or

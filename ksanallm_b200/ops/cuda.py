@@ -80,13 +80,19 @@ class _Sig:
     ksana_layer_norm = ([P, I, P, I, P, P, P, I, I, I, F, I, P], I)
     ksana_embedding_f32 = ([P, P, P, I, I, I, F, P, P, I, I, P], I)
     ksana_append_act = ([P, P, I, P, P, I, I, I, I, P, I, I, I, I, P], I)
-    ksana_moe_topk = ([P, I, P, I, I, I, I, I, P, P, P], I)
+    ksana_moe_topk = ([P, I, P, I, I, I, I, I, I, F, P, P, P], I)
     ksana_moe_sort = ([P, I, I, I, P, P, P, P], I)
     ksana_moe_gemm_any = ([P, I, P, I, P, P, P, I, I, I, I, I, P], I)
     ksana_silu_mul_any = ([P, P, I, I, I, P], I)
     ksana_gelu_mul = ([P, I, P, I, I, I, I, P], I)
     ksana_qk_norm_cache = ([P, I, P, I, P, I, P, P, P, P, F, P, P, I, I, I, I, I, I, I, I, P], I)
-    ksana_relu2 = ([P, P, LL, I, P], I)
+    ksana_relu2 = ([P, I, P, I, I, I, P], I)
+    ksana_gated_stream_norm = ([P, I, P, I, P, P, P, I, P, I, P, I, P, I, F, P, P, P, P, P, I, I, F, I, P], I)
+    ksana_qk_row_norm_cache = ([P, I, P, I, P, I, P, P, P, P, F, P, P, I, I, I, I, I, I, I, I, P], I)
+    ksana_talking_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, F, P, P, F, P, I, P, I, I, I, I, P], I)
+    ksana_token_mix = ([P, P, P, LL, LL, P, P, P, P, P, I, I, I, I, P], I)
+    ksana_tanh_parts = ([P, I, P, I, I, P], I)
+    ksana_time_mix_recurrent = ([P, I, P, I, P, I, P, I, P, P, P, LL, P, P, P, I, I, P, I, I, I, I, P], I)
     ksana_clamped_gate_mul = ([P, P, I, I, F, F, I, P], I)
     ksana_hyper_norm = ([P, I, P, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, F, I, P], I)
     ksana_head_gemm_any = ([P, LL, LL, P, P, LL, LL, I, I, I, I, I, P], I)
@@ -99,7 +105,7 @@ class _Sig:
     ksana_recurrence_step = ([P, I, P, I, P, P, P, P, P, P, P, P, P, I, I, I, P, I, I, I, P], I)
     ksana_recurrence_conv = ([P, I, P, P, P, P, P, P, P, I, I, P, I, I, I, P], I)
     ksana_recurrence_scan = ([P, I, P, I, P, P, P, P, P, P, P, P, I, I, I, P, I, I, I, I, I, P], I)
-    ksana_gated_norm = ([P, P, I, P, P, I, I, I, I, F, I, F, I, P], I)
+    ksana_gated_norm = ([P, P, I, P, P, I, I, I, I, F, I, F, I, I, P], I)
     ksana_softcap = ([P, I, P, I, I, F, P], I)
     ksana_window_attention_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, I, I, I, F, P, I, F, F, I, P, I, P, I, I, I, I, P], I)
     ksana_window_prefill = ([P, I, I, P, I, P, I, P, P, I, I, I, I, I, I, I, I, F, P, I, F, F, I, P, I, P, I, I, I, I, P], I)

@@ -66,9 +66,30 @@ def hyper_norm(x, scale, routed, streams, mix, out_w, streams_out, in_w, weight,
 
 
 def relu2(x: torch.Tensor) -> torch.Tensor:
-    x = x.contiguous()
-    out = torch.empty_like(x)
-    _check(lib().ksana_relu2(_ptr(x), _ptr(out), x.numel(), _KIND[x.dtype], _stream()), "relu2")
+    x2 = _rows(x)
+    out = torch.empty(x2.shape, dtype=x.dtype, device=x.device)
+    _check(lib().ksana_relu2(_ptr(x2), x2.stride(0), _ptr(out), x2.shape[0], x2.shape[1], _KIND[x.dtype], _stream()),
+           "relu2")
+    return out.view(x.shape)
+
+
+def gated_stream_norm(x, x_gate, routed, y, y_scale, y_gate, scale: float, stream_in, stream_out, weights, eps: float,
+                      out_dtype) -> torch.Tensor:
+    T, H = stream_in.shape
+    out = torch.empty(len(weights), T, H, dtype=out_dtype, device=stream_in.device)
+    rows, pos, wts = routed if routed is not None else (None, None, None)
+    assert stream_in.is_contiguous() and (stream_out is None or stream_out.is_contiguous()) and len(weights) in (1, 2)
+    assert all(t is None or t.is_contiguous() for t in (rows, pos, wts))
+    assert all(t is None or t.stride(1) == 1 and t.dtype == out_dtype for t in (x, x_gate, y, y_gate))
+    assert all(w.dtype == out_dtype and w.is_contiguous() for w in weights)
+
+    def ld(t):
+        return t.stride(0) if t is not None else 0
+    _check(lib().ksana_gated_stream_norm(
+        _ptr(x), ld(x), _ptr(x_gate), ld(x_gate), _ptr(rows), _ptr(pos), _ptr(wts), wts.shape[1] if wts is not None else 0,
+        _ptr(y), ld(y), _ptr(y_scale), ld(y_scale), _ptr(y_gate), ld(y_gate), float(scale), _ptr(stream_in),
+        _ptr(stream_out), _ptr(weights[0]), _ptr(weights[1]) if len(weights) > 1 else None, _ptr(out), T, H, float(eps),
+        _KIND[out_dtype], _stream()), "gated_stream_norm")
     return out
 
 
@@ -132,18 +153,21 @@ def _packed_heads(x: torch.Tensor) -> torch.Tensor:
 
 
 def qk_norm_cache(q, k, v, slot_mapping, cache, block_size: int, q_norm, k_norm, eps: float, positions=None,
-                  rotary=None) -> None:
+                  rotary=None, norm_all: bool = False, halves: bool = False) -> None:
     T, h, d = q.shape
+    if norm_all or halves:
+        assert norm_all and halves and k is not None and q_norm is not None
     hk, dv = (v.shape[1], v.shape[2]) if v is not None else (0, 0)
     for x in (q, k, v):
         if x is not None:
             _packed_heads(x)
     assert cache.dtype == q.dtype and cache.is_contiguous()
-    _check(lib().ksana_qk_norm_cache(_ptr(q), q.stride(0), _ptr(k), k.stride(0) if k is not None else 0, _ptr(v),
-                                     v.stride(0) if v is not None else 0, _ptr(slot_mapping), _ptr(cache), _ptr(q_norm),
-                                     _ptr(k_norm), float(eps), _ptr(positions) if rotary is not None else None,
-                                     _ptr(rotary), rotary.shape[1] if rotary is not None else 0, T, h, hk, d, dv,
-                                     block_size, _KIND[q.dtype], _stream()), "qk_norm_cache")
+    fn = lib().ksana_qk_row_norm_cache if norm_all else lib().ksana_qk_norm_cache
+    _check(fn(_ptr(q), q.stride(0), _ptr(k), k.stride(0) if k is not None else 0, _ptr(v),
+              v.stride(0) if v is not None else 0, _ptr(slot_mapping), _ptr(cache), _ptr(q_norm), _ptr(k_norm), float(eps),
+              _ptr(positions) if rotary is not None else None, _ptr(rotary),
+              rotary.shape[1] if rotary is not None else 0, T, h, hk, d, dv, block_size, _KIND[q.dtype], _stream()),
+           "qk_norm_cache")
 
 
 def window_attention(q, cache, meta, block_size: int, kv_heads: int, vdim: int, scale: float, window: int, bias,
@@ -235,12 +259,12 @@ def linear_attention(q, k, v, state, meta, decay, act: str, rotary, key_scale: f
     return out
 
 
-def gated_norm(o, g, weight, eps: float, gate: str, out_scale: float, out: torch.Tensor) -> None:
+def gated_norm(o, g, weight, eps: float, gate: str, out_scale: float, out: torch.Tensor, per_head: bool = False) -> None:
     T, h, dv = o.shape
     assert o.is_contiguous() and g.stride(1) == 1 and out.stride(1) == 1
     _check(lib().ksana_gated_norm(_ptr(o), _ptr(g), g.stride(0), _ptr(weight), _ptr(out), out.stride(0), T, h, dv,
-                                  float(eps), 1 if gate == "sigmoid" else 0, float(out_scale), _KIND[o.dtype],
-                                  _stream()), "gated_norm")
+                                  float(eps), 1 if gate == "sigmoid" else 0, float(out_scale), int(per_head),
+                                  _KIND[o.dtype], _stream()), "gated_norm")
 
 
 def softcap(logits: torch.Tensor, cap: float) -> torch.Tensor:

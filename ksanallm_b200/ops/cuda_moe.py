@@ -30,23 +30,23 @@ def moe_route(logits, top_k, scoring="softmax", norm_topk=False, n_group=1, topk
     return ids, w
 
 
-def moe_topk(logits, experts, top_k, bias=None, groups=1, keep=1):
+def moe_topk(logits, experts, top_k, bias=None, groups=1, keep=1, scoring="softmax", scale=1.0):
     """The ``top_k`` largest of the first ``experts`` logits (+ bias) of each token, in its ``keep`` best groups, softmax
-    over just those."""
+    over just those or each one's sigmoid, times ``scale``."""
     from . import cuda
     T = logits.shape[0]
     x = logits if logits.dtype == torch.float32 and logits.stride(1) == 1 else logits.float().contiguous()
     ids = torch.empty(T, top_k, dtype=torch.int32, device=logits.device)
     w = torch.empty(T, top_k, dtype=torch.float32, device=logits.device)
     code = cuda.lib().ksana_moe_topk(cuda._ptr(x), x.stride(0), cuda._ptr(bias), T, experts, top_k, groups, keep,
-                                     cuda._ptr(ids), cuda._ptr(w), cuda._stream())
+                                     int(scoring == "sigmoid"), float(scale), cuda._ptr(ids), cuda._ptr(w), cuda._stream())
     if code == -1:
-        return ref.moe_topk(logits, experts, top_k, bias, groups, keep)
+        return ref.moe_topk(logits, experts, top_k, bias, groups, keep, scoring, scale)
     cuda._check(code, "moe_topk")
     return ids, w
 
 
-def _pipeline_any(x, ids, w_gate_up, w_down, expert_offset, limit=0.0, alpha=1.0):
+def _pipeline_any(x, ids, w_gate_up, w_down, expert_offset, limit=0.0, alpha=1.0, plain=False):
     """expert_pipeline for fp32, and for sizes the tensor-core GEMM does not take: the same sort, plain GEMMs."""
     from . import cuda
     T, H = x.shape
@@ -61,29 +61,32 @@ def _pipeline_any(x, ids, w_gate_up, w_down, expert_offset, limit=0.0, alpha=1.0
     h1 = torch.empty(n, two_i, dtype=x.dtype, device=dev)
     cuda._check(lib.ksana_moe_gemm_any(p(x), x.stride(0), p(row_src), k, p(w_gate_up.contiguous()), p(h1), p(offsets), E,
                                        n, two_i, H, kind, st), "moe_gemm_any(gate_up)")
-    if limit:
+    if plain:
+        from . import cuda_mixer
+        a = cuda_mixer.relu2(h1)
+    elif limit:
         from . import cuda_mixer
         a = cuda_mixer.clamped_gate_mul(h1, limit, alpha)
     else:
         a = torch.empty(n, two_i // 2, dtype=x.dtype, device=dev)
         cuda._check(lib.ksana_silu_mul_any(p(h1), p(a), n, two_i // 2, kind, st), "silu_mul_any")
     y = torch.empty(n, H, dtype=x.dtype, device=dev)
-    cuda._check(lib.ksana_moe_gemm_any(p(a), two_i // 2, None, 1, p(w_down.contiguous()), p(y), p(offsets), E, n, H,
-                                       two_i // 2, kind, st), "moe_gemm_any(down)")
+    cuda._check(lib.ksana_moe_gemm_any(p(a), a.shape[1], None, 1, p(w_down.contiguous()), p(y), p(offsets), E, n, H,
+                                       a.shape[1], kind, st), "moe_gemm_any(down)")
     return y, pos
 
 
-def expert_pipeline(x, ids, w_gate_up, w_down, expert_offset=0, limit=0.0, alpha=1.0):
+def expert_pipeline(x, ids, w_gate_up, w_down, expert_offset=0, limit=0.0, alpha=1.0, plain=False):
     """Sort the (token, slot) pairs by local expert and run gate_up -> SiLU*mul (``limit`` > 0: the clamped gate of
-    ``reference.clamped_gate_mul``) -> down on the sorted rows.
+    ``reference.clamped_gate_mul``; ``plain``: up -> squared ReLU) -> down on the sorted rows.
     Returns (y [T*k, H] sorted expert outputs, pos [T*k] sorted row of each pair or -1 for non-local experts)."""
     from . import cuda
     if not supports(x, w_gate_up, w_down):
-        return _pipeline_any(x, ids, w_gate_up, w_down, expert_offset, limit, alpha)
+        return _pipeline_any(x, ids, w_gate_up, w_down, expert_offset, limit, alpha, plain)
     T, H = x.shape
     k = ids.shape[1]
     E_local, two_i, _ = w_gate_up.shape
-    I_ = two_i // 2
+    I_ = two_i if plain else two_i // 2
     dev = x.device
     key = (dev.index, E_local)
     meta = _meta.get(key)
@@ -103,7 +106,10 @@ def expert_pipeline(x, ids, w_gate_up, w_down, expert_offset=0, limit=0.0, alpha
     h1 = torch.empty(n, two_i, dtype=torch.bfloat16, device=dev)
     cuda._check(lib.ksana_moe_grouped_gemm(cuda._ptr(xs), cuda._ptr(w_gate_up), cuda._ptr(h1), cuda._ptr(offsets),
                                            E_local, n, two_i, H, st), "moe_grouped_gemm(gate_up)")
-    if limit:
+    if plain:
+        from . import cuda_mixer
+        a = cuda_mixer.relu2(h1)
+    elif limit:
         from . import cuda_mixer
         a = cuda_mixer.clamped_gate_mul(h1, limit, alpha)
     else:
