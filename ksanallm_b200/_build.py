@@ -82,14 +82,16 @@ def cuda_sources():
 FAMILY_SOURCES = {
     family: ("host_common", "elementwise", "sampling", "gemm_bf16", "gemm_bf16_2cta", "gemm_bf16_cluster_splitk", "moe",
              "moe_topk", "mixer_elementwise", "window_attention", "linear_attention", "hyper_connections", "head_gemm",
-             "gemm_batched", "latent_attention", "gated_recurrence", "talking_attention", "time_mix", "mixer_executor")
+             "gemm_batched", "latent_attention", "gated_recurrence", "talking_attention",
+             "talking_prefill", "talking_decode", "time_mix", "mixer_executor")
     for family in ("molopel", "givirax", "ladusun", "vibunex")
 }
 
 # Files compiled with IEEE division, square root and the accurate math functions: what they compute is specified in
 # 32-bit floats.
 EXACT_MATH = {"moe_topk", "mixer_elementwise", "window_attention", "linear_attention", "hyper_connections", "head_gemm",
-              "latent_attention", "gated_recurrence", "talking_attention", "time_mix"}
+              "latent_attention", "gated_recurrence", "talking_attention", "talking_prefill", "talking_decode",
+              "time_mix"}
 
 
 def cuda_library(family: str = "") -> Path:

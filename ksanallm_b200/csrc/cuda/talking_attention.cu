@@ -3,32 +3,9 @@
 //   o_ih = sum_j (sum_g talk[h][g] p_g(i, j)) v_j,
 // each head with the keys and values of its own key / value head, times the sigmoid of a gate per output. Scores, softmax,
 // mix and sums are 32-bit. Cache of a layer: [block][keys hk x bs x d | values hk x bs x dv]. Query i sees every j <= i.
-#include "host_common.h"
-#include "mixer_common.cuh"
+#include "talking.cuh"
 
 namespace ksana {
-
-struct TalkArgs {
-  const void* q;
-  int ldq;
-  const void* cache;
-  const int* block_tables;
-  int max_blocks;
-  const int* cu_q;
-  const int* kv_lens;
-  const int* seq_of_token;
-  int h, hk, d, dv, bs;
-  float scale;
-  const float* sink;   // [h]
-  const float* talk;   // [h][h]: to, from
-  float out_scale;
-  const void* gate;    // [T][ldg >= h * dv] in the storage type of q, or null
-  int ldg;
-  void* out;
-  int ldo;
-  __host__ __device__ size_t v_off() const { return static_cast<size_t>(hk) * bs * d; }
-  __host__ __device__ size_t block_elems() const { return static_cast<size_t>(hk) * bs * (d + dv); }
-};
 
 // ---- any size, any storage type -----------------------------------------------------------------------------------------
 // One CTA per new token, in two passes over its keys, 32 at a time: every head's maximum and sum, then the weights again,

@@ -569,28 +569,6 @@ static int launch_latent(const WindowAttnArgs& a, int total_tokens, const void* 
 // so nothing is computed for more than 8 NT - heads columns of padding. SHARED: values are keys, both products read the
 // same page. Head sizes below DP / DVP are filled up with zeros by TMA. The kernel is a stream over the cache; the tensor
 // instructions only keep the arithmetic out of its way.
-__device__ __forceinline__ void mma_16816(float* c, const uint32_t* a, uint32_t b0, uint32_t b1) {
-  asm volatile(
-      "mma.sync.aligned.m16n8k16.row.col.f32.bf16.bf16.f32 {%0, %1, %2, %3}, {%4, %5, %6, %7}, {%8, %9}, {%0, %1, %2, %3};"
-      : "+f"(c[0]), "+f"(c[1]), "+f"(c[2]), "+f"(c[3])
-      : "r"(a[0]), "r"(a[1]), "r"(a[2]), "r"(a[3]), "r"(b0), "r"(b1));
-}
-template <bool TRANS>
-__device__ __forceinline__ void ldmatrix_x4(uint32_t* r, uint32_t addr) {
-  if constexpr (TRANS)
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.trans.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-  else
-    asm volatile("ldmatrix.sync.aligned.m8n8.x4.shared.b16 {%0, %1, %2, %3}, [%4];"
-                 : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr) : "memory");
-}
-// an 8 x 8 matrix of 16-bit values held across the warp, transposed
-__device__ __forceinline__ uint32_t transpose_8x8(uint32_t v) {
-  uint32_t r;
-  asm volatile("movmatrix.sync.aligned.m8n8.trans.b16 %0, %1;" : "=r"(r) : "r"(v));
-  return r;
-}
-
 template <int DP, int DVP, bool SHARED>
 struct WindowDecodeSmem {
   static constexpr int K_BYTES = 16 * DP * 2;

@@ -90,6 +90,10 @@ class _Sig:
     ksana_gated_stream_norm = ([P, I, P, I, P, P, P, I, P, I, P, I, P, I, F, P, P, P, P, P, I, I, F, I, P], I)
     ksana_qk_row_norm_cache = ([P, I, P, I, P, I, P, P, P, P, F, P, P, I, I, I, I, I, I, I, I, P], I)
     ksana_talking_any = ([P, I, P, P, I, P, P, P, I, I, I, I, I, F, P, P, F, P, I, P, I, I, I, I, P], I)
+    ksana_talking_prefill_bytes = ([I, I, P, P], LL)
+    ksana_talking_prefill = ([P, I, I, P, I, P, I, P, P, I, I, I, I, I, F, P, P, F, P, I, P, I, I, P, P, P, LL, P, P], I)
+    ksana_talking_decode_bytes = ([I, I, I], LL)
+    ksana_talking_decode = ([P, I, P, I, P, I, P, P, I, I, I, I, I, F, P, P, F, P, I, P, I, I, I, I, P, LL, P], I)
     ksana_token_mix = ([P, P, P, LL, LL, P, P, P, P, P, I, I, I, I, P], I)
     ksana_tanh_parts = ([P, I, P, I, I, P], I)
     ksana_time_mix_recurrent = ([P, I, P, I, P, I, P, I, P, P, P, LL, P, P, P, I, I, P, I, I, I, I, P], I)
