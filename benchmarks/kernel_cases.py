@@ -21,6 +21,11 @@ each case is small (at most a few GB on the device) and launches its kernel a ha
     python benchmarks/kernel_cases.py recurrence_prefill [T C blocks taps sequences]
     python benchmarks/kernel_cases.py recurrence_decode [B C blocks taps]
     python benchmarks/kernel_cases.py ladusun_rows [T H streams h hk d rank rot]
+    python benchmarks/kernel_cases.py talking_prefill [T h hk d dv]
+    python benchmarks/kernel_cases.py talking_decode [B ctx h hk d dv]
+    python benchmarks/kernel_cases.py timemix_prefill [T heads dim sequences]
+    python benchmarks/kernel_cases.py timemix_decode [B heads dim]
+    python benchmarks/kernel_cases.py vibunex_rows [T H h hk d]
     python benchmarks/kernel_cases.py all
 """
 import json
@@ -31,7 +36,7 @@ import torch
 
 sys.path.insert(0, os.path.dirname(os.path.dirname(os.path.abspath(__file__))))
 from ksanallm_b200.engine.step_input import make_step_input  # noqa: E402
-from ksanallm_b200.ops import cuda, cuda_latent, cuda_mixer, cuda_moe, cuda_recurrence  # noqa: E402
+from ksanallm_b200.ops import cuda, cuda_latent, cuda_mixer, cuda_moe, cuda_recurrence, cuda_talking, cuda_timemix  # noqa: E402
 from ksanallm_b200.ops import reference as ref  # noqa: E402
 
 DEV = "cuda"
@@ -439,6 +444,120 @@ def case_ladusun_rows():
     return dict(kernel="ladusun_rows", T=T, H=H, streams=S, **out)
 
 
+def _talking_setup(q_lens, kv_lens, h, hk, d, dv, prefill):
+    _, _, bt, cu = _attn_setup(q_lens, kv_lens, 1, 1)
+    T = cu[-1]
+    bf = lambda *s: torch.randn(*s, device=DEV).to(torch.bfloat16)  # noqa: E731
+    cache = bf(int(bt.max()) + 2, 16 * hk * (d + dv))
+    pos = [n - q + i for n, q in zip(kv_lens, q_lens) for i in range(q)]
+    meta = make_step_input([0] * T, pos, [0] * T, cu, kv_lens, bt, num_prefill=prefill, device=DEV)
+    x, out = bf(T, h * (d + dv)), bf(T, h * dv)
+    sink, talk = torch.randn(h, device=DEV), (torch.eye(h, device=DEV) + 0.3 * torch.randn(h, h, device=DEV)).bfloat16().float()
+    return lambda i: cuda_talking.talking_attention(x[:, :h * d].unflatten(1, (h, d)), cache, meta, 16, hk, dv, d ** -0.5, sink,
+                                                    talk, 1.0, out, x[:, h * d:])
+
+
+def case_talking_prefill():
+    T, h, hk, d, dv = args_or([8192, 32, 8, 128, 128])
+    us = timeit(_talking_setup([T], [T], h, hk, d, dv, 1), iters=5)
+    pairs = T * (T + 1) / 2
+    fl, mix = 2.0 * h * (d + dv) * pairs, 2.0 * h * h * pairs
+    p = peaks()
+    return dict(kernel="talking_prefill", T=T, h=h, hk=hk, d=d, dv=dv, us=round(us, 1), tflops=round((fl + mix) / us / 1e6, 1),
+                frac_of_measured_bf16=round((fl + mix) / us / 1e6 / p["bf16_tflops"], 3),
+                frac_without_the_mix=round(fl / us / 1e6 / p["bf16_tflops"], 3))
+
+
+def case_talking_decode():
+    B, ctx, h, hk, d, dv = args_or([128, 1024, 32, 8, 128, 128])
+    us = timeit(_talking_setup([1] * B, [ctx] * B, h, hk, d, dv, 0))
+    by, p = B * ctx * hk * (d + dv) * 2, peaks()
+    return dict(kernel="talking_decode", B=B, ctx=ctx, h=h, hk=hk, d=d, dv=dv, us=round(us, 1), kv_gb=round(by / 1e9, 3),
+                gbs=round(by / us / 1e3, 1), frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+
+
+def _timemix_setup(lens, q_lens, h, d, prefill, copies=2):
+    B, T, n = len(lens), sum(q_lens), h * d
+    cu = [0]
+    for q in q_lens:
+        cu.append(cu[-1] + q)
+    meta = make_step_input([0] * T, [0] * T, [0] * T, cu, lens, torch.zeros(B, 1), num_prefill=prefill, device=DEV,
+                           state_slots=list(range(B)))
+    xs = [(torch.randn(3, T, n, device=DEV) * 0.3).to(torch.bfloat16) for _ in range(copies)]
+    zs = [torch.randn(T, n, device=DEV) for _ in range(copies)]
+    states = [torch.zeros(B, 1, 1, h * d * d + n, device=DEV) for _ in range(copies)]
+    w0, u = torch.randn(n, device=DEV) - 3, torch.randn(h, d, device=DEV)
+    return lambda i: cuda_timemix.time_mix(xs[i % copies][0], xs[i % copies][1], xs[i % copies][2], zs[i % copies], w0, u,
+                                           states[i % copies], meta)
+
+
+def case_timemix_prefill():
+    T, h, d, n = args_or([8192, 64, 64, 1])
+    us = timeit(_timemix_setup([T // n] * n, [T // n] * n, h, d, n), iters=5)
+    by = T * h * d * (4 * 2 + 4)  # r, k, v, o in 16 bits and the decay's exponent in 32
+    fl = T * h * (2.0 * d * d * 2 + 64 * 2 * d)  # state update and read-out + the causal half of a chunk of 64
+    p = peaks()
+    floor = max(by / p["hbm_gbs"] / 1e3, fl / p["bf16_tflops"] / 1e6)
+    return dict(kernel="timemix_prefill", T=T, h=h, d=d, sequences=n, us=round(us, 1), roofline_us=round(floor, 1),
+                frac_of_roofline=round(floor / us, 3))
+
+
+def case_timemix_decode():
+    B, h, d = args_or([128, 64, 64])
+    us = timeit(_timemix_setup([100] * B, [1] * B, h, d, 0))
+    by, p = 2 * B * h * d * d * 4, peaks()
+    return dict(kernel="timemix_decode", B=B, h=h, d=d, us=round(us, 1), state_gb=round(by / 2e9, 3), gbs=round(by / us / 1e3, 1),
+                frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+
+
+def case_vibunex_rows():
+    """Row-wise kernels of gated residuals, time mixing and weight-mixing attention."""
+    T, H, h, hk, d = args_or([8192, 4096, 32, 8, 128])
+    bf = lambda *s: torch.randn(*s, device=DEV).to(torch.bfloat16)  # noqa: E731
+    p, out = peaks(), {}
+
+    def add(name, us, by):
+        out[name] = dict(us=round(us, 1), gbs=round(by / us / 1e3, 1), frac_of_measured_hbm=round(by / us / 1e3 / p["hbm_gbs"], 3))
+    xs, r32, w, k = [bf(T, 4 * H) for _ in range(2)], [torch.randn(T, H, device=DEV) for _ in range(2)], bf(H), 2
+    y2, pos, wts = bf(T * k, H), torch.randperm(T * k, dtype=torch.int32, device=DEV), torch.rand(T, k, device=DEV)
+    z = torch.randn(T, 24, device=DEV)
+
+    def norm(i, routed):
+        x = xs[i % 2]
+        cuda_mixer.gated_stream_norm(x[:, :H], x[:, H:2 * H], (y2, pos, wts) if routed else None, x[:, 2 * H:3 * H], z[:, 16],
+                                     x[:, 3 * H:], 0.5, r32[i % 2], r32[i % 2], [w, w], 1e-6, torch.bfloat16)
+    add("gated_stream_norm", timeit(lambda i: norm(i, False)), T * H * 20)
+    add("gated_stream_norm_routed", timeit(lambda i: norm(i, True)), T * H * (20 + 2 * k))
+    r16 = [bf(T, H) for _ in range(2)]
+    add("rms_norm", timeit(lambda i: cuda.rms_norm(r16[i % 2], w, 1e-6, r16[1 - i % 2])), T * H * 8)
+    meta = make_step_input([0] * T, [0] * T, [0] * T, [0, T], [T], torch.zeros(1, 1), num_prefill=1, device=DEV, state_slots=[0])
+    mu, state = torch.rand(5, H, device=DEV), torch.zeros(1, 1, 1, H, device=DEV)
+    add("token_mix", timeit(lambda i: cuda_timemix.token_mix(r16[i % 2], mu, state, meta)), T * H * 12)
+    o, g, y, wf = bf(T, H // 64, 64), [bf(T, H) for _ in range(2)], bf(T, H), torch.ones(H, device=DEV)
+    add("gated_head_norm_weight", timeit(lambda i: cuda_mixer.gated_norm(o, g[i % 2], wf, 1e-6, "silu", 1.0, y, True)), T * H * 6)
+    add("gated_head_norm", timeit(lambda i: cuda_mixer.gated_norm(o, g[i % 2], None, 1e-6, "silu", 1.0, y)), T * H * 6)
+    slots, table = torch.arange(T, dtype=torch.int32, device=DEV), torch.randn(T, d // 2, device=DEV)
+    cache = torch.zeros((T + 15) // 16, hk * 16 * 2 * d, dtype=torch.bfloat16, device=DEV)
+    qkv = [bf(T, (h + 2 * hk) * d) for _ in range(3)]
+    wq, wk, wb = torch.ones(h * d, device=DEV), torch.ones(hk * d, device=DEV), torch.ones(d, device=DEV, dtype=torch.bfloat16)
+
+    def parts(x):
+        return x[:, :h * d].unflatten(1, (h, d)), x[:, h * d:(h + hk) * d].unflatten(1, (hk, d)), x[:, (h + hk) * d:].unflatten(1, (hk, d))
+    by = T * d * 2 * (2 * h + 4 * hk)
+    add("qk_row_norm_cache", timeit(lambda i: cuda_mixer.qk_norm_cache(*parts(qkv[i % 3]), slots, cache, 16, wq, wk, 1e-6, slots, table,
+                                                                       True, True)), by)
+    full = torch.randn(T, d, device=DEV)
+    add("rope_cache", timeit(lambda i: cuda.rope_qknorm_cache(*parts(qkv[i % 3]), slots, full, slots, cache.view(-1, 2, hk, 16, d), wb, wb,
+                                                              1e-6)), by)
+    a32 = torch.randn(T, 64, device=DEV)
+    add("tanh_parts", timeit(lambda i: cuda_timemix.tanh_parts(a32, torch.bfloat16)), T * 64 * 8)
+    add("moe_topk_sigmoid", timeit(lambda i: cuda_moe.moe_topk(z, 16, 2, None, 1, 1, "sigmoid", 1.5)), T * (16 + 4) * 4)
+    add("moe_route", timeit(lambda i: cuda_moe.moe_route(z, 2, "softmax", True)), T * (16 + 4) * 4)
+    us = [bf(T, 2 * H) for _ in range(2)]
+    add("relu2_strided", timeit(lambda i: cuda_mixer.relu2(us[i % 2][:, H:])), T * H * 4)
+    return dict(kernel="vibunex_rows", T=T, H=H, h=h, hk=hk, d=d, **out)
+
+
 def case_mixer_rows():
     """The row-wise kernels, each beside its counterpart of the dense models."""
     T, H, h, hk, d = args_or([8192, 4096, 32, 8, 128])
@@ -502,7 +621,9 @@ CASES = dict(gemm=case_gemm, gemm_fp8=case_gemm_fp8, gemm_int4=case_gemm_int4, d
              moe=case_moe, window_prefill=case_window_prefill, window_decode=case_window_decode,
              linear_prefill=case_linear_prefill, linear_decode=case_linear_decode, mixer_rows=case_mixer_rows,
              latent_prefill=case_latent_prefill, latent_decode=case_latent_decode, recurrence_prefill=case_recurrence_prefill,
-             recurrence_decode=case_recurrence_decode, ladusun_rows=case_ladusun_rows)
+             recurrence_decode=case_recurrence_decode, ladusun_rows=case_ladusun_rows, talking_prefill=case_talking_prefill,
+             talking_decode=case_talking_decode, timemix_prefill=case_timemix_prefill, timemix_decode=case_timemix_decode,
+             vibunex_rows=case_vibunex_rows)
 
 if __name__ == "__main__":
     which = sys.argv[1] if len(sys.argv) > 1 else "all"
