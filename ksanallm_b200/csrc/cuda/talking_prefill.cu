@@ -46,8 +46,9 @@ talking_stats_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
                      float* __restrict__ lse, unsigned int* err) {
   using L_ = TalkStatsSmem<DP>;
   int b, qt;
-  if (!find_unit(a, rd.num_seqs, rd.unit0 + blockIdx.x, &b, &qt)) return;
-  const int head = blockIdx.y, kh = head / (a.h / a.hk);
+  // (blocks further along a prompt are longer: they go first)
+  if (!find_unit(a, rd.num_seqs, rd.unit0 + gridDim.y - 1 - blockIdx.y, &b, &qt)) return;
+  const int head = blockIdx.x, kh = head / (a.h / a.hk);
   const int q0 = a.cu_q[b], q_len = a.cu_q[b + 1] - q0, L = a.kv_lens[b];
   const int row_pos = L - q_len + qt * 128;
   const int tid = threadIdx.x, warp = tid >> 5;
@@ -278,6 +279,7 @@ talking_weights_kernel(const __grid_constant__ CUtensorMap tmK, TalkArgs a, Talk
   bool ok = true;
   for (int t = 0; t < live; ++t) {
     const int key = key0 + t * 32;
+    const bool edge = key + 31 > pos0;  // some of these keys are later than some query
     for (int ci = 0; ci < nc; ++ci) {
       const int n = t * nc + ci;
       if (ok) ok = mbar_wait_bounded(&full[warp * 2 + (n & 1)], (n >> 1) & 1, abort_flag, err);
@@ -316,13 +318,18 @@ talking_weights_kernel(const __grid_constant__ CUtensorMap tmK, TalkArgs a, Talk
           for (int e = 0; e < 2; ++e) {
             if (at[k][e] < 0) continue;
             uint8_t* dst = sP + at[k][e] + j2 * 2;
+            if (edge) {
+#pragma unroll
+              for (int nt = 0; nt < 4; ++nt) {
+                const int j = key + nt * 8 + j2;
+                if (j > pos[k][e]) acc[k][nt][e * 2] = -INFINITY;
+                if (j + 1 > pos[k][e]) acc[k][nt][e * 2 + 1] = -INFINITY;
+              }
+            }
 #pragma unroll
             for (int nt = 0; nt < 4; ++nt) {
-              const int j = key + nt * 8 + j2;
-              float x = ex2_ftz(fmaf(acc[k][nt][e * 2], scale2, -ls[k][e]));
-              float y = ex2_ftz(fmaf(acc[k][nt][e * 2 + 1], scale2, -ls[k][e]));
-              if (j > pos[k][e]) x = 0.f;
-              if (j + 1 > pos[k][e]) y = 0.f;
+              const float x = ex2_ftz(fmaf(acc[k][nt][e * 2], scale2, -ls[k][e]));
+              const float y = ex2_ftz(fmaf(acc[k][nt][e * 2 + 1], scale2, -ls[k][e]));
               uint32_t low;
               *reinterpret_cast<uint32_t*>(dst + nt * 16) = split_bf16(x, y, &low);
               *reinterpret_cast<uint32_t*>(dst + HP * ROW + nt * 16) = low;
@@ -370,10 +377,17 @@ talking_weights_kernel(const __grid_constant__ CUtensorMap tmK, TalkArgs a, Talk
         }
       }
       __syncwarp();
-      for (int x = lane; x < 2 * a.h * 4; x += 32) {
-        const int part = x / (a.h * 4), g = (x >> 2) % a.h, ch = x & 3;
-        *reinterpret_cast<uint4*>(wout + part * plane + (static_cast<size_t>(g) * 128 + i) * rd.pitch + key + ch * 8) =
-            *reinterpret_cast<const uint4*>(P + (part * HP + g) * ROW + ch * 16);
+      {
+        const int ch = lane & 3;
+        const uint8_t* src = P + (lane >> 2) * ROW + ch * 16;
+        __nv_bfloat16* dst = wout + (static_cast<size_t>(lane >> 2) * 128 + i) * rd.pitch + key + ch * 8;
+        const size_t step = static_cast<size_t>(8 * 128) * rd.pitch;
+#pragma unroll
+        for (int g0 = 0; g0 < HP; g0 += 8, src += 8 * ROW, dst += step)
+          if (g0 + (lane >> 2) < a.h) {
+            *reinterpret_cast<uint4*>(dst) = *reinterpret_cast<const uint4*>(src);
+            *reinterpret_cast<uint4*>(dst + plane) = *reinterpret_cast<const uint4*>(src + HP * ROW);
+          }
       }
     }
     __syncthreads();
@@ -406,8 +420,9 @@ __global__ void __launch_bounds__(192)
 talking_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmV, TalkArgs a,
                       TalkRound rd, unsigned int* err) {
   using L_ = TalkValuesSmem<DVP>;
+  const int unit = gridDim.y - 1 - blockIdx.y;  // longest first
   int b, qt;
-  if (!find_unit(a, rd.num_seqs, rd.unit0 + blockIdx.y, &b, &qt)) return;
+  if (!find_unit(a, rd.num_seqs, rd.unit0 + unit, &b, &qt)) return;
   const int head = blockIdx.x, kh = head / (a.h / a.hk);
   const int q_len = a.cu_q[b + 1] - a.cu_q[b], L = a.kv_lens[b];
   const int n = (min(L, L - q_len + qt * 128 + 128) + 127) / 128;
@@ -440,7 +455,7 @@ talking_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
     if ((tid & 31) == 0) {
       const int* bt = a.block_tables + static_cast<size_t>(b) * a.max_blocks;
       const int n_pages = (L + TALK_PAGE - 1) / TALK_PAGE;
-      const int row_hi = (blockIdx.y * 2 * a.h + head) * 128, row_lo = row_hi + a.h * 128;
+      const int row_hi = (unit * 2 * a.h + head) * 128, row_lo = row_hi + a.h * 128;
       bool ok = true;
       int loads = 0;
       for (int i = 0; i < n; ++i) {
@@ -512,7 +527,7 @@ talking_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
 }
 
 // ---- launches ----------------------------------------------------------------------------------------------------------
-constexpr long long TALK_W_BYTES = 256ll << 20;  // weights written out at a time, unless one block of rows needs more
+constexpr long long TALK_W_BYTES = 1ll << 30;  // weights written out at a time, unless one block of rows needs more
 
 static int talk_units(const int* cu, int b) { return (cu[b + 1] - cu[b] + 127) / 128; }
 // keys of a block's rows, up to the multiple of 128 that its tiles cover
@@ -548,7 +563,7 @@ static int launch_stats(const TalkArgs& a, const CUtensorMap& tq, const CUtensor
                         float* lse, cudaStream_t st) {
   auto kern = talking_stats_kernel<DP>;
   if (KSANA_SMEM_ONCE(kern, TalkStatsSmem<DP>::TOTAL) != 0) return -4;
-  kern<<<dim3(units, a.h), 160, TalkStatsSmem<DP>::TOTAL, st>>>(tq, tk, a, rd, lse, error_word());
+  kern<<<dim3(a.h, units), 160, TalkStatsSmem<DP>::TOTAL, st>>>(tq, tk, a, rd, lse, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
 template <int DP, int HK>
