@@ -96,6 +96,8 @@ class _Sig:
     ksana_talking_decode = ([P, I, P, I, P, I, P, P, I, I, I, I, I, F, P, P, F, P, I, P, I, I, I, I, P, LL, P], I)
     ksana_token_mix = ([P, P, P, LL, LL, P, P, P, P, P, I, I, I, I, P], I)
     ksana_tanh_parts = ([P, I, P, I, I, P], I)
+    ksana_time_mix_scratch = ([I, I, I, I], LL)
+    ksana_time_mix_chunked = ([P, I, P, I, P, I, P, I, P, P, P, LL, P, P, P, I, I, P, I, I, I, P, P], I)
     ksana_time_mix_recurrent = ([P, I, P, I, P, I, P, I, P, P, P, LL, P, P, P, I, I, P, I, I, I, I, P], I)
     ksana_clamped_gate_mul = ([P, P, I, I, F, F, I, P], I)
     ksana_hyper_norm = ([P, I, P, P, P, P, I, P, I, P, P, P, P, P, P, I, I, I, F, I, P], I)
