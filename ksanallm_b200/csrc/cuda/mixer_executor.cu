@@ -97,9 +97,52 @@ int ksana_recurrence_scan(const void* y, int ldy, const void* x, int ldx, float*
                           const int* kv_lens, const void* u, const float* z, const float* gates_b, const float* rate,
                           int C, int K, int B, void* out, int ldo, int seq_base, int num_seqs, int tok_base, int kind,
                           cudaStream_t st);
+int ksana_gated_stream_norm(const void* x, int ldx, const void* xg, int ldxg, const void* rows, const int* pos,
+                            const float* weights, int k, const void* y, int ldy, const float* ys, int ldys, const void* yg,
+                            int ldyg, float scale, const float* in, float* stream, const void* w0, const void* w1, void* out,
+                            int tokens, int H, float eps, int kind, cudaStream_t st);
+int ksana_qk_row_norm_cache(void* q, int ldq, const void* k, int ldk, const void* v, int ldv, const int* slots, void* cache,
+                            const float* qw, const float* kw, float eps, const int* positions, const float* rotary, int rd,
+                            int tokens, int h, int hk, int d, int dv, int bs, int kind, cudaStream_t st);
+int ksana_talking_any(const void* q, int ldq, const void* cache, const int* block_tables, int max_blocks, const int* cu_q,
+                      const int* kv_lens, const int* seq_of_token, int h, int hk, int d, int dv, int bs, float scale,
+                      const float* sink, const float* talk, float out_scale, const void* gate, int ldg, void* out, int ldo,
+                      int tok_base, int tokens, int kind, cudaStream_t st);
+long long ksana_talking_prefill_bytes(int h, int num_seqs, const int* cu_q_host, const int* kv_lens_host);
+int ksana_talking_prefill(const void* q, int ldq, int total_tokens, const void* cache, int num_blocks,
+                          const int* block_tables, int max_blocks, const int* cu_q, const int* kv_lens, int h, int hk, int d,
+                          int dv, int bs, float scale, const float* sink, const float* talk, float out_scale,
+                          const void* gate, int ldg, void* out, int ldo, int num_seqs, const int* cu_q_host,
+                          const int* kv_lens_host, void* scratch, long long scratch_bytes, int* launches, cudaStream_t st);
+long long ksana_talking_decode_bytes(int h, int num_seqs, int max_kv);
+int ksana_talking_decode(const void* q, int ldq, const void* cache, int num_blocks, const int* block_tables, int max_blocks,
+                         const int* cu_q, const int* kv_lens, int h, int hk, int d, int dv, int bs, float scale,
+                         const float* sink, const float* talk, float out_scale, const void* gate, int ldg, void* out,
+                         int ldo, int seq_base, int num_seqs, int max_kv, void* scratch, long long scratch_bytes,
+                         cudaStream_t st);
+int ksana_token_mix(const void* h, const float* mu, float* last, long long slot_pitch, long long slots_total,
+                    const int* slots, const int* cu_q, const int* kv_lens, const int* seq_of_token, void* out, int tokens,
+                    int W, int rows, int kind, cudaStream_t st);
+int ksana_tanh_parts(const float* x, int n, void* out, int rows, int kind, cudaStream_t st);
+int ksana_time_mix_recurrent(const void* r, int ldr, const void* k, int ldk, const void* v, int ldv, const float* z, int ldz,
+                             const float* w0, const float* u, float* state, long long slot_pitch, const int* slots,
+                             const int* cu_q, const int* kv_lens, int h, int d, void* out, int seq_base, int num_seqs,
+                             int one_token, int kind, cudaStream_t st);
+long long ksana_time_mix_scratch(int tokens, int num_seqs, int h, int d);
+int ksana_time_mix_chunked(const void* r, int ldr, const void* k, int ldk, const void* v, int ldv, const float* z, int ldz,
+                           const float* w0, const float* u, float* state, long long slot_pitch, const int* slots,
+                           const int* cu_q, const int* kv_lens, int h, int d, void* out, int seq_base, int num_seqs,
+                           int max_q, float* scratch, cudaStream_t st);
 }
 
 namespace {
+
+// Scratch of weight-mixing attention in a step.
+static long long talking_bytes(const KsanaMixerStep* s, const KsanaMixerLayer& w) {
+  const long long p = ksana_talking_prefill_bytes(w.h, s->num_prefill, s->cu_q_host, s->kv_lens_host);
+  const long long d = s->one_token ? ksana_talking_decode_bytes(w.h, s->num_decode, s->max_kv_decode) : 0;
+  return p > d ? p : d;
+}
 
 // How latent attention uses its scratch in a step: contexts of prompts (latents, then keys and values) in rounds of at
 // most expand_bytes, absorbed queries and weighted latents for the tokens from `first` on.
@@ -367,17 +410,19 @@ struct Exec {
   bool experts(const KsanaMixerLayer& w) {
     const int T = s->total_tokens, H = m->hidden, I = w.expert_inter, n = T * w.top;
     const int* offsets = m->sort_meta + w.experts;
+    const int in_rows = w.experts_plain ? I : 2 * I;
     if (!step(15, gemm(h, H, w.w_router, nullptr, m->router_buf, w.router_rows, w.router_rows, 1))) return false;
     if (!step(16, ksana_moe_topk(m->router_buf, w.router_rows, w.b_router, T, w.experts, w.top, w.groups, w.keep_groups,
-                                 0, 1.f, m->expert_ids, m->expert_weights, st)))
+                                 w.scoring, w.router_scale, m->expert_ids, m->expert_weights, st)))
       return false;
     ++*launches;
     if (!step(17, ksana_moe_permute(h, H, m->expert_ids, T, w.top, H, 0, w.experts, m->sort_meta, m->pair_pos,
                                     m->pair_src, m->rows_buf, st)))
       return false;
-    if (!step(18, ksana_moe_grouped_gemm(m->rows_buf, w.w_expert_gu, m->rows_gu_buf, offsets, w.experts, n, 2 * I, H, st)))
+    if (!step(18, ksana_moe_grouped_gemm(m->rows_buf, w.w_expert_gu, m->rows_gu_buf, offsets, w.experts, n, in_rows, H, st)))
       return false;
-    int rc = w.limit > 0.f ? ksana_clamped_gate_mul(m->rows_gu_buf, m->rows_act_buf, n, I, w.limit, w.alpha, 1, st)
+    int rc = w.experts_plain ? ksana_relu2(m->rows_gu_buf, I, m->rows_act_buf, n, I, 1, st)
+             : w.limit > 0.f ? ksana_clamped_gate_mul(m->rows_gu_buf, m->rows_act_buf, n, I, w.limit, w.alpha, 1, st)
                            : ksana_silu_mul(m->rows_gu_buf, 2 * I, m->rows_act_buf, I, n, I, st);
     if (rc == -1) rc = ksana_silu_mul_any(m->rows_gu_buf, m->rows_act_buf, n, I, 1, st);
     if (!step(19, rc)) return false;
@@ -399,7 +444,120 @@ struct Exec {
     return step(13, gemm(m->act_buf, I, w.w_down, w.plain ? w.b_down : nullptr, m->proj_buf, H, H));
   }
 
+  bool talking(const KsanaMixerLayer& w, char* x, void* out) {
+    const int T = s->total_tokens, ld = w.n_in;
+    char *k = x + static_cast<size_t>(w.h * w.d) * 2, *v = k + static_cast<size_t>(w.hk * w.d) * 2;
+    const char* gate = w.out_gate ? v + static_cast<size_t>(w.hk * w.dv) * 2 : nullptr;
+    auto append = w.qk_norm_all ? ksana_qk_row_norm_cache : ksana_qk_norm_cache;
+    if (!step(2, append(x, ld, k, ld, v, ld, s->slot_mapping, w.kv, w.q_norm, w.k_norm, m->eps, s->positions, w.rot_table,
+                        w.rot, T, w.h, w.hk, w.d, w.dv, m->block_size, 1, st)))
+      return false;
+    auto general = [&](int first, int count) {
+      return ksana_talking_any(x, ld, w.kv, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, s->seq_of_token, w.h, w.hk,
+                               w.d, w.dv, m->block_size, w.scale, w.talk_sink, w.talk_mix, w.attn_out_scale, gate, ld, out,
+                               w.k_out, first, count, 1, st);
+    };
+    if (s->num_prefill > 0) {
+      int n = 0;
+      int rc = ksana_talking_prefill(x, ld, T, w.kv, m->num_blocks, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, w.h,
+                                     w.hk, w.d, w.dv, m->block_size, w.scale, w.talk_sink, w.talk_mix, w.attn_out_scale, gate,
+                                     ld, out, w.k_out, s->num_prefill, s->cu_q_host, s->kv_lens_host, m->lat_buf,
+                                     m->lat_bytes, &n, st);
+      if (rc == -1) rc = general(0, s->prefill_tokens); else *launches += n - 1;
+      if (!step(31, rc)) return false;
+    }
+    if (s->num_decode > 0) {
+      int rc = -1;
+      if (s->one_token) {
+        rc = ksana_talking_decode(x, ld, w.kv, m->num_blocks, s->block_tables, s->max_blocks, s->cu_q, s->kv_lens, w.h, w.hk,
+                                  w.d, w.dv, m->block_size, w.scale, w.talk_sink, w.talk_mix, w.attn_out_scale, gate, ld, out,
+                                  w.k_out, s->num_prefill, s->num_decode, s->max_kv_decode, m->lat_buf, m->lat_bytes, st);
+        if (rc == 0) ++*launches;
+      }
+      if (rc == -1) rc = general(s->prefill_tokens, T - s->prefill_tokens);
+      if (!step(32, rc)) return false;
+    }
+    return true;
+  }
+
+  bool time_mix(const KsanaMixerLayer& w, char* out) {
+    const int T = s->total_tokens, H = m->hidden, n = w.mh * w.md, ld = w.mpad;
+    const long long pitch = static_cast<long long>(n) * w.md + H;  // of a state slot: the heads' states, the last token
+    if (!step(33, ksana_token_mix(h, w.mu, w.state + pitch - H, pitch, 1, s->state_slots, s->cu_q, s->kv_lens,
+                                  s->seq_of_token, m->mixes_buf, T, H, 5, 1, st)))
+      return false;
+    const char* mixes = static_cast<const char*>(m->mixes_buf);
+    char* rkvg = static_cast<char*>(m->rkvg_buf);
+    const size_t in = static_cast<size_t>(T) * H * 2, to = static_cast<size_t>(T) * ld * 2;
+    for (int i = 0; i < 4; ++i)
+      if (!step(34, gemm(mixes + i * in, H, static_cast<const char*>(w.w_mix) + static_cast<size_t>(i) * ld * H * 2, nullptr,
+                         rkvg + i * to, ld, ld)))
+        return false;
+    if (!step(35, gemm(mixes + 4 * in, H, w.w_decay1, nullptr, m->rank_buf, w.mrank, w.mrank, 1))) return false;
+    if (!step(36, ksana_tanh_parts(m->rank_buf, w.mrank, m->tanh_buf, T, 1, st))) return false;
+    if (!step(37, gemm(m->tanh_buf, 2 * w.mrank, w.w_decay2, nullptr, m->decay_buf, ld, ld, 1))) return false;
+    const char *r = rkvg, *k = r + to, *v = k + to, *g = v + to;
+    int n_long = s->num_long;
+    if (n_long > 0) {
+      int rc = -1;
+      if (ksana_time_mix_scratch(s->long_tokens, n_long, w.mh, w.md) <= m->chunk_floats)
+        rc = ksana_time_mix_chunked(r, ld, k, ld, v, ld, m->decay_buf, ld, w.w_decay0, w.bonus, w.state, pitch, s->state_slots,
+                                    s->cu_q, s->kv_lens, w.mh, w.md, m->o_buf, 0, n_long, s->max_q_prefill, m->chunk_buf, st);
+      if (rc == -1) {
+        n_long = 0;  // not a size of the chunked form
+      } else {
+        *launches += 2;
+        if (!step(38, rc)) return false;
+      }
+    }
+    const int base[2] = {n_long, s->num_prefill}, count[2] = {s->num_prefill - n_long, s->num_decode};
+    for (int i = 0; i < 2; ++i)
+      if (count[i] > 0 &&
+          !step(39, ksana_time_mix_recurrent(r, ld, k, ld, v, ld, m->decay_buf, ld, w.w_decay0, w.bonus, w.state, pitch,
+                                             s->state_slots, s->cu_q, s->kv_lens, w.mh, w.md, m->o_buf, base[i], count[i],
+                                             i == 1 && s->one_token, 1, st)))
+        return false;
+    return step(40, ksana_gated_norm(m->o_buf, g, ld, w.mix_norm, out, w.k_out, T, w.mh, w.md, m->eps, 0, w.mix_out_scale, 1,
+                                     1, st));
+  }
+
+  bool gated_layer(const KsanaMixerLayer& w) {
+    const int T = s->total_tokens, H = m->hidden;
+    char *x = static_cast<char*>(m->in_buf), *mix = static_cast<char*>(m->mix_buf);
+    const char* h0 = static_cast<const char*>(h);
+    if (!step(1, gemm(h, H, w.w_in, w.b_in, x, w.n_in, w.n_in))) return false;
+    const int used = w.h * w.dv + w.mh * w.md;
+    if (used < w.k_out &&
+        cudaMemset2DAsync(mix + static_cast<size_t>(used) * 2, static_cast<size_t>(w.k_out) * 2, 0,
+                          static_cast<size_t>(w.k_out - used) * 2, T, st) != cudaSuccess)
+      return step(8, -5);
+    if (!talking(w, x, mix)) return false;
+    if (w.mh > 0 && !time_mix(w, mix + static_cast<size_t>(w.h * w.dv) * 2)) return false;
+    if (!step(9, gemm(mix, w.k_out, w.w_out, w.b_out, m->proj_buf, H, H))) return false;
+    const int attn_in = w.h * w.d + w.hk * (w.d + w.dv) + (w.out_gate ? w.h * w.dv : 0), n = H + w.shared_ff;
+    if (w.experts > 0) {
+      h = h0 + static_cast<size_t>(T) * H * 2;
+      if (!experts(w)) return false;
+      if (!step(41, gemm(h, H, w.w_ff_in, w.b_ff_in, m->gu_buf, n, n))) return false;
+      if (!step(42, ksana_relu2(static_cast<char*>(m->gu_buf) + static_cast<size_t>(H) * 2, n, m->act_buf, T, w.shared_ff, 1, st)))
+        return false;
+      if (!step(43, gemm(m->act_buf, w.shared_ff, w.w_shared_down, nullptr, m->shared_buf, H, H))) return false;
+    }
+    const bool ff = w.experts > 0;
+    void* out = m->h_buf[pp];
+    if (!step(44, ksana_gated_stream_norm(m->proj_buf, H, x + static_cast<size_t>(attn_in) * 2, w.n_in,
+                                          ff ? m->rows_out_buf : nullptr, m->pair_pos, m->expert_weights, w.top,
+                                          ff ? m->shared_buf : nullptr, H, ff ? m->router_buf + w.experts : nullptr,
+                                          w.router_rows, ff ? m->gu_buf : nullptr, n, m->residual_scale, residual, residual,
+                                          w.next_ln, w.next_ln2, out, T, H, m->eps, 1, st)))
+      return false;
+    h = out;
+    pp ^= 1;
+    return true;
+  }
+
   bool layer(const KsanaMixerLayer& w, bool first) {
+    if (w.gated_residual) return gated_layer(w);
     const int T = s->total_tokens, H = m->hidden;
     char* x = static_cast<char*>(m->in_buf);
     char* mix = static_cast<char*>(m->mix_buf);
@@ -433,7 +591,10 @@ struct Exec {
 KSANA_API long long ksana_mixer_latent_bytes(const KsanaMixerModel* m, const KsanaMixerStep* s, int layers) {
   long long most = 0;
   for (int i = 0; i < layers; ++i)
-    if (m->layers[i].ah > 0) {
+    if (m->layers[i].talk) {
+      const long long n = talking_bytes(s, m->layers[i]);
+      if (n > most) most = n;
+    } else if (m->layers[i].ah > 0) {
       const long long n = latent_plan(m, s, m->layers[i]).bytes;
       if (n > most) most = n;
     }

@@ -1,6 +1,6 @@
 // Native forward pass of layers with mixers of their own sizes (windowed attention and / or linear attention, latent
-// attention, a gated recurrence; a norm over a 32-bit residual stream, or over several hyper-connected ones; a dense or
-// routed FFN behind or beside the mixers), driven from ONE call per step. A layer that runs several times is listed once
+// attention, a gated recurrence, weight-mixing attention beside time mixing; a norm over a 32-bit residual stream, or over
+// several hyper-connected ones; a dense or routed FFN behind or beside the mixers), driven from ONE call per step. A layer that runs several times is listed once
 // per run. Mirrored with ctypes on the Python side.
 #pragma once
 #include <cuda_runtime.h>
@@ -73,16 +73,37 @@ struct KsanaMixerLayer {
   const float* hc_mix[2];
   const float* hc_out[2];
   const float* next_in;        // how the next layer (or the final norm) reads the streams
+  // gated residual: mixers and experts side by side, over norms of their own (h_buf: two planes [T, H])
+  int gated_residual, experts_plain, scoring, shared_ff;  // scoring: of the router, 1 sigmoid
+  float router_scale;
+  const void* next_ln2;        // the next layer's second norm (null: it has one)
+  const void* w_ff_in;         // [H + shared_ff, H]: the experts' residual gate, the shared expert's input
+  const void* b_ff_in;
+  const void* w_shared_down;   // [H, shared_ff]
+  // weight-mixing attention
+  int talk, out_gate, qk_norm_all;
+  const float* talk_mix;       // [h, h]
+  const float* talk_sink;      // [h]
+  // time mixing (mh == 0: none)
+  int mh, md, mrank, mpad;     // mpad: rows of one projection (mh * md filled up)
+  float mix_out_scale;
+  const float* mu;             // [5, H]
+  const void* w_mix;           // [4, mpad, H]: r, k, v, gate
+  const void* w_decay1;        // [mrank, H]
+  const void* w_decay2;        // [mpad, 2 mrank]
+  const float* w_decay0;       // [mh * md]
+  const float* bonus;          // [mh * md]
+  const float* mix_norm;       // [mh * md]
 };
 
 struct KsanaMixerModel {
   int hidden, block_size, num_blocks, center;  // center: LayerNorm, else RMS norm
   int streams;                                 // 0: one residual stream
-  float eps;
+  float eps, residual_scale;                   // residual_scale: of gated sublayers
   // scratch for max_tokens rows
   void* in_buf;    // [T, max n_in]
   void* mix_buf;   // [T, max k_out]
-  void* o_buf;     // [T, max lh * ldv]
+  void* o_buf;     // [T, max lh * ldv or mh * md]
   void* gu_buf;    // [T, 2 max I]
   void* act_buf;   // [T, max I]
   void* proj_buf;  // [T, H]
@@ -101,7 +122,14 @@ struct KsanaMixerModel {
   void* rows_out_buf;
   float* chunk_buf;
   long long chunk_floats;
-  void* lat_buf;           // scratch of latent attention
+  // gated layers: [T, H] (shared expert), time mixing's [5][T, H], [4][T, mpad], [T, mrank] fp32, [T, 2 mrank], [T, mpad] fp32
+  void* shared_buf;
+  void* mixes_buf;
+  void* rkvg_buf;
+  float* rank_buf;
+  void* tanh_buf;
+  float* decay_buf;
+  void* lat_buf;           // scratch of latent and of weight-mixing attention
   long long lat_bytes, expand_bytes;  // expand_bytes: keys and values that prompts have written out at a time
   float* gemm_ws;
   long long gemm_ws_floats;

@@ -311,16 +311,22 @@ class _MixerLayer(ctypes.Structure):
         [(n, I) for n in ("ah", "adim", "avdim", "arank")] + [("ascale", F)] + \
         [(n, P) for n in ("anorm", "a_uk_t", "a_uv", "a_expand")] + [(n, I) for n in ("rc", "rk", "rb")] + \
         [(n, P) for n in ("conv_w", "conv_b", "gates", "gates_by_block", "gates_b", "rate")] + \
-        [(n, P * 2) for n in ("ls", "hc_in", "hc_mix", "hc_out")] + [("next_in", P)]
+        [(n, P * 2) for n in ("ls", "hc_in", "hc_mix", "hc_out")] + [("next_in", P)] + \
+        [(n, I) for n in ("gated_residual", "experts_plain", "scoring", "shared_ff")] + [("router_scale", F)] + \
+        [(n, P) for n in ("next_ln2", "w_ff_in", "b_ff_in", "w_shared_down")] + \
+        [(n, I) for n in ("talk", "out_gate", "qk_norm_all")] + [("talk_mix", P), ("talk_sink", P)] + \
+        [(n, I) for n in ("mh", "md", "mrank", "mpad")] + [("mix_out_scale", F)] + \
+        [(n, P) for n in ("mu", "w_mix", "w_decay1", "w_decay2", "w_decay0", "bonus", "mix_norm")]
 
 
 class _MixerModel(ctypes.Structure):
-    _fields_ = [("hidden", I), ("block_size", I), ("num_blocks", I), ("center", I), ("streams", I), ("eps", F), ("in_buf", P),
+    _fields_ = [("hidden", I), ("block_size", I), ("num_blocks", I), ("center", I), ("streams", I), ("eps", F), ("residual_scale", F), ("in_buf", P),
                 ("mix_buf", P), ("o_buf", P), ("gu_buf", P), ("act_buf", P), ("proj_buf", P), ("h_buf", P * 2)] + \
                [(n, P) for n in ("router_buf", "expert_ids", "expert_weights", "pair_pos", "pair_src", "sort_meta",
                                  "rows_buf", "rows_gu_buf", "rows_act_buf", "rows_out_buf")] + \
-               [("chunk_buf", P),
-                ("chunk_floats", LL), ("lat_buf", P), ("lat_bytes", LL), ("expand_bytes", LL), ("gemm_ws", P), ("gemm_ws_floats", LL), ("gemm_counters", P), ("n_counters", I),
+               [("chunk_buf", P), ("chunk_floats", LL)] + \
+               [(n, P) for n in ("shared_buf", "mixes_buf", "rkvg_buf", "rank_buf", "tanh_buf", "decay_buf")] + \
+               [("lat_buf", P), ("lat_bytes", LL), ("expand_bytes", LL), ("gemm_ws", P), ("gemm_ws_floats", LL), ("gemm_counters", P), ("n_counters", I),
                 ("layers", P)]
 
 
@@ -341,10 +347,9 @@ class MixerExecutor:
             return False
         if model.device.type != "cuda" or model.dtype != torch.bfloat16 or not model.layers or model.norm_w is None:
             return False
-        if model.gated_layers:
-            return False
         for layer in model.layers:
-            lins = [layer.in_proj, layer.o_proj] + ([layer.ffn.up, layer.ffn.down] if layer.ffn is not None else [])
+            lins = [x for x in (layer.ff_in, layer.shared_down) if x is not None]
+            lins += [layer.in_proj, layer.o_proj] + ([layer.ffn.up, layer.ffn.down] if layer.ffn is not None else [])
             if any(lin.kind != "dense" or lin.pre is not None or lin.weight.dtype != torch.bfloat16 or
                    not lin.weight.is_contiguous() or lin.weight.shape[0] % 8 or lin.weight.shape[1] % 8 for lin in lins):
                 return False
@@ -353,8 +358,10 @@ class MixerExecutor:
                     f.up.bias is not None or f.down.bias is not None or not f.gated or f.act != "gelu_tanh"):
                 return False
             e = layer.experts
+            if layer.spec.gated_residual and model.cfg.hidden_size % 8:
+                return False
             if e is not None:
-                H, two_i = model.cfg.hidden_size, e.w_gate_up.shape[1]
+                H, two_i = model.cfg.hidden_size, e.w_gate_up.shape[1] * (2 if layer.spec.moe.plain else 1)
                 if e.perm is not None or e._eplb_counts is not None or e.gate_w.dtype != torch.bfloat16 or H % 8 or \
                         two_i % 16 or any(t.dtype != torch.bfloat16 or not t.is_contiguous()
                                           for t in (e.gate_w, e.w_gate_up, e.w_down)) or layer.spec.moe.experts > 2048:
@@ -384,6 +391,7 @@ class MixerExecutor:
                 e, s = layer.experts, layer.spec.moe
                 L.experts, L.top, L.expert_inter = s.experts, s.top, e.w_down.shape[2]
                 L.groups, L.keep_groups, L.limit, L.alpha = s.groups, s.keep, s.limit, s.alpha
+                L.experts_plain, L.scoring, L.router_scale = int(s.plain), int(s.scoring == "sigmoid"), s.scale
                 L.ln2 = _p(layer.ln2)
                 L.router_rows, L.w_router, L.b_router = e.gate_w.shape[0], _p(e.gate_w), _p(e.logit_bias)
                 L.w_expert_gu, L.w_expert_down = _p(e.w_gate_up), _p(e.w_down)
@@ -407,6 +415,19 @@ class MixerExecutor:
                 L.q_norm, L.k_norm = _p(a.q_norm), _p(a.k_norm)
                 L.softcap, L.sink, L.head_gate = s.softcap, int(s.sink), int(s.head_gate)
                 L.reads, L.rot = int(s.kv_from is not None), s.rot.dims if s.rot else 0
+                L.talk, L.out_gate, L.qk_norm_all = int(s.talk), int(s.out_gate), int(s.qk_norm_all)
+                L.talk_mix, L.talk_sink = _p(a.talk), _p(a.sink)
+            L.gated_residual = int(layer.spec.gated_residual)
+            if L.gated_residual:
+                L.next_ln2 = _p(model.layers[i + 1].ln2 if i + 1 < n else None)
+                if layer.ff_in is not None:
+                    L.w_ff_in, L.b_ff_in = _p(layer.ff_in.weight), _p(layer.ff_in.bias)
+                    L.w_shared_down, L.shared_ff = _p(layer.shared_down.weight), layer.shared_down.in_features
+            if layer.timemix is not None:
+                a, s = layer.timemix, layer.timemix.spec
+                L.mh, L.md, L.mpad, L.mrank = s.heads, s.dim, a.proj.shape[1], a.w1.shape[0]
+                L.mix_out_scale, L.mu, L.w_mix = s.out_scale, _p(a.mu), _p(a.proj)
+                L.w_decay1, L.w_decay2, L.w_decay0, L.bonus, L.mix_norm = _p(a.w1), _p(a.w2), _p(a.w0), _p(a.u), _p(a.norm)
             if layer.latent is not None:
                 a, s = layer.latent, layer.latent.spec
                 L.ah, L.adim, L.avdim, L.arank, L.rot, L.ascale = s.heads, s.dim, s.vdim, s.rank, s.rot_dim, s.scale
@@ -425,6 +446,7 @@ class MixerExecutor:
                 L.decay, L.norm_w = _p(a.decay), _p(a.norm)
         m = self._m = _MixerModel()
         m.hidden, m.eps = model.cfg.hidden_size, float(model.cfg.rms_norm_eps)
+        m.residual_scale = float(model.cfg.residual_scale)
         m.center, m.streams = int(model.cfg.norm_type == "layernorm"), model.cfg.streams
         m.expand_bytes = cuda_latent.EXPAND_BYTES
         ws = self._ws = kcuda.workspace(model.device)
@@ -447,12 +469,21 @@ class MixerExecutor:
         cap = (max(T, 1024) + 1023) // 1024 * 1024
         L, H = self._layers, self._m.hidden
         cols = [max(max(f(x) for x in L), 8) for f in (
-            lambda x: x.n_in, lambda x: x.k_out, lambda x: x.lh * x.ldv, lambda x: 0 if x.parallel else 2 * x.inter,
-            lambda x: 0 if x.parallel else x.inter)] + [H] * 3
+            lambda x: x.n_in, lambda x: x.k_out, lambda x: max(x.lh * x.ldv, x.mh * x.md),
+            lambda x: H + x.shared_ff if x.shared_ff else 0 if x.parallel else 2 * x.inter,
+            lambda x: x.shared_ff if x.shared_ff else 0 if x.parallel else x.inter)]
+        planes = 2 if any(x.gated_residual for x in L) else 1
+        cols += [H] + [H * planes] * 2
         dev = self.model.device
         self._bufs = [torch.empty(cap, c, dtype=torch.bfloat16, device=dev) for c in cols]
         m = self._m
         m.in_buf, m.mix_buf, m.o_buf, m.gu_buf, m.act_buf, m.proj_buf, m.h_buf[0], m.h_buf[1] = (_p(b) for b in self._bufs)
+        if planes > 1:
+            pad, rank = (max(f(x) for x in L) for f in (lambda x: x.mpad, lambda x: x.mrank))
+            self._gated = [torch.empty(cap, c, dtype=t, device=dev) for c, t in (
+                (H, torch.bfloat16), (5 * H, torch.bfloat16), (4 * pad, torch.bfloat16), (rank, torch.float32),
+                (2 * rank, torch.bfloat16), (pad, torch.float32))]
+            m.shared_buf, m.mixes_buf, m.rkvg_buf, m.rank_buf, m.tanh_buf, m.decay_buf = (_p(b) for b in self._gated)
         routed = [x for x in L if x.experts]
         if routed:
             top = max(x.top for x in routed)
@@ -511,10 +542,12 @@ class MixerExecutor:
         s.max_kv_decode = int(meta.kv_lens_host[n_pre:].max()) if n_dec else 0
         s.one_token = int(T - s.prefill_tokens == n_dec)
         s.max_q_decode = int((cu[n_pre + 1:] - cu[n_pre:-1]).max()) if n_dec else 0
-        s.num_long = long_portions(meta) if any(x.lh for x in self._layers) else 0
+        s.num_long = long_portions(meta) if any(x.lh or x.mh for x in self._layers) else 0
         s.long_tokens = int(cu[s.num_long])
         if s.num_long:
             self._chunk_floats(max((s.long_tokens // 128 + s.num_long) * x.lh * x.ld * x.ldv for x in self._layers))
+            self._chunk_floats(max(kcuda.lib().ksana_time_mix_scratch(s.long_tokens, s.num_long, x.mh, x.md)
+                                   for x in self._layers))
         if self._rec_width:  # chunks of prompts, or the gates' products where the general kernels run
             self._chunk_floats(max(T * self._rec_width * 5 // 2 + 4, kcuda.lib().ksana_recurrence_scratch(
                 s.prefill_tokens, n_pre, s.max_q_prefill, self._rec_width)))
@@ -530,4 +563,5 @@ class MixerExecutor:
         if rc != 0:
             raise RuntimeError(f"native mixer forward failed at layer {rc // 100 - 1}, step {rc % 100}, "
                                f"code {self._fail.value}")
-        return self._bufs[6 if self._out.value == self._bufs[6].data_ptr() else 7][:T]
+        out = self._bufs[6 if self._out.value == self._bufs[6].data_ptr() else 7]
+        return out.view(-1)[:T * m.hidden].view(T, m.hidden)

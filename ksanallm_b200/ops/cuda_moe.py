@@ -81,7 +81,7 @@ def expert_pipeline(x, ids, w_gate_up, w_down, expert_offset=0, limit=0.0, alpha
     ``reference.clamped_gate_mul``; ``plain``: up -> squared ReLU) -> down on the sorted rows.
     Returns (y [T*k, H] sorted expert outputs, pos [T*k] sorted row of each pair or -1 for non-local experts)."""
     from . import cuda
-    if not supports(x, w_gate_up, w_down):
+    if not supports(x, w_gate_up, w_down, 8 if plain else 16):
         return _pipeline_any(x, ids, w_gate_up, w_down, expert_offset, limit, alpha, plain)
     T, H = x.shape
     k = ids.shape[1]
@@ -120,9 +120,9 @@ def expert_pipeline(x, ids, w_gate_up, w_down, expert_offset=0, limit=0.0, alpha
     return y, pos
 
 
-def supports(x, w_gate_up, w_down) -> bool:
+def supports(x, w_gate_up, w_down, multiple: int = 16) -> bool:
     two_i, H = w_gate_up.shape[1], x.shape[1]
-    return (x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and two_i % 16 == 0 and H % 8 == 0 and
+    return (x.dtype == torch.bfloat16 and w_gate_up.dtype == torch.bfloat16 and two_i % multiple == 0 and H % 8 == 0 and
             w_gate_up.is_contiguous() and w_down.is_contiguous())
 
 

@@ -71,14 +71,13 @@ def talking_attention(q, k, v, scale, sink, talk, first=0):
     """q [n, H, d] at positions first .. first + n - 1, k [N, G, d], v [N, G, dv] at positions 0 .. N - 1. The weights of
     all heads are mixed by talk [to, from] before each head sums up the values of its own key/value head."""
     n, H = q.shape[:2]
-    R = H // k.shape[1]
+    mine = [h // (H // k.shape[1]) for h in range(H)]  # every query head's key/value head
     out = q.new_zeros(n, H, v.shape[2])
     for i in range(n):
         N = first + i + 1
-        p = torch.stack([sink_weights((k[:N, h // R] @ q[i, h]) * scale, sink[h]) for h in range(H)])
-        mixed = talk @ p
-        for h in range(H):
-            out[i, h] = mixed[h] @ v[:N, h // R]
+        scores = torch.einsum("nhd,hd->hn", k[:N, mine], q[i]) * scale
+        p = torch.stack([sink_weights(s, x) for s, x in zip(scores, sink)])
+        out[i] = torch.einsum("hn,nhv->hv", talk @ p, v[:N, mine])
     return out
 
 
@@ -113,7 +112,7 @@ def bonus_recurrence(r, k, v, w, u, s0=None):
         kv = k[t].unsqueeze(2) * v[t].unsqueeze(1)
         out.append(((s + u.unsqueeze(2) * kv) * r[t].unsqueeze(2)).sum(1))
         s = w[t].unsqueeze(2) * s + kv
-    return torch.stack(out), s
+    return torch.stack(out) if out else torch.zeros_like(v), s
 
 
 def time_mixer(h, c, w, p, eps):
@@ -203,7 +202,7 @@ def tensor_shapes(cfg: dict) -> Dict[str, tuple]:
                        x + "q.norm": (H * a["dim"],), x + "k.norm": (G * a["dim"],), x + "talk": (H, H), x + "sink": (H,),
                        x + "g": (H * a["vdim"], W), x + "o": (W, H * a["vdim"])})
         n, x = r["heads"] * r["dim"], p + ".mix.right."
-        rank = layer.get("decay_rank", 12)  # (not part of a config: the tensors' shapes tell)
+        rank = (6, 16, 11, 3)[i % 4]  # (not part of a configuration: the tensors' shapes tell)
         shapes.update({f"{x}mu.{c}": (W,) for c in "rkvgw"})
         shapes.update({x + c: (n, W) for c in "rkvg"})
         shapes.update({x + "w1": (rank, W), x + "w2": (n, rank), x + "w0": (n,), x + "u": (r["heads"], r["dim"]),
