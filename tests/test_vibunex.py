@@ -224,7 +224,7 @@ def test_the_comparison_would_show(cases, mistake, monkeypatch):
     elif mistake == "whose values":  # of the head that the weights come from
         patch("talking_attention", lambda f: lambda q, k, v, scale, sink, talk, first=0: f(q, k, v.flip(1), scale, sink, talk, first))
     elif mistake == "scale":
-        L[0]["left"]["scale"] *= 1.01
+        L[0]["left"]["scale"] *= 1.03
     elif mistake == "rotation":
         patch("rotate_halves", lambda f: lambda x, pos, *a: f(x, [p + 1 if p > 50 else p for p in pos], *a))
     elif mistake == "pairs":
@@ -242,7 +242,7 @@ def test_the_comparison_would_show(cases, mistake, monkeypatch):
     elif mistake == "output gate":
         w["l0.mix.left.g"] = w["l0.mix.left.g"].roll(1, 0)
     elif mistake == "left scale":
-        L[1]["left_scale"] *= 1.01
+        L[1]["left_scale"] *= 1.03
     elif mistake == "right scale":
         L[0]["right_scale"] *= 1.01
     elif mistake == "bonus":

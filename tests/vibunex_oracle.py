@@ -232,7 +232,9 @@ def random_weights(cfg: dict, seed: int = 0) -> Dict[str, torch.Tensor]:
             t = torch.eye(shape[0]) + 0.5 * t
         elif last == "w0":
             t = -3.0 + 1.7 * t
-        elif last in ("sink", "u"):
+        elif last == "sink":
+            t = 2.0 + t
+        elif last == "u":
             pass
         elif last == "b":
             t = 0.5 * t
