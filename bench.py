@@ -15,7 +15,7 @@ distribution are admitted so that exactly K steps are timed. Other named workloa
                       tokens, 128 output tokens, prefix caching on, 128 x 128 block-scaled fp8 weights.
 * ``deepseek-v3-fp8`` 2048 requests, prompts uniform [512, 4096], 512 output tokens, ``--max-batch`` = decode batch.
 
-``--throughput molopel`` (or ``givirax``, ``ladusun``) measures something else: prefill and decode throughput of that design at a few
+``--throughput molopel`` (or ``givirax``, ``ladusun``, ``vibunex``) measures something else: prefill and decode throughput of that design at a few
 layer sizes, beside the closest other model of the same size (benchmarks/layer_throughput.py).
 
 A "step" is one engine step through the public ``LLMEngine.step()``: schedule -> one H2D copy of the step's inputs
@@ -79,7 +79,7 @@ def parse_args():
     ap.add_argument("--kv-fraction", type=float, default=0.0,
                     help="fraction of device memory given to the KV cache (0: everything but a fixed reserve)")
     ap.add_argument("--no-tp1-check", action="store_true", help="skip the comparison of TP=N tokens with TP=1")
-    ap.add_argument("--throughput", default="", choices=["", "molopel", "givirax", "ladusun"],
+    ap.add_argument("--throughput", default="", choices=["", "molopel", "givirax", "ladusun", "vibunex"],
                     help="prefill and decode throughput of a model design at several layer sizes beside the closest "
                          "other model of equal size (one GPU; replaces the serving workload)")
     return ap.parse_args()

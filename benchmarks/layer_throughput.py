@@ -5,12 +5,16 @@ closest other model of the same width, heads and depth. Random weights, bf16, on
     python bench.py --throughput molopel
     python bench.py --throughput givirax
     python bench.py --throughput ladusun
+    python bench.py --throughput vibunex
 
 Molopel: beside the dense model (Qwen3 blocks: QK norm, grouped-query attention, SwiGLU) whose feed-forward is as wide as
 makes the parameter counts equal. Givirax (half of its layers run twice): beside Qwen3-MoE blocks, dense and routed in
 turn, as many layers as Givirax has runs, with the same experts and a gated feed-forward of the same number of weights.
 Ladusun (four residual streams): beside DeepSeek blocks (latent attention, routed experts) of the same width, depth, heads
 and latent size, dense and routed in turn, with the same experts and a gated feed-forward of the same number of weights.
+Vibunex: beside two models, each closest in one respect: Qwen2-MoE blocks (grouped-query attention, routed and shared
+experts) with the same experts and the same number of feed-forward weights, and Molopel blocks (attention to all keys beside
+retention with as many channels) with a dense feed-forward of as many weights as a Vibunex token meets.
 
 prefill: prompts of 4096 tokens, 8192 tokens a step. decode: 128 sequences behind prompts of 1024 tokens, one token each
 per step. Weights and caches are larger than L2, so each step starts cold. CUDA events around the timed steps; the host
@@ -23,7 +27,8 @@ import time
 
 import torch
 
-from ksanallm_b200.config.model_config import givirax_config, ladusun_config, model_config_from_dict, molopel_config
+from ksanallm_b200.config.model_config import (givirax_config, ladusun_config, model_config_from_dict, molopel_config,
+                                               vibunex_config)
 from ksanallm_b200.config.schema import parse_serving_config
 from ksanallm_b200.engine.llm_engine import LLMEngine
 from ksanallm_b200.engine.sampling_params import SamplingParams
@@ -39,6 +44,9 @@ GIVIRAX_SIZES = [(2048, 8, 8192, 16, 2, 2048, 16, 4, 1024), (4096, 8, 16384, 16,
 # width, depth, feed-forward, experts, experts per token, expert width, heads, key / value heads, latent size
 LADUSUN_SIZES = [(2048, 8, 8192, 16, 2, 2048, 16, 4, 512), (4096, 8, 16384, 16, 2, 4096, 32, 8, 512),
                  (8192, 4, 32768, 8, 2, 8192, 64, 8, 512)]
+# width, depth, experts, experts per token, expert width, shared expert's width, heads, key / value heads, time-mixing heads of 64
+VIBUNEX_SIZES = [(2048, 8, 16, 2, 2048, 2048, 16, 4, 32), (4096, 8, 16, 2, 4096, 4096, 32, 8, 64),
+                 (8192, 4, 8, 2, 8192, 8192, 64, 8, 128)]
 PROMPT, STEP_TOKENS = 4096, 8192
 BATCH, CONTEXT, DECODE_STEPS = 128, 1024, 40
 
@@ -61,6 +69,25 @@ def moe_config(width, depth, ff, experts, top, expert_ff, heads, kv_heads):
         num_experts=experts, num_experts_per_tok=top, norm_topk_prob=True, rms_norm_eps=1e-6, vocab_size=32000,
         mlp_layer_types=["sparse" if i % 2 else "dense" for i in range(depth)],
         max_position_embeddings=8192, torch_dtype="bfloat16", eos_token_id=2))
+
+
+def shared_moe_config(width, depth, experts, top, expert_ff, shared_ff, heads, kv_heads):
+    return model_config_from_dict(dict(
+        model_type="qwen2_moe", hidden_size=width, num_hidden_layers=depth, num_attention_heads=heads,
+        num_key_value_heads=kv_heads, head_dim=128, intermediate_size=shared_ff, moe_intermediate_size=expert_ff,
+        shared_expert_intermediate_size=shared_ff, num_experts=experts, num_experts_per_tok=top, norm_topk_prob=False,
+        rms_norm_eps=1e-6, vocab_size=32000, decoder_sparse_step=1, max_position_embeddings=8192, torch_dtype="bfloat16",
+        eos_token_id=2))
+
+
+def retention_config(width, depth, ff, heads, kv_heads, channels):
+    """Molopel whose layers all have attention to every key beside retention over ``channels``."""
+    cfg = molopel_config(width, 1, ff, heads, kv_heads, 128, 8192)
+    raw = json.loads(json.dumps(cfg.raw))
+    layer = raw["layers"][0]
+    layer["mixer"]["right"].update(heads=channels // 64, dim=64, vdim=64, decay=[0.99] * (channels // 64), rot=dict(dims=64, base=10000.0))
+    raw["layers"] = [layer] * depth
+    return model_config_from_dict(raw)
 
 
 def mla_config(width, depth, ff, experts, top, expert_ff, heads, rank):
@@ -177,7 +204,26 @@ def run_ladusun() -> None:
                               data="synthetic", **rows)), flush=True)
 
 
+def run_vibunex() -> None:
+    for width, depth, experts, top, expert_ff, shared_ff, heads, kv, mix in VIBUNEX_SIZES:
+        rows = {}
+        third = lambda n: n * 2 // 3 // 128 * 128  # noqa: E731  (a gated feed-forward has three matrices)
+        for name, cfg in (
+                ("vibunex", vibunex_config(width, depth, experts, top, expert_ff, shared_ff, heads, kv, 128, mix, 64)),
+                ("shared_moe", shared_moe_config(width, depth, experts, top, third(expert_ff), third(shared_ff), heads, kv)),
+                ("molopel", retention_config(width, depth, third(top * expert_ff + shared_ff), heads, kv, mix * 64))):
+            model, n = build(cfg)
+            rows[name] = dict(parameters_m=round(n / 1e6), **measure(model))
+            del model
+            torch.cuda.empty_cache()
+        print(json.dumps(dict(metric="throughput", design="vibunex", width=width, layers=depth, experts=experts, top=top,
+                              expert_ff=expert_ff, shared_ff=shared_ff, heads=heads, kv_heads=kv, mix_heads=mix, dtype="bf16",
+                              data="synthetic", **rows)), flush=True)
+
+
 def run(design: str) -> None:
+    if design == "vibunex":
+        return run_vibunex()
     if design == "givirax":
         return run_givirax()
     if design == "ladusun":
