@@ -1,8 +1,11 @@
 // Weight-mixing attention (see talking_attention.cu) over prompts on the tensor cores, bf16. A head's output needs all heads'
 // normalised weights, so the work goes in three launches per round of 128-row query blocks:
 //   statistics   the logarithm of every (query, head)'s softmax denominator, sink included
-//   weights      scores again, weights of all heads, their mix -> W[block][hi | lo][head][row][key] as two bf16 matrices
+//   weights      scores again, weights of all heads, their mix -> W[block][hi | lo][head] as two bf16 matrices
 //   values       O = (W_hi + W_lo) V per (block, head), times the output gate
+// The weights' kernel comes in two forms. For 16, 32 or 64 heads in groups of 2, 4 or 8 both of its products run on tcgen05,
+// and a matrix of W is [16][key][8 rows], which is the layout of an MMA operand without swizzle; for other sizes they run on
+// mma.sync, and it is [row][key].
 // Rounds keep W within a budget; keys beyond a query's position have zero weights in it.
 #include "talking.cuh"
 
@@ -168,7 +171,276 @@ talking_stats_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   }
 }
 
-// ---- weights -----------------------------------------------------------------------------------------------------------
+// ---- weights, tcgen05 ----------------------------------------------------------------------------------------------------
+// One CTA = (QN query rows of a block, all HP heads, a range of keys), 128 keys at a time; QN x HP = 256. Keys are the MMA
+// rows, so that a thread owns one key, all heads of half of the queries of which are in its registers:
+//   S = K_c Q_c^T          per key / value head c: 128 keys x (QN queries x R heads of the group)
+//   P = exp(S - lse)       written back to TMEM as two bf16 matrices hi + lo, [query][head]
+//   D_i = P_i talk^T       per query i, A = P_i from TMEM
+//   W                      D as hi + lo, eight queries of a head side by side
+// Two regions of 256 columns change places from tile to tile: S and then D of a tile are in one, its P in the other. Q K^T of
+// the next tile runs while this one's D is written out. Warps 0-3 and 4-7 cover the 128 lanes once each; warp 8 loads, warp 9
+// issues the MMAs.
+template <int DP, int HP>
+struct TalkWeightsTcSmem {
+  static constexpr int QN = 256 / HP, STAGES = 4;
+  static constexpr int TILE = 128 * DP * 2;           // 128 keys of one head
+  static constexpr int OFF_Q = STAGES * TILE;
+  static constexpr int Q_BYTES = 256 * DP * 2;
+  static constexpr int OFF_T = OFF_Q + Q_BYTES;       // the mix, K-major
+  static constexpr int OFF_LSE = OFF_T + HP * 128;
+  static constexpr int OFF_BAR = OFF_LSE + 256 * 4;
+  static constexpr int USED = OFF_BAR + 128 + 1024;
+  // at least half of the SM's shared memory: two CTAs would compete for the 512 TMEM columns each of them takes
+  static constexpr int TOTAL = USED > 120 * 1024 ? USED : 120 * 1024;
+};
+
+template <int DP, int HP, int R>
+__global__ void __launch_bounds__(320, 1)
+talking_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_constant__ CUtensorMap tmK, TalkArgs a,
+                          TalkRound rd, int keys_per, unsigned int* err) {
+  using L_ = TalkWeightsTcSmem<DP, HP>;
+  constexpr int QN = L_::QN, STAGES = L_::STAGES, G = HP / R, N = QN * R;
+  constexpr int QP = 64 / HP;                        // queries whose scores a thread has at a time
+  constexpr int WP = QP * R < 8 ? QP * R : 8;        // columns per load of them
+  constexpr int DW = QN == 16 ? 4 : 8;               // heads of D at a time
+  static_assert(N % 16 == 0 && (WP == 4 || WP == 8), "");
+  const int unit = gridDim.x - 1 - blockIdx.x;  // blocks further along a prompt are longer: they go first
+  int b, qb;
+  if (!find_unit(a, rd.num_seqs, rd.unit0 + unit, &b, &qb)) return;
+  const int q_len = a.cu_q[b + 1] - a.cu_q[b], L = a.kv_lens[b];
+  const int row0 = qb * 128 + blockIdx.y * QN;  // first query row, within the sequence's new tokens
+  if (row0 >= q_len) return;
+  const int pos0 = L - q_len + row0, t0 = a.cu_q[b] + row0;
+  const int filled = (min(L, L - q_len + qb * 128 + 128) + 127) / 128 * 128;  // what the values' kernel reads
+  const int key0 = blockIdx.z * keys_per, key1 = min(key0 + keys_per, filled);
+  if (key0 >= key1) return;
+  const int tiles = (key1 - key0) / 128;
+  const int live = max(0, min(tiles, (min(pos0 + QN, L) - key0 + 127) / 128));  // tiles with a visible key
+  extern __shared__ uint8_t smem_raw[];
+  uint8_t* smem = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(smem_raw) + 1023) & ~uintptr_t(1023));
+  uint8_t *sQ = smem + L_::OFF_Q, *sT = smem + L_::OFF_T;
+  float* sLse = reinterpret_cast<float*>(smem + L_::OFF_LSE);  // [QN][HP]
+  uint64_t* q_bar = reinterpret_cast<uint64_t*>(smem + L_::OFF_BAR);
+  uint64_t* k_full = q_bar + 1;           // [STAGES]
+  uint64_t* k_free = k_full + STAGES;     // [STAGES]
+  uint64_t* s_done = k_free + STAGES;
+  uint64_t* p_ready = s_done + 1;
+  uint64_t* d_done = p_ready + 1;
+  uint32_t* holder = reinterpret_cast<uint32_t*>(d_done + 1);
+  volatile int* abort_flag = reinterpret_cast<volatile int*>(holder + 1);
+  const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
+  if (tid == 0) {
+    mbar_init(q_bar, 1);
+    for (int s = 0; s < STAGES; ++s) {
+      mbar_init(&k_full[s], 1);
+      mbar_init(&k_free[s], 1);
+    }
+    mbar_init(s_done, 1);
+    mbar_init(p_ready, 256);
+    mbar_init(d_done, 1);
+    *abort_flag = 0;
+    fence_mbar_init();
+  }
+  if (warp == 0) {
+    tmem_alloc(holder, 512);
+    tmem_relinquish();
+  }
+  for (int i = tid; i < HP * 8; i += 320) {  // talk[to][from .. from + 7], rows of 128 bytes in the 128-byte swizzle
+    const int to = i >> 3, ch = i & 7;
+    uint32_t v[4];
+#pragma unroll
+    for (int u = 0; u < 4; ++u) {
+      const int from = ch * 8 + u * 2;
+      v[u] = from < HP ? pack_bf16(a.talk[to * HP + from], a.talk[to * HP + from + 1]) : 0u;
+    }
+    *reinterpret_cast<uint4*>(sT + (to >> 3) * 1024 + (to & 7) * 128 + ((ch ^ (to & 7)) << 4)) = make_uint4(v[0], v[1], v[2], v[3]);
+  }
+  for (int i = tid; i < 256; i += 320)
+    sLse[i] = row0 + i / HP < q_len ? rd.lse[static_cast<size_t>(t0 + i / HP) * HP + i % HP] : 0.f;
+  fence_async_smem();
+  tc_fence_before();
+  __syncthreads();
+  tc_fence_after();
+  const uint32_t tmem = *holder;
+  if (warp == 8) {
+    if (lane == 0 && live > 0) {
+      const int* bt = a.block_tables + static_cast<size_t>(b) * a.max_blocks;
+      const int n_pages = (L + TALK_PAGE - 1) / TALK_PAGE;
+      mbar_expect_tx(q_bar, L_::Q_BYTES);
+      for (int c = 0; c < G; ++c)
+        for (int hf = 0; hf < DP / 64; ++hf)
+          tma_load_3d(sQ + (c * (DP / 64) + hf) * (N * 128), &tmQ, q_bar, hf * 64, c * R, t0);
+      bool ok = true;
+      int n = 0;
+      for (int t = 0; ok && t < live; ++t)
+        for (int c = 0; c < G; ++c, ++n) {
+          const int st = n % STAGES;
+          if (n >= STAGES) ok = mbar_wait_bounded(&k_free[st], (n / STAGES - 1) & 1, abort_flag, err);
+          if (!ok) break;
+          mbar_expect_tx(&k_full[st], L_::TILE);
+          for (int p = 0; p < 128 / TALK_PAGE; ++p) {
+            const int blk = bt[min((key0 + t * 128) / TALK_PAGE + p, n_pages - 1)];  // (past the end: masked keys)
+            for (int hf = 0; hf < DP / 64; ++hf)
+              tma_load_3d(smem + st * L_::TILE + hf * (128 * 128) + p * (TALK_PAGE * 128), &tmK, &k_full[st], hf * 64,
+                          c * TALK_PAGE, blk);
+          }
+        }
+      if (!ok) {  // copies in flight still write to this CTA's memory: give them their (bounded) time before leaving
+        for (int it = 0; it < (1 << 20) && !mbar_try_wait(q_bar, 0); ++it) {}
+        for (int i = max(n - STAGES, 0); i < n; ++i)
+          for (int it = 0; it < (1 << 20) && !mbar_try_wait(&k_full[i % STAGES], (i / STAGES) & 1); ++it) {}
+      }
+    }
+    __syncwarp();
+  } else if (warp == 9) {
+    if (lane == 0 && live > 0) {
+      bool ok = mbar_wait_bounded(q_bar, 0, abort_flag, err);
+      int n = 0;
+      for (int t = 0; ok && t < live; ++t) {
+        const uint32_t own = tmem + (t & 1) * 256, other = tmem + 256 - (t & 1) * 256;
+        for (int c = 0; c < G; ++c, ++n) {
+          const int st = n % STAGES;
+          ok = mbar_wait_bounded(&k_full[st], (n / STAGES) & 1, abort_flag, err);
+          if (!ok) break;
+          tc_fence_after();
+          constexpr uint32_t idesc = umma_idesc(128, N, 1, 1);
+          const uint32_t kb = smem_u32(smem + st * L_::TILE), qa = smem_u32(sQ + c * (DP / 64) * (N * 128));
+#pragma unroll
+          for (int k = 0; k < DP / 16; ++k)
+            umma_f16(own + c * N, umma_desc_k128(kb + (k >> 2) * (128 * 128) + (k & 3) * 32),
+                     umma_desc_k128(qa + (k >> 2) * (N * 128) + (k & 3) * 32), idesc, k > 0 ? 1u : 0u);
+          umma_commit(&k_free[st]);
+        }
+        if (!ok) break;
+        umma_commit(s_done);
+        ok = mbar_wait_bounded(p_ready, t & 1, abort_flag, err);
+        if (!ok) break;
+        tc_fence_after();
+        constexpr uint32_t idesc = umma_idesc(128, HP, 1, 1);
+        const uint32_t tb = smem_u32(sT);
+#pragma unroll 2
+        for (int i = 0; i < QN; ++i)
+#pragma unroll
+          for (int k = 0; k < HP / 8; ++k)  // hi, then lo
+            umma_f16_ts(own + i * HP, other + i * HP + k * 8, umma_desc_k128(tb + (k % (HP / 16)) * 32), idesc, k > 0 ? 1u : 0u);
+        umma_commit(d_done);
+        ok = mbar_wait_bounded(d_done, t & 1, abort_flag, err);  // (the next scores go over this tile's weights)
+      }
+    }
+    __syncwarp();
+  } else {
+    const int wg = warp >> 2, j = (warp & 3) * 32 + lane;
+    const uint32_t lane_off = static_cast<uint32_t>((warp & 3) * 32) << 16;
+    const float scale2 = a.scale * LOG2E;
+    const size_t step = static_cast<size_t>(16) * rd.pitch * 8, plane = step * HP;
+    __nv_bfloat16* wout = rd.w + unit * 2 * plane + static_cast<size_t>(blockIdx.y * QN / 8) * rd.pitch * 8 + blockIdx.y * QN % 8 +
+                          (wg * (HP / 2)) * step + static_cast<size_t>(key0 + j) * 8;
+    bool ok = true;
+    for (int t = 0; t < live; ++t) {
+      const uint32_t own = tmem + (t & 1) * 256 + lane_off, other = tmem + 256 - (t & 1) * 256 + lane_off;
+      if (ok) ok = mbar_wait_bounded(s_done, t & 1, abort_flag, err);
+      ok = __all_sync(0xffffffffu, ok);
+      tc_fence_before();
+      asm volatile("bar.sync 1, 256;" ::: "memory");  // everybody has read the last tile's D, which P goes over
+      if (ok) {
+        tc_fence_after();
+        const int past = pos0 + wg * (QN / 2) - (key0 + t * 128 + j);  // queries up to -past - 1 do not see this key
+        const bool edge = __any_sync(0xffffffffu, past < 0);
+#pragma unroll 1
+        for (int i0 = 0; i0 < QN / 2; i0 += QP) {
+          float s[64];  // [key / value head][query of this pass][head of the group]
+          const uint32_t src = own + (wg * (QN / 2) + i0) * R;
+#pragma unroll
+          for (int f = 0; f < 64; f += WP) {
+            if constexpr (WP == 4)
+              tmem_ld4(src + (f / (QP * R)) * N + f % (QP * R), reinterpret_cast<uint32_t*>(s) + f);
+            else
+              tmem_ld8(src + (f / (QP * R)) * N + f % (QP * R), reinterpret_cast<uint32_t*>(s) + f);
+          }
+          tmem_wait_ld();
+#pragma unroll
+          for (int i = 0; i < QP; ++i) {
+            const float* lse = sLse + (wg * (QN / 2) + i0 + i) * HP;
+            uint32_t p[HP];  // hi, then lo
+#pragma unroll
+            for (int g = 0; g < HP; g += 2) {
+              const int f = (g / R) * (QP * R) + i * R + g % R;
+              const float2 l = *reinterpret_cast<const float2*>(lse + g);
+              float x = ex2_ftz(fmaf(s[f], scale2, -l.x)), y = ex2_ftz(fmaf(s[f + 1], scale2, -l.y));
+              if (edge && i0 + i + past < 0) x = y = 0.f;
+              p[g / 2] = split_bf16(x, y, &p[HP / 2 + g / 2]);
+            }
+            const uint32_t dst = other + (wg * (QN / 2) + i0 + i) * HP;
+            if constexpr (HP == 16) {
+              tmem_st16(dst, p);
+            } else {
+#pragma unroll
+              for (int c = 0; c < HP; c += 32) tmem_st32(dst + c, p + c);
+            }
+          }
+        }
+        tmem_wait_st();
+        tc_fence_before();
+        mbar_arrive(p_ready);
+        ok = mbar_wait_bounded(d_done, t & 1, abort_flag, err);
+      }
+      ok = __all_sync(0xffffffffu, ok);
+      if (!ok) continue;  // keep meeting the other warps at the barrier
+      tc_fence_after();
+#pragma unroll 1
+      for (int g = 0; g < HP / 2; g += DW) {
+        float d[QN][DW];
+#pragma unroll
+        for (int i = 0; i < QN; ++i) {
+          if constexpr (DW == 4)
+            tmem_ld4(own + i * HP + wg * (HP / 2) + g, reinterpret_cast<uint32_t*>(d[i]));
+          else
+            tmem_ld8(own + i * HP + wg * (HP / 2) + g, reinterpret_cast<uint32_t*>(d[i]));
+        }
+        tmem_wait_ld();
+        __nv_bfloat16* dst = wout + g * step + static_cast<size_t>(t) * (128 * 8);
+#pragma unroll
+        for (int x = 0; x < DW; ++x) {
+          uint32_t hi[QN / 2], lo[QN / 2];
+#pragma unroll
+          for (int i = 0; i < QN; i += 2) hi[i / 2] = split_bf16(d[i][x], d[i + 1][x], &lo[i / 2]);
+          if constexpr (QN == 4) {
+            *reinterpret_cast<uint2*>(dst + x * step) = make_uint2(hi[0], hi[1]);
+            *reinterpret_cast<uint2*>(dst + x * step + plane) = make_uint2(lo[0], lo[1]);
+          } else {
+#pragma unroll
+            for (int q = 0; q < QN / 8; ++q) {
+              const size_t at = x * step + static_cast<size_t>(q) * rd.pitch * 8;
+              *reinterpret_cast<uint4*>(dst + at) = make_uint4(hi[q * 4], hi[q * 4 + 1], hi[q * 4 + 2], hi[q * 4 + 3]);
+              *reinterpret_cast<uint4*>(dst + at + plane) = make_uint4(lo[q * 4], lo[q * 4 + 1], lo[q * 4 + 2], lo[q * 4 + 3]);
+            }
+          }
+        }
+      }
+    }
+    for (int t = live; t < tiles; ++t)
+      for (int g = 0; g < HP / 2; ++g)
+        for (int part = 0; part < 2; ++part) {
+          __nv_bfloat16* dst = wout + g * step + part * plane + static_cast<size_t>(t) * (128 * 8);
+          if constexpr (QN == 4) {
+            *reinterpret_cast<uint2*>(dst) = make_uint2(0, 0);
+          } else {
+#pragma unroll
+            for (int q = 0; q < QN / 8; ++q)
+              *reinterpret_cast<uint4*>(dst + static_cast<size_t>(q) * rd.pitch * 8) = make_uint4(0, 0, 0, 0);
+          }
+        }
+  }
+  tc_fence_before();
+  __syncthreads();
+  if (warp == 0) {
+    tc_fence_after();
+    tmem_dealloc(tmem, 512);
+  }
+}
+
+// ---- weights, other sizes --------------------------------------------------------------------------------------------------
 // One CTA of 8 warps = (QN query rows of a block, all heads, a range of keys), 32 keys at a time, QN x (heads filled up to
 // HP = 16 HK) = 512 rows. Scores: the rows of one key / value head are cut into units of 16 (queries x heads of the group);
 // a warp keeps the queries of up to four units in registers and streams those heads' keys through a ring of its own with
@@ -406,7 +678,8 @@ talking_weights_kernel(const __grid_constant__ CUtensorMap tmK, TalkArgs a, Talk
 
 // ---- values ------------------------------------------------------------------------------------------------------------
 // One CTA = (block of 128 query rows, head): warp 4 loads tiles of 128 keys (both parts of W, the values' pages), warp 5
-// issues the MMAs, warps 0-3 write the result out.
+// issues the MMAs, warps 0-3 write the result out. BLOCKED: the layout of W that the tcgen05 form of the weights' kernel
+// leaves.
 template <int DVP>
 struct TalkValuesSmem {
   static constexpr int W_BYTES = 128 * 128 * 2;  // one part
@@ -415,7 +688,18 @@ struct TalkValuesSmem {
   static constexpr int TOTAL = OFF_BAR + 128 + 1024;
 };
 
-template <int DVP>
+// MN-major operand without swizzle: 8 elements along MN are 16 bytes, 8 K-rows of them 128 bytes; the next 8 K-rows lie lbo
+// bytes on, the next 8 elements along MN sbo bytes.
+__device__ __forceinline__ uint64_t umma_desc_mn_plain(uint32_t smem_addr, uint32_t lbo_bytes, uint32_t sbo_bytes) {
+  uint64_t d = 0;
+  d |= static_cast<uint64_t>((smem_addr >> 4) & 0x3FFF);
+  d |= static_cast<uint64_t>((lbo_bytes >> 4) & 0x3FFF) << 16;
+  d |= static_cast<uint64_t>((sbo_bytes >> 4) & 0x3FFF) << 32;
+  d |= static_cast<uint64_t>(1) << 46;
+  return d;
+}
+
+template <int DVP, bool BLOCKED>
 __global__ void __launch_bounds__(192)
 talking_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_constant__ CUtensorMap tmV, TalkArgs a,
                       TalkRound rd, unsigned int* err) {
@@ -464,7 +748,13 @@ talking_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
         uint8_t* dst = smem + (i & 1) * L_::STAGE;
         uint64_t* bar = &full[i & 1];
         mbar_expect_tx(bar, L_::STAGE);
-        for (int hf = 0; hf < 2; ++hf) {
+        if constexpr (BLOCKED) {
+          for (int part = 0; part < 2; ++part)
+            for (int c = 0; c < 16; ++c)
+              bulk_load(dst + part * L_::W_BYTES + c * 2048,
+                        rd.w + (static_cast<size_t>(part ? row_lo : row_hi) / 8 + c) * rd.pitch * 8 + i * (128 * 8), 2048, bar);
+        }
+        for (int hf = 0; hf < (BLOCKED ? 0 : 2); ++hf) {
           tma_load_2d(dst + hf * (128 * 128), &tmW, bar, i * 128 + hf * 64, row_hi);
           tma_load_2d(dst + L_::W_BYTES + hf * (128 * 128), &tmW, bar, i * 128 + hf * 64, row_lo);
         }
@@ -488,12 +778,14 @@ talking_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
         ok = mbar_wait_bounded(&full[i & 1], (i >> 1) & 1, abort_flag, err);
         if (!ok) break;
         tc_fence_after();
-        constexpr uint32_t idesc = umma_idesc_major(128, DVP, false, true);
+        constexpr uint32_t idesc = umma_idesc_major(128, DVP, BLOCKED, true);
         const uint32_t wb = smem_u32(smem + (i & 1) * L_::STAGE), vb = wb + 2 * L_::W_BYTES;
 #pragma unroll
         for (int k = 0; k < 16; ++k) {  // hi, then lo
-          const uint32_t off = (k >> 3) * L_::W_BYTES + ((k >> 2) & 1) * (128 * 128) + (k & 3) * 32;
-          umma_f16(tmem, umma_desc_k128(wb + off), umma_desc_mn128(vb + (k & 7) * (16 * 128), 128 * 128), idesc,
+          const uint32_t part = wb + (k >> 3) * L_::W_BYTES;
+          const uint64_t aw = BLOCKED ? umma_desc_mn_plain(part + (k & 7) * 256, 128, 2048)
+                                      : umma_desc_k128(part + ((k >> 2) & 1) * (128 * 128) + (k & 3) * 32);
+          umma_f16(tmem, aw, umma_desc_mn128(vb + (k & 7) * (16 * 128), 128 * 128), idesc,
                    i > 0 || k > 0 ? 1u : 0u);
         }
         umma_commit(&freed[i & 1]);
@@ -580,13 +872,52 @@ static int launch_weights(const TalkArgs& a, const CUtensorMap& tk, const TalkRo
   kern<<<dim3(units, subs, (rd.pitch + keys_per - 1) / keys_per), 256, L_::TOTAL, st>>>(tk, a, rd, keys_per, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
 }
-template <int DVP>
+template <int DP, int HP, int R>
+static int launch_weights_tc(const TalkArgs& a, int total_tokens, const CUtensorMap& tk, const TalkRound& rd, int units,
+                             cudaStream_t st) {
+  using L_ = TalkWeightsTcSmem<DP, HP>;
+  static_assert(L_::TOTAL <= 232448, "does not fit");
+  CUtensorMap tq;
+  const uint64_t dims[3] = {static_cast<uint64_t>(a.d), static_cast<uint64_t>(a.h), static_cast<uint64_t>(total_tokens)};
+  const uint64_t str[2] = {static_cast<uint64_t>(a.d) * 2, static_cast<uint64_t>(a.ldq) * 2};
+  const uint32_t box[3] = {64, R, L_::QN};
+  if (make_tmap_nd(&tq, a.q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, dims, str, box, CU_TENSOR_MAP_SWIZZLE_128B)) return -2;
+  auto kern = talking_weights_tc_kernel<DP, HP, R>;
+  if (KSANA_SMEM_ONCE(kern, L_::TOTAL) != 0) return -4;
+  const int subs = 128 / L_::QN;
+  // key ranges: several waves of CTAs, none of them shorter than 512 keys
+  int parts = 1;
+  while (static_cast<long long>(units) * subs * parts < 6ll * sm_count() && rd.pitch / (parts + 1) >= 512) ++parts;
+  const int keys_per = ((rd.pitch + parts - 1) / parts + 127) / 128 * 128;
+  kern<<<dim3(units, subs, (rd.pitch + keys_per - 1) / keys_per), 320, L_::TOTAL, st>>>(tq, tk, a, rd, keys_per, error_word());
+  return cudaGetLastError() == cudaSuccess ? 0 : -5;
+}
+// -1: not a size of the tcgen05 form
+static int weights_tc(const TalkArgs& a, int total_tokens, const CUtensorMap& tk, const TalkRound& rd, int units,
+                      cudaStream_t st) {
+  const int r = a.h / a.hk;
+#define KSANA_TWT(HP, R)                                                                                 \
+  if (a.h == HP && r == R)                                                                               \
+    return a.d <= 64 ? launch_weights_tc<64, HP, R>(a, total_tokens, tk, rd, units, st)                  \
+                     : launch_weights_tc<128, HP, R>(a, total_tokens, tk, rd, units, st)
+  KSANA_TWT(16, 2);
+  KSANA_TWT(16, 4);
+  KSANA_TWT(16, 8);
+  KSANA_TWT(32, 2);
+  KSANA_TWT(32, 4);
+  KSANA_TWT(32, 8);
+  KSANA_TWT(64, 4);
+  KSANA_TWT(64, 8);
+#undef KSANA_TWT
+  return -1;
+}
+template <int DVP, bool BLOCKED>
 static int launch_values(const TalkArgs& a, const CUtensorMap& tv, const TalkRound& rd, int units, cudaStream_t st) {
-  CUtensorMap tw;
+  CUtensorMap tw = tv;
   const uint64_t rows = static_cast<uint64_t>(units) * 2 * a.h * 128;
-  if (make_tmap_2d(&tw, rd.w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, rd.pitch, rd.pitch, 128, 64, CU_TENSOR_MAP_SWIZZLE_128B))
+  if (!BLOCKED && make_tmap_2d(&tw, rd.w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, rd.pitch, rd.pitch, 128, 64, CU_TENSOR_MAP_SWIZZLE_128B))
     return -2;
-  auto kern = talking_values_kernel<DVP>;
+  auto kern = talking_values_kernel<DVP, BLOCKED>;
   if (KSANA_SMEM_ONCE(kern, TalkValuesSmem<DVP>::TOTAL) != 0) return -4;
   kern<<<dim3(a.h, units), 192, TalkValuesSmem<DVP>::TOTAL, st>>>(tw, tv, a, rd, error_word());
   return cudaGetLastError() == cudaSuccess ? 0 : -5;
@@ -647,14 +978,20 @@ KSANA_API int ksana_talking_prefill(const void* q, int ldq, int total_tokens, co
   for (int b = 0, block = 0; rd.unit0 < all;) {
     const TalkPlan p = talk_plan(h, num_seqs, cu_q_host, kv_lens_host, &b, &block);
     rd.pitch = p.pitch;
-    int rc;
+    int rc = weights_tc(a, total_tokens, tk, rd, p.units, st);
+    const bool blocked = rc != -1;
 #define KSANA_TW(DP) \
   rc = h <= 16 ? launch_weights<DP, 1>(a, tk, rd, p.units, st) \
        : h <= 32 ? launch_weights<DP, 2>(a, tk, rd, p.units, st) : launch_weights<DP, 4>(a, tk, rd, p.units, st)
-    if (d <= 64) KSANA_TW(64); else KSANA_TW(128);
+    if (!blocked) {
+      if (d <= 64) KSANA_TW(64); else KSANA_TW(128);
+    }
 #undef KSANA_TW
     if (rc) return rc;
-    rc = dv <= 64 ? launch_values<64>(a, tv, rd, p.units, st) : launch_values<128>(a, tv, rd, p.units, st);
+    if (blocked)
+      rc = dv <= 64 ? launch_values<64, true>(a, tv, rd, p.units, st) : launch_values<128, true>(a, tv, rd, p.units, st);
+    else
+      rc = dv <= 64 ? launch_values<64, false>(a, tv, rd, p.units, st) : launch_values<128, false>(a, tv, rd, p.units, st);
     if (rc) return rc;
     *launches += 2;
     rd.unit0 += p.units;
