@@ -88,18 +88,23 @@ talking_stats_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_const
   const int* bt = a.block_tables + static_cast<size_t>(b) * a.max_blocks;
   if (warp == 4) {
     if ((tid & 31) == 0) {
-      int loads = 0;
+      int loads = 0, blk[128 / TALK_PAGE];
+      auto pages = [&](int i) {  // of a tile, ahead of its turn
+#pragma unroll
+        for (int p = 0; p < 128 / TALK_PAGE; ++p) blk[p] = bt[min(i * (128 / TALK_PAGE) + p, n_pages - 1)];  // (past the end: masked)
+      };
       auto load_k = [&](int i) {
         uint64_t* bar = &k_full[i & 1];
         mbar_expect_tx(bar, L_::TILE);
-        for (int p = 0; p < 128 / TALK_PAGE; ++p) {
-          const int blk = bt[min(i * (128 / TALK_PAGE) + p, n_pages - 1)];  // (past the end: masked keys)
+#pragma unroll
+        for (int p = 0; p < 128 / TALK_PAGE; ++p)
           for (int hf = 0; hf < DP / 64; ++hf)
             tma_load_3d(sK + (i & 1) * L_::TILE + hf * (128 * 128) + p * (TALK_PAGE * 128), &tmK, bar, hf * 64,
-                        kh * TALK_PAGE, blk);
-        }
+                        kh * TALK_PAGE, blk[p]);
         loads = i + 1;
+        pages(i + 1);
       };
+      pages(0);
       mbar_expect_tx(q_bar, L_::TILE);
       for (int hf = 0; hf < DP / 64; ++hf) tma_load_3d(sQ + hf * (128 * 128), &tmQ, q_bar, hf * 64, head, q0 + qt * 128);
       for (int i = 0; i < 2 && i < n; ++i) load_k(i);
@@ -272,20 +277,23 @@ talking_weights_tc_kernel(const __grid_constant__ CUtensorMap tmQ, const __grid_
         for (int hf = 0; hf < DP / 64; ++hf)
           tma_load_3d(sQ + (c * (DP / 64) + hf) * (N * 128), &tmQ, q_bar, hf * 64, c * R, t0);
       bool ok = true;
-      int n = 0;
-      for (int t = 0; ok && t < live; ++t)
+      int n = 0, blk[128 / TALK_PAGE];
+      for (int t = 0; ok && t < live; ++t) {
+#pragma unroll
+        for (int p = 0; p < 128 / TALK_PAGE; ++p)
+          blk[p] = bt[min((key0 + t * 128) / TALK_PAGE + p, n_pages - 1)];  // (past the end: masked keys)
         for (int c = 0; c < G; ++c, ++n) {
           const int st = n % STAGES;
           if (n >= STAGES) ok = mbar_wait_bounded(&k_free[st], (n / STAGES - 1) & 1, abort_flag, err);
           if (!ok) break;
           mbar_expect_tx(&k_full[st], L_::TILE);
-          for (int p = 0; p < 128 / TALK_PAGE; ++p) {
-            const int blk = bt[min((key0 + t * 128) / TALK_PAGE + p, n_pages - 1)];  // (past the end: masked keys)
+#pragma unroll
+          for (int p = 0; p < 128 / TALK_PAGE; ++p)
             for (int hf = 0; hf < DP / 64; ++hf)
               tma_load_3d(smem + st * L_::TILE + hf * (128 * 128) + p * (TALK_PAGE * 128), &tmK, &k_full[st], hf * 64,
-                          c * TALK_PAGE, blk);
-          }
+                          c * TALK_PAGE, blk[p]);
         }
+      }
       if (!ok) {  // copies in flight still write to this CTA's memory: give them their (bounded) time before leaving
         for (int it = 0; it < (1 << 20) && !mbar_try_wait(q_bar, 0); ++it) {}
         for (int i = max(n - STAGES, 0); i < n; ++i)
@@ -743,27 +751,27 @@ talking_values_kernel(const __grid_constant__ CUtensorMap tmW, const __grid_cons
       bool ok = true;
       int loads = 0;
       for (int i = 0; i < n; ++i) {
+        int blk[128 / TALK_PAGE];
+#pragma unroll
+        for (int p = 0; p < 128 / TALK_PAGE; ++p) blk[p] = bt[min(i * (128 / TALK_PAGE) + p, n_pages - 1)];  // (past the end: zero weights)
         if (i >= 2) ok = mbar_wait_bounded(&freed[i & 1], ((i >> 1) - 1) & 1, abort_flag, err);
         if (!ok) break;
         uint8_t* dst = smem + (i & 1) * L_::STAGE;
         uint64_t* bar = &full[i & 1];
         mbar_expect_tx(bar, L_::STAGE);
         if constexpr (BLOCKED) {
-          for (int part = 0; part < 2; ++part)
-            for (int c = 0; c < 16; ++c)
-              bulk_load(dst + part * L_::W_BYTES + c * 2048,
-                        rd.w + (static_cast<size_t>(part ? row_lo : row_hi) / 8 + c) * rd.pitch * 8 + i * (128 * 8), 2048, bar);
+          tma_load_2d(dst, &tmW, bar, i * 256, row_hi / 8);  // (128 keys x 8 rows as 256 words of 8 bytes, 16 times)
+          tma_load_2d(dst + L_::W_BYTES, &tmW, bar, i * 256, row_lo / 8);
         }
         for (int hf = 0; hf < (BLOCKED ? 0 : 2); ++hf) {
           tma_load_2d(dst + hf * (128 * 128), &tmW, bar, i * 128 + hf * 64, row_hi);
           tma_load_2d(dst + L_::W_BYTES + hf * (128 * 128), &tmW, bar, i * 128 + hf * 64, row_lo);
         }
-        for (int p = 0; p < 128 / TALK_PAGE; ++p) {
-          const int blk = bt[min(i * (128 / TALK_PAGE) + p, n_pages - 1)];  // (past the end: zero weights)
+#pragma unroll
+        for (int p = 0; p < 128 / TALK_PAGE; ++p)
           for (int hf = 0; hf < DVP / 64; ++hf)
             tma_load_3d(dst + 2 * L_::W_BYTES + hf * (128 * 128) + p * (TALK_PAGE * 128), &tmV, bar, hf * 64,
-                        kh * TALK_PAGE, blk);
-        }
+                        kh * TALK_PAGE, blk[p]);
         loads = i + 1;
       }
       if (!ok)  // copies in flight still write to this CTA's memory: give them their (bounded) time before leaving
@@ -913,9 +921,13 @@ static int weights_tc(const TalkArgs& a, int total_tokens, const CUtensorMap& tk
 }
 template <int DVP, bool BLOCKED>
 static int launch_values(const TalkArgs& a, const CUtensorMap& tv, const TalkRound& rd, int units, cudaStream_t st) {
-  CUtensorMap tw = tv;
+  CUtensorMap tw;
   const uint64_t rows = static_cast<uint64_t>(units) * 2 * a.h * 128;
-  if (!BLOCKED && make_tmap_2d(&tw, rd.w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, rd.pitch, rd.pitch, 128, 64, CU_TENSOR_MAP_SWIZZLE_128B))
+  if (BLOCKED) {
+    const uint64_t dims[2] = {static_cast<uint64_t>(rd.pitch) * 2, rows / 8}, str[1] = {static_cast<uint64_t>(rd.pitch) * 16};
+    const uint32_t box[2] = {256, 16};
+    if (make_tmap_nd(&tw, rd.w, CU_TENSOR_MAP_DATA_TYPE_FLOAT64, 2, dims, str, box, CU_TENSOR_MAP_SWIZZLE_NONE)) return -2;
+  } else if (make_tmap_2d(&tw, rd.w, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 2, rows, rd.pitch, rd.pitch, 128, 64, CU_TENSOR_MAP_SWIZZLE_128B))
     return -2;
   auto kern = talking_values_kernel<DVP, BLOCKED>;
   if (KSANA_SMEM_ONCE(kern, TalkValuesSmem<DVP>::TOTAL) != 0) return -4;
