@@ -36,18 +36,20 @@ def test_attention_with_mixed_weights(dtype, kind, H, G, d, dv, dims):
 
 
 @pytest.mark.parametrize("H,G,d,dv", [(1, 1, 8, 8), (3, 1, 24, 128), (64, 4, 16, 16), (33, 11, 40, 72), (24, 8, 72, 64), (7, 7, 128, 64),
-                                      (65, 13, 16, 24), (64, 64, 16, 16), (4, 1, 136, 32)])
+                                      (16, 8, 64, 64), (16, 4, 40, 128), (16, 2, 128, 24), (32, 16, 32, 64), (32, 4, 128, 72),
+                                      (64, 16, 64, 16), (64, 8, 128, 128), (65, 13, 16, 24), (64, 64, 16, 16), (4, 1, 136, 32)])
 def test_attention_sizes(H, G, d, dv):
-    """Groups of 1 to 16 heads, heads of every size, and what only the general kernel takes."""
+    """Groups of 1 to 16 heads, heads of every size, both forms of the weights' kernel, and what only the general kernel takes."""
     M.attention_case(BF16, "cuda", H, G, d, dv, 8, kind="random")
 
 
-def test_weights_written_out_in_several_rounds():
+@pytest.mark.parametrize("hk", [4, 8])
+def test_weights_written_out_in_several_rounds(hk):
     """Prompts whose weights do not fit into one round's budget, blocks of several sequences in a round."""
     from ksanallm_b200.engine.step_input import make_step_input
     from ksanallm_b200.ops import cuda_talking, reference as ref
     g = torch.Generator(device="cuda").manual_seed(3)
-    h, hk, d, dv, lens, news = 64, 4, 32, 16, [4100, 40, 2500], [4100, 40, 1200]
+    h, d, dv, lens, news = 64, 32, 16, [4100, 40, 2500], [4100, 40, 1200]
     cu = [0, 4100, 4140, 5340]
     table = torch.zeros(3, 260, dtype=torch.int32)
     for b, first in enumerate((1, 300, 310)):
