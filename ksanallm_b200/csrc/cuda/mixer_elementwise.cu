@@ -635,6 +635,48 @@ gated_head_norm_kernel(const T* __restrict__ o, const T* __restrict__ g, int ldg
   }
 }
 
+// The same for heads of exactly 8 LANES columns (16-bit): LANES lanes take a head, and every lane two heads at a time.
+template <int LANES>
+__global__ void __launch_bounds__(256)
+gated_head_norm_packed_kernel(const __nv_bfloat16* __restrict__ o, const __nv_bfloat16* __restrict__ g, int ldg,
+                              const float* __restrict__ w, __nv_bfloat16* __restrict__ out, int ldo, long long units, int h,
+                              float eps, int gate, float out_scale) {
+  const int l = threadIdx.x % LANES, c = l * 8;
+  const long long stride = static_cast<long long>(gridDim.x) * (256 / LANES);  // (both heads of a lane are far apart: no matter)
+  const long long u0 = static_cast<long long>(blockIdx.x) * (256 / LANES) + threadIdx.x / LANES;
+  float f[2][8], gg[2][8];
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const long long u = u0 + i * stride;  // (token, head)
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[i][j] = gg[i][j] = 0.f;
+    if (u < units) {
+      load_n<8>(o + u * (8 * LANES) + c, f[i]);
+      load_n<8>(g + (u / h) * ldg + (u % h) * (8 * LANES) + c, gg[i]);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < 2; ++i) {
+    const long long u = u0 + i * stride;
+    float ss = 0.f;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) ss += f[i][j] * f[i][j];
+#pragma unroll
+    for (int x = LANES / 2; x > 0; x >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, x);
+    const float inv = out_scale / sqrtf(ss / static_cast<float>(8 * LANES) + eps);
+    if (u >= units) continue;
+    const int col = static_cast<int>(u % h) * (8 * LANES) + c;
+#pragma unroll
+    for (int j = 0; j < 8; ++j) f[i][j] *= inv * gate_f<__nv_bfloat16>(gg[i][j], gate);
+    if (w) {
+      load_n<8>(w + col, gg[i]);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) f[i][j] *= gg[i][j];
+    }
+    store_n<8>(out + (u / h) * ldo + col, f[i]);
+  }
+}
+
 // over all heads of a token, with a weight: one CTA per token
 template <typename T, int N>
 __global__ void __launch_bounds__(256)
@@ -867,6 +909,17 @@ KSANA_API int ksana_gated_norm(const void* o, const void* g, int ldg, const floa
   const int esz = kind ? 2 : 4;
   const int width = h * dv;
   const bool vec = !((dv | ldg | ldo) & 3) && aligned(o, 4 * esz) && aligned(g, 4 * esz) && aligned(out, 4 * esz);
+  if (kind && (!w || per_head) && (dv == 32 || dv == 64 || dv == 128) && !((ldg | ldo) & 7) && aligned(o, 16) && aligned(g, 16) &&
+      aligned(out, 16) && aligned(w, 16)) {
+    const long long units = static_cast<long long>(tokens) * h;
+#define KSANA_GHP(L)                                                                                                     \
+  gated_head_norm_packed_kernel<L><<<static_cast<unsigned>((units + 2 * (256 / L) - 1) / (2 * (256 / L))), 256, 0, st>>>(  \
+      static_cast<const bf16*>(o), static_cast<const bf16*>(g), ldg, w, static_cast<bf16*>(out), ldo, units, h, eps, gate,  \
+      out_scale)
+    if (dv == 32) KSANA_GHP(4); else if (dv == 64) KSANA_GHP(8); else KSANA_GHP(16);
+#undef KSANA_GHP
+    return done();
+  }
   const bool wide = kind && (!w || per_head) && dv > 128 && !((dv | ldg | ldo) & 7) && aligned(o, 16) && aligned(g, 16) && aligned(out, 16);
   const unsigned grid = static_cast<unsigned>((static_cast<long long>(tokens) * ((h + 3) / 4) + 7) / 8);
 #define KSANA_GN(T, N)                                                                                               \
